@@ -7,6 +7,7 @@ Behavioural contract (same as MaxText's `pyconfig.initialize`, src/maxtext/confi
   packaged ``configs/`` directory); parents are applied first;
 * ``model_name=<x>`` merges ``configs/models/<x>.yml``; those architecture constants beat the YAML
   chain, and a CLI override of one of them is an error unless ``override_model_config=true``;
+* ``model_dir=<folder>`` takes the architecture constants from the folder's config.json instead (`models/registry.py`);
 * ``M_<KEY>`` environment variables override like CLI arguments; setting the same key on the CLI
   and in the environment is an error (pyconfig.py:128);
 * unknown keys are errors;
@@ -292,6 +293,16 @@ def initialize(argv: list[str] | None = None, num_devices: int | None = None, **
               f"{k} is fixed by model_name={model_name}; pass override_model_config=true to change it")
         continue
       table[k] = _coerce(k, v, _defaults.DEFAULTS[k])
+
+  # model folder: its config.json plays the role of the catalog entry
+  if table.get("model_dir"):
+    from ..models import registry
+    for k, v in registry.config_keys(str(table["model_dir"])).items():
+      if k in cli or k in env:
+        if not table.get("override_model_config"):
+          raise ConfigError(f"{k} is fixed by model_dir={table['model_dir']}; pass override_model_config=true to change it")
+        continue
+      table[k] = v
 
   if num_devices is None:
     num_devices = _types.detect_num_devices(table)

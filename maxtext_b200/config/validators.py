@@ -299,7 +299,17 @@ def check_misc(t):
     _fail("dataset_name can't be empty when dataset_type=tfds")
 
 
-ALL_CHECKS = (check_checkpointing, check_attention, check_block_diffusion, check_quantization, check_moe, check_families, check_post_training,
+def check_layer_specs(t):
+  if t.get("decoder_block") != "silinex":
+    return
+  from ..models import silinex
+  try:
+    silinex.validate(t)
+  except (KeyError, TypeError, ValueError) as e:
+    _fail(f"layer_specs: {e!r}" if isinstance(e, KeyError) else str(e))
+
+
+ALL_CHECKS = (check_layer_specs, check_checkpointing, check_attention, check_block_diffusion, check_quantization, check_moe, check_families, check_post_training,
               check_batch_and_vocab, check_parallelism, check_schedules_and_distillation, check_misc)
 
 

@@ -301,6 +301,7 @@ int mt_num_sms() { return num_sms(); }
 void register_attention(pybind11::module_& m);
 void register_moe(pybind11::module_& m);
 void register_comm(pybind11::module_& m);
+void register_serving(pybind11::module_& m);
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_supported", &gemm_supported);
@@ -329,4 +330,5 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   register_attention(m);
   register_moe(m);
   register_comm(m);
+  register_serving(m);
 }

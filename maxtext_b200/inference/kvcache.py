@@ -4,8 +4,9 @@ The reference keeps two caches per layer (prefill and AR) with configurable axis
 attention partials (src/maxtext/inference/kvcache.py:249-1137; attention_op.py:2730). On a GPU one contiguous cache
 per layer is simpler and faster: `[slots, max_len, kv_heads, head_dim]`, written in place at each slot's current
 length; a prefill result is inserted by copying its rows into a slot. Optional int8 / fp8 storage with per
-(token, head) scales mirrors `KVQuant` (kvcache.py:49-150). `MlaKVCache` stores the compressed latent and the
-shared RoPE key (kvcache.py:1204) and expands them with `wkv_b` at attention time.
+(token, head) scales mirrors `KVQuant` (kvcache.py:49-150). `MlaLayerCache` stores the compressed latent and the
+shared RoPE key (kvcache.py:1204); prefill expands them with `wkv_b`, decoding attends in the latent space (`ops/latent.py`).
+Recurrent layers keep a `layers.gdn.RecurrentState` instead of keys and values.
 """
 from __future__ import annotations
 
@@ -52,9 +53,20 @@ class LayerKVCache:
       self.vs = torch.ones(slots, max_len, kv_heads, 1, dtype=torch.float32, device=device)
     self.slot_ids: torch.Tensor | None = None     # which cache rows the current batch maps to
     self.lengths: torch.Tensor | None = None      # tokens already cached per batch row (before this call)
+    self.new_lens: torch.Tensor | None = None     # real tokens per row of a right-padded batch
 
-  def bind(self, slot_ids, lengths):
-    self.slot_ids, self.lengths = slot_ids, lengths
+  def bind(self, slot_ids, lengths, new_lens=None):
+    """`new_lens` [B]: real tokens per row when the batch is right padded; the padding is not written."""
+    self.slot_ids, self.lengths, self.new_lens = slot_ids, lengths, new_lens
+
+  def _places(self, B: int, S: int, device):
+    """(cache rows, positions, selector) of the new tokens that enter the cache."""
+    pos = self.lengths[:, None] + torch.arange(S, device=device)[None]
+    rows = self.slot_ids[:, None].expand(B, S)
+    if self.new_lens is None:
+      return rows, pos, lambda x: x
+    real = torch.arange(S, device=device)[None] < self.new_lens[:, None]
+    return rows[real], pos[real], lambda x: x[real]
 
   def rows_for(self, n: int) -> int:
     """Rows of this rank's part that hold a prompt of n tokens."""
@@ -94,9 +106,9 @@ class LayerKVCache:
     O = torch.stack(outs).float()                                          # [N, B, S, H, D]
     return (O * w.permute(0, 1, 3, 2)[..., None]).sum(0).to(q.dtype)
 
-  def _write(self, buf, sbuf, x, pos):
-    B, S = x.shape[:2]
-    rows = self.slot_ids[:, None].expand(B, S)
+  def _write(self, buf, sbuf, x):
+    rows, pos, pick = self._places(x.shape[0], x.shape[1], x.device)
+    x = pick(x)
     if self.quant:
       q, s = self.quant.quantize(x)
       buf[rows, pos] = q
@@ -126,8 +138,8 @@ class LayerKVCache:
         raise NotImplementedError("a sequence-split cache does not take bidirectional image blocks")
       return self._attend_split(q, k, v, ctx, window, soft_cap, sinks)
     pos = self.lengths[:, None] + torch.arange(S, device=q.device)[None]           # absolute positions of the new tokens
-    self._write(self.k, getattr(self, "ks", None), k, pos)
-    self._write(self.v, getattr(self, "vs", None), v, pos)
+    self._write(self.k, getattr(self, "ks", None), k)
+    self._write(self.v, getattr(self, "vs", None), v)
     if self._decode_kernel_ok(q, S, sinks):
       # one new token per sequence: split-KV decode kernel straight on the cache, lengths stay on the device (no host sync)
       from ..ops import backend
@@ -137,6 +149,8 @@ class LayerKVCache:
                                      out, 1.0, float(soft_cap), int(window), splits)
       return out[:, None]
     upto = int((self.lengths.max() + S).item()) if ctx.mode != "prefill" else int(S + self.lengths.max().item())
+    if self.new_lens is not None:
+      upto = min(upto, self.max_len)                      # padding may run past the end of the cache
     K, V = self._read(self.k, getattr(self, "ks", None), upto), self._read(self.v, getattr(self, "vs", None), upto)
     kv_pos = torch.arange(upto, device=q.device)[None].expand(B, upto)
     valid_len = (self.lengths + S)[:, None]
@@ -162,25 +176,17 @@ class MlaLayerCache(LayerKVCache):
     self.seq_group, self.seq_rank, self.seq_size, self.global_len = None, 0, 1, max_len        # latent caches are not split along the sequence
     self.latent = torch.zeros(slots, max_len, kv_lora_rank, dtype=dtype, device=device)
     self.k_rope = torch.zeros(slots, max_len, rope_dim, dtype=dtype, device=device)
-    self.slot_ids = self.lengths = None
+    self.slot_ids = self.lengths = self.new_lens = None
+
+  def write(self, latent, k_rope):
+    """latent [B, S, R], k_rope [B, S, dr] of the new tokens to the rows after what each sequence holds."""
+    rows, pos, pick = self._places(latent.shape[0], latent.shape[1], latent.device)
+    self.latent[rows, pos] = pick(latent).to(self.dtype)
+    self.k_rope[rows, pos] = pick(k_rope).to(self.dtype)
 
   def attend_mla(self, q, latent, k_rope, mla, ctx):
-    from ..ops import functional as F
-    B, S = q.shape[:2]
-    pos = self.lengths[:, None] + torch.arange(S, device=q.device)[None]
-    rows = self.slot_ids[:, None].expand(B, S)
-    self.latent[rows, pos] = latent.to(self.dtype)
-    self.k_rope[rows, pos] = k_rope.reshape(B, S, -1).to(self.dtype)
-    upto = int((self.lengths.max() + S).item())
-    lat, kr = self.latent[self.slot_ids, :upto], self.k_rope[self.slot_ids, :upto]
-    kv = F.linear(lat, mla.wkv_b).view(B, upto, mla.h, mla.nope + mla.vd)
-    k = torch.cat([kv[..., :mla.nope], kr[:, :, None, :].expand(B, upto, mla.h, mla.rope_d)], dim=-1)
-    v = kv[..., mla.nope:]
-    kv_pos = torch.arange(upto, device=q.device)[None].expand(B, upto)
-    mask = ref.attention_mask(pos, kv_pos) & (kv_pos < (self.lengths + S)[:, None])[:, None, None, :]
-    if ctx.segment_ids is not None and ctx.mode == "prefill" and ctx.segment_ids.shape[1] == upto:
-      mask = mask & (ctx.segment_ids[:, None, :, None] == ctx.segment_ids[:, None, None, :])      # packed prompts (prefill_concat)
-    return ref.attention(q, k, v, mask, 1.0)
+    from ..ops import latent as lat_ops
+    return lat_ops.attend_cached(q, latent, k_rope, mla, self, ctx)
 
 
 def make_caches(model, slots: int, max_len: int, device, quantize: bool = False):
@@ -195,16 +201,14 @@ def make_caches(model, slots: int, max_len: int, device, quantize: bool = False)
   for layer in model.layers:
     per_layer = []
     for blk in layer.blocks:
-      if seq_size > 1 and blk.plan.attention in ("mla", "gdn", "compressed"):
+      if seq_size > 1 and blk.plan.attention in ("mla", "gdn", "gla", "compressed"):
         raise NotImplementedError("context_autoregressive parallelism splits plain key / value caches only")
       if blk.plan.attention == "mla":
-        per_layer.append(MlaLayerCache(slots, max_len, c.kv_lora_rank, c.qk_rope_head_dim, dt, device))
+        per_layer.append(MlaLayerCache(slots, max_len, blk.attn.kv_rank, blk.attn.rope_d, dt, device))
       elif blk.plan.attention == "compressed":
         per_layer.append(blk.attn.make_cache(slots, max_len, dt, device))
-      elif blk.plan.attention == "gdn":
-        from ..layers.gdn import GDNState
-        a = blk.attn
-        per_layer.append(GDNState(slots, a.conv_dim, a.K, a.hv, a.dk, a.dv, device))
+      elif blk.plan.attention in ("gdn", "gla"):
+        per_layer.append(blk.attn.make_state(slots, device))
       else:
         a = blk.attn
         per_layer.append(LayerKVCache(slots, max_len, a.hkv_l, a.dh, a.dh, dt, device, quant, **seq))

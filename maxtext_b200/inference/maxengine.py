@@ -60,10 +60,15 @@ class MaxEngine:
 
   # ------------------------------------------------------------------ params
   def load_params(self, path: str | None = None, seed: int | None = None):
-    """Params-only checkpoint (`load_parameters_path`) or random init when no path is configured."""
+    """Params-only checkpoint (`load_parameters_path`), the weights of a model folder (`model_dir`), or random init when neither is
+    configured."""
     from ..checkpoint import manager as ckpt
     path = path or self.config.load_parameters_path
-    if path:
+    model_dir = str(getattr(self.config, "model_dir", "") or "")
+    if model_dir and not path:
+      from ..models import registry
+      registry.load_weights(model_dir, self.model.store, self.config)
+    elif path:
       ckpt.load_params_only(path, _EngineView(self), self.model.mesh)
     else:
       self.model.store.initialize(seed=self.config.init_weights_seed if seed is None else seed)
@@ -139,10 +144,45 @@ class MaxEngine:
                        torch.zeros(slots, dtype=torch.long, device=dev),
                        torch.zeros(slots, device=dev) if c.return_log_prob else None)
 
-  def _bind(self, caches, slot_ids, lengths):
+  def _bind(self, caches, slot_ids, lengths, new_lens=None):
     for per_layer in caches:
       for cch in per_layer:
-        cch.bind(slot_ids, lengths)
+        cch.bind(slot_ids, lengths, new_lens)
+
+  @staticmethod
+  def _recurrent_buffers(caches) -> list:
+    """Fixed-size state tensors, which every step rewrites (key / value rows are only appended)."""
+    return [getattr(cch, n) for per_layer in caches for cch in per_layer for n in getattr(cch, "recurrent_buffers", ())]
+
+  @torch.no_grad()
+  def extend(self, state: DecodeState, slots: list[int], tokens: list, want: list | None = None):
+    """Feed every slot of `slots` its next tokens, as one right-padded batch, and return the logits [n, V] at the wanted places.
+
+    `tokens[i]` continues what slot `slots[i]` holds (nothing, for a slot that is new or was freed); `want[i]` lists places among
+    tokens[i] (None: the last place of every row). Nothing is sampled: this is the teacher-forced form of prefill (rows that start at
+    their first token) and of generate (rows that go on by one token)."""
+    dev = self.device
+    lens = [len(t) for t in tokens]
+    if not slots or min(lens) < 1 or len(set(slots)) != len(slots):
+      raise ValueError("extend: needs at least one token for each of a set of distinct slots")
+    starts = state.next_pos[torch.tensor(slots, device=dev)].tolist()
+    for s, a, n in zip(slots, starts, lens):
+      if not 0 <= s < int(state.tokens.shape[0]) or a + n > self.max_len:
+        raise ValueError(f"extend: slot {s} cannot take {n} more tokens (holds {a} of {self.max_len})")
+    S = max(lens)
+    padded = torch.zeros(len(slots), S, dtype=torch.long)
+    for i, t in enumerate(tokens):
+      padded[i, :lens[i]] = torch.as_tensor(t, dtype=torch.long)
+    want = [[n - 1] for n in lens] if want is None else want
+    rows = torch.tensor([i * S + p for i, w in enumerate(want) for p in w], dtype=torch.long)
+    ids, begin, n_new = (torch.tensor(v, dtype=torch.long, device=dev) for v in (slots, starts, lens))
+    self._bind(state.caches, ids, begin, n_new if min(lens) != S else None)
+    pos = begin[:, None] + torch.arange(S, device=dev)[None]
+    mode = "prefill" if max(starts) == 0 else "decode"
+    logits = self.model.forward(padded.to(dev), pos, None, mode=mode, caches=state.caches, new_lens=n_new if min(lens) != S else None,
+                                logit_rows=rows.to(dev))
+    state.next_pos[ids] = begin + n_new
+    return logits
 
   def _check_length(self, n: int, what: str):
     """A prompt must leave room for at least one generated token: a prefix of max_target_length tokens would make the next
@@ -176,7 +216,8 @@ class MaxEngine:
       mm_kw = dict(images=images[None].to(dev), image_mask=image_mask[:true_length][None].to(dev))
     if audio is not None:
       mm_kw.update(audio=audio[None].to(dev), audio_mask=audio_mask[:true_length][None].to(dev))
-    logits = self.model.forward(toks, pos, None, mode="prefill", caches=caches, **mm_kw)[:, -1]
+    last = torch.full((1,), true_length - 1, dtype=torch.long, device=dev)
+    logits = self.model.forward(toks, pos, None, mode="prefill", caches=caches, logit_rows=last, **mm_kw)
     tok = self._sample(logits)
     lp = inference_utils.log_prob_of(logits, tok) if self.config.return_log_prob else None
     res = ResultTokens(torch.tensor([[int(tok), 1, 1]], device=dev), lp)
@@ -198,15 +239,19 @@ class MaxEngine:
   def prefill_concat(self, prompts: list[torch.Tensor]) -> list[Prefix]:
     """Several short prompts in one prefill pass (maxengine.py:1180 `prefill_concat`): the prompts are packed into one row
     with segment ids and per-prompt positions, and the cached keys / values of each segment become that prompt's prefix.
-    Layers with a recurrent state (gated delta networks) cannot be packed this way; such models prefill one by one."""
+    A recurrent state would run on from one prompt into the next, so models with recurrent layers run the prompts as the rows of one
+    right-padded batch instead."""
     dev = self.device
     lens = [int(p.numel()) for p in prompts]
     for n in lens:
       self._check_length(n, "prefill_concat")
     total = sum(lens)
-    packable = total <= self.max_len and not any(b.plan.attention in ("gdn", "compressed") for l in self.model.layers for b in l.blocks)
-    if not packable or len(prompts) == 1:
+    kinds = {b.plan.attention for l in self.model.layers for b in l.blocks}
+    packable = total <= self.max_len and not kinds & {"gdn", "gla", "compressed"}
+    if len(prompts) == 1 or "compressed" in kinds:
       return [self.prefill(p, n)[0] for p, n in zip(prompts, lens)]
+    if not packable:
+      return self._prefill_padded(prompts, lens)
     toks = torch.cat([p.to(dev).long() for p in prompts])[None]
     seg = torch.cat([torch.full((n,), i + 1, dtype=torch.int32, device=dev) for i, n in enumerate(lens)])[None]
     pos = torch.cat([torch.arange(n, device=dev) for n in lens])[None]
@@ -226,6 +271,18 @@ class MaxEngine:
       tok = self._sample(lg)
       out.append(Prefix(caches, n, tok, lg, inference_utils.log_prob_of(lg, tok) if self.config.return_log_prob else None))
       start += n
+    return out
+
+  def _prefill_padded(self, prompts, lens) -> list[Prefix]:
+    """One pass over a right-padded batch; prefix i is row i of the shared caches."""
+    state = self.init_decode_state(len(prompts))
+    logits = self.extend(state, list(range(len(prompts))), [p.tolist() for p in prompts])
+    out = []
+    for i, n in enumerate(lens):
+      caches = [[_CacheRow(cch, i) for cch in per_layer] for per_layer in state.caches]
+      lg = logits[i][None]
+      tok = self._sample(lg)
+      out.append(Prefix(caches, n, tok, lg, inference_utils.log_prob_of(lg, tok) if self.config.return_log_prob else None))
     return out
 
   @torch.no_grad()
@@ -249,7 +306,9 @@ class MaxEngine:
         e = min(n, s + chunk)
         self._bind(caches, slot, torch.full((1,), s, dtype=torch.long, device=dev))
         pos = torch.arange(s, e, device=dev)[None]
-        logits = self.model.forward(tokens[s:e].to(dev).long()[None], pos, None, mode="decode", caches=caches)[:, -1]
+        last = torch.full((1,), e - s - 1, dtype=torch.long, device=dev)
+        logits = self.model.forward(tokens[s:e].to(dev).long()[None], pos, None, mode="prefill" if s == 0 else "decode", caches=caches,
+                                    logit_rows=last)
     tok = self._sample(logits)
     return Prefix(caches, n, tok, logits), ResultTokens(torch.tensor([[int(tok), 1, 1]], device=dev))
 
@@ -265,9 +324,8 @@ class MaxEngine:
         for name in ("k", "v", "ks", "vs", "latent", "k_rope") + tuple(getattr(s, "token_buffers", ())):
           if hasattr(s, name) and hasattr(d, name):
             getattr(d, name)[slot, :m] = getattr(s, name)[0, :m]
-        for name in ("conv", "rec"):                 # fixed-size recurrent state (gated delta layers)
-          if hasattr(s, name) and hasattr(d, name):
-            getattr(d, name)[slot] = getattr(s, name)[0]
+        for name in getattr(s, "recurrent_buffers", ()):        # fixed-size recurrent state
+          getattr(d, name)[slot] = getattr(s, name)[0]
     state.tokens[slot] = prefix.first_token.reshape(-1)[0]
     state.next_pos[slot] = n
     state.active[slot] = True
@@ -310,21 +368,22 @@ class MaxEngine:
     entry = self._graphs.get(key)
     if entry is None:
       try:
-        keep = [t.clone() for t in (state.tokens, state.next_pos, state.active, state.generated)]
+        live = (state.tokens, state.next_pos, state.active, state.generated, *self._recurrent_buffers(state.caches))
+        keep = [t.clone() for t in live]
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):                       # warm-up: lazy initialisation must happen outside the capture
           for _ in range(2):
             self._step_inplace(state)
         torch.cuda.current_stream().wait_stream(side)
-        for t, k in zip((state.tokens, state.next_pos, state.active, state.generated), keep):
-          t.copy_(k)                                        # the warm-up steps wrote only beyond the cached lengths
+        for t, k in zip(live, keep):
+          t.copy_(k)                                        # key / value rows: the warm-up steps wrote only beyond the cached lengths
         g = torch.cuda.CUDAGraph()
         if hasattr(g, "register_generator_state"):
           g.register_generator_state(self.generator)
         with torch.cuda.graph(g):
           data = self._step_inplace(state)
-        for t, k in zip((state.tokens, state.next_pos, state.active, state.generated), keep):
+        for t, k in zip(live, keep):
           t.copy_(k)                                        # capture does not execute, but keep the contract explicit
         entry = (g, data)
       except Exception as e:  # pylint: disable=broad-except
@@ -359,6 +418,17 @@ class MaxEngine:
     state.active[slot] = False
     state.next_pos[slot] = 0
     state.generated[slot] = 0
+
+
+class _CacheRow:
+  """One slot of a cache, seen as a single-row cache (what `insert` copies from)."""
+
+  def __init__(self, cache, row: int):
+    self._cache, self._row = cache, row
+
+  def __getattr__(self, name):
+    v = getattr(self._cache, name)
+    return v[self._row:self._row + 1] if isinstance(v, torch.Tensor) and v.dim() >= 2 else v
 
 
 class _EngineView:

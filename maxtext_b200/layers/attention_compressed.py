@@ -344,5 +344,7 @@ class CompressedLayerCache:
     self.token_buffers = tuple(names)
     self.slot_ids = self.lengths = None
 
-  def bind(self, slot_ids, lengths):
+  def bind(self, slot_ids, lengths, new_lens=None):
+    if new_lens is not None:
+      raise NotImplementedError("compressed attention does not take right-padded batches of unequal rows")
     self.slot_ids, self.lengths = slot_ids, lengths

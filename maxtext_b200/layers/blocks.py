@@ -9,6 +9,7 @@ wi_0|wi_1 are adjacent in the unit's flat buffer and are consumed as single fuse
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 
 import torch
 import torch.distributed as dist
@@ -462,6 +463,19 @@ class Attention:
 
 
 # ------------------------------------------------------------------------------------------ MLA
+@dataclass(frozen=True)
+class LatentSizes:
+  """Sizes of one latent-attention layer; `scale` multiplies the scores, `window` limits the keys (0: all)."""
+  heads: int
+  nope: int
+  rope: int
+  vd: int
+  q_rank: int
+  kv_rank: int
+  scale: float
+  window: int = 0
+
+
 class MLA:
   """DeepSeek multi-head latent attention (src/maxtext/layers/attention_mla.py:785-1115).
 
@@ -469,43 +483,59 @@ class MLA:
   kv_norm on the latent; wkv_b -> per head [k_nope | v]; the single RoPE'd k_rope head is broadcast to
   all heads. Softmax scale (incl. YaRN mscale) multiplies the query at runtime."""
 
-  def __init__(self, b: Builder, config, rope_inv_ts, interleaved, name="self_attention"):
+  def __init__(self, b: Builder, config, rope_inv_ts, interleaved, name="self_attention", sizes: LatentSizes | None = None):
     c = config
     self.c = c
-    self.h = c.num_query_heads // b.tp_size
-    self.nope, self.rope_d, self.vd = c.qk_nope_head_dim, c.qk_rope_head_dim, c.v_head_dim
+    if sizes is None:
+      scale = (c.qk_nope_head_dim + c.qk_rope_head_dim) ** -0.5
+      if c.max_position_embeddings > c.original_max_position_embeddings and c.rope_type == "yarn":
+        m = 0.1 * c.mscale * math.log(c.rope_factor) + 1.0
+        scale = scale * m * m
+      sizes = LatentSizes(c.num_query_heads, c.qk_nope_head_dim, c.qk_rope_head_dim, c.v_head_dim, c.q_lora_rank, c.kv_lora_rank, scale)
+    self.heads, self.h = sizes.heads, sizes.heads // b.tp_size
+    self.nope, self.rope_d, self.vd = sizes.nope, sizes.rope, sizes.vd
+    self.q_rank, self.kv_rank, self.softmax_scale, self.window = sizes.q_rank, sizes.kv_rank, sizes.scale, sizes.window
     self.qk = self.nope + self.rope_d
     self.inv_ts, self.interleaved = rope_inv_ts, interleaved
     ab = b.sub(name)
     d = c.emb_dim
-    if c.q_lora_rank > 0:
-      self.wq_a = ab.sub("wq_a").linear("kernel", (d,), (c.q_lora_rank,), ("embed", "q_lora"))
-      self.q_norm = Norm(ab, "q_norm", c.q_lora_rank, c.normalization_layer_epsilon)
-      self.wq_b = ab.sub("wq_b").linear("kernel", (c.q_lora_rank,), (c.num_query_heads, self.qk),
-                                        ("q_lora", "q_heads", "kv"), tp="col")
+    if self.q_rank > 0:
+      self.wq_a = ab.sub("wq_a").linear("kernel", (d,), (self.q_rank,), ("embed", "q_lora"))
+      self.q_norm = Norm(ab, "q_norm", self.q_rank, c.normalization_layer_epsilon)
+      self.wq_b = ab.sub("wq_b").linear("kernel", (self.q_rank,), (self.heads, self.qk), ("q_lora", "q_heads", "kv"), tp="col")
       self.query = None
     else:
-      self.query = ab.sub("query").linear("kernel", (d,), (c.num_query_heads, self.qk), ("embed", "q_heads", "kv"), tp="col")
-    self.wkv_a = ab.sub("wkv_a").linear("kernel", (d,), (c.kv_lora_rank + self.rope_d,), ("embed", "kv_lora"))
-    self.kv_norm = Norm(ab, "kv_norm", c.kv_lora_rank, c.normalization_layer_epsilon)
-    self.wkv_b = ab.sub("wkv_b").linear("kernel", (c.kv_lora_rank,), (c.num_query_heads, self.nope + self.vd),
+      self.query = ab.sub("query").linear("kernel", (d,), (self.heads, self.qk), ("embed", "q_heads", "kv"), tp="col")
+    self.wkv_a = ab.sub("wkv_a").linear("kernel", (d,), (self.kv_rank + self.rope_d,), ("embed", "kv_lora"))
+    self.kv_norm = Norm(ab, "kv_norm", self.kv_rank, c.normalization_layer_epsilon)
+    self.wkv_b = ab.sub("wkv_b").linear("kernel", (self.kv_rank,), (self.heads, self.nope + self.vd),
                                         ("kv_lora", "kv_heads", "kv_head_dim"), tp="col")
-    self.o = ab.sub("out").linear("kernel", (c.num_query_heads, self.vd), (d,), ("heads", "kv", "embed"), tp="row")
+    self.o = ab.sub("out").linear("kernel", (self.heads, self.vd), (d,), ("heads", "kv", "embed"), tp="row")
     self.indexer = None
     if bool(getattr(c, "use_indexer", False)):
       # src/maxtext/layers/attention_mla.py:735-750: DeepSeek-V3.2 sparse attention; shares the rotary table, not the layout
       from .indexer import Indexer
       assert b.tp_size == 1, "use_indexer is not split over the tensor axis"
       self.indexer = Indexer(ab, c, rope_inv_ts)
-    scale = self.qk ** -0.5
-    if c.max_position_embeddings > c.original_max_position_embeddings and c.rope_type == "yarn":
-      m = 0.1 * c.mscale * math.log(c.rope_factor) + 1.0
-      scale = scale * m * m
-    self.softmax_scale = scale
+
+  def _serve(self, x, ctx):
+    """Inference: the latent and the rotated key part go to the cache, which attends (`kvcache.MlaLayerCache`)."""
+    from ..ops import latent
+    B, S, _ = x.shape
+    kva = F.linear(x, self.wkv_a)
+    if self.query is not None:
+      q, lat, kr = F.linear(x, self.query), *latent.prep(None, kva, self, ctx)[1:]
+    else:
+      cq, lat, kr = latent.prep(F.linear(x, self.wq_a), kva, self, ctx)
+      q = F.linear(cq, self.wq_b)
+    out = ctx.cache.attend_mla(q.view(B, S, self.h, self.qk), lat, kr, self, ctx)
+    return tp_exit(F.linear(out.reshape(B, S, -1), self.o), ctx)
 
   def __call__(self, x, ctx):
     c = self.c
     x = tp_enter(x, ctx)
+    if ctx.cache is not None:
+      return self._serve(x, ctx)
     B, S, _ = x.shape
     low_rank_q = None
     if self.query is not None:
@@ -518,27 +548,24 @@ class MLA:
     q_rope = F.rope(q_rope, ctx.positions, self.inv_ts, self.interleaved)
     q = torch.cat([q_nope, q_rope], dim=-1) * self.softmax_scale
     kva = F.linear(x, self.wkv_a)
-    latent, k_rope = kva[..., :c.kv_lora_rank], kva[..., c.kv_lora_rank:]
+    latent, k_rope = kva[..., :self.kv_rank], kva[..., self.kv_rank:]
     k_rope = F.rope(k_rope.reshape(B, S, 1, self.rope_d), ctx.positions, self.inv_ts, self.interleaved)
     latent = self.kv_norm(latent.contiguous())
-    if ctx.cache is not None:
-      out = ctx.cache.attend_mla(q, latent, k_rope, self, ctx)
+    kv = F.linear(latent, self.wkv_b).view(B, S, self.h, self.nope + self.vd)
+    k = torch.cat([kv[..., :self.nope], k_rope.expand(B, S, self.h, self.rope_d)], dim=-1)
+    v = kv[..., self.nope:]
+    if c.use_qk_clip and ctx.mode == "train" and not ctx.recompute and ctx.max_logits is not None:
+      ctx.max_logits[(ctx.layer_index, self)] = _max_logit_per_head(q, k, ctx.positions, ctx.segment_ids)
+    sparse = None
+    if self.indexer is not None:
+      sparse, score, allowed = self.indexer(x, low_rank_q, ctx.positions, ctx.segment_ids)
+      if sparse is not None and ctx.mode == "train" and float(c.indexer_loss_scaling_factor) > 0:
+        ctx.aux_losses.append(("indexer_loss", self.indexer.loss(score, q, k, allowed, sparse)))
+    if sparse is not None:
+      # a per-query key set is not a mask form of the flash kernels: this path is the fp32 definition with an explicit mask
+      out = ref.attention(q, k, v, sparse, 1.0)
     else:
-      kv = F.linear(latent, self.wkv_b).view(B, S, self.h, self.nope + self.vd)
-      k = torch.cat([kv[..., :self.nope], k_rope.expand(B, S, self.h, self.rope_d)], dim=-1)
-      v = kv[..., self.nope:]
-      if c.use_qk_clip and ctx.mode == "train" and not ctx.recompute and ctx.max_logits is not None:
-        ctx.max_logits[(ctx.layer_index, self)] = _max_logit_per_head(q, k, ctx.positions, ctx.segment_ids)
-      sparse = None
-      if self.indexer is not None:
-        sparse, score, allowed = self.indexer(x, low_rank_q, ctx.positions, ctx.segment_ids)
-        if sparse is not None and ctx.mode == "train" and float(c.indexer_loss_scaling_factor) > 0:
-          ctx.aux_losses.append(("indexer_loss", self.indexer.loss(score, q, k, allowed, sparse)))
-      if sparse is not None:
-        # a per-query key set is not a mask form of the flash kernels: this path is the fp32 definition with an explicit mask
-        out = ref.attention(q, k, v, sparse, 1.0)
-      else:
-        out = F.attention(q, k.contiguous(), v.contiguous(), ctx.positions, ctx.segment_ids, 1.0, 0.0, 0)
+      out = F.attention(q, k.contiguous(), v.contiguous(), ctx.positions, ctx.segment_ids, 1.0, 0.0, self.window)
     y = F.linear(out.reshape(B, S, -1), self.o)
     return tp_exit(y, ctx)
 
@@ -594,7 +621,7 @@ class MLP:
       h = F.gated_act(gu, self.acts[0])
     else:
       h = F.linear(x, self.wi_0, bias=self.bi)
-      h = ref.act_fn(self.acts[0])(h.float()).to(x.dtype) if self.acts[0] != "linear" else h
+      h = F.act(h, self.acts[0])
     if tp_rt is not None and ctx.reuse("mlpwo") is None and self.bo is None and self.wo.lora is None:
       y = F.linear(h, self.wo, tp_reduce=tp_rt)
     else:

@@ -72,6 +72,9 @@ class LayerCtx:
   bidir: torch.Tensor | None = None  # [B, 1, S, S] extra allowed (query, key) pairs: tokens of one image see each other
   positions3: torch.Tensor | None = None  # [B, S, 3] (temporal, height, width) positions of a multimodal prompt (`use_mrope`)
   deepstack: tuple | None = None     # (image mask [B, S], [features [B, N*K, D], ...]): feature i is added after decoder layer i
+  new_lens: torch.Tensor | None = None  # [B] real tokens per row of a right-padded inference batch (None: all of them)
+  next_norm: object = None           # fp32 residual streams: the norm that reads the stream after the current layer ...
+  normed: torch.Tensor | None = None  # ... and its output, handed from the layer that computed it to the one that reads it
   name_prefix: str = ""              # disambiguates blocks that share a layer (gemma2 local/global)
   batch_split: int = 1               # > 1: every decoder layer runs the batch as that many micro-batches on alternating streams
   micro_slot: int = 0                # which micro-batch of a split layer this context describes

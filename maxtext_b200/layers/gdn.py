@@ -10,14 +10,17 @@ with q, k L2-normalised, q scaled by Dk^-1/2, and q | k | v first passed through
 SiLU. Training and prefill evaluate the recurrence chunk by chunk so that almost all of the work is matrix products:
 inside a chunk of C tokens the dependence of the written values on each other is a unit lower triangular system
 (solved once per chunk), and only the [Dk, Dv] state crosses chunk borders. Decode applies the three lines above to
-the cached state.
+the cached state. Inference on a GPU runs the kernels behind `ops.recurrent`; training and CPU evaluate the forms below.
 """
 from __future__ import annotations
+
+from dataclasses import dataclass
 
 import torch
 import torch.nn.functional as tF
 
 from ..ops import functional as F
+from ..ops import recurrent
 from .blocks import Builder
 
 
@@ -87,17 +90,46 @@ def gated_delta_chunked(q, k, v, g, beta, chunk: int = 64, state=None):
   return o.transpose(1, 2), S
 
 
-class GDNState:
-  """Decode-time state of one gated-delta layer for `slots` sequences: the last K-1 convolution inputs and S."""
+class RecurrentState:
+  """Inference state of one recurrent layer for `slots` sequences: the matrix state S per head in fp32 and, where the layer has a
+  short convolution, its last taps - 1 inputs. A sequence of length 0 reads zeros whatever its slot holds, so a slot needs no
+  clearing between requests."""
 
-  def __init__(self, slots, conv_dim, kernel, heads, dk, dv, device):
-    self.conv = torch.zeros(slots, kernel - 1, conv_dim, dtype=torch.float32, device=device)
+  recurrent_buffers = ("conv", "rec")
+
+  def __init__(self, slots, heads, dk, dv, device, conv_dim: int = 0, taps: int = 1):
+    self.conv = torch.zeros(slots, taps - 1, conv_dim, dtype=torch.float32, device=device)
     self.rec = torch.zeros(slots, heads, dk, dv, dtype=torch.float32, device=device)
-    self.slot_ids = None
-    self.lengths = None
+    self.slot_ids = self.lengths = self.new_lens = None
 
-  def bind(self, slot_ids, lengths):
-    self.slot_ids, self.lengths = slot_ids, lengths
+  def bind(self, slot_ids, lengths, new_lens=None):
+    self.slot_ids, self.lengths, self.new_lens = slot_ids, lengths, new_lens
+
+  def fresh(self, B: int) -> "RecurrentState":
+    """Bind to rows 0 .. B-1 with nothing cached (a forward pass without a cache)."""
+    z = torch.zeros(B, dtype=torch.long, device=self.rec.device)
+    self.bind(torch.arange(B, device=self.rec.device), z)
+    return self
+
+  def read(self, name: str) -> torch.Tensor:
+    buf = getattr(self, name)[self.slot_ids]
+    return buf * (self.lengths > 0).to(buf.dtype).view(-1, *([1] * (buf.dim() - 1)))
+
+  def real(self, S: int) -> torch.Tensor:
+    """[B, S] True at the tokens that are not right padding."""
+    n = self.new_lens if self.new_lens is not None else torch.full_like(self.lengths, S)
+    return torch.arange(S, device=n.device)[None] < n[:, None]
+
+
+@dataclass(frozen=True)
+class DeltaSizes:
+  """Key heads, value heads, key / value width per head, convolution taps, chunk length of the chunked form."""
+  hk: int
+  hv: int
+  dk: int
+  dv: int
+  taps: int
+  chunk: int = 64
 
 
 class GatedDeltaNet:
@@ -106,15 +138,15 @@ class GatedDeltaNet:
   `in_proj_qkvz` packs, per key head, [q (Dk) | k (Dk) | v (r Dv) | z (r Dv)] with r value heads per key head, and
   `in_proj_ba` packs per key head [b (r) | a (r)]."""
 
-  def __init__(self, b: Builder, config, name="attention"):
+  def __init__(self, b: Builder, config, name="attention", sizes: DeltaSizes | None = None):
     c = config
     assert b.tp_size == 1, "the gated delta network is not split over the tensor axis"
     self.c = c
-    self.hk, self.hv = int(c.gdn_num_key_heads), int(c.gdn_num_value_heads)
-    self.dk, self.dv = int(c.gdn_key_head_dim), int(c.gdn_value_head_dim)
+    if sizes is None:
+      sizes = DeltaSizes(int(c.gdn_num_key_heads), int(c.gdn_num_value_heads), int(c.gdn_key_head_dim), int(c.gdn_value_head_dim),
+                         int(c.gdn_conv_kernel_dim), int(c.gdn_chunk_size))
+    self.hk, self.hv, self.dk, self.dv, self.K, self.chunk = sizes.hk, sizes.hv, sizes.dk, sizes.dv, sizes.taps, sizes.chunk
     self.r = self.hv // self.hk
-    self.K = int(c.gdn_conv_kernel_dim)
-    self.chunk = int(c.gdn_chunk_size)
     self.key_dim, self.value_dim = self.hk * self.dk, self.hv * self.dv
     self.conv_dim = 2 * self.key_dim + self.value_dim
     d = c.emb_dim
@@ -128,33 +160,46 @@ class GatedDeltaNet:
     self.norm = ab.sub("norm", "rms_norm").vector("scale", self.dv, ("norm",))
     self.out = ab.sub("out_proj").linear("kernel", (self.value_dim,), (d,), ("gdn_head", "embed"))
 
+  def make_state(self, slots: int, device) -> RecurrentState:
+    return RecurrentState(slots, self.hv, self.dk, self.dv, device, self.conv_dim, self.K)
+
   def __call__(self, x, ctx):
     B, S, _ = x.shape
     hk, r, dk, dv = self.hk, self.r, self.dk, self.dv
-    qkvz = F.linear(x, self.in_qkvz).view(B, S, hk, 2 * dk + 2 * r * dv)
-    ba = F.linear(x, self.in_ba).view(B, S, hk, 2 * r)
+    qkvz, ba = F.linear(x, self.in_qkvz), F.linear(x, self.in_ba)
+    st = ctx.cache if isinstance(ctx.cache, RecurrentState) else None
+    if recurrent.kernels_ok(qkvz):
+      y = recurrent.delta_forward(self, qkvz, ba, st if st is not None else self.make_state(B, x.device).fresh(B))
+      return F.linear(y, self.out)
+    qkvz, ba = qkvz.view(B, S, hk, 2 * dk + 2 * r * dv), ba.view(B, S, hk, 2 * r)
     q, k, v, z = torch.split(qkvz, [dk, dk, r * dv, r * dv], dim=-1)
     bb, aa = ba[..., :r].reshape(B, S, self.hv), ba[..., r:].reshape(B, S, self.hv)
     z = z.reshape(B, S, self.hv, dv)
     mixed = torch.cat([q.reshape(B, S, -1), k.reshape(B, S, -1), v.reshape(B, S, -1)], dim=-1).float()   # [B,S,conv_dim]
-    st = ctx.cache if isinstance(ctx.cache, GDNState) else None
     if st is not None:
-      hist = st.conv[st.slot_ids]                                                                      # [B,K-1,conv_dim]
+      hist = st.read("conv")                                                                           # [B,K-1,conv_dim]
     else:
       hist = torch.zeros(B, self.K - 1, self.conv_dim, dtype=torch.float32, device=x.device)
     seq = torch.cat([hist, mixed], dim=1)
     wconv = self.conv.leaf().float().view(self.K, self.conv_dim)
     conv = sum(seq[:, j:j + S] * wconv[j] for j in range(self.K))
     conv = tF.silu(conv)
-    if st is not None:
-      st.conv[st.slot_ids] = seq[:, -(self.K - 1):]
+    if st is not None and self.K > 1:
+      # the inputs before each row's first missing token: rows n .. n + K - 2 of [history | new tokens]
+      last = st.real(S).sum(1)[:, None] + torch.arange(self.K - 1, device=x.device)[None]
+      st.conv[st.slot_ids] = seq.gather(1, last[..., None].expand(-1, -1, self.conv_dim))
     q, k, v = torch.split(conv, [self.key_dim, self.key_dim, self.value_dim], dim=-1)
     q, k, v = q.view(B, S, hk, dk), k.view(B, S, hk, dk), v.view(B, S, self.hv, dv)
     if r > 1:
       q, k = q.repeat_interleave(r, dim=2), k.repeat_interleave(r, dim=2)
     beta = torch.sigmoid(bb.float())
     g = -torch.exp(self.A_log.leaf().float()) * tF.softplus(aa.float() + self.dt_bias.leaf().float())
-    s0 = st.rec[st.slot_ids] if st is not None else None
+    s0 = None
+    if st is not None:
+      s0 = st.read("rec")
+      if st.new_lens is not None:                # padding neither decays nor writes
+        keep = st.real(S)[..., None].to(g.dtype)
+        g, beta = g * keep, beta * keep
     if S == 1:
       o, s1 = gated_delta_recurrent(q, k, v, g, beta, s0)
     else:
@@ -162,7 +207,5 @@ class GatedDeltaNet:
     if st is not None:
       st.rec[st.slot_ids] = s1
     # RMS norm over the value head dim, learned scale, then the SiLU gate
-    eps = self.c.normalization_layer_epsilon
-    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * self.norm.leaf().float()
-    o = (o * tF.silu(z.float())).to(x.dtype)
+    o = recurrent.gated_head_norm(o, z, self.norm.leaf(), self.c.normalization_layer_epsilon).to(x.dtype)
     return F.linear(o.reshape(B, S, self.value_dim), self.out)

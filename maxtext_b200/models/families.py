@@ -18,6 +18,7 @@ class Family:
   norm_kind: str = "rms"
   norm_offset: float = 0.0
   scale_embedding: bool = False
+  residual_fp32: bool = False              # the residual stream and the logits are fp32 whatever the compute dtype
 
 
 def describe(c) -> Family:
@@ -29,6 +30,8 @@ def describe(c) -> Family:
     return Family(norm_kind="layernorm")
   if blk in ("qwen3_next", "qwen3_5"):
     return Family(norm_offset=1.0)           # every RMS scale is stored zero-centred and applied as (1 + scale)
+  if blk == "silinex":
+    return Family(norm_offset=1.0, residual_fp32=True)
   return Family()
 
 
@@ -164,6 +167,9 @@ def layer_plans(c) -> list[LayerPlan]:
     for i in range(nh, n, 2):
       plans.append(LayerPlan("scanned_blocks", [v4(ratios[i], "layers_0"), v4(ratios[i + 1], "layers_1")]))
     return plans
+  if blk == "silinex":
+    from .silinex import layer_plans as silinex_plans
+    return silinex_plans(c)
   if blk == "gemma":
     bp = BlockPlan(pre_attn_norm="pre_self_attention_norm", pre_mlp_norm="pre_ffw_norm", soft_cap=c.attn_logits_soft_cap)
     return [LayerPlan("layers", [bp]) for _ in range(n)]
@@ -221,4 +227,4 @@ def layer_plans(c) -> list[LayerPlan]:
     return plans
   raise NotImplementedError(
       f"decoder_block={blk!r} parses but has no model implementation here yet (implemented: llama2, mistral, mixtral, "
-      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, simple)")
+      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, silinex, simple)")

@@ -34,7 +34,8 @@ class BlockPlan:
   post_mlp_norm: str | None = None
   attn_name: str = "self_attention"
   mlp_name: str = "mlp"
-  attention: str = "gqa"                 # gqa | mla | gdn (gated delta network, qwen3-next)
+  attention: str = "gqa"                 # gqa | mla | gdn (gated delta network, qwen3-next) | gla | compressed
+  mixer: dict | None = None              # sizes of this block's mixer, for families whose layers differ (None: the config's)
   gated_attn: bool = False               # qwen3-next full attention: sigmoid output gate from a widened query projection
   window: int = 0
   rope: str = "default"                  # key into Transformer.rope_tables
@@ -44,7 +45,7 @@ class BlockPlan:
   query_scalar: float | None = None
   soft_cap: float = 0.0
   sinks: bool = False
-  mlp: str = "dense"                     # dense | moe | moe_shared
+  mlp: str = "dense"                     # dense | moe | moe_shared | none (the block is its mixer alone)
   mlp_hidden: int | None = None
   mlp_bias: bool = False
   norm_kind: str = "rms"
@@ -62,6 +63,8 @@ class BlockPlan:
   share_kv: bool = False                 # value = key projection
   v_norm: str = ""                       # "" | "noscale" | "scale": RMS normalisation of the value heads
   layer_scalar: bool = False             # learned scalar on the layer output
+  residual_mult: float = 1.0             # factor on each branch before it joins the residual stream
+  residual_fp32: bool = False            # fp32 residual stream with sandwich norms, fused with the residual add (`F.residual_norm`)
   compress_ratio: int = 0                # DeepSeek-V4 compressed attention: 0 (window only), 4 (sparse) or 128 (heavy)
 
 
@@ -90,10 +93,22 @@ class DecoderBlock:
     inv_ts, interleaved = rope_tables[plan.rope]
     rot = int(c.head_dim * c.partial_rotary_factor) if 0 < c.partial_rotary_factor < 1.0 else None
     if plan.attention == "mla":
-      self.attn = L.MLA(b, c, inv_ts, interleaved, plan.attn_name + s)
+      if plan.mixer is not None:
+        m = plan.mixer
+        inv_ts, interleaved = ref.rope_inv_timescale(int(m["rot_dim"]), 1.0, float(m["rot"]["base"])).to(inv_ts.device), True
+        sizes = L.LatentSizes(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["q_rank"]), int(m["kv_rank"]),
+                              float(m["scale"]), int(m["mask"]["size"]))
+      self.attn = L.MLA(b, c, inv_ts, interleaved, plan.attn_name + s, sizes if plan.mixer is not None else None)
     elif plan.attention == "gdn":
-      from ..layers.gdn import GatedDeltaNet
-      self.attn = GatedDeltaNet(b, c, plan.attn_name + s)
+      from ..layers.gdn import DeltaSizes, GatedDeltaNet
+      m = plan.mixer
+      self.attn = GatedDeltaNet(b, c, plan.attn_name + s, DeltaSizes(int(m["kv_heads"]), int(m["heads"]), int(m["dim"]), int(m["vdim"]),
+                                                                     int(m["conv"])) if m is not None else None)
+    elif plan.attention == "gla":
+      from ..layers.gla import GatedLinearAttention
+      m = plan.mixer
+      self.attn = GatedLinearAttention(b, c, plan.attn_name + s, int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"]),
+                                       int(m["decay_rank"]))
     elif plan.attention == "compressed":
       from ..layers.attention_compressed import CompressedAttention
       self.attn = CompressedAttention(b, c, plan.attn_name + s, plan.compress_ratio, int(c.sliding_window_size))
@@ -113,6 +128,8 @@ class DecoderBlock:
       self.mlp = M.RoutedAndSharedMoE(b, c, plan.mlp_name + s, style=plan.moe_style, hash_routing=hashed)
     elif plan.mlp == "gemma4_moe":
       self.mlp = M.Gemma4MoE(b, c, plan.mlp_name + s)
+    elif plan.mlp == "none":
+      self.mlp = None
     else:
       self.mlp = L.MLP(b, c, plan.mlp_name + s, plan.mlp_hidden, bias=plan.mlp_bias)
     self.n2b = mk(plan.post_mlp_norm) if plan.post_mlp_norm else None
@@ -138,6 +155,8 @@ class DecoderBlock:
     if self.mhc_attn is not None:               # x [B, S, k, D]: the residual adds live inside the hyper-connections
       x = self.mhc_attn(self.n1, lambda h: self.attn(h, ctx), x)
       return self.mhc_mlp(self.n2, lambda h: self.mlp(h, ctx), x)
+    if self.plan.residual_fp32:
+      return self._call_fp32_stream(x, ctx)
     a = self.attn(self.n1(x) if self.n1 is not None else x, ctx)
     if self.n1b is not None:
       a = self.n1b(a)
@@ -149,6 +168,23 @@ class DecoderBlock:
     x = x + ctx.dropout(m, 1)
     if self.layer_scalar is not None:
       x = x * self.layer_scalar.leaf().to(x.dtype)
+    return x
+
+
+  def _call_fp32_stream(self, x, ctx: LayerCtx):
+    """x fp32 [B, S, D]. One kernel per sublayer border: the branch's norm, the residual add and the norm in front of the next
+    sublayer (of this block, or of the next layer through `ctx.next_norm` / `ctx.normed`)."""
+    m = self.plan.residual_mult
+    dt = self.n1.scale.data.dtype
+    h = ctx.normed if ctx.normed is not None else F.stream_norm(x, self.n1, dt)
+    ctx.normed = None
+    a = self.attn(h, ctx)
+    if self.mlp is None:
+      x, ctx.normed = F.residual_norm(x, a, self.n1b, m, ctx.next_norm)
+      return x
+    x, h = F.residual_norm(x, a, self.n1b, m, self.n2)
+    f = self.mlp(h, ctx)
+    x, ctx.normed = F.residual_norm(x, f, self.n2b, m, ctx.next_norm)
     return x
 
 
@@ -447,6 +483,8 @@ class Transformer:
     """mm: (soft tokens, mask) of one modality, or a list of such pairs (images, audio) merged one after the other."""
     c = self.config
     x = F.embedding(tokens, self.embedding)
+    if self.family.residual_fp32:
+      x = x.float()
     if mm is not None:
       from ..multimodal.utils import merge_mm_embeddings
       for soft, mask in ([mm] if isinstance(mm, tuple) else mm):
@@ -475,21 +513,27 @@ class Transformer:
       return 1.0 / math.sqrt(c.emb_dim)
     return 1.0
 
-  def logits(self, x):
+  def logits(self, x, normed=None):
+    """`normed`: the final norm's output when the last layer already produced it (fp32 residual streams)."""
+    if self.family.residual_fp32:
+      h = normed if normed is not None else F.stream_norm(x, self.final_norm, self.final_norm.scale.data.dtype)
+      return F.head_logits(h, self.head_param(), self.config.final_logits_soft_cap, self.head_logit_scale(), fp32_out=True)
     h = self.final_norm(x)
     return F.head_logits(h, self.head_param(), self.config.final_logits_soft_cap, self.head_logit_scale())
 
   # ------------------------------------------------------------------ plain forward (eval / inference / tests)
   @torch.no_grad()
   def forward(self, tokens, positions=None, segment_ids=None, mode="train", caches=None, images=None, image_mask=None, positions3=None,
-              audio=None, audio_mask=None):
-    """Full logits [B,S,V] in fp32; every unit must be resident (single rank or gathered by the caller).
+              audio=None, audio_mask=None, new_lens=None, logit_rows=None):
+    """Full logits [B,S,V] in fp32, or [n,V] at the flat (b * S + s) places `logit_rows`; every unit must be resident (single rank or gathered by the caller).
     `images` [B, N, 3, H, W] with `image_mask` [B, S] (True at the soft-token positions) makes the prompt multimodal;
-    `audio` (mel spectrograms, one clip per sequence) with `audio_mask` [B, S] does the same for the audio tower."""
+    `audio` (mel spectrograms, one clip per sequence) with `audio_mask` [B, S] does the same for the audio tower.
+    `new_lens` [B]: how many of the S tokens of each row are real (the rest is right padding that enters no cache or state)."""
     B, S = tokens.shape
     if positions is None:
       positions = torch.arange(S, device=tokens.device)[None].expand(B, S)
     ctx = self.make_ctx(positions, segment_ids, mode, tokens)
+    ctx.new_lens = new_lens
     ctx.positions3 = positions3.to(tokens.device) if positions3 is not None else None
     if str(getattr(self.config, "attention_type", "global")) == "block_diffusion" and caches is None:
       from ..diffusion.block_diffusion import same_block_mask
@@ -508,8 +552,15 @@ class Transformer:
     for i, layer in enumerate(self.layers):
       ctx.layer_index = i
       ctx.cache = caches[i] if caches is not None else None
+      if self.family.residual_fp32 and not torch.is_grad_enabled():
+        ctx.next_norm = self.layers[i + 1].blocks[0].n1 if i + 1 < len(self.layers) else self.final_norm
       x = layer(x, ctx)
-    return self.logits(x)
+    normed = ctx.normed
+    if logit_rows is None:
+      return self.logits(x, normed)
+    if normed is not None:
+      return self.logits(None, normed.flatten(0, 1)[logit_rows])
+    return self.logits(x.flatten(0, 1)[logit_rows][None])[0]
 
 
 class _SingleMesh:

@@ -89,7 +89,10 @@ def mm(a: torch.Tensor, b: torch.Tensor, ta: bool, tb: bool, out: torch.Tensor |
     if out.dtype == a.dtype:
       torch.mm(opa, opb, out=out)
     elif a.is_cuda:
-      out.copy_(torch.mm(opa, opb))
+      if out.dtype == torch.float32 and a.dtype == torch.bfloat16:
+        torch.mm(opa, opb, out_dtype=torch.float32, out=out)      # keep the fp32 accumulators
+      else:
+        out.copy_(torch.mm(opa, opb))
     else:
       out.copy_(torch.mm(opa.float(), opb.float()))
   return out
@@ -257,6 +260,51 @@ def rmsnorm(x: torch.Tensor, p, eps: float, offset: float = 0.0) -> torch.Tensor
   if not x2.is_contiguous():
     x2 = x2.contiguous()
   return _RMSNormFn.apply(x2, scale, p, eps, offset).view(x.shape)
+
+
+# =============================================================================== fp32 residual stream
+def _stream_kernel_ok(*ts) -> bool:
+  return not torch.is_grad_enabled() and backend.use_cuda_kernels(ts[0]) and all(t.dtype in (torch.bfloat16, torch.float32) for t in ts)
+
+
+def stream_norm(x: torch.Tensor, norm, dtype) -> torch.Tensor:
+  """RMS norm of an fp32 stream, rounded once to `dtype` (`norm` is a `layers.blocks.Norm`)."""
+  if _stream_kernel_ok(x) and x.dtype == torch.float32:
+    x2 = x.reshape(-1, x.shape[-1]).contiguous()
+    y = torch.empty(x2.shape, dtype=dtype, device=x.device)
+    backend.ext().residual_norm(x2, None, None, 0.0, norm.scale.data, y, float(norm.eps), float(norm.eps), float(norm.offset))
+    return y.view(x.shape)
+  return ref.rmsnorm_f32(x, norm.scale.leaf(), norm.eps, norm.offset).to(dtype)
+
+
+def residual_norm(x: torch.Tensor, branch: torch.Tensor, post, mult: float, nxt=None):
+  """(x + mult * post(branch), nxt(of that) in the branch's dtype or None): the fp32 residual add of a sandwich-normed branch
+  together with the norm that reads the stream next. On a GPU one kernel, which updates x in place."""
+  if _stream_kernel_ok(x, branch) and x.dtype == torch.float32 and x.is_contiguous():
+    x2, b2 = x.view(-1, x.shape[-1]), branch.reshape(-1, x.shape[-1]).contiguous()
+    y = torch.empty_like(b2) if nxt is not None else None
+    assert nxt is None or nxt.offset == post.offset
+    backend.ext().residual_norm(x2, b2, post.scale.data, float(mult), nxt.scale.data if nxt is not None else None, y, float(post.eps),
+                                float(nxt.eps) if nxt is not None else 0.0, float(post.offset))
+    return x, (y.view(x.shape) if y is not None else None)
+  x = x.float() + mult * ref.rmsnorm_f32(branch, post.scale.leaf(), post.eps, post.offset)
+  return x, (ref.rmsnorm_f32(x, nxt.scale.leaf(), nxt.eps, nxt.offset).to(branch.dtype) if nxt is not None else None)
+
+
+# =============================================================================== activation (ungated)
+_PLAIN_ACT_CODE = {"silu": 0, "swish": 0, "gelu": 1, "relu": 2, "gelu_exact": 4}
+
+
+def act(h: torch.Tensor, name: str) -> torch.Tensor:
+  """act(h) elementwise, fp32 inside, in h's dtype."""
+  if name == "linear":
+    return h
+  if not torch.is_grad_enabled() and name in _PLAIN_ACT_CODE and backend.use_cuda_kernels(h) and h.is_contiguous() \
+      and h.dtype in (torch.bfloat16, torch.float32):
+    out = torch.empty_like(h)
+    backend.ext().act_fwd(h.view(-1), out.view(-1), _PLAIN_ACT_CODE[name])
+    return out
+  return ref.act_fn(name)(h.float()).to(h.dtype)
 
 
 # =============================================================================== gated activation
@@ -668,9 +716,11 @@ def fused_head_loss(h: torch.Tensor, head, targets: torch.Tensor, weights: torch
   return loss_sum, z_sum, dh
 
 
-def head_logits(h: torch.Tensor, head, soft_cap: float = 0.0, logit_scale: float = 1.0) -> torch.Tensor:
-  """Full fp32 logits (inference / evaluation of small batches)."""
-  lg = mm(h.reshape(-1, h.shape[-1]), head.data, False, True).float().view(*h.shape[:-1], head.data.shape[0])
+def head_logits(h: torch.Tensor, head, soft_cap: float = 0.0, logit_scale: float = 1.0, fp32_out: bool = False) -> torch.Tensor:
+  """Full fp32 logits (inference / evaluation of small batches). `fp32_out` keeps the product's fp32 accumulators instead of rounding
+  the logits to the compute dtype first."""
+  lg = mm(h.reshape(-1, h.shape[-1]), head.data, False, True, out_dtype=torch.float32 if fp32_out else None)
+  lg = lg.float().view(*h.shape[:-1], head.data.shape[0])
   if logit_scale != 1.0:
     lg = lg * logit_scale
   if soft_cap and soft_cap > 0:

@@ -1,0 +1,69 @@
+"""Inference kernels of the recurrent layers (gated delta network, gated linear attention): `csrc/recurrent_sm100.cu`.
+
+Both layers keep a matrix state per head; the kernels take the layer's raw projections and return its gated, normalised head outputs
+[B, S, H * Dv] ready for the output projection. One token per sequence is one fused launch (convolution, gates, state update,
+read-out, norm); longer inputs run convolution -> recurrence -> norm. States are read and written in the rows `slot_ids` of the
+layer's `RecurrentState`; rows with `lengths` 0 start from zero, and only the first `new_lens` tokens of a row count.
+"""
+from __future__ import annotations
+
+import torch
+
+from . import backend
+
+
+def kernels_ok(t: torch.Tensor) -> bool:
+  return not torch.is_grad_enabled() and t.dtype in (torch.bfloat16, torch.float32) and backend.use_cuda_kernels(t)
+
+
+def gated_head_norm(o, z, scale, eps):
+  """Definition: o [.., H, Dv] RMS-normalised over Dv, times scale, times silu(z); fp32."""
+  o = o.float()
+  o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * scale.float()
+  return o * torch.nn.functional.silu(z.float())
+
+
+def delta_forward(layer, qkvz, ba, st):
+  """layer: GatedDeltaNet; qkvz [B,S,hk*(2dk+2r dv)], ba [B,S,2hv]."""
+  B, S, _ = qkvz.shape
+  E = backend.ext()
+  N = B * S
+  dev, dt = qkvz.device, qkvz.dtype
+  eps = float(layer.c.normalization_layer_epsilon)
+  out = torch.empty(B, S, layer.value_dim, dtype=dt, device=dev)
+  q2, b2 = qkvz.view(N, -1), ba.reshape(N, -1)
+  w = layer.conv.data.view(layer.K, layer.conv_dim)
+  if S == 1:
+    E.delta_decode(q2, b2, w, layer.A_log.data, layer.dt_bias.data, layer.norm.data, eps, layer.hk, layer.hv, layer.dk, layer.dv, st.conv,
+                   st.rec, st.slot_ids, st.lengths, out.view(N, -1))
+    return out
+  mixed = torch.empty(N, layer.conv_dim, dtype=dt, device=dev)
+  E.delta_conv(q2, w, layer.hk, layer.hv, layer.dk, layer.dv, S, st.conv, st.slot_ids, st.lengths, st.new_lens, mixed)
+  o = torch.empty(N, layer.value_dim, dtype=dt, device=dev)
+  E.delta_scan(mixed, b2, layer.A_log.data, layer.dt_bias.data, layer.hk, layer.hv, layer.dk, layer.dv, S, st.rec, st.slot_ids, st.lengths,
+               st.new_lens, o)
+  r = layer.r
+  E.gated_head_norm(o, q2, layer.hv, layer.dv, r, 2 * layer.dk + r * layer.dv, 2 * layer.dk + 2 * r * layer.dv, layer.norm.data, eps,
+                    out.view(N, -1))
+  return out
+
+
+def gla_forward(layer, p, st):
+  """layer: GatedLinearAttention; p [B,S,2H(dk+dv)+rank]."""
+  B, S, _ = p.shape
+  E = backend.ext()
+  N = B * S
+  H, dk, dv = layer.heads, layer.dk, layer.dv
+  eps = float(layer.c.normalization_layer_epsilon)
+  out = torch.empty(B, S, H * dv, dtype=p.dtype, device=p.device)
+  p2 = p.view(N, -1)
+  if S == 1:
+    E.gla_decode(p2, layer.decay.data, layer.decay_bias.data, layer.norm.data, eps, layer.tau, H, dk, dv, st.rec, st.slot_ids, st.lengths,
+                 out.view(N, -1))
+    return out
+  log_alpha = torch.empty(N, H * dk, dtype=torch.float32, device=p.device)
+  E.gla_decay(p2, 2 * H * (dk + dv), layer.decay.data, layer.decay_bias.data, layer.tau, log_alpha)
+  o = torch.empty(N, H * dv, dtype=p.dtype, device=p.device)
+  E.gla_scan(p2, log_alpha, H, dk, dv, S, st.rec, st.slot_ids, st.lengths, st.new_lens, o)
+  E.gated_head_norm(o, p2, H, dv, 1, 2 * H * dk + H * dv, dv, layer.norm.data, eps, out.view(N, -1))
+  return out

@@ -24,6 +24,13 @@ def rmsnorm(x: torch.Tensor, scale: torch.Tensor | None, eps: float, offset: flo
   return y * (scale.to(x.dtype) + offset)
 
 
+def rmsnorm_f32(x: torch.Tensor, scale: torch.Tensor | None, eps: float, offset: float = 0.0) -> torch.Tensor:
+  """The norm of an fp32 residual stream: everything, the scale included, in fp32; fp32 result."""
+  xf = x.float()
+  y = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
+  return y if scale is None else y * (scale.float() + offset)
+
+
 def rmsnorm_bwd(dy, x, scale, eps, offset=0.0):
   xf, dyf = x.float(), dy.float()
   rstd = torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)

@@ -73,10 +73,28 @@ def training_tflops_per_device(c, batch_per_device: float | None = None) -> tupl
   return 3 * (weight + attention) * g / 1e12, 3 * weight * g / 1e12, 3 * attention * g / 1e12
 
 
+def _sized_mixer(bp, B, S, d):
+  """The same for a block that brings its own mixer sizes (`layer_specs`)."""
+  bs, m = B * S, bp.mixer
+  H, dv = m["heads"], m["vdim"]
+  if bp.attention == "mla":
+    qk = m["dim"] + m["rot_dim"]
+    w = d * m["q_rank"] + m["q_rank"] * H * qk + d * (m["kv_rank"] + m["rot_dim"]) + m["kv_rank"] * H * (m["dim"] + dv) + H * dv * d
+    win = min(int(m["mask"]["size"]), S)
+    return 2 * bs * w, 2 * B * (S * win - 0.5 * win * win) * H * (qk + dv)
+  if bp.attention == "gdn":
+    kd = m["kv_heads"] * m["dim"]
+    return 2 * bs * (d * (2 * kd + 2 * H * dv + 2 * H) + H * dv * d + m["conv"] * (2 * kd + H * dv)), bs * H * m["dim"] * dv * 8
+  w = d * (2 * H * m["dim"] + 2 * H * dv + m["decay_rank"]) + m["decay_rank"] * H * m["dim"] + H * dv * d
+  return 2 * bs * w, bs * H * m["dim"] * dv * 6
+
+
 def _block(c, bp, B, S, n_act):
   """(weight FLOPs, attention FLOPs) of one block, forward."""
   bs, d = B * S, c.emb_dim
-  if bp.attention == "mla":
+  if bp.mixer is not None:
+    proj_w, attn = _sized_mixer(bp, B, S, d)
+  elif bp.attention == "mla":
     qk = c.qk_nope_head_dim + c.qk_rope_head_dim
     if c.q_lora_rank > 0:
       q = 2 * bs * (d * c.q_lora_rank + c.q_lora_rank * c.num_query_heads * qk)
@@ -103,7 +121,9 @@ def _block(c, bp, B, S, n_act):
       attn = 4 * B * (n * bp.chunk ** 2 + rem ** 2) * c.num_query_heads * dh / 2   # causal triangles of the chunks
     else:
       attn = 4 * bs * S * c.num_query_heads * dh / 2
-  if bp.mlp in ("moe", "moe_shared", "gemma4_moe"):
+  if bp.mlp == "none":
+    ffn = 0
+  elif bp.mlp in ("moe", "moe_shared", "gemma4_moe"):
     ffn = 2 * bs * d * c.num_experts + _ffn(bs, d, c.moe_mlp_dim, n_act) * c.num_experts_per_tok
     if bp.mlp == "moe_shared" and c.shared_experts > 0:
       ffn += _ffn(bs, d, c.moe_mlp_dim * c.shared_experts, n_act)
