@@ -23,7 +23,7 @@ class Suite:
 
   def check(self, got, want, dtype, what=""):
     e = M.rel_rows(got, want)
-    assert float(e.max()) < self.tol[dtype] and float(e.median()) < self.mid[dtype], f"{what}: worst {float(e.max())}, middle {float(e.median())}"
+    assert float(e.max()) < self.tol[dtype] and (len(e) < 8 or float(e.median()) < self.mid[dtype]), f"{what}: worst {float(e.max())}, middle {float(e.median())}"
 
   # ---- every mechanism alone and together, whole prompts
   @pytest.mark.parametrize("name", sorted(M.SPECS))
