@@ -239,7 +239,16 @@ def main():
   ap.add_argument("--no-precheck", action="store_true", help="skip the untimed fused-vs-NCCL equivalence check that multi-GPU runs do first")
   ap.add_argument("--comm", default="fused", choices=["fused", "nccl"],
                   help="FSDP collectives: this repository's NVLink kernels fused with the GEMMs (default) or plain NCCL (comparison arm)")
+  ap.add_argument("--serving", action="store_true", help="instead of the training step: prefill and decode throughput of silinex-1b and of plain "
+                  "models of equal size, one JSON line per model (maxtext_b200/benchmarks/serving_bench.py; one GPU)")
+  ap.add_argument("--serving-models", default="")
+  ap.add_argument("--serving-lengths", default="512,2048,8192")
+  ap.add_argument("--serving-slots", default="1,32,128")
+  ap.add_argument("--serving-context", type=int, default=2048)
   args = ap.parse_args()
+  if args.serving:
+    from maxtext_b200.benchmarks import serving_bench
+    return serving_bench.main(args.serving_models, args.serving_lengths, args.serving_slots, args.serving_context, max(args.steps, 5))
   preset = PRESETS[args.config]
   args.model = args.model or preset["model"]
   args.seq = args.seq or preset["seq"]

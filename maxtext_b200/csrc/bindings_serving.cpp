@@ -20,6 +20,12 @@ int mt_delta_scan(int f32, const void* mixed, const void* ba, long ldb, const vo
                   float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* o, int B, cudaStream_t st);
 int mt_gla_scan(int f32, const void* x, long ldx, const float* log_alpha, int H, int dk, int dv, int S, float* rec, const int64_t* slots,
                 const int64_t* lengths, const int64_t* new_lens, void* o, int B, cudaStream_t st);
+int mt_chunk_supported(int dk, int dv);
+int mt_delta_chunks(const void* mixed, long ldx, const void* ba, long ldb, const void* A_log, const void* dt_bias, int hk, int hv, int dk, int dv, int S,
+                    int t_lo, int t_hi, float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* tp, float* gates, float* ends,
+                    void* o, int B, cudaStream_t st);
+int mt_gla_chunks(const void* x, long ldx, const float* log_alpha, int H, int dk, int dv, int S, int t_lo, int t_hi, float* rec, const int64_t* slots,
+                  const int64_t* lengths, const int64_t* new_lens, void* aa, void* qkg, float* ends, void* o, int B, cudaStream_t st);
 int mt_gla_decay(int f32, const void* lo, long ldx, const void* w, const void* bias, int rank, float inv_tau, float* out, long N, int C, cudaStream_t st);
 int mt_gated_head_norm(int f32, const void* o, const void* x, long ldx, long rows, int H, int dv, int r, long zoff, long zstride, const void* w, float eps,
                        void* out, cudaStream_t st);
@@ -187,6 +193,56 @@ void gla_scan(const Tensor& x, const Tensor& log_alpha, int64_t H, int64_t dk, i
                    longs(lengths, B, "lengths"), longs(new_lens, B, "new_lens"), o.data_ptr(), (int)B, stream()), "gla_scan");
 }
 
+// tokens of every row handled per launch pair, so that the per-chunk scratch stays near 256 MB
+int64_t chunk_segment(int64_t B, int64_t H, int64_t S, int64_t bytes_per_token_head) {
+  const int64_t fit = (int64_t(256) << 20) / std::max<int64_t>(1, B * H * bytes_per_token_head);
+  return std::min((S + 63) / 64 * 64, std::max<int64_t>(64, fit / 64 * 64));
+}
+
+bool chunk_supported(int64_t dk, int64_t dv) { return mt_chunk_supported((int)dk, (int)dv) != 0; }
+
+// the chunked form of delta_scan (bf16)
+void delta_chunks(const Tensor& mixed, const Tensor& ba, const Tensor& A_log, const Tensor& dt_bias, int64_t hk, int64_t hv, int64_t dk, int64_t dv,
+                  int64_t S, Tensor& rec, const Tensor& slots, const Tensor& lengths, const OptTensor& new_lens, Tensor& o) {
+  TORCH_CHECK(!f32(mixed) && chunk_supported(dk, dv), "delta_chunks: bf16 and head widths of 16 .. 128 in steps of 16");
+  const int64_t B = slots.numel(), cd = 2 * hk * dk + hv * dv;
+  same(mixed, mixed, B * S * cd, "mixed");
+  TORCH_CHECK((reinterpret_cast<uintptr_t>(mixed.data_ptr()) % 16) == 0);
+  rows2d(ba, mixed, B * S, 2 * hv, "gates");
+  same(A_log, mixed, hv, "A_log"); same(dt_bias, mixed, hv, "dt_bias"); same(o, mixed, B * S * hv * dv, "o");
+  float* rp = state(rec, {hv, dk, dv}, "rec");
+  const int64_t *sl = longs(slots, B, "slots"), *le = longs(lengths, B, "lengths"), *nl = longs(new_lens, B, "new_lens");
+  c10::cuda::CUDAGuard guard(mixed.device());
+  const int64_t seg = chunk_segment(B, hv, S, 4 * 64 * 2), tiles = B * (seg / 64) * hv;
+  auto fo = torch::dtype(torch::kFloat32).device(mixed.device());
+  auto tp = torch::empty({tiles * 4 * 64 * 64}, mixed.options());
+  auto gates = torch::empty({tiles * 4 * 64}, fo), ends = torch::empty({tiles}, fo);
+  for (int64_t t = 0; t < S; t += seg)
+    done(mt_delta_chunks(mixed.data_ptr(), cd, ba.data_ptr(), ba.stride(0), A_log.data_ptr(), dt_bias.data_ptr(), (int)hk, (int)hv, (int)dk, (int)dv, (int)S,
+                         (int)t, (int)std::min(S, t + seg), rp, sl, le, nl, tp.data_ptr(), gates.data_ptr<float>(), ends.data_ptr<float>(), o.data_ptr(), (int)B,
+                         stream()), "delta_chunks", 2);
+}
+
+// the chunked form of gla_scan (bf16)
+void gla_chunks(const Tensor& x, const Tensor& log_alpha, int64_t H, int64_t dk, int64_t dv, int64_t S, Tensor& rec, const Tensor& slots,
+                const Tensor& lengths, const OptTensor& new_lens, Tensor& o) {
+  TORCH_CHECK(!f32(x) && chunk_supported(dk, dv), "gla_chunks: bf16 and head widths of 16 .. 128 in steps of 16");
+  const int64_t B = slots.numel();
+  rows2d(x, x, B * S, 2 * H * (dk + dv), "packed projection");
+  TORCH_CHECK((reinterpret_cast<uintptr_t>(x.data_ptr()) % 16) == 0 && x.stride(0) % 8 == 0);
+  TORCH_CHECK(log_alpha.is_cuda() && log_alpha.scalar_type() == torch::kFloat32 && log_alpha.is_contiguous() && log_alpha.numel() == B * S * H * dk);
+  same(o, x, B * S * H * dv, "o");
+  float* rp = state(rec, {H, dk, dv}, "rec");
+  const int64_t *sl = longs(slots, B, "slots"), *le = longs(lengths, B, "lengths"), *nl = longs(new_lens, B, "new_lens");
+  c10::cuda::CUDAGuard guard(x.device());
+  const int64_t seg = chunk_segment(B, H, S, 2 * 64 * 2 + 4 * dk * 2), tiles = B * (seg / 64) * H;
+  auto aa = torch::empty({tiles * 2 * 64 * 64}, x.options()), qkg = torch::empty({tiles * 4 * 64 * dk}, x.options());
+  auto ends = torch::empty({tiles * dk}, torch::dtype(torch::kFloat32).device(x.device()));
+  for (int64_t t = 0; t < S; t += seg)
+    done(mt_gla_chunks(x.data_ptr(), x.stride(0), log_alpha.data_ptr<float>(), (int)H, (int)dk, (int)dv, (int)S, (int)t, (int)std::min(S, t + seg), rp, sl, le,
+                       nl, aa.data_ptr(), qkg.data_ptr(), ends.data_ptr<float>(), o.data_ptr(), (int)B, stream()), "gla_chunks", 2);
+}
+
 void gated_head_norm(const Tensor& o, const Tensor& x, int64_t H, int64_t dv, int64_t r, int64_t zoff, int64_t zstride, const Tensor& w, double eps,
                      Tensor& out) {
   const bool f = f32(o);
@@ -285,6 +341,9 @@ void register_serving(pybind11::module_& m) {
   m.def("gla_decode", &gla_decode);
   m.def("gla_decay", &gla_decay);
   m.def("gla_scan", &gla_scan);
+  m.def("chunk_supported", &chunk_supported);
+  m.def("delta_chunks", &delta_chunks);
+  m.def("gla_chunks", &gla_chunks);
   m.def("gated_head_norm", &gated_head_norm);
   m.def("mla_prep", &mla_prep);
   m.def("mla_pack", &mla_pack);

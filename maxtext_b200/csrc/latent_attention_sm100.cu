@@ -8,6 +8,7 @@
 //    fit that form (fp32, latents not a multiple of 64) take a plain kernel with fp32 arithmetic.
 // Lengths and slots are device memory: nothing synchronises with the host, so a decode step can be captured in a graph.
 #include "serving_common.cuh"
+#include "warp_mma.cuh"
 
 namespace mt {
 
@@ -262,30 +263,6 @@ __global__ void __launch_bounds__(256) mla_attn_plain_kernel(AttnArgs a, const T
 
 // Tensor-core form (bf16): grid (splits, ceil(H / 16), B), 256 threads. Tiles of 64 keys, two in flight. Warp w: scores of keys 8 w .. 8 w + 7
 // for 16 heads; then columns [w * R / 8, (w + 1) * R / 8) of the weighted sum. CT = R / 64 column tiles of 8 per warp.
-__device__ __forceinline__ void la_cp_async16(void* smem, const void* gmem, int src_bytes) {
-  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(s), "l"(gmem), "r"(src_bytes));
-}
-__device__ __forceinline__ void la_commit() { asm volatile("cp.async.commit_group;\n" ::); }
-template <int N> __device__ __forceinline__ void la_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
-__device__ __forceinline__ void la_ldm4(unsigned* r, const void* p) {
-  const unsigned s = (unsigned)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
-}
-__device__ __forceinline__ void la_ldm4t(unsigned* r, const void* p) {
-  const unsigned s = (unsigned)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));
-}
-__device__ __forceinline__ void la_ldm2t(unsigned* r, const void* p) {
-  const unsigned s = (unsigned)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(s));
-}
-__device__ __forceinline__ void la_mma(float* d, const unsigned* a, unsigned b0, unsigned b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
 constexpr int TC_KEYS = 64, TC_NT = 256, TC_PLD = TC_KEYS + 8;
 
 template <int CT>

@@ -1,0 +1,522 @@
+// Prompts through the recurrent layers in chunks of 64 tokens (bf16 models, head widths that are multiples of 16 up to 128). The recurrences are
+// those of recurrent_sm100.cu. Two kernels per layer:
+//
+//  * prepare, parallel over (chunk, head, sequence): everything that does not depend on the incoming state.
+//      gated delta: with G_i the log-decay summed from the chunk's start, r the inverse norms of q and k,
+//        L_ij = beta_i rk_i rk_j (k_i . k_j) e^(G_i - G_j)  (j < i),   T = (I + L)^-1,   P_ij = rq_i rk_j (q_i . k_j) e^(G_i - G_j)  (j <= i)
+//      gated linear attention: G per key channel;  A_ij = sum_d q_id k_jd e^(G_id - G_jd)  (j <= i),  q e^G,  k e^(G_end - G).
+//        Exponents are formed so that none is positive: 16 x 16 blocks below the diagonal are split at the first row of their block row,
+//        diagonal blocks are summed with their own exponent per term.
+//  * carry, one CTA per (16 state columns, head, sequence), chunk after chunk with the state in fp32 registers and the next chunk's tiles in flight:
+//      gated delta:  X = K S, Y = Q S;  R = beta (V - rk e^G X);  U = T R;  O = rq e^G Y + P U;  S <- e^G_end S + K^T (rk e^(G_end - G) U)
+//      linear:       O = (q e^G) S + A V;  S <- diag(e^G_end) S + (k e^(G_end - G))^T V
+//
+// Products run on mma.sync m16n8k16. q, k, v are exact bf16 operands; every fp32 operand (S, T, P, A, R, U, the decayed q and k) enters as a
+// (high, low) bf16 pair, so no factor loses more than its last 8 bits of 24. The tiles are 64 x 16 with a strict chain from chunk to chunk: the
+// round trip of an accumulator through tensor memory would cost more than the products themselves.
+#include "serving_common.cuh"
+#include "warp_mma.cuh"
+
+namespace mt {
+
+typedef __nv_bfloat16 bf16;
+
+constexpr int CH = 64;           // tokens per chunk
+constexpr int CN = 16;           // state columns per carry CTA
+constexpr int CLD = CH + 8;      // padded row of a 64-wide tile
+constexpr int NLD = CN + 8;      // padded row of a 16-wide tile
+
+struct ChunkArgs {
+  int H, r, dk, dv, S;           // value heads, value heads per key head, widths, tokens per row of the batch
+  int t_lo, t_hi, chunks;        // this launch covers tokens [t_lo, t_hi) of every row in `chunks` chunks
+  const int64_t* slots;
+  const int64_t* lengths;
+  const int64_t* new_lens;       // or null
+  float* rec;                    // [slots, H, dk, dv]
+};
+
+__device__ __forceinline__ int real_tokens(const ChunkArgs& a, int b) { return min(a.t_hi, a.new_lens ? (int)a.new_lens[b] : a.S); }
+__device__ __forceinline__ long chunk_id(const ChunkArgs& a, int b, int c, int h) { return ((long)b * a.chunks + c) * a.H + h; }
+
+// rows [0, CH) of a [CH, dk] bf16 tile to shared memory (row length ld), zeros past row m; dk is a multiple of 8
+__device__ __forceinline__ void tile_async(bf16* dst, int ld, const bf16* src, long stride, int cols, int m, int tid, int nt) {
+  const int v = cols / 8;
+  for (int i = tid; i < CH * v; i += nt) {
+    const int r = i / v, c = (i % v) * 8;
+    la_cp_async16(dst + r * ld + c, src + (long)(r < m ? r : 0) * stride + c, r < m ? 16 : 0);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ gated delta: prepare
+// grid (chunks, H, B), 128 threads. tp: per chunk and head four [64][64] bf16 tiles: T high, T low, P high, P low;
+// gates: per chunk and head [4][64] floats: rk e^G, beta, rq e^G, rk e^(G_end - G), and e^G_end in gate_end.
+__global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(ChunkArgs a, const bf16* __restrict__ mixed, long ldx, const bf16* __restrict__ ba, long ldb,
+                                                                  const bf16* __restrict__ A_log, const bf16* __restrict__ dt_bias, bf16* __restrict__ tp,
+                                                                  float* __restrict__ gates, float* __restrict__ gate_end) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int dk = a.dk, r = a.r, kh = h / r, LD = dk + 8, t0 = a.t_lo + c * CH;
+  const int m = min(CH, real_tokens(a, b) - t0);
+  if (m <= 0) return;
+  bf16* ks = reinterpret_cast<bf16*>(raw);               // [64][LD]
+  bf16* qs = ks + CH * LD;
+  float* L = reinterpret_cast<float*>(qs + CH * LD);     // [64][68]
+  __shared__ float G[CH], beta[CH], rk[CH], rq[CH], half_sum;
+  const bf16* row0 = mixed + ((long)b * a.S + t0) * ldx;
+  tile_async(qs, LD, row0 + (long)kh * dk, ldx, dk, m, tid, 128);
+  tile_async(ks, LD, row0 + (long)(a.H / r + kh) * dk, ldx, dk, m, tid, 128);
+  la_commit();
+  float lg = 0.f;
+  if (tid < CH) {
+    float be = 0.f;
+    if (tid < m) {
+      const bf16* bb = ba + ((long)b * a.S + t0 + tid) * ldb + (long)kh * 2 * r + (h - kh * r);
+      lg = -expf(to_f(A_log[h])) * softplus_f(to_f(bb[r]) + to_f(dt_bias[h]));
+      be = sigmoid_f(to_f(bb[0]));
+    }
+    beta[tid] = be;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float x = __shfl_up_sync(0xffffffffu, lg, o);
+      if (lane >= o) lg += x;
+    }
+    if (tid == 31) half_sum = lg;
+  }
+  la_wait<0>();
+  __syncthreads();
+  if (tid < CH) G[tid] = lg + (tid >= 32 ? half_sum : 0.f);
+  // inverse norms: eight lanes per row, 16 rows of q and k per warp
+  for (int i = 0; i < 16; i += 4) {
+    const int row = warp * 16 + i + (lane >> 3);
+    float sk = 0.f, sq = 0.f;
+    for (int d = (lane & 7) * 2; d < dk; d += 16) {
+      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(ks + row * LD + d));
+      const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(qs + row * LD + d));
+      sk += x.x * x.x + x.y * x.y;
+      sq += y.x * y.x + y.y * y.y;
+    }
+#pragma unroll
+    for (int o = 1; o < 8; o <<= 1) {
+      sk += __shfl_xor_sync(0xffffffffu, sk, o);
+      sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    }
+    if ((lane & 7) == 0) {
+      rk[row] = rsqrtf(sk + 1e-6f);
+      rq[row] = rsqrtf(sq + 1e-6f) * rsqrtf((float)dk);
+    }
+  }
+  __syncthreads();
+  // rows 16 warp .. 16 warp + 15 of K K^T and Q K^T, columns up to the diagonal block
+  float kk[8][4], qk[8][4];
+#pragma unroll
+  for (int n = 0; n < 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) kk[n][e] = qk[n][e] = 0.f;
+  for (int k = 0; k < dk; k += 16) {
+    unsigned fk[4], fq[4];
+    la_ldm4(fk, ks + (warp * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+    la_ldm4(fq, qs + (warp * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+#pragma unroll
+    for (int n = 0; n < 8; n += 2) {
+      if (n <= 2 * warp) {
+        unsigned fb[4];                                  // columns 8 n .. 8 n + 15
+        la_ldm4(fb, ks + (n * 8 + (lane & 7) + ((lane >> 4) << 3)) * LD + k + ((lane >> 3) & 1) * 8);
+        la_mma(kk[n], fk, fb[0], fb[1]);
+        la_mma(kk[n + 1], fk, fb[2], fb[3]);
+        la_mma(qk[n], fq, fb[0], fb[1]);
+        la_mma(qk[n + 1], fq, fb[2], fb[3]);
+      }
+    }
+  }
+  bf16* out = tp + chunk_id(a, b, c, h) * 4 * CH * CH;
+#pragma unroll
+  for (int n = 0; n < 8; ++n) {
+#pragma unroll
+    for (int e = 0; e < 4; e += 2) {
+      const int i = warp * 16 + (lane >> 2) + (e ? 8 : 0), j = n * 8 + (lane & 3) * 2;
+      float l[2] = {0.f, 0.f}, p[2] = {0.f, 0.f};
+      if (n <= 2 * warp + 1) {
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          if (j + x <= i) {
+            const float f = expf(G[i] - G[j + x]) * rk[j + x];
+            p[x] = qk[n][e + x] * f * rq[i];
+            if (j + x < i) l[x] = kk[n][e + x] * f * rk[i] * beta[i];
+          }
+        }
+        __nv_bfloat162 hi, lo;
+        la_split2(p[0], p[1], hi, lo);
+        *reinterpret_cast<__nv_bfloat162*>(out + 2 * CH * CH + i * CH + j) = hi;
+        *reinterpret_cast<__nv_bfloat162*>(out + 3 * CH * CH + i * CH + j) = lo;
+      }
+      *reinterpret_cast<float2*>(L + i * 68 + j) = make_float2(l[0], l[1]);
+    }
+  }
+  __syncthreads();
+  if (tid < CH) {
+    // column tid of T by forward substitution: T_i = [i == tid] - sum_{k < i} L_ik T_k
+    float t[CH];
+#pragma unroll
+    for (int i = 0; i < CH; ++i) {
+      float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+#pragma unroll
+      for (int k = 0; k < (i & ~3); k += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(L + i * 68 + k);
+        s0 += l.x * t[k]; s1 += l.y * t[k + 1]; s2 += l.z * t[k + 2]; s3 += l.w * t[k + 3];
+      }
+#pragma unroll
+      for (int k = i & ~3; k < i; ++k) s0 += L[i * 68 + k] * t[k];
+      t[i] = (i == tid ? 1.f : 0.f) - ((s0 + s1) + (s2 + s3));
+      const bf16 hi = __float2bfloat16_rn(t[i]);
+      out[i * CH + tid] = hi;
+      out[CH * CH + i * CH + tid] = __float2bfloat16_rn(t[i] - __bfloat162float(hi));
+    }
+  } else {
+    const int i = tid - CH;
+    float* g = gates + chunk_id(a, b, c, h) * 4 * CH;
+    const float end = G[CH - 1];
+    g[i] = rk[i] * expf(G[i]);
+    g[CH + i] = beta[i];
+    g[2 * CH + i] = rq[i] * expf(G[i]);
+    g[3 * CH + i] = rk[i] * expf(end - G[i]);
+    if (i == 0) gate_end[chunk_id(a, b, c, h)] = expf(end);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ gated linear attention: prepare
+// grid (chunks, H, B), 256 threads. aa: per chunk and head A high, A low [64][64]; qkg: per chunk and head four [64][dk] tiles: q e^G high, low,
+// k e^(G_end - G) high, low; end: e^G_end [dk].
+__global__ void __launch_bounds__(256) gla_chunk_prepare_kernel(ChunkArgs a, const bf16* __restrict__ x, long ldx, const float* __restrict__ log_alpha,
+                                                                bf16* __restrict__ aa, bf16* __restrict__ qkg, float* __restrict__ end) {
+  extern __shared__ __align__(16) float sm[];
+  const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
+  const int dk = a.dk, H = a.H, LD = dk + 4, t0 = a.t_lo + c * CH;
+  const int m = min(CH, real_tokens(a, b) - t0);
+  if (m <= 0) return;
+  float* G = sm;                                         // [64][LD]
+  float* ksc = G + CH * LD;                              // [48][LD] scaled keys of the blocks left of the diagonal
+  float* qsc = ksc + 48 * LD;                            // [16][LD]
+  bf16* q = reinterpret_cast<bf16*>(qsc + 16 * LD);      // [64][dk + 8]
+  bf16* k = q + CH * (dk + 8);
+  const int QLD = dk + 8;
+  const bf16* row0 = x + ((long)b * a.S + t0) * ldx;
+  tile_async(q, QLD, row0 + (long)h * dk, ldx, dk, m, tid, 256);
+  tile_async(k, QLD, row0 + (long)(H + h) * dk, ldx, dk, m, tid, 256);
+  la_commit();
+  if (tid < dk) {
+    const float* la = log_alpha + ((long)b * a.S + t0) * H * dk + (long)h * dk + tid;
+    float g = 0.f;
+#pragma unroll 8
+    for (int i = 0; i < CH; ++i) {
+      if (i < m) g += la[(long)i * H * dk];
+      G[i * LD + tid] = g;
+    }
+  }
+  la_wait<0>();
+  __syncthreads();
+  const float scale = rsqrtf((float)dk);
+  const long id = chunk_id(a, b, c, h);
+  bf16* qg = qkg + id * 4 * CH * dk;
+  for (int i = tid; i < CH * dk / 2; i += 256) {
+    const int t = i / (dk / 2), d = (i % (dk / 2)) * 2;
+    const float2 qv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(q + t * QLD + d));
+    const float2 kv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + t * QLD + d));
+    const float g0 = G[t * LD + d], g1 = G[t * LD + d + 1], e0 = G[(CH - 1) * LD + d], e1 = G[(CH - 1) * LD + d + 1];
+    __nv_bfloat162 hi, lo;
+    la_split2(qv.x * scale * expf(g0), qv.y * scale * expf(g1), hi, lo);
+    *reinterpret_cast<__nv_bfloat162*>(qg + t * dk + d) = hi;
+    *reinterpret_cast<__nv_bfloat162*>(qg + CH * dk + t * dk + d) = lo;
+    la_split2(kv.x * expf(e0 - g0), kv.y * expf(e1 - g1), hi, lo);
+    *reinterpret_cast<__nv_bfloat162*>(qg + 2 * CH * dk + t * dk + d) = hi;
+    *reinterpret_cast<__nv_bfloat162*>(qg + 3 * CH * dk + t * dk + d) = lo;
+  }
+  if (tid < dk) end[id * dk + tid] = expf(G[(CH - 1) * LD + tid]);
+  bf16* ah = aa + id * 2 * CH * CH;
+  auto put = [&](int i, int j, float v) {
+    const bf16 hi = __float2bfloat16_rn(v);
+    ah[i * CH + j] = hi;
+    ah[CH * CH + i * CH + j] = __float2bfloat16_rn(v - __bfloat162float(hi));
+  };
+  // diagonal blocks: thread (i, j) of each 16 x 16 block, the exponent of every term on its own
+  {
+    const int i0 = tid >> 4, j0 = tid & 15;
+    for (int blk = 0; blk < 4; ++blk) {
+      const int i = blk * 16 + i0, j = blk * 16 + j0;
+      float s = 0.f;
+      if (j <= i)
+        for (int d = 0; d < dk; ++d) s += to_f(q[i * QLD + d]) * to_f(k[j * QLD + d]) * expf(G[i * LD + d] - G[j * LD + d]);
+      put(i, j, s * scale);
+    }
+  }
+  // blocks below the diagonal, block row by block row: exponents split at the last token before the block row
+  for (int I = 1; I < 4; ++I) {
+    const float* ref = G + (I * 16 - 1) * LD;
+    __syncthreads();
+    for (int i = tid; i < 16 * dk; i += 256) {
+      const int t = i / dk, d = i % dk;
+      qsc[t * LD + d] = to_f(q[(I * 16 + t) * QLD + d]) * scale * expf(G[(I * 16 + t) * LD + d] - ref[d]);
+    }
+    for (int i = tid; i < I * 16 * dk; i += 256) {
+      const int t = i / dk, d = i % dk;
+      ksc[t * LD + d] = to_f(k[t * QLD + d]) * expf(ref[d] - G[t * LD + d]);
+    }
+    __syncthreads();
+    const int i0 = tid >> 4, j0 = tid & 15;
+    float s[3] = {0.f, 0.f, 0.f};
+    for (int d = 0; d < dk; d += 4) {
+      const float4 u = *reinterpret_cast<const float4*>(qsc + i0 * LD + d);
+#pragma unroll
+      for (int J = 0; J < 3; ++J) {
+        if (J < I) {
+          const float4 w = *reinterpret_cast<const float4*>(ksc + (J * 16 + j0) * LD + d);
+          s[J] += u.x * w.x + u.y * w.y + u.z * w.z + u.w * w.w;
+        }
+      }
+    }
+#pragma unroll
+    for (int J = 0; J < 3; ++J)
+      if (J < I) put(I * 16 + i0, J * 16 + j0, s[J]);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ carry
+// grid (dv / 16, H, B), 256 threads: warp (rg, half) = (w & 3, w >> 2) forms rows 16 rg .. of the token-by-column tiles, columns 8 half ..;
+// warp w holds state rows 16 w .. 16 w + 15.
+template <bool DELTA>
+__global__ void __launch_bounds__(256) chunk_carry_kernel(ChunkArgs a, const bf16* __restrict__ x, long ldx, long koff, long voff,
+                                                          const bf16* __restrict__ tiles, const bf16* __restrict__ qkg, const float* __restrict__ gates,
+                                                          const float* __restrict__ ends, bf16* __restrict__ o) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rg = warp & 3, half = warp >> 2;
+  const int dk = a.dk, dv = a.dv, H = a.H, LD = dk + 8, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * CN, kh = h / a.r;
+  const int n = real_tokens(a, b), chunks = (n - a.t_lo + CH - 1) / CH;
+  constexpr int NQK = DELTA ? 2 : 4, NTP = DELTA ? 4 : 2;
+  // one stage: q / k tiles, v tile, 64 x 64 tiles, gates
+  const size_t st_qk = (size_t)CH * LD, st_v = (size_t)CH * NLD, st_tp = (size_t)CH * CLD;
+  const size_t stage = (NQK * st_qk + st_v + NTP * st_tp) * 2 + 4 * CH * 4;
+  auto qkt = [&](int buf, int i) { return reinterpret_cast<bf16*>(raw + buf * stage) + i * st_qk; };
+  auto vt = [&](int buf) { return reinterpret_cast<bf16*>(raw + buf * stage) + NQK * st_qk; };
+  auto tpt = [&](int buf, int i) { return reinterpret_cast<bf16*>(raw + buf * stage) + NQK * st_qk + st_v + i * st_tp; };
+  auto gt = [&](int buf) { return reinterpret_cast<float*>(raw + buf * stage + (NQK * st_qk + st_v + NTP * st_tp) * 2); };
+  bf16* Sh = reinterpret_cast<bf16*>(raw + 2 * stage);   // [dk][NLD] high, low
+  bf16* Sl = Sh + dk * NLD;
+  bf16* W = Sl + dk * NLD;                               // gated delta: R high, low, U high, low, decayed U high, low: [64][NLD] each
+
+  auto issue = [&](int c, int buf) {
+    const int t0 = a.t_lo + c * CH, m = min(CH, n - t0);
+    const long id = chunk_id(a, b, c, h);
+    const bf16* row0 = x + ((long)b * a.S + t0) * ldx;
+    if constexpr (DELTA) {
+      tile_async(qkt(buf, 0), LD, row0 + (long)kh * dk, ldx, dk, m, tid, 256);
+      tile_async(qkt(buf, 1), LD, row0 + koff + (long)kh * dk, ldx, dk, m, tid, 256);
+    } else {
+      for (int i = 0; i < 4; ++i) tile_async(qkt(buf, i), LD, qkg + (id * 4 + i) * CH * dk, dk, dk, CH, tid, 256);
+    }
+    tile_async(vt(buf), NLD, row0 + voff + (long)h * dv + c0, ldx, CN, m, tid, 256);
+    for (int i = 0; i < NTP; ++i) tile_async(tpt(buf, i), CLD, tiles + (id * NTP + i) * CH * CH, CH, CH, CH, tid, 256);
+    const float* g = DELTA ? gates + id * 4 * CH : ends + id * dk;
+    for (int i = tid; i < (DELTA ? CH : dk / 4); i += 256) la_cp_async16(gt(buf) + i * 4, g + i * 4, 16);
+    la_commit();
+  };
+
+  const long slot = a.slots[b];
+  const bool fresh = a.lengths[b] == 0 && a.t_lo == 0;
+  float* sp = a.rec + (slot * H + h) * (long)dk * dv + c0;
+  const bool owns = warp * 16 < dk;                      // warps past the key width hold no state rows
+  float S[2][4];
+  const int gr = lane >> 2, kc = (lane & 3) * 2;
+#pragma unroll
+  for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      S[nt][e] = (!fresh && owns) ? sp[(long)(warp * 16 + gr + (e >> 1) * 8) * dv + nt * 8 + kc + (e & 1)] : 0.f;
+  auto publish = [&]() {
+    if (!owns) return;
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        const int at = (warp * 16 + gr + (e >> 1) * 8) * NLD + nt * 8 + kc;
+        la_split2(S[nt][e], S[nt][e + 1], *reinterpret_cast<__nv_bfloat162*>(Sh + at), *reinterpret_cast<__nv_bfloat162*>(Sl + at));
+      }
+  };
+  publish();
+  if (chunks > 0) issue(0, 0);
+  for (int c = 0; c < chunks; ++c) {
+    const int buf = c & 1, t0 = a.t_lo + c * CH;
+    la_wait<0>();
+    __syncthreads();                                     // this chunk's tiles and S are visible; the other stage is free
+    if (c + 1 < chunks) issue(c + 1, buf ^ 1);
+    const float* g = gt(buf);
+    const int arow = rg * 16 + (lane & 15), acol = (lane >> 4) * 8, brow = lane & 15;
+    const int i0 = rg * 16 + gr;                         // this thread's rows of a token tile: i0, i0 + 8
+    float y[4] = {0.f, 0.f, 0.f, 0.f};
+    if constexpr (DELTA) {
+      float xx[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int k = 0; k < dk; k += 16) {
+        unsigned fq[4], fk[4], sh[2], sl[2];
+        la_ldm4(fq, qkt(buf, 0) + arow * LD + k + acol);
+        la_ldm4(fk, qkt(buf, 1) + arow * LD + k + acol);
+        la_ldm2t(sh, Sh + (k + brow) * NLD + half * 8);
+        la_ldm2t(sl, Sl + (k + brow) * NLD + half * 8);
+        la_mma(xx, fk, sl[0], sl[1]);
+        la_mma(y, fq, sl[0], sl[1]);
+        la_mma(xx, fk, sh[0], sh[1]);
+        la_mma(y, fq, sh[0], sh[1]);
+      }
+      const bf16* v = vt(buf);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int i = i0 + e * 8, at = i * NLD + half * 8 + kc;
+        const float2 vv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(v + at));
+        const float be = g[CH + i], ek = g[i];
+        la_split2(be * (vv.x - ek * xx[2 * e]), be * (vv.y - ek * xx[2 * e + 1]), *reinterpret_cast<__nv_bfloat162*>(W + at),
+                  *reinterpret_cast<__nv_bfloat162*>(W + CH * NLD + at));
+      }
+      __syncthreads();
+      float u[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int k = 0; k <= rg * 16; k += 16) {           // T is lower triangular
+        unsigned th[4], tl[4], rh[2], rl[2];
+        la_ldm4(th, tpt(buf, 0) + arow * CLD + k + acol);
+        la_ldm4(tl, tpt(buf, 1) + arow * CLD + k + acol);
+        la_ldm2t(rh, W + (k + brow) * NLD + half * 8);
+        la_ldm2t(rl, W + CH * NLD + (k + brow) * NLD + half * 8);
+        la_mma(u, tl, rh[0], rh[1]);
+        la_mma(u, th, rl[0], rl[1]);
+        la_mma(u, th, rh[0], rh[1]);
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int i = i0 + e * 8, at = i * NLD + half * 8 + kc;
+        const float kd = g[3 * CH + i];
+        la_split2(u[2 * e], u[2 * e + 1], *reinterpret_cast<__nv_bfloat162*>(W + 2 * CH * NLD + at),
+                  *reinterpret_cast<__nv_bfloat162*>(W + 3 * CH * NLD + at));
+        la_split2(kd * u[2 * e], kd * u[2 * e + 1], *reinterpret_cast<__nv_bfloat162*>(W + 4 * CH * NLD + at),
+                  *reinterpret_cast<__nv_bfloat162*>(W + 5 * CH * NLD + at));
+      }
+      __syncthreads();
+      y[0] *= g[2 * CH + i0]; y[1] *= g[2 * CH + i0]; y[2] *= g[2 * CH + i0 + 8]; y[3] *= g[2 * CH + i0 + 8];
+      for (int k = 0; k <= rg * 16; k += 16) {
+        unsigned ph[4], pl[4], uh[2], ul[2];
+        la_ldm4(ph, tpt(buf, 2) + arow * CLD + k + acol);
+        la_ldm4(pl, tpt(buf, 3) + arow * CLD + k + acol);
+        la_ldm2t(uh, W + 2 * CH * NLD + (k + brow) * NLD + half * 8);
+        la_ldm2t(ul, W + 3 * CH * NLD + (k + brow) * NLD + half * 8);
+        la_mma(y, pl, uh[0], uh[1]);
+        la_mma(y, ph, ul[0], ul[1]);
+        la_mma(y, ph, uh[0], uh[1]);
+      }
+      if (owns) {
+        const float ge = ends[chunk_id(a, b, c, h)];
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) S[nt][e] *= ge;
+#pragma unroll
+        for (int k = 0; k < CH; k += 16) {
+          unsigned fk[4], uh[4], ul[4];
+          la_ldm4t(fk, qkt(buf, 1) + (k + la_at_row(lane)) * LD + warp * 16 + la_at_col(lane));
+          la_ldm4t(uh, W + 4 * CH * NLD + (k + brow) * NLD + (lane >> 4) * 8);
+          la_ldm4t(ul, W + 5 * CH * NLD + (k + brow) * NLD + (lane >> 4) * 8);
+          la_mma(S[0], fk, ul[0], ul[1]);
+          la_mma(S[1], fk, ul[2], ul[3]);
+          la_mma(S[0], fk, uh[0], uh[1]);
+          la_mma(S[1], fk, uh[2], uh[3]);
+        }
+      }
+    } else {
+      for (int k = 0; k < dk; k += 16) {
+        unsigned qh[4], ql[4], sh[2], sl[2];
+        la_ldm4(qh, qkt(buf, 0) + arow * LD + k + acol);
+        la_ldm4(ql, qkt(buf, 1) + arow * LD + k + acol);
+        la_ldm2t(sh, Sh + (k + brow) * NLD + half * 8);
+        la_ldm2t(sl, Sl + (k + brow) * NLD + half * 8);
+        la_mma(y, ql, sh[0], sh[1]);
+        la_mma(y, qh, sl[0], sl[1]);
+        la_mma(y, qh, sh[0], sh[1]);
+      }
+      for (int k = 0; k <= rg * 16; k += 16) {           // A is lower triangular
+        unsigned fh[4], fl[4], fv[2];
+        la_ldm4(fh, tpt(buf, 0) + arow * CLD + k + acol);
+        la_ldm4(fl, tpt(buf, 1) + arow * CLD + k + acol);
+        la_ldm2t(fv, vt(buf) + (k + brow) * NLD + half * 8);
+        la_mma(y, fl, fv[0], fv[1]);
+        la_mma(y, fh, fv[0], fv[1]);
+      }
+      if (owns) {
+        const float e0 = g[warp * 16 + gr], e1 = g[warp * 16 + gr + 8];
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) { S[nt][0] *= e0; S[nt][1] *= e0; S[nt][2] *= e1; S[nt][3] *= e1; }
+#pragma unroll
+        for (int k = 0; k < CH; k += 16) {
+          unsigned kh_[4], kl[4], fv[4];
+          la_ldm4t(kh_, qkt(buf, 2) + (k + la_at_row(lane)) * LD + warp * 16 + la_at_col(lane));
+          la_ldm4t(kl, qkt(buf, 3) + (k + la_at_row(lane)) * LD + warp * 16 + la_at_col(lane));
+          la_ldm4t(fv, vt(buf) + (k + brow) * NLD + (lane >> 4) * 8);
+          la_mma(S[0], kl, fv[0], fv[1]);
+          la_mma(S[1], kl, fv[2], fv[3]);
+          la_mma(S[0], kh_, fv[0], fv[1]);
+          la_mma(S[1], kh_, fv[2], fv[3]);
+        }
+      }
+      __syncthreads();                                   // every warp has read S
+    }
+    publish();
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = t0 + i0 + e * 8;
+      if (t < n)
+        *reinterpret_cast<__nv_bfloat162*>(o + (((long)b * a.S + t) * H + h) * dv + c0 + half * 8 + kc) = __floats2bfloat162_rn(y[2 * e], y[2 * e + 1]);
+    }
+  }
+  if (owns) {
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sp[(long)(warp * 16 + gr + (e >> 1) * 8) * dv + nt * 8 + kc + (e & 1)] = S[nt][e];
+  }
+  for (int i = tid; i < (a.t_hi - max(n, a.t_lo)) * CN; i += 256)         // padding positions are read by the norm kernel: give them a value
+    o[(((long)b * a.S + max(n, a.t_lo) + i / CN) * H + h) * dv + c0 + i % CN] = __float2bfloat16_rn(0.f);
+}
+
+size_t carry_smem(int delta, int dk) {
+  const size_t nqk = delta ? 2 : 4, ntp = delta ? 4 : 2;
+  const size_t stage = (nqk * CH * (dk + 8) + (size_t)CH * NLD + ntp * CH * CLD) * 2 + 4 * CH * 4;
+  return 2 * stage + 2 * (2 * (size_t)dk * NLD + (delta ? 6 * CH * NLD : 0));
+}
+
+}  // namespace mt
+
+using namespace mt;
+
+// both halves of the layer fit the chunked kernels
+extern "C" int mt_chunk_supported(int dk, int dv) { return dk % 16 == 0 && dk >= 16 && dk <= 128 && dv % 16 == 0 && dv >= 16; }
+
+extern "C" int mt_delta_chunks(const void* mixed, long ldx, const void* ba, long ldb, const void* A_log, const void* dt_bias, int hk, int hv, int dk, int dv,
+                               int S, int t_lo, int t_hi, float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* tp,
+                               float* gates, float* ends, void* o, int B, cudaStream_t st) {
+  if (!mt_chunk_supported(dk, dv) || ldx % 8) return -1;
+  const ChunkArgs a{hv, hv / hk, dk, dv, S, t_lo, t_hi, (t_hi - t_lo + CH - 1) / CH, slots, lengths, new_lens, rec};
+  const size_t s1 = 2 * 2 * (size_t)CH * (dk + 8) + 4 * CH * 68, s2 = carry_smem(1, dk);
+  if (cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2;
+  if (cudaFuncSetAttribute(chunk_carry_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2) != cudaSuccess) return -2;
+  delta_chunk_prepare_kernel<<<dim3(a.chunks, hv, B), 128, s1, st>>>(a, (const bf16*)mixed, ldx, (const bf16*)ba, ldb, (const bf16*)A_log,
+                                                                    (const bf16*)dt_bias, (bf16*)tp, gates, ends);
+  chunk_carry_kernel<true><<<dim3(dv / CN, hv, B), 256, s2, st>>>(a, (const bf16*)mixed, ldx, (long)hk * dk, 2L * hk * dk, (const bf16*)tp, nullptr, gates,
+                                                                ends, (bf16*)o);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int mt_gla_chunks(const void* x, long ldx, const float* log_alpha, int H, int dk, int dv, int S, int t_lo, int t_hi, float* rec,
+                             const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* aa, void* qkg, float* ends, void* o, int B,
+                             cudaStream_t st) {
+  if (!mt_chunk_supported(dk, dv) || ldx % 8) return -1;
+  const ChunkArgs a{H, 1, dk, dv, S, t_lo, t_hi, (t_hi - t_lo + CH - 1) / CH, slots, lengths, new_lens, rec};
+  const size_t s1 = 4 * (size_t)(CH + 64) * (dk + 4) + 2 * 2 * (size_t)CH * (dk + 8), s2 = carry_smem(0, dk);
+  if (cudaFuncSetAttribute(gla_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2;
+  if (cudaFuncSetAttribute(chunk_carry_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2) != cudaSuccess) return -2;
+  gla_chunk_prepare_kernel<<<dim3(a.chunks, H, B), 256, s1, st>>>(a, (const bf16*)x, ldx, log_alpha, (bf16*)aa, (bf16*)qkg, ends);
+  chunk_carry_kernel<false><<<dim3(dv / CN, H, B), 256, s2, st>>>(a, (const bf16*)x, ldx, 0, 2L * H * dk, (const bf16*)aa, (const bf16*)qkg, nullptr, ends,
+                                                                (bf16*)o);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}

@@ -16,6 +16,14 @@ def kernels_ok(t: torch.Tensor) -> bool:
   return not torch.is_grad_enabled() and t.dtype in (torch.bfloat16, torch.float32) and backend.use_cuda_kernels(t)
 
 
+CHUNK_FROM = 24          # tokens from which the chunked kernels replace the token scan
+
+
+def chunked_ok(t: torch.Tensor, S: int, dk: int, dv: int) -> bool:
+  """bf16 prompts run chunk by chunk on the tensor cores; fp32, very short inputs and unusual head widths run the token scan."""
+  return t.dtype == torch.bfloat16 and S >= CHUNK_FROM and backend.ext().chunk_supported(dk, dv)
+
+
 def gated_head_norm(o, z, scale, eps):
   """Definition: o [.., H, Dv] RMS-normalised over Dv, times scale, times silu(z); fp32."""
   o = o.float()
@@ -40,8 +48,8 @@ def delta_forward(layer, qkvz, ba, st):
   mixed = torch.empty(N, layer.conv_dim, dtype=dt, device=dev)
   E.delta_conv(q2, w, layer.hk, layer.hv, layer.dk, layer.dv, S, st.conv, st.slot_ids, st.lengths, st.new_lens, mixed)
   o = torch.empty(N, layer.value_dim, dtype=dt, device=dev)
-  E.delta_scan(mixed, b2, layer.A_log.data, layer.dt_bias.data, layer.hk, layer.hv, layer.dk, layer.dv, S, st.rec, st.slot_ids, st.lengths,
-               st.new_lens, o)
+  scan = E.delta_chunks if chunked_ok(mixed, S, layer.dk, layer.dv) else E.delta_scan
+  scan(mixed, b2, layer.A_log.data, layer.dt_bias.data, layer.hk, layer.hv, layer.dk, layer.dv, S, st.rec, st.slot_ids, st.lengths, st.new_lens, o)
   r = layer.r
   E.gated_head_norm(o, q2, layer.hv, layer.dv, r, 2 * layer.dk + r * layer.dv, 2 * layer.dk + 2 * r * layer.dv, layer.norm.data, eps,
                     out.view(N, -1))
@@ -64,6 +72,7 @@ def gla_forward(layer, p, st):
   log_alpha = torch.empty(N, H * dk, dtype=torch.float32, device=p.device)
   E.gla_decay(p2, 2 * H * (dk + dv), layer.decay.data, layer.decay_bias.data, layer.tau, log_alpha)
   o = torch.empty(N, H * dv, dtype=p.dtype, device=p.device)
-  E.gla_scan(p2, log_alpha, H, dk, dv, S, st.rec, st.slot_ids, st.lengths, st.new_lens, o)
+  scan = E.gla_chunks if chunked_ok(p2, S, dk, dv) else E.gla_scan
+  scan(p2, log_alpha, H, dk, dv, S, st.rec, st.slot_ids, st.lengths, st.new_lens, o)
   E.gated_head_norm(o, p2, H, dv, 1, 2 * H * dk + H * dv, dv, layer.norm.data, eps, out.view(N, -1))
   return out

@@ -85,13 +85,15 @@ SCAN_CASES = [(2, 150, 2, 1, 128, 128, None), (1, 300, 1, 2, 64, 128, None), (3,
 def test_delta_scan(B, S, hk, r, dk, dv, lens):
   from maxtext_b200.ops import backend
   E = backend.ext(required=True)
-  for dtype, tol in ((torch.float32, 2e-5), (torch.bfloat16, 1e-2)):
+  for dtype, scan, tol in ((torch.float32, E.delta_scan, 2e-5), (torch.bfloat16, E.delta_scan, 1e-2), (torch.bfloat16, E.delta_chunks, 1e-2)):
+    if scan is E.delta_chunks and not E.chunk_supported(dk, dv):
+      continue
     args = _delta_inputs(B, S, hk, r, dk, dv, dtype)
     rec = torch.full((B + 1, hk * r, dk, dv), 7.0, device="cuda")             # row 0 unused, dirty states elsewhere
     slots, lengths = torch.arange(B, device="cuda") + 1, torch.zeros(B, dtype=torch.long, device="cuda")
     n = torch.tensor(lens, device="cuda") if lens else None
     o = torch.empty(B * S, hk * r * dv, dtype=dtype, device="cuda")
-    E.delta_scan(*args, hk, hk * r, dk, dv, S, rec, slots, lengths, n, o)
+    scan(*args, hk, hk * r, dk, dv, S, rec, slots, lengths, n, o)
     for b in range(B):
       m = lens[b] if lens else S
       want = _delta_want(*args, B, S, hk, r, dk, dv, b, m)
@@ -107,7 +109,7 @@ def test_delta_scan(B, S, hk, r, dk, dv, lens):
       outs = []
       for lo, hi, done in ((0, half, 0), (half, S, half)):
         oo = torch.empty(B * (hi - lo), hk * r * dv, dtype=dtype, device="cuda")
-        E.delta_scan(*[t[:, lo:hi].reshape(B * (hi - lo), -1).contiguous() for t in cut], *args[2:], hk, hk * r, dk, dv, hi - lo, rec2, slots,
+        scan(*[t[:, lo:hi].reshape(B * (hi - lo), -1).contiguous() for t in cut], *args[2:], hk, hk * r, dk, dv, hi - lo, rec2, slots,
                      torch.full_like(lengths, done), None, oo)
         outs.append(oo.view(B, hi - lo, -1))
       both = torch.cat(outs, 1).view(B * S, -1)
@@ -127,12 +129,14 @@ def test_gla_scan(B, S, H, dk, dv, lens, decay):
   x = torch.randn(B * S, ld, generator=g)
   z = torch.rand(B * S, H * dk, generator=g)
   la = {"slow": -0.01 * z, "fast": -30.0 * z, "mixed": -10.0 ** (4 * z - 3)}[decay].cuda()
-  for dtype, tol in ((torch.float32, 2e-5), (torch.bfloat16, 1e-2)):
+  for dtype, scan, tol in ((torch.float32, E.gla_scan, 2e-5), (torch.bfloat16, E.gla_scan, 1e-2), (torch.bfloat16, E.gla_chunks, 1e-2)):
+    if scan is E.gla_chunks and not E.chunk_supported(dk, dv):
+      continue
     xd = x.to(dtype).cuda()
     rec = torch.full((B, H, dk, dv), 3.0, device="cuda")
     slots, lengths = torch.arange(B, device="cuda"), torch.zeros(B, dtype=torch.long, device="cuda")
     o = torch.empty(B * S, H * dv, dtype=dtype, device="cuda")
-    E.gla_scan(xd, la, H, dk, dv, S, rec, slots, lengths, torch.tensor(lens, device="cuda") if lens else None, o)
+    scan(xd, la, H, dk, dv, S, rec, slots, lengths, torch.tensor(lens, device="cuda") if lens else None, o)
     for b in range(B):
       n = lens[b] if lens else S
       xb = xd.double().cpu().view(B, S, -1)[b, :n]
