@@ -131,7 +131,7 @@ void gla_decode(const Tensor& x, const Tensor& w, const Tensor& bias, const Tens
                 Tensor& rec, const Tensor& slots, const Tensor& lengths, Tensor& out) {
   const bool f = f32(x);
   const int64_t B = x.size(0);
-  TORCH_CHECK(w.dim() == 2 && w.size(0) == H * dk);
+  TORCH_CHECK(w.dim() == 2 && w.size(0) == H * dk && w.size(1) % 8 == 0, "gla_decode: the rank is padded to a multiple of 8");
   rows2d(x, x, B, 2 * H * (dk + dv) + w.size(1), "packed projection");
   same(w, x, H * dk * w.size(1), "decay projection"); same(bias, x, H * dk, "decay bias"); same(norm, x, dv, "norm"); same(out, x, B * H * dv, "out");
   float* rp = state(rec, {H, dk, dv}, "rec");

@@ -31,7 +31,29 @@ __device__ __forceinline__ float rotated(const T* x, const float* cs, int e, int
 }
 
 // ------------------------------------------------------------------------------------------------ projection epilogue
-template <typename T>
+// rms norm of p [n] times w, VEC elements per access; the result also goes to `also` when that is not null
+template <typename T, int VEC>
+__device__ __forceinline__ void norm_row(const T* __restrict__ p, const T* __restrict__ w, int n, float eps, float* red, T* __restrict__ y, T* __restrict__ also) {
+  float ss = 0.f;
+  for (int i = threadIdx.x * VEC; i < n; i += blockDim.x * VEC) {
+    float v[VEC];
+    load_vec<VEC>(p + i, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
+  }
+  const float rstd = rsqrtf(block_add(ss, red) / (float)n + eps);
+  for (int i = threadIdx.x * VEC; i < n; i += blockDim.x * VEC) {
+    float v[VEC], g[VEC];
+    load_vec<VEC>(p + i, v);
+    load_vec<VEC>(w + i, g);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = v[e] * rstd * g[e];
+    store_vec<VEC>(y + i, v);
+    if (also) store_vec<VEC>(also + i, v);
+  }
+}
+
+template <typename T, int VEC>
 __global__ void __launch_bounds__(128) mla_prep_kernel(const T* __restrict__ qa, long ldq, const T* __restrict__ qw, int Q, const T* __restrict__ kva,
                                                        long ldk, const T* __restrict__ kw, int R, int dr, float eps, const int64_t* __restrict__ pos,
                                                        const float* __restrict__ inv_ts, int interleaved, int S, T* __restrict__ cq, T* __restrict__ lat,
@@ -43,25 +65,12 @@ __global__ void __launch_bounds__(128) mla_prep_kernel(const T* __restrict__ qa,
   const long n = blockIdx.x;
   const int b = (int)(n / S), t = (int)(n % S);
   rotation_table(cs, pos[n], inv_ts, dr / 2);
-  if (qa) {
-    const T* p = qa + n * ldq;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < Q; i += blockDim.x) { const float v = to_f(p[i]); ss += v * v; }
-    const float rstd = rsqrtf(block_add(ss, red) / (float)Q + eps);
-    for (int i = threadIdx.x; i < Q; i += blockDim.x) cq[n * Q + i] = from_f<T>(to_f(p[i]) * rstd * to_f(qw[i]));
-  }
+  if (qa) norm_row<T, VEC>(qa + n * ldq, qw, Q, eps, red, cq + n * Q, (T*)nullptr);
   const T* p = kva + n * ldk;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < R; i += blockDim.x) { const float v = to_f(p[i]); ss += v * v; }
-  const float rstd = rsqrtf(block_add(ss, red) / (float)R + eps);       // its barriers also publish the rotation table
   const long at = lengths[b] + t;
   const bool real = (!new_lens || t < new_lens[b]) && at < max_len;
   const long row = slots[b] * max_len + at;
-  for (int i = threadIdx.x; i < R; i += blockDim.x) {
-    const T v = from_f<T>(to_f(p[i]) * rstd * to_f(kw[i]));
-    lat[n * R + i] = v;
-    if (real) cache_lat[row * R + i] = v;
-  }
+  norm_row<T, VEC>(p, kw, R, eps, red, lat + n * R, real ? cache_lat + row * R : (T*)nullptr);       // its barriers also publish the rotation table
   for (int e = threadIdx.x; e < dr; e += blockDim.x) {
     const T v = from_f<T>(rotated(p + R, cs, e, dr / 2, interleaved));
     kr[n * dr + e] = v;
@@ -79,10 +88,30 @@ __global__ void __launch_bounds__(256) mla_pack_q_kernel(const T* __restrict__ q
   rotation_table(cs, pos[n], inv_ts, dr / 2);
   __syncthreads();
   const int qk = nope + dr, C = DQ / 8;
+  const bool vec = interleaved && nope % 8 == 0 && dr % 8 == 0;
   for (int i = threadIdx.x; i < H * C; i += blockDim.x) {
     const int h = i / C, e0 = (i % C) * 8;
     const T* x = q + (n * H + h) * qk;
     float v[8];
+    if (vec) {
+      if (e0 < qk) {
+        load_vec<8>(x + e0, v);
+        if (e0 >= nope) {
+          const float* t = cs + (e0 - nope);             // (cos, sin) of four pairs
+#pragma unroll
+          for (int j = 0; j < 8; j += 2) {
+            const float u = v[j], w = v[j + 1];
+            v[j] = u * t[j] - w * t[j + 1];
+            v[j + 1] = w * t[j] + u * t[j + 1];
+          }
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = 0.f;
+      }
+      store_vec<8>(qp + (n * H + h) * DQ + e0, v);
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const int e = e0 + j;
@@ -283,12 +312,14 @@ __global__ void __launch_bounds__(TC_NT) mla_attn_tc_kernel(AttnArgs a, const __
   const long base = a.slots[b] * a.max_len;
   const int vec_row = D / 8, vec_lat = R / 8;
   auto issue = [&](int t0, int buf) {
-    for (int i = tid; i < TC_KEYS * vec_row; i += TC_NT) {
-      const int r = i / vec_row, v = i % vec_row;
+    for (int r = warp; r < TC_KEYS; r += TC_NT / 32) {
       const bool in = t0 + r < hi;
       const long row = base + (in ? t0 + r : lo);
-      const __nv_bfloat16* src = v < vec_lat ? lat + row * R + v * 8 : kr + row * a.dr + (v - vec_lat) * 8;
-      la_cp_async16(xs + ((long)buf * TC_KEYS + r) * LD + v * 8, src, in ? 16 : 0);          // rows past the end are zero-filled
+      __nv_bfloat16* dst = xs + ((long)buf * TC_KEYS + r) * LD;
+      const int bytes = in ? 16 : 0;                                                         // rows past the end are zero-filled
+#pragma unroll
+      for (int v = lane; v < CT * 8; v += 32) la_cp_async16(dst + v * 8, lat + row * R + v * 8, bytes);
+      for (int v = lane; v < vec_row - vec_lat; v += 32) la_cp_async16(dst + R + v * 8, kr + row * a.dr + v * 8, bytes);
     }
     la_commit();
   };
@@ -312,25 +343,42 @@ __global__ void __launch_bounds__(TC_NT) mla_attn_tc_kernel(AttnArgs a, const __
     __syncthreads();
     const __nv_bfloat16* xt = xs + (long)buf * TC_KEYS * LD;
     // scores of 8 keys: A = q (16 x 16 pieces), B = keys (8 rows); one ldmatrix.x4 of the keys covers two k-steps
-    float s[4] = {0.f, 0.f, 0.f, 0.f};
+    float sc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[i][e] = 0.f;
     const __nv_bfloat16* qrow = qs + (lane & 15) * LD + (lane >> 4) * 8;
     const __nv_bfloat16* krow = xt + (warp * 8 + (lane & 7)) * LD + (lane >> 3) * 8;
     int k = 0;
+#pragma unroll 2
+    for (; k + 64 <= D; k += 64) {
+      unsigned fa[4][4], fb[2][4];
+      la_ldm4(fb[0], krow + k);
+      la_ldm4(fb[1], krow + k + 32);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) la_ldm4(fa[i], qrow + k + 16 * i);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) la_mma(sc[i], fa[i], fb[i >> 1][2 * (i & 1)], fb[i >> 1][2 * (i & 1) + 1]);
+    }
     for (; k + 32 <= D; k += 32) {
       unsigned fa[4], fb[4];
       la_ldm4(fb, krow + k);
       la_ldm4(fa, qrow + k);
-      la_mma(s, fa, fb[0], fb[1]);
+      la_mma(sc[0], fa, fb[0], fb[1]);
       la_ldm4(fa, qrow + k + 16);
-      la_mma(s, fa, fb[2], fb[3]);
+      la_mma(sc[1], fa, fb[2], fb[3]);
     }
     if (k < D) {                                         // D is a multiple of 16: one k-step is left
       unsigned fa[4], fb[2];
       const unsigned p = (unsigned)__cvta_generic_to_shared(xt + (warp * 8 + (lane & 7)) * LD + k + ((lane >> 3) & 1) * 8);
       asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(fb[0]), "=r"(fb[1]) : "r"(p));
       la_ldm4(fa, qrow + k);
-      la_mma(s, fa, fb[0], fb[1]);
+      la_mma(sc[2], fa, fb[0], fb[1]);
     }
+    float s[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[e] = (sc[0][e] + sc[1][e]) + (sc[2][e] + sc[3][e]);
     const int key = t0 + warp * 8 + kc;
 #pragma unroll
     for (int e = 0; e < 4; ++e) s[e] = key + (e & 1) < hi ? s[e] * a.scale : -INFINITY;
@@ -470,6 +518,143 @@ __global__ void __launch_bounds__(256) mla_value_up_kernel(const float* __restri
   }
 }
 
+// ------------------------------------------------------------------------------------------------ decode: the two per-head products on tensor cores
+// bf16, batches of eight and more. Batch rows in the M position, 64 columns per CTA.
+constexpr int HB = 64;                                   // batch rows per absorb CTA
+constexpr int VB = 32;                                   // batch rows per value CTA
+
+// grid (H, R / 64, ceil(B / 64)), 128 threads; warp w: columns 16 w .. 16 w + 15, four row tiles
+__global__ void __launch_bounds__(128) mla_absorb_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ w,
+                                                            const int64_t* __restrict__ pos, const float* __restrict__ inv_ts, int interleaved, int B, int H,
+                                                            int nope, int dr, int vd, int R, __nv_bfloat16* __restrict__ qa) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int h = blockIdx.x, j0 = blockIdx.y * 64, b0 = blockIdx.z * HB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int qk = nope + dr, QL = nope + 8, nb = min(HB, B - b0);
+  __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(raw);                     // [nope][72]
+  __nv_bfloat16* qs = ws + nope * 72;                                            // [64][QL]
+  const __nv_bfloat16* wb = w + (long)h * (nope + vd) * R + j0;
+  for (int i = tid; i < nope * 8; i += 128) la_cp_async16(ws + (i >> 3) * 72 + (i & 7) * 8, wb + (long)(i >> 3) * R + (i & 7) * 8, 16);
+  for (int r = warp; r < HB; r += 4)
+    for (int v = lane; v < nope / 8; v += 32)
+      la_cp_async16(qs + r * QL + v * 8, q + ((long)(b0 + (r < nb ? r : 0)) * H + h) * qk + v * 8, r < nb ? 16 : 0);
+  la_commit();
+  if (blockIdx.y == 0) {                                 // the rotated part, while the copies run
+    const int half = dr / 2;
+    for (int i = tid; i < nb * half; i += 128) {
+      const int r = i / half, p = i % half;
+      float s, c;
+      sincosf((float)pos[b0 + r] * inv_ts[p], &s, &c);
+      const __nv_bfloat16* x = q + ((long)(b0 + r) * H + h) * qk + nope;
+      __nv_bfloat16* y = qa + ((long)(b0 + r) * H + h) * (R + dr) + R;
+      const int iu = interleaved ? 2 * p : p, iv = interleaved ? 2 * p + 1 : p + half;
+      const float u = to_f(x[iu]), v = to_f(x[iv]);
+      y[iu] = __float2bfloat16_rn(u * c - v * s);
+      y[iv] = __float2bfloat16_rn(v * c + u * s);
+    }
+  }
+  float acc[4][2][4];
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[m][n][e] = 0.f;
+  la_wait<0>();
+  __syncthreads();
+#pragma unroll 2
+  for (int k = 0; k < nope; k += 16) {
+    unsigned fb[4];
+    la_ldm4t(fb, ws + (k + (lane & 15)) * 72 + warp * 16 + (lane >> 4) * 8);
+#pragma unroll
+    for (int m = 0; m < 4; ++m) {
+      if (m * 16 < nb) {
+        unsigned fa[4];
+        la_ldm4(fa, qs + (m * 16 + (lane & 15)) * QL + k + (lane >> 4) * 8);
+        la_mma(acc[m][0], fa, fb[0], fb[1]);
+        la_mma(acc[m][1], fa, fb[2], fb[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+#pragma unroll
+    for (int e = 0; e < 4; e += 2) {
+      const int r = m * 16 + (lane >> 2) + (e ? 8 : 0);
+      if (r < nb) {
+        __nv_bfloat16* y = qa + ((long)(b0 + r) * H + h) * (R + dr) + j0 + warp * 16 + (lane & 3) * 2;
+        *reinterpret_cast<__nv_bfloat162*>(y) = __floats2bfloat162_rn(acc[m][0][e], acc[m][0][e + 1]);
+        *reinterpret_cast<__nv_bfloat162*>(y + 8) = __floats2bfloat162_rn(acc[m][1][e], acc[m][1][e + 1]);
+      }
+    }
+}
+
+// grid (H, ceil(vd / 64), ceil(B / 32)), 256 threads; warp: columns 16 (w & 3) .., row tile w >> 2. The merged latent sums enter as bf16 pairs.
+__global__ void __launch_bounds__(256) mla_value_up_tc_kernel(const float* __restrict__ part, const float* __restrict__ ml, const __nv_bfloat16* __restrict__ w,
+                                                              int B, int H, int nope, int vd, int R, int splits, __nv_bfloat16* __restrict__ out) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  __shared__ float wt[VB][64];
+  const int h = blockIdx.x, e0 = blockIdx.y * 64, b0 = blockIdx.z * VB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int LD = R + 8, nb = min(VB, B - b0), ne = min(64, vd - e0);
+  __nv_bfloat16* ws = reinterpret_cast<__nv_bfloat16*>(raw);                     // [64][LD]
+  __nv_bfloat16* ch = ws + 64 * LD;                                              // [32][LD] high, low
+  __nv_bfloat16* cl = ch + VB * LD;
+  const __nv_bfloat16* wb = w + ((long)h * (nope + vd) + nope + e0) * R;
+  for (int r = warp; r < 64; r += 8)
+    for (int v = lane; v < R / 8; v += 32) la_cp_async16(ws + r * LD + v * 8, wb + (long)(r < ne ? r : 0) * R + v * 8, r < ne ? 16 : 0);
+  la_commit();
+  if (tid < nb) {
+    const float* p = ml + ((long)(b0 + tid) * H + h) * splits * 2;
+    float m = -INFINITY, den = 0.f;
+    for (int s = 0; s < splits; ++s) m = fmaxf(m, p[2 * s]);
+    for (int s = 0; s < splits; ++s) den += p[2 * s + 1] > 0.f ? p[2 * s + 1] * expf(p[2 * s] - m) : 0.f;
+    for (int s = 0; s < splits; ++s) wt[tid][s] = p[2 * s + 1] > 0.f ? expf(p[2 * s] - m) / den : 0.f;
+  }
+  __syncthreads();
+  for (int r = warp; r < VB; r += 8) {
+    const float* p = part + ((long)(b0 + (r < nb ? r : 0)) * H + h) * splits * R;
+    for (int j = lane * 4; j < R; j += 128) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < nb)
+        for (int s = 0; s < splits; ++s) {
+          const float f = wt[r][s];
+          if (f > 0.f) {
+            const float4 x = *reinterpret_cast<const float4*>(p + (long)s * R + j);
+            v.x += f * x.x; v.y += f * x.y; v.z += f * x.z; v.w += f * x.w;
+          }
+        }
+      __nv_bfloat162 hi, lo;
+      la_split2(v.x, v.y, hi, lo);
+      *reinterpret_cast<__nv_bfloat162*>(ch + r * LD + j) = hi;
+      *reinterpret_cast<__nv_bfloat162*>(cl + r * LD + j) = lo;
+      la_split2(v.z, v.w, hi, lo);
+      *reinterpret_cast<__nv_bfloat162*>(ch + r * LD + j + 2) = hi;
+      *reinterpret_cast<__nv_bfloat162*>(cl + r * LD + j + 2) = lo;
+    }
+  }
+  la_wait<0>();
+  __syncthreads();
+  const int n0 = (warp & 3) * 16, m0 = (warp >> 2) * 16;
+  float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}}, low[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll 4
+  for (int k = 0; k < R; k += 16) {
+    unsigned fb[4], fh[4], fl[4];
+    la_ldm4(fb, ws + (n0 + (lane & 7) + ((lane >> 4) << 3)) * LD + k + ((lane >> 3) & 1) * 8);
+    la_ldm4(fh, ch + (m0 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+    la_ldm4(fl, cl + (m0 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+    la_mma(acc[0], fh, fb[0], fb[1]);
+    la_mma(acc[1], fh, fb[2], fb[3]);
+    la_mma(low[0], fl, fb[0], fb[1]);
+    la_mma(low[1], fl, fb[2], fb[3]);
+  }
+#pragma unroll
+  for (int n = 0; n < 2; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = m0 + (lane >> 2) + (e >> 1) * 8, c = n0 + n * 8 + (lane & 3) * 2 + (e & 1);
+      if (r < nb && c < ne) out[((long)(b0 + r) * H + h) * vd + e0 + c] = __float2bfloat16_rn(acc[n][e] + low[n][e]);
+    }
+}
+
 template <typename K>
 int raise_smem(K k, size_t smem) {
   if (smem > 227 * 1024) return -1;
@@ -493,10 +678,12 @@ extern "C" int mt_mla_prep(int f32, const void* qa, long ldq, const void* qw, in
                            long max_len, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, long N, cudaStream_t st) {
   if (N <= 0) return 0;
   const size_t smem = sizeof(float) * dr;
-#define CALL(T) mla_prep_kernel<T><<<(unsigned)N, 128, smem, st>>>((const T*)qa, ldq, (const T*)qw, Q, (const T*)kva, ldk, (const T*)kw, R, dr, eps, pos, \
-                                                                   inv_ts, interleaved, S, (T*)cq, (T*)lat, (T*)kr, (T*)cache_lat, (T*)cache_kr, max_len, \
-                                                                   slots, lengths, new_lens)
-  if (f32) CALL(float); else CALL(bf16);
+  const bool v4 = Q % 4 == 0 && R % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0;
+#define CALL(T, V) mla_prep_kernel<T, V><<<(unsigned)N, 128, smem, st>>>((const T*)qa, ldq, (const T*)qw, Q, (const T*)kva, ldk, (const T*)kw, R, dr, eps, pos, \
+                                                                        inv_ts, interleaved, S, (T*)cq, (T*)lat, (T*)kr, (T*)cache_lat, (T*)cache_kr, \
+                                                                        max_len, slots, lengths, new_lens)
+  if (f32) { if (v4) CALL(float, 4); else CALL(float, 1); }
+  else { if (v4) CALL(bf16, 4); else CALL(bf16, 1); }
 #undef CALL
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
@@ -515,6 +702,13 @@ extern "C" int mt_mla_pack(const void* q, const void* kv, const void* kr, const 
 extern "C" int mt_mla_absorb(int f32, const void* q, const void* w, const int64_t* pos, const float* inv_ts, int interleaved, int B, int H, int nope, int dr,
                              int vd, int R, void* qa, cudaStream_t st) {
   if (B <= 0) return 0;
+  if (!f32 && B >= 8 && R % 64 == 0 && nope % 16 == 0 && dr % 8 == 0 && nope <= 512) {
+    const size_t smem = 2 * ((size_t)nope * 72 + HB * (nope + 8));
+    if (int rc = raise_smem(mla_absorb_tc_kernel, smem)) return rc;
+    mla_absorb_tc_kernel<<<dim3(H, R / 64, (B + HB - 1) / HB), 128, smem, st>>>((const bf16*)q, (const bf16*)w, pos, inv_ts, interleaved, B, H, nope, dr, vd, R,
+                                                                             (bf16*)qa);
+    return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  }
   const size_t smem = sizeof(float) * (8 * AB_BT * 256 + dr);
   const dim3 grid(H, (B + AB_BT - 1) / AB_BT, (R + 255) / 256);
 #define GO(T, AL) { if (int rc = raise_smem(mla_absorb_kernel<T, AL>, smem)) return rc; \
@@ -556,6 +750,12 @@ extern "C" int mt_mla_value_up(int f32, const float* part, const float* ml, cons
                                cudaStream_t st) {
   if (B <= 0) return 0;
   if (splits < 1 || splits > 64) return -1;
+  if (!f32 && B >= 8 && R % 16 == 0 && R <= 512) {
+    const size_t tc = 2 * (size_t)(64 + 2 * VB) * (R + 8);
+    if (int rc = raise_smem(mla_value_up_tc_kernel, tc)) return rc;
+    mla_value_up_tc_kernel<<<dim3(H, (vd + 63) / 64, (B + VB - 1) / VB), 256, tc, st>>>(part, ml, (const bf16*)w, B, H, nope, vd, R, splits, (bf16*)out);
+    return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  }
   const size_t smem = sizeof(float) * AB_BT * (size_t)((R + 3) & ~3);
   const dim3 grid(H, (B + AB_BT - 1) / AB_BT, (vd + 63) / 64);
 #define GO(T, AL) { if (int rc = raise_smem(mla_value_up_kernel<T, AL>, smem)) return rc; \

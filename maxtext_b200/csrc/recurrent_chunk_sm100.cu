@@ -5,8 +5,8 @@
 //      gated delta: with G_i the log-decay summed from the chunk's start, r the inverse norms of q and k,
 //        L_ij = beta_i rk_i rk_j (k_i . k_j) e^(G_i - G_j)  (j < i),   T = (I + L)^-1,   P_ij = rq_i rk_j (q_i . k_j) e^(G_i - G_j)  (j <= i)
 //      gated linear attention: G per key channel;  A_ij = sum_d q_id k_jd e^(G_id - G_jd)  (j <= i),  q e^G,  k e^(G_end - G).
-//        Exponents are formed so that none is positive: 16 x 16 blocks below the diagonal are split at the first row of their block row,
-//        diagonal blocks are summed with their own exponent per term.
+//        Exponents are split at the token before each block row of 16, so that no factor below the diagonal exceeds one; a diagonal block uses the
+//        same split while its decay is at most 2^60, and otherwise sums its terms with their own exponents.
 //  * carry, one CTA per (16 state columns, head, sequence), chunk after chunk with the state in fp32 registers and the next chunk's tiles in flight:
 //      gated delta:  X = K S, Y = Q S;  R = beta (V - rk e^G X);  U = T R;  O = rq e^G Y + P U;  S <- e^G_end S + K^T (rk e^(G_end - G) U)
 //      linear:       O = (q e^G) S + A V;  S <- diag(e^G_end) S + (k e^(G_end - G))^T V
@@ -194,8 +194,8 @@ __global__ void __launch_bounds__(256) gla_chunk_prepare_kernel(ChunkArgs a, con
   const int m = min(CH, real_tokens(a, b) - t0);
   if (m <= 0) return;
   float* G = sm;                                         // [64][LD]
-  float* ksc = G + CH * LD;                              // [48][LD] scaled keys of the blocks left of the diagonal
-  float* qsc = ksc + 48 * LD;                            // [16][LD]
+  float* ksc = G + CH * LD;                              // [64][LD] scaled keys up to the diagonal block
+  float* qsc = ksc + CH * LD;                            // [16][LD]
   bf16* q = reinterpret_cast<bf16*>(qsc + 16 * LD);      // [64][dk + 8]
   bf16* k = q + CH * (dk + 8);
   const int QLD = dk + 8;
@@ -208,7 +208,7 @@ __global__ void __launch_bounds__(256) gla_chunk_prepare_kernel(ChunkArgs a, con
     float g = 0.f;
 #pragma unroll 8
     for (int i = 0; i < CH; ++i) {
-      if (i < m) g += la[(long)i * H * dk];
+      if (i < m) g += la[(long)i * H * dk] * 1.4426950408889634f;         // base 2
       G[i * LD + tid] = g;
     }
   }
@@ -223,77 +223,80 @@ __global__ void __launch_bounds__(256) gla_chunk_prepare_kernel(ChunkArgs a, con
     const float2 kv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + t * QLD + d));
     const float g0 = G[t * LD + d], g1 = G[t * LD + d + 1], e0 = G[(CH - 1) * LD + d], e1 = G[(CH - 1) * LD + d + 1];
     __nv_bfloat162 hi, lo;
-    la_split2(qv.x * scale * expf(g0), qv.y * scale * expf(g1), hi, lo);
+    la_split2(qv.x * scale * exp2f(g0), qv.y * scale * exp2f(g1), hi, lo);
     *reinterpret_cast<__nv_bfloat162*>(qg + t * dk + d) = hi;
     *reinterpret_cast<__nv_bfloat162*>(qg + CH * dk + t * dk + d) = lo;
-    la_split2(kv.x * expf(e0 - g0), kv.y * expf(e1 - g1), hi, lo);
+    la_split2(kv.x * exp2f(e0 - g0), kv.y * exp2f(e1 - g1), hi, lo);
     *reinterpret_cast<__nv_bfloat162*>(qg + 2 * CH * dk + t * dk + d) = hi;
     *reinterpret_cast<__nv_bfloat162*>(qg + 3 * CH * dk + t * dk + d) = lo;
   }
-  if (tid < dk) end[id * dk + tid] = expf(G[(CH - 1) * LD + tid]);
+  if (tid < dk) end[id * dk + tid] = exp2f(G[(CH - 1) * LD + tid]);
   bf16* ah = aa + id * 2 * CH * CH;
   auto put = [&](int i, int j, float v) {
     const bf16 hi = __float2bfloat16_rn(v);
     ah[i * CH + j] = hi;
     ah[CH * CH + i * CH + j] = __float2bfloat16_rn(v - __bfloat162float(hi));
   };
-  // diagonal blocks: thread (i, j) of each 16 x 16 block, the exponent of every term on its own
-  {
-    const int i0 = tid >> 4, j0 = tid & 15;
-    for (int blk = 0; blk < 4; ++blk) {
-      const int i = blk * 16 + i0, j = blk * 16 + j0;
-      float s = 0.f;
-      if (j <= i)
-        for (int d = 0; d < dk; ++d) s += to_f(q[i * QLD + d]) * to_f(k[j * QLD + d]) * expf(G[i * LD + d] - G[j * LD + d]);
-      put(i, j, s * scale);
-    }
-  }
-  // blocks below the diagonal, block row by block row: exponents split at the last token before the block row
-  for (int I = 1; I < 4; ++I) {
-    const float* ref = G + (I * 16 - 1) * LD;
-    __syncthreads();
+  // block row by block row: exponents split at the last token before the block row, where no factor can overflow below the diagonal. The diagonal
+  // block joins in when its own decay is at most 2^60 in every channel; otherwise its terms are summed with their own exponents.
+  const int i0 = tid >> 4, j0 = tid & 15;
+  for (int I = 0; I < 4; ++I) {
+    const float* ref = G + (I * 16 - 1) * LD;            // not read for I = 0: nothing has decayed there
+    bool mild = true;
+    if (tid < dk) mild = (I ? ref[tid] : 0.f) - G[(I * 16 + 15) * LD + tid] <= 60.f;
+    mild = __syncthreads_and(mild);
     for (int i = tid; i < 16 * dk; i += 256) {
       const int t = i / dk, d = i % dk;
-      qsc[t * LD + d] = to_f(q[(I * 16 + t) * QLD + d]) * scale * expf(G[(I * 16 + t) * LD + d] - ref[d]);
+      qsc[t * LD + d] = to_f(q[(I * 16 + t) * QLD + d]) * scale * exp2f(G[(I * 16 + t) * LD + d] - (I ? ref[d] : 0.f));
     }
-    for (int i = tid; i < I * 16 * dk; i += 256) {
+    const int krows = mild ? I * 16 + 16 : I * 16;
+    for (int i = tid; i < krows * dk; i += 256) {
       const int t = i / dk, d = i % dk;
-      ksc[t * LD + d] = to_f(k[t * QLD + d]) * expf(ref[d] - G[t * LD + d]);
+      ksc[t * LD + d] = to_f(k[t * QLD + d]) * exp2f((I ? ref[d] : 0.f) - G[t * LD + d]);
     }
     __syncthreads();
-    const int i0 = tid >> 4, j0 = tid & 15;
-    float s[3] = {0.f, 0.f, 0.f};
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
     for (int d = 0; d < dk; d += 4) {
       const float4 u = *reinterpret_cast<const float4*>(qsc + i0 * LD + d);
 #pragma unroll
-      for (int J = 0; J < 3; ++J) {
-        if (J < I) {
+      for (int J = 0; J < 4; ++J) {
+        if (J * 16 < krows) {
           const float4 w = *reinterpret_cast<const float4*>(ksc + (J * 16 + j0) * LD + d);
           s[J] += u.x * w.x + u.y * w.y + u.z * w.z + u.w * w.w;
         }
       }
     }
+    if (!mild) {
+      const int i = I * 16 + i0, j = I * 16 + j0;
+      float t = 0.f;
+      if (j <= i)
+        for (int d = 0; d < dk; ++d) t += to_f(q[i * QLD + d]) * to_f(k[j * QLD + d]) * exp2f(G[i * LD + d] - G[j * LD + d]);
 #pragma unroll
-    for (int J = 0; J < 3; ++J)
-      if (J < I) put(I * 16 + i0, J * 16 + j0, s[J]);
+      for (int J = 0; J < 4; ++J)
+        if (J == I) s[J] = t * scale;
+    }
+#pragma unroll
+    for (int J = 0; J < 4; ++J)
+      if (J <= I) put(I * 16 + i0, J * 16 + j0, J == I && j0 > i0 ? 0.f : s[J]);
   }
 }
 
 // ------------------------------------------------------------------------------------------------ carry
 // grid (dv / 16, H, B), 256 threads: warp (rg, half) = (w & 3, w >> 2) forms rows 16 rg .. of the token-by-column tiles, columns 8 half ..;
 // warp w holds state rows 16 w .. 16 w + 15.
-template <bool DELTA>
+template <bool DELTA, int DK>
 __global__ void __launch_bounds__(256) chunk_carry_kernel(ChunkArgs a, const bf16* __restrict__ x, long ldx, long koff, long voff,
                                                           const bf16* __restrict__ tiles, const bf16* __restrict__ qkg, const float* __restrict__ gates,
                                                           const float* __restrict__ ends, bf16* __restrict__ o) {
   extern __shared__ __align__(16) unsigned char raw[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, rg = warp & 3, half = warp >> 2;
-  const int dk = a.dk, dv = a.dv, H = a.H, LD = dk + 8, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * CN, kh = h / a.r;
+  constexpr int dk = DK, LD = DK + 8;
+  const int dv = a.dv, H = a.H, h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * CN, kh = h / a.r;
   const int n = real_tokens(a, b), chunks = (n - a.t_lo + CH - 1) / CH;
   constexpr int NQK = DELTA ? 2 : 4, NTP = DELTA ? 4 : 2;
   // one stage: q / k tiles, v tile, 64 x 64 tiles, gates
-  const size_t st_qk = (size_t)CH * LD, st_v = (size_t)CH * NLD, st_tp = (size_t)CH * CLD;
-  const size_t stage = (NQK * st_qk + st_v + NTP * st_tp) * 2 + 4 * CH * 4;
+  constexpr size_t st_qk = (size_t)CH * LD, st_v = (size_t)CH * NLD, st_tp = (size_t)CH * CLD;
+  constexpr size_t stage = (NQK * st_qk + st_v + NTP * st_tp) * 2 + 4 * CH * 4;
   auto qkt = [&](int buf, int i) { return reinterpret_cast<bf16*>(raw + buf * stage) + i * st_qk; };
   auto vt = [&](int buf) { return reinterpret_cast<bf16*>(raw + buf * stage) + NQK * st_qk; };
   auto tpt = [&](int buf, int i) { return reinterpret_cast<bf16*>(raw + buf * stage) + NQK * st_qk + st_v + i * st_tp; };
@@ -352,18 +355,21 @@ __global__ void __launch_bounds__(256) chunk_carry_kernel(ChunkArgs a, const bf1
     const int i0 = rg * 16 + gr;                         // this thread's rows of a token tile: i0, i0 + 8
     float y[4] = {0.f, 0.f, 0.f, 0.f};
     if constexpr (DELTA) {
-      float xx[4] = {0.f, 0.f, 0.f, 0.f};
+      float xx[4] = {0.f, 0.f, 0.f, 0.f}, xl[4] = {0.f, 0.f, 0.f, 0.f}, yl[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
       for (int k = 0; k < dk; k += 16) {
         unsigned fq[4], fk[4], sh[2], sl[2];
         la_ldm4(fq, qkt(buf, 0) + arow * LD + k + acol);
         la_ldm4(fk, qkt(buf, 1) + arow * LD + k + acol);
         la_ldm2t(sh, Sh + (k + brow) * NLD + half * 8);
         la_ldm2t(sl, Sl + (k + brow) * NLD + half * 8);
-        la_mma(xx, fk, sl[0], sl[1]);
-        la_mma(y, fq, sl[0], sl[1]);
+        la_mma(xl, fk, sl[0], sl[1]);
+        la_mma(yl, fq, sl[0], sl[1]);
         la_mma(xx, fk, sh[0], sh[1]);
         la_mma(y, fq, sh[0], sh[1]);
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { xx[e] += xl[e]; y[e] += yl[e]; }
       const bf16* v = vt(buf);
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
@@ -374,17 +380,21 @@ __global__ void __launch_bounds__(256) chunk_carry_kernel(ChunkArgs a, const bf1
                   *reinterpret_cast<__nv_bfloat162*>(W + CH * NLD + at));
       }
       __syncthreads();
-      float u[4] = {0.f, 0.f, 0.f, 0.f};
-      for (int k = 0; k <= rg * 16; k += 16) {           // T is lower triangular
+      float u[4] = {0.f, 0.f, 0.f, 0.f}, u1[4] = {0.f, 0.f, 0.f, 0.f}, u2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int k = 0; k < CH; k += 16) {
+        if (k > rg * 16) break;                          // T is lower triangular
         unsigned th[4], tl[4], rh[2], rl[2];
         la_ldm4(th, tpt(buf, 0) + arow * CLD + k + acol);
         la_ldm4(tl, tpt(buf, 1) + arow * CLD + k + acol);
         la_ldm2t(rh, W + (k + brow) * NLD + half * 8);
         la_ldm2t(rl, W + CH * NLD + (k + brow) * NLD + half * 8);
-        la_mma(u, tl, rh[0], rh[1]);
-        la_mma(u, th, rl[0], rl[1]);
+        la_mma(u1, tl, rh[0], rh[1]);
+        la_mma(u2, th, rl[0], rl[1]);
         la_mma(u, th, rh[0], rh[1]);
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) u[e] += u1[e] + u2[e];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int i = i0 + e * 8, at = i * NLD + half * 8 + kc;
@@ -396,16 +406,21 @@ __global__ void __launch_bounds__(256) chunk_carry_kernel(ChunkArgs a, const bf1
       }
       __syncthreads();
       y[0] *= g[2 * CH + i0]; y[1] *= g[2 * CH + i0]; y[2] *= g[2 * CH + i0 + 8]; y[3] *= g[2 * CH + i0 + 8];
-      for (int k = 0; k <= rg * 16; k += 16) {
+      float y1[4] = {0.f, 0.f, 0.f, 0.f}, y2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int k = 0; k < CH; k += 16) {
+        if (k > rg * 16) break;
         unsigned ph[4], pl[4], uh[2], ul[2];
         la_ldm4(ph, tpt(buf, 2) + arow * CLD + k + acol);
         la_ldm4(pl, tpt(buf, 3) + arow * CLD + k + acol);
         la_ldm2t(uh, W + 2 * CH * NLD + (k + brow) * NLD + half * 8);
         la_ldm2t(ul, W + 3 * CH * NLD + (k + brow) * NLD + half * 8);
-        la_mma(y, pl, uh[0], uh[1]);
-        la_mma(y, ph, ul[0], ul[1]);
+        la_mma(y1, pl, uh[0], uh[1]);
+        la_mma(y2, ph, ul[0], ul[1]);
         la_mma(y, ph, uh[0], uh[1]);
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[e] += y1[e] + y2[e];
       if (owns) {
         const float ge = ends[chunk_id(a, b, c, h)];
 #pragma unroll
@@ -425,24 +440,30 @@ __global__ void __launch_bounds__(256) chunk_carry_kernel(ChunkArgs a, const bf1
         }
       }
     } else {
+      float y1[4] = {0.f, 0.f, 0.f, 0.f}, y2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
       for (int k = 0; k < dk; k += 16) {
         unsigned qh[4], ql[4], sh[2], sl[2];
         la_ldm4(qh, qkt(buf, 0) + arow * LD + k + acol);
         la_ldm4(ql, qkt(buf, 1) + arow * LD + k + acol);
         la_ldm2t(sh, Sh + (k + brow) * NLD + half * 8);
         la_ldm2t(sl, Sl + (k + brow) * NLD + half * 8);
-        la_mma(y, ql, sh[0], sh[1]);
-        la_mma(y, qh, sl[0], sl[1]);
+        la_mma(y1, ql, sh[0], sh[1]);
+        la_mma(y2, qh, sl[0], sl[1]);
         la_mma(y, qh, sh[0], sh[1]);
       }
-      for (int k = 0; k <= rg * 16; k += 16) {           // A is lower triangular
+#pragma unroll
+      for (int k = 0; k < CH; k += 16) {
+        if (k > rg * 16) break;                          // A is lower triangular
         unsigned fh[4], fl[4], fv[2];
         la_ldm4(fh, tpt(buf, 0) + arow * CLD + k + acol);
         la_ldm4(fl, tpt(buf, 1) + arow * CLD + k + acol);
         la_ldm2t(fv, vt(buf) + (k + brow) * NLD + half * 8);
-        la_mma(y, fl, fv[0], fv[1]);
-        la_mma(y, fh, fv[0], fv[1]);
+        la_mma(y1, fl, fv[0], fv[1]);
+        la_mma(y2, fh, fv[0], fv[1]);
       }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[e] += y1[e] + y2[e];
       if (owns) {
         const float e0 = g[warp * 16 + gr], e1 = g[warp * 16 + gr + 8];
 #pragma unroll
@@ -485,6 +506,26 @@ size_t carry_smem(int delta, int dk) {
   return 2 * stage + 2 * (2 * (size_t)dk * NLD + (delta ? 6 * CH * NLD : 0));
 }
 
+template <bool DELTA, int DK>
+int launch_carry_dk(const ChunkArgs& a, const bf16* x, long ldx, long koff, long voff, const bf16* tiles, const bf16* qkg, const float* gates,
+                    const float* ends, bf16* o, int B, cudaStream_t st) {
+  const size_t smem = carry_smem(DELTA, DK);
+  auto k = chunk_carry_kernel<DELTA, DK>;
+  if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return -2;
+  k<<<dim3(a.dv / CN, a.H, B), 256, smem, st>>>(a, x, ldx, koff, voff, tiles, qkg, gates, ends, o);
+  return 0;
+}
+template <bool DELTA>
+int launch_carry(const ChunkArgs& a, const bf16* x, long ldx, long koff, long voff, const bf16* tiles, const bf16* qkg, const float* gates,
+                 const float* ends, bf16* o, int B, cudaStream_t st) {
+  switch (a.dk) {
+#define GO(DK) case DK: return launch_carry_dk<DELTA, DK>(a, x, ldx, koff, voff, tiles, qkg, gates, ends, o, B, st);
+    GO(16) GO(32) GO(48) GO(64) GO(80) GO(96) GO(112) GO(128)
+#undef GO
+    default: return -1;
+  }
+}
+
 }  // namespace mt
 
 using namespace mt;
@@ -497,13 +538,11 @@ extern "C" int mt_delta_chunks(const void* mixed, long ldx, const void* ba, long
                                float* gates, float* ends, void* o, int B, cudaStream_t st) {
   if (!mt_chunk_supported(dk, dv) || ldx % 8) return -1;
   const ChunkArgs a{hv, hv / hk, dk, dv, S, t_lo, t_hi, (t_hi - t_lo + CH - 1) / CH, slots, lengths, new_lens, rec};
-  const size_t s1 = 2 * 2 * (size_t)CH * (dk + 8) + 4 * CH * 68, s2 = carry_smem(1, dk);
+  const size_t s1 = 2 * 2 * (size_t)CH * (dk + 8) + 4 * CH * 68;
   if (cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2;
-  if (cudaFuncSetAttribute(chunk_carry_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2) != cudaSuccess) return -2;
   delta_chunk_prepare_kernel<<<dim3(a.chunks, hv, B), 128, s1, st>>>(a, (const bf16*)mixed, ldx, (const bf16*)ba, ldb, (const bf16*)A_log,
                                                                     (const bf16*)dt_bias, (bf16*)tp, gates, ends);
-  chunk_carry_kernel<true><<<dim3(dv / CN, hv, B), 256, s2, st>>>(a, (const bf16*)mixed, ldx, (long)hk * dk, 2L * hk * dk, (const bf16*)tp, nullptr, gates,
-                                                                ends, (bf16*)o);
+  if (int rc = launch_carry<true>(a, (const bf16*)mixed, ldx, (long)hk * dk, 2L * hk * dk, (const bf16*)tp, nullptr, gates, ends, (bf16*)o, B, st)) return rc;
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -512,11 +551,9 @@ extern "C" int mt_gla_chunks(const void* x, long ldx, const float* log_alpha, in
                              cudaStream_t st) {
   if (!mt_chunk_supported(dk, dv) || ldx % 8) return -1;
   const ChunkArgs a{H, 1, dk, dv, S, t_lo, t_hi, (t_hi - t_lo + CH - 1) / CH, slots, lengths, new_lens, rec};
-  const size_t s1 = 4 * (size_t)(CH + 64) * (dk + 4) + 2 * 2 * (size_t)CH * (dk + 8), s2 = carry_smem(0, dk);
+  const size_t s1 = 4 * (size_t)(2 * CH + 16) * (dk + 4) + 2 * 2 * (size_t)CH * (dk + 8);
   if (cudaFuncSetAttribute(gla_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2;
-  if (cudaFuncSetAttribute(chunk_carry_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2) != cudaSuccess) return -2;
   gla_chunk_prepare_kernel<<<dim3(a.chunks, H, B), 256, s1, st>>>(a, (const bf16*)x, ldx, log_alpha, (bf16*)aa, (bf16*)qkg, ends);
-  chunk_carry_kernel<false><<<dim3(dv / CN, H, B), 256, s2, st>>>(a, (const bf16*)x, ldx, 0, 2L * H * dk, (const bf16*)aa, (const bf16*)qkg, nullptr, ends,
-                                                                (bf16*)o);
+  if (int rc = launch_carry<false>(a, (const bf16*)x, ldx, 0, 2L * H * dk, (const bf16*)aa, (const bf16*)qkg, nullptr, ends, (bf16*)o, B, st)) return rc;
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

@@ -3,18 +3,18 @@
 //   gated linear attention:    S <- diag(alpha) S + k v^T;                        o = S^T q       (alpha per key channel)
 // Three families:
 //  * decode (one token per sequence): one CTA per sequence and key head does everything between the input and the output projection:
-//    short convolution, unit norms, gates, state update, read-out, head norm and output gate. Bound by reading and writing S once:
-//    a thread keeps its part of S in registers, and S^T k and S^T q come out of the same pass because
-//    S_new^T q = g S^T q + (k . q) u.
+//    short convolution, unit norms, gates, state update, read-out, head norm and output gate. Bound by reading and writing S once: it passes through
+//    shared memory, and S^T k and S^T q come out of the same pass because S_new^T q = g S^T q + (k . q) u.
 //  * scan (prompts): S stays in registers over the whole prompt. The columns of S never mix, so a CTA takes 16 of them and a warp 4;
 //    eight lanes share a column and reduce with three shuffles.
 //  * the elementwise parts of a prompt: convolution, per-channel decay, head norm with output gate.
 // Rows of a batch read the state of slot slot_ids[b] (zeros when lengths[b] == 0) and stop after new_lens[b] tokens.
 #include "serving_common.cuh"
+#include "warp_mma.cuh"
 
 namespace mt {
 
-constexpr int DEC_NT = 512;      // threads of a decode CTA
+constexpr int DEC_NT = 256;      // threads of a decode CTA
 constexpr int SCAN_NT = 128;     // threads of a scan CTA
 constexpr int SCAN_COLS = 16;    // state columns per scan CTA
 constexpr int SCAN_TC = 16;      // tokens staged in shared memory at a time
@@ -47,45 +47,43 @@ __device__ __forceinline__ float beta_gate(float b) { return sigmoid_f(b); }
 __device__ __forceinline__ float log_decay(float a, float A_log, float dt) { return -expf(A_log) * softplus_f(a + dt); }
 
 // ------------------------------------------------------------------------------------------------ decode
-// grid (hk, B). RPT: rows of S a thread keeps in registers; 0: S is read twice instead (wide states).
-template <typename T, bool DELTA, int RPT>
+// grid (hk, B). TILE: the state of a head passes through shared memory (cp.async, several CTAs per SM hide each other's phases); otherwise it is read
+// twice from global memory (states too wide for shared memory, or not a multiple of 16 bytes).
+template <typename T, bool DELTA, bool TILE>
 __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, DeltaArgs<T> d, GlaArgs<T> gl, const T* __restrict__ norm_w, float eps,
-                                                                 T* __restrict__ out, int dvp) {
+                                                                 T* __restrict__ out, int dvp, int rows) {
   extern __shared__ __align__(16) float sm[];
   const int kh = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const int dk = a.dk, dv = a.dv, r = a.r, H = a.hk * r;
-  const int nrg = DEC_NT / dvp;                         // row groups
+  const int nrg = DEC_NT / dvp;                         // row groups of `rows` rows each
   const int rg = tid / dvp, c = tid % dvp;
-  const int rows = RPT > 0 ? RPT : (dk + nrg - 1) / nrg;
-  float* qs = sm;                                       // [rows * nrg] each, zero above dk
+  float* tile = sm;                                     // [dk * dv]
+  float* qs = tile + (TILE ? dk * dv : 0);              // [rows * nrg] each
   float* ks = qs + rows * nrg;
   float* al = ks + rows * nrg;                          // alpha (GLA)
-  float* vs = al + (DELTA ? 0 : rows * nrg);            // [r * dv]
-  float* redk = vs + ((r * dv + 3) & ~3);               // [DEC_NT]
+  float* redk = al + (DELTA ? 0 : rows * nrg);          // [DEC_NT]
   float* redq = redk + DEC_NT;
   float* wsum = redq + DEC_NT;                          // [DEC_NT / 32]
+  float* vs = wsum + DEC_NT / 32;                       // [r * dv]
   const long slot = a.slot_ids[b];
   const bool fresh = a.lengths[b] == 0;
   const bool col = c < dv;
-  const int row0 = rg * rows;
+  const int row0 = rg * rows, nrows = min(rows, dk - row0);
 
-  float S[RPT > 0 ? RPT : 1];
   auto state_of = [&](int h) { return a.rec + ((slot * H + h) * dk) * (long)dv; };
-  auto load_state = [&](int h) {
-    if constexpr (RPT > 0) {
+  auto load_tile = [&](int h) {
+    if constexpr (TILE) {
       const float* p = state_of(h);
-#pragma unroll
-      for (int i = 0; i < RPT; ++i) S[i] = (!fresh && col && row0 + i < dk) ? p[(long)(row0 + i) * dv + c] : 0.f;
+      if (!fresh)
+        for (int i = tid * 4; i < dk * dv; i += DEC_NT * 4) la_cp_async16(tile + i, p + i, 16);
+      else
+        for (int i = tid * 4; i < dk * dv; i += DEC_NT * 4) *reinterpret_cast<float4*>(tile + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+      la_commit();
     }
   };
-  load_state(kh * r);                                   // in flight while the convolution and the gates are computed
+  load_tile(kh * r);                                    // in flight while the convolution and the gates are computed
 
   const T* xr;
-  for (int i = tid; i < rows * nrg; i += DEC_NT) {
-    qs[i] = 0.f; ks[i] = 0.f;
-    if (!DELTA) al[i] = 0.f;
-  }
-  __syncthreads();
   if constexpr (DELTA) {
     const int per = 2 * dk + 2 * r * dv, key_dim = a.hk * dk, conv_dim = 2 * key_dim + H * dv, K = d.taps;
     xr = d.x + b * d.ldx + (long)kh * per;
@@ -100,7 +98,7 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
         if (j > 0) cs[(long)(j - 1) * conv_dim + ch] = old;
       }
       if (K > 1) cs[(long)(K - 2) * conv_dim + ch] = xv;
-      const float y = to_f(from_f<T>(silu_f(acc)));
+      const float y = to_f(from_f<T>(silu_t<T>(acc)));
       if (i < dk) qs[i] = y;
       else if (i < 2 * dk) ks[i - dk] = y;
       else vs[i - 2 * dk] = y;
@@ -111,9 +109,13 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
       const T* w = gl.w + ((long)kh * dk + i) * gl.rank;
       const T* lo = xr + 2L * H * (dk + dv);
       float z = to_f(gl.bias[kh * dk + i]);
-      for (int j = 0; j < gl.rank; ++j) z += to_f(w[j]) * to_f(lo[j]);
-      const float alpha = expf(log_sigmoid_f(z) * gl.inv_tau);
-      al[i] = alpha;
+      for (int j = 0; j < gl.rank; j += 8) {
+        float wv[8];
+        load_vec<8>(w + j, wv);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) z += wv[e] * to_f(lo[j + e]);
+      }
+      al[i] = expf(log_sigmoid_f(z) * gl.inv_tau);
       qs[i] = to_f(xr[(long)kh * dk + i]);
       ks[i] = to_f(xr[(long)H * dk + kh * dk + i]);
     }
@@ -132,18 +134,26 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
     rk = rsqrtf(warp_add(kk) + 1e-6f);
   }
   qk *= rq * rk;
+  if (!DELTA) {                                         // S_new^T q = S^T (alpha q) + (k . q) v
+    __syncthreads();
+    for (int i = tid; i < dk; i += DEC_NT) qs[i] *= al[i];
+  }
   for (int j = 0; j < r; ++j) {
     const int h = kh * r + j;
-    if (j > 0) load_state(h);
-    const float* sp = state_of(h);
+    if (j > 0) load_tile(h);
+    la_wait<0>();
+    __syncthreads();
+    float* gp = state_of(h);
+    const float* sp = (TILE ? tile : gp) + (long)row0 * dv + c;
+    const bool read = col && (TILE || !fresh);
     float pk = 0.f, pq = 0.f;
-#pragma unroll
-    for (int i = 0; i < rows; ++i) {
-      float s;
-      if constexpr (RPT > 0) s = S[i];
-      else s = (!fresh && col && row0 + i < dk) ? sp[(long)(row0 + i) * dv + c] : 0.f;
-      if constexpr (DELTA) { pk += s * ks[row0 + i]; pq += s * qs[row0 + i]; }
-      else pq += s * (al[row0 + i] * qs[row0 + i]);
+    if (read) {
+#pragma unroll 8
+      for (int i = 0; i < nrows; ++i) {
+        const float s = sp[(long)i * dv];
+        if (DELTA) pk += s * ks[row0 + i];
+        pq += s * qs[row0 + i];
+      }
     }
     if (DELTA) redk[tid] = pk;
     redq[tid] = pq;
@@ -163,16 +173,13 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
       u = v;
     }
     const float o = col ? decay * rq * sq + qk * u : 0.f;
-    float* wp = state_of(h);
+    const float ku = rk * u;
     if (col) {
-#pragma unroll
-      for (int i = 0; i < rows; ++i) {
-        if (row0 + i < dk) {
-          float s;
-          if constexpr (RPT > 0) s = S[i];
-          else s = fresh ? 0.f : wp[(long)(row0 + i) * dv + c];
-          wp[(long)(row0 + i) * dv + c] = (DELTA ? decay : al[row0 + i]) * s + ks[row0 + i] * rk * u;
-        }
+      float* wp = gp + (long)row0 * dv + c;
+#pragma unroll 8
+      for (int i = 0; i < nrows; ++i) {
+        const float s = read ? sp[(long)i * dv] : 0.f;
+        wp[(long)i * dv] = (DELTA ? decay : al[row0 + i]) * s + ks[row0 + i] * ku;
       }
     }
     // head norm over dv and output gate
@@ -184,16 +191,15 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
     if (rg == 0 && col) {
       const float rstd = rsqrtf(ss / (float)dv + eps);
       const T* zp = DELTA ? xr + 2 * dk + r * dv + j * dv : xr + 2L * H * dk + (long)H * dv + kh * dv;
-      out[((long)b * H + h) * dv + c] = from_f<T>(o * rstd * to_f(norm_w[c]) * silu_f(to_f(zp[c])));
+      out[((long)b * H + h) * dv + c] = from_f<T>(o * rstd * to_f(norm_w[c]) * silu_t<T>(to_f(zp[c])));
     }
-    __syncthreads();
   }
 }
 
 // ------------------------------------------------------------------------------------------------ convolution of a prompt
 // y[n, ch] = silu(sum_j w[j, ch] x[t - taps + 1 + j]) with inputs before the row's first new token taken from the state.
 // grid (channel groups, token tiles, B); a thread owns VEC channels and walks CONV_TT tokens.
-constexpr int CONV_TT = 32;
+constexpr int CONV_TT = 16;
 
 template <typename T, int VEC, int MAXK>
 __global__ void delta_conv_kernel(RecArgs a, DeltaArgs<T> d, T* __restrict__ y) {
@@ -206,7 +212,7 @@ __global__ void delta_conv_kernel(RecArgs a, DeltaArgs<T> d, T* __restrict__ y) 
   if (ch < key_dim) src = (long)(ch / dk) * per + ch % dk;
   else if (ch < 2 * key_dim) src = (long)((ch - key_dim) / dk) * per + dk + (ch - key_dim) % dk;
   else src = (long)((ch - 2 * key_dim) / (r * dv)) * per + 2 * dk + (ch - 2 * key_dim) % (r * dv);
-  const T* xb = d.x + (long)b * a.S * d.ldx + src;
+  const T* __restrict__ xb = d.x + (long)b * a.S * d.ldx + src;
   const bool fresh = a.lengths[b] == 0;
   const float* cs = d.conv + a.slot_ids[b] * (long)(K - 1) * conv_dim + ch;
   float w[MAXK][VEC], hist[MAXK][VEC];                   // hist[j]: input of tap j; the last K entries are used
@@ -224,22 +230,34 @@ __global__ void delta_conv_kernel(RecArgs a, DeltaArgs<T> d, T* __restrict__ y) 
     }
   }
   const int t1 = min(t0 + CONV_TT, a.S);
-  for (int t = t0; t < t1; ++t) {
-    load_vec<VEC>(xb + (long)t * d.ldx, hist[MAXK - 1]);
-    float acc[VEC];
+  T* __restrict__ yb = y + (long)b * a.S * conv_dim + ch;
+  for (int t = t0; t < t1; t += 4) {
+    float in[4][VEC];                                    // four loads in flight
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+    for (int u = 0; u < 4; ++u)
+      if (t + u < t1) load_vec<VEC>(xb + (long)(t + u) * d.ldx, in[u]);
 #pragma unroll
-    for (int j = 0; j < MAXK; ++j)
+    for (int u = 0; u < 4; ++u) {
+      if (t + u < t1) {
+        float acc[VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) acc[e] += w[j][e] * hist[j][e];
+        for (int e = 0; e < VEC; ++e) {
+          hist[MAXK - 1][e] = in[u][e];
+          acc[e] = 0.f;
+        }
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) acc[e] = silu_f(acc[e]);
-    store_vec<VEC>(y + ((long)b * a.S + t) * conv_dim + ch, acc);
+        for (int j = 0; j < MAXK; ++j)
 #pragma unroll
-    for (int j = 0; j < MAXK - 1; ++j)
+          for (int e = 0; e < VEC; ++e) acc[e] += w[j][e] * hist[j][e];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) hist[j][e] = hist[j + 1][e];
+        for (int e = 0; e < VEC; ++e) acc[e] = silu_t<T>(acc[e]);
+        store_vec<VEC>(yb + (long)(t + u) * conv_dim, acc);
+#pragma unroll
+        for (int j = 0; j < MAXK - 1; ++j)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) hist[j][e] = hist[j + 1][e];
+      }
+    }
   }
 }
 
@@ -400,31 +418,35 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
 
 // ------------------------------------------------------------------------------------------------ head norm + output gate
 // out[n, h, :] = rms(o[n, h, :]) * w * silu(z), one warp per (n, h); z of head h sits at x[n * ldx + zoff + (h / r) * zstride + (h % r) * dv].
-template <typename T, int VEC>
-__global__ void gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ x, long ldx, long rows, int H, int dv, int r, long zoff, long zstride,
-                                       const T* __restrict__ w, float eps, T* __restrict__ out) {
-  const long row = ((long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-  if (row >= rows) return;
-  const int lane = threadIdx.x & 31;
-  const long n = row / H;
-  const int h = (int)(row % H);
-  const T* op = o + row * dv;
+// LPR lanes share a row.
+template <typename T, int VEC, int LPR>
+__global__ void __launch_bounds__(256) gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ x, long ldx, long rows, int H, int dv, int r,
+                                                              long zoff, long zstride, const T* __restrict__ w, float eps, T* __restrict__ out) {
+  const long row = ((long)blockIdx.x * blockDim.x + threadIdx.x) / LPR;
+  const int lane = threadIdx.x % LPR;
+  const bool in = row < rows;
+  const long n = in ? row / H : 0;
+  const int h = in ? (int)(row % H) : 0;
+  const T* op = o + (in ? row : 0) * dv;
   const T* zp = x + n * ldx + zoff + (long)(h / r) * zstride + (long)(h % r) * dv;
-  float ss = 0.f;
-  for (int c = lane * VEC; c < dv; c += 32 * VEC) {
-    float v[VEC];
+  float ss = 0.f, v[VEC];
+  for (int c = lane * VEC; c < dv; c += LPR * VEC) {
     load_vec<VEC>(op + c, v);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
   }
-  const float rstd = rsqrtf(warp_add(ss) / (float)dv + eps);
-  for (int c = lane * VEC; c < dv; c += 32 * VEC) {
-    float v[VEC], z[VEC], g[VEC];
-    load_vec<VEC>(op + c, v);
+#pragma unroll
+  for (int s = LPR / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  if (!in) return;
+  const float rstd = rsqrtf(ss / (float)dv + eps);
+  const bool once = dv <= LPR * VEC;                     // the row is still in registers
+  for (int c = lane * VEC; c < dv; c += LPR * VEC) {
+    float z[VEC], g[VEC];
+    if (!once) load_vec<VEC>(op + c, v);
     load_vec<VEC>(zp + c, z);
     load_vec<VEC>(w + c, g);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) v[e] = v[e] * rstd * g[e] * silu_f(z[e]);
+    for (int e = 0; e < VEC; ++e) v[e] = v[e] * rstd * g[e] * silu_t<T>(z[e]);
     store_vec<VEC>(out + row * dv + c, v);
   }
 }
@@ -435,15 +457,16 @@ int launch_decode(const RecArgs& a, const DeltaArgs<T>& d, const GlaArgs<T>& g, 
   int dvp = 32;
   while (dvp < a.dv) dvp <<= 1;
   if (dvp > DEC_NT) return -1;
-  const int nrg = DEC_NT / dvp, need = (a.dk + nrg - 1) / nrg;
-  const int rpt = need <= 8 ? 8 : need <= 16 ? 16 : need <= 32 ? 32 : need <= 64 ? 64 : 0;
-  const int rows = rpt ? rpt : need;
-  const size_t smem = sizeof(float) * ((DELTA ? 2 : 3) * (size_t)rows * nrg + ((a.r * a.dv + 3) & ~3) + 2 * DEC_NT + DEC_NT / 32);
-  if (smem > 200 * 1024) return -1;
-  auto k = rpt == 8 ? recurrent_decode_kernel<T, DELTA, 8> : rpt == 16 ? recurrent_decode_kernel<T, DELTA, 16> : rpt == 32
-      ? recurrent_decode_kernel<T, DELTA, 32> : rpt == 64 ? recurrent_decode_kernel<T, DELTA, 64> : recurrent_decode_kernel<T, DELTA, 0>;
+  const int nrg = DEC_NT / dvp, rows = ((a.dk + nrg - 1) / nrg + 3) & ~3;
+  const size_t state = sizeof(float) * (size_t)a.dk * a.dv;
+  const bool tile = state % 16 == 0 && state <= 160 * 1024;
+  const size_t smem = (tile ? state : 0) + sizeof(float) * ((DELTA ? 2 : 3) * (size_t)rows * nrg + (size_t)a.r * a.dv + 2 * DEC_NT + DEC_NT / 32);
+  if (smem > 220 * 1024) return -1;
+  auto k1 = recurrent_decode_kernel<T, DELTA, true>;
+  auto k0 = recurrent_decode_kernel<T, DELTA, false>;
+  auto k = tile ? k1 : k0;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return -2;
-  k<<<dim3(a.hk, B), DEC_NT, smem, st>>>(a, d, g, (const T*)norm, eps, (T*)out, dvp);
+  k<<<dim3(a.hk, B), DEC_NT, smem, st>>>(a, d, g, (const T*)norm, eps, (T*)out, dvp, rows);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -482,11 +505,14 @@ int launch_conv(const RecArgs& a, const DeltaArgs<T>& d, void* y, int B, cudaStr
 template <typename T>
 int launch_head_norm(const void* o, const void* x, long ldx, long rows, int H, int dv, int r, long zoff, long zstride, const void* w, float eps, void* out,
                      cudaStream_t st) {
-  const unsigned blocks = (unsigned)((rows + 7) / 8);
-  const bool v4 = dv % 4 == 0 && ldx % 4 == 0 && zoff % 4 == 0 && zstride % 4 == 0;
-  auto k4 = gated_head_norm_kernel<T, 4>;
-  auto k1 = gated_head_norm_kernel<T, 1>;
-  (v4 ? k4 : k1)<<<blocks, 256, 0, st>>>((const T*)o, (const T*)x, ldx, rows, H, dv, r, zoff, zstride, (const T*)w, eps, (T*)out);
+  const bool v8 = dv % 8 == 0 && ldx % 8 == 0 && zoff % 8 == 0 && zstride % 8 == 0;
+#define GO(V, L) gated_head_norm_kernel<T, V, L><<<(unsigned)((rows * L + 255) / 256), 256, 0, st>>>((const T*)o, (const T*)x, ldx, rows, H, dv, r, zoff, \
+                                                                                                  zstride, (const T*)w, eps, (T*)out)
+  if (!v8) GO(1, 32);
+  else if (dv <= 64) GO(8, 8);
+  else if (dv <= 128) GO(8, 16);
+  else GO(8, 32);
+#undef GO
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 

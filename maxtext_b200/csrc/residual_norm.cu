@@ -63,6 +63,18 @@ __device__ __forceinline__ float act_value(float x, int code) {
   }
 }
 
+// Gelu for a bf16 result: Abramowitz and Stegun 7.1.26, erfc(z) = t (a1 + t (a2 + t (a3 + t (a4 + t a5)))) e^(-z^2) with t = 1 / (1 + p z), absolute
+// error below 1.5e-7; 1 + erf is formed without cancellation for negative arguments.
+__device__ __forceinline__ float gelu_erf_bf16(float x) {
+  const float z = fabsf(x) * 0.7071067811865476f, t = __fdividef(1.f, 1.f + 0.3275911f * z);
+  const float c = t * (0.254829592f + t * (-0.284496736f + t * (1.421413741f + t * (-1.453152027f + t * 1.061405429f)))) * __expf(-z * z);
+  return 0.5f * x * (x < 0.f ? c : 2.f - c);
+}
+template <typename T> __device__ __forceinline__ float act_typed(float x, int code) { return act_value(x, code); }
+template <> __device__ __forceinline__ float act_typed<__nv_bfloat16>(float x, int code) {
+  return code == 4 ? gelu_erf_bf16(x) : (code == 0 ? silu_t<__nv_bfloat16>(x) : act_value(x, code));
+}
+
 template <typename T>
 __global__ void act_kernel(const T* __restrict__ x, T* __restrict__ y, long n, int code) {
   const long nv = n / 8;
@@ -70,10 +82,10 @@ __global__ void act_kernel(const T* __restrict__ x, T* __restrict__ y, long n, i
     float v[8];
     load_vec<8>(x + i * 8, v);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = act_value(v[e], code);
+    for (int e = 0; e < 8; ++e) v[e] = act_typed<T>(v[e], code);
     store_vec<8>(y + i * 8, v);
   }
-  if (blockIdx.x == 0 && threadIdx.x < n - nv * 8) y[nv * 8 + threadIdx.x] = from_f<T>(act_value(to_f(x[nv * 8 + threadIdx.x]), code));
+  if (blockIdx.x == 0 && threadIdx.x < n - nv * 8) y[nv * 8 + threadIdx.x] = from_f<T>(act_typed<T>(to_f(x[nv * 8 + threadIdx.x]), code));
 }
 
 template <typename T>

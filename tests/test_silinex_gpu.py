@@ -182,6 +182,42 @@ def test_latent_decode_attention(H, R, dr, window, lens):
   assert _status() == 0
 
 
+@pytest.mark.parametrize("B, H, nope, dr, vd, R", [(3, 2, 20, 6, 14, 36), (1, 5, 32, 16, 48, 64), (8, 3, 48, 16, 40, 128), (70, 2, 128, 64, 128, 512), (33, 4, 16, 8, 80, 320)])
+def test_latent_decode_products(B, H, nope, dr, vd, R):
+  from maxtext_b200.ops import backend
+  E = backend.ext(required=True)
+  g = torch.Generator().manual_seed(4)
+  for dtype, tol in ((torch.float32, 1e-5), (torch.bfloat16, 6e-3)):
+    q, w = (torch.randn(*s, generator=g).to(dtype).cuda() for s in ((B, H, nope + dr), (H * (nope + vd), R)))
+    pos = torch.randint(0, 5000, (B,), generator=g).cuda()
+    inv = (10000.0 ** (-torch.arange(dr // 2, dtype=torch.float64) * 2 / dr)).float().cuda()
+    wd = w.double().view(H, nope + vd, R)
+    for inter in (True, False):
+      qa = torch.empty(B, H, R + dr, dtype=dtype, device="cuda")
+      E.mla_absorb(q, w, pos, inv, inter, nope, vd, qa)
+      qd = q.double()
+      ang = pos.double()[:, None, None] * inv.double()
+      u, v = (qd[..., nope::2], qd[..., nope + 1::2]) if inter else (qd[..., nope:nope + dr // 2], qd[..., nope + dr // 2:])
+      a, b = u * ang.cos() - v * ang.sin(), v * ang.cos() + u * ang.sin()
+      rot = torch.stack([a, b], -1).flatten(-2) if inter else torch.cat([a, b], -1)
+      want = torch.cat([torch.einsum("bhd,hdr->bhr", qd[..., :nope], wd[:, :nope]), rot], -1)
+      for part in (slice(0, R), slice(R, R + dr)):
+        assert (qa.double() - want)[..., part].pow(2).mean().sqrt() < max(tol, 2e-4 if part.start else 0) * want[..., part].pow(2).mean().sqrt(), (dtype, inter, part)
+    for splits in (1, 3):
+      part, ml = torch.randn(B, H, splits, R, generator=g).cuda(), torch.rand(B, H, splits, 2, generator=g).cuda() + 0.1
+      if splits > 1:
+        ml[:, :, 1] = torch.tensor([float("-inf"), 0.0])                   # a split without keys
+        part[:, :, 1] = float("nan")
+      out = torch.empty(B, H, vd, dtype=dtype, device="cuda")
+      E.mla_value_up(part, ml, w, nope, out)
+      m = ml[..., 0].double().max(-1, keepdim=True).values
+      f = torch.where(ml[..., 1] > 0, torch.exp(ml[..., 0].double() - m), torch.zeros_like(m))
+      ctx = (torch.nan_to_num(part.double()) * f[..., None]).sum(2) / (f * ml[..., 1].double()).sum(2)[..., None]
+      want = torch.einsum("bhr,her->bhe", ctx, wd[:, nope:])
+      assert (out.double() - want).pow(2).mean().sqrt() < tol * want.pow(2).mean().sqrt(), (dtype, splits)
+  assert _status() == 0
+
+
 def test_fp32_stream_kernels():
   from maxtext_b200.ops import functional as F
   g = torch.Generator().manual_seed(0)
