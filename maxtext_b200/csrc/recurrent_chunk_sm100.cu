@@ -39,8 +39,9 @@ __device__ __forceinline__ int real_tokens(const ChunkArgs& a, int b) { return m
 __device__ __forceinline__ long chunk_id(const ChunkArgs& a, int b, int c, int h) { return ((long)b * a.chunks + c) * a.H + h; }
 
 // rows [0, CH) of a [CH, dk] bf16 tile to shared memory (row length ld), zeros past row m; dk is a multiple of 8
-__device__ __forceinline__ void tile_async(bf16* dst, int ld, const bf16* src, long stride, int cols, int m, int tid, int nt) {
-  const int v = cols / 8;
+template <int cols>
+__device__ __forceinline__ void tile_async(bf16* dst, int ld, const bf16* src, long stride, int m, int tid, int nt) {
+  constexpr int v = cols / 8;
   for (int i = tid; i < CH * v; i += nt) {
     const int r = i / v, c = (i % v) * 8;
     la_cp_async16(dst + r * ld + c, src + (long)(r < m ? r : 0) * stride + c, r < m ? 16 : 0);
@@ -50,12 +51,14 @@ __device__ __forceinline__ void tile_async(bf16* dst, int ld, const bf16* src, l
 // ------------------------------------------------------------------------------------------------ gated delta: prepare
 // grid (chunks, H, B), 128 threads. tp: per chunk and head four [64][64] bf16 tiles: T high, T low, P high, P low;
 // gates: per chunk and head [4][64] floats: rk e^G, beta, rq e^G, rk e^(G_end - G), and e^G_end in gate_end.
+template <int DK>
 __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(ChunkArgs a, const bf16* __restrict__ mixed, long ldx, const bf16* __restrict__ ba, long ldb,
                                                                   const bf16* __restrict__ A_log, const bf16* __restrict__ dt_bias, bf16* __restrict__ tp,
                                                                   float* __restrict__ gates, float* __restrict__ gate_end) {
   extern __shared__ __align__(16) unsigned char raw[];
   const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int dk = a.dk, r = a.r, kh = h / r, LD = dk + 8, t0 = a.t_lo + c * CH;
+  constexpr int dk = DK, LD = DK + 8;
+  const int r = a.r, kh = h / r, t0 = a.t_lo + c * CH;
   const int m = min(CH, real_tokens(a, b) - t0);
   if (m <= 0) return;
   bf16* ks = reinterpret_cast<bf16*>(raw);               // [64][LD]
@@ -63,8 +66,8 @@ __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(ChunkArgs a, c
   float* L = reinterpret_cast<float*>(qs + CH * LD);     // [64][68]
   __shared__ float G[CH], beta[CH], rk[CH], rq[CH], half_sum;
   const bf16* row0 = mixed + ((long)b * a.S + t0) * ldx;
-  tile_async(qs, LD, row0 + (long)kh * dk, ldx, dk, m, tid, 128);
-  tile_async(ks, LD, row0 + (long)(a.H / r + kh) * dk, ldx, dk, m, tid, 128);
+  tile_async<dk>(qs, LD, row0 + (long)kh * dk, ldx, m, tid, 128);
+  tile_async<dk>(ks, LD, row0 + (long)(a.H / r + kh) * dk, ldx, m, tid, 128);
   la_commit();
   float lg = 0.f;
   if (tid < CH) {
@@ -153,24 +156,32 @@ __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(ChunkArgs a, c
     }
   }
   __syncthreads();
-  if (tid < CH) {
-    // column tid of T by forward substitution: T_i = [i == tid] - sum_{k < i} L_ik T_k
-    float t[CH];
+  // T in blocks of 32: the diagonal blocks by forward substitution (a warp each, a lane per column), T21 = -T22 (L21 T11) by all threads
+  __shared__ __align__(16) float Ts[CH][36], Ms[32][36];
+  auto put = [&](int i, int j, float t) {
+    const bf16 hi = __float2bfloat16_rn(t);
+    out[i * CH + j] = hi;
+    out[CH * CH + i * CH + j] = __float2bfloat16_rn(t - __bfloat162float(hi));
+  };
+  if (warp < 2) {
+    const float* l0 = L + warp * 32 * 68 + warp * 32;
+    float t[32];
 #pragma unroll
-    for (int i = 0; i < CH; ++i) {
-      float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    for (int i = 0; i < 32; ++i) {
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int k = 0; k < (i & ~3); k += 4) {
-        const float4 l = *reinterpret_cast<const float4*>(L + i * 68 + k);
-        s0 += l.x * t[k]; s1 += l.y * t[k + 1]; s2 += l.z * t[k + 2]; s3 += l.w * t[k + 3];
+      for (int k = 0; k < i; k += 4) {                   // entries at and right of the diagonal are zero
+        const float4 l = *reinterpret_cast<const float4*>(l0 + i * 68 + k);
+        s[0] += l.x * t[k];
+        if (k + 1 < i) s[1] += l.y * t[k + 1];
+        if (k + 2 < i) s[2] += l.z * t[k + 2];
+        if (k + 3 < i) s[3] += l.w * t[k + 3];
       }
-#pragma unroll
-      for (int k = i & ~3; k < i; ++k) s0 += L[i * 68 + k] * t[k];
-      t[i] = (i == tid ? 1.f : 0.f) - ((s0 + s1) + (s2 + s3));
-      const bf16 hi = __float2bfloat16_rn(t[i]);
-      out[i * CH + tid] = hi;
-      out[CH * CH + i * CH + tid] = __float2bfloat16_rn(t[i] - __bfloat162float(hi));
+      t[i] = (i == lane ? 1.f : 0.f) - ((s[0] + s[1]) + (s[2] + s[3]));
+      Ts[warp * 32 + i][lane] = t[i];
     }
+#pragma unroll 8
+    for (int i = 0; i < 32; ++i) put(warp * 32 + i, warp * 32 + lane, Ts[warp * 32 + i][lane]);
   } else {
     const int i = tid - CH;
     float* g = gates + chunk_id(a, b, c, h) * 4 * CH;
@@ -181,16 +192,44 @@ __global__ void __launch_bounds__(128) delta_chunk_prepare_kernel(ChunkArgs a, c
     g[3 * CH + i] = rk[i] * expf(end - G[i]);
     if (i == 0) gate_end[chunk_id(a, b, c, h)] = expf(end);
   }
+  __syncthreads();
+  const int row = tid >> 2, c8 = (tid & 3) * 8;
+  float acc[8];
+  auto product = [&](const float* x, const float (*y)[36]) {         // acc = x[0 .. 31] . y[0 .. 31][c8 .. c8 + 7]
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+#pragma unroll 4
+    for (int k = 0; k < 32; ++k) {
+      const float f = x[k];
+      const float4 u = *reinterpret_cast<const float4*>(&y[k][c8]), v = *reinterpret_cast<const float4*>(&y[k][c8 + 4]);
+      acc[0] += f * u.x; acc[1] += f * u.y; acc[2] += f * u.z; acc[3] += f * u.w;
+      acc[4] += f * v.x; acc[5] += f * v.y; acc[6] += f * v.z; acc[7] += f * v.w;
+    }
+  };
+  product(L + (32 + row) * 68, Ts);
+  store_vec<8>(&Ms[row][c8], acc);
+  __syncthreads();
+  product(&Ts[32 + row][0], Ms);
+  float neg[8], low[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    neg[e] = -acc[e];
+    low[e] = neg[e] - __bfloat162float(__float2bfloat16_rn(neg[e]));
+  }
+  store_vec<8>(out + (32 + row) * CH + c8, neg);
+  store_vec<8>(out + CH * CH + (32 + row) * CH + c8, low);
 }
 
 // ------------------------------------------------------------------------------------------------ gated linear attention: prepare
 // grid (chunks, H, B), 256 threads. aa: per chunk and head A high, A low [64][64]; qkg: per chunk and head four [64][dk] tiles: q e^G high, low,
 // k e^(G_end - G) high, low; end: e^G_end [dk].
+template <int DK>
 __global__ void __launch_bounds__(256) gla_chunk_prepare_kernel(ChunkArgs a, const bf16* __restrict__ x, long ldx, const float* __restrict__ log_alpha,
                                                                 bf16* __restrict__ aa, bf16* __restrict__ qkg, float* __restrict__ end) {
   extern __shared__ __align__(16) float sm[];
   const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
-  const int dk = a.dk, H = a.H, LD = dk + 4, t0 = a.t_lo + c * CH;
+  constexpr int dk = DK, LD = DK + 4;
+  const int H = a.H, t0 = a.t_lo + c * CH;
   const int m = min(CH, real_tokens(a, b) - t0);
   if (m <= 0) return;
   float* G = sm;                                         // [64][LD]
@@ -198,21 +237,43 @@ __global__ void __launch_bounds__(256) gla_chunk_prepare_kernel(ChunkArgs a, con
   float* qsc = ksc + CH * LD;                            // [16][LD]
   bf16* q = reinterpret_cast<bf16*>(qsc + 16 * LD);      // [64][dk + 8]
   bf16* k = q + CH * (dk + 8);
-  const int QLD = dk + 8;
+  constexpr int QLD = dk + 8;
   const bf16* row0 = x + ((long)b * a.S + t0) * ldx;
-  tile_async(q, QLD, row0 + (long)h * dk, ldx, dk, m, tid, 256);
-  tile_async(k, QLD, row0 + (long)(H + h) * dk, ldx, dk, m, tid, 256);
+  tile_async<dk>(q, QLD, row0 + (long)h * dk, ldx, m, tid, 256);
+  tile_async<dk>(k, QLD, row0 + (long)(H + h) * dk, ldx, m, tid, 256);
+  const float* la = log_alpha + ((long)b * a.S + t0) * H * dk + (long)h * dk;
+  for (int i = tid; i < CH * dk / 4; i += 256) {
+    const int t = i / (dk / 4), d = (i % (dk / 4)) * 4;
+    la_cp_async16(G + t * LD + d, la + (long)(t < m ? t : 0) * H * dk + d, t < m ? 16 : 0);
+  }
   la_commit();
-  if (tid < dk) {
-    const float* la = log_alpha + ((long)b * a.S + t0) * H * dk + (long)h * dk + tid;
-    float g = 0.f;
-#pragma unroll 8
-    for (int i = 0; i < CH; ++i) {
-      if (i < m) g += la[(long)i * H * dk] * 1.4426950408889634f;         // base 2
-      G[i * LD + tid] = g;
+  la_wait<0>();
+  __syncthreads();
+  // running sums down the 64 tokens, in base 2: four segments of 16 tokens per channel, then the segments' offsets
+  for (int w = tid; w < 4 * dk; w += 256) {
+    float* g = G + (w / dk) * 16 * LD + w % dk;
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) { s += g[i * LD] * 1.4426950408889634f; g[i * LD] = s; }
+  }
+  __syncthreads();
+  float off[2] = {0.f, 0.f};                             // 4 dk <= 512 segments over 256 threads
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int w = tid + x * 256;
+    if (w < 4 * dk)
+      for (int s = 0; s < w / dk; ++s) off[x] += G[(s * 16 + 15) * LD + w % dk];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int w = tid + x * 256;
+    if (w < 4 * dk && w >= dk) {
+      float* g = G + (w / dk) * 16 * LD + w % dk;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) g[i * LD] += off[x];
     }
   }
-  la_wait<0>();
   __syncthreads();
   const float scale = rsqrtf((float)dk);
   const long id = chunk_id(a, b, c, h);
@@ -310,13 +371,13 @@ __global__ void __launch_bounds__(256) chunk_carry_kernel(ChunkArgs a, const bf1
     const long id = chunk_id(a, b, c, h);
     const bf16* row0 = x + ((long)b * a.S + t0) * ldx;
     if constexpr (DELTA) {
-      tile_async(qkt(buf, 0), LD, row0 + (long)kh * dk, ldx, dk, m, tid, 256);
-      tile_async(qkt(buf, 1), LD, row0 + koff + (long)kh * dk, ldx, dk, m, tid, 256);
+      tile_async<dk>(qkt(buf, 0), LD, row0 + (long)kh * dk, ldx, m, tid, 256);
+      tile_async<dk>(qkt(buf, 1), LD, row0 + koff + (long)kh * dk, ldx, m, tid, 256);
     } else {
-      for (int i = 0; i < 4; ++i) tile_async(qkt(buf, i), LD, qkg + (id * 4 + i) * CH * dk, dk, dk, CH, tid, 256);
+      for (int i = 0; i < 4; ++i) tile_async<dk>(qkt(buf, i), LD, qkg + (id * 4 + i) * CH * dk, dk, CH, tid, 256);
     }
-    tile_async(vt(buf), NLD, row0 + voff + (long)h * dv + c0, ldx, CN, m, tid, 256);
-    for (int i = 0; i < NTP; ++i) tile_async(tpt(buf, i), CLD, tiles + (id * NTP + i) * CH * CH, CH, CH, CH, tid, 256);
+    tile_async<CN>(vt(buf), NLD, row0 + voff + (long)h * dv + c0, ldx, m, tid, 256);
+    for (int i = 0; i < NTP; ++i) tile_async<CH>(tpt(buf, i), CLD, tiles + (id * NTP + i) * CH * CH, CH, CH, tid, 256);
     const float* g = DELTA ? gates + id * 4 * CH : ends + id * dk;
     for (int i = tid; i < (DELTA ? CH : dk / 4); i += 256) la_cp_async16(gt(buf) + i * 4, g + i * 4, 16);
     la_commit();
@@ -539,9 +600,14 @@ extern "C" int mt_delta_chunks(const void* mixed, long ldx, const void* ba, long
   if (!mt_chunk_supported(dk, dv) || ldx % 8) return -1;
   const ChunkArgs a{hv, hv / hk, dk, dv, S, t_lo, t_hi, (t_hi - t_lo + CH - 1) / CH, slots, lengths, new_lens, rec};
   const size_t s1 = 2 * 2 * (size_t)CH * (dk + 8) + 4 * CH * 68;
-  if (cudaFuncSetAttribute(delta_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2;
-  delta_chunk_prepare_kernel<<<dim3(a.chunks, hv, B), 128, s1, st>>>(a, (const bf16*)mixed, ldx, (const bf16*)ba, ldb, (const bf16*)A_log,
-                                                                    (const bf16*)dt_bias, (bf16*)tp, gates, ends);
+  switch (dk) {
+#define GO(DK) case DK: \
+    if (cudaFuncSetAttribute(delta_chunk_prepare_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2; \
+    delta_chunk_prepare_kernel<DK><<<dim3(a.chunks, hv, B), 128, s1, st>>>(a, (const bf16*)mixed, ldx, (const bf16*)ba, ldb, (const bf16*)A_log, \
+                                                                          (const bf16*)dt_bias, (bf16*)tp, gates, ends); break;
+    GO(16) GO(32) GO(48) GO(64) GO(80) GO(96) GO(112) GO(128)
+#undef GO
+  }
   if (int rc = launch_carry<true>(a, (const bf16*)mixed, ldx, (long)hk * dk, 2L * hk * dk, (const bf16*)tp, nullptr, gates, ends, (bf16*)o, B, st)) return rc;
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
@@ -552,8 +618,13 @@ extern "C" int mt_gla_chunks(const void* x, long ldx, const float* log_alpha, in
   if (!mt_chunk_supported(dk, dv) || ldx % 8) return -1;
   const ChunkArgs a{H, 1, dk, dv, S, t_lo, t_hi, (t_hi - t_lo + CH - 1) / CH, slots, lengths, new_lens, rec};
   const size_t s1 = 4 * (size_t)(2 * CH + 16) * (dk + 4) + 2 * 2 * (size_t)CH * (dk + 8);
-  if (cudaFuncSetAttribute(gla_chunk_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2;
-  gla_chunk_prepare_kernel<<<dim3(a.chunks, H, B), 256, s1, st>>>(a, (const bf16*)x, ldx, log_alpha, (bf16*)aa, (bf16*)qkg, ends);
+  switch (dk) {
+#define GO(DK) case DK: \
+    if (cudaFuncSetAttribute(gla_chunk_prepare_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1) != cudaSuccess) return -2; \
+    gla_chunk_prepare_kernel<DK><<<dim3(a.chunks, H, B), 256, s1, st>>>(a, (const bf16*)x, ldx, log_alpha, (bf16*)aa, (bf16*)qkg, ends); break;
+    GO(16) GO(32) GO(48) GO(64) GO(80) GO(96) GO(112) GO(128)
+#undef GO
+  }
   if (int rc = launch_carry<false>(a, (const bf16*)x, ldx, 0, 2L * H * dk, (const bf16*)aa, (const bf16*)qkg, nullptr, ends, (bf16*)o, B, st)) return rc;
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
