@@ -129,6 +129,7 @@ void gemm(const torch::Tensor& a, const torch::Tensor& b, torch::Tensor& out, bo
   check(rc, "mt_gemm_bf16");
 }
 
+#ifndef MT_SERVING_ONLY
 // x [R, C] bf16 -> (q [R, C] uint8 or None, qt [C, R] uint8 or None, dequant scale [1]); fmt 0 = E4M3, 1 = E5M2. Current scaling:
 // the scale comes from this tensor's own absolute maximum, computed on the device.
 std::tuple<c10::optional<torch::Tensor>, c10::optional<torch::Tensor>, torch::Tensor, torch::Tensor> quantize_fp8_with(
@@ -179,6 +180,7 @@ void gemm_fp8(const torch::Tensor& a, const torch::Tensor& b, torch::Tensor& out
                     status_tensor().data_ptr<int>(), num_sms(), cur_stream()),
         "mt_gemm_fp8");
 }
+#endif
 
 // the CTA-pair (cta_group::2) variant of `gemm`; N must be a multiple of 128
 void gemm_pair(const torch::Tensor& a, const torch::Tensor& b, torch::Tensor& out, bool ta, bool tb, bool accumulate) {
@@ -262,6 +264,7 @@ void embedding_bwd(const torch::Tensor& tok, const torch::Tensor& dy, torch::Ten
         "embedding_bwd");
 }
 
+#ifndef MT_SERVING_ONLY
 void xent_fwd_bwd(torch::Tensor& logits, const torch::Tensor& targets, const torch::Tensor& weights, double z_loss, torch::Tensor& loss,
                   torch::Tensor& z, bool write_grad) {
   TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1 && logits.scalar_type() == torch::kBFloat16);
@@ -291,6 +294,7 @@ void sumsq(const torch::Tensor& x, torch::Tensor& out) {
   auto partials = torch::empty({parts}, x.options());
   check(mt_sumsq(x.data_ptr<float>(), x.numel(), partials.data_ptr<float>(), out.data_ptr<float>(), num_sms(), cur_stream()), "mt_sumsq", 2);
 }
+#endif
 
 }  // namespace
 
@@ -312,9 +316,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_use_pair", [](bool v) { g_use_pair = v; });
   m.def("gemm_set_raster", [](int64_t v) { mt_gemm_set_raster((int)v); });
   m.def("gemm_set_group_m", [](int64_t v) { TORCH_CHECK(mt_gemm_set_group_m((int)v) == 0, "bad group size"); });
-  m.def("quantize_fp8", &quantize_fp8);
-  m.def("quantize_fp8_with", &quantize_fp8_with);
-  m.def("gemm_fp8", &gemm_fp8);
   m.def("kernel_status", &kernel_status);
   m.def("launch_count", &launch_count);
   m.def("rmsnorm_fwd", &rmsnorm_fwd);
@@ -324,11 +325,16 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gated_act_bwd", &gated_act_bwd);
   m.def("embedding_fwd", &embedding_fwd);
   m.def("embedding_bwd", &embedding_bwd);
+  register_attention(m);
+  register_serving(m);
+#ifndef MT_SERVING_ONLY
+  m.def("quantize_fp8", &quantize_fp8);
+  m.def("quantize_fp8_with", &quantize_fp8_with);
+  m.def("gemm_fp8", &gemm_fp8);
   m.def("xent_fwd_bwd", &xent_fwd_bwd);
   m.def("adamw", &adamw);
   m.def("sumsq", &sumsq);
-  register_attention(m);
   register_moe(m);
   register_comm(m);
-  register_serving(m);
+#endif
 }

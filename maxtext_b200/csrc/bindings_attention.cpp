@@ -74,6 +74,7 @@ void flash_fwd(const torch::Tensor& q, const torch::Tensor& k, const torch::Tens
   mt_count_launches(pos_q ? 3 : 1);
 }
 
+#ifndef MT_SERVING_ONLY
 bool flash_bwd_supported(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v) {
   return flash_fwd_supported(q, k, v) && mt_flash_bwd_supported((int)q.size(3), (int)v.size(3));
 }
@@ -102,6 +103,7 @@ void flash_bwd(const torch::Tensor& dout, const torch::Tensor& q, const torch::T
   TORCH_CHECK(rc == 0, "mt_flash_bwd failed with code ", rc);
   mt_count_launches(pos_q ? 5 : 3);
 }
+#endif
 
 // q [B, Hq, D], caches [slots, max_len, Hkv, D] (bf16), slot_ids / lengths int32 [B] (lengths include the new token); out [B, Hq, D].
 void decode_attention(const torch::Tensor& q, const torch::Tensor& k_cache, const torch::Tensor& v_cache, const torch::Tensor& slot_ids,
@@ -144,7 +146,9 @@ void register_attention(pybind11::module_& m) {
   m.def("sample_tokens", &sample_tokens);
   m.def("decode_attention", &decode_attention);
   m.def("flash_fwd_supported", &flash_fwd_supported);
-  m.def("flash_bwd_supported", &flash_bwd_supported);
   m.def("flash_fwd", &flash_fwd);
+#ifndef MT_SERVING_ONLY
+  m.def("flash_bwd_supported", &flash_bwd_supported);
   m.def("flash_bwd", &flash_bwd);
+#endif
 }

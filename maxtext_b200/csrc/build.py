@@ -34,6 +34,24 @@ def build_extension(verbose: bool = True):
   return mod
 
 
+# what inference needs: a machine that only serves and has no built library compiles this part of it
+SERVING_DIR = os.path.join(HERE, "build_serving")
+SERVING_NAME = "maxtext_b200_serving_C"
+SERVING_SOURCES = ("bindings.cpp", "bindings_attention.cpp", "bindings_serving.cpp", "gemm_sm100.cu", "gemm_small_m.cu", "elementwise.cu",
+                   "attention_fwd_sm100.cu", "decode_attention.cu", "sampling_sm100.cu", "residual_norm.cu", "recurrent_sm100.cu",
+                   "recurrent_chunk_sm100.cu", "latent_attention_sm100.cu")
+
+
+def build_serving_extension(verbose: bool = True):
+  from torch.utils import cpp_extension
+  os.makedirs(SERVING_DIR, exist_ok=True)
+  os.environ.setdefault("MAX_JOBS", str(min(16, os.cpu_count() or 4)))
+  flag = ["-DMT_SERVING_ONLY"]
+  return cpp_extension.load(
+      name=SERVING_NAME, sources=[os.path.join(HERE, f) for f in SERVING_SOURCES], extra_cflags=["-O2", "-std=c++17"] + flag,
+      extra_cuda_cflags=NVCC_FLAGS + flag, extra_include_paths=[HERE], build_directory=SERVING_DIR, with_cuda=True, verbose=verbose)
+
+
 HOST_DIR = os.path.join(HERE, "host")
 HOST_BUILD_DIR = os.path.join(HERE, "build_host")
 HOST_EXT_NAME = "maxtext_b200_host"
@@ -81,6 +99,10 @@ if __name__ == "__main__":
   if "--sanitize" in sys.argv:
     build_host_extension_sanitized(verbose="-q" not in sys.argv)
     print("built", os.path.join(HOST_ASAN_BUILD_DIR, HOST_ASAN_EXT_NAME + ".so"))
+    sys.exit(0)
+  if "--serving" in sys.argv:
+    build_serving_extension(verbose="-q" not in sys.argv)
+    print("built", os.path.join(SERVING_DIR, SERVING_NAME + ".so"))
     sys.exit(0)
   build_host_extension(verbose="-q" not in sys.argv)
   build_extension(verbose="-q" not in sys.argv)

@@ -76,6 +76,8 @@ def decode(config, prompt: str | None = None, engine: MaxEngine | None = None) -
 
 def main(argv=None):
   argv = list(sys.argv if argv is None else argv)
+  from ..ops import backend
+  backend.serving_only()
   config = pyconfig.initialize(argv)
   text = decode(config)
   max_logging.log(f"Input `{config.prompt}` -> `{text}`")

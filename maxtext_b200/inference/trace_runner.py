@@ -55,9 +55,11 @@ class TraceRunner:
 
 def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str = "cuda"):
   from ..config import pyconfig
+  from ..ops import backend
   from .maxengine import MaxEngine
   if device == "cuda" and not torch.cuda.is_available():
     raise RuntimeError("a CUDA device is needed")
+  backend.serving_only()
   if dtype == "float32":
     torch.set_float32_matmul_precision("highest")          # no reduced-precision products
   cfg = pyconfig.initialize(["trace_run", os.path.join(pyconfig.CONFIG_ROOT, "base.yml"), f"model_dir={model_dir}"], num_devices=1, dtype=dtype,

@@ -19,15 +19,26 @@ EXT_NAME = "maxtext_b200_C"
 BUILD_DIR = os.path.normpath(os.path.join(os.path.dirname(__file__), "..", "csrc", "build"))
 
 
+_SERVING_ONLY = False
+
+
 def so_path() -> str:
   return os.path.join(BUILD_DIR, EXT_NAME + ".so")
 
 
+def serving_only():
+  """Called by command lines that only run inference: when no full library has been built, the serving part of it is compiled and
+  loaded instead (`csrc.build.build_serving_extension`)."""
+  global _SERVING_ONLY
+  _SERVING_ONLY = True
+
+
 def _import_so(path: str):
-  spec = importlib.util.spec_from_file_location(EXT_NAME, path)
+  name = os.path.splitext(os.path.basename(path))[0]
+  spec = importlib.util.spec_from_file_location(name, path)
   mod = importlib.util.module_from_spec(spec)
   spec.loader.exec_module(mod)
-  sys.modules[EXT_NAME] = mod
+  sys.modules[name] = mod
   return mod
 
 
@@ -42,6 +53,9 @@ def ext(required: bool | None = None):
     return None
   _TRIED = True
   path = so_path()
+  if _SERVING_ONLY and not os.path.isfile(path):
+    from ..csrc import build as _build
+    path = os.path.join(_build.SERVING_DIR, _build.SERVING_NAME + ".so")
   err = None
   if os.path.isfile(path):
     try:
@@ -52,7 +66,7 @@ def ext(required: bool | None = None):
   if required:
     if os.environ.get("MAXTEXT_B200_JIT_BUILD", "1") == "1" and err is None:
       from ..csrc import build as _build
-      _build.build_extension(verbose=False)
+      (_build.build_serving_extension if _SERVING_ONLY else _build.build_extension)(verbose=False)
       _EXT = _import_so(path)
       return _EXT
     raise RuntimeError(
