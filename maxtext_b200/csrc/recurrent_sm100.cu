@@ -8,6 +8,7 @@
 //  * scan (prompts): S stays in registers over the whole prompt. The columns of S never mix, so a CTA takes 16 of them and a warp 4;
 //    eight lanes share a column and reduce with three shuffles.
 //  * the elementwise parts of a prompt: convolution, per-channel decay, head norm with output gate.
+// The decay multiplies as S + (g - 1) S with g - 1 from expm1: a slow decay is applied thousands of times, and the rounding of g itself would add up.
 // Rows of a batch read the state of slot slot_ids[b] (zeros when lengths[b] == 0) and stop after new_lens[b] tokens.
 #include "serving_common.cuh"
 #include "warp_mma.cuh"
@@ -60,7 +61,7 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
   float* tile = sm;                                     // [dk * dv]
   float* qs = tile + (TILE ? dk * dv : 0);              // [rows * nrg] each
   float* ks = qs + rows * nrg;
-  float* al = ks + rows * nrg;                          // alpha (GLA)
+  float* al = ks + rows * nrg;                          // alpha - 1 (GLA)
   float* redk = al + (DELTA ? 0 : rows * nrg);          // [DEC_NT]
   float* redq = redk + DEC_NT;
   float* wsum = redq + DEC_NT;                          // [DEC_NT / 32]
@@ -115,7 +116,7 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
 #pragma unroll
         for (int e = 0; e < 8; ++e) z += wv[e] * to_f(lo[j + e]);
       }
-      al[i] = expf(log_sigmoid_f(z) * gl.inv_tau);
+      al[i] = expm1f(log_sigmoid_f(z) * gl.inv_tau);
       qs[i] = to_f(xr[(long)kh * dk + i]);
       ks[i] = to_f(xr[(long)H * dk + kh * dk + i]);
     }
@@ -136,7 +137,7 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
   qk *= rq * rk;
   if (!DELTA) {                                         // S_new^T q = S^T (alpha q) + (k . q) v
     __syncthreads();
-    for (int i = tid; i < dk; i += DEC_NT) qs[i] *= al[i];
+    for (int i = tid; i < dk; i += DEC_NT) qs[i] += al[i] * qs[i];
   }
   for (int j = 0; j < r; ++j) {
     const int h = kh * r + j;
@@ -163,23 +164,25 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
       if (DELTA) sk += redk[g * dvp + c];
       sq += redq[g * dvp + c];
     }
-    float decay = 1.f, u = 0.f;
+    float dm1 = 0.f, u = 0.f;
     const float v = col ? vs[j * dv + c] : 0.f;
     if constexpr (DELTA) {
       const T* bb = d.ba + b * d.ldb + (long)kh * 2 * r;
-      decay = expf(log_decay(to_f(bb[r + j]), to_f(d.A_log[h]), to_f(d.dt_bias[h])));
-      u = beta_gate(to_f(bb[j])) * (v - decay * rk * sk);
+      dm1 = expm1f(log_decay(to_f(bb[r + j]), to_f(d.A_log[h]), to_f(d.dt_bias[h])));
+      sk += dm1 * sk;
+      sq += dm1 * sq;
+      u = beta_gate(to_f(bb[j])) * (v - rk * sk);
     } else {
       u = v;
     }
-    const float o = col ? decay * rq * sq + qk * u : 0.f;
+    const float o = col ? rq * sq + qk * u : 0.f;
     const float ku = rk * u;
     if (col) {
       float* wp = gp + (long)row0 * dv + c;
 #pragma unroll 8
       for (int i = 0; i < nrows; ++i) {
         const float s = read ? sp[(long)i * dv] : 0.f;
-        wp[(long)i * dv] = (DELTA ? decay : al[row0 + i]) * s + ks[row0 + i] * ku;
+        wp[(long)i * dv] = s + (DELTA ? dm1 : al[row0 + i]) * s + ks[row0 + i] * ku;
       }
     }
     // head norm over dv and output gate
@@ -328,7 +331,7 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
   float* ks = qs + SCAN_TC * 8 * GS;
   float* as = ks + SCAN_TC * 8 * GS;                     // GLA only
   float* vs = as + (DELTA ? 0 : SCAN_TC * 8 * GS);       // [TC][16]
-  float* sc = vs + SCAN_TC * SCAN_COLS;                  // [TC][4]: decay, beta, rq, k.q (normalised)  (and rk folded into ks)
+  float* sc = vs + SCAN_TC * SCAN_COLS;                  // [TC][4]: decay - 1, beta, rq, k.q (normalised); rk is folded into ks
   const int c0 = blockIdx.x * SCAN_COLS, cl = warp * 4 + (lane & 3), c = c0 + cl, rg = lane >> 2;
   const bool col = c < dv;
   const long slot = a.slot_ids[b];
@@ -352,7 +355,7 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
       const int at = t * 8 * GS + (e / RPT) * GS + e % RPT;
       qs[at] = to_f(q[row * ldx + (long)kh * dk + e]);
       ks[at] = to_f(k[row * ldx + (long)kh * dk + e]);
-      if (!DELTA) as[at] = expf(log_alpha[row * (long)H * dk + (long)h * dk + e]);
+      if (!DELTA) as[at] = expm1f(log_alpha[row * (long)H * dk + (long)h * dk + e]);
     }
     for (int i = tid; i < m * SCAN_COLS; i += SCAN_NT) {
       const int t = i / SCAN_COLS, e = c0 + i % SCAN_COLS;
@@ -373,7 +376,7 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
         for (int e = lane; e < dk; e += 32) ks[t * 8 * GS + (e / RPT) * GS + e % RPT] *= rk;
         if (lane == 0) {
           const T* bb = ba + ((long)b * a.S + t0 + t) * ldb + (long)kh * 2 * r + (h - kh * r);
-          sc[t * 4] = expf(log_decay(to_f(bb[r]), to_f(A_log[h]), to_f(dt_bias[h])));
+          sc[t * 4] = expm1f(log_decay(to_f(bb[r]), to_f(A_log[h]), to_f(dt_bias[h])));
           sc[t * 4 + 1] = beta_gate(to_f(bb[0]));
         }
       }
@@ -388,7 +391,7 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
 #pragma unroll
       for (int i = 0; i < RPT; ++i) {
         if constexpr (DELTA) { sk += S[i] * kt[i]; sq += S[i] * qt[i]; }
-        else { S[i] *= at[i]; sq += S[i] * qt[i]; }
+        else { S[i] += at[i] * S[i]; sq += S[i] * qt[i]; }
       }
 #pragma unroll
       for (int w = 4; w <= 16; w <<= 1) {
@@ -396,14 +399,18 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
         sq += __shfl_xor_sync(0xffffffffu, sq, w);
       }
       const float rq = sc[t * 4 + 2], kq = sc[t * 4 + 3];
-      float u = vs[t * SCAN_COLS + cl], decay = 1.f;
+      float u = vs[t * SCAN_COLS + cl];
       if constexpr (DELTA) {
-        decay = sc[t * 4];
-        u = sc[t * 4 + 1] * (u - decay * sk);
+        const float dm1 = sc[t * 4];
+        sk += dm1 * sk;
+        sq += dm1 * sq;
+        u = sc[t * 4 + 1] * (u - sk);
+#pragma unroll
+        for (int i = 0; i < RPT; ++i) S[i] += dm1 * S[i];
       }
 #pragma unroll
-      for (int i = 0; i < RPT; ++i) S[i] = (DELTA ? decay * S[i] : S[i]) + kt[i] * u;
-      if (rg == 0 && col) o[((long)b * a.S + t0 + t) * (long)H * dv + (long)h * dv + c] = from_f<T>(decay * rq * sq + kq * u);
+      for (int i = 0; i < RPT; ++i) S[i] += kt[i] * u;
+      if (rg == 0 && col) o[((long)b * a.S + t0 + t) * (long)H * dv + (long)h * dv + c] = from_f<T>(rq * sq + kq * u);
     }
   }
   // padding positions of the output are read by the norm kernel: give them a value
