@@ -248,7 +248,11 @@ def main():
   args = ap.parse_args()
   if args.serving:
     from maxtext_b200.benchmarks import serving_bench
-    return serving_bench.main(args.serving_models, args.serving_lengths, args.serving_slots, args.serving_context, max(args.steps, 5))
+    sampler = ClockSampler(0 if "CUDA_VISIBLE_DEVICES" not in os.environ else int(os.environ["CUDA_VISIBLE_DEVICES"].split(",")[0]))
+    sampler.start()
+    rc = serving_bench.main(args.serving_models, args.serving_lengths, args.serving_slots, args.serving_context, max(args.steps, 5))
+    print(json.dumps({"clocks": sampler.stop()}))
+    return rc
   preset = PRESETS[args.config]
   args.model = args.model or preset["model"]
   args.seq = args.seq or preset["seq"]

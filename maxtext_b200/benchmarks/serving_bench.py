@@ -6,11 +6,16 @@
   decode:  tokens/s of a full decode state per slot count, every slot holding `context` tokens, CUDA-graph replay
   kernels: device microseconds per launch by kernel (PyTorch profiler, a separate untimed pass), one prompt and one decode step
 
+and one last line `rooflines`: every serving kernel at silinex-1b's layer sizes (8192 prompt tokens; 128 sequences with 2048 cached tokens),
+its time by CUDA events with L2 flushed, its algorithmic bytes or products, and the fraction of the measured copy bandwidth or GEMM rate,
+beside the like operation of the models that existed before (`like`).
+
 Weights are random; the work does not depend on their values. The models:
 
   silinex-1b   the catalog entry: gated delta, sliding-window latent attention and gated linear attention layers in turn
   mla-1b       the same width, depth and feed-forward size with the DeepSeek block (latent attention in every layer, gated MLP of equal size)
   llama-1b     the same with grouped-query attention
+  silinex-5b, mla-5b   the same two at width 4096, 32 heads, 24 layers
 """
 from __future__ import annotations
 
@@ -20,31 +25,51 @@ import statistics
 
 import torch
 
+def _silinex(width, heads, ff, layers, q_rank):
+  """Gated delta, latent attention (window 2048) and gated linear attention layers in turn, sized by `heads` of 128 lanes."""
+  mlp = {"kind": "dense", "ff": ff}
+  kinds = [
+      {"type": "delta", "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}, "mlp": mlp},
+      {"type": "latent_attention", "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": 512, "scale": 192 ** -0.5,
+                                             "mask": {"size": 2048}, "rot": {"base": 500000.0, "dims": 64}}, "mlp": mlp},
+      {"type": "gla", "mixer": {"heads": heads, "dim": 64, "vdim": 128, "tau": 16.0, "decay_rank": 32}, "mlp": mlp}]
+  return dict(decoder_block="silinex", base_emb_dim=width, base_num_decoder_layers=layers, layer_specs=[kinds[i % 3] for i in range(layers)],
+              mlp_activations=["gelu_exact"], residual_multiplier=0.6, vocab_size=65536, logits_via_embedding=False)
+
+
+def _plain(width, heads, ff, layers, q_rank=0):
+  """The same width, depth and feed-forward weights (gated, so two thirds of the hidden width) with one attention kind in every layer."""
+  keys = dict(base_emb_dim=width, base_num_query_heads=heads, base_num_decoder_layers=layers, base_mlp_dim=-(-2 * ff // 3 // 64) * 64, vocab_size=65536,
+              logits_via_embedding=False)
+  if q_rank:
+    return dict(keys, decoder_block="deepseek", attention_type="mla", base_num_kv_heads=heads, first_num_dense_layers=layers, q_lora_rank=q_rank,
+                kv_lora_rank=512, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128)
+  return dict(keys, decoder_block="llama2", base_num_kv_heads=heads // 2, head_dim=128)
+
+
 MODELS = {
-    "silinex-1b": ["model_name=silinex-1b"],
-    "mla-1b": ["decoder_block=deepseek", "attention_type=mla", "base_emb_dim=2048", "base_num_query_heads=16", "base_num_kv_heads=16", "first_num_dense_layers=18",
-               "base_num_decoder_layers=18", "base_mlp_dim=5461", "q_lora_rank=768", "kv_lora_rank=512", "qk_nope_head_dim=128",
-               "qk_rope_head_dim=64", "v_head_dim=128", "vocab_size=65536", "logits_via_embedding=false"],
-    "llama-1b": ["decoder_block=llama2", "base_emb_dim=2048", "base_num_query_heads=16", "base_num_kv_heads=8", "head_dim=128",
-                 "base_num_decoder_layers=18", "base_mlp_dim=5461", "vocab_size=65536", "logits_via_embedding=false"],
+    "silinex-1b": dict(model_name="silinex-1b"),
+    "mla-1b": _plain(2048, 16, 8192, 18, 768),
+    "llama-1b": _plain(2048, 16, 8192, 18),
+    "silinex-5b": _silinex(4096, 32, 16384, 24, 1536),
+    "mla-5b": _plain(4096, 32, 16384, 24, 1536),
 }
 
 
 def make_engine(name: str, max_len: int, slots: int = 1):
   from ..config import pyconfig
   from ..inference.maxengine import MaxEngine
-  over = [o if not o.startswith("base_mlp_dim=") else f"base_mlp_dim={-(-int(o.split('=')[1]) // 64) * 64}" for o in MODELS[name]]
-  cfg = pyconfig.initialize(["serving", os.path.join(pyconfig.CONFIG_ROOT, "base.yml")] + over +
-                            [f"max_target_length={max_len}", f"max_prefill_predict_length={max_len - 64}", f"per_device_batch_size={slots}", "dtype=bfloat16",
-                             "weight_dtype=bfloat16", "hardware=gpu", "enable_checkpointing=false", "log_config=false", "cuda_graphs=true",
-                             "decode_sampling_strategy=greedy"], num_devices=1)
+  cfg = pyconfig.initialize(["serving", os.path.join(pyconfig.CONFIG_ROOT, "base.yml")], num_devices=1, max_target_length=max_len,
+                            max_prefill_predict_length=max_len - 64, per_device_batch_size=slots, dtype="bfloat16", weight_dtype="bfloat16", hardware="gpu",
+                            enable_checkpointing=False, log_config=False, cuda_graphs=True, decode_sampling_strategy="greedy", **MODELS[name])
   eng = MaxEngine(cfg, device=torch.device("cuda", torch.cuda.current_device()))
   eng.load_params()
   return eng
 
 
-def _events(fn, iters: int, warmup: int = 3) -> float:
-  """Median device milliseconds of fn over `iters` calls, L2 flushed in between."""
+def _events(fn, iters: int, warmup: int = 3, drain: bool = True) -> float:
+  """Median device milliseconds of fn over `iters` calls, L2 flushed in between. `drain` waits for the flush before fn is issued, so that
+  the host's part of a multi-launch fn counts; without it a single kernel is queued behind the flush and timed alone."""
   flush = torch.empty(256 * 1024 * 1024, dtype=torch.uint8, device="cuda")
   for _ in range(warmup):
     fn()
@@ -52,7 +77,8 @@ def _events(fn, iters: int, warmup: int = 3) -> float:
   for _ in range(iters):
     flush.zero_()
     a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-    torch.cuda.synchronize()
+    if drain:
+      torch.cuda.synchronize()
     a.record()
     fn()
     b.record()
@@ -120,8 +146,102 @@ def run(names, lengths, slot_counts, context: int, iters: int = 10, kernels: boo
   return rows
 
 
+def rooflines(iters: int = 10) -> dict:
+  """name -> {us, bytes | flops, fraction of roofline, like}."""
+  from ..layers.gdn import gated_delta_chunked, gated_delta_recurrent
+  from ..ops import backend
+  E = backend.ext(required=True)
+  root = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+  peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+  if os.path.isfile(os.path.join(root, "MEASURED_PEAKS.json")):
+    with open(os.path.join(root, "MEASURED_PEAKS.json"), encoding="utf-8") as fh:
+      peaks = {**json.load(fh), "source": "measured"}
+  bf, dev = torch.bfloat16, "cuda"
+  rows = {}
+
+  def t(*shape, dtype=bf):
+    return torch.randn(*shape, dtype=dtype, device=dev) if dtype.is_floating_point else torch.zeros(*shape, dtype=dtype, device=dev)
+
+  def add(name, fn, nbytes=0, flops=0, like="", it=iters):
+    us = _events(fn, it, 2, drain=False) * 1e3
+    ideal = max(nbytes / (peaks["hbm_gbs"] * 1e3), flops / (peaks["bf16_tflops"] * 1e6))
+    rows[name] = {"us": round(us, 1), "bytes": int(nbytes), "flops": int(flops), "fraction": round(ideal / us, 3), "like": like}
+
+  def longs(n, v=0):
+    return torch.full((n,), v, dtype=torch.long, device=dev)
+  N, D, F_ = 8192, 2048, 8192
+  hk, hv, dk, dv = 8, 16, 128, 128
+  # ---- prompts
+  x32, b, w, y = t(N, D, dtype=torch.float32), t(N, D), t(D), t(N, D)
+  add("residual_norm", lambda: E.residual_norm(x32, b, w, 0.5, w, y, 1e-6, 1e-6, 1.0), 12 * N * D, like="rmsnorm")
+  add("rmsnorm", lambda: E.rmsnorm_fwd(b, w, 1e-6, 0.0, y, None), 4 * N * D)
+  h, h2 = t(N, F_), t(N, F_)
+  add("act gelu_exact", lambda: E.act_fwd(h.view(-1), h2.view(-1), 4), 4 * N * F_, like="gated_act")
+  add("gated_act", lambda: E.gated_act_fwd(h, h2.view(-1)[: N * F_ // 2].view(N, F_ // 2), 0), 3 * N * F_)
+  cd, per = 2 * hk * dk + hv * dv, 2 * hk * dk + 2 * hv * dv
+  qkvz, ba, cw, mixed, o = t(N, per), t(N, 2 * hv), t(4, cd), t(N, cd), t(N, hv * dv)
+  conv, rec, one, A, nw = t(1, 3, cd, dtype=torch.float32), t(1, hv, dk, dv, dtype=torch.float32), longs(1), t(hv), t(dv)
+  add("delta_conv", lambda: E.delta_conv(qkvz, cw, hk, hv, dk, dv, N, conv, one, one, None, mixed), 4 * N * cd, like="rmsnorm")
+  add("delta_chunks (both kernels)", lambda: E.delta_chunks(mixed, ba, A, A, hk, hv, dk, dv, N, rec, one, one, None, o), 2 * N * (cd + hv * dv + 2 * hv),
+      like="gated delta composition")
+  q, k, v = (t(1, N, hv, d) for d in (dk, dk, dv))
+  g, be = -torch.rand(1, N, hv, device=dev), torch.rand(1, N, hv, device=dev)
+  add("gated delta composition", lambda: gated_delta_chunked(q, k, v, g, be, 64), 2 * N * (cd + hv * dv + 2 * hv), it=3)
+  add("gated_head_norm", lambda: E.gated_head_norm(o, qkvz, hv, dv, 2, 512, 768, nw, 1e-6, y.view(-1)[: N * hv * dv].view(N, hv * dv)), 6 * N * hv * dv,
+      like="rmsnorm")
+  H, gk, rank = 16, 64, 32
+  gx, la, dw, db = t(N, 2 * H * (gk + dv) + rank), -torch.rand(N, H * gk, device=dev) * 0.05, t(H * gk, rank), t(H * gk)
+  rec2 = t(1, H, gk, dv, dtype=torch.float32)
+  add("gla_decay", lambda: E.gla_decay(gx, 2 * H * (gk + dv), dw, db, 16.0, la), 2 * N * rank + 4 * N * H * gk, like="rmsnorm")
+  la.uniform_(-0.05, 0.0)
+  add("gla_chunks (both kernels)", lambda: E.gla_chunks(gx, la, H, gk, dv, N, rec2, one, one, None, o), N * (2 * 2 * H * (gk + dv) + 4 * H * gk),
+      like="gated delta composition")
+  nope, dr, vd, R, Q = 128, 64, 128, 512, 768
+  inv, pos = torch.rand(dr // 2, device=dev), torch.arange(N, device=dev)
+  qa, kva, qw, kw, cq, lat, kr = t(N, Q), t(N, R + dr), t(Q), t(R), t(N, Q), t(N, R), t(N, dr)
+  c_lat, c_kr = t(1, N, R), t(1, N, dr)
+  add("mla_prep", lambda: E.mla_prep(qa, qw, kva, kw, 1e-6, pos, inv, True, cq, lat, kr, c_lat, c_kr, one, one, None), 2 * N * (2 * Q + 3 * (R + dr)),
+      like="rmsnorm")
+  qh, kv = t(N, H, nope + dr), t(N, H, nope + vd)
+  qp, kp, vp = t(N, H, 192), t(N, H, 192), t(N, H, 128)
+  add("mla_pack (both kernels)", lambda: E.mla_pack(qh, kv, kr, pos, inv, True, nope, vd, qp, kp, vp), 2 * N * H * (2 * 192 + 256 + 192 + 128), like="rmsnorm")
+  from ..ops import functional as F
+  with torch.no_grad():
+    win = 2048
+    pairs = N * win - win * win // 2
+    add("flash forward, window 2048", lambda: F.attention_fwd(qp[None], kp[None], vp[None], None, None, 0.1, 0.0, win), 0, 2 * pairs * H * (192 + 128),
+        like="flash forward, causal")
+    add("flash forward, causal", lambda: F.attention_fwd(qp[None], kp[None], vp[None], None, None, 0.1, 0.0, 0), 0, N * N * H * (192 + 128))
+  # ---- decoding: 128 sequences, 2048 cached tokens
+  B, L = 128, 2048
+  ids, lens = torch.arange(B, device=dev), longs(B, L - 1)
+  dconv, drec, dout = t(B, 3, cd, dtype=torch.float32), t(B, hv, dk, dv, dtype=torch.float32), t(B, hv * dv)
+  st = 8 * B * hv * dk * dv + 2 * B * (per + hv * dv) + 8 * B * 3 * cd
+  add("delta_decode", lambda: E.delta_decode(qkvz[:B], ba[:B], cw, A, A, nw, 1e-6, hk, hv, dk, dv, dconv, drec, ids, lens, dout), st,
+      like="gated delta step composition")
+  q1, k1, v1 = (t(B, 1, hv, d) for d in (dk, dk, dv))
+  g1, b1 = -torch.rand(B, 1, hv, device=dev), torch.rand(B, 1, hv, device=dev)
+  add("gated delta step composition", lambda: gated_delta_recurrent(q1, k1, v1, g1, b1, drec), 8 * B * hv * dk * dv)
+  grec = t(B, H, gk, dv, dtype=torch.float32)
+  add("gla_decode", lambda: E.gla_decode(gx[:B], dw, db, nw, 1e-6, 16.0, H, gk, dv, grec, ids, lens, dout), 8 * B * H * gk * dv, like="gated delta step composition")
+  lc, kc, qd = t(B, L, R), t(B, L, dr), t(B, H, R + dr)
+  sp = E.mla_decode_splits(B, H, L)
+  part, ml = t(B, H, sp, R, dtype=torch.float32), torch.rand(B, H, sp, 2, device=dev) + 0.1
+  add("mla_decode_attn", lambda: E.mla_decode_attn(qd, lc, kc, ids, lens, 0.1, 2048, sp, part, ml), 2 * B * L * (R + dr), like="decode_attention")
+  kc8, vc8, q8, o8 = t(B, L, 8, 128), t(B, L, 8, 128), t(B, 16, 128), t(B, 16, 128)
+  i32, l32 = ids.int(), (lens + 1).int()
+  add("decode_attention", lambda: E.decode_attention(q8, kc8, vc8, i32, l32, o8, 1.0, 0.0, 0, 1), 2 * 2 * B * L * 8 * 128)
+  wb, qin, vout = t(H * (nope + vd), R), t(B, H, nope + dr), t(B, H, vd)
+  add("mla_absorb", lambda: E.mla_absorb(qin, wb, pos[:B], inv, True, nope, vd, qd), 2 * (H * nope * R + B * H * (nope + 2 * dr + R)), like="gemm, M = 128")
+  add("mla_value_up", lambda: E.mla_value_up(part, ml, wb, nope, vout), 2 * H * vd * R + 4 * B * H * R + 2 * B * H * vd, like="gemm, M = 128")
+  ga, gw, go = t(B, 2048), t(2048, 2048), t(B, 2048)
+  add("gemm, M = 128", lambda: F.mm(ga, gw, False, True, out=go), 2 * (2048 * 2048 + 2 * B * 2048))
+  return {"rooflines": rows, "hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "peaks": peaks["source"]}
+
+
 def main(models: str = "", lengths: str = "512,2048,8192", slots: str = "1,32,128", context: int = 2048, iters: int = 10) -> int:
   names = [m for m in models.split(",") if m] or list(MODELS)
   for row in run(names, [int(x) for x in lengths.split(",")], [int(x) for x in slots.split(",")], context, iters):
     print(json.dumps(row))
+  print(json.dumps(rooflines(iters)))
   return 0

@@ -317,6 +317,55 @@ __global__ void __launch_bounds__(128) gla_decay_kernel(const T* __restrict__ lo
   }
 }
 
+// The same with the product on tensor cores (bf16): grid (ceil(C / 64), ceil(N / 64)), 128 threads; rows of lo and w start on 16 bytes.
+__global__ void __launch_bounds__(128) gla_decay_tc_kernel(const __nv_bfloat16* __restrict__ lo, long ldx, const __nv_bfloat16* __restrict__ w,
+                                                           const __nv_bfloat16* __restrict__ bias, int rank, float inv_tau, float* __restrict__ out, long N,
+                                                           int C) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int kp = (rank + 15) & ~15, LD = kp + 8, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c0 = blockIdx.x * 64;
+  const long n0 = (long)blockIdx.y * 64;
+  __nv_bfloat16* as = reinterpret_cast<__nv_bfloat16*>(raw);       // [64][LD]
+  __nv_bfloat16* ws = as + 64 * LD;
+  for (int i = tid; i < 64 * (kp / 8); i += 128) {
+    const int r = i / (kp / 8), k = (i % (kp / 8)) * 8;
+    const bool ka = k < rank, na = n0 + r < N, ca = c0 + r < C;
+    la_cp_async16(as + r * LD + k, lo + (na ? n0 + r : 0) * ldx + (ka ? k : 0), ka && na ? 16 : 0);
+    la_cp_async16(ws + r * LD + k, w + (long)(ca ? c0 + r : 0) * rank + (ka ? k : 0), ka && ca ? 16 : 0);
+  }
+  la_commit();
+  float acc[8][4];
+#pragma unroll
+  for (int n = 0; n < 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = c0 + n * 8 + (lane & 3) * 2 + (e & 1);
+      acc[n][e] = c < C ? to_f(bias[c]) : 0.f;
+    }
+  la_wait<0>();
+  __syncthreads();
+  for (int k = 0; k < kp; k += 16) {
+    unsigned fa[4];
+    la_ldm4(fa, as + (warp * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+#pragma unroll
+    for (int n = 0; n < 8; n += 2) {
+      unsigned fb[4];
+      la_ldm4(fb, ws + (n * 8 + (lane & 7) + ((lane >> 4) << 3)) * LD + k + ((lane >> 3) & 1) * 8);
+      la_mma(acc[n], fa, fb[0], fb[1]);
+      la_mma(acc[n + 1], fa, fb[2], fb[3]);
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const long n = n0 + warp * 16 + (lane >> 2) + e * 8;
+    if (n >= N) continue;
+#pragma unroll
+    for (int x = 0; x < 8; ++x) {
+      const int c = c0 + x * 8 + (lane & 3) * 2;           // C is even
+      if (c < C) *reinterpret_cast<float2*>(out + n * C + c) = make_float2(log_sigmoid_f(acc[x][2 * e]) * inv_tau, log_sigmoid_f(acc[x][2 * e + 1]) * inv_tau);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ scan over a prompt
 // grid (ceil(dv / 16), heads, B). q / k of token n sit at q[n * ldq + (h / r) * dk]; likewise v and, for GLA, log_alpha (fp32).
 template <typename T, bool DELTA, int RPT>
@@ -583,6 +632,12 @@ extern "C" int mt_gla_decay(int f32, const void* lo, long ldx, const void* w, co
                             cudaStream_t st) {
   if (N <= 0) return 0;
   if (rank % 8) return -1;
+  if (!f32 && C % 2 == 0 && ldx % 8 == 0 && reinterpret_cast<uintptr_t>(lo) % 16 == 0 && rank <= 160) {
+    const size_t smem = 2 * 2 * 64 * (size_t)(((rank + 15) & ~15) + 8);
+    gla_decay_tc_kernel<<<dim3((C + 63) / 64, (unsigned)((N + 63) / 64)), 128, smem, st>>>((const __nv_bfloat16*)lo, ldx, (const __nv_bfloat16*)w,
+                                                                                       (const __nv_bfloat16*)bias, rank, inv_tau, out, N, C);
+    return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  }
   const dim3 grid((C + 127) / 128, (unsigned)((N + 31) / 32));
   if (f32) gla_decay_kernel<float><<<grid, 128, 0, st>>>((const float*)lo, ldx, (const float*)w, (const float*)bias, rank, inv_tau, out, N, C);
   else gla_decay_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>((const __nv_bfloat16*)lo, ldx, (const __nv_bfloat16*)w, (const __nv_bfloat16*)bias, rank,

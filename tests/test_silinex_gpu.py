@@ -156,6 +156,19 @@ def test_gla_scan(B, S, H, dk, dv, lens, decay):
   assert _status() == 0
 
 
+@pytest.mark.parametrize("N, C, rank, at", [(70, 96, 32, 64), (5, 30, 8, 13), (129, 128, 24, 16), (64, 66, 40, 8)])
+def test_gla_decay(N, C, rank, at):
+  from maxtext_b200.ops import backend
+  E = backend.ext(required=True)
+  g = torch.Generator().manual_seed(5)
+  for dtype in (torch.float32, torch.bfloat16):
+    x, w, b = ((torch.randn(*s, generator=g) * 3).to(dtype).cuda() for s in ((N, at + rank + 8), (C, rank), (C,)))
+    out = torch.empty(N, C, device="cuda")
+    E.gla_decay(x, at, w, b, 8.0, out)
+    want = torch.nn.functional.logsigmoid(x[:, at:at + rank].double() @ w.double().T + b.double()) / 8.0
+    assert torch.allclose(out.double(), want, rtol=2e-5, atol=1e-6), dtype
+
+
 @pytest.mark.parametrize("H, R, dr, window, lens", [(5, 128, 32, 0, [1, 300, 64]), (16, 512, 64, 100, [101, 100, 700]), (33, 64, 16, 65, [65, 66, 1]),
                                                     (3, 40, 6, 9, [9, 10, 30]), (4, 448, 48, 0, [65, 128, 129])])
 def test_latent_decode_attention(H, R, dr, window, lens):
