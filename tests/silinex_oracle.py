@@ -9,7 +9,7 @@ import torch
 
 
 def rms(x, eps):
-  """x divided by the root of its mean square over the last dimension, eps inside the root."""
+  """RMS normalisation over the last dimension; eps is added to the mean square."""
   return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
 
 
