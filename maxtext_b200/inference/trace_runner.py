@@ -17,6 +17,8 @@ import sys
 
 import torch
 
+from ..ops import backend
+
 
 class TraceRunner:
   """Maps request ids to slots of a decode state; the state grows when a batch needs more slots than it has and none is in use."""
@@ -46,6 +48,8 @@ class TraceRunner:
       want = [list(e.get("want") or []) for e in entries]
       logits = self.engine.extend(self.state, [self.slot_of[e["id"]] for e in entries], [e["tokens"] for e in entries], want)
       out = logits.float().cpu() if any(want) else None
+      if self.engine.device.type == "cuda" and backend.ext(required=True).kernel_status(True) != 0:
+        raise RuntimeError("a kernel gave up a bounded wait: the results of this step are not valid")
     for rid in end:
       slot = self.slot_of.pop(rid)
       self.engine.free_slot(self.state, slot)
@@ -55,7 +59,6 @@ class TraceRunner:
 
 def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str = "cuda"):
   from ..config import pyconfig
-  from ..ops import backend
   from .maxengine import MaxEngine
   if device == "cuda" and not torch.cuda.is_available():
     raise RuntimeError("a CUDA device is needed")

@@ -281,6 +281,16 @@ class _CollapsingNorm:
     return self.norm(x)
 
 
+class _StreamNorm:
+  """Final norm of a model with an fp32 residual stream: reads fp32, returns the compute dtype."""
+
+  def __init__(self, norm):
+    self.norm, self.scale, self.bias, self.eps, self.offset = norm, norm.scale, norm.bias, norm.eps, norm.offset
+
+  def __call__(self, x):
+    return F.stream_norm(x, self.norm, self.scale.data.dtype)
+
+
 class MTPLayer:
   """One multi-token-prediction module (src/maxtext/layers/multi_token_prediction.py:160-310): the previous hidden state and
   the embedding of the token one step further ahead are normalised separately, concatenated [embedding | hidden], projected
@@ -381,7 +391,7 @@ class Transformer:
     if self.mhc_k > 1 and c.decoder_block == "deepseek4":
       from ..layers.mhc import HyperHead
       hyper_head = HyperHead(hb.sub("decoder"), c, "hc_head")
-    self.final_norm = _CollapsingNorm(norm, hyper_head) if self.mhc_k > 1 else norm
+    self.final_norm = _CollapsingNorm(norm, hyper_head) if self.mhc_k > 1 else (_StreamNorm(norm) if self.family.residual_fp32 else norm)
     self.logits_dense = None
     if not c.logits_via_embedding:
       self.logits_dense = hb.sub("decoder", "logits_dense").linear("kernel", (c.emb_dim,), (c.vocab_size,),
@@ -515,11 +525,8 @@ class Transformer:
 
   def logits(self, x, normed=None):
     """`normed`: the final norm's output when the last layer already produced it (fp32 residual streams)."""
-    if self.family.residual_fp32:
-      h = normed if normed is not None else F.stream_norm(x, self.final_norm, self.final_norm.scale.data.dtype)
-      return F.head_logits(h, self.head_param(), self.config.final_logits_soft_cap, self.head_logit_scale(), fp32_out=True)
-    h = self.final_norm(x)
-    return F.head_logits(h, self.head_param(), self.config.final_logits_soft_cap, self.head_logit_scale())
+    h = normed if normed is not None else self.final_norm(x)
+    return F.head_logits(h, self.head_param(), self.config.final_logits_soft_cap, self.head_logit_scale(), fp32_out=self.family.residual_fp32)
 
   # ------------------------------------------------------------------ plain forward (eval / inference / tests)
   @torch.no_grad()

@@ -263,3 +263,20 @@ def test_every_kernel_path_is_taken_in_bf16(tmp_path):
   before = F.attention_fallbacks()
   M.run_pieces(eng, M.prompt(60, sp), [30, 20, 1])
   assert F.attention_fallbacks() == before
+
+
+def test_training_step_in_bf16(tmp_path):
+  """The layers train through their differentiable forms, with the fp32 stream crossing units."""
+  from helpers import BASE_YML
+  from maxtext_b200.config import pyconfig
+  from maxtext_b200.input_pipeline.synthetic import SyntheticDataIterator
+  from maxtext_b200.train.engine import TrainEngine
+  sp = M.spec([M.delta(4, 2, 32, 32, 2), M.gla(2, 32, 32, 2.0, 8), M.latent(4, 32, 32, 64, 64, 64, 40, 0.15)], 256, vocab=512)
+  path = M.write_folder(tmp_path / "m", sp, M.weights(sp))
+  cfg = pyconfig.initialize(["t", BASE_YML, f"model_dir={path}"], num_devices=1, dtype="bfloat16", max_target_length=64, per_device_batch_size=2,
+                            dataset_type="synthetic", hardware="gpu", enable_checkpointing=False, log_config=False, steps=5, learning_rate=5e-3,
+                            warmup_steps_fraction=0.0)
+  eng = TrainEngine(cfg, None, torch.device("cuda", 0))
+  batch = next(SyntheticDataIterator(cfg))
+  losses = [float(eng.train_step(batch)["learning/loss"]) for _ in range(5)]
+  assert losses[-1] < losses[0] and all(x == x for x in losses)
