@@ -300,11 +300,12 @@ def check_misc(t):
 
 
 def check_layer_specs(t):
-  if t.get("decoder_block") != "silinex":
+  from ..models import silinex, tipidra
+  family = {"silinex": silinex, "tipidra": tipidra}.get(t.get("decoder_block"))
+  if family is None:
     return
-  from ..models import silinex
   try:
-    silinex.validate(t)
+    family.validate(t)
   except (KeyError, TypeError, ValueError) as e:
     _fail(f"layer_specs: {e!r}" if isinstance(e, KeyError) else str(e))
 

@@ -201,16 +201,16 @@ def make_caches(model, slots: int, max_len: int, device, quantize: bool = False)
   for layer in model.layers:
     per_layer = []
     for blk in layer.blocks:
-      if seq_size > 1 and blk.plan.attention in ("mla", "gdn", "gla", "compressed"):
+      if seq_size > 1 and blk.plan.attention in ("mla", "gdn", "gla", "ssm", "compressed"):
         raise NotImplementedError("context_autoregressive parallelism splits plain key / value caches only")
       if blk.plan.attention == "mla":
         per_layer.append(MlaLayerCache(slots, max_len, blk.attn.kv_rank, blk.attn.rope_d, dt, device))
       elif blk.plan.attention == "compressed":
         per_layer.append(blk.attn.make_cache(slots, max_len, dt, device))
-      elif blk.plan.attention in ("gdn", "gla"):
+      elif blk.plan.attention in ("gdn", "gla", "ssm"):
         per_layer.append(blk.attn.make_state(slots, device))
       else:
         a = blk.attn
-        per_layer.append(LayerKVCache(slots, max_len, a.hkv_l, a.dh, a.dh, dt, device, quant, **seq))
+        per_layer.append(LayerKVCache(slots, max_len, a.hkv_l, a.dh, a.dv, dt, device, quant, **seq))
     out.append(per_layer)
   return out

@@ -247,7 +247,7 @@ class MaxEngine:
       self._check_length(n, "prefill_concat")
     total = sum(lens)
     kinds = {b.plan.attention for l in self.model.layers for b in l.blocks}
-    packable = total <= self.max_len and not kinds & {"gdn", "gla", "compressed"}
+    packable = total <= self.max_len and not kinds & {"gdn", "gla", "ssm", "compressed"}
     if len(prompts) == 1 or "compressed" in kinds:
       return [self.prefill(p, n)[0] for p, n in zip(prompts, lens)]
     if not packable:

@@ -284,6 +284,17 @@ class Norm:
 
 
 # ------------------------------------------------------------------------------------------ attention (MHA / GQA / MQA)
+@dataclass(frozen=True)
+class HeadSizes:
+  """Sizes of one attention layer; `scale` multiplies q . k, `soft_cap` (0: none) bounds the result."""
+  heads: int
+  kv_heads: int
+  dim: int
+  vdim: int
+  scale: float
+  soft_cap: float = 0.0
+
+
 class Attention:
   """Multi/grouped-query attention with RoPE; the 1/sqrt(head_dim) factor lives in the query weights
   (src/maxtext/layers/attentions.py:663-677) unless QK-norm or an explicit query scalar is used."""
@@ -291,11 +302,19 @@ class Attention:
   def __init__(self, b: Builder, config, name="self_attention", window: int = 0, rope_inv_ts=None, interleaved=False,
                use_rope=True, qk_norm=False, query_scalar: float | None = None, soft_cap: float = 0.0, bias=False,
                rotary_dim=None, sinks=False, l2_qk_norm=False, temperature_tuning=False, chunk=0, out_bias=None, global_qk_norm=False, gated=False, qk_norm_offset=0.0,
-               head_dim: int | None = None, num_kv_heads: int | None = None, share_kv: bool = False, v_norm: str = ""):
+               head_dim: int | None = None, num_kv_heads: int | None = None, share_kv: bool = False, v_norm: str = "",
+               sizes: HeadSizes | None = None):
+    """With `sizes` the layer has head counts and widths of its own (values may be narrower or wider than keys), and `gated` means an
+    output gate from a projection of its own instead of a widened query projection."""
     c = config
     self.config = c
+    if sizes is not None:
+      head_dim, num_kv_heads, query_scalar, soft_cap = sizes.dim, sizes.kv_heads, sizes.scale, sizes.soft_cap
     # gemma4 global layers have their own head width and key/value head count (src/maxtext/models/gemma4.py:186-196)
     self.hq, self.hkv, self.dh, self.d = c.num_query_heads, int(num_kv_heads or c.num_kv_heads), int(head_dim or c.head_dim), c.emb_dim
+    self.dv = self.dh
+    if sizes is not None:
+      self.hq, self.dv = sizes.heads, sizes.vdim
     self.share_kv, self.v_norm = bool(share_kv), str(v_norm or "")
     tp = b.tp_size
     self.hq_l = self.hq // tp
@@ -310,7 +329,7 @@ class Attention:
       self.logit_scale = (0.1 * math.log(float(c.rope_factor)) + 1.0) ** 2
     # qwen3-next (src/maxtext/layers/attentions.py:685-686,1266-1270,1360-1362): the query projection is twice as wide,
     # per head [query | gate], and sigmoid(gate) multiplies the attention output before the output projection
-    self.gated = bool(gated)
+    self.gated = bool(gated) and sizes is None
     ab = b.sub(*name.split("/"))
     depth_scale = 1.0 if (qk_norm or (query_scalar is not None and query_scalar != 1.0)) else 1.0 / math.sqrt(self.dh)
     kv_tp = "col" if self.hkv >= tp else None
@@ -319,11 +338,16 @@ class Attention:
     self.k = ab.sub("key").linear("kernel", (self.d,), (self.hkv, self.dh), ("embed", "kv_heads", "kv_head_dim"),
                                   "fan_in_normal", tp=kv_tp)
     # share_kv_projections (src/maxtext/layers/attentions.py:289): the value is the (un-normalised, un-rotated) key projection
-    self.v = None if self.share_kv else ab.sub("value").linear("kernel", (self.d,), (self.hkv, self.dh), ("embed", "kv_heads", "kv_head_dim"),
+    self.v = None if self.share_kv else ab.sub("value").linear("kernel", (self.d,), (self.hkv, self.dv), ("embed", "kv_heads", "kv_head_dim"),
                                                                "fan_in_normal", tp=kv_tp)
-    self.o = ab.sub("out").linear("kernel", (self.hq, self.dh), (self.d,), ("heads", "kv", "embed"), "fan_in_normal",
+    self.g = ab.sub("gate").linear("kernel", (self.d,), (self.hq, self.dv), ("embed", "q_heads", "kv"), "fan_in_normal", tp="col") \
+        if gated and sizes is not None else None
+    self.o = ab.sub("out").linear("kernel", (self.hq, self.dv), (self.d,), ("heads", "kv", "embed"), "fan_in_normal",
                                   tp="row")
-    self.qkv = FusedParam([self.q, self.k, self.v]) if (not self.gated and not self.share_kv and FusedParam.possible([self.q, self.k, self.v])) else None
+    self.qkv = FusedParam([self.q, self.k, self.v]) if (not self.gated and not self.share_kv and sizes is None
+                                                        and FusedParam.possible([self.q, self.k, self.v])) else None
+    # everything that reads the layer input as one product [q | k | v | gate] (inference)
+    self.qkvg = FusedParam([self.q, self.k, self.v, self.g]) if self.g is not None and FusedParam.possible([self.q, self.k, self.v, self.g]) else None
     self.vn = Norm(ab, "value_norm", self.dh, c.normalization_layer_epsilon, with_scale=(self.v_norm == "scale"), axes=("norm",)) if self.v_norm else None
     self.bq = self.bk = self.bv = None
     if bias:
@@ -364,10 +388,26 @@ class Attention:
     q = ctx.keep("query_proj", F.linear(x, self.q, ctx.reuse("query_proj"), self.bq))
     k = ctx.keep("key_proj", F.linear(x, self.k, ctx.reuse("key_proj"), self.bk))
     v = k if self.share_kv else ctx.keep("value_proj", F.linear(x, self.v, ctx.reuse("value_proj"), self.bv))
-    return None, (q.view(B, S, hq, -1), k.view(B, S, hkv, dh), v.view(B, S, hkv, dh))
+    return None, (q.view(B, S, hq, -1), k.view(B, S, hkv, dh), v.view(B, S, hkv, self.dv))
+
+  def _serve(self, x, ctx):
+    """Inference kernels: one product for q | k | v | gate, rotation and norms in one pass that also fills the cache, attention over
+    the cache, and the gate with the last step of it (`ops.cached_attention`)."""
+    from ..ops import cached_attention as CA
+    B, S, _ = x.shape
+    if self.qkvg is not None and self.qkvg.fusable():
+      p = F.linear(x, self.qkvg).view(B * S, -1)
+      q, k, v, g = torch.split(p, self.qkvg.rows, dim=-1)
+    else:
+      q, k, v, g = (F.linear(x, w).view(B * S, -1) for w in (self.q, self.k, self.v, self.g))
+    return F.linear(CA.serve(self, q, k, v, g, ctx).view(B, S, -1), self.o)
 
   def __call__(self, x, ctx):
     B, S, _ = x.shape
+    if self.g is not None and self.l2_qk_norm and ctx.cache is not None:
+      from ..ops import cached_attention as CA
+      if CA.servable(x, self, ctx):
+        return self._serve(x, ctx)
     # tensor parallelism: with the fused runtime the two all-reduces of this block run inside GEMM epilogues
     tp_rt = tp_fused.runtime_for(ctx, x, self.d) if ctx.tp_size > 1 else None
     fuse_in = tp_rt is not None and self.qkv is not None and self.bq is None and self.qkv.fusable()
@@ -375,8 +415,9 @@ class Attention:
       x = tp_enter(x, ctx)
       B, S, _ = x.shape                      # sequence parallelism: the gathered length
     packed, sep = self._project(x, ctx, tp_rt if fuse_in else None)
+    gate = F.linear(x, self.g) if self.g is not None else None
     moba = bool(getattr(self.config, "moba", False)) and ctx.cache is None and ctx.cp_size == 1
-    plain = (ctx.positions3 is None and not self.qk_norm and self.vn is None and not self.share_kv and self.sinks is None and self.rotary_dim is None and not self.gated and ctx.bidir is None and not moba and ctx.cache is None and ctx.cp_size == 1
+    plain = (ctx.positions3 is None and not self.qk_norm and self.g is None and self.vn is None and not self.share_kv and self.sinks is None and self.rotary_dim is None and not self.gated and ctx.bidir is None and not moba and ctx.cache is None and ctx.cp_size == 1
              and not self.l2_qk_norm and not self.temperature_tuning and not (self.chunk and S > self.chunk))
     saved_ctx = ctx.reuse("context")
     if saved_ctx is not None and packed is not None and plain:
@@ -391,7 +432,6 @@ class Attention:
         q, k, v = packed[:, :, :self.hq_l], packed[:, :, self.hq_l:self.hq_l + self.hkv_l], packed[:, :, self.hq_l + self.hkv_l:]
       else:
         q, k, v = sep
-      gate = None
       if self.gated:
         q, gate = q[..., :self.dh], q[..., self.dh:].reshape(B, S, -1)
       if self.global_qk_norm:
@@ -445,7 +485,7 @@ class Attention:
       else:
         out = F.attention(q, k, v, ctx.positions, ctx.segment_ids, 1.0, self.soft_cap, self.window)
     ctx.keep("context", out)
-    if self.gated:
+    if gate is not None:
       out = (out.reshape(B, S, -1).float() * torch.sigmoid(gate.float())).to(out.dtype)
     if tp_rt is not None and ctx.reuse("out_proj") is None and self.bo is None and self.o.lora is None:
       y = F.linear(out.reshape(B, S, -1), self.o, tp_reduce=tp_rt)

@@ -91,7 +91,8 @@ def gated_delta_chunked(q, k, v, g, beta, chunk: int = 64, state=None):
 
 
 class RecurrentState:
-  """Inference state of one recurrent layer for `slots` sequences: the matrix state S per head in fp32 and, where the layer has a
+  """Inference state of one recurrent layer for `slots` sequences: the matrix state S per head in fp32 (a selective scan has one head of
+  [channels, state]) and, where the layer has a
   short convolution, its last taps - 1 inputs. A sequence of length 0 reads zeros whatever its slot holds, so a slot needs no
   clearing between requests."""
 

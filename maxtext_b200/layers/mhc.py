@@ -107,6 +107,20 @@ class HyperConnection:
     return (res_out + post_out).to(x.dtype)
 
 
+class StaticHyperConnection:
+  """A hyper-connection whose maps are constants of the model: the branch reads sum_s in[s] x_s, and afterwards stream t is
+  sum_s mix[s, t] x_s + out[t] * branch (mix is indexed [from, to]). Streams and maps are fp32 (`ops.functional.stream_mix`)."""
+
+  def __init__(self, b: L.Builder, config, name: str, k: int):
+    self.k = k
+    sb = b.sub(name)
+    add = lambda n, shape, init: sb._add(n, shape=shape, ref_shape=shape, logical_axes=(None,) * len(shape), kind="same", init=init)  # noqa: E731
+    # at the start every stream carries the same residual sum: read their mean, keep each, write to each
+    self.read = sb._add("in", shape=(k,), ref_shape=(k,), logical_axes=(None,), kind="same", init="const", init_scale=1.0 / k)
+    self.mix = add("mix", (k, k), "identity")
+    self.write = add("out", (k,), "ones")
+
+
 class HyperHead:
   """Final collapse of the k streams (DeepSeek-V4): scale-free RMS statistic of the flattened stream, a [k*D, k] projection,
   sigmoid gates, weighted sum of the streams."""

@@ -10,6 +10,7 @@ a variable-size all-to-all whose split sizes come from an exchanged count matrix
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 
 import torch
 import torch.distributed as dist
@@ -85,27 +86,41 @@ class _AllReduceMean(torch.autograd.Function):
     return g / ctx.n, None, None
 
 
+@dataclass(frozen=True)
+class MoESizes:
+  """Experts, experts per token, expert width and activation clamp of one routed layer."""
+  experts: int
+  top: int
+  ff: int
+  limit: float = 0.0
+
+
 class RoutedMoE:
-  def __init__(self, b: Builder, config, name="MoeBlock_0", deepseek_style=False, style: str = "", hash_routing: bool = False):
+  def __init__(self, b: Builder, config, name="MoeBlock_0", deepseek_style=False, style: str = "", hash_routing: bool = False,
+               sizes: MoESizes | None = None):
     """style: "llama4" (raw top-k logits, sigmoid score applied to the expert input, unit combine weights;
     src/maxtext/layers/moe.py:752,902-906,1051-1053) or "gpt_oss" (router bias on the logits, per-expert biases and the
-    clamped x * sigmoid(1.702 x) * (up + 1) activation; moe.py:617-637,841-853,2239-2242)."""
+    clamped x * sigmoid(1.702 x) * (up + 1) activation; moe.py:617-637,841-853,2239-2242), or "scaled_input": the top-k sigmoid
+    scores, not renormalised, scale what each chosen expert reads, experts with the clamped activation and no biases; the router and
+    the scores are fp32. `sizes` replaces the config's sizes."""
     c = config
     self.c = c
     self.style = style
-    self.E, self.k = c.num_experts, c.num_experts_per_tok
+    if sizes is None:
+      sizes = MoESizes(c.num_experts, c.num_experts_per_tok, c.moe_mlp_dim, float(c.mlp_activations_limit or 0.0))
+    self.E, self.k, self.limit = sizes.experts, sizes.top, sizes.limit
     self.deepseek = deepseek_style
     mb = b.sub(name)
-    d, f = c.emb_dim, c.moe_mlp_dim
+    d, f = c.emb_dim, sizes.ff
     self.gate = mb.sub("gate").linear("kernel", (d,), (self.E,), ("embed", None))
-    self.gate_bias = mb.sub("gate").vector("bias", self.E, (None,), init="zeros") if c.routed_bias else None
+    self.gate_bias = mb.sub("gate").vector("bias", self.E, (None,), init="zeros") if c.routed_bias and style != "scaled_input" else None
     self.wi_0 = mb.experts("wi_0", self.E, d, f, ("exp", "embed_moe", "mlp_moe"), tp="col")
     self.wi_1 = mb.experts("wi_1", self.E, d, f, ("exp", "embed_moe", "mlp_moe"), tp="col")
     self.wo = mb.experts("wo", self.E, f, d, ("exp", "mlp_moe", "embed_moe"), tp="row")
     self.act = c.mlp_activations[0]
     self.e_local = self.E // b.ep_size
     self.b0 = self.b1 = self.bo = None
-    if c.mlp_bias:
+    if c.mlp_bias and style != "scaled_input":
       self.b0 = mb.table("wi_0_bias", (self.E, f), ("exp", "activation_mlp"), init="zeros")
       self.b1 = mb.table("wi_1_bias", (self.E, f), ("exp", "activation_mlp"), init="zeros")
       self.bo = mb.table("wo_bias", (self.E, d), ("exp", "activation_embed"), init="zeros")
@@ -125,6 +140,10 @@ class RoutedMoE:
     src = x2 if gate_inputs is None else gate_inputs
     xg = src.float() if c.float32_gate_logits else src
     w = self.gate.leaf()
+    if self.style == "scaled_input":
+      probs = torch.sigmoid(torch.nn.functional.linear(src.float(), w.float()))
+      wts, idx = probs.topk(self.k, dim=-1)
+      return wts, idx, self._aux(probs, idx, B, S, ctx)
     logits = torch.nn.functional.linear(xg, w.to(xg.dtype))
     if self.style == "gemma4":
       probs = torch.softmax(logits.float(), -1)
@@ -222,8 +241,8 @@ class RoutedMoE:
       row_e = torch.repeat_interleave(torch.arange(sizes.numel(), device=rows.device), sizes.long(), output_size=rows.shape[0])
       g = g + self.b0.leaf()[row_e].to(g.dtype)
       u = u + self.b1.leaf()[row_e].to(u.dtype)
-    if self.style == "gpt_oss":
-      lim = float(self.c.mlp_activations_limit)
+    if self.style in ("gpt_oss", "scaled_input"):
+      lim = self.limit
       gf, uf = g.float().clamp(max=lim), u.float().clamp(-lim, lim)
       h = (gf * torch.sigmoid(1.702 * gf) * (uf + 1.0)).to(rows.dtype)
     else:
@@ -255,7 +274,11 @@ class RoutedMoE:
     red = _ReduceScatterRows.apply(out, ctx.ep_group) if torch.is_grad_enabled() else _ReduceScatterRows.forward(F._Dummy(), out, ctx.ep_group)
     return red
 
-  def __call__(self, x, ctx, gate_inputs=None):
+  def __call__(self, x, ctx, gate_inputs=None, rows_ok=False):
+    """`rows_ok`: a GPU inference pass may return the experts' output rows (`moe_ops.ExpertRows`) instead of their sum per token."""
+    if self.style == "scaled_input" and moe_ops.serve_ok(x, ctx):
+      out = moe_ops.serve_scaled(x.reshape(-1, x.shape[-1]), self)
+      return out if rows_ok else out.combine(x)
     if ctx.sp and ctx.tp_size > 1:
       assert gate_inputs is None, "a separate router input is not implemented under tensor-sequence parallelism"
       # sequence-parallel residual stream: routing needs every token, so the block runs the plain tensor-parallel form on
@@ -285,6 +308,10 @@ class RoutedMoE:
       assert self.k == 1, "llama4 routing scales the expert input by its single score"
       x2 = (x2.float() * torch.sigmoid(wts)).to(x2.dtype)
       wts = torch.ones_like(wts)
+    row_scale = None
+    if self.style == "scaled_input":
+      assert ctx.ep_size == 1, "expert inputs scaled per choice are not exchanged between ranks"
+      row_scale, wts = wts.reshape(-1), torch.ones_like(wts)
     if ctx.tp_size > 1:
       # the experts' hidden dim is split over the tensor ranks: what flows back into the tokens and into the combine weights
       # is a partial sum on every rank (the router itself runs replicated and stays outside). The fused paths combine before
@@ -292,7 +319,7 @@ class RoutedMoE:
       x2, wts_fused = tp_enter(x2, ctx), tp_enter(wts, ctx)
     else:
       wts_fused = wts
-    plain_ffn = self.b0 is None and self.style != "gpt_oss"
+    plain_ffn = self.b0 is None and self.style not in ("gpt_oss", "scaled_input")
     if plain_ffn and ctx.ep_size == 1 and self.act in F._ACT_CODE and moe_ops.padded_path_supported(x2, D, self.wi_0.data.shape[1], self.E):
       # GPU path: device-side stable sort into 128-row-padded expert groups, grouped tcgen05 GEMMs, no host synchronisation
       out = moe_ops.moe_ffn_padded(x2, wts_fused, idx, self.wi_0, self.wi_1, self.wo, self.E, self.act)
@@ -308,6 +335,8 @@ class RoutedMoE:
           out = tp_exit(out, ctx)
         return out.view(B, S, D)
     rows, order, sizes = moe_ops.permute(x2, idx, self.E)          # rows sorted by global expert id
+    if row_scale is not None:
+      rows = (rows.float() * row_scale[order][:, None]).to(rows.dtype)
     y = self._expert_parallel(rows, sizes, ctx) if ctx.ep_size > 1 else self.experts_ffn(rows, sizes)
     if ctx.tp_size > 1:
       y = tp_exit(y, ctx)           # the experts' hidden dim is split over the tensor ranks: sum the partial outputs

@@ -19,6 +19,7 @@ class Family:
   norm_offset: float = 0.0
   scale_embedding: bool = False
   residual_fp32: bool = False              # the residual stream and the logits are fp32 whatever the compute dtype
+  static_streams: bool = False             # mhc_expansion_rate fp32 streams, mixed by constants of the model instead of per-token maps
 
 
 def describe(c) -> Family:
@@ -32,6 +33,8 @@ def describe(c) -> Family:
     return Family(norm_offset=1.0)           # every RMS scale is stored zero-centred and applied as (1 + scale)
   if blk == "silinex":
     return Family(norm_offset=1.0, residual_fp32=True)
+  if blk == "tipidra":
+    return Family(norm_kind="layernorm", residual_fp32=True, static_streams=True)
   return Family()
 
 
@@ -170,6 +173,9 @@ def layer_plans(c) -> list[LayerPlan]:
   if blk == "silinex":
     from .silinex import layer_plans as silinex_plans
     return silinex_plans(c)
+  if blk == "tipidra":
+    from .tipidra import layer_plans as tipidra_plans
+    return tipidra_plans(c)
   if blk == "gemma":
     bp = BlockPlan(pre_attn_norm="pre_self_attention_norm", pre_mlp_norm="pre_ffw_norm", soft_cap=c.attn_logits_soft_cap)
     return [LayerPlan("layers", [bp]) for _ in range(n)]
@@ -227,4 +233,4 @@ def layer_plans(c) -> list[LayerPlan]:
     return plans
   raise NotImplementedError(
       f"decoder_block={blk!r} parses but has no model implementation here yet (implemented: llama2, mistral, mixtral, "
-      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, silinex, simple)")
+      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, silinex, tipidra, simple)")

@@ -13,9 +13,9 @@ import struct
 
 import torch
 
-from . import silinex
+from . import silinex, tipidra
 
-ARCHITECTURES = {"Silinex": silinex}
+ARCHITECTURES = {"Silinex": silinex, "Tipidra": tipidra}
 
 
 def _safetensors_files(path: str) -> list[str]:

@@ -34,9 +34,9 @@ class BlockPlan:
   post_mlp_norm: str | None = None
   attn_name: str = "self_attention"
   mlp_name: str = "mlp"
-  attention: str = "gqa"                 # gqa | mla | gdn (gated delta network, qwen3-next) | gla | compressed
+  attention: str = "gqa"                 # gqa | mla | gdn (gated delta network, qwen3-next) | gla | ssm (selective scan) | compressed
   mixer: dict | None = None              # sizes of this block's mixer, for families whose layers differ (None: the config's)
-  gated_attn: bool = False               # qwen3-next full attention: sigmoid output gate from a widened query projection
+  gated_attn: bool = False               # sigmoid output gate: from a widened query projection (qwen3-next) or, with `mixer`, a projection of its own
   window: int = 0
   rope: str = "default"                  # key into Transformer.rope_tables
   use_rope: bool = True
@@ -57,12 +57,14 @@ class BlockPlan:
   l2_qk_norm: bool = False               # llama4: scale-free RMS normalisation of q and k after RoPE
   temperature_tuning: bool = False       # llama4 NoPE layers: position-dependent query scale
   chunk: int = 0                         # llama4 RoPE layers: attention restricted to chunks of this many tokens
-  moe_style: str = ""                    # "" | "llama4" | "gpt_oss"
+  moe_style: str = ""                    # "" | "llama4" | "gpt_oss" | "scaled_input"
+  moe: dict | None = None                # router and expert sizes of this block, for families whose layers differ (None: the config's)
   head_dim: int | None = None            # gemma4 global layers: own head width ...
   kv_heads: int | None = None            # ... and key / value head count
   share_kv: bool = False                 # value = key projection
   v_norm: str = ""                       # "" | "noscale" | "scale": RMS normalisation of the value heads
   layer_scalar: bool = False             # learned scalar on the layer output
+  hyper: str = ""                        # "static": hyper-connections with constant maps around the two sublayers
   residual_mult: float = 1.0             # factor on each branch before it joins the residual stream
   residual_fp32: bool = False            # fp32 residual stream with sandwich norms, fused with the residual add (`F.residual_norm`)
   compress_ratio: int = 0                # DeepSeek-V4 compressed attention: 0 (window only), 4 (sparse) or 128 (heavy)
@@ -109,20 +111,32 @@ class DecoderBlock:
       m = plan.mixer
       self.attn = GatedLinearAttention(b, c, plan.attn_name + s, int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"]),
                                        int(m["decay_rank"]))
+    elif plan.attention == "ssm":
+      from ..layers.ssm import ScanSizes, SelectiveScan
+      m = plan.mixer
+      self.attn = SelectiveScan(b, c, plan.attn_name + s, ScanSizes(int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m["conv"])))
     elif plan.attention == "compressed":
       from ..layers.attention_compressed import CompressedAttention
       self.attn = CompressedAttention(b, c, plan.attn_name + s, plan.compress_ratio, int(c.sliding_window_size))
     else:
-      self.attn = L.Attention(b, c, plan.attn_name + s, plan.window, inv_ts, interleaved, plan.use_rope, plan.qk_norm,
+      sizes = None
+      if plan.mixer is not None:
+        m = plan.mixer
+        rot, interleaved = int(m["rot"]["dims"]), False
+        inv_ts = ref.rope_inv_timescale(rot, 1.0, float(m["rot"]["base"])).to(inv_ts.device)
+        sizes = L.HeadSizes(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), float(m["softcap"]))
+      self.attn = L.Attention(b, c, plan.attn_name + s, plan.window, inv_ts, interleaved, plan.use_rope and rot != 0, plan.qk_norm,
                               plan.query_scalar, plan.soft_cap, plan.attn_bias,
                               rotary_dim=rot, sinks=plan.sinks, l2_qk_norm=plan.l2_qk_norm,
                               temperature_tuning=plan.temperature_tuning, chunk=plan.chunk, out_bias=plan.attn_out_bias,
                               global_qk_norm=plan.global_qk_norm, gated=plan.gated_attn, qk_norm_offset=plan.norm_offset,
-                              head_dim=plan.head_dim, num_kv_heads=plan.kv_heads, share_kv=plan.share_kv, v_norm=plan.v_norm)
+                              head_dim=plan.head_dim, num_kv_heads=plan.kv_heads, share_kv=plan.share_kv, v_norm=plan.v_norm, sizes=sizes)
     self.n1b = mk(plan.post_attn_norm) if plan.post_attn_norm else None
     self.n2 = mk(plan.pre_mlp_norm) if plan.pre_mlp_norm else None
     if plan.mlp == "moe":
-      self.mlp = M.RoutedMoE(b, c, plan.mlp_name + s, style=plan.moe_style)
+      r = plan.moe
+      self.mlp = M.RoutedMoE(b, c, plan.mlp_name + s, style=plan.moe_style, sizes=M.MoESizes(
+          int(r["router"]["experts"]), int(r["router"]["top"]), int(r["expert"]["ff"]), float(r["expert"]["limit"])) if r is not None else None)
     elif plan.mlp == "moe_shared":
       hashed = layer_index is not None and layer_index < int(getattr(c, "first_num_hash_layers", 0) or 0) and plan.moe_style == ""
       self.mlp = M.RoutedAndSharedMoE(b, c, plan.mlp_name + s, style=plan.moe_style, hash_routing=hashed)
@@ -136,7 +150,12 @@ class DecoderBlock:
     self.layer_scalar = b._add("layer_scalar" + s, shape=(1,), ref_shape=(1,), logical_axes=(None,), kind="same", init="ones") \
         if plan.layer_scalar else None
     self.mhc_attn = self.mhc_mlp = None
-    if int(getattr(c, "mhc_expansion_rate", 1)) > 1:
+    self.hc1 = self.hc2 = None
+    if plan.hyper == "static":
+      from ..layers.mhc import StaticHyperConnection
+      self.hc1 = StaticHyperConnection(b, c, "mixer_streams" + s, int(c.mhc_expansion_rate))
+      self.hc2 = StaticHyperConnection(b, c, "mlp_streams" + s, int(c.mhc_expansion_rate)) if self.mlp is not None else None
+    elif int(getattr(c, "mhc_expansion_rate", 1)) > 1:
       # src/maxtext/models/deepseek.py:177-179: each branch of the block is wrapped by its own hyper-connection
       from ..layers.mhc import HyperConnection
       self.mhc_attn = HyperConnection(b, c, "mhc_attention", c.emb_dim)
@@ -155,6 +174,8 @@ class DecoderBlock:
     if self.mhc_attn is not None:               # x [B, S, k, D]: the residual adds live inside the hyper-connections
       x = self.mhc_attn(self.n1, lambda h: self.attn(h, ctx), x)
       return self.mhc_mlp(self.n2, lambda h: self.mlp(h, ctx), x)
+    if self.hc1 is not None:
+      return self._call_static_streams(x, ctx)
     if self.plan.residual_fp32:
       return self._call_fp32_stream(x, ctx)
     a = self.attn(self.n1(x) if self.n1 is not None else x, ctx)
@@ -170,6 +191,23 @@ class DecoderBlock:
       x = x * self.layer_scalar.leaf().to(x.dtype)
     return x
 
+  def reader(self):
+    """What reads the residual stream first in this block: its norm, with the weights of the streams where there are several."""
+    return F.StreamReader(self.hc1, self.n1) if self.hc1 is not None else self.n1
+
+  def _call_static_streams(self, x, ctx: LayerCtx):
+    """x fp32 [B, S, k, D]. One kernel per sublayer border: the streams mixed among themselves, the branch added to each, and the
+    normalised input of the next sublayer (of this block, or of the next layer through `ctx.next_norm` / `ctx.normed`)."""
+    h = ctx.normed if ctx.normed is not None else F.stream_read(x, self.reader(), self.n1.scale.data.dtype)
+    ctx.normed = None
+    a = self.attn(h, ctx)
+    if self.mlp is None:
+      x, ctx.normed = F.stream_mix(x, a, self.hc1, ctx.next_norm)
+      return x
+    x, h = F.stream_mix(x, a, self.hc1, F.StreamReader(self.hc2, self.n2))
+    f = self.mlp(h, ctx, rows_ok=True) if self.plan.moe_style == "scaled_input" else self.mlp(h, ctx)
+    x, ctx.normed = F.stream_mix(x, f, self.hc2, ctx.next_norm)
+    return x
 
   def _call_fp32_stream(self, x, ctx: LayerCtx):
     """x fp32 [B, S, D]. One kernel per sublayer border: the branch's norm, the residual add and the norm in front of the next
@@ -290,6 +328,19 @@ class _StreamNorm:
   def __call__(self, x):
     return F.stream_norm(x, self.norm, self.scale.data.dtype)
 
+  def reader(self):
+    return self
+
+
+class _StreamSumNorm(_StreamNorm):
+  """Final norm of a model with several fp32 streams: their plain sum, normalised; returns the compute dtype."""
+
+  def __call__(self, x):
+    return F.stream_read(x, self.reader(), self.scale.data.dtype)
+
+  def reader(self):
+    return F.StreamReader(None, self.norm)
+
 
 class MTPLayer:
   """One multi-token-prediction module (src/maxtext/layers/multi_token_prediction.py:160-310): the previous hidden state and
@@ -391,7 +442,10 @@ class Transformer:
     if self.mhc_k > 1 and c.decoder_block == "deepseek4":
       from ..layers.mhc import HyperHead
       hyper_head = HyperHead(hb.sub("decoder"), c, "hc_head")
-    self.final_norm = _CollapsingNorm(norm, hyper_head) if self.mhc_k > 1 else (_StreamNorm(norm) if self.family.residual_fp32 else norm)
+    if self.family.static_streams:
+      self.final_norm = _StreamSumNorm(norm)
+    else:
+      self.final_norm = _CollapsingNorm(norm, hyper_head) if self.mhc_k > 1 else (_StreamNorm(norm) if self.family.residual_fp32 else norm)
     self.logits_dense = None
     if not c.logits_via_embedding:
       self.logits_dense = hb.sub("decoder", "logits_dense").linear("kernel", (c.emb_dim,), (c.vocab_size,),
@@ -495,6 +549,8 @@ class Transformer:
     x = F.embedding(tokens, self.embedding)
     if self.family.residual_fp32:
       x = x.float()
+    if float(c.embedding_multiplier) != 1.0:
+      x = x * float(c.embedding_multiplier)
     if mm is not None:
       from ..multimodal.utils import merge_mm_embeddings
       for soft, mask in ([mm] if isinstance(mm, tuple) else mm):
@@ -509,7 +565,7 @@ class Transformer:
       x = x + torch.cat([torch.sin(ang), torch.cos(ang)], dim=-1).to(x.dtype)
     if self.pos_embedding is not None:
       x = x + self.pos_embedding.leaf()[positions.long()].to(x.dtype)
-    if self.mhc_k > 1:
+    if self.mhc_k > 1 or self.family.static_streams:
       from ..layers.mhc import expand_streams
       x = expand_streams(x, self.mhc_k)        # src/maxtext/layers/decoders.py:880-883
     return x
@@ -560,7 +616,8 @@ class Transformer:
       ctx.layer_index = i
       ctx.cache = caches[i] if caches is not None else None
       if self.family.residual_fp32 and not torch.is_grad_enabled():
-        ctx.next_norm = self.layers[i + 1].blocks[0].n1 if i + 1 < len(self.layers) else self.final_norm
+        nxt = self.layers[i + 1].blocks[0] if i + 1 < len(self.layers) else self.final_norm
+        ctx.next_norm = nxt.reader()
       x = layer(x, ctx)
     normed = ctx.normed
     if logit_rows is None:

@@ -1,0 +1,130 @@
+"""Attention over a slot-indexed key/value cache on the inference kernels (`csrc/cached_attention_sm100.cu`).
+
+`serve` is the whole attention part of a layer whose q and k are rotated and then RMS-normalised per head: one kernel rotates, normalises,
+fills the cache and lays the operands out for what follows; prompts run the flash kernel (head widths padded to the next variant), one new
+token per sequence runs the split decode kernel, and everything else (fp32, unusual widths) a plain kernel that reads the cache. Sinks,
+soft caps, windows and a sigmoid output gate are parameters. `decode` and `prompt` also serve `inference.kvcache.LayerKVCache.attend`.
+"""
+from __future__ import annotations
+
+import torch
+
+from . import backend, functional as F
+
+FAR = 1 << 30            # position of a key row that holds nothing: after every query, so the causal mask removes it
+
+
+def kernels_ok(t: torch.Tensor) -> bool:
+  return not torch.is_grad_enabled() and t.dtype in (torch.bfloat16, torch.float32) and backend.use_cuda_kernels(t)
+
+
+def servable(x, layer, ctx) -> bool:
+  """Can this call of a `layers.blocks.Attention` run `serve`? (It normalises q and k after the rotation.)"""
+  from ..inference.kvcache import LayerKVCache
+  c = ctx.cache
+  return (kernels_ok(x) and type(c) is LayerKVCache and c.quant is None and c.seq_size == 1 and c.k.dtype == x.dtype and ctx.tp_size == 1
+          and ctx.positions3 is None and ctx.bidir is None and not layer.interleaved and not layer.qk_norm and layer.vn is None
+          and layer.bq is None and not layer.chunk and not layer.temperature_tuning and not (ctx.segment_ids is not None and x.dtype != torch.bfloat16))
+
+
+def flash_widths(qk: int, vd: int):
+  """Head widths (query/key, value) of the smallest flash variant that holds a head, or None."""
+  for dq, dv in ((64, 64), (128, 128), (192, 128)):
+    if qk <= dq and vd <= dv:
+      return dq, dv
+  return None
+
+
+def _gate(o, g, H, dv):
+  """o [N, H, >= dv] times sigmoid(g [N, H * dv]) (g None: only the padding is dropped)."""
+  if g is None:
+    return o[..., :dv].reshape(o.shape[0], H * dv)
+  out = torch.empty(o.shape[0], H * dv, dtype=o.dtype, device=o.device)
+  backend.ext().head_gate(o, g, dv, out)
+  return out
+
+
+def serve(layer, q, k, v, g, ctx):
+  """q [N, H*D], k [N, G*D], v [N, G*Dv] rows of the projections (not rotated yet), g [N, H*Dv] logits of the gate -> [N, H*Dv]."""
+  E, cache = backend.ext(), ctx.cache
+  B, S = ctx.positions.shape
+  N, H, G, D, Dv = B * S, layer.hq_l, layer.hkv_l, layer.dh, layer.dv
+  bf = q.dtype == torch.bfloat16
+  scale, cap, win = float(layer.query_scalar or 1.0) * layer.logit_scale, float(layer.soft_cap), int(layer.window)
+  sinks = layer.sinks.data if layer.sinks is not None else None
+  eps = float(layer.config.normalization_layer_epsilon)
+  rot = (int(layer.rotary_dim or D) if layer.use_rope else 0)
+  widths = flash_widths(D, Dv) if bf and S > 1 else None
+  fresh = ctx.mode == "prefill"
+  dq, dvp = widths if widths is not None else (D, Dv)
+  pack_k = widths is not None and fresh                  # later portions read their keys from the cache
+  qp = torch.empty(N, H, dq, dtype=q.dtype, device=q.device)
+  kp = torch.empty(N, G, dq, dtype=q.dtype, device=q.device) if pack_k else None
+  vp = torch.empty(N, G, dvp, dtype=q.dtype, device=q.device) if pack_k and dvp != Dv else None
+  E.qkv_prep(q, k, v, D, Dv, ctx.positions.contiguous(), layer.inv_ts if rot else None, rot, eps if layer.l2_qk_norm else -1.0, qp, kp, vp, cache.k, cache.v,
+             cache.slot_ids, cache.lengths, cache.new_lens)
+  if S == 1:
+    return decode(qp, cache, scale, cap, win, sinks, g)
+  if widths is None:
+    return plain(qp, cache, S, scale, cap, win, sinks, g)
+  if fresh:
+    vv = vp if vp is not None else v
+    o = _flash(qp.view(B, S, H, dq), kp.view(B, S, G, dq), vv.view(B, S, G, dvp) if vp is not None else _rows(vv, B, S, G, Dv), ctx.positions,
+               ctx.segment_ids, scale, cap, win, sinks)
+  else:
+    o = _portion(qp.view(B, S, H, dq), cache, ctx, scale, cap, win, sinks, D, Dv)
+  return _gate(o.view(N, H, dvp), g, H, Dv)
+
+
+def _rows(v, B, S, G, Dv):
+  """[N, G*Dv] rows of a wider matrix as [B, S, G, Dv] without a copy."""
+  return v.as_strided((B, S, G, Dv), (S * v.stride(0), v.stride(0), Dv, 1), v.storage_offset())
+
+
+def _flash(q, k, v, positions, segment_ids, scale, cap, win, sinks, kv_positions=None):
+  return F.attention_fwd(q, k, v, positions, segment_ids, scale, cap, win, kv_positions=kv_positions, sinks=sinks)[0]
+
+
+def _portion(q, cache, ctx, scale, cap, win, sinks, D, Dv):
+  """Queries that follow cached tokens: the keys they can see are gathered from the cache (padded to the flash widths)."""
+  B, S, H, dq = q.shape
+  dvp = flash_widths(D, Dv)[1]
+  if win > 0:
+    idx = cache.lengths[:, None] - (win - 1) + torch.arange(win - 1 + S, device=q.device)[None]
+  else:
+    idx = torch.arange(int((cache.lengths.max() + S).item()), device=q.device)[None].expand(B, -1)
+  kv_pos = torch.where((idx < 0) | (idx >= (cache.lengths + S)[:, None]), torch.full_like(idx, FAR), idx)
+  rows = idx.clamp(0, cache.max_len - 1)
+  slots = cache.slot_ids[:, None].expand_as(rows)
+  k, v = cache.k[slots, rows], cache.v[slots, rows]
+  k = torch.nn.functional.pad(k, (0, dq - D)) if dq != D else k
+  v = torch.nn.functional.pad(v, (0, dvp - Dv)) if dvp != Dv else v
+  return _flash(q, k, v, ctx.positions, None, scale, cap, win, sinks, kv_pos)
+
+
+def decode_widths_ok(D: int, Dv: int, dtype) -> bool:
+  return dtype == torch.bfloat16 and D % 8 == 0 and Dv % 8 == 0 and max(D, Dv) <= 256
+
+
+def decode(q, cache, scale, cap, win, sinks, g=None):
+  """One new token per sequence (its own key is in the cache already): q [B, H, D] -> [B, H*Dv], gated by sigmoid(g) if given."""
+  E = backend.ext()
+  B, H, D = q.shape
+  G, Dv = cache.k.shape[2], cache.v.shape[3]
+  if not decode_widths_ok(D, Dv, q.dtype):
+    return plain(q, cache, 1, scale, cap, win, sinks, g)
+  span = min(cache.max_len, win) if win > 0 else cache.max_len
+  splits = E.cached_decode_splits(B, H, G, span)
+  part = torch.empty(B, H, splits, Dv, dtype=torch.float32, device=q.device)
+  ml = torch.empty(B, H, splits, 2, dtype=torch.float32, device=q.device)
+  out = torch.empty(B, H * Dv, dtype=q.dtype, device=q.device)
+  E.cached_decode(q, cache.k, cache.v, cache.slot_ids, cache.lengths, scale, cap, win, sinks, g, splits, part, ml, out)
+  return out
+
+
+def plain(q, cache, S, scale, cap, win, sinks, g=None):
+  """Any widths up to 512, fp32 or bf16, any number of new tokens: q [B*S, H, D] over the cache -> [B*S, H*Dv]."""
+  H, Dv = q.shape[1], cache.v.shape[3]
+  o = torch.empty(q.shape[0], H, Dv, dtype=q.dtype, device=q.device)
+  backend.ext().cached_attention(q, cache.k, cache.v, cache.slot_ids, cache.lengths, S, scale, cap, win, sinks, o)
+  return _gate(o, g, H, Dv)

@@ -291,6 +291,51 @@ def residual_norm(x: torch.Tensor, branch: torch.Tensor, post, mult: float, nxt=
   return x, (ref.rmsnorm_f32(x, nxt.scale.leaf(), nxt.eps, nxt.offset).to(branch.dtype) if nxt is not None else None)
 
 
+# =============================================================================== several fp32 residual streams
+class StreamReader:
+  """What reads the streams in front of a sublayer: the weights of the streams (of a `layers.mhc.StaticHyperConnection`; None: their plain
+  sum) and the layer norm applied to the weighted sum."""
+
+  def __init__(self, connection, norm):
+    self.weights, self.norm = connection.read if connection is not None else None, norm
+
+
+def _read_streams(x, reader, dtype):
+  u = x.sum(2) if reader.weights is None else torch.einsum("s,bnsd->bnd", reader.weights.leaf().float(), x)
+  n = reader.norm
+  return ref.layernorm(u, n.scale.leaf().float(), n.bias.leaf().float(), n.eps).to(dtype)
+
+
+def stream_read(x: torch.Tensor, reader: StreamReader, dtype) -> torch.Tensor:
+  """x fp32 [B, S, k, D] -> the normalised input [B, S, D] of a sublayer, rounded once to `dtype`."""
+  if _stream_kernel_ok(x) and x.dtype == torch.float32 and x.is_contiguous():
+    B, S, k, D = x.shape
+    n = reader.norm
+    y = torch.empty(B * S, D, dtype=dtype, device=x.device)
+    backend.ext().stream_mix(x.view(B * S, k, D), None, None, 1, None, None, reader.weights.data if reader.weights is not None else None,
+                             n.scale.data, n.bias.data, y, float(n.eps))
+    return y.view(B, S, D)
+  return _read_streams(x.float(), reader, dtype)
+
+
+def stream_mix(x: torch.Tensor, branch, connection, nxt: StreamReader | None = None):
+  """(streams after a sublayer, input of the next one or None): x_t <- sum_s mix[s, t] x_s + write[t] * branch on fp32 x [B, S, k, D].
+  `branch` is [B, S, D] or expert rows that are summed per token (`moe_ops.ExpertRows`). On a GPU one kernel, which updates x in place."""
+  rows, dest, per_token = (branch, None, 1) if isinstance(branch, torch.Tensor) else (branch.rows, branch.dest, branch.k)
+  if _stream_kernel_ok(x, rows) and x.dtype == torch.float32 and x.is_contiguous():
+    B, S, k, D = x.shape
+    n = nxt.norm if nxt is not None else None
+    dt = connection.mix.data.dtype
+    y = torch.empty(B * S, D, dtype=dt, device=x.device) if nxt is not None else None
+    backend.ext().stream_mix(x.view(B * S, k, D), rows.reshape(-1, D), dest, per_token, connection.mix.data, connection.write.data,
+                             nxt.weights.data if nxt is not None and nxt.weights is not None else None, n.scale.data if n is not None else None,
+                             n.bias.data if n is not None else None, y, float(n.eps) if n is not None else 0.0)
+    return x, (y.view(B, S, D) if y is not None else None)
+  y = branch.float()
+  x = torch.einsum("st,bnsd->bntd", connection.mix.leaf().float(), x.float()) + connection.write.leaf().float()[:, None] * y[:, :, None, :]
+  return x, (_read_streams(x, nxt, branch.dtype) if nxt is not None else None)
+
+
 # =============================================================================== activation (ungated)
 _PLAIN_ACT_CODE = {"silu": 0, "swish": 0, "gelu": 1, "relu": 2, "gelu_exact": 4}
 
