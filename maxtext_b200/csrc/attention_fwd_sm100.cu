@@ -43,6 +43,7 @@ struct Params {
   attn::Mask mk;
   float scale;           // logits = scale * q.k
   float softcap;         // 0 = none; logits = softcap * tanh(scale * q.k / softcap)
+  int cap_mode;          // CAP_FAST: the tanh instruction (11 bits); CAP_EXACT: fp32; CAP_SMALL: fp32, for |scale * q.k| <= 0.3 softcap
   const float* sinks;    // [Hq] or nullptr
   float* lse;            // [B,Hq,Sq]
   int* status;
@@ -61,6 +62,23 @@ __device__ __forceinline__ float fast_tanh(float x) {
   float y;
   asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+enum { CAP_FAST = 0, CAP_EXACT = 1, CAP_SMALL = 2 };
+// tanh(x * pre) of two values. CAP_EXACT from one exponential; CAP_SMALL from the Taylor series up to x^9 (below 2e-8 for |x| <= 0.3)
+__device__ __forceinline__ float2 tanh2(float2 x, float pre, int mode) {
+  if (mode == CAP_SMALL) {
+    const float2 y = __fmul2_rn(x, make_float2(pre, pre)), z = __fmul2_rn(y, y);
+    float2 t = __ffma2_rn(z, make_float2(62.f / 2835.f, 62.f / 2835.f), make_float2(-17.f / 315.f, -17.f / 315.f));
+    t = __ffma2_rn(z, t, make_float2(2.f / 15.f, 2.f / 15.f));
+    t = __ffma2_rn(z, t, make_float2(-1.f / 3.f, -1.f / 3.f));
+    return __ffma2_rn(__fmul2_rn(y, z), t, y);
+  }
+  if (mode == CAP_EXACT) {
+    const float c = 2.f * LOG2E * pre;
+    return make_float2(1.f - __fdividef(2.f, 1.f + fast_exp2(x.x * c)), 1.f - __fdividef(2.f, 1.f + fast_exp2(x.y * c)));
+  }
+  return make_float2(fast_tanh(x.x * pre), fast_tanh(x.y * pre));
 }
 
 struct alignas(8) Ctl {
@@ -272,12 +290,17 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
         none = hi_p < lo_p;
         if (cap) pre = p.scale / p.softcap;
       }
-      // soft-cap and mask of 32 score columns starting at column c0 of the tile
-      auto prepare = [&](uint32_t (&r)[32], int c0) {
+      // soft-cap (only where the values are needed: it is monotonic, so a maximum can be capped afterwards) and mask of 32 score columns
+      // starting at column c0 of the tile
+      auto prepare = [&](uint32_t (&r)[32], int c0, bool values) {
         if constexpr (MASKED) {
-          if (cap) {
+          if (cap && values) {
 #pragma unroll
-            for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(fast_tanh(__uint_as_float(r[e]) * pre));
+            for (int e = 0; e < 32; e += 2) {
+              const float2 t = tanh2(make_float2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), pre, p.cap_mode);
+              r[e] = __float_as_uint(t.x);
+              r[e + 1] = __float_as_uint(t.y);
+            }
           }
           if (arrays) {
             const int* kp = sk_pos + (i * 2 + par) * 128 + c0;
@@ -304,20 +327,21 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
       tmem_ld_32x32b_x32(tS, r0);
       tmem_ld_wait_dep(r0);
       tmem_ld_32x32b_x32(tS + 32, r1);
-      prepare(r0, 0);
+      prepare(r0, 0, false);
       tmax = max32(r0);
       tmem_ld_wait_dep(r1);
       tmem_ld_32x32b_x32(tS + 64, r0);
-      prepare(r1, 32);
+      prepare(r1, 32, false);
       tmax = fmaxf(tmax, max32(r1));
       tmem_ld_wait_dep(r0);
       tmem_ld_32x32b_x32(tS + 96, r1);
-      prepare(r0, 64);
+      prepare(r0, 64, false);
       tmax = fmaxf(tmax, max32(r0));
       tmem_ld_wait_dep(r1);
       tmem_ld_32x32b_x32(tS, r0);              // first chunk of pass 2
-      prepare(r1, 96);
+      prepare(r1, 96, false);
       tmax = fmaxf(tmax, max32(r1));
+      if (MASKED && cap && tmax != -INFINITY) tmax = tanh2(make_float2(tmax, 0.f), pre, p.cap_mode).x;
       const float mt_ = a * tmax;                                    // -inf when the whole row is masked
       const bool grow = mt_ > m + RESCALE_THRESHOLD;                 // m = -inf: any finite maximum grows it
       if (__any_sync(0xffffffffu, grow)) {
@@ -344,7 +368,7 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
       const float2 a2 = make_float2(a, a), neg2 = make_float2(neg, neg);
       float2 rsa = make_float2(0.f, 0.f), rsb = make_float2(0.f, 0.f);
       auto exps = [&](uint32_t (&r)[32], int c) {
-        prepare(r, c * 32);
+        prepare(r, c * 32, true);
         uint32_t pk[16];
 #pragma unroll
         for (int e = 0; e < 16; ++e) {
@@ -544,7 +568,7 @@ void mt_attn_tile_minmax(const int* pos, int B, int S, int* out, cudaStream_t st
 int mt_flash_fwd(const void* q, const void* k, const void* v, void* out, float* lse, const int* seg_q, const int* seg_k, const int* pos_q,
                  const int* pos_k, int* tiles, const float* sinks, int B, int Sq, int Skv, int Hq, int Hkv, int Dqk, int Dv, long ldq, long bsq,
                  long ldk, long bsk, long ldv, long bsv, long ldo, long bso, float scale, float softcap, int causal, int window, int chunk,
-                 int q_off, int* status, cudaStream_t st) {
+                 int q_off, int cap_mode, int* status, cudaStream_t st) {
   using namespace mt::fwd;
   if (!mt_flash_fwd_supported(Dqk, Dv) || Hq % Hkv || Sq < 1 || Skv < 1 || (pos_q == nullptr) != (pos_k == nullptr) ||
       (seg_q == nullptr) != (seg_k == nullptr) || (pos_q && !tiles))
@@ -557,7 +581,7 @@ int mt_flash_fwd(const void* q, const void* k, const void* v, void* out, float* 
   Params p{};
   p.B = B; p.Hq = Hq; p.Hkv = Hkv;
   p.n_pairs = (Sq + 128 * nq - 1) / (128 * nq);
-  p.scale = scale; p.softcap = softcap; p.sinks = sinks; p.lse = lse; p.status = status;
+  p.scale = scale; p.softcap = softcap; p.cap_mode = cap_mode; p.sinks = sinks; p.lse = lse; p.status = status;
   p.head_major = 0;                       // tile-major: longest query tiles of every head first
   mt::attn::Mask& msk = p.mk;
   msk.Sq = Sq; msk.Skv = Skv; msk.n_qt = (Sq + 127) / 128; msk.n_kt = (Skv + 127) / 128;

@@ -306,6 +306,7 @@ void register_attention(pybind11::module_& m);
 void register_moe(pybind11::module_& m);
 void register_comm(pybind11::module_& m);
 void register_serving(pybind11::module_& m);
+void register_hybrid(pybind11::module_& m);
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_supported", &gemm_supported);
@@ -327,6 +328,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("embedding_bwd", &embedding_bwd);
   register_attention(m);
   register_serving(m);
+  register_hybrid(m);
+  register_moe(m);
 #ifndef MT_SERVING_ONLY
   m.def("quantize_fp8", &quantize_fp8);
   m.def("quantize_fp8_with", &quantize_fp8_with);
@@ -334,7 +337,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("xent_fwd_bwd", &xent_fwd_bwd);
   m.def("adamw", &adamw);
   m.def("sumsq", &sumsq);
-  register_moe(m);
   register_comm(m);
 #endif
 }

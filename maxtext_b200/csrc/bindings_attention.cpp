@@ -10,7 +10,7 @@ long mt_attn_tile_ints(int B, int Sq, int Skv);
 int mt_flash_fwd(const void* q, const void* k, const void* v, void* out, float* lse, const int* seg_q, const int* seg_k, const int* pos_q,
                  const int* pos_k, int* tiles, const float* sinks, int B, int Sq, int Skv, int Hq, int Hkv, int Dqk, int Dv, long ldq, long bsq,
                  long ldk, long bsk, long ldv, long bsv, long ldo, long bso, float scale, float softcap, int causal, int window, int chunk,
-                 int q_off, int* status, cudaStream_t st);
+                 int q_off, int cap_mode, int* status, cudaStream_t st);
 int mt_flash_bwd_supported(int Dqk, int Dv);
 int mt_flash_bwd(const void* dout, const void* q, const void* k, const void* v, const void* out, const float* lse, float* delta, void* dq,
                  void* dk, void* dv, const int* seg_q, const int* seg_k, const int* pos_q, const int* pos_k, int* tiles, int B, int Sq, int Skv,
@@ -55,7 +55,7 @@ const int* opt_int(const c10::optional<torch::Tensor>& t, int64_t numel, const c
 void flash_fwd(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, torch::Tensor& out, torch::Tensor& lse,
                const c10::optional<torch::Tensor>& seg_q, const c10::optional<torch::Tensor>& seg_k, const c10::optional<torch::Tensor>& pos_q,
                const c10::optional<torch::Tensor>& pos_k, const c10::optional<torch::Tensor>& sinks, double scale, double softcap, bool causal,
-               int64_t window, int64_t chunk, int64_t q_off) {
+               int64_t window, int64_t chunk, int64_t q_off, int64_t cap_mode) {
   TORCH_CHECK(flash_fwd_supported(q, k, v) && tma_view(out) && lse.is_contiguous() && lse.scalar_type() == torch::kFloat32);
   const int B = (int)q.size(0), Sq = (int)q.size(1), Skv = (int)k.size(1), Hq = (int)q.size(2);
   TORCH_CHECK(out.size(0) == B && out.size(1) == Sq && out.size(2) == Hq && out.size(3) == v.size(3) && lse.numel() == (int64_t)B * Hq * Sq);
@@ -68,7 +68,7 @@ void flash_fwd(const torch::Tensor& q, const torch::Tensor& k, const torch::Tens
                         opt_int(seg_k, (int64_t)B * Skv, "seg_k"), opt_int(pos_q, (int64_t)B * Sq, "pos_q"), opt_int(pos_k, (int64_t)B * Skv, "pos_k"),
                         pos_q ? tiles.data_ptr<int>() : nullptr, sinks ? sinks->data_ptr<float>() : nullptr, B, Sq, Skv, Hq, (int)k.size(2),
                         (int)q.size(3), (int)v.size(3), q.stride(1), q.stride(0), k.stride(1), k.stride(0), v.stride(1), v.stride(0),
-                        out.stride(1), out.stride(0), (float)scale, (float)softcap, causal ? 1 : 0, (int)window, (int)chunk, (int)q_off,
+                        out.stride(1), out.stride(0), (float)scale, (float)softcap, causal ? 1 : 0, (int)window, (int)chunk, (int)q_off, (int)cap_mode,
                         mt_status_ptr(), at::cuda::getCurrentCUDAStream().stream());
   TORCH_CHECK(rc == 0, "mt_flash_fwd failed with code ", rc);
   mt_count_launches(pos_q ? 3 : 1);
@@ -146,7 +146,9 @@ void register_attention(pybind11::module_& m) {
   m.def("sample_tokens", &sample_tokens);
   m.def("decode_attention", &decode_attention);
   m.def("flash_fwd_supported", &flash_fwd_supported);
-  m.def("flash_fwd", &flash_fwd);
+  m.def("flash_fwd", &flash_fwd, pybind11::arg("q"), pybind11::arg("k"), pybind11::arg("v"), pybind11::arg("out"), pybind11::arg("lse"), pybind11::arg("seg_q"),
+        pybind11::arg("seg_k"), pybind11::arg("pos_q"), pybind11::arg("pos_k"), pybind11::arg("sinks"), pybind11::arg("scale"), pybind11::arg("softcap"),
+        pybind11::arg("causal"), pybind11::arg("window"), pybind11::arg("chunk"), pybind11::arg("q_off"), pybind11::arg("cap_mode") = 0);
 #ifndef MT_SERVING_ONLY
   m.def("flash_bwd_supported", &flash_bwd_supported);
   m.def("flash_bwd", &flash_bwd);

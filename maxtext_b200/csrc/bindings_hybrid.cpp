@@ -1,0 +1,267 @@
+// Bindings of the inference kernels for several residual streams, selective scans, attention over a key/value cache and routed experts with
+// scaled inputs. Every entry checks types, layouts and sizes before it launches; pointers handed to the kernels are in bounds for the sizes
+// given with them.
+#include <torch/extension.h>
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <cuda_runtime.h>
+
+extern "C" {
+int mt_stream_mix(float* x, int k, const void* branch, const int* dest, int per_token, const void* mix, const void* write, const void* read, const void* w,
+                  const void* b, void* y, int f32, long rows, int D, float eps, cudaStream_t st);
+int mt_ssm_conv(int f32, const void* x, long ldx, const void* w, const void* bias, int taps, int C, int S, float* hist, const int64_t* slots,
+                const int64_t* lengths, const int64_t* new_lens, void* y, int B, cudaStream_t st);
+int mt_ssm_scan(int f32, const void* x, const void* z, long ldz, const void* q, long ldq, int off, const float* dt, const void* dt_bias, const void* A_log,
+                const void* D, int C, int N, int S, float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* y, int B,
+                cudaStream_t st);
+int mt_qkv_prep(int f32, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int H, int G, int D, int Dv, const int64_t* pos,
+                const float* inv_ts, int rot, float eps, int S, void* qp, int dq, void* kp, void* vp, int dvp, void* kc, void* vc, long max_len,
+                const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, long N, cudaStream_t st);
+int mt_cached_decode(const void* q, const void* k, const void* v, const int64_t* slots, const int64_t* lengths, long max_len, int B, int H, int G, int D, int Dv,
+                     float scale, float cap, int window, const void* sinks, const void* gate, long ldg, int splits, float* part, float* ml, void* out,
+                     cudaStream_t st);
+int mt_cached_attention(int f32, const void* q, const void* k, const void* v, long max_len, const int64_t* slots, const int64_t* lengths, int B, int S, int H,
+                        int G, int D, int Dv, float scale, float cap, int window, const void* sinks, void* out, cudaStream_t st);
+int mt_head_gate(int f32, const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, void* out, int sms, cudaStream_t st);
+int mt_expert_up(int f32, const void* x, const void* w0, const void* w1, const float* wts, const int* idx, const int* sizes, const int* offs,
+                 const int* row_pair, int n, int k, int E, int F, int D, float limit, void* h, int sms, cudaStream_t st);
+int mt_expert_down(int f32, const void* h, const void* w, const int* idx, const int* sizes, const int* offs, const int* row_pair, int n, int E, int D, int F,
+                   void* y, int sms, cudaStream_t st);
+int mt_expert_act(const void* gu, const float* wts, const int* row_pair, const int* offs, int E, int F, float limit, void* h, int rows_max, int sms,
+                  cudaStream_t st);
+}
+
+void mt_count_launches(int n); // defined in bindings.cpp
+int mt_num_sms();              // defined in bindings.cpp
+
+namespace {
+
+using torch::Tensor;
+using OptTensor = c10::optional<Tensor>;
+
+cudaStream_t stream() { return at::cuda::getCurrentCUDAStream().stream(); }
+
+void done(int rc, const char* what, int launches = 1) {
+  TORCH_CHECK(rc == 0, what, " failed with code ", rc);
+  mt_count_launches(launches);
+}
+bool f32(const Tensor& t) {
+  TORCH_CHECK(t.is_cuda() && (t.scalar_type() == torch::kFloat32 || t.scalar_type() == torch::kBFloat16), "bf16 or fp32 CUDA tensor expected");
+  return t.scalar_type() == torch::kFloat32;
+}
+void same(const Tensor& t, const Tensor& like, int64_t numel, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == like.scalar_type() && t.is_contiguous() && t.numel() == numel, what, ": contiguous tensor of ", numel,
+              " elements of the compute type expected");
+}
+const void* same(const OptTensor& t, const Tensor& like, int64_t numel, const char* what) {
+  if (!t) return nullptr;
+  same(*t, like, numel, what);
+  return t->data_ptr();
+}
+void rows2d(const Tensor& t, const Tensor& like, int64_t n, int64_t cols, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == like.scalar_type() && t.dim() == 2 && t.size(0) == n && t.size(1) >= cols && t.stride(1) == 1, what,
+              ": [", n, ", >= ", cols, "] rows expected");
+}
+void floats(const Tensor& t, int64_t numel, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kFloat32 && t.is_contiguous() && t.numel() == numel, what, ": contiguous fp32 tensor of ", numel,
+              " elements expected");
+}
+const int64_t* longs(const Tensor& t, int64_t n, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kInt64 && t.is_contiguous() && t.numel() == n, what, ": int64 [", n, "] expected");
+  return t.data_ptr<int64_t>();
+}
+const int64_t* longs(const OptTensor& t, int64_t n, const char* what) { return t ? longs(*t, n, what) : nullptr; }
+const int* ints(const Tensor& t, int64_t n, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kInt32 && t.is_contiguous() && t.numel() == n, what, ": int32 [", n, "] expected");
+  return t.data_ptr<int>();
+}
+
+void stream_mix(Tensor& x, const OptTensor& branch, const OptTensor& dest, int64_t per_token, const OptTensor& mix, const OptTensor& write,
+                const OptTensor& read, const OptTensor& w, const OptTensor& b, const OptTensor& y, double eps) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 3 && x.is_contiguous() && x.scalar_type() == torch::kFloat32, "stream_mix: x fp32 [rows, k, D]");
+  const int64_t N = x.size(0), k = x.size(1), D = x.size(2);
+  TORCH_CHECK(branch || y, "stream_mix: nothing to do");
+  TORCH_CHECK(bool(branch) == bool(mix) && bool(branch) == bool(write) && bool(w) == bool(y) && bool(b) == bool(y) && per_token >= 1);
+  const Tensor& like = branch ? *branch : *y;
+  const bool f = f32(like);
+  if (branch) {
+    TORCH_CHECK(branch->dim() == 2 && branch->is_contiguous() && branch->size(1) == D, "stream_mix: branch rows of the model width");
+    if (dest) ints(*dest, N * per_token, "dest");
+    else TORCH_CHECK(branch->size(0) == N * per_token, "stream_mix: ", per_token, " branch rows per token");
+    same(*mix, like, k * k, "mix");
+    same(*write, like, k, "write");
+  }
+  if (y) { same(*y, like, N * D, "y"); same(*w, like, D, "norm weight"); same(*b, like, D, "norm bias"); }
+  const void* rd = same(read, like, k, "read");
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_stream_mix(x.data_ptr<float>(), (int)k, branch ? branch->data_ptr() : nullptr, dest ? dest->data_ptr<int>() : nullptr, (int)per_token,
+                     mix ? mix->data_ptr() : nullptr, write ? write->data_ptr() : nullptr, rd, w ? w->data_ptr() : nullptr, b ? b->data_ptr() : nullptr,
+                     y ? y->data_ptr() : nullptr, f, N, (int)D, (float)eps, stream()), "stream_mix");
+}
+
+// x [B*S, >= C] projection rows, w [taps, C], bias [C], hist [slots, taps-1, C] -> y [B*S, C]
+void ssm_conv(const Tensor& x, const Tensor& w, const Tensor& bias, int64_t S, Tensor& hist, const Tensor& slots, const Tensor& lengths,
+              const OptTensor& new_lens, Tensor& y) {
+  const bool f = f32(x);
+  TORCH_CHECK(w.dim() == 2 && w.size(0) >= 1);
+  const int64_t B = slots.numel(), taps = w.size(0), C = w.size(1);
+  rows2d(x, x, B * S, C, "projection");
+  TORCH_CHECK((reinterpret_cast<uintptr_t>(x.data_ptr()) % 16) == 0);
+  same(w, x, taps * C, "filter"); same(bias, x, C, "bias"); same(y, x, B * S * C, "y");
+  TORCH_CHECK(hist.is_cuda() && hist.scalar_type() == torch::kFloat32 && hist.is_contiguous() && hist.dim() == 3 && hist.size(1) == taps - 1 && hist.size(2) == C);
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_ssm_conv(f, x.data_ptr(), x.stride(0), w.data_ptr(), bias.data_ptr(), (int)taps, (int)C, (int)S, hist.data_ptr<float>(), longs(slots, B, "slots"),
+                   longs(lengths, B, "lengths"), longs(new_lens, B, "new_lens"), y.data_ptr(), (int)B, stream()), "ssm_conv");
+}
+
+// x [B*S, C]; p [B*S, 2C] projection rows whose second half is the gate; q [B*S, >= off + 2N]; dt fp32 [B*S, C]; rec [slots, 1, C, N] -> y [B*S, C]
+void ssm_scan(const Tensor& x, const Tensor& p, const Tensor& q, const Tensor& dt, const Tensor& dt_bias, const Tensor& A_log, const Tensor& D, int64_t off,
+              int64_t N, int64_t S, Tensor& rec, const Tensor& slots, const Tensor& lengths, const OptTensor& new_lens, Tensor& y) {
+  const bool f = f32(x);
+  const int64_t B = slots.numel(), C = D.numel();
+  same(x, x, B * S * C, "x"); same(y, x, B * S * C, "y");
+  rows2d(p, x, B * S, 2 * C, "projection");
+  rows2d(q, x, B * S, off + 2 * N, "step size, B, C");
+  floats(dt, B * S * C, "dt");
+  same(dt_bias, x, C, "dt bias"); same(A_log, x, C * N, "A_log"); same(D, x, C, "D");
+  TORCH_CHECK(rec.is_cuda() && rec.scalar_type() == torch::kFloat32 && rec.is_contiguous() && rec.dim() == 4 && rec.size(1) == 1 && rec.size(2) == C &&
+              rec.size(3) == N, "ssm_scan: state of the wrong size");
+  c10::cuda::CUDAGuard guard(x.device());
+  const char* z = static_cast<const char*>(p.data_ptr()) + C * p.element_size();
+  done(mt_ssm_scan(f, x.data_ptr(), z, p.stride(0), q.data_ptr(), q.stride(0), (int)off, dt.data_ptr<float>(), dt_bias.data_ptr(), A_log.data_ptr(),
+                   D.data_ptr(), (int)C, (int)N, (int)S, rec.data_ptr<float>(), longs(slots, B, "slots"), longs(lengths, B, "lengths"),
+                   longs(new_lens, B, "new_lens"), y.data_ptr(), (int)B, stream()), "ssm_scan");
+}
+
+void check_cache(const Tensor& k, const Tensor& v, const Tensor& like, int64_t D) {
+  TORCH_CHECK(k.dim() == 4 && v.dim() == 4 && k.size(0) == v.size(0) && k.size(1) == v.size(1) && k.size(2) == v.size(2) && k.size(3) == D,
+              "cache: keys and values of different shapes");
+  same(k, like, k.numel(), "key cache");
+  same(v, like, v.numel(), "value cache");
+}
+
+// q / k / v rows of the projections -> qp [N, H, dq], kp [N, G, dq] or None, vp [N, G, dvp] or None, cache rows; rot: rotated lanes; eps < 0: no norm
+void qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, int64_t D, int64_t Dv, const Tensor& pos, const OptTensor& inv_ts, int64_t rot, double eps,
+              Tensor& qp, const OptTensor& kp, const OptTensor& vp, Tensor& kc, Tensor& vc, const Tensor& slots, const Tensor& lengths,
+              const OptTensor& new_lens) {
+  const bool f = f32(q);
+  TORCH_CHECK(qp.dim() == 3 && rot % 2 == 0 && rot >= 0 && rot <= D && bool(inv_ts) == (rot > 0));
+  const int64_t N = q.size(0), H = qp.size(1), dq = qp.size(2), B = slots.numel();
+  check_cache(kc, vc, q, D);
+  const int64_t G = kc.size(2);
+  TORCH_CHECK(vc.size(3) == Dv && B > 0 && N % B == 0 && dq >= D && H % G == 0);
+  rows2d(q, q, N, H * D, "q"); rows2d(k, q, N, G * D, "k"); rows2d(v, q, N, G * Dv, "v");
+  same(qp, q, N * H * dq, "packed q");
+  if (kp) same(*kp, q, N * G * dq, "packed k");
+  int64_t dvp = Dv;
+  if (vp) { dvp = vp->size(vp->dim() - 1); TORCH_CHECK(dvp >= Dv); same(*vp, q, N * G * dvp, "packed v"); }
+  if (inv_ts) floats(*inv_ts, rot / 2, "inverse timescales");
+  c10::cuda::CUDAGuard guard(q.device());
+  done(mt_qkv_prep(f, q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), (int)H, (int)G, (int)D, (int)Dv,
+                   longs(pos, N, "positions"), inv_ts ? inv_ts->data_ptr<float>() : nullptr, (int)rot, (float)eps, (int)(N / B), qp.data_ptr(), (int)dq,
+                   kp ? kp->data_ptr() : nullptr, vp ? vp->data_ptr() : nullptr, (int)dvp, kc.data_ptr(), vc.data_ptr(), kc.size(1), longs(slots, B, "slots"),
+                   longs(lengths, B, "lengths"), longs(new_lens, B, "new_lens"), N, stream()), "qkv_prep");
+}
+
+// parts of the key range that fill the machine twice over without making a part shorter than four tiles
+int64_t cached_decode_splits(int64_t B, int64_t H, int64_t G, int64_t span) {
+  const int64_t ctas = std::max<int64_t>(1, B * G * ((H / G + 15) / 16));
+  return std::max<int64_t>(1, std::min<int64_t>({64, 2 * mt_num_sms() / ctas, (span + 63) / 64}));
+}
+
+void cached_decode(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& slots, const Tensor& lengths, double scale, double cap, int64_t window,
+                   const OptTensor& sinks, const OptTensor& gate, int64_t splits, Tensor& part, Tensor& ml, Tensor& out) {
+  TORCH_CHECK(!f32(q) && q.dim() == 3 && q.is_contiguous());
+  const int64_t B = q.size(0), H = q.size(1), D = q.size(2);
+  check_cache(k, v, q, D);
+  const int64_t G = k.size(2), Dv = v.size(3);
+  TORCH_CHECK(H % G == 0 && splits >= 1);
+  floats(part, B * H * splits * Dv, "part"); floats(ml, B * H * splits * 2, "ml");
+  same(out, q, B * H * Dv, "out");
+  const void* sk = same(sinks, q, H, "sinks");
+  if (gate) rows2d(*gate, q, B, H * Dv, "gate");
+  c10::cuda::CUDAGuard guard(q.device());
+  done(mt_cached_decode(q.data_ptr(), k.data_ptr(), v.data_ptr(), longs(slots, B, "slots"), longs(lengths, B, "lengths"), k.size(1), (int)B, (int)H, (int)G,
+                        (int)D, (int)Dv, (float)scale, (float)cap, (int)window, sk, gate ? gate->data_ptr() : nullptr, gate ? gate->stride(0) : 0, (int)splits,
+                        part.data_ptr<float>(), ml.data_ptr<float>(), out.data_ptr(), stream()), "cached_decode", 2);
+}
+
+void cached_attention(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& slots, const Tensor& lengths, int64_t S, double scale, double cap,
+                      int64_t window, const OptTensor& sinks, Tensor& out) {
+  const bool f = f32(q);
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous());
+  const int64_t B = slots.numel(), H = q.size(1), D = q.size(2);
+  check_cache(k, v, q, D);
+  const int64_t G = k.size(2), Dv = v.size(3);
+  TORCH_CHECK(q.size(0) == B * S && H % G == 0);
+  same(out, q, B * S * H * Dv, "out");
+  const void* sk = same(sinks, q, H, "sinks");
+  c10::cuda::CUDAGuard guard(q.device());
+  done(mt_cached_attention(f, q.data_ptr(), k.data_ptr(), v.data_ptr(), k.size(1), longs(slots, B, "slots"), longs(lengths, B, "lengths"), (int)B, (int)S, (int)H,
+                           (int)G, (int)D, (int)Dv, (float)scale, (float)cap, (int)window, sk, out.data_ptr(), stream()), "cached_attention");
+}
+
+// o [N, H, >= dv], g [N, >= H * dv] -> out [N, H * dv]
+void head_gate(const Tensor& o, const Tensor& g, int64_t dv, Tensor& out) {
+  const bool f = f32(o);
+  TORCH_CHECK(o.dim() == 3 && o.is_contiguous() && o.size(2) >= dv);
+  const int64_t N = o.size(0), H = o.size(1);
+  rows2d(g, o, N, H * dv, "gate");
+  same(out, o, N * H * dv, "out");
+  c10::cuda::CUDAGuard guard(o.device());
+  done(mt_head_gate(f, o.data_ptr(), (int)o.size(2), g.data_ptr(), g.stride(0), N, (int)(H * dv), (int)dv, out.data_ptr(), mt_num_sms(), stream()), "head_gate");
+}
+
+void check_plan(const Tensor& sizes, const Tensor& offs, const Tensor& row_pair, int64_t E) {
+  ints(sizes, E, "sizes"); ints(offs, E + 1, "offs"); ints(row_pair, row_pair.numel(), "row_pair");
+}
+
+void expert_up(const Tensor& x, const Tensor& w0, const Tensor& w1, const Tensor& wts, const Tensor& idx, const Tensor& sizes, const Tensor& offs,
+               const Tensor& row_pair, int64_t k, double limit, Tensor& h) {
+  const bool f = f32(x);
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w0.dim() == 3 && w0.sizes() == w1.sizes() && w0.size(2) == x.size(1));
+  const int64_t E = w0.size(0), F = w0.size(1), D = w0.size(2), n = x.size(0) * k;
+  same(w0, x, E * F * D, "w0"); same(w1, x, E * F * D, "w1"); same(h, x, n * F, "h");
+  floats(wts, n, "scores");
+  check_plan(sizes, offs, row_pair, E);
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_expert_up(f, x.data_ptr(), w0.data_ptr(), w1.data_ptr(), wts.data_ptr<float>(), ints(idx, n, "idx"), sizes.data_ptr<int>(), offs.data_ptr<int>(),
+                    row_pair.data_ptr<int>(), (int)n, (int)k, (int)E, (int)F, (int)D, (float)limit, h.data_ptr(), mt_num_sms(), stream()), "expert_up");
+}
+
+void expert_down(const Tensor& h, const Tensor& w, const Tensor& idx, const Tensor& sizes, const Tensor& offs, const Tensor& row_pair, Tensor& y) {
+  const bool f = f32(h);
+  TORCH_CHECK(h.dim() == 2 && h.is_contiguous() && w.dim() == 3 && w.size(2) == h.size(1));
+  const int64_t E = w.size(0), D = w.size(1), F = w.size(2), n = h.size(0);
+  same(w, h, E * F * D, "w"); same(y, h, n * D, "y");
+  check_plan(sizes, offs, row_pair, E);
+  c10::cuda::CUDAGuard guard(h.device());
+  done(mt_expert_down(f, h.data_ptr(), w.data_ptr(), ints(idx, n, "idx"), sizes.data_ptr<int>(), offs.data_ptr<int>(), row_pair.data_ptr<int>(), (int)n, (int)E,
+                      (int)D, (int)F, y.data_ptr(), mt_num_sms(), stream()), "expert_down");
+}
+
+// gu [rows_max, 2F] of the padded layout -> h [rows_max, F]
+void expert_act(const Tensor& gu, const Tensor& wts, const Tensor& row_pair, const Tensor& offs, double limit, Tensor& h) {
+  TORCH_CHECK(!f32(gu) && gu.dim() == 2 && gu.is_contiguous() && h.dim() == 2 && gu.size(1) == 2 * h.size(1) && h.size(1) % 8 == 0);
+  same(h, gu, gu.size(0) * h.size(1), "h");
+  ints(row_pair, gu.size(0), "row_pair"); ints(offs, offs.numel(), "offs"); floats(wts, wts.numel(), "scores");
+  c10::cuda::CUDAGuard guard(gu.device());
+  done(mt_expert_act(gu.data_ptr(), wts.data_ptr<float>(), row_pair.data_ptr<int>(), offs.data_ptr<int>(), (int)offs.numel() - 1, (int)h.size(1), (float)limit,
+                     h.data_ptr(), (int)gu.size(0), mt_num_sms(), stream()), "expert_act");
+}
+
+}  // namespace
+
+void register_hybrid(pybind11::module_& m) {
+  m.def("stream_mix", &stream_mix);
+  m.def("ssm_conv", &ssm_conv);
+  m.def("ssm_scan", &ssm_scan);
+  m.def("qkv_prep", &qkv_prep);
+  m.def("cached_decode_splits", &cached_decode_splits);
+  m.def("cached_decode", &cached_decode);
+  m.def("cached_attention", &cached_attention);
+  m.def("head_gate", &head_gate);
+  m.def("expert_up", &expert_up);
+  m.def("expert_down", &expert_down);
+  m.def("expert_act", &expert_act);
+}

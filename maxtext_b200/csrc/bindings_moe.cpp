@@ -43,6 +43,7 @@ bool bf16_rows(const torch::Tensor& t) {
 }
 
 // idx [n] int32 -> fills sizes [E], offs [E+1], blk_expert [rows_max/128], dest [n], row_pair [rows_max]
+#ifndef MT_SERVING_ONLY
 // ---- block-scaled FP8 (gemm_fp8_block_sm100.cu)
 // x [R, C] bf16 -> (q [R, C] uint8 holding e4m3, scales_t [ceil(C/128), R] fp32)
 std::vector<torch::Tensor> quant_fp8_rows(const torch::Tensor& x) {
@@ -101,6 +102,8 @@ void gemm_fp8_block(const torch::Tensor& aq, const torch::Tensor& sa, const torc
   TORCH_CHECK(rc == 0, "mt_gemm_fp8_block failed with code ", rc);
   mt_count_launches(1);
 }
+
+#endif
 
 // logits [T,E] fp32 / bf16 -> (idx [T,k] int32, wts [T,k] fp32, probs [T,E] fp32, counts [E] int32), see router_sm100.cu
 std::vector<torch::Tensor> router_topk(const torch::Tensor& logits, const c10::optional<torch::Tensor>& bias, int64_t k, int64_t mode,
@@ -201,6 +204,7 @@ void grouped_gemm(int64_t mode, const torch::Tensor& a, const torch::Tensor& b, 
   mt_count_launches(1);
 }
 
+#ifndef MT_SERVING_ONLY
 // ---- expert-parallel dispatch over peer memory. `*_table` tensors are int64 device arrays of per-rank base addresses.
 void ep_put_counts(const torch::Tensor& sizes, int64_t my_rank, const torch::Tensor& counts_table) {
   TORCH_CHECK(i32(sizes) && counts_table.is_cuda() && counts_table.scalar_type() == torch::kInt64);
@@ -257,18 +261,24 @@ void ep_zero_pads(torch::Tensor& buf, const torch::Tensor& offs, const torch::Te
   mt_count_launches(1);
 }
 
+#endif
+
 }  // namespace
 
 void register_moe(pybind11::module_& m) {
+#ifndef MT_SERVING_ONLY
   m.def("ep_put_counts", &ep_put_counts);
   m.def("ep_index", &ep_index);
   m.def("ep_push", &ep_push);
   m.def("ep_pull", &ep_pull);
   m.def("ep_zero_pads", &ep_zero_pads);
+#endif
   m.def("router_topk", &router_topk);
+#ifndef MT_SERVING_ONLY
   m.def("quant_fp8_rows", &quant_fp8_rows);
   m.def("quant_fp8_blocks", &quant_fp8_blocks);
   m.def("gemm_fp8_block", &gemm_fp8_block);
+#endif
   m.def("moe_sort", &moe_sort);
   m.def("moe_gather", &moe_gather);
   m.def("moe_combine", &moe_combine);

@@ -6,7 +6,7 @@
 //   mode 0  selection on the logits (plus an optional per-expert bias); weights = softmax over the k selected logits, or
 //           the raw logits (`raw_weights`, Llama-4 style); probs = softmax over all experts (for the load-balance loss)
 //   mode 1  DeepSeek style: scores = softmax or sigmoid of the logits, selection on scores + bias, weights = the selected
-//           scores (renormalised over the k for sigmoid scores) times a scaling factor; probs = scores
+//           scores (renormalised over the k for sigmoid scores unless `raw_weights`) times a scaling factor; probs = scores
 // The gradient of these few small tensors is taken in PyTorch from the saved outputs.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -110,7 +110,7 @@ __global__ void router_topk_kernel(const T* __restrict__ logits, const float* __
   float w;
   if (mode == 1) {
     w = lane < k ? wscore : 0.f;
-    if (sigmoid_scores) { const float tot = warp_sum(w); w = w / (tot + 1e-20f); }
+    if (sigmoid_scores && !raw_weights) { const float tot = warp_sum(w); w = w / (tot + 1e-20f); }
     w *= scaling;
   } else if (raw_weights) {
     w = lane < k ? wscore : 0.f;

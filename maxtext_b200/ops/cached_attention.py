@@ -60,19 +60,21 @@ def serve(layer, q, k, v, g, ctx):
   pack_k = widths is not None and fresh                  # later portions read their keys from the cache
   qp = torch.empty(N, H, dq, dtype=q.dtype, device=q.device)
   kp = torch.empty(N, G, dq, dtype=q.dtype, device=q.device) if pack_k else None
-  vp = torch.empty(N, G, dvp, dtype=q.dtype, device=q.device) if pack_k and dvp != Dv else None
+  copy_v = pack_k and (dvp != Dv or v.stride(0) % 8 != 0 or v.data_ptr() % 16 != 0)
+  vp = torch.empty(N, G, dvp, dtype=q.dtype, device=q.device) if copy_v else None
   E.qkv_prep(q, k, v, D, Dv, ctx.positions.contiguous(), layer.inv_ts if rot else None, rot, eps if layer.l2_qk_norm else -1.0, qp, kp, vp, cache.k, cache.v,
              cache.slot_ids, cache.lengths, cache.new_lens)
   if S == 1:
     return decode(qp, cache, scale, cap, win, sinks, g)
   if widths is None:
     return plain(qp, cache, S, scale, cap, win, sinks, g)
+  # normalised q and k bound every score by D * scale
+  mode = F.CAP_SMALL if layer.l2_qk_norm and D * abs(scale) <= 0.3 * cap else F.CAP_EXACT
   if fresh:
-    vv = vp if vp is not None else v
-    o = _flash(qp.view(B, S, H, dq), kp.view(B, S, G, dq), vv.view(B, S, G, dvp) if vp is not None else _rows(vv, B, S, G, Dv), ctx.positions,
-               ctx.segment_ids, scale, cap, win, sinks)
+    o = _flash(qp.view(B, S, H, dq), kp.view(B, S, G, dq), vp.view(B, S, G, dvp) if vp is not None else _rows(v, B, S, G, Dv), ctx.positions,
+               ctx.segment_ids, scale, cap, win, sinks, mode)
   else:
-    o = _portion(qp.view(B, S, H, dq), cache, ctx, scale, cap, win, sinks, D, Dv)
+    o = _portion(qp.view(B, S, H, dq), cache, ctx, scale, cap, win, sinks, mode, D, Dv)
   return _gate(o.view(N, H, dvp), g, H, Dv)
 
 
@@ -81,11 +83,11 @@ def _rows(v, B, S, G, Dv):
   return v.as_strided((B, S, G, Dv), (S * v.stride(0), v.stride(0), Dv, 1), v.storage_offset())
 
 
-def _flash(q, k, v, positions, segment_ids, scale, cap, win, sinks, kv_positions=None):
-  return F.attention_fwd(q, k, v, positions, segment_ids, scale, cap, win, kv_positions=kv_positions, sinks=sinks)[0]
+def _flash(q, k, v, positions, segment_ids, scale, cap, win, sinks, mode, kv_positions=None):
+  return F.attention_fwd(q, k, v, positions, segment_ids, scale, cap, win, kv_positions=kv_positions, sinks=sinks, cap_mode=mode)[0]
 
 
-def _portion(q, cache, ctx, scale, cap, win, sinks, D, Dv):
+def _portion(q, cache, ctx, scale, cap, win, sinks, mode, D, Dv):
   """Queries that follow cached tokens: the keys they can see are gathered from the cache (padded to the flash widths)."""
   B, S, H, dq = q.shape
   dvp = flash_widths(D, Dv)[1]
@@ -99,7 +101,7 @@ def _portion(q, cache, ctx, scale, cap, win, sinks, D, Dv):
   k, v = cache.k[slots, rows], cache.v[slots, rows]
   k = torch.nn.functional.pad(k, (0, dq - D)) if dq != D else k
   v = torch.nn.functional.pad(v, (0, dvp - Dv)) if dvp != Dv else v
-  return _flash(q, k, v, ctx.positions, None, scale, cap, win, sinks, kv_pos)
+  return _flash(q, k, v, ctx.positions, None, scale, cap, win, sinks, mode, kv_pos)
 
 
 def decode_widths_ok(D: int, Dv: int, dtype) -> bool:

@@ -465,8 +465,11 @@ def _i32(t):
   return None if t is None else t.to(torch.int32).contiguous()
 
 
+CAP_FAST, CAP_EXACT, CAP_SMALL = 0, 1, 2      # the flash kernel's soft cap: tanh instruction; fp32; fp32 for |scale * q.k| <= 0.3 soft_cap
+
+
 def attention_fwd(q, k, v, positions, segment_ids, scale, soft_cap, window, causal=True, kv_positions=None,
-                  kv_segment_ids=None, chunk=0, sinks=None):
+                  kv_segment_ids=None, chunk=0, sinks=None, cap_mode=CAP_FAST):
   """Returns (out [B,Sq,Hq,Dv], lse [B,Hq,Sq] fp32). Strided q/k/v views are accepted.
 
   On a GPU this is the tcgen05 flash kernel for every mask form the models use: causal or not, sliding window, chunked
@@ -487,7 +490,7 @@ def attention_fwd(q, k, v, positions, segment_ids, scale, soft_cap, window, caus
       pos_k = _i32(kv_positions if kv_positions is not None else positions) if by_arrays else None
       sk = sinks.detach().float().contiguous() if sinks is not None else None
       E.flash_fwd(q, k, v, out, lse, seg_q, seg_k, pos_q, pos_k, sk, float(scale), float(soft_cap or 0.0), bool(causal), int(window or 0),
-                  int(chunk or 0), int(k.shape[1] - q.shape[1]) if not by_arrays else 0)
+                  int(chunk or 0), int(k.shape[1] - q.shape[1]) if not by_arrays else 0, int(cap_mode))
       return out, lse
   mask_args = dict(q_pos=positions, kv_pos=kv_positions if kv_positions is not None else positions, q_seg=segment_ids,
                    kv_seg=kv_segment_ids if kv_segment_ids is not None else segment_ids, causal=causal,

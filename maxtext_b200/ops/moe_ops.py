@@ -371,7 +371,7 @@ def serve_scaled(x2: torch.Tensor, layer) -> ExpertRows:
     E_.grouped_gemm(1, h, wo, rows, plan.offs, plan.blk_expert, False)
     return ExpertRows(rows, plan.dest, k)
   h = torch.empty(n, Fdim, dtype=dt, device=dev)
-  E_.expert_up(x2, w0, w1, wts.view(-1), plan.sizes, plan.offs, plan.row_pair, k, float(layer.limit), h)
+  E_.expert_up(x2, w0, w1, wts.view(-1), idx.view(-1), plan.sizes, plan.offs, plan.row_pair, k, float(layer.limit), h)
   y = torch.empty(n, D, dtype=dt, device=dev)
-  E_.expert_down(h, wo, plan.sizes, plan.offs, plan.row_pair, y)
+  E_.expert_down(h, wo, idx.view(-1), plan.sizes, plan.offs, plan.row_pair, y)
   return ExpertRows(y, None, k)
