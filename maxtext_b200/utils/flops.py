@@ -76,7 +76,13 @@ def training_tflops_per_device(c, batch_per_device: float | None = None) -> tupl
 def _sized_mixer(bp, B, S, d):
   """The same for a block that brings its own mixer sizes (`layer_specs`)."""
   bs, m = B * S, bp.mixer
+  if bp.attention == "ssm":
+    c, n, r = m["inner"], m["state"], m["dt_rank"]
+    return 2 * bs * (3 * d * c + c * (r + 2 * n) + r * c + m["conv"] * c), 7 * bs * c * n
   H, dv = m["heads"], m["vdim"]
+  if bp.attention == "gqa":
+    w = d * (H * m["dim"] + m["kv_heads"] * (m["dim"] + dv) + 2 * H * dv)
+    return 2 * bs * w, bs * S * H * (m["dim"] + dv)
   if bp.attention == "mla":
     qk = m["dim"] + m["rot_dim"]
     w = d * m["q_rank"] + m["q_rank"] * H * qk + d * (m["kv_rank"] + m["rot_dim"]) + m["kv_rank"] * H * (m["dim"] + dv) + H * dv * d
@@ -123,6 +129,9 @@ def _block(c, bp, B, S, n_act):
       attn = 4 * bs * S * c.num_query_heads * dh / 2
   if bp.mlp == "none":
     ffn = 0
+  elif bp.moe is not None:
+    r = bp.moe["router"]
+    ffn = 2 * bs * d * r["experts"] + _ffn(bs, d, bp.moe["expert"]["ff"], n_act) * r["top"]
   elif bp.mlp in ("moe", "moe_shared", "gemma4_moe"):
     ffn = 2 * bs * d * c.num_experts + _ffn(bs, d, c.moe_mlp_dim, n_act) * c.num_experts_per_tok
     if bp.mlp == "moe_shared" and c.shared_experts > 0:
