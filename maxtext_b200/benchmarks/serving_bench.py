@@ -1,4 +1,4 @@
-"""Serving throughput of a mixed-mixer model beside plain models of equal size, and the device time of every serving kernel.
+"""Serving throughput of the mixed-mixer models beside plain models of equal size, and the device time of every serving kernel.
 
 `python bench.py --serving [--serving-models a,b] [--serving-lengths 512,2048] [--serving-slots 1,32]` prints one JSON line per model:
 
@@ -6,7 +6,7 @@
   decode:  tokens/s of a full decode state per slot count, every slot holding `context` tokens, CUDA-graph replay
   kernels: device microseconds per launch by kernel (PyTorch profiler, a separate untimed pass), one prompt and one decode step
 
-and one last line `rooflines`: every serving kernel at silinex-1b's layer sizes (8192 prompt tokens; 128 sequences with 2048 cached tokens),
+and one last line `rooflines`: every serving kernel at silinex-1b's and tipidra-1b's layer sizes (8192 prompt tokens; 128 sequences with 2048 cached tokens),
 its time by CUDA events with L2 flushed, its algorithmic bytes or products, and the fraction of the measured copy bandwidth or GEMM rate,
 beside the like operation of the models that existed before (`like`).
 
@@ -16,6 +16,9 @@ Weights are random; the work does not depend on their values. The models:
   mla-1b       the same width, depth and feed-forward size with the DeepSeek block (latent attention in every layer, gated MLP of equal size)
   llama-1b     the same with grouped-query attention
   silinex-5b, mla-5b   the same two at width 4096, 32 heads, 24 layers
+  tipidra-1b   the catalog entry: capped attention and selective-scan layers in turn, every other pair with routed experts, two residual streams
+  moe-1b       the same width, depth and active weights with the Mixtral block (grouped-query attention, routed experts in every layer)
+  tipidra-5b, moe-5b   the same two at width 4096, 32 heads, 24 layers
 """
 from __future__ import annotations
 
@@ -47,12 +50,33 @@ def _plain(width, heads, ff, layers, q_rank=0):
   return dict(keys, decoder_block="llama2", base_num_kv_heads=heads // 2, head_dim=128)
 
 
+def _tipidra(width, heads, ff, expert_ff, layers):
+  """Capped attention and selective scans (twice the width, 16 states) in turn; dense, routed, routed, dense feed-forwards in turn."""
+  a = {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "rot": {"base": 500000.0, "dims": 64}, "scale": 128 ** -0.5, "softcap": 40.0}
+  s = {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}
+  dense, routed = {"kind": "dense", "ff": ff}, {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": expert_ff, "limit": 7.0}}
+  kinds = [{"type": "attention", "mixer": a, "mlp": dense}, {"type": "mamba1", "mixer": s, "mlp": routed},
+           {"type": "attention", "mixer": a, "mlp": routed}, {"type": "mamba1", "mixer": s, "mlp": dense}]
+  return dict(decoder_block="tipidra", base_emb_dim=width, base_num_decoder_layers=layers, layer_specs=[kinds[i % 4] for i in range(layers)],
+              mlp_activations=["gelu", "linear"], embedding_multiplier=width ** 0.5, mhc_expansion_rate=2, final_logits_soft_cap=30.0, vocab_size=65536,
+              logits_via_embedding=False)
+
+
+def _moe(width, heads, expert_ff, layers):
+  return dict(decoder_block="mixtral", base_emb_dim=width, base_num_query_heads=heads, base_num_kv_heads=heads // 4, head_dim=128, base_mlp_dim=expert_ff,
+              base_moe_mlp_dim=expert_ff, num_experts=16, num_experts_per_tok=2, base_num_decoder_layers=layers, vocab_size=65536, logits_via_embedding=False)
+
+
 MODELS = {
     "silinex-1b": dict(model_name="silinex-1b"),
     "mla-1b": _plain(2048, 16, 8192, 18, 768),
     "llama-1b": _plain(2048, 16, 8192, 18),
     "silinex-5b": _silinex(4096, 32, 16384, 24, 1536),
     "mla-5b": _plain(4096, 32, 16384, 24, 1536),
+    "tipidra-1b": dict(model_name="tipidra-1b"),
+    "moe-1b": _moe(2048, 16, 2560, 16),
+    "tipidra-5b": _tipidra(4096, 32, 12288, 4096, 24),
+    "moe-5b": _moe(4096, 32, 5120, 24),
 }
 
 
@@ -212,6 +236,47 @@ def rooflines(iters: int = 10) -> dict:
     add("flash forward, window 2048", lambda: F.attention_fwd(qp[None], kp[None], vp[None], None, None, 0.1, 0.0, win), 0, 2 * pairs * H * (192 + 128),
         like="flash forward, causal")
     add("flash forward, causal", lambda: F.attention_fwd(qp[None], kp[None], vp[None], None, None, 0.1, 0.0, 0), 0, N * N * H * (192 + 128))
+  # several residual streams, selective scan, capped attention with a gate, experts with scaled inputs
+  xs, mix, wr = t(N, 2, D, dtype=torch.float32), t(2, 2) * 0.1, t(2)
+  add("stream_mix, 2 streams", lambda: E.stream_mix(xs, b, None, 1, mix, wr, wr, w, w, y, 1e-5), N * D * (2 * 2 * 4 + 4), like="rmsnorm")
+  C, NS, rk = 4096, 16, 128
+  px, sx, sy, cw4, cb, q2 = t(N, 2 * C), t(N, C), t(N, C), t(4, C), t(C), t(N, rk + 2 * NS)
+  hist, srec, sdt = t(1, 3, C, dtype=torch.float32), t(1, 1, C, NS, dtype=torch.float32), t(N, C, dtype=torch.float32)
+  A16, D16 = torch.rand(C, NS, device=dev).to(bf), t(C)
+  add("ssm_conv", lambda: E.ssm_conv(px, cw4, cb, N, hist, one, one, None, sx), 4 * N * C, like="delta_conv")
+  add("ssm_scan", lambda: E.ssm_scan(sx, px, q2, sdt, cb, A16, D16, rk, NS, N, srec, one, one, None, sy), N * C * 10 + 4 * N * NS,
+      like="gla_chunks (both kernels)")
+  HQ, HG, hd = 16, 4, 128
+  pk, qo, ko = t(N, (2 * HQ + 2 * HG) * hd), t(N, HQ, hd), t(N, HG, hd)
+  ck, cv, inv64 = t(1, N, HG, hd), t(1, N, HG, hd), torch.rand(32, device=dev)
+  qs, ks, vs, gs = torch.split(pk, [HQ * hd, HG * hd, HG * hd, HQ * hd], -1)
+  pos0 = torch.arange(N, device=dev)
+  add("qkv_prep", lambda: E.qkv_prep(qs, ks, vs, hd, hd, pos0, inv64, 64, 1e-5, qo, ko, None, ck, cv, one, one, None), 2 * N * hd * (2 * HQ + 5 * HG),
+      like="rmsnorm")
+  from ..ops import functional as F
+  with torch.no_grad():
+    vv = vs.as_strided((1, N, HG, hd), (N * vs.stride(0), vs.stride(0), hd, 1), vs.storage_offset())
+    sink = torch.zeros(HQ, device=dev)
+    qn, kn = qo[None] * 0.1, ko[None]
+    add("flash forward, capped, sink", lambda: F.attention_fwd(qn, kn, vv, None, None, 0.09, 40.0, 0, sinks=sink, cap_mode=F.CAP_SMALL), 0, N * N * HQ * 2 * hd,
+        like="flash forward, causal, 128")
+    add("flash forward, capped by an exponential", lambda: F.attention_fwd(qn, kn, vv, None, None, 0.09, 40.0, 0, sinks=sink, cap_mode=F.CAP_EXACT), 0,
+        N * N * HQ * 2 * hd, like="flash forward, causal, 128")
+    add("flash forward, causal, 128", lambda: F.attention_fwd(qn, kn, vv, None, None, 0.09, 0.0, 0), 0, N * N * HQ * 2 * hd)
+  go_ = t(N, HQ * hd)
+  add("head_gate", lambda: E.head_gate(qo, gs, hd, go_), 6 * N * HQ * hd, like="rmsnorm")
+  from ..ops import moe_ops
+  nE, top, Fe = 16, 2, 2048
+  P = lambda *s: type("P", (), {"data": t(*s)})()  # noqa: E731
+  lay = type("L", (), dict(k=top, E=nE, limit=7.0, gate=P(nE, D), wi_0=P(nE, Fe, D), wi_1=P(nE, Fe, D), wo=P(nE, D, Fe)))()
+  xin = t(N, D)
+  idx, wts, _, _ = E.router_topk(F.mm(xin, lay.gate.data, False, True, out_dtype=torch.float32), None, top, 1, True, True, 1.0)
+  with torch.no_grad():
+    add("experts, scaled inputs (whole layer)", lambda: moe_ops.serve_scaled(xin, lay), 0, 6 * N * top * D * Fe, like="experts, silu (whole layer)")
+    add("experts, silu (whole layer)", lambda: moe_ops.moe_ffn_padded(xin, wts, idx, lay.wi_0, lay.wi_1, lay.wo, nE, "silu"), 0, 6 * N * top * D * Fe)
+  plan = moe_ops.GroupPlan(idx, nE)
+  gu, he = t(plan.rows_max, 2 * Fe), t(plan.rows_max, Fe)
+  add("expert_act", lambda: E.expert_act(gu, wts.view(-1), plan.row_pair, plan.offs, 7.0, he), 6 * N * top * Fe, like="gated_act")
   # ---- decoding: 128 sequences, 2048 cached tokens
   B, L = 128, 2048
   ids, lens = torch.arange(B, device=dev), longs(B, L - 1)
@@ -236,6 +301,38 @@ def rooflines(iters: int = 10) -> dict:
   add("mla_value_up", lambda: E.mla_value_up(part, ml, wb, nope, vout), 2 * H * vd * R + 4 * B * H * R + 2 * B * H * vd, like="gemm, M = 128")
   ga, gw, go = t(B, 2048), t(2048, 2048), t(B, 2048)
   add("gemm, M = 128", lambda: F.mm(ga, gw, False, True, out=go), 2 * (2048 * 2048 + 2 * B * 2048))
+  for Bd in (1, 128):
+    xd = xin[:Bd].contiguous()
+    with torch.no_grad():
+      idx, wts, _, _ = E.router_topk(F.mm(xd, lay.gate.data, False, True, out_dtype=torch.float32), None, top, 1, True, True, 1.0)
+      plan = moe_ops.GroupPlan(idx, nE)
+    hit = int((plan.sizes > 0).sum())
+    hd_, yd = t(Bd * top, Fe), t(Bd * top, D)
+    add(f"expert_up, {Bd} tokens", lambda: E.expert_up(xd, lay.wi_0.data, lay.wi_1.data, wts.view(-1), idx.view(-1), plan.sizes, plan.offs, plan.row_pair, top, 7.0,
+                                                       hd_), 2 * hit * 2 * Fe * D, like=f"experts, silu (whole layer), {Bd} tokens")
+    add(f"expert_down, {Bd} tokens", lambda: E.expert_down(hd_, lay.wo.data, idx.view(-1), plan.sizes, plan.offs, plan.row_pair, yd), 2 * hit * Fe * D,
+        like=f"experts, silu (whole layer), {Bd} tokens")
+    with torch.no_grad():
+      add(f"experts, scaled inputs (whole layer), {Bd} tokens", lambda: moe_ops.serve_scaled(xd, lay), 2 * hit * 3 * Fe * D,
+          like=f"experts, silu (whole layer), {Bd} tokens")
+      add(f"experts, silu (whole layer), {Bd} tokens", lambda: moe_ops.moe_ffn_padded(xd, wts, idx, lay.wi_0, lay.wi_1, lay.wo, nE, "silu"), 2 * hit * 3 * Fe * D)
+  brec, bhist = t(B, 1, C, NS, dtype=torch.float32), t(B, 3, C, dtype=torch.float32)
+  add("ssm_conv, 128 tokens", lambda: E.ssm_conv(px[:B], cw4, cb, 1, bhist, ids, lens, None, sx[:B]), B * C * (4 + 8 * 3), like="delta_decode")
+  add("ssm_scan, 128 tokens", lambda: E.ssm_scan(sx[:B], px[:B], q2[:B], sdt[:B], cb, A16, D16, rk, NS, 1, brec, ids, lens, None, sy[:B]),
+      B * C * (8 * NS + 10) + 2 * C * NS, like="gla_decode")
+  kc4, vc4, q16, g16 = t(B, L, HG, hd), t(B, L, HG, hd), t(B, HQ, hd), t(B, HQ * hd)
+  sinkb = t(HQ)
+  for Bd in (1, 32, 128):
+    sp = E.cached_decode_splits(Bd, HQ, HG, L)
+    pt, ml2, od = t(Bd, HQ, sp, hd, dtype=torch.float32), t(Bd, HQ, sp, 2, dtype=torch.float32), t(Bd, HQ * hd)
+    add(f"cached_decode, {Bd} sequences", lambda: E.cached_decode(q16[:Bd], kc4[:Bd], vc4[:Bd], ids[:Bd], lens[:Bd], 0.09, 40.0, 0, sinkb, g16[:Bd], sp, pt, ml2, od),
+        2 * 2 * Bd * L * HG * hd, like=f"decode_attention, {Bd} sequences")
+    o16 = t(Bd, HQ, hd)
+    sp1 = max(1, min(16, 296 // (Bd * HG)))
+    add(f"decode_attention, {Bd} sequences", lambda: E.decode_attention(q16[:Bd], kc4[:Bd], vc4[:Bd], i32[:Bd], l32[:Bd], o16, 1.0, 0.0, 0, sp1),
+        2 * 2 * Bd * L * HG * hd)
+  add("stream_mix, 128 tokens", lambda: E.stream_mix(xs[:B], b[:B], None, 1, mix, wr, wr, w, w, y[:B], 1e-5), B * D * (2 * 2 * 4 + 4), like="rmsnorm, 128 tokens")
+  add("rmsnorm, 128 tokens", lambda: E.rmsnorm_fwd(b[:B], w, 1e-6, 0.0, y[:B], None), 4 * B * D)
   return {"rooflines": rows, "hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "peaks": peaks["source"]}
 
 

@@ -43,7 +43,6 @@ struct Params {
   attn::Mask mk;
   float scale;           // logits = scale * q.k
   float softcap;         // 0 = none; logits = softcap * tanh(scale * q.k / softcap)
-  int cap_mode;          // CAP_FAST: the tanh instruction (11 bits); CAP_EXACT: fp32; CAP_SMALL: fp32, for |scale * q.k| <= 0.3 softcap
   const float* sinks;    // [Hq] or nullptr
   float* lse;            // [B,Hq,Sq]
   int* status;
@@ -64,21 +63,25 @@ __device__ __forceinline__ float fast_tanh(float x) {
   return y;
 }
 
-enum { CAP_FAST = 0, CAP_EXACT = 1, CAP_SMALL = 2 };
-// tanh(x * pre) of two values. CAP_EXACT from one exponential; CAP_SMALL from the Taylor series up to x^9 (below 2e-8 for |x| <= 0.3)
-__device__ __forceinline__ float2 tanh2(float2 x, float pre, int mode) {
-  if (mode == CAP_SMALL) {
+// Forms of the soft cap. CAP_FAST: the tanh instruction (11 bits); CAP_EXACT: fp32, from one exponential; CAP_SMALL: fp32 for
+// |scale * q.k| <= 0.3 softcap, from the Taylor series up to x^9 (error below 2e-8)
+enum { CAP_NONE = -1, CAP_FAST = 0, CAP_EXACT = 1, CAP_SMALL = 2 };
+// tanh(x * pre) of two values
+template <int CAP>
+__device__ __forceinline__ float2 tanh2(float2 x, float pre) {
+  if constexpr (CAP == CAP_SMALL) {
     const float2 y = __fmul2_rn(x, make_float2(pre, pre)), z = __fmul2_rn(y, y);
     float2 t = __ffma2_rn(z, make_float2(62.f / 2835.f, 62.f / 2835.f), make_float2(-17.f / 315.f, -17.f / 315.f));
     t = __ffma2_rn(z, t, make_float2(2.f / 15.f, 2.f / 15.f));
     t = __ffma2_rn(z, t, make_float2(-1.f / 3.f, -1.f / 3.f));
     return __ffma2_rn(__fmul2_rn(y, z), t, y);
   }
-  if (mode == CAP_EXACT) {
+  else if constexpr (CAP == CAP_EXACT) {
     const float c = 2.f * LOG2E * pre;
     return make_float2(1.f - __fdividef(2.f, 1.f + fast_exp2(x.x * c)), 1.f - __fdividef(2.f, 1.f + fast_exp2(x.y * c)));
+  } else {
+    return make_float2(fast_tanh(x.x * pre), fast_tanh(x.y * pre));
   }
-  return make_float2(fast_tanh(x.x * pre), fast_tanh(x.y * pre));
 }
 
 struct alignas(8) Ctl {
@@ -88,7 +91,7 @@ struct alignas(8) Ctl {
   int pad[2];
 };
 
-template <int DQK, int DV, int NQ>
+template <int DQK, int DV, int NQ, int CAP>
 __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const CUtensorMap& map_k, const CUtensorMap& map_v,
                                                const CUtensorMap& map_o, const Params& p) {
   constexpr int QT = 128 * DQK * 2;          // bytes of a Q or K tile
@@ -253,7 +256,8 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
     const bool row_ok = row < t.rows;
     const bool has_seg = mk.seg_q != nullptr;
     const bool arrays = mk.pos_k != nullptr;
-    const bool cap = p.softcap > 0.f;
+    constexpr bool cap = CAP != CAP_NONE;
+    const float pre = cap ? p.scale / p.softcap : 1.f;
     const float a = cap ? p.softcap * LOG2E : p.scale * LOG2E;     // y = a * s' is the logit in log2 units
     float m = -INFINITY, l = 0.f;                                  // reference maximum (log2 units) and row sum
     int cnt = 0;
@@ -280,7 +284,6 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
       bool none = false;
       [[maybe_unused]] const bool has_seg = MASKED && mk.seg_q != nullptr;
       [[maybe_unused]] const bool arrays = MASKED && mk.pos_k != nullptr;
-      float pre = 1.f;
       if constexpr (MASKED) {
         const int qpos = mk.pos_q ? (row_ok ? mk.pos_q[(long)b * mk.Sq + qg] : 0) : qg + mk.q_off;
         if (has_seg) my_seg = row_ok ? mk.seg_q[(long)b * mk.Sq + qg] : 0;
@@ -288,20 +291,19 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
         attn::key_interval(mk, qpos, lo_p, hi_p);                   // keys this row may attend to, as a closed position interval
         span = (uint32_t)hi_p - (uint32_t)lo_p;                     // lo_p <= position <= hi_p as one unsigned comparison
         none = hi_p < lo_p;
-        if (cap) pre = p.scale / p.softcap;
       }
       // soft-cap (only where the values are needed: it is monotonic, so a maximum can be capped afterwards) and mask of 32 score columns
       // starting at column c0 of the tile
-      auto prepare = [&](uint32_t (&r)[32], int c0, bool values) {
-        if constexpr (MASKED) {
-          if (cap && values) {
+      auto prepare = [&](uint32_t (&r)[32], int c0, auto values) {
+        if constexpr (cap && decltype(values)::value) {
 #pragma unroll
-            for (int e = 0; e < 32; e += 2) {
-              const float2 t = tanh2(make_float2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), pre, p.cap_mode);
-              r[e] = __float_as_uint(t.x);
-              r[e + 1] = __float_as_uint(t.y);
-            }
+          for (int e = 0; e < 32; e += 2) {
+            const float2 t = tanh2<CAP>(make_float2(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), pre);
+            r[e] = __float_as_uint(t.x);
+            r[e + 1] = __float_as_uint(t.y);
           }
+        }
+        if constexpr (MASKED) {
           if (arrays) {
             const int* kp = sk_pos + (i * 2 + par) * 128 + c0;
 #pragma unroll
@@ -327,21 +329,24 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
       tmem_ld_32x32b_x32(tS, r0);
       tmem_ld_wait_dep(r0);
       tmem_ld_32x32b_x32(tS + 32, r1);
-      prepare(r0, 0, false);
+      constexpr std::false_type order{};
+      prepare(r0, 0, order);
       tmax = max32(r0);
       tmem_ld_wait_dep(r1);
       tmem_ld_32x32b_x32(tS + 64, r0);
-      prepare(r1, 32, false);
+      prepare(r1, 32, order);
       tmax = fmaxf(tmax, max32(r1));
       tmem_ld_wait_dep(r0);
       tmem_ld_32x32b_x32(tS + 96, r1);
-      prepare(r0, 64, false);
+      prepare(r0, 64, order);
       tmax = fmaxf(tmax, max32(r0));
       tmem_ld_wait_dep(r1);
       tmem_ld_32x32b_x32(tS, r0);              // first chunk of pass 2
-      prepare(r1, 96, false);
+      prepare(r1, 96, order);
       tmax = fmaxf(tmax, max32(r1));
-      if (MASKED && cap && tmax != -INFINITY) tmax = tanh2(make_float2(tmax, 0.f), pre, p.cap_mode).x;
+      if constexpr (cap) {
+        if (tmax != -INFINITY) tmax = tanh2<CAP>(make_float2(tmax, 0.f), pre).x;
+      }
       const float mt_ = a * tmax;                                    // -inf when the whole row is masked
       const bool grow = mt_ > m + RESCALE_THRESHOLD;                 // m = -inf: any finite maximum grows it
       if (__any_sync(0xffffffffu, grow)) {
@@ -368,7 +373,7 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
       const float2 a2 = make_float2(a, a), neg2 = make_float2(neg, neg);
       float2 rsa = make_float2(0.f, 0.f), rsb = make_float2(0.f, 0.f);
       auto exps = [&](uint32_t (&r)[32], int c) {
-        prepare(r, c * 32, true);
+        prepare(r, c * 32, std::true_type{});
         uint32_t pk[16];
 #pragma unroll
         for (int e = 0; e < 16; ++e) {
@@ -408,7 +413,7 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
       if (cls == 0) continue;
       const int k0 = kt * 128;
       const int par = cnt & 1;
-      const bool masked = cls == 2 || cap;
+      const bool masked = cls == 2;
       if (masked && (mk.pos_k != nullptr || mk.seg_q != nullptr)) {
         const int kg = k0 + wt;
         if (mk.pos_k) sk_pos[(i * 2 + par) * 128 + wt] = kg < mk.Skv ? mk.pos_k[(long)b * mk.Skv + kg] : INT_MAX;
@@ -478,11 +483,11 @@ __device__ __forceinline__ void flash_fwd_body(const CUtensorMap& map_q, const C
 
 // The register file gives 320 threads 168 registers each (warps are allocated in groups of four, so ten warps cost twelve):
 // the 128 scores of a row stay in registers with a few spilled temporaries.
-template <int DQK, int DV, int NQ>
+template <int DQK, int DV, int NQ, int CAP>
 __global__ void __launch_bounds__(64 + 128 * NQ, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                  const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_o, const __grid_constant__ Params p) {
-  flash_fwd_body<DQK, DV, NQ>(map_q, map_k, map_v, map_o, p);
+  flash_fwd_body<DQK, DV, NQ, CAP>(map_q, map_k, map_v, map_o, p);
 }
 
 // (min, max) of every 128-token tile of a position array [B, S]; tiles beyond S are not written. One warp per tile.
@@ -533,17 +538,28 @@ static int tok_map(CUtensorMap* m, const void* ptr, long batch, long tokens, lon
   return r == CUDA_SUCCESS ? 0 : (int)r;
 }
 
-template <int DQK, int DV, int NQ>
-static int run(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mo, const Params& p, cudaStream_t st) {
+template <int DQK, int DV, int NQ, int CAP>
+static int run_cap(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mo, const Params& p, cudaStream_t st) {
   const int smem = NQ * 128 * DQK * 2 + 2 * 128 * DQK * 2 + 2 * 128 * DV * 2 + (int)sizeof(Ctl) + 4096 + 1024;
   static bool cfg = false;
   if (!cfg) {
-    if (cudaFuncSetAttribute(flash_fwd_kernel<DQK, DV, NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
+    if (cudaFuncSetAttribute(flash_fwd_kernel<DQK, DV, NQ, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
     cfg = true;
   }
   const long ctas = (long)p.n_pairs * p.Hq * p.B;
-  flash_fwd_kernel<DQK, DV, NQ><<<(unsigned)ctas, 64 + 128 * NQ, smem, st>>>(mq, mk, mv, mo, p);
+  flash_fwd_kernel<DQK, DV, NQ, CAP><<<(unsigned)ctas, 64 + 128 * NQ, smem, st>>>(mq, mk, mv, mo, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+template <int DQK, int DV, int NQ>
+static int run(int cap_mode, const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mo, const Params& p, cudaStream_t st) {
+  if (!(p.softcap > 0.f)) return run_cap<DQK, DV, NQ, CAP_NONE>(mq, mk, mv, mo, p, st);
+  switch (cap_mode) {
+    case CAP_FAST: return run_cap<DQK, DV, NQ, CAP_FAST>(mq, mk, mv, mo, p, st);
+    case CAP_EXACT: return run_cap<DQK, DV, NQ, CAP_EXACT>(mq, mk, mv, mo, p, st);
+    case CAP_SMALL: return run_cap<DQK, DV, NQ, CAP_SMALL>(mq, mk, mv, mo, p, st);
+    default: return -1;
+  }
 }
 
 }  // namespace fwd
@@ -581,7 +597,7 @@ int mt_flash_fwd(const void* q, const void* k, const void* v, void* out, float* 
   Params p{};
   p.B = B; p.Hq = Hq; p.Hkv = Hkv;
   p.n_pairs = (Sq + 128 * nq - 1) / (128 * nq);
-  p.scale = scale; p.softcap = softcap; p.cap_mode = cap_mode; p.sinks = sinks; p.lse = lse; p.status = status;
+  p.scale = scale; p.softcap = softcap; p.sinks = sinks; p.lse = lse; p.status = status;
   p.head_major = 0;                       // tile-major: longest query tiles of every head first
   mt::attn::Mask& msk = p.mk;
   msk.Sq = Sq; msk.Skv = Skv; msk.n_qt = (Sq + 127) / 128; msk.n_kt = (Skv + 127) / 128;
@@ -593,9 +609,9 @@ int mt_flash_fwd(const void* q, const void* k, const void* v, void* out, float* 
     msk.tile_q = tiles;
     msk.tile_k = tiles + 2l * B * msk.n_qt;
   }
-  if (Dqk == 128) return run<128, 128, 2>(mq, mk, mv, mo, p, st);
-  if (Dqk == 64) return run<64, 64, 2>(mq, mk, mv, mo, p, st);
-  return run<192, 128, 1>(mq, mk, mv, mo, p, st);
+  if (Dqk == 128) return run<128, 128, 2>(cap_mode, mq, mk, mv, mo, p, st);
+  if (Dqk == 64) return run<64, 64, 2>(cap_mode, mq, mk, mv, mo, p, st);
+  return run<192, 128, 1>(cap_mode, mq, mk, mv, mo, p, st);
 }
 
 }  // extern "C"

@@ -3,9 +3,9 @@
 // up-projections in fp32, in front of the clamps:
 //   up:    h[pair] = act(s (Wg x), s (Wu x)),  act(g, u) = min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1)
 //   down:  y[pair] = Wd h[pair]
-// A CTA owns 16 * MW weight rows of one expert. Its four warps sit MW along the rows and 4 / MW along the contraction, operands pass through
-// a three-stage cp.async ring, mma.sync m16n8k16 takes the weights in the M position (a step is bound by reading weights: with a handful of
-// tokens per expert the 128-row tiles of tcgen05 would be empty). Also here: the activation of the padded path, and plain kernels for fp32
+// A persistent CTA works through items of 16 * MW weight rows of one expert. Its four warps sit MW along the rows and 4 / MW along the
+// contraction, operands pass through a cp.async ring of three or four stages, mma.sync m16n8k16 takes the weights in the M position (a step is bound by
+// reading weights: with a handful of tokens per expert the 128-row tiles of tcgen05 would be empty). Also here: the activation of the padded path, and plain kernels for fp32
 // and for widths that are not multiples of 8.
 #include "serving_common.cuh"
 #include "warp_mma.cuh"
@@ -30,49 +30,98 @@ struct Args {
 };
 
 constexpr int NT = 32;        // rows per pass
-constexpr int STAGES = 3;
+// per warp layout: contraction of a stage, and stages, so that at least two CTAs fit an SM
+constexpr int depth(int mw) { return mw == 4 ? 64 : 128; }
+constexpr int stages(int mw) { return mw == 2 ? 3 : 4; }
 
+// One work item: BM weight rows of one expert against up to NT of its rows. Items are numbered expert by expert (experts without rows have
+// none), and a CTA takes every gridDim.x-th one.
+struct Item {
+  int e, r0, m0;              // expert, first of its rows, first weight row
+  int base;                   // number of the expert's first item
+};
+
+template <int BM>
+__device__ __forceinline__ bool find(const Args& a, int E, int number, Item& it) {
+  const int tiles = (a.M + BM - 1) / BM;
+  while (it.e < E) {
+    const int count = (a.sizes[it.e] + NT - 1) / NT * tiles;
+    if (number < it.base + count) {
+      it.r0 = (number - it.base) / tiles * NT;
+      it.m0 = (number - it.base) % tiles * BM;
+      return true;
+    }
+    it.base += count;
+    ++it.e;
+  }
+  return false;
+}
+
+// The ring runs on over item borders: while an item's sums are finished the loads of the next one are in flight.
 template <bool UP, int MW>
 __global__ void __launch_bounds__(128)
-stream_kernel(const Args a) {
-  constexpr int KW = 4 / MW, BM = 16 * MW, BK = MW == 4 ? 64 : (MW == 2 ? 128 : 256), LD = BK + 8, NWT = UP ? 2 : 1;
+stream_kernel(const Args a, int E) {
+  constexpr int KW = 4 / MW, BM = 16 * MW, BK = depth(MW), STAGES = stages(MW), LD = BK + 8, NWT = UP ? 2 : 1, PL = BM + 1;
+  constexpr int V = BK / 8, XR = NT * V / 128;                        // 16-byte pieces of a row; pieces of x per thread
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16* sw = sm;                                             // [STAGES][NWT][BM][LD]
   __nv_bfloat16* sx = sm + STAGES * NWT * BM * LD;                    // [STAGES][NT][LD]
-  __shared__ int rows[NT], pairs[NT];
-  __shared__ float score[NT];
-  const int e = blockIdx.y, m0 = blockIdx.x * BM;
-  const int size = a.sizes[e], off = a.offs[e];
+  float* part = reinterpret_cast<float*>(sx + STAGES * NT * LD);      // [KW][NWT][NT][PL]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wm = warp % MW, wk = warp / MW;
   const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x);
-  const __nv_bfloat16* w[2] = {reinterpret_cast<const __nv_bfloat16*>(a.w0) + (long)e * a.M * a.K,
-                               UP ? reinterpret_cast<const __nv_bfloat16*>(a.w1) + (long)e * a.M * a.K : nullptr};
   const int steps = (a.K + BK - 1) / BK;
-  for (int r0 = 0; r0 < size; r0 += NT) {
-    __syncthreads();
-    if (tid < NT) {
-      const int p = r0 + tid < size ? a.row_pair[off + r0 + tid] : -1;
-      pairs[tid] = p;
-      rows[tid] = p < 0 ? -1 : (UP ? p / a.k : p);
-      if (UP) score[tid] = p < 0 ? 0.f : a.wts[p];
-    }
-    __syncthreads();
-    auto load = [&](int step) {
-      const int st = step % STAGES, k0 = step * BK;
-      constexpr int V = BK / 8;
+
+  // ---- loader: item, step, and what this thread copies of it
+  Item ld{0, 0, 0, 0};
+  int ld_number = blockIdx.x, ld_step = 0, ld_stage = 0;
+  bool ld_more = find<BM>(a, E, ld_number, ld);
+  const __nv_bfloat16* xrow[XR];
+  const __nv_bfloat16 *w0 = nullptr, *w1 = nullptr;
+  auto enter = [&]() {
+    if (!ld_more) return;
+    w0 = reinterpret_cast<const __nv_bfloat16*>(a.w0) + ((long)ld.e * a.M + ld.m0) * a.K;
+    if (UP) w1 = reinterpret_cast<const __nv_bfloat16*>(a.w1) + ((long)ld.e * a.M + ld.m0) * a.K;
+    const int size = a.sizes[ld.e], off = a.offs[ld.e];
 #pragma unroll
-      for (int wt = 0; wt < NWT; ++wt)
-        for (int i = tid; i < BM * V; i += 128) {
-          const int r = i / V, c = (i % V) * 8;
-          const bool ok = m0 + r < a.M && k0 + c < a.K;
-          la_cp_async16(sw + ((st * NWT + wt) * BM + r) * LD + c, ok ? w[wt] + (long)(m0 + r) * a.K + k0 + c : w[wt], ok ? 16 : 0);
-        }
-      for (int i = tid; i < NT * V; i += 128) {
+    for (int j = 0; j < XR; ++j) {
+      const int r = ld.r0 + (tid + j * 128) / V;
+      const int p = r < size ? a.row_pair[off + r] : -1;
+      xrow[j] = p < 0 ? nullptr : x + (long)(UP ? p / a.k : p) * a.K;
+    }
+  };
+  enter();
+  auto load = [&]() {
+    if (ld_more) {
+      const int k0 = ld_step * BK;
+      for (int i = tid; i < BM * V; i += 128) {
         const int r = i / V, c = (i % V) * 8;
-        const bool ok = rows[r] >= 0 && k0 + c < a.K;
-        la_cp_async16(sx + (st * NT + r) * LD + c, ok ? x + (long)rows[r] * a.K + k0 + c : x, ok ? 16 : 0);
+        const bool ok = ld.m0 + r < a.M && k0 + c < a.K;
+        const long at = ok ? (long)r * a.K + k0 + c : 0;
+        la_cp_async16(sw + ((ld_stage * NWT) * BM + r) * LD + c, w0 + at, ok ? 16 : 0);
+        if (UP) la_cp_async16(sw + ((ld_stage * NWT + NWT - 1) * BM + r) * LD + c, w1 + at, ok ? 16 : 0);
       }
-    };
+#pragma unroll
+      for (int j = 0; j < XR; ++j) {
+        const int i = tid + j * 128, r = i / V, c = (i % V) * 8;
+        const bool ok = xrow[j] != nullptr && k0 + c < a.K;
+        la_cp_async16(sx + (ld_stage * NT + r) * LD + c, ok ? xrow[j] + k0 + c : x, ok ? 16 : 0);
+      }
+      if (++ld_step == steps) {
+        ld_step = 0;
+        ld_number += gridDim.x;
+        ld_more = find<BM>(a, E, ld_number, ld);
+        enter();
+      }
+    }
+    ld_stage = ld_stage + 1 == STAGES ? 0 : ld_stage + 1;
+    la_commit();
+  };
+#pragma unroll
+  for (int s = 0; s < STAGES - 1; ++s) load();
+
+  Item it{0, 0, 0, 0};
+  int stage = 0;
+  for (int number = blockIdx.x; find<BM>(a, E, number, it); number += gridDim.x) {
     float acc[NWT][4][4];
 #pragma unroll
     for (int wt = 0; wt < NWT; ++wt)
@@ -80,17 +129,11 @@ stream_kernel(const Args a) {
       for (int j = 0; j < 4; ++j)
 #pragma unroll
         for (int q = 0; q < 4; ++q) acc[wt][j][q] = 0.f;
-    for (int s = 0; s < STAGES - 1; ++s) {
-      if (s < steps) load(s);
-      la_commit();
-    }
     for (int s = 0; s < steps; ++s) {
       la_wait<STAGES - 2>();
       __syncthreads();
-      if (s + STAGES - 1 < steps) load(s + STAGES - 1);
-      la_commit();
-      const int st = s % STAGES;
-      const __nv_bfloat16* xs = sx + st * NT * LD;
+      load();
+      const __nv_bfloat16* xs = sx + stage * NT * LD;
 #pragma unroll
       for (int kk = 0; kk < BK / 16 / KW; ++kk) {
         const int kc = (kk * KW + wk) * 16;
@@ -101,7 +144,7 @@ stream_kernel(const Args a) {
 #pragma unroll
         for (int wt = 0; wt < NWT; ++wt) {
           unsigned aw[4];
-          la_ldm4(aw, sw + ((st * NWT + wt) * BM + wm * 16 + (lane & 15)) * LD + kc + (lane >> 4) * 8);
+          la_ldm4(aw, sw + ((stage * NWT + wt) * BM + wm * 16 + (lane & 15)) * LD + kc + (lane >> 4) * 8);
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
             la_mma(acc[wt][2 * j], aw, bx[j][0], bx[j][1]);
@@ -109,12 +152,9 @@ stream_kernel(const Args a) {
           }
         }
       }
+      stage = stage + 1 == STAGES ? 0 : stage + 1;
     }
-    la_wait<0>();
-    __syncthreads();
-    // partial products of the KW warps through shared memory: part [KW][NWT][NT][BM + 1]
-    float* part = reinterpret_cast<float*>(sm);
-    constexpr int PL = BM + 1;
+    // the KW partial products meet in shared memory (the previous item's were read before this item's first barrier)
 #pragma unroll
     for (int wt = 0; wt < NWT; ++wt)
 #pragma unroll
@@ -123,9 +163,11 @@ stream_kernel(const Args a) {
         for (int q = 0; q < 4; ++q)
           part[((wk * NWT + wt) * NT + j * 8 + (lane & 3) * 2 + (q & 1)) * PL + wm * 16 + (lane >> 2) + (q >> 1) * 8] = acc[wt][j][q];
     __syncthreads();
+    const int left = a.sizes[it.e] - it.r0, off = a.offs[it.e] + it.r0;
     for (int i = tid; i < NT * BM; i += 128) {
       const int t = i / BM, r = i % BM;
-      if (pairs[t] < 0 || m0 + r >= a.M) continue;
+      if (t >= left || it.m0 + r >= a.M) continue;
+      const int p = a.row_pair[off + t];
       float v[NWT];
 #pragma unroll
       for (int wt = 0; wt < NWT; ++wt) {
@@ -134,10 +176,11 @@ stream_kernel(const Args a) {
         for (int q = 0; q < KW; ++q) v[wt] += part[((q * NWT + wt) * NT + t) * PL + r];
       }
       float o = v[0];
-      if constexpr (UP) o = clamped_act(score[t] * v[0], score[t] * v[NWT - 1], a.limit);
-      reinterpret_cast<__nv_bfloat16*>(a.out)[(long)pairs[t] * a.M + m0 + r] = __float2bfloat16_rn(o);
+      if constexpr (UP) o = clamped_act(a.wts[p] * v[0], a.wts[p] * v[NWT - 1], a.limit);
+      reinterpret_cast<__nv_bfloat16*>(a.out)[(long)p * a.M + it.m0 + r] = __float2bfloat16_rn(o);
     }
   }
+  la_wait<0>();
 }
 
 // one warp per output row, one pair at a time
@@ -184,13 +227,14 @@ act_kernel(const __nv_bfloat16* __restrict__ gu, const float* __restrict__ wts, 
 }
 
 template <bool UP, int MW>
-int stream(const Args& a, int E, cudaStream_t st) {
-  constexpr int BM = 16 * MW, BK = MW == 4 ? 64 : (MW == 2 ? 128 : 256), LD = BK + 8, NWT = UP ? 2 : 1, KW = 4 / MW;
-  constexpr int ring = STAGES * (NWT * BM + NT) * LD * 2, part = KW * NWT * NT * (BM + 1) * 4;
-  constexpr int smem = ring > part ? ring : part;
+int stream(const Args& a, int E, int sms, cudaStream_t st) {
+  constexpr int BM = 16 * MW, STAGES = stages(MW), LD = depth(MW) + 8, NWT = UP ? 2 : 1, KW = 4 / MW;
+  constexpr int smem = STAGES * (NWT * BM + NT) * LD * 2 + KW * NWT * NT * (BM + 1) * 4;
   auto k = stream_kernel<UP, MW>;
   if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
-  k<<<dim3((a.M + BM - 1) / BM, E), 128, smem, st>>>(a);
+  const long items = ((long)(a.n < E ? a.n : E) + a.n / NT) * ((a.M + BM - 1) / BM);       // at most
+  const long slots = (long)sms * (227 * 1024 / (smem + 1024));
+  k<<<(unsigned)(items < slots ? items : slots), 128, smem, st>>>(a, E);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -198,11 +242,10 @@ template <bool UP>
 int run(int f32, const Args& a, int E, int sms, cudaStream_t st) {
   if (a.n <= 0) return 0;
   if (!f32 && a.K % 8 == 0) {
-    // CTAs that will find rows: at most one expert per pair
-    const long hit = a.n < E ? a.n : E;
-    if (hit * ((a.M + 63) / 64) >= 2l * sms) return stream<UP, 4>(a, E, st);
-    if (hit * ((a.M + 31) / 32) >= 2l * sms) return stream<UP, 2>(a, E, st);
-    return stream<UP, 1>(a, E, st);
+    const long hit = a.n < E ? a.n : E;                     // experts that will find rows, at most
+    if (hit * ((a.M + 63) / 64) >= 2l * sms) return stream<UP, 4>(a, E, sms, st);
+    if (hit * ((a.M + 31) / 32) >= 2l * sms) return stream<UP, 2>(a, E, sms, st);
+    return stream<UP, 1>(a, E, sms, st);
   }
   const dim3 grid((a.M + 7) / 8, a.n < 65535 ? a.n : 65535);
   if (f32) plain_kernel<float, UP><<<grid, 256, 0, st>>>(a);

@@ -3,11 +3,13 @@
 //   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,   y_c = (sum_n S[c, n] C_n + D_c x_c) * silu(z_c)
 // with dt = softplus(pre-activation + bias) and A = -exp(A_log). States, decays and step sizes are fp32.
 //
-// A channel's states are spread over P neighbouring lanes, NS per lane, and stay in registers over the whole prompt. Half of a CTA's warps
-// run the recurrence; the other half load and prepare the next tile of tokens (softplus, dt * x, B and C as fp32) and finish the previous
-// one (skip, gate, store), so the chain of steps never waits for memory. The read-out of four steps is reduced over the lanes in one
-// transposed exchange. One token per sequence runs a streaming kernel of its own, bound by reading and writing the states.
+// A channel's states are spread over P neighbouring lanes, NS per lane, and stay in registers over the whole prompt. Four of a CTA's twelve
+// warps run the recurrence; the others load and prepare the next tile of tokens (softplus, dt * x, B and C as fp32) and finish the previous
+// one (skip, gate, store), with all loads of a tile in flight together, so the chain of steps never waits for memory. The read-out of four
+// steps is reduced over the lanes in one transposed exchange. One token per sequence runs a streaming kernel of its own, bound by reading
+// and writing the states.
 #include "serving_common.cuh"
+#include <type_traits>
 
 namespace mt {
 namespace ssm {
@@ -118,10 +120,113 @@ struct ScanArgs {
   void* y;
 };
 
-constexpr int SCAN_THREADS = 128;                           // of each role
+constexpr int SCAN_THREADS = 128;                           // that run the recurrence
+constexpr int FEED_THREADS = 256;                           // that load, prepare and finish
+
+// Step size for a bf16 model: hardware exponential and logarithm, the series of log(1 + y) where the logarithm would cancel (relative error
+// below 1e-5 everywhere)
+template <typename T> __device__ __forceinline__ float softplus_t(float x) { return softplus_f(x); }
+template <> __device__ __forceinline__ float softplus_t<__nv_bfloat16>(float x) {
+  const float y = __expf(-fabsf(x));
+  const float series = y * (1.f + y * (-1.f / 2 + y * (1.f / 3 + y * (-1.f / 4 + y * (1.f / 5)))));
+  return fmaxf(x, 0.f) + (y < 0.0625f ? series : __logf(1.f + y));
+}
+
+// both roles of the scan kernel, from their own code
+__device__ __forceinline__ void tile_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(SCAN_THREADS + FEED_THREADS) : "memory"); }
+
+// W values as they lie in memory: converting them where they are loaded would make one load wait for the other
+template <typename T, int W> struct alignas(sizeof(T) * W) Raw { T e[W]; };
+template <typename T, int W> __device__ __forceinline__ Raw<T, W> read_raw(const T* p) { return *reinterpret_cast<const Raw<T, W>*>(p); }
+template <typename T, int W> __device__ __forceinline__ Raw<T, W> fill_raw(float v) {
+  Raw<T, W> r;
+#pragma unroll
+  for (int i = 0; i < W; ++i) r.e[i] = from_f<T>(v);
+  return r;
+}
+
+// What a feeding thread holds of tile `in` on its way to shared memory and of tile `out` on its way to y, W channels at a time, G pieces each.
+// `issue` starts the global loads, `settle` uses them. Tiles outside 0 .. tiles - 1 are skipped.
+template <typename T, int CH, int NP, int TT, int W, int G>
+struct Feeder {
+  static constexpr int CW = CH / W, STEP = FEED_THREADS / CW, ND = (TT + STEP - 1) / STEP;
+  static constexpr int BW = W == 4 ? 16 / (int)sizeof(T) : 1, NB = (TT * 2 * NP / BW + FEED_THREADS - 1) / FEED_THREADS;
+  static constexpr int PIECES = ND > NB ? ND : NB;
+  Raw<float, W> d[G];
+  Raw<T, W> x[G], xo[G], z[G];
+  Raw<T, BW> v[G];
+  float bias[W], skip[W];
+  const T *xb, *zb, *qb;
+  const float* db;
+  T* yb;
+  float *sBC, *sy;
+  float2* sdt;
+  long ldz, ldq;
+  int C, N, tiles, t_end, tid, c, ft;
+  bool live;
+
+  __device__ __forceinline__ void issue(int g, int in, int out) {
+    const bool has_in = in < tiles, has_out = out >= 0 && out < tiles;
+#pragma unroll
+    for (int j = 0; j < G; ++j) {
+      const int r = ft + (g + j) * STEP, t = in * TT + r, to = out * TT + r;
+      const bool row = g + j < ND && r < TT && live;
+      d[j] = fill_raw<float, W>(-INFINITY);                 // padding: softplus 0, so it neither decays nor writes
+      x[j] = fill_raw<T, W>(0.f);
+      if (row && has_in && t < t_end) {
+        d[j] = read_raw<float, W>(db + (long)t * C + c);
+        x[j] = read_raw<T, W>(xb + (long)t * C + c);
+      }
+      if (row && has_out && to < t_end) {
+        xo[j] = read_raw<T, W>(xb + (long)to * C + c);
+        z[j] = read_raw<T, W>(zb + (long)to * ldz + c);
+      }
+      // B and C of a token are neighbours; wide loads are only taken when N fills the padded width
+      const int i = (tid + (g + j) * FEED_THREADS) * BW, tb = in * TT + i / (2 * NP), k = i % (2 * NP), n = k % NP;
+      v[j] = fill_raw<T, BW>(0.f);
+      if (has_in && g + j < NB && i < TT * 2 * NP && tb < t_end && n < N) v[j] = read_raw<T, BW>(qb + (long)tb * ldq + (k / NP) * N + n);
+    }
+  }
+
+  __device__ __forceinline__ void settle(int g, int in, int out) {
+    const bool has_in = in < tiles, has_out = out >= 0 && out < tiles;
+    const int lc = (tid % CW) * W;
+    const float* yy = sy + (out & 1) * TT * CH + lc;
+    float* bc = sBC + (in & 1) * TT * 2 * NP;
+    float2* dd = sdt + (in & 1) * TT * CH + lc;
+#pragma unroll
+    for (int j = 0; j < G; ++j) {
+      const int r = ft + (g + j) * STEP, to = out * TT + r, i = (tid + (g + j) * FEED_THREADS) * BW;
+      const bool row = g + j < ND && r < TT;
+      if (row && live && has_out && to < t_end) {
+        float o[W];
+        load_vec<W>(yy + r * CH, o);
+#pragma unroll
+        for (int e = 0; e < W; ++e) o[e] = (o[e] + skip[e] * to_f(xo[j].e[e])) * silu_t<T>(to_f(z[j].e[e]));
+        store_vec<W>(yb + (long)to * C + c, o);
+      }
+      if (has_in && row) {
+        float p[2 * W];
+#pragma unroll
+        for (int e = 0; e < W; ++e) {
+          p[2 * e] = live && d[j].e[e] != -INFINITY ? softplus_t<T>(d[j].e[e] + bias[e]) : 0.f;
+          p[2 * e + 1] = p[2 * e] * to_f(x[j].e[e]);
+        }
+        if constexpr (W == 4) store_vec<8>(reinterpret_cast<float*>(dd + r * CH), p);
+        else dd[r * CH] = make_float2(p[0], p[1]);
+      }
+      if (has_in && g + j < NB && i < TT * 2 * NP) {
+        float o[BW];
+#pragma unroll
+        for (int e = 0; e < BW; ++e) o[e] = to_f(v[j].e[e]);
+        store_vec<BW>(bc + i, o);
+      }
+    }
+  }
+};
 
 template <typename T, int P, int NS>
-__global__ void __launch_bounds__(2 * SCAN_THREADS)
+__global__ void __launch_bounds__(SCAN_THREADS + FEED_THREADS)
 scan_kernel(const ScanArgs a) {
   constexpr int CH = SCAN_THREADS / P;                      // channels of the CTA
   constexpr int NP = P * NS;                                // states, padded
@@ -141,33 +246,35 @@ scan_kernel(const ScanArgs a) {
   const float* db = a.dt + (long)b * a.S * a.C;
   T* yb = reinterpret_cast<T*>(a.y) + (long)b * a.S * a.C;
 
-  auto prepare = [&](int tile) {
-    const int t0 = tile * TT;
-    float* bc = sBC + (tile & 1) * TT * 2 * NP;
-    float2* dd = sdt + (tile & 1) * TT * CH;
-    for (int i = tid; i < TT * CH; i += SCAN_THREADS) {
-      const int t = t0 + i / CH, c = c0 + i % CH;
-      float2 v = make_float2(0.f, 0.f);                     // padding neither decays nor writes
-      if (t < n_real && t < a.S && c < a.C) {
-        v.x = softplus_f(db[(long)t * a.C + c] + to_f(reinterpret_cast<const T*>(a.dt_bias)[c]));
-        v.y = v.x * to_f(xb[(long)t * a.C + c]);
-      }
-      dd[i] = v;
+  const int t_end = min(n_real, a.S);
+  // Round n (-1 .. tiles) brings tile n + 1 in and takes tile n - 1 out. Where registers allow it the loads of round n + 1 start at the end of
+  // round n and stay in flight across the barrier.
+  auto feed = [&](auto width) {
+    constexpr int W = decltype(width)::value;
+    using Probe = Feeder<T, CH, NP, TT, W, 1>;
+    constexpr bool AHEAD = W == 4 && Probe::PIECES <= 2;
+    Feeder<T, CH, NP, TT, W, AHEAD ? Probe::PIECES : (W == 4 ? 2 : 4)> f;
+    f.xb = xb; f.zb = zb; f.qb = qb; f.db = db; f.yb = yb; f.sBC = sBC; f.sy = sy; f.sdt = sdt; f.ldz = a.ldz; f.ldq = a.ldq;
+    f.C = a.C; f.N = a.N; f.tiles = tiles; f.t_end = t_end; f.tid = tid; f.ft = tid / f.CW;
+    f.c = c0 + (tid % f.CW) * W;
+    f.live = f.c < a.C;
+    if (f.live) {
+      load_vec<W>(reinterpret_cast<const T*>(a.dt_bias) + f.c, f.bias);
+      load_vec<W>(reinterpret_cast<const T*>(a.D) + f.c, f.skip);
     }
-    for (int i = tid; i < TT * 2 * NP; i += SCAN_THREADS) {
-      const int t = t0 + i / (2 * NP), j = i % (2 * NP), which = j / NP, n = j % NP;
-      bc[i] = (t < n_real && t < a.S && n < a.N) ? to_f(qb[(long)t * a.ldq + which * a.N + n]) : 0.f;
-    }
-  };
-  auto finish = [&](int tile) {
-    const int t0 = tile * TT;
-    const float* yy = sy + (tile & 1) * TT * CH;
-    for (int i = tid; i < TT * CH; i += SCAN_THREADS) {
-      const int t = t0 + i / CH, c = c0 + i % CH;
-      if (t < n_real && t < a.S && c < a.C) {
-        const float x = to_f(xb[(long)t * a.C + c]), z = to_f(zb[(long)t * a.ldz + c]);
-        yb[(long)t * a.C + c] = from_f<T>((yy[i] + to_f(reinterpret_cast<const T*>(a.D)[c]) * x) * silu_t<T>(z));
+    if constexpr (AHEAD) f.issue(0, 0, -2);
+    for (int n = -1; n <= tiles; ++n) {
+      if constexpr (AHEAD) {
+        f.settle(0, n + 1, n - 1);
+        f.issue(0, n + 2, n);
+      } else {
+#pragma unroll 1
+        for (int g = 0; g < f.PIECES; g += W == 4 ? 2 : 4) {
+          f.issue(g, n + 1, n - 1);
+          f.settle(g, n + 1, n - 1);
+        }
       }
+      if (n < tiles) tile_barrier();
     }
   };
 
@@ -182,65 +289,93 @@ scan_kernel(const ScanArgs a) {
       S[i] = (ok && cached) ? rec[i] : 0.f;
       A[i] = ok ? Decay<T>::arg(to_f(reinterpret_cast<const T*>(a.A_log)[(long)c * a.N + ln * NS + i])) : 0.f;
     }
-  } else if (tiles > 0) {
-    prepare(0);
   }
-  __syncthreads();
-  for (int tile = 0; tile < tiles; ++tile) {
-    if (consumer) {
+  // the two roles meet at the same barriers: one before the first tile and one after every tile
+  if (consumer) {
+    tile_barrier();
+    for (int tile = 0; tile < tiles; ++tile) {
       const float* bc = sBC + (tile & 1) * TT * 2 * NP + ln * NS;
       const float2* dd = sdt + (tile & 1) * TT * CH + lc;
       float* yy = sy + (tile & 1) * TT * CH + lc;
-      for (int t = 0; t < TT; t += 4) {
-        float r[4];
+      // Four steps at a time. Operands are read one group ahead and a group's read-outs are reduced while the next group computes, without
+      // a branch in the loop, so that loads, exchanges and exponentials of neighbouring groups overlap in one warp.
+      float2 d[4];
+      float Bv[4][NS], Cv[4][NS], r[4];
+      auto fetch = [&](int t) {
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
-          const float2 d = dd[(t + u) * CH];
-          float Bv[NS], Cv[NS];
-          load_vec<NS>(bc + (t + u) * 2 * NP, Bv);
-          load_vec<NS>(bc + (t + u) * 2 * NP + NP, Cv);
+          d[u] = dd[(t + u) * CH];
+          load_vec<NS>(bc + (t + u) * 2 * NP, Bv[u]);
+          load_vec<NS>(bc + (t + u) * 2 * NP + NP, Cv[u]);
+        }
+      };
+      auto steps = [&]() {
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
           float acc = 0.f;
 #pragma unroll
           for (int i = 0; i < NS; ++i) {
-            S[i] = Decay<T>::step(S[i], d.x, A[i], d.y * Bv[i]);
-            acc = fmaf(S[i], Cv[i], acc);
+            S[i] = Decay<T>::step(S[i], d[u].x, A[i], d[u].y * Bv[u][i]);
+            acc = fmaf(S[i], Cv[u][i], acc);
           }
           r[u] = acc;
         }
+      };
+      // sums of q[0..3] over the P lanes: lane bit 0 takes steps {0,1} or {2,3}, lane bit 1 one of the two, the remaining bits add up
+      const bool b0 = ln & 1, b1 = ln & 2;
+      float* mine = yy + (P == 1 ? 0 : (b0 ? 2 : 0) + (P > 2 && b1 ? 1 : 0)) * CH;
+      auto reduce = [&](const float (&q)[4], float (&o)[4]) {
         if constexpr (P == 1) {
 #pragma unroll
-          for (int u = 0; u < 4; ++u) yy[(t + u) * CH] = r[u];
-        } else if constexpr (P == 2) {
-          const bool odd = ln & 1;
-          const float s0 = odd ? r[0] : r[2], s1 = odd ? r[1] : r[3];
-          const float k0 = (odd ? r[2] : r[0]) + __shfl_xor_sync(0xffffffffu, s0, 1), k1 = (odd ? r[3] : r[1]) + __shfl_xor_sync(0xffffffffu, s1, 1);
-          yy[(t + (odd ? 2 : 0)) * CH] = k0;
-          yy[(t + (odd ? 3 : 1)) * CH] = k1;
+          for (int u = 0; u < 4; ++u) o[u] = q[u];
         } else {
-          // lane bit 0 picks steps {0,1} or {2,3}, lane bit 1 one of the two; the remaining bits add up
-          const bool o1 = ln & 1, o2 = ln & 2;
-          const float s0 = o1 ? r[0] : r[2], s1 = o1 ? r[1] : r[3];
-          const float k0 = (o1 ? r[2] : r[0]) + __shfl_xor_sync(0xffffffffu, s0, 1), k1 = (o1 ? r[3] : r[1]) + __shfl_xor_sync(0xffffffffu, s1, 1);
-          float v = (o2 ? k1 : k0) + __shfl_xor_sync(0xffffffffu, o2 ? k0 : k1, 2);
+          const float s0 = b0 ? q[0] : q[2], s1 = b0 ? q[1] : q[3];
+          o[0] = (b0 ? q[2] : q[0]) + __shfl_xor_sync(0xffffffffu, s0, 1);
+          o[1] = (b0 ? q[3] : q[1]) + __shfl_xor_sync(0xffffffffu, s1, 1);
+          if constexpr (P > 2) {
+            o[0] = (b1 ? o[1] : o[0]) + __shfl_xor_sync(0xffffffffu, b1 ? o[0] : o[1], 2);
 #pragma unroll
-          for (int o = 4; o < P; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-          if (ln < 4) yy[(t + (o1 ? 2 : 0) + (o2 ? 1 : 0)) * CH] = v;
+            for (int x = 4; x < P; x <<= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], x);
+          }
         }
+      };
+      auto put = [&](int t, const float (&o)[4]) {
+        if constexpr (P == 1) {
+#pragma unroll
+          for (int u = 0; u < 4; ++u) mine[(t + u) * CH] = o[u];
+        } else if constexpr (P == 2) {
+          mine[t * CH] = o[0];
+          mine[(t + 1) * CH] = o[1];
+        } else {
+          mine[t * CH] = o[0];                              // lanes above the fourth hold the same sum
+        }
+      };
+      fetch(0);
+      steps();
+      fetch(4);
+#pragma unroll 2
+      for (int t = 4; t < TT; t += 4) {
+        const float q[4] = {r[0], r[1], r[2], r[3]};
+        float o[4];
+        reduce(q, o);
+        steps();
+        fetch(min(t + 4, TT - 4));
+        put(t - 4, o);
       }
-    } else {
-      if (tile + 1 < tiles) prepare(tile + 1);
-      if (tile > 0) finish(tile - 1);
+      float o[4];
+      reduce(r, o);
+      put(TT - 4, o);
+      tile_barrier();
     }
-    __syncthreads();
-  }
-  if (consumer) {
 #pragma unroll
     for (int i = 0; i < NS; ++i)
       if (c < a.C && ln * NS + i < a.N) rec[i] = S[i];
   } else {
-    if (tiles > 0) finish(tiles - 1);
+    const bool wide = CH % 4 == 0 && a.C % 4 == 0 && a.N == NP && a.ldz % 4 == 0 && a.ldq % 8 == 0 && a.off % 8 == 0;
+    if (wide) feed(std::integral_constant<int, 4>{});
+    else feed(std::integral_constant<int, 1>{});
     // right padding: nothing reads it as a value, but later products multiply it by zero
-    for (int i = max(n_real, 0) * CH + tid; i < a.S * CH; i += SCAN_THREADS)
+    for (int i = max(n_real, 0) * CH + tid; i < a.S * CH; i += FEED_THREADS)
       if (c0 + i % CH < a.C) yb[(long)(i / CH) * a.C + c0 + i % CH] = from_f<T>(0.f);
   }
 }
@@ -322,7 +457,7 @@ int run(const ScanArgs& a, int B, cudaStream_t st) {
   constexpr int smem = (2 * TT * 2 * NP + 2 * TT * CH * 2 + 2 * TT * CH) * 4;
   auto k = scan_kernel<T, P, NS>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
-  k<<<dim3((a.C + CH - 1) / CH, B), 2 * SCAN_THREADS, smem, st>>>(a);
+  k<<<dim3((a.C + CH - 1) / CH, B), SCAN_THREADS + FEED_THREADS, smem, st>>>(a);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -332,8 +467,8 @@ int run_t(const ScanArgs& a, int B, cudaStream_t st) {
   if (a.N <= 8) return run<T, 2, 4>(a, B, st);
   if (a.N <= 16) return run<T, 4, 4>(a, B, st);
   if (a.N <= 32) return run<T, 8, 4>(a, B, st);
-  if (a.N <= 64) return run<T, 8, 8>(a, B, st);
-  if (a.N <= 128) return run<T, 16, 8>(a, B, st);
+  if (a.N <= 64) return run<T, 16, 4>(a, B, st);
+  if (a.N <= 128) return run<T, 32, 4>(a, B, st);
   if (a.N <= 256) return run<T, 32, 8>(a, B, st);
   return -1;
 }
