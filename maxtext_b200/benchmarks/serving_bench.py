@@ -292,10 +292,7 @@ def rooflines(iters: int = 10) -> dict:
   lc, kc, qd = t(B, L, R), t(B, L, dr), t(B, H, R + dr)
   sp = E.mla_decode_splits(B, H, L)
   part, ml = t(B, H, sp, R, dtype=torch.float32), torch.rand(B, H, sp, 2, device=dev) + 0.1
-  add("mla_decode_attn", lambda: E.mla_decode_attn(qd, lc, kc, ids, lens, 0.1, 2048, sp, part, ml), 2 * B * L * (R + dr), like="decode_attention")
-  kc8, vc8, q8, o8 = t(B, L, 8, 128), t(B, L, 8, 128), t(B, 16, 128), t(B, 16, 128)
-  i32, l32 = ids.int(), (lens + 1).int()
-  add("decode_attention", lambda: E.decode_attention(q8, kc8, vc8, i32, l32, o8, 1.0, 0.0, 0, 1), 2 * 2 * B * L * 8 * 128)
+  add("mla_decode_attn", lambda: E.mla_decode_attn(qd, lc, kc, ids, lens, 0.1, 2048, sp, part, ml), 2 * B * L * (R + dr), like="cached_decode, 128 sequences")
   wb, qin, vout = t(H * (nope + vd), R), t(B, H, nope + dr), t(B, H, vd)
   add("mla_absorb", lambda: E.mla_absorb(qin, wb, pos[:B], inv, True, nope, vd, qd), 2 * (H * nope * R + B * H * (nope + 2 * dr + R)), like="gemm, M = 128")
   add("mla_value_up", lambda: E.mla_value_up(part, ml, wb, nope, vout), 2 * H * vd * R + 4 * B * H * R + 2 * B * H * vd, like="gemm, M = 128")
@@ -317,7 +314,7 @@ def rooflines(iters: int = 10) -> dict:
           like=f"experts, silu (whole layer), {Bd} tokens")
       add(f"experts, silu (whole layer), {Bd} tokens", lambda: moe_ops.moe_ffn_padded(xd, wts, idx, lay.wi_0, lay.wi_1, lay.wo, nE, "silu"), 2 * hit * 3 * Fe * D)
   brec, bhist = t(B, 1, C, NS, dtype=torch.float32), t(B, 3, C, dtype=torch.float32)
-  add("ssm_conv, 128 tokens", lambda: E.ssm_conv(px[:B], cw4, cb, 1, bhist, ids, lens, None, sx[:B]), B * C * (4 + 8 * 3), like="delta_decode")
+  add("ssm_conv, 128 tokens", lambda: E.ssm_conv(px[:B], cw4, cb, 1, bhist, ids, lens, None, sx[:B]), B * C * (4 + 8 * 3), like="rmsnorm, 128 tokens")
   add("ssm_scan, 128 tokens", lambda: E.ssm_scan(sx[:B], px[:B], q2[:B], sdt[:B], cb, A16, D16, rk, NS, 1, brec, ids, lens, None, sy[:B]),
       B * C * (8 * NS + 10) + 2 * C * NS, like="gla_decode")
   kc4, vc4, q16, g16 = t(B, L, HG, hd), t(B, L, HG, hd), t(B, HQ, hd), t(B, HQ * hd)
@@ -326,11 +323,7 @@ def rooflines(iters: int = 10) -> dict:
     sp = E.cached_decode_splits(Bd, HQ, HG, L)
     pt, ml2, od = t(Bd, HQ, sp, hd, dtype=torch.float32), t(Bd, HQ, sp, 2, dtype=torch.float32), t(Bd, HQ * hd)
     add(f"cached_decode, {Bd} sequences", lambda: E.cached_decode(q16[:Bd], kc4[:Bd], vc4[:Bd], ids[:Bd], lens[:Bd], 0.09, 40.0, 0, sinkb, g16[:Bd], sp, pt, ml2, od),
-        2 * 2 * Bd * L * HG * hd, like=f"decode_attention, {Bd} sequences")
-    o16 = t(Bd, HQ, hd)
-    sp1 = max(1, min(16, 296 // (Bd * HG)))
-    add(f"decode_attention, {Bd} sequences", lambda: E.decode_attention(q16[:Bd], kc4[:Bd], vc4[:Bd], i32[:Bd], l32[:Bd], o16, 1.0, 0.0, 0, sp1),
-        2 * 2 * Bd * L * HG * hd)
+        2 * 2 * Bd * L * HG * hd, like="mla_decode_attn")
   add("stream_mix, 128 tokens", lambda: E.stream_mix(xs[:B], b[:B], None, 1, mix, wr, wr, w, w, y[:B], 1e-5), B * D * (2 * 2 * 4 + 4), like="rmsnorm, 128 tokens")
   add("rmsnorm, 128 tokens", lambda: E.rmsnorm_fwd(b[:B], w, 1e-6, 0.0, y[:B], None), 4 * B * D)
   return {"rooflines": rows, "hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "peaks": peaks["source"]}

@@ -3,7 +3,8 @@
 `serve` is the whole attention part of a layer whose q and k are rotated and then RMS-normalised per head: one kernel rotates, normalises,
 fills the cache and lays the operands out for what follows; prompts run the flash kernel (head widths padded to the next variant), one new
 token per sequence runs the split decode kernel, and everything else (fp32, unusual widths) a plain kernel that reads the cache. Sinks,
-soft caps, windows and a sigmoid output gate are parameters. `decode` and `prompt` also serve `inference.kvcache.LayerKVCache.attend`.
+soft caps, windows and a sigmoid output gate are parameters. `attend` is the same for layers that prepare q, k and v themselves
+(`inference.kvcache.LayerKVCache.attend`).
 """
 from __future__ import annotations
 
@@ -33,6 +34,36 @@ def flash_widths(qk: int, vd: int):
     if qk <= dq and vd <= dv:
       return dq, dv
   return None
+
+
+def attends(q, cache, ctx) -> bool:
+  """Can `attend` take q [B, S, H, D] over this cache? (bf16 caches that are neither quantised nor split, no image blocks)"""
+  B, S, H, D = q.shape
+  return (q.dtype == torch.bfloat16 and kernels_ok(q) and cache.quant is None and cache.k.dtype == q.dtype and H % cache.k.shape[2] == 0
+          and getattr(ctx, "bidir", None) is None and max(D, cache.v.shape[3]) <= 512 and (S == 1 or ctx.segment_ids is None or ctx.mode == "prefill")
+          and (S == 1 or ctx.segment_ids is None or flash_widths(D, cache.v.shape[3]) is not None))
+
+
+def attend(q, k, v, cache, ctx, window, soft_cap, sinks):
+  """q [B, S, H, D] (scaled) and the S new tokens' k, v, which the cache holds by now -> [B, S, H, Dv]."""
+  B, S, H, D = q.shape
+  Dv = v.shape[3]
+  cap, win, sk = float(soft_cap or 0.0), int(window or 0), sinks.data if sinks is not None else None
+  widths = flash_widths(D, Dv)
+  if S == 1:
+    out = decode(q[:, 0].contiguous(), cache, 1.0, cap, win, sk)
+  elif widths is None:
+    out = plain(q.reshape(B * S, H, D).contiguous(), cache, S, 1.0, cap, win, sk)
+  else:
+    def wide(t, n):
+      return t if t.shape[3] == n else torch.nn.functional.pad(t, (0, n - t.shape[3]))
+    q = wide(q, widths[0]).contiguous()
+    if ctx.mode == "prefill":
+      out = _flash(q, wide(k, widths[0]).contiguous(), wide(v, widths[1]).contiguous(), ctx.positions, ctx.segment_ids, 1.0, cap, win, sk, F.CAP_EXACT)
+    else:
+      out = _portion(q, cache, ctx, 1.0, cap, win, sk, F.CAP_EXACT, D, Dv)
+    out = out[..., :Dv]
+  return out.reshape(B, S, H, Dv)
 
 
 def _gate(o, g, H, dv):

@@ -126,14 +126,15 @@ def test_decode_attention_matches_reference(B, Hq, Hkv, D, window):
   kc = (torch.randn(slots, max_len, Hkv, D, device="cuda") * 0.5).bfloat16()
   vc = (torch.randn(slots, max_len, Hkv, D, device="cuda") * 0.5).bfloat16()
   q = (torch.randn(B, Hq, D, device="cuda") * 0.3).bfloat16()
-  slot_ids = torch.randperm(slots, device="cuda")[:B].to(torch.int32)
-  lengths = torch.tensor([1, 64, 333, 700][:B] if B <= 4 else None, device="cuda", dtype=torch.int32)
+  slot_ids = torch.randperm(slots, device="cuda")[:B]
+  lengths = torch.tensor([1, 64, 333, 700][:B], device="cuda")
   out = torch.empty(B, Hq, D, device="cuda", dtype=torch.bfloat16)
   for splits in (1, 5):
-    E.decode_attention(q, kc, vc, slot_ids, lengths, out, 1.0, 0.0, window, splits)
+    part, ml = torch.empty(B, Hq, splits, D, device="cuda"), torch.empty(B, Hq, splits, 2, device="cuda")
+    E.cached_decode(q, kc, vc, slot_ids, lengths - 1, 1.0, 0.0, window, None, None, splits, part, ml, out.view(B, -1))
     for b in range(B):
       n = int(lengths[b])
-      K, V = kc[slot_ids[b].long(), :n][None], vc[slot_ids[b].long(), :n][None]
+      K, V = kc[slot_ids[b], :n][None], vc[slot_ids[b], :n][None]
       qpos = torch.tensor([[n - 1]], device="cuda")
       kpos = torch.arange(n, device="cuda")[None]
       m = ref.attention_mask(qpos, kpos, None, None, True, window)

@@ -335,3 +335,40 @@ def test_every_row_of_an_expert_is_computed():
     w0, w1, wo = (p.data.double().cpu() for p in (layer.wi_0, layer.wi_1, layer.wo))
     want = sum(O.clamped_expert(float(torch.sigmoid(torch.tensor(v, dtype=torch.float64))) * x.double(), w0[e], w1[e], wo[e], 1.0) for e, v in ((3, 2.0), (5, 1.0)))
     assert _rows(got, want) < 2.5e-2
+
+
+# ------------------------------------------------------------------------------------------ the same kernels behind the other families' caches
+@pytest.mark.parametrize("D, Dv, H, G, window, cap, sinks", [(64, 64, 4, 2, 0, 0.0, False), (128, 128, 8, 1, 9, 4.0, True), (32, 32, 4, 4, 0, 0.0, True),
+                                                             (48, 80, 6, 2, 5, 3.0, False), (208, 144, 2, 1, 0, 2.0, True)])
+def test_layer_cache_attends_on_the_kernels(D, Dv, H, G, window, cap, sinks):
+  """Prompts, portions, single tokens and packed prompts through LayerKVCache.attend against the definition on fp32 copies."""
+  from maxtext_b200.inference.kvcache import LayerKVCache
+  from maxtext_b200.ops import cached_attention as CA, reference as ref
+  g = torch.Generator().manual_seed(D)
+  B, total, bf = 2, 40, torch.bfloat16
+  q, k, v = (torch.randn(B, total, n, w, generator=g).to(bf).cuda() for n, w in ((H, D), (G, D), (G, Dv)))
+  q = (q * (2.0 / D ** 0.5)).to(bf)
+  sk = torch.randn(H, generator=g).to(bf).cuda() if sinks else None
+  param = type("P", (), {"data": sk})() if sinks else None
+  pos = torch.arange(total, device="cuda")[None].expand(B, -1)
+  want = ref.attention(q.float(), k.float(), v.float(), ref.attention_mask(pos, pos, None, None, True, window), 1.0, cap, sinks=sk)
+  slots = torch.tensor([2, 0], device="cuda")
+
+  def ctx(mode, lo, hi, seg=None):
+    return type("C", (), {"mode": mode, "positions": pos[:, lo:hi].contiguous(), "segment_ids": seg, "bidir": None})()
+  with torch.no_grad():
+    for cuts in ([0, total], [0, 17, 19, 39, 40], [0, 1, 2, 3, total]):
+      cache = LayerKVCache(3, 64, G, D, Dv, bf, "cuda")
+      outs = []
+      for lo, hi in zip(cuts, cuts[1:]):
+        cache.bind(slots, torch.full((B,), lo, dtype=torch.long, device="cuda"))
+        c = ctx("prefill" if lo == 0 else "decode", lo, hi)
+        assert CA.attends(q[:, lo:hi], cache, c)
+        outs.append(cache.attend(q[:, lo:hi], k[:, lo:hi], v[:, lo:hi], c, window, cap, param))
+      assert _rows(torch.cat(outs, 1), want) < 2e-2, cuts
+    if CA.flash_widths(D, Dv) is not None:
+      seg = torch.cat([torch.full((B, 15), 1), torch.full((B, 25), 2)], 1).int().cuda()
+      want2 = ref.attention(q.float(), k.float(), v.float(), ref.attention_mask(pos, pos, seg, seg, True, window), 1.0, cap, sinks=sk)
+      cache = LayerKVCache(3, 64, G, D, Dv, bf, "cuda")
+      cache.bind(slots, torch.zeros(B, dtype=torch.long, device="cuda"))
+      assert _rows(cache.attend(q, k, v, ctx("prefill", 0, total, seg), window, cap, param), want2) < 2e-2
