@@ -163,10 +163,12 @@ void qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, int64_t D, int6
                    longs(lengths, B, "lengths"), longs(new_lens, B, "new_lens"), N, stream()), "qkv_prep");
 }
 
-// parts of the key range that fill the machine twice over without making a part shorter than four tiles
+// parts of the key range that fill the machine twice over without making a part shorter than four tiles; long ranges are cut up to four times
+// anyway, so that the last wave of CTAs is short
 int64_t cached_decode_splits(int64_t B, int64_t H, int64_t G, int64_t span) {
   const int64_t ctas = std::max<int64_t>(1, B * G * ((H / G + 15) / 16));
-  return std::max<int64_t>(1, std::min<int64_t>({64, 2 * mt_num_sms() / ctas, (span + 63) / 64}));
+  const int64_t fill = 2 * mt_num_sms() / ctas, even = std::min<int64_t>(4, span / 1024);
+  return std::max<int64_t>(1, std::min<int64_t>({64, std::max(fill, even), (span + 63) / 64}));
 }
 
 void cached_decode(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& slots, const Tensor& lengths, double scale, double cap, int64_t window,

@@ -136,19 +136,29 @@ decode_kernel(const DecodeArgs a) {
   }
   __syncthreads();
   const int n_tiles = hi > lo ? (hi - lo + KEYS - 1) / KEYS : 0;
+  // a lane keeps its 16-byte column of a row and walks down the keys; columns beyond the width are filled with zeros once per tile
+  constexpr int KP = DK / 8, VP = DVT / 8, KR = 32 / KP, VR = 32 / VP;
+  const int kr = lane / KP, kcol = (lane % KP) * 8, vr = lane / VP, vcol = (lane % VP) * 8;
+  const bool kin = kcol < a.D, vin = vcol < a.Dv, kpad = kcol < D16 * 16, vpad = vcol < V16 * 16;
+  const __nv_bfloat16 *kp = kb + (kin ? (lo + kr) * ldk + kcol : 0), *vp = vb + (vin ? (lo + vr) * ldv + vcol : 0);
   auto load = [&](int tile, int stage) {
-    __nv_bfloat16* sk = ring + stage * TILE;
-    __nv_bfloat16* sv = sk + KEYS * LK;
-    const int t0 = lo + tile * KEYS;
-    for (int i = lane; i < KEYS * D16 * 2; i += 32) {
-      const int r = i / (D16 * 2), c = (i % (D16 * 2)) * 8;
-      const bool ok = t0 + r < hi && c < a.D;
-      la_cp_async16(sk + r * LK + c, ok ? kb + (long)(t0 + r) * ldk + c : kb, ok ? 16 : 0);
+    __nv_bfloat16* sk = ring + stage * TILE + kr * LK + kcol;
+    __nv_bfloat16* sv = ring + stage * TILE + KEYS * LK + vr * LV + vcol;
+    const int left = hi - lo - tile * KEYS;
+    const __nv_bfloat16 *kt = kp + (kin ? (long)tile * KEYS * ldk : 0), *vt = vp + (vin ? (long)tile * KEYS * ldv : 0);
+    if (kpad) {
+#pragma unroll
+      for (int j = 0; j < KEYS / KR; ++j) {
+        const bool ok = kin && kr + j * KR < left;
+        la_cp_async16(sk + j * KR * LK, ok ? kt + j * KR * ldk : kb, ok ? 16 : 0);
+      }
     }
-    for (int i = lane; i < KEYS * V16 * 2; i += 32) {
-      const int r = i / (V16 * 2), c = (i % (V16 * 2)) * 8;
-      const bool ok = t0 + r < hi && c < a.Dv;
-      la_cp_async16(sv + r * LV + c, ok ? vb + (long)(t0 + r) * ldv + c : vb, ok ? 16 : 0);
+    if (vpad) {
+#pragma unroll
+      for (int j = 0; j < KEYS / VR; ++j) {
+        const bool ok = vin && vr + j * VR < left;
+        la_cp_async16(sv + j * VR * LV, ok ? vt + j * VR * ldv : vb, ok ? 16 : 0);
+      }
     }
   };
   float o[DVT / 8][4];

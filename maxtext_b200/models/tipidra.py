@@ -41,7 +41,7 @@ def validate(t: dict) -> None:
       raise ValueError(why)
   need(len(t["layer_specs"]) == int(t["base_num_decoder_layers"]),
        f"layer_specs names {len(t['layer_specs'])} layers, base_num_decoder_layers is {t['base_num_decoder_layers']}")
-  need(int(t["mhc_expansion_rate"]) >= 1, "mhc_expansion_rate: there is at least one residual stream")
+  need(1 <= int(t["mhc_expansion_rate"]) <= 16, "mhc_expansion_rate: between 1 and 16 residual streams are supported")
   for i, lay in enumerate(t["layer_specs"]):
     m, kind, mlp = lay["mixer"], lay["type"], lay["mlp"]
     need(kind in MIXERS, f"layer_specs[{i}]: unknown mixer type {kind!r}")
@@ -51,11 +51,12 @@ def validate(t: dict) -> None:
       need(m["softcap"] > 0, f"layer_specs[{i}]: softcap must be positive")
       need(max(m["dim"], m["vdim"]) <= 512, f"layer_specs[{i}]: head widths above 512 are not supported")
     else:
-      need(m["conv"] >= 1, f"layer_specs[{i}]: the convolution needs at least one tap")
-      need(m["state"] >= 1 and m["dt_rank"] >= 1, f"layer_specs[{i}]: state and dt_rank must be positive")
+      need(1 <= m["conv"] <= 17, f"layer_specs[{i}]: the convolution needs between one tap and 17")
+      need(1 <= m["state"] <= 256 and m["dt_rank"] >= 1, f"layer_specs[{i}]: state (up to 256) and dt_rank must be positive")
     if mlp is not None and mlp["kind"] == "moe":
       r = mlp["router"]
       need(1 <= r["top"] <= r["experts"], f"layer_specs[{i}]: router.top must lie between 1 and router.experts")
+      need(r["experts"] <= 512 and r["top"] <= 32, f"layer_specs[{i}]: at most 512 experts and 32 of them per token are supported")
       need(mlp["expert"]["limit"] > 0, f"layer_specs[{i}]: expert.limit must be positive")
 
 

@@ -372,3 +372,20 @@ def test_layer_cache_attends_on_the_kernels(D, Dv, H, G, window, cap, sinks):
       cache = LayerKVCache(3, 64, G, D, Dv, bf, "cuda")
       cache.bind(slots, torch.zeros(B, dtype=torch.long, device="cuda"))
       assert _rows(cache.attend(q, k, v, ctx("prefill", 0, total, seg), window, cap, param), want2) < 2e-2
+
+
+def test_training_step_in_bf16(tmp_path):
+  """The layers train through their differentiable forms, with the fp32 streams crossing units."""
+  from helpers import BASE_YML
+  from maxtext_b200.config import pyconfig
+  from maxtext_b200.input_pipeline.synthetic import SyntheticDataIterator
+  from maxtext_b200.train.engine import TrainEngine
+  sp = M.spec([(M.scan(128, 8, 16, 3), M.dense(128)), (M.attention(4, 2, 64, 64, 32, 0.1, 9.0), M.moe(4, 2, 64, 2.0))], 128, streams=3, vocab=512)
+  path = M.write_folder(tmp_path / "m", sp, M.weights(sp))
+  cfg = pyconfig.initialize(["t", BASE_YML, f"model_dir={path}"], num_devices=1, dtype="bfloat16", max_target_length=64, per_device_batch_size=2,
+                            dataset_type="synthetic", hardware="gpu", enable_checkpointing=False, log_config=False, steps=5, learning_rate=2e-3,
+                            warmup_steps_fraction=0.0)
+  eng = TrainEngine(cfg, None, torch.device("cuda", 0))
+  batch = next(SyntheticDataIterator(cfg))
+  losses = [float(eng.train_step(batch)["learning/loss"]) for _ in range(5)]
+  assert losses[-1] < losses[0] and all(x == x for x in losses), losses
