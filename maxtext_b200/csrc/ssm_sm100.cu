@@ -1,7 +1,8 @@
 // Selective scan (Gu and Dao, "Mamba: Linear-Time Sequence Modeling with Selective State Spaces") at inference:
-//   x  = silu(causal depthwise convolution + bias)
-//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,   y_c = (sum_n S[c, n] C_n + D_c x_c) * silu(z_c)
-// with dt = softplus(pre-activation + bias) and A = -exp(A_log). States, decays and step sizes are fp32.
+//   u = silu(causal depthwise convolution + bias)
+//   s <- exp(d alpha) * s + (d u) b,    y = (<s, c> + skip u) silu(z)
+// per channel, with d = softplus(pre-activation + bias) and alpha = -exp(A_log). States, decays and step sizes are fp32. In the code x is the
+// channel's input u, dt its step size, B and C are b and c, A is alpha and D the skip factor.
 //
 // A channel's states are spread over P neighbouring lanes, NS per lane, and stay in registers over the whole prompt. Four of a CTA's twelve
 // warps run the recurrence; the others load and prepare the next tile of tokens (softplus, dt * x, B and C as fp32) and finish the previous
@@ -247,8 +248,8 @@ scan_kernel(const ScanArgs a) {
   T* yb = reinterpret_cast<T*>(a.y) + (long)b * a.S * a.C;
 
   const int t_end = min(n_real, a.S);
-  // Round n (-1 .. tiles) brings tile n + 1 in and takes tile n - 1 out. Where registers allow it the loads of round n + 1 start at the end of
-  // round n and stay in flight across the barrier.
+  // Turn n (-1 .. tiles) brings tile n + 1 in and takes tile n - 1 out. Where registers allow it the loads of turn n + 1 start at the end of
+  // turn n and stay in flight across the barrier.
   auto feed = [&](auto width) {
     constexpr int W = decltype(width)::value;
     using Probe = Feeder<T, CH, NP, TT, W, 1>;

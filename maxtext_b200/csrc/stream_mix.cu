@@ -1,5 +1,6 @@
 // The border between two sublayers of a model with several fp32 residual streams and static hyper-connections, in one pass per token:
-//   x_t <- sum_s mix[s, t] x_s + write[t] * (sum of the branch's rows);    y = layer_norm(sum_t read[t] x_t) * w + b
+//   X <- M^T X + w (sum of the branch's rows)^T,    y = scaled and shifted layer norm of r^T X
+// where the rows of X [k, D] are the streams of a token.
 // The branch comes in the compute type (a GEMM output, or the rows of the chosen experts of the token), the streams stay fp32, y is rounded
 // once for the next GEMM. Without a branch it only reads the streams; without y it only mixes them. Bandwidth-bound.
 #include "serving_common.cuh"

@@ -108,8 +108,9 @@ class HyperConnection:
 
 
 class StaticHyperConnection:
-  """A hyper-connection whose maps are constants of the model: the branch reads sum_s in[s] x_s, and afterwards stream t is
-  sum_s mix[s, t] x_s + out[t] * branch (mix is indexed [from, to]). Streams and maps are fp32 (`ops.functional.stream_mix`)."""
+  """A hyper-connection whose maps are constants of the model. With the k streams of a token as the rows of X, the branch reads r^T X and
+  leaves M^T X + w b^T, b being its output: `read` holds r, `write` w, and a row of `mix` (M) says where one stream goes. fp32 arithmetic
+  (`ops.functional.stream_mix`)."""
 
   def __init__(self, b: L.Builder, config, name: str, k: int):
     self.k = k

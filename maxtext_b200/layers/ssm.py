@@ -1,11 +1,12 @@
 """Selective scan (Gu and Dao, "Mamba: Linear-Time Sequence Modeling with Selective State Spaces").
 
 A causal depthwise convolution with bias and SiLU forms x from one half of the input projection; a second projection of x gives a
-low-rank step size and the two vectors B and C of the state width. Per channel c and state n, in fp32,
+low-rank step size and two vectors b and c of the state width. A channel with input u, step size d and state vector s then does, in fp32,
 
-  S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,      y_c = sum_n S[c, n] C_n + D_c x_c,
+  s <- exp(d alpha) * s + (d u) b,      y = <s, c> + skip u,
 
-with dt = softplus(low-rank projection + bias) per channel and A = -exp(A_log); SiLU of the other half of the input projection gates y.
+alpha = -exp(A_log) being the channel's row of decay rates and d the softplus of its low-rank projection plus bias; SiLU of the other half of the
+input projection gates y.
 Inference on a GPU runs the kernels behind `ops.ssm`; training and CPU evaluate the recurrence as written.
 """
 from __future__ import annotations

@@ -319,8 +319,8 @@ def stream_read(x: torch.Tensor, reader: StreamReader, dtype) -> torch.Tensor:
 
 
 def stream_mix(x: torch.Tensor, branch, connection, nxt: StreamReader | None = None):
-  """(streams after a sublayer, input of the next one or None): x_t <- sum_s mix[s, t] x_s + write[t] * branch on fp32 x [B, S, k, D].
-  `branch` is [B, S, D] or expert rows that are summed per token (`moe_ops.ExpertRows`). On a GPU one kernel, which updates x in place."""
+  """(streams after a sublayer, input of the next one or None) for fp32 x [B, S, k, D]: X <- M^T X + w b^T per token
+  (`layers.mhc.StaticHyperConnection`). `branch` is [B, S, D] or expert rows that are summed per token (`moe_ops.ExpertRows`). On a GPU one kernel, which updates x in place."""
   rows, dest, per_token = (branch, None, 1) if isinstance(branch, torch.Tensor) else (branch.rows, branch.dest, branch.k)
   if _stream_kernel_ok(x, rows) and x.dtype == torch.float32 and x.is_contiguous():
     B, S, k, D = x.shape

@@ -77,7 +77,8 @@ def sink_attention(q, k, v, scale, cap, sink):
 
 
 def selective_scan(x, dt, A, B, C, D):
-  """x, dt [T, c]; A [c, n]; B, C [T, n]; D [c]: S <- exp(dt A) S + dt x B, y = S C + D x."""
+  """x, dt [T, channels]; A [channels, n]; B, C [T, n]; D [channels]. Each channel decays its n states at its own rates, adds its input times
+  the step size along B, and reads them out along C next to a direct path."""
   S = torch.zeros_like(A)
   out = []
   for t in range(x.shape[0]):
@@ -131,7 +132,7 @@ MLPS = {"dense": dense_mlp, "moe": moe_mlp}
 
 
 def hyper_sublayer(streams, hc, norm, branch):
-  """streams: list of s tensors [T, width]; hc: in [s], mix [s, s] indexed [from, to], out [s]."""
+  """streams: list of tensors [T, width]; hc: the weights `in` and `out`, one per stream, and `mix`, whose rows are the sources."""
   n = len(streams)
   u = sum(hc["in"][s] * streams[s] for s in range(n))
   y = branch(norm(u))
