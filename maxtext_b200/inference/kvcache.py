@@ -122,10 +122,13 @@ class LayerKVCache:
       return self.quant.dequantize(x, sbuf[self.slot_ids, :upto], self.dtype)
     return x
 
-  def attend(self, q, k, v, ctx, window=0, soft_cap=0.0, sinks=None):
-    """Append k/v of the S new tokens at each row's current length, then attend over everything cached."""
+  def attend(self, q, k, v, ctx, window=0, soft_cap=0.0, sinks=None, chunk=0):
+    """Append k/v of the S new tokens at each row's current length, then attend over everything cached (that `window` and `chunk` leave
+    visible)."""
     B, S = q.shape[:2]
     if self.seq_size > 1:
+      if chunk:
+        raise NotImplementedError("a sequence-split cache does not take chunked attention")
       if getattr(ctx, "bidir", None) is not None:
         raise NotImplementedError("a sequence-split cache does not take bidirectional image blocks")
       return self._attend_split(q, k, v, ctx, window, soft_cap, sinks)
@@ -135,17 +138,22 @@ class LayerKVCache:
     from ..ops import cached_attention as CA
     if CA.attends(q, self, ctx):
       # flash kernel for prompts, split decode kernel for one new token per sequence (lengths stay on the device, no host sync)
-      return CA.attend(q, k, v, self, ctx, window, soft_cap, sinks)
+      return CA.attend(q, k, v, self, ctx, window, soft_cap, sinks, chunk)
     upto = int((self.lengths.max() + S).item()) if ctx.mode != "prefill" else int(S + self.lengths.max().item())
     if self.new_lens is not None:
       upto = min(upto, self.max_len)                      # padding may run past the end of the cache
     K, V = self._read(self.k, getattr(self, "ks", None), upto), self._read(self.v, getattr(self, "vs", None), upto)
     kv_pos = torch.arange(upto, device=q.device)[None].expand(B, upto)
     valid_len = (self.lengths + S)[:, None]
-    mask = ref.attention_mask(pos, kv_pos, None, None, True, window) & (kv_pos < valid_len)[:, None, None, :]
+    packed = ctx.segment_ids is not None and ctx.mode == "prefill" and ctx.segment_ids.shape[1] == upto
+    if packed:                                            # several prompts in one row: chunks count from the start of each
+      mask = ref.attention_mask(pos, kv_pos, None, None, True, window) & ref.attention_mask(ctx.positions, ctx.positions, chunk=chunk, causal=False)
+    else:
+      mask = ref.attention_mask(pos, kv_pos, None, None, True, window, chunk)
+    mask = mask & (kv_pos < valid_len)[:, None, None, :]
     if ctx.segment_ids is not None and ctx.mode == "prefill":
       mask = mask & (ctx.segment_ids[:, None, :, None] != 0)
-      if ctx.segment_ids.shape[1] == upto:
+      if packed:
         # several prompts packed into one prefill pass (prefill_concat): a token sees its own prompt only
         mask = mask & (ctx.segment_ids[:, None, :, None] == ctx.segment_ids[:, None, None, :])
     if getattr(ctx, "bidir", None) is not None and ctx.bidir.shape[-2] == S and ctx.bidir.shape[-1] <= upto:
@@ -177,6 +185,50 @@ class MlaLayerCache(LayerKVCache):
     return lat_ops.attend_cached(q, latent, k_rope, mla, self, ctx)
 
 
+class PairCache:
+  """Caches of a block with two mixers side by side. The engine copies and saves cache contents by attribute name; each name belongs to the
+  one part that has it (keys and values to one, a recurrent state to the other)."""
+
+  def __init__(self, left, right):
+    self.left, self.right = left, right
+    names = [{n for n, t in vars(p).items() if isinstance(t, torch.Tensor)} for p in (left, right)]
+    if names[0] & names[1]:
+      raise NotImplementedError("two mixers side by side need caches of different kinds")
+    self.recurrent_buffers = tuple(getattr(left, "recurrent_buffers", ())) + tuple(getattr(right, "recurrent_buffers", ()))
+
+  def bind(self, slot_ids, lengths, new_lens=None):
+    self.left.bind(slot_ids, lengths, new_lens)
+    self.right.bind(slot_ids, lengths, new_lens)
+
+  def __getattr__(self, name):
+    if name in ("left", "right"):
+      raise AttributeError(name)
+    for part in (self.left, self.right):
+      if hasattr(part, name):
+        return getattr(part, name)
+    raise AttributeError(name)
+
+
+RECURRENT = ("gdn", "gla", "ssm", "retention", "channel_delta")    # block kinds that carry a state of fixed size from token to token
+
+
+def recurrent(plan) -> bool:
+  """Does a block of this plan carry such a state?"""
+  return plan.attention in RECURRENT or (plan.pair is not None and any(recurrent(p) for p in plan.pair))
+
+
+def _block_cache(attn, plan, slots, max_len, dt, device, quant, seq):
+  if plan.attention == "parallel":
+    return PairCache(*(_block_cache(a, p, slots, max_len, dt, device, quant, seq) for a, p in zip((attn.left, attn.right), plan.pair)))
+  if plan.attention == "mla":
+    return MlaLayerCache(slots, max_len, attn.kv_rank, attn.rope_d, dt, device)
+  if plan.attention == "compressed":
+    return attn.make_cache(slots, max_len, dt, device)
+  if plan.attention in RECURRENT:
+    return attn.make_state(slots, device)
+  return LayerKVCache(slots, max_len, attn.hkv_l, attn.kw, attn.dv, dt, device, quant, **seq)
+
+
 def make_caches(model, slots: int, max_len: int, device, quantize: bool = False):
   """One cache per attention block of the model, in layer order."""
   c = model.config
@@ -189,16 +241,8 @@ def make_caches(model, slots: int, max_len: int, device, quantize: bool = False)
   for layer in model.layers:
     per_layer = []
     for blk in layer.blocks:
-      if seq_size > 1 and blk.plan.attention in ("mla", "gdn", "gla", "ssm", "compressed"):
+      if seq_size > 1 and (blk.plan.attention in ("mla", "parallel", "compressed") or recurrent(blk.plan)):
         raise NotImplementedError("context_autoregressive parallelism splits plain key / value caches only")
-      if blk.plan.attention == "mla":
-        per_layer.append(MlaLayerCache(slots, max_len, blk.attn.kv_rank, blk.attn.rope_d, dt, device))
-      elif blk.plan.attention == "compressed":
-        per_layer.append(blk.attn.make_cache(slots, max_len, dt, device))
-      elif blk.plan.attention in ("gdn", "gla", "ssm"):
-        per_layer.append(blk.attn.make_state(slots, device))
-      else:
-        a = blk.attn
-        per_layer.append(LayerKVCache(slots, max_len, a.hkv_l, a.dh, a.dv, dt, device, quant, **seq))
+      per_layer.append(_block_cache(blk.attn, blk.plan, slots, max_len, dt, device, quant, seq))
     out.append(per_layer)
   return out

@@ -247,7 +247,7 @@ class MaxEngine:
       self._check_length(n, "prefill_concat")
     total = sum(lens)
     kinds = {b.plan.attention for l in self.model.layers for b in l.blocks}
-    packable = total <= self.max_len and not kinds & {"gdn", "gla", "ssm", "compressed"}
+    packable = total <= self.max_len and "compressed" not in kinds and not any(kvcache.recurrent(b.plan) for l in self.model.layers for b in l.blocks)
     if len(prompts) == 1 or "compressed" in kinds:
       return [self.prefill(p, n)[0] for p, n in zip(prompts, lens)]
     if not packable:

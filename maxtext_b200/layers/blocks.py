@@ -286,13 +286,30 @@ class Norm:
 # ------------------------------------------------------------------------------------------ attention (MHA / GQA / MQA)
 @dataclass(frozen=True)
 class HeadSizes:
-  """Sizes of one attention layer; `scale` multiplies q . k, `soft_cap` (0: none) bounds the result."""
+  """Sizes of one attention layer; `scale` multiplies q . k, `soft_cap` (0: none) bounds the result. `gate`: an output gate per lane
+  ("lane"), per head ("head") or none. `q_temp` = (coef, every): q grows by 1 + coef ln(floor((p + 1) / every) + 1) at position p.
+  `diff`: differential attention (Ye et al., "Differential Transformer"): two maps per head over the same values, the second subtracted
+  with a learned weight around `diff`. `sink`: a constant score in the softmax denominator, without a value."""
   heads: int
   kv_heads: int
   dim: int
   vdim: int
   scale: float
   soft_cap: float = 0.0
+  gate: str = "lane"
+  q_temp: tuple | None = None
+  diff: float | None = None
+  sink: float | None = None
+
+
+class Constant:
+  """A fixed tensor where layers expect a parameter."""
+
+  def __init__(self, t: torch.Tensor):
+    self.data = t
+
+  def leaf(self):
+    return self.data
 
 
 class Attention:
@@ -307,7 +324,7 @@ class Attention:
     """With `sizes` the layer has head counts and widths of its own (values may be narrower or wider than keys), and `gated` means an
     output gate from a projection of its own instead of a widened query projection."""
     c = config
-    self.config = c
+    self.config, self.sizes = c, sizes
     if sizes is not None:
       head_dim, num_kv_heads, query_scalar, soft_cap = sizes.dim, sizes.kv_heads, sizes.scale, sizes.soft_cap
     # gemma4 global layers have their own head width and key/value head count (src/maxtext/models/gemma4.py:186-196)
@@ -322,6 +339,13 @@ class Attention:
     self.window, self.inv_ts, self.interleaved, self.use_rope = window, rope_inv_ts, interleaved, use_rope
     self.qk_norm, self.query_scalar, self.soft_cap, self.rotary_dim = qk_norm, query_scalar, soft_cap, rotary_dim
     self.l2_qk_norm, self.temperature_tuning, self.chunk = l2_qk_norm, temperature_tuning, int(chunk)
+    # maps per head (two in differential attention); the cache keeps them side by side as one key of width kw
+    self.maps = 2 if sizes is not None and sizes.diff is not None else 1
+    self.kw = self.dh * self.maps
+    self.q_temp = sizes.q_temp if sizes is not None else None
+    if temperature_tuning and not use_rope:
+      # llama4 NoPE layers (src/maxtext/layers/attentions.py:1302-1308)
+      self.q_temp = (float(getattr(c, "temperature_tuning_scale", 0.1)), float(getattr(c, "temperature_tuning_floor_scale", 8192.0)))
     # YaRN "attention scaling" (src/maxtext/layers/embeddings.py:1020-1022): rotated q and k are each multiplied by
     # 0.1 ln(factor) + 1; here the product of the two factors scales the logits
     self.logit_scale = 1.0
@@ -333,27 +357,30 @@ class Attention:
     ab = b.sub(*name.split("/"))
     depth_scale = 1.0 if (qk_norm or (query_scalar is not None and query_scalar != 1.0)) else 1.0 / math.sqrt(self.dh)
     kv_tp = "col" if self.hkv >= tp else None
-    self.q = ab.sub("query").linear("kernel", (self.d,), (self.hq, self.dh * (2 if self.gated else 1)), ("embed", "q_heads", "kv"),
+    self.q = ab.sub("query").linear("kernel", (self.d,), (self.hq, self.kw * (2 if self.gated else 1)), ("embed", "q_heads", "kv"),
                                     "fan_in_normal", depth_scale, tp="col")
-    self.k = ab.sub("key").linear("kernel", (self.d,), (self.hkv, self.dh), ("embed", "kv_heads", "kv_head_dim"),
+    self.k = ab.sub("key").linear("kernel", (self.d,), (self.hkv, self.kw), ("embed", "kv_heads", "kv_head_dim"),
                                   "fan_in_normal", tp=kv_tp)
     # share_kv_projections (src/maxtext/layers/attentions.py:289): the value is the (un-normalised, un-rotated) key projection
     self.v = None if self.share_kv else ab.sub("value").linear("kernel", (self.d,), (self.hkv, self.dv), ("embed", "kv_heads", "kv_head_dim"),
                                                                "fan_in_normal", tp=kv_tp)
-    self.g = ab.sub("gate").linear("kernel", (self.d,), (self.hq, self.dv), ("embed", "q_heads", "kv"), "fan_in_normal", tp="col") \
+    self.gate_per_head = sizes is not None and sizes.gate == "head"
+    self.g = ab.sub("gate").linear("kernel", (self.d,), (self.hq,) if self.gate_per_head else (self.hq, self.dv),
+                                   ("embed", "q_heads") if self.gate_per_head else ("embed", "q_heads", "kv"), "fan_in_normal", tp="col") \
         if gated and sizes is not None else None
     self.o = ab.sub("out").linear("kernel", (self.hq, self.dv), (self.d,), ("heads", "kv", "embed"), "fan_in_normal",
                                   tp="row")
     self.qkv = FusedParam([self.q, self.k, self.v]) if (not self.gated and not self.share_kv and sizes is None
                                                         and FusedParam.possible([self.q, self.k, self.v])) else None
     # everything that reads the layer input as one product [q | k | v | gate] (inference)
-    self.qkvg = FusedParam([self.q, self.k, self.v, self.g]) if self.g is not None and FusedParam.possible([self.q, self.k, self.v, self.g]) else None
+    self.in_parts = [p for p in (self.q, self.k, self.v, self.g) if p is not None]
+    self.qkvg = FusedParam(self.in_parts) if sizes is not None and FusedParam.possible(self.in_parts) else None
     self.vn = Norm(ab, "value_norm", self.dh, c.normalization_layer_epsilon, with_scale=(self.v_norm == "scale"), axes=("norm",)) if self.v_norm else None
     self.bq = self.bk = self.bv = None
     if bias:
-      self.bq = ab.sub("query").vector("bias", self.hq * self.dh, ("q_heads",), init="zeros", tp=True)
-      self.bk = ab.sub("key").vector("bias", self.hkv * self.dh, ("kv_heads",), init="zeros", tp=kv_tp is not None)
-      self.bv = ab.sub("value").vector("bias", self.hkv * self.dh, ("kv_heads",), init="zeros", tp=kv_tp is not None)
+      self.bq = ab.sub("query").vector("bias", self.hq * self.kw, ("q_heads",), init="zeros", tp=True)
+      self.bk = ab.sub("key").vector("bias", self.hkv * self.kw, ("kv_heads",), init="zeros", tp=kv_tp is not None)
+      self.bv = ab.sub("value").vector("bias", self.hkv * self.dv, ("kv_heads",), init="zeros", tp=kv_tp is not None)
     # the output projection carries a bias whenever q/k/v do, except for qwen2 (src/maxtext/layers/attentions.py:833)
     self.bo = ab.sub("out").vector("bias", self.d, ("embed",), init="zeros") if (bias if out_bias is None else out_bias) else None
     if self.bo is not None and tp > 1 and sp_enabled(c):
@@ -363,8 +390,8 @@ class Attention:
     if self.global_qk_norm:
       # olmo3 (src/maxtext/layers/attentions.py:486-494): one RMS statistic over all heads of a token, scale per lane
       assert tp == 1, "the all-head q/k normalisation of olmo3 is not implemented under tensor parallelism"
-      self.qn = Norm(ab, "query_norm", self.hq * self.dh, c.normalization_layer_epsilon, axes=("norm",))
-      self.kn = Norm(ab, "key_norm", self.hkv * self.dh, c.normalization_layer_epsilon, axes=("norm",))
+      self.qn = Norm(ab, "query_norm", self.hq * self.kw, c.normalization_layer_epsilon, axes=("norm",))
+      self.kn = Norm(ab, "key_norm", self.hkv * self.kw, c.normalization_layer_epsilon, axes=("norm",))
     elif qk_norm:
       ws = bool(getattr(c, "qk_norm_with_scale", True))         # false: plain RMS normalisation without a learned scale
       self.qn = Norm(ab, "query_norm", self.dh, c.normalization_layer_epsilon, qk_norm_offset, with_scale=ws, axes=("norm",))
@@ -374,6 +401,32 @@ class Attention:
         if n_ is not None and n_.scale is not None:
           n_.scale.pdef.tp_partial = True        # every rank normalises its own heads with the shared per-lane scale
     self.sinks = ab.vector("sinks", self.hq, ("q_heads",), init="zeros", tp=True) if sinks else None
+    if sizes is not None and sizes.sink is not None:
+      self.sinks = Constant(torch.full((self.hq * self.maps,), float(sizes.sink), device=rope_inv_ts.device))
+    self.lam = None
+    if self.maps == 2:
+      assert tp == 1, "differential attention is not split over the tensor axis"
+      self.lam = [ab.sub("lambda").vector(n, self.dh, ("norm",), init="zeros") for n in ("q1", "k1", "q2", "k2")]
+
+  def sink_data(self, dtype):
+    """The sink scores in the compute type, or None."""
+    if isinstance(self.sinks, Constant) and self.sinks.data.dtype != dtype:
+      self.sinks.data = self.sinks.data.to(dtype)
+    return self.sinks.data if self.sinks is not None else None
+
+  def _maps_apart(self, q):
+    """q [B, S, heads * 2, dim] -> [B, S, heads * 2, 2 * dim]: map j of a head meets its own half of the cached key (both halves share the
+    values), so that the two maps are two query heads of ordinary grouped attention."""
+    z = torch.zeros_like(q[:, :, 0::2])
+    return torch.stack([torch.cat([q[:, :, 0::2], z], -1), torch.cat([z, q[:, :, 1::2]], -1)], 3).flatten(2, 3)
+
+  def _difference(self, o):
+    """o [B, S, heads * 2, Dv] -> [B, S, heads, Dv]: (map 1 - lambda map 2), normalised per head, times 1 - diff; fp32 inside."""
+    d = float(self.sizes.diff)
+    lq1, lk1, lq2, lk2 = (p.leaf().float() for p in self.lam)
+    lam = torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + d
+    y = o[:, :, 0::2].float() - lam * o[:, :, 1::2].float()
+    return (y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + self.config.normalization_layer_epsilon) * (1.0 - d)).to(o.dtype)
 
   def _project(self, x, ctx, tp_rt=None):
     B, S, _ = x.shape
@@ -388,26 +441,34 @@ class Attention:
     q = ctx.keep("query_proj", F.linear(x, self.q, ctx.reuse("query_proj"), self.bq))
     k = ctx.keep("key_proj", F.linear(x, self.k, ctx.reuse("key_proj"), self.bk))
     v = k if self.share_kv else ctx.keep("value_proj", F.linear(x, self.v, ctx.reuse("value_proj"), self.bv))
-    return None, (q.view(B, S, hq, -1), k.view(B, S, hkv, dh), v.view(B, S, hkv, self.dv))
+    return None, (q.view(B, S, hq * self.maps, -1), k.view(B, S, hkv * self.maps, dh), v.view(B, S, hkv, self.dv))
 
-  def _serve(self, x, ctx):
-    """Inference kernels: one product for q | k | v | gate, rotation and norms in one pass that also fills the cache, attention over
-    the cache, and the gate with the last step of it (`ops.cached_attention`)."""
+  def serves(self, x, ctx) -> bool:
+    """Will this call run the inference kernels?"""
+    if self.sizes is None or ctx.cache is None:
+      return False
+    from ..ops import cached_attention as CA
+    return CA.servable(x, self, ctx)
+
+  def _serve(self, x, ctx, rows=None):
+    """Inference kernels: one product for q | k | v | gate (`rows`: its result, one matrix per part), rotation and norms in one pass that
+    also fills the cache, attention over the cache, and the gate with the last step of it (`ops.cached_attention`)."""
     from ..ops import cached_attention as CA
     B, S, _ = x.shape
-    if self.qkvg is not None and self.qkvg.fusable():
-      p = F.linear(x, self.qkvg).view(B * S, -1)
-      q, k, v, g = torch.split(p, self.qkvg.rows, dim=-1)
-    else:
-      q, k, v, g = (F.linear(x, w).view(B * S, -1) for w in (self.q, self.k, self.v, self.g))
-    return F.linear(CA.serve(self, q, k, v, g, ctx).view(B, S, -1), self.o)
+    if rows is None:
+      if self.qkvg is not None and self.qkvg.fusable():
+        rows = torch.split(F.linear(x, self.qkvg).view(B * S, -1), self.qkvg.rows, dim=-1)
+      else:
+        rows = [F.linear(x, w).view(B * S, -1) for w in self.in_parts]
+    q, k, v = rows[:3]
+    return F.linear(CA.serve(self, q, k, v, rows[3] if self.g is not None else None, ctx).view(B, S, -1), self.o)
 
-  def __call__(self, x, ctx):
+  def __call__(self, x, ctx, rows=None, out_bias=True):
+    """`out_bias=False` leaves the output projection's bias to the caller (it may join a later step)."""
     B, S, _ = x.shape
-    if self.g is not None and self.l2_qk_norm and ctx.cache is not None:
-      from ..ops import cached_attention as CA
-      if CA.servable(x, self, ctx):
-        return self._serve(x, ctx)
+    if self.serves(x, ctx):
+      y = self._serve(x, ctx, rows)
+      return y + self.bo.data if self.bo is not None and out_bias else y
     # tensor parallelism: with the fused runtime the two all-reduces of this block run inside GEMM epilogues
     tp_rt = tp_fused.runtime_for(ctx, x, self.d) if ctx.tp_size > 1 else None
     fuse_in = tp_rt is not None and self.qkv is not None and self.bq is None and self.qkv.fusable()
@@ -417,7 +478,7 @@ class Attention:
     packed, sep = self._project(x, ctx, tp_rt if fuse_in else None)
     gate = F.linear(x, self.g) if self.g is not None else None
     moba = bool(getattr(self.config, "moba", False)) and ctx.cache is None and ctx.cp_size == 1
-    plain = (ctx.positions3 is None and not self.qk_norm and self.g is None and self.vn is None and not self.share_kv and self.sinks is None and self.rotary_dim is None and not self.gated and ctx.bidir is None and not moba and ctx.cache is None and ctx.cp_size == 1
+    plain = (ctx.positions3 is None and self.maps == 1 and not self.qk_norm and self.g is None and self.vn is None and not self.share_kv and self.sinks is None and self.rotary_dim is None and not self.gated and ctx.bidir is None and not moba and ctx.cache is None and ctx.cp_size == 1
              and not self.l2_qk_norm and not self.temperature_tuning and not (self.chunk and S > self.chunk))
     saved_ctx = ctx.reuse("context")
     if saved_ctx is not None and packed is not None and plain:
@@ -435,8 +496,8 @@ class Attention:
       if self.gated:
         q, gate = q[..., :self.dh], q[..., self.dh:].reshape(B, S, -1)
       if self.global_qk_norm:
-        q = self.qn(q.reshape(B, S, -1)).view(B, S, self.hq_l, self.dh)
-        k = self.kn(k.reshape(B, S, -1)).view(B, S, self.hkv_l, self.dh)
+        q = self.qn(q.reshape(B, S, -1)).view(q.shape)
+        k = self.kn(k.reshape(B, S, -1)).view(k.shape)
       elif self.qk_norm:
         q, k = self.qn(q), self.kn(k)
       if self.vn is not None:
@@ -456,12 +517,12 @@ class Attention:
         k = (k.float() * torch.rsqrt(k.float().pow(2).mean(-1, keepdim=True) + eps)).to(k.dtype)
       if (self.query_scalar and self.query_scalar != 1.0) or self.logit_scale != 1.0:
         q = q * ((self.query_scalar or 1.0) * self.logit_scale)
-      if self.temperature_tuning and not self.use_rope:
-        # llama4 NoPE layers (attentions.py:1302-1308): log(floor((pos + 1) / floor_scale) + 1) * scale + 1
-        c_ = self.config
-        sc = torch.log(torch.floor((ctx.positions.float() + 1.0) / float(getattr(c_, "temperature_tuning_floor_scale", 8192.0))) + 1.0) \
-            * float(getattr(c_, "temperature_tuning_scale", 0.1)) + 1.0
+      if self.q_temp is not None:
+        coef, every = self.q_temp
+        sc = torch.log(torch.floor((ctx.positions.float() + 1.0) / float(every)) + 1.0) * float(coef) + 1.0
         q = (q.float() * sc[:, :, None, None]).to(q.dtype)
+      if self.maps == 2:
+        q, k = self._maps_apart(q), k.reshape(B, S, self.hkv_l, self.kw)
       if moba:
         # mixture-of-block attention: each query attends its own block and the best `moba_topk` earlier key blocks
         seg = None
@@ -476,7 +537,7 @@ class Attention:
         out = F.attention(q, k, v, ctx.positions, ctx.segment_ids, 1.0, self.soft_cap, self.window, chunk=self.chunk,
                           sinks=self.sinks.leaf() if self.sinks is not None else None)
       elif ctx.cache is not None:
-        out = ctx.cache.attend(q, k, v, ctx, window=self.window, soft_cap=self.soft_cap, sinks=self.sinks)
+        out = ctx.cache.attend(q, k, v, ctx, window=self.window, soft_cap=self.soft_cap, sinks=self.sinks, chunk=self.chunk)
       elif ctx.cp_size > 1:
         from ..parallel.context_parallel import context_attention
         out = context_attention(q, k, v, ctx.positions, ctx.segment_ids, ctx, 1.0, self.soft_cap, self.window)
@@ -485,12 +546,14 @@ class Attention:
       else:
         out = F.attention(q, k, v, ctx.positions, ctx.segment_ids, 1.0, self.soft_cap, self.window)
     ctx.keep("context", out)
+    if self.maps == 2:
+      out = self._difference(out)
     if gate is not None:
-      out = (out.reshape(B, S, -1).float() * torch.sigmoid(gate.float())).to(out.dtype)
+      out = (out.reshape(*gate.shape, -1).float() * torch.sigmoid(gate.float())[..., None]).to(out.dtype)
     if tp_rt is not None and ctx.reuse("out_proj") is None and self.bo is None and self.o.lora is None:
       y = F.linear(out.reshape(B, S, -1), self.o, tp_reduce=tp_rt)
     else:
-      y = F.linear(out.reshape(B, S, -1), self.o, ctx.reuse("out_proj"), self.bo if ctx.tp_size == 1 else None)
+      y = F.linear(out.reshape(B, S, -1), self.o, ctx.reuse("out_proj"), self.bo if ctx.tp_size == 1 and out_bias else None)
       if ctx.reuse("out_proj") is None:
         y = tp_exit(y, ctx)
         if self.bo is not None and ctx.tp_size > 1:

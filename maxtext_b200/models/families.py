@@ -33,6 +33,8 @@ def describe(c) -> Family:
     return Family(norm_offset=1.0)           # every RMS scale is stored zero-centred and applied as (1 + scale)
   if blk == "silinex":
     return Family(norm_offset=1.0, residual_fp32=True)
+  if blk == "sitivik":
+    return Family(residual_fp32=True)
   if blk == "tipidra":
     return Family(norm_kind="layernorm", residual_fp32=True, static_streams=True)
   return Family()
@@ -173,6 +175,9 @@ def layer_plans(c) -> list[LayerPlan]:
   if blk == "silinex":
     from .silinex import layer_plans as silinex_plans
     return silinex_plans(c)
+  if blk == "sitivik":
+    from .sitivik import layer_plans as sitivik_plans
+    return sitivik_plans(c)
   if blk == "tipidra":
     from .tipidra import layer_plans as tipidra_plans
     return tipidra_plans(c)
@@ -233,4 +238,4 @@ def layer_plans(c) -> list[LayerPlan]:
     return plans
   raise NotImplementedError(
       f"decoder_block={blk!r} parses but has no model implementation here yet (implemented: llama2, mistral, mixtral, "
-      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, silinex, tipidra, simple)")
+      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, silinex, sitivik, tipidra, simple)")

@@ -34,7 +34,7 @@ class BlockPlan:
   post_mlp_norm: str | None = None
   attn_name: str = "self_attention"
   mlp_name: str = "mlp"
-  attention: str = "gqa"                 # gqa | mla | gdn (gated delta network, qwen3-next) | gla | ssm (selective scan) | compressed
+  attention: str = "gqa"                 # gqa | mla | gdn (gated delta network, qwen3-next) | gla | ssm (selective scan) | retention | channel_delta | parallel (two of them) | compressed
   mixer: dict | None = None              # sizes of this block's mixer, for families whose layers differ (None: the config's)
   gated_attn: bool = False               # sigmoid output gate: from a widened query projection (qwen3-next) or, with `mixer`, a projection of its own
   window: int = 0
@@ -67,6 +67,14 @@ class BlockPlan:
   hyper: str = ""                        # "static": hyper-connections with constant maps around the two sublayers
   residual_mult: float = 1.0             # factor on each branch before it joins the residual stream
   residual_fp32: bool = False            # fp32 residual stream with sandwich norms, fused with the residual add (`F.residual_norm`)
+  pair: tuple | None = None              # "parallel": the plans of the two mixers that read the same input ...
+  join: tuple = (1.0, 1.0, False)        # ... their factors, and whether each result is RMS-normalised before the sum
+  mask: str = ""                         # `mixer` attention: "window" | "chunk" | "" (every earlier token); the size is the mixer's
+  interleaved: bool = False              # `mixer` attention: neighbouring lanes rotate together instead of the halves
+  gate: str = "lane"                     # `mixer` attention: one output gate per "lane" or per "head"
+  sink_value: float | None = None        # `mixer` attention: a constant sink score instead of learned ones
+  layer_scale: bool = False              # one learned factor per lane on every branch before it joins the stream
+  token_side: int = 0                    # width of the per-layer token input that joins the stream after the feed-forward (0: none)
   compress_ratio: int = 0                # DeepSeek-V4 compressed attention: 0 (window only), 4 (sparse) or 128 (heavy)
 
 
@@ -74,6 +82,58 @@ class BlockPlan:
 class LayerPlan:
   stack: str = "layers"                  # name of the stacked collection in the checkpoint tree
   blocks: list = field(default_factory=lambda: [BlockPlan()])
+
+
+def build_mixer(b: L.Builder, c, plan: BlockPlan, name: str, rope_tables: dict):
+  """The token mixer of a block: the attention kind, recurrence or pair of them that its plan names."""
+  inv_ts, interleaved = rope_tables[plan.rope]
+  rot = int(c.head_dim * c.partial_rotary_factor) if 0 < c.partial_rotary_factor < 1.0 else None
+  m = plan.mixer
+  if plan.attention == "parallel":
+    from ..layers.parallel import ParallelMixer
+    return ParallelMixer(b, c, name, *(lambda ab, n, p=p: build_mixer(ab, c, p, n, rope_tables) for p in plan.pair), plan.join)
+  if plan.attention == "mla":
+    if m is not None:
+      inv_ts, interleaved = ref.rope_inv_timescale(int(m["rot_dim"]), 1.0, float(m["rot"]["base"])).to(inv_ts.device), True
+      sizes = L.LatentSizes(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["q_rank"]), int(m["kv_rank"]),
+                            float(m["scale"]), int(m["mask"]["size"]))
+    return L.MLA(b, c, inv_ts, interleaved, name, sizes if m is not None else None)
+  if plan.attention == "gdn":
+    from ..layers.gdn import DeltaSizes, GatedDeltaNet
+    return GatedDeltaNet(b, c, name, DeltaSizes(int(m["kv_heads"]), int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]))
+                         if m is not None else None)
+  if plan.attention == "gla":
+    from ..layers.gla import GatedLinearAttention
+    return GatedLinearAttention(b, c, name, int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"]), int(m["decay_rank"]))
+  if plan.attention == "ssm":
+    from ..layers.ssm import ScanSizes, SelectiveScan
+    return SelectiveScan(b, c, name, ScanSizes(int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m["conv"])))
+  if plan.attention == "retention":
+    from ..layers.retention import Retention, RetentionSizes
+    return Retention(b, c, name, RetentionSizes(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["rot"]["dims"]), float(m["rot"]["base"]),
+                                                tuple(float(x) for x in m["decay"])), inv_ts.device)
+  if plan.attention == "channel_delta":
+    from ..layers.channel_delta import ChannelDeltaNet, ChannelDeltaSizes
+    return ChannelDeltaNet(b, c, name, ChannelDeltaSizes(int(m["kv_heads"]), int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]),
+                                                         int(m["decay_rank"]), int(m["gate_rank"])))
+  if plan.attention == "compressed":
+    from ..layers.attention_compressed import CompressedAttention
+    return CompressedAttention(b, c, name, plan.compress_ratio, int(c.sliding_window_size))
+  sizes, window, chunk = None, plan.window, plan.chunk
+  if m is not None:
+    turn = m.get("rot") or {"dims": 0, "base": 1.0}
+    rot, interleaved = int(turn["dims"]), plan.interleaved
+    inv_ts = ref.rope_inv_timescale(rot, 1.0, float(turn["base"]), stretch=turn.get("scaling")).to(inv_ts.device)
+    temp = m.get("q_temp")
+    sizes = L.HeadSizes(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), float(m.get("softcap", 0.0)), plan.gate,
+                        (float(temp["coef"]), float(temp["every"])) if temp else None, float(m["diff"]) if "diff" in m else None, plan.sink_value)
+    window, chunk = (int(m["mask"]["size"]) if plan.mask == kind else 0 for kind in ("window", "chunk"))
+  return L.Attention(b, c, name, window, inv_ts, interleaved, plan.use_rope and rot != 0, plan.qk_norm,
+                     plan.query_scalar, plan.soft_cap, plan.attn_bias,
+                     rotary_dim=rot, sinks=plan.sinks, l2_qk_norm=plan.l2_qk_norm,
+                     temperature_tuning=plan.temperature_tuning, chunk=chunk, out_bias=plan.attn_out_bias,
+                     global_qk_norm=plan.global_qk_norm, gated=plan.gated_attn, qk_norm_offset=plan.norm_offset,
+                     head_dim=plan.head_dim, num_kv_heads=plan.kv_heads, share_kv=plan.share_kv, v_norm=plan.v_norm, sizes=sizes)
 
 
 class DecoderBlock:
@@ -92,45 +152,7 @@ class DecoderBlock:
     eps = c.normalization_layer_epsilon
     mk = lambda n: L.Norm(b, n + s, c.emb_dim, eps, plan.norm_offset, kind=plan.norm_kind)  # noqa: E731
     self.n1 = mk(plan.pre_attn_norm) if plan.pre_attn_norm else None
-    inv_ts, interleaved = rope_tables[plan.rope]
-    rot = int(c.head_dim * c.partial_rotary_factor) if 0 < c.partial_rotary_factor < 1.0 else None
-    if plan.attention == "mla":
-      if plan.mixer is not None:
-        m = plan.mixer
-        inv_ts, interleaved = ref.rope_inv_timescale(int(m["rot_dim"]), 1.0, float(m["rot"]["base"])).to(inv_ts.device), True
-        sizes = L.LatentSizes(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["q_rank"]), int(m["kv_rank"]),
-                              float(m["scale"]), int(m["mask"]["size"]))
-      self.attn = L.MLA(b, c, inv_ts, interleaved, plan.attn_name + s, sizes if plan.mixer is not None else None)
-    elif plan.attention == "gdn":
-      from ..layers.gdn import DeltaSizes, GatedDeltaNet
-      m = plan.mixer
-      self.attn = GatedDeltaNet(b, c, plan.attn_name + s, DeltaSizes(int(m["kv_heads"]), int(m["heads"]), int(m["dim"]), int(m["vdim"]),
-                                                                     int(m["conv"])) if m is not None else None)
-    elif plan.attention == "gla":
-      from ..layers.gla import GatedLinearAttention
-      m = plan.mixer
-      self.attn = GatedLinearAttention(b, c, plan.attn_name + s, int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"]),
-                                       int(m["decay_rank"]))
-    elif plan.attention == "ssm":
-      from ..layers.ssm import ScanSizes, SelectiveScan
-      m = plan.mixer
-      self.attn = SelectiveScan(b, c, plan.attn_name + s, ScanSizes(int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m["conv"])))
-    elif plan.attention == "compressed":
-      from ..layers.attention_compressed import CompressedAttention
-      self.attn = CompressedAttention(b, c, plan.attn_name + s, plan.compress_ratio, int(c.sliding_window_size))
-    else:
-      sizes = None
-      if plan.mixer is not None:
-        m = plan.mixer
-        rot, interleaved = int(m["rot"]["dims"]), False
-        inv_ts = ref.rope_inv_timescale(rot, 1.0, float(m["rot"]["base"])).to(inv_ts.device)
-        sizes = L.HeadSizes(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), float(m["softcap"]))
-      self.attn = L.Attention(b, c, plan.attn_name + s, plan.window, inv_ts, interleaved, plan.use_rope and rot != 0, plan.qk_norm,
-                              plan.query_scalar, plan.soft_cap, plan.attn_bias,
-                              rotary_dim=rot, sinks=plan.sinks, l2_qk_norm=plan.l2_qk_norm,
-                              temperature_tuning=plan.temperature_tuning, chunk=plan.chunk, out_bias=plan.attn_out_bias,
-                              global_qk_norm=plan.global_qk_norm, gated=plan.gated_attn, qk_norm_offset=plan.norm_offset,
-                              head_dim=plan.head_dim, num_kv_heads=plan.kv_heads, share_kv=plan.share_kv, v_norm=plan.v_norm, sizes=sizes)
+    self.attn = build_mixer(b, c, plan, plan.attn_name + s, rope_tables)
     self.n1b = mk(plan.post_attn_norm) if plan.post_attn_norm else None
     self.n2 = mk(plan.pre_mlp_norm) if plan.pre_mlp_norm else None
     if plan.mlp == "moe":
@@ -147,6 +169,12 @@ class DecoderBlock:
     else:
       self.mlp = L.MLP(b, c, plan.mlp_name + s, plan.mlp_hidden, bias=plan.mlp_bias)
     self.n2b = mk(plan.post_mlp_norm) if plan.post_mlp_norm else None
+    self.ls1 = b.sub("layer_scale").vector("mixer" + s, c.emb_dim) if plan.layer_scale else None
+    self.ls2 = b.sub("layer_scale").vector("mlp" + s, c.emb_dim) if plan.layer_scale and self.mlp is not None else None
+    self.side = None
+    if plan.token_side:
+      from ..layers.parallel import TokenSide
+      self.side = TokenSide(b, c, plan.token_side)
     self.layer_scalar = b._add("layer_scalar" + s, shape=(1,), ref_shape=(1,), logical_axes=(None,), kind="same", init="ones") \
         if plan.layer_scalar else None
     self.mhc_attn = self.mhc_mlp = None
@@ -177,7 +205,7 @@ class DecoderBlock:
     if self.hc1 is not None:
       return self._call_static_streams(x, ctx)
     if self.plan.residual_fp32:
-      return self._call_fp32_stream(x, ctx)
+      return self._call_fp32_stream(x, ctx) if self.n1b is not None else self._call_joined_stream(x, ctx)
     a = self.attn(self.n1(x) if self.n1 is not None else x, ctx)
     if self.n1b is not None:
       a = self.n1b(a)
@@ -223,6 +251,21 @@ class DecoderBlock:
     x, h = F.residual_norm(x, a, self.n1b, m, self.n2)
     f = self.mlp(h, ctx)
     x, ctx.normed = F.residual_norm(x, f, self.n2b, m, ctx.next_norm)
+    return x
+
+
+  def _call_joined_stream(self, x, ctx: LayerCtx):
+    """x fp32 [B, S, D], pre-norm. One kernel per border between sublayers: the branches (weighted, normalised, scaled lane by lane) join the
+    stream, and what reads it next comes out of the same pass: a norm, or the stream itself in the compute type for the token input."""
+    h = ctx.normed if ctx.normed is not None else F.stream_norm(x, self.n1, self.n1.scale.data.dtype)
+    ctx.normed = None
+    last = F.AS_IS if self.side is not None else ctx.next_norm
+    x, h = F.residual_join(x, self.attn(h, ctx), self.ls1, self.n2 if self.mlp is not None else last)
+    if self.mlp is not None:
+      x, h = F.residual_join(x, self.mlp(h, ctx), self.ls2, last)
+    if self.side is not None:
+      x, h = F.residual_norm(x, self.side(h, ctx), self.side.norm, 1.0, ctx.next_norm)
+    ctx.normed = h
     return x
 
 

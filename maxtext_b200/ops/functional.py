@@ -291,6 +291,64 @@ def residual_norm(x: torch.Tensor, branch: torch.Tensor, post, mult: float, nxt=
   return x, (ref.rmsnorm_f32(x, nxt.scale.leaf(), nxt.eps, nxt.offset).to(branch.dtype) if nxt is not None else None)
 
 
+class Branch:
+  """One addend of a residual step: `factor` * [RMS norm of] (`out` + bias)."""
+
+  def __init__(self, out, bias=None, norm=None, factor=1.0):
+    self.out, self.bias, self.norm, self.factor = out, bias, norm, float(factor)
+
+
+class Branches(list):
+  """The addends of one residual step."""
+
+
+AS_IS = object()          # `residual_join(nxt=AS_IS)`: what reads the stream next takes it as it is, in the compute type
+
+
+def residual_join(x: torch.Tensor, branch, lanes=None, nxt=None):
+  """(x + lanes * sum of the branches, nxt(of that) in the branch's dtype or None). `branch` is a tensor or `Branches` (up to two), `lanes` a
+  parameter with one factor per lane, `nxt` a norm or AS_IS. On a GPU one kernel, which updates x in place."""
+  parts = branch if isinstance(branch, Branches) else [Branch(branch)]
+  dt = parts[0].out.dtype
+  if _stream_kernel_ok(x, *(p.out for p in parts)) and x.dtype == torch.float32 and x.is_contiguous():
+    x2 = x.view(-1, x.shape[-1])
+    outs = [p.out.reshape(x2.shape).contiguous() for p in parts]
+    y = torch.empty(x2.shape, dtype=dt, device=x.device) if nxt is not None else None
+    a, b = parts[0], parts[1] if len(parts) > 1 else Branch(None)
+
+    def data(p):
+      return p.data if p is not None else None
+    eps = float(next((n.eps for n in (a.norm, b.norm, nxt) if n is not None and n is not AS_IS), 0.0))
+    assert all(n is None or n is AS_IS or (n.eps == eps and n.offset == 0) for n in (a.norm, b.norm, nxt))
+    backend.ext().residual_join(x2, outs[0], data(a.bias), data(a.norm.scale if a.norm is not None else None), a.factor, outs[1] if len(parts) > 1 else None,
+                                data(b.bias), data(b.norm.scale if b.norm is not None else None), b.factor, data(lanes),
+                                nxt.scale.data if nxt is not None and nxt is not AS_IS else None, y, eps)
+    return x, (y.view(x.shape) if y is not None else None)
+  total = 0.0
+  for p in parts:
+    t = p.out.float()
+    if p.bias is not None:
+      t = t + p.bias.leaf().float()
+    if p.norm is not None:
+      t = ref.rmsnorm_f32(t, p.norm.scale.leaf(), p.norm.eps, p.norm.offset)
+    total = total + p.factor * t
+  x = x.float() + (total if lanes is None else lanes.leaf().float() * total)
+  if nxt is None:
+    return x, None
+  return x, (x if nxt is AS_IS else ref.rmsnorm_f32(x, nxt.scale.leaf(), nxt.eps, nxt.offset)).to(dt)
+
+
+def token_gate(g: torch.Tensor, table, tokens: torch.Tensor) -> torch.Tensor:
+  """gelu_tanh(g) * table[tokens] for g [B, S, dim]."""
+  if not torch.is_grad_enabled() and backend.use_cuda_kernels(g) and g.dtype in (torch.bfloat16, torch.float32) and table.data.dtype == g.dtype:
+    g2 = g.reshape(-1, g.shape[-1])
+    out = torch.empty(g2.shape, dtype=g.dtype, device=g.device)
+    backend.ext().token_gate(g2 if g2.is_contiguous() else g2.contiguous(), table.data, tokens.reshape(-1).long().contiguous(), out)
+    return out.view(g.shape)
+  e = embedding(tokens, table)
+  return (ref.act_fn("gelu")(g.float()) * e.float()).to(g.dtype)
+
+
 # =============================================================================== several fp32 residual streams
 class StreamReader:
   """What reads the streams in front of a sublayer: the weights of the streams (of a `layers.mhc.StaticHyperConnection`; None: their plain

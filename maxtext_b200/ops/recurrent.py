@@ -24,11 +24,13 @@ def chunked_ok(t: torch.Tensor, S: int, dk: int, dv: int) -> bool:
   return t.dtype == torch.bfloat16 and S >= CHUNK_FROM and backend.ext().chunk_supported(dk, dv)
 
 
-def gated_head_norm(o, z, scale, eps):
-  """Definition: o [.., H, Dv] RMS-normalised over Dv, times scale, times silu(z); fp32."""
+def gated_head_norm(o, z, scale, eps, gate="silu"):
+  """Definition: o [.., H, Dv] RMS-normalised over Dv, times scale (None: no weight), times silu(z) or sigmoid(z); fp32."""
   o = o.float()
-  o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * scale.float()
-  return o * torch.nn.functional.silu(z.float())
+  o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+  if scale is not None:
+    o = o * scale.float()
+  return o * (torch.nn.functional.silu(z.float()) if gate == "silu" else torch.sigmoid(z.float()))
 
 
 def delta_forward(layer, qkvz, ba, st):

@@ -52,11 +52,13 @@ def layernorm(x, scale, bias, eps):
 
 # ----------------------------------------------------------------------------- rope
 def rope_inv_timescale(head_dim: int, min_ts: float, max_ts: float, linear_scaling: float = 1.0,
-                       rope_type: str = "default", use_scale: bool = True, yarn: dict | None = None) -> torch.Tensor:
+                       rope_type: str = "default", use_scale: bool = True, yarn: dict | None = None,
+                       stretch: dict | None = None) -> torch.Tensor:
   """1/timescale per rotated pair, shape [head_dim/2] fp32.
 
   default: timescale_i = min*(max/min)^(2i/d) (x linear factor) (src/maxtext/layers/embeddings.py:318-334)
-  llama3.1: same base, then the Llama-3.1 wavelength-dependent rescale (embeddings.py:646-672)
+  llama3.1: same base, then the Llama-3.1 wavelength-dependent rescale (embeddings.py:646-672); `stretch` (factor, low, high, original)
+  asks for the same rescale with constants of its own
   yarn: blend of interpolated and extrapolated frequencies (embeddings.py:880-1027)
   """
   half = head_dim // 2
@@ -65,8 +67,9 @@ def rope_inv_timescale(head_dim: int, min_ts: float, max_ts: float, linear_scali
   if rope_type == "default" and linear_scaling != 1.0:
     ts = ts * linear_scaling
   inv = 1.0 / ts
-  if rope_type.startswith("llama3.1") and use_scale:
-    scale_factor, low_f, high_f, old_len = 8.0, 1.0, 4.0, 8192.0
+  if stretch is not None or (rope_type.startswith("llama3.1") and use_scale):
+    st = stretch or {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192.0}
+    scale_factor, low_f, high_f, old_len = (float(st[k]) for k in ("factor", "low", "high", "original"))
     wavelen = 2 * math.pi / inv
     smooth = (old_len / wavelen - low_f) / (high_f - low_f)
     mid = (1 - smooth) * inv / scale_factor + smooth * inv
