@@ -5,6 +5,7 @@
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <cuda_runtime.h>
+#include "cached_attention.h"
 
 extern "C" {
 int mt_stream_mix(float* x, int k, const void* branch, const int* dest, int per_token, const void* mix, const void* write, const void* read, const void* w,
@@ -14,15 +15,15 @@ int mt_ssm_conv(int f32, const void* x, long ldx, const void* w, const void* bia
 int mt_ssm_scan(int f32, const void* x, const void* z, long ldz, const void* q, long ldq, int off, const float* dt, const void* dt_bias, const void* A_log,
                 const void* D, int C, int N, int S, float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* y, int B,
                 cudaStream_t st);
-int mt_qkv_prep(int f32, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int H, int G, int D, int Dv, const int64_t* pos,
-                const float* inv_ts, int rot, float eps, int S, void* qp, int dq, void* kp, void* vp, int dvp, void* kc, void* vc, long max_len,
-                const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, long N, cudaStream_t st);
+int mt_qkv_prep(int f32, const mt::cattn::PrepArgs* a, long N, cudaStream_t st);
 int mt_cached_decode(const void* q, const void* k, const void* v, const int64_t* slots, const int64_t* lengths, long max_len, int B, int H, int G, int D, int Dv,
-                     float scale, float cap, int window, const void* sinks, const void* gate, long ldg, int splits, float* part, float* ml, void* out,
-                     cudaStream_t st);
+                     float scale, float cap, int window, int chunk, const void* sinks, const void* gate, long ldg, int per_head,
+                     const mt::cattn::DiffArgs* diff, int splits, float* part, float* ml, void* out, cudaStream_t st);
 int mt_cached_attention(int f32, const void* q, const void* k, const void* v, long max_len, const int64_t* slots, const int64_t* lengths, int B, int S, int H,
-                        int G, int D, int Dv, float scale, float cap, int window, const void* sinks, void* out, cudaStream_t st);
-int mt_head_gate(int f32, const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, void* out, int sms, cudaStream_t st);
+                        int G, int D, int Dv, float scale, float cap, int window, int chunk, const void* sinks, void* out, cudaStream_t st);
+int mt_head_gate(int f32, const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, int per_head, void* out, int sms, cudaStream_t st);
+int mt_diff_combine(int f32, const void* o, int dvp, const mt::cattn::DiffArgs* a, long N, int H, int Dv, const void* gate, long ldg, int per_head, void* out,
+                    int sms, cudaStream_t st);
 int mt_expert_up(int f32, const void* x, const void* w0, const void* w1, const float* wts, const int* idx, const int* sizes, const int* offs,
                  const int* row_pair, int n, int k, int E, int F, int D, float limit, void* h, int sms, cudaStream_t st);
 int mt_expert_down(int f32, const void* h, const void* w, const int* idx, const int* sizes, const int* offs, const int* row_pair, int n, int E, int D, int F,
@@ -99,18 +100,18 @@ void stream_mix(Tensor& x, const OptTensor& branch, const OptTensor& dest, int64
                      y ? y->data_ptr() : nullptr, f, N, (int)D, (float)eps, stream()), "stream_mix");
 }
 
-// x [B*S, >= C] projection rows, w [taps, C], bias [C], hist [slots, taps-1, C] -> y [B*S, C]
-void ssm_conv(const Tensor& x, const Tensor& w, const Tensor& bias, int64_t S, Tensor& hist, const Tensor& slots, const Tensor& lengths,
+// x [B*S, >= C] projection rows, w [taps, C], bias [C] or None, hist [slots, taps-1, C] -> y [B*S, C]
+void ssm_conv(const Tensor& x, const Tensor& w, const OptTensor& bias, int64_t S, Tensor& hist, const Tensor& slots, const Tensor& lengths,
               const OptTensor& new_lens, Tensor& y) {
   const bool f = f32(x);
   TORCH_CHECK(w.dim() == 2 && w.size(0) >= 1);
   const int64_t B = slots.numel(), taps = w.size(0), C = w.size(1);
   rows2d(x, x, B * S, C, "projection");
   TORCH_CHECK((reinterpret_cast<uintptr_t>(x.data_ptr()) % 16) == 0);
-  same(w, x, taps * C, "filter"); same(bias, x, C, "bias"); same(y, x, B * S * C, "y");
+  same(w, x, taps * C, "filter"); same(y, x, B * S * C, "y");
   TORCH_CHECK(hist.is_cuda() && hist.scalar_type() == torch::kFloat32 && hist.is_contiguous() && hist.dim() == 3 && hist.size(1) == taps - 1 && hist.size(2) == C);
   c10::cuda::CUDAGuard guard(x.device());
-  done(mt_ssm_conv(f, x.data_ptr(), x.stride(0), w.data_ptr(), bias.data_ptr(), (int)taps, (int)C, (int)S, hist.data_ptr<float>(), longs(slots, B, "slots"),
+  done(mt_ssm_conv(f, x.data_ptr(), x.stride(0), w.data_ptr(), same(bias, x, C, "bias"), (int)taps, (int)C, (int)S, hist.data_ptr<float>(), longs(slots, B, "slots"),
                    longs(lengths, B, "lengths"), longs(new_lens, B, "new_lens"), y.data_ptr(), (int)B, stream()), "ssm_conv");
 }
 
@@ -140,27 +141,60 @@ void check_cache(const Tensor& k, const Tensor& v, const Tensor& like, int64_t D
   same(v, like, v.numel(), "value cache");
 }
 
-// q / k / v rows of the projections -> qp [N, H, dq], kp [N, G, dq] or None, vp [N, G, dvp] or None, cache rows; rot: rotated lanes; eps < 0: no norm
+// q / k / v rows of the projections -> qp [N, H * maps, dq], kp [N, G, dq] or None, vp [N, G, dvp] or None, cache rows. rot: rotated lanes;
+// eps < 0: no norm; without norm weights the norm follows the rotation, with them it precedes it (one head's weights, or all heads').
+// temp_every 0: no query temperature. maps 2: differential attention, D being the width of one map.
 void qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, int64_t D, int64_t Dv, const Tensor& pos, const OptTensor& inv_ts, int64_t rot, double eps,
               Tensor& qp, const OptTensor& kp, const OptTensor& vp, Tensor& kc, Tensor& vc, const Tensor& slots, const Tensor& lengths,
-              const OptTensor& new_lens) {
+              const OptTensor& new_lens, const OptTensor& bq, const OptTensor& bk, const OptTensor& bv, const OptTensor& wq, const OptTensor& wk, bool paired,
+              int64_t maps, double temp_coef, double temp_every) {
   const bool f = f32(q);
-  TORCH_CHECK(qp.dim() == 3 && rot % 2 == 0 && rot >= 0 && rot <= D && bool(inv_ts) == (rot > 0));
-  const int64_t N = q.size(0), H = qp.size(1), dq = qp.size(2), B = slots.numel();
-  check_cache(kc, vc, q, D);
+  TORCH_CHECK(qp.dim() == 3 && rot % 2 == 0 && rot >= 0 && rot <= D && bool(inv_ts) == (rot > 0) && maps >= 1 && qp.size(1) % maps == 0);
+  const int64_t N = q.size(0), H = qp.size(1) / maps, dq = qp.size(2), B = slots.numel();
+  check_cache(kc, vc, q, D * maps);
   const int64_t G = kc.size(2);
-  TORCH_CHECK(vc.size(3) == Dv && B > 0 && N % B == 0 && dq >= D && H % G == 0);
-  rows2d(q, q, N, H * D, "q"); rows2d(k, q, N, G * D, "k"); rows2d(v, q, N, G * Dv, "v");
-  same(qp, q, N * H * dq, "packed q");
+  TORCH_CHECK(vc.size(3) == Dv && B > 0 && N % B == 0 && dq >= D * maps && H % G == 0);
+  rows2d(q, q, N, H * maps * D, "q"); rows2d(k, q, N, G * maps * D, "k"); rows2d(v, q, N, G * Dv, "v");
+  same(qp, q, N * H * maps * dq, "packed q");
   if (kp) same(*kp, q, N * G * dq, "packed k");
   int64_t dvp = Dv;
   if (vp) { dvp = vp->size(vp->dim() - 1); TORCH_CHECK(dvp >= Dv); same(*vp, q, N * G * dvp, "packed v"); }
   if (inv_ts) floats(*inv_ts, rot / 2, "inverse timescales");
+  TORCH_CHECK(bool(wq) == bool(wk) && (!wq || eps >= 0));
+  const bool all = wq && (wq->numel() != D || wk->numel() != D || (H * maps == 1 && G * maps == 1));
+  mt::cattn::PrepArgs a{};
+  a.q = q.data_ptr(); a.k = k.data_ptr(); a.v = v.data_ptr();
+  a.ldq = q.stride(0); a.ldk = k.stride(0); a.ldv = v.stride(0);
+  a.bq = same(bq, q, H * maps * D, "q bias"); a.bk = same(bk, q, G * maps * D, "k bias"); a.bv = same(bv, q, G * Dv, "v bias");
+  a.wq = same(wq, q, all ? H * maps * D : D, "q norm"); a.wk = same(wk, q, all ? G * maps * D : D, "k norm");
+  a.norm = eps < 0 ? mt::cattn::NORM_NONE : !wq ? mt::cattn::NORM_AFTER : all ? mt::cattn::NORM_ALL : mt::cattn::NORM_HEAD;
+  a.H = (int)H; a.G = (int)G; a.D = (int)D; a.Dv = (int)Dv; a.maps = (int)maps;
+  a.pos = longs(pos, N, "positions");
+  a.inv_ts = inv_ts ? inv_ts->data_ptr<float>() : nullptr;
+  a.rot = (int)rot; a.paired = paired;
+  a.eps = (float)eps; a.temp_coef = (float)temp_coef; a.temp_every = (float)temp_every;
+  a.S = (int)(N / B);
+  a.qp = qp.data_ptr(); a.kp = kp ? kp->data_ptr() : nullptr; a.vp = vp ? vp->data_ptr() : nullptr;
+  a.dq = (int)dq; a.dvp = (int)dvp;
+  a.kc = kc.data_ptr(); a.vc = vc.data_ptr(); a.max_len = kc.size(1);
+  a.slots = longs(slots, B, "slots"); a.lengths = longs(lengths, B, "lengths"); a.new_lens = longs(new_lens, B, "new_lens");
   c10::cuda::CUDAGuard guard(q.device());
-  done(mt_qkv_prep(f, q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), (int)H, (int)G, (int)D, (int)Dv,
-                   longs(pos, N, "positions"), inv_ts ? inv_ts->data_ptr<float>() : nullptr, (int)rot, (float)eps, (int)(N / B), qp.data_ptr(), (int)dq,
-                   kp ? kp->data_ptr() : nullptr, vp ? vp->data_ptr() : nullptr, (int)dvp, kc.data_ptr(), vc.data_ptr(), kc.size(1), longs(slots, B, "slots"),
-                   longs(lengths, B, "lengths"), longs(new_lens, B, "new_lens"), N, stream()), "qkv_prep");
+  done(mt_qkv_prep(f, &a, N, stream()), "qkv_prep");
+}
+
+// lam: the four lambda vectors of differential attention
+mt::cattn::DiffArgs diff_args(const std::vector<Tensor>& lam, const Tensor& like, double diff, double eps) {
+  TORCH_CHECK(lam.size() == 4, "differential attention: four lambda vectors");
+  const int64_t D = lam[0].numel();
+  for (const Tensor& t : lam) same(t, like, D, "lambda");
+  return {lam[0].data_ptr(), lam[1].data_ptr(), lam[2].data_ptr(), lam[3].data_ptr(), (int)D, (float)diff, (float)eps};
+}
+
+// gate rows [N, >= H * Dv], or [N, >= H] with one gate per head
+const void* gate_rows(const OptTensor& gate, const Tensor& like, int64_t N, int64_t H, int64_t Dv, bool per_head) {
+  if (!gate) return nullptr;
+  rows2d(*gate, like, N, per_head ? H : H * Dv, "gate");
+  return gate->data_ptr();
 }
 
 // parts of the key range that fill the machine twice over without making a part shorter than four tiles; long ranges are cut up to four times
@@ -172,24 +206,27 @@ int64_t cached_decode_splits(int64_t B, int64_t H, int64_t G, int64_t span) {
 }
 
 void cached_decode(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& slots, const Tensor& lengths, double scale, double cap, int64_t window,
-                   const OptTensor& sinks, const OptTensor& gate, int64_t splits, Tensor& part, Tensor& ml, Tensor& out) {
+                   const OptTensor& sinks, const OptTensor& gate, int64_t splits, Tensor& part, Tensor& ml, Tensor& out, int64_t chunk, bool per_head,
+                   const std::vector<Tensor>& lam, double diff, double eps) {
   TORCH_CHECK(!f32(q) && q.dim() == 3 && q.is_contiguous());
-  const int64_t B = q.size(0), H = q.size(1), D = q.size(2);
+  const int64_t B = q.size(0), H = q.size(1), D = q.size(2), heads = lam.empty() ? H : H / 2;
   check_cache(k, v, q, D);
   const int64_t G = k.size(2), Dv = v.size(3);
-  TORCH_CHECK(H % G == 0 && splits >= 1);
+  TORCH_CHECK(H % G == 0 && splits >= 1 && (lam.empty() || H % 2 == 0));
   floats(part, B * H * splits * Dv, "part"); floats(ml, B * H * splits * 2, "ml");
-  same(out, q, B * H * Dv, "out");
+  same(out, q, B * heads * Dv, "out");
   const void* sk = same(sinks, q, H, "sinks");
-  if (gate) rows2d(*gate, q, B, H * Dv, "gate");
+  const void* gp = gate_rows(gate, q, B, heads, Dv, per_head);
+  mt::cattn::DiffArgs d{};
+  if (!lam.empty()) d = diff_args(lam, q, diff, eps);
   c10::cuda::CUDAGuard guard(q.device());
   done(mt_cached_decode(q.data_ptr(), k.data_ptr(), v.data_ptr(), longs(slots, B, "slots"), longs(lengths, B, "lengths"), k.size(1), (int)B, (int)H, (int)G,
-                        (int)D, (int)Dv, (float)scale, (float)cap, (int)window, sk, gate ? gate->data_ptr() : nullptr, gate ? gate->stride(0) : 0, (int)splits,
-                        part.data_ptr<float>(), ml.data_ptr<float>(), out.data_ptr(), stream()), "cached_decode", 2);
+                        (int)D, (int)Dv, (float)scale, (float)cap, (int)window, (int)chunk, sk, gp, gate ? gate->stride(0) : 0, per_head,
+                        lam.empty() ? nullptr : &d, (int)splits, part.data_ptr<float>(), ml.data_ptr<float>(), out.data_ptr(), stream()), "cached_decode", 2);
 }
 
 void cached_attention(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& slots, const Tensor& lengths, int64_t S, double scale, double cap,
-                      int64_t window, const OptTensor& sinks, Tensor& out) {
+                      int64_t window, const OptTensor& sinks, Tensor& out, int64_t chunk) {
   const bool f = f32(q);
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous());
   const int64_t B = slots.numel(), H = q.size(1), D = q.size(2);
@@ -200,18 +237,32 @@ void cached_attention(const Tensor& q, const Tensor& k, const Tensor& v, const T
   const void* sk = same(sinks, q, H, "sinks");
   c10::cuda::CUDAGuard guard(q.device());
   done(mt_cached_attention(f, q.data_ptr(), k.data_ptr(), v.data_ptr(), k.size(1), longs(slots, B, "slots"), longs(lengths, B, "lengths"), (int)B, (int)S, (int)H,
-                           (int)G, (int)D, (int)Dv, (float)scale, (float)cap, (int)window, sk, out.data_ptr(), stream()), "cached_attention");
+                           (int)G, (int)D, (int)Dv, (float)scale, (float)cap, (int)window, (int)chunk, sk, out.data_ptr(), stream()), "cached_attention");
 }
 
-// o [N, H, >= dv], g [N, >= H * dv] -> out [N, H * dv]
-void head_gate(const Tensor& o, const Tensor& g, int64_t dv, Tensor& out) {
+// o [N, H, >= dv], g [N, >= H * dv] (or [N, >= H]) -> out [N, H * dv]
+void head_gate(const Tensor& o, const Tensor& g, int64_t dv, Tensor& out, bool per_head) {
   const bool f = f32(o);
   TORCH_CHECK(o.dim() == 3 && o.is_contiguous() && o.size(2) >= dv);
   const int64_t N = o.size(0), H = o.size(1);
-  rows2d(g, o, N, H * dv, "gate");
+  gate_rows(g, o, N, H, dv, per_head);
   same(out, o, N * H * dv, "out");
   c10::cuda::CUDAGuard guard(o.device());
-  done(mt_head_gate(f, o.data_ptr(), (int)o.size(2), g.data_ptr(), g.stride(0), N, (int)(H * dv), (int)dv, out.data_ptr(), mt_num_sms(), stream()), "head_gate");
+  done(mt_head_gate(f, o.data_ptr(), (int)o.size(2), g.data_ptr(), g.stride(0), N, (int)(H * dv), (int)dv, per_head, out.data_ptr(), mt_num_sms(), stream()),
+       "head_gate");
+}
+
+// o [N, 2 H, >= dv] (two maps per head) -> out [N, H * dv]
+void diff_combine(const Tensor& o, const std::vector<Tensor>& lam, double diff, double eps, const OptTensor& gate, int64_t dv, Tensor& out, bool per_head) {
+  const bool f = f32(o);
+  TORCH_CHECK(o.dim() == 3 && o.is_contiguous() && o.size(2) >= dv && o.size(1) % 2 == 0);
+  const int64_t N = o.size(0), H = o.size(1) / 2;
+  const void* gp = gate_rows(gate, o, N, H, dv, per_head);
+  same(out, o, N * H * dv, "out");
+  const auto d = diff_args(lam, o, diff, eps);
+  c10::cuda::CUDAGuard guard(o.device());
+  done(mt_diff_combine(f, o.data_ptr(), (int)o.size(2), &d, N, (int)H, (int)dv, gp, gate ? gate->stride(0) : 0, per_head, out.data_ptr(), mt_num_sms(),
+                       stream()), "diff_combine");
 }
 
 void check_plan(const Tensor& sizes, const Tensor& offs, const Tensor& row_pair, int64_t E) {
@@ -258,11 +309,19 @@ void register_hybrid(pybind11::module_& m) {
   m.def("stream_mix", &stream_mix);
   m.def("ssm_conv", &ssm_conv);
   m.def("ssm_scan", &ssm_scan);
-  m.def("qkv_prep", &qkv_prep);
+  using pybind11::arg;
+  const auto none = pybind11::none();
+  m.def("qkv_prep", &qkv_prep, arg("q"), arg("k"), arg("v"), arg("D"), arg("Dv"), arg("pos"), arg("inv_ts"), arg("rot"), arg("eps"), arg("qp"), arg("kp"),
+        arg("vp"), arg("kc"), arg("vc"), arg("slots"), arg("lengths"), arg("new_lens"), arg("bq") = none, arg("bk") = none, arg("bv") = none, arg("wq") = none,
+        arg("wk") = none, arg("paired") = false, arg("maps") = 1, arg("temp_coef") = 0.0, arg("temp_every") = 0.0);
   m.def("cached_decode_splits", &cached_decode_splits);
-  m.def("cached_decode", &cached_decode);
-  m.def("cached_attention", &cached_attention);
-  m.def("head_gate", &head_gate);
+  m.def("cached_decode", &cached_decode, arg("q"), arg("k"), arg("v"), arg("slots"), arg("lengths"), arg("scale"), arg("cap"), arg("window"), arg("sinks"),
+        arg("gate"), arg("splits"), arg("part"), arg("ml"), arg("out"), arg("chunk") = 0, arg("per_head") = false, arg("lam") = std::vector<Tensor>{},
+        arg("diff") = 0.0, arg("eps") = 0.0);
+  m.def("cached_attention", &cached_attention, arg("q"), arg("k"), arg("v"), arg("slots"), arg("lengths"), arg("S"), arg("scale"), arg("cap"), arg("window"),
+        arg("sinks"), arg("out"), arg("chunk") = 0);
+  m.def("head_gate", &head_gate, arg("o"), arg("g"), arg("dv"), arg("out"), arg("per_head") = false);
+  m.def("diff_combine", &diff_combine);
   m.def("expert_up", &expert_up);
   m.def("expert_down", &expert_down);
   m.def("expert_act", &expert_act);

@@ -8,6 +8,9 @@
 extern "C" {
 int mt_residual_norm(float* x, const void* branch, const void* w_post, float mult, const void* w_next, void* y, int f32, long rows, int D, float eps_post,
                      float eps_next, float offset, cudaStream_t st);
+int mt_residual_join(float* x, const void* a, const void* a_bias, const void* a_norm, float a_factor, const void* b, const void* b_bias, const void* b_norm,
+                     float b_factor, const void* lanes, const void* w_next, void* y, int f32, long rows, int D, float eps, cudaStream_t st);
+int mt_token_gate(const void* g, const void* table, const int64_t* tokens, void* out, int f32, long N, int dim, long vocab, int sms, cudaStream_t st);
 int mt_act_fwd(const void* x, void* y, int f32, long n, int code, int sms, cudaStream_t st);
 int mt_delta_decode(int f32, const void* x, long ldx, const void* ba, long ldb, const void* conv_w, int taps, const void* A_log, const void* dt_bias,
                     const void* norm, float eps, int hk, int hv, int dk, int dv, float* conv, float* rec, const int64_t* slots, const int64_t* lengths,
@@ -28,7 +31,23 @@ int mt_gla_chunks(const void* x, long ldx, const float* log_alpha, int H, int dk
                   const int64_t* lengths, const int64_t* new_lens, void* aa, void* qkg, float* ends, void* o, int B, cudaStream_t st);
 int mt_gla_decay(int f32, const void* lo, long ldx, const void* w, const void* bias, int rank, float inv_tau, float* out, long N, int C, cudaStream_t st);
 int mt_gated_head_norm(int f32, const void* o, const void* x, long ldx, long rows, int H, int dv, int r, long zoff, long zstride, const void* w, float eps,
-                       void* out, cudaStream_t st);
+                       int sig, void* out, cudaStream_t st);
+int mt_retention_decode(int f32, const void* x, long ldx, const float* log_decay, const float* inv_ts, int rot, float eps, int H, int dk, int dv, float* rec,
+                        const int64_t* slots, const int64_t* lengths, void* out, int B, cudaStream_t st);
+int mt_retention_scan(int f32, const void* x, long ldx, const float* log_decay, const float* inv_ts, int rot, int H, int dk, int dv, int S, float* rec,
+                      const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* o, int B, cudaStream_t st);
+int mt_retention_chunks(const void* x, long ldx, const float* log_decay, const float* inv_ts, int rot, int H, int dk, int dv, int S, int t_lo, int t_hi,
+                        float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* aa, void* qkg, float* ends, void* o, int B,
+                        cudaStream_t st);
+int mt_channel_delta_decode(int f32, const void* x, long ldx, const void* beta, long ldb, const void* conv_w, int taps, const float* da, const void* A_log,
+                            const void* dt_bias, const void* z, long ldz, const void* norm, float eps, int hk, int hv, int dk, int dv, float* conv, float* rec,
+                            const int64_t* slots, const int64_t* lengths, void* out, int B, cudaStream_t st);
+int mt_channel_delta_scan(int f32, const void* mixed, const void* beta, long ldb, const float* da, const void* A_log, const void* dt_bias, int hk, int hv,
+                          int dk, int dv, int S, float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* o, int B,
+                          cudaStream_t st);
+int mt_channel_delta_chunks(const void* mixed, long ldx, const void* beta, long ldb, const float* da, const void* A_log, const void* dt_bias, int hk, int hv,
+                            int dk, int dv, int S, int t_lo, int t_hi, float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens,
+                            void* tp, void* qkg, float* betas, float* ends, void* o, int B, cudaStream_t st);
 int mt_mla_prep(int f32, const void* qa, long ldq, const void* qw, int Q, const void* kva, long ldk, const void* kw, int R, int dr, float eps,
                 const int64_t* pos, const float* inv_ts, int interleaved, int S, void* cq, void* lat, void* kr, void* cache_lat, void* cache_kr, long max_len,
                 const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, long N, cudaStream_t st);
@@ -94,6 +113,39 @@ void residual_norm(Tensor& x, const OptTensor& branch, const OptTensor& w_post, 
   done(mt_residual_norm(x.data_ptr<float>(), branch ? branch->data_ptr() : nullptr, w_post ? w_post->data_ptr() : nullptr, (float)mult,
                         w_next ? w_next->data_ptr() : nullptr, y ? y->data_ptr() : nullptr, f, x.size(0), (int)x.size(1), (float)eps_post, (float)eps_next,
                         (float)offset, stream()), "residual_norm");
+}
+
+const void* lane_vector(const OptTensor& t, const Tensor& like, int64_t D, const char* what) {
+  if (!t) return nullptr;
+  same(*t, like, D, what);
+  return t->data_ptr();
+}
+
+// x [rows, D] fp32 += lanes * (a + b), each branch [norm of](out + bias) * factor; y: rms(x) * w_next, x itself without w_next, or None
+void residual_join(Tensor& x, const Tensor& a, const OptTensor& a_bias, const OptTensor& a_norm, double a_factor, const OptTensor& b, const OptTensor& b_bias,
+                   const OptTensor& b_norm, double b_factor, const OptTensor& lanes, const OptTensor& w_next, const OptTensor& y, double eps) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.is_contiguous() && x.scalar_type() == torch::kFloat32 && x.size(1) <= 8192, "residual_join: x fp32 [rows, <= 8192]");
+  const bool f = f32(a);
+  const int64_t D = x.size(1);
+  TORCH_CHECK(y || !w_next, "residual_join: a norm without a result");
+  same(a, a, x.numel(), "branch");
+  if (b) same(*b, a, x.numel(), "second branch");
+  if (y) same(*y, a, x.numel(), "y");
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_residual_join(x.data_ptr<float>(), a.data_ptr(), lane_vector(a_bias, a, D, "bias"), lane_vector(a_norm, a, D, "norm"), (float)a_factor,
+                        b ? b->data_ptr() : nullptr, lane_vector(b_bias, a, D, "bias"), lane_vector(b_norm, a, D, "norm"), (float)b_factor,
+                        lane_vector(lanes, a, D, "lane factors"), lane_vector(w_next, a, D, "next norm"), y ? y->data_ptr() : nullptr, f, x.size(0), (int)D,
+                        (float)eps, stream()), "residual_join");
+}
+
+// g [N, dim], table [V, dim], tokens [N] -> out [N, dim]
+void token_gate(const Tensor& g, const Tensor& table, const Tensor& tokens, Tensor& out) {
+  const bool f = f32(g);
+  TORCH_CHECK(g.dim() == 2 && table.dim() == 2 && table.size(1) == g.size(1) && table.size(0) > 0);
+  same(g, g, g.numel(), "g"); same(table, g, table.numel(), "table"); same(out, g, g.numel(), "out");
+  c10::cuda::CUDAGuard guard(g.device());
+  done(mt_token_gate(g.data_ptr(), table.data_ptr(), longs(tokens, g.size(0), "tokens"), out.data_ptr(), f, g.size(0), (int)g.size(1), table.size(0),
+                     mt_num_sms(), stream()), "token_gate");
 }
 
 void act_fwd(const Tensor& x, Tensor& y, int64_t code) {
@@ -243,15 +295,129 @@ void gla_chunks(const Tensor& x, const Tensor& log_alpha, int64_t H, int64_t dk,
                        nl, aa.data_ptr(), qkg.data_ptr(), ends.data_ptr<float>(), o.data_ptr(), (int)B, stream()), "gla_chunks", 2);
 }
 
-void gated_head_norm(const Tensor& o, const Tensor& x, int64_t H, int64_t dv, int64_t r, int64_t zoff, int64_t zstride, const Tensor& w, double eps,
-                     Tensor& out) {
+// out = rms(o) [* w] * silu(z), or sigmoid(z) with `sig`; z at column zoff + (h / r) * zstride + (h % r) * dv of x
+void gated_head_norm(const Tensor& o, const Tensor& x, int64_t H, int64_t dv, int64_t r, int64_t zoff, int64_t zstride, const OptTensor& w, double eps,
+                     Tensor& out, bool sig) {
   const bool f = f32(o);
   const int64_t N = x.size(0);
   rows2d(x, o, N, zoff + (H / r - 1) * zstride + r * dv, "packed projection");
-  same(o, o, N * H * dv, "o"); same(w, o, dv, "norm"); same(out, o, N * H * dv, "out");
+  same(o, o, N * H * dv, "o"); same(out, o, N * H * dv, "out");
+  if (w) same(*w, o, dv, "norm");
   c10::cuda::CUDAGuard guard(o.device());
-  done(mt_gated_head_norm(f, o.data_ptr(), x.data_ptr(), x.stride(0), N * H, (int)H, (int)dv, (int)r, zoff, zstride, w.data_ptr(), (float)eps,
-                          out.data_ptr(), stream()), "gated_head_norm");
+  done(mt_gated_head_norm(f, o.data_ptr(), x.data_ptr(), x.stride(0), N * H, (int)H, (int)dv, (int)r, zoff, zstride, w ? w->data_ptr() : nullptr, (float)eps,
+                          sig, out.data_ptr(), stream()), "gated_head_norm");
+}
+
+void check_fp32(const Tensor& t, int64_t numel, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == torch::kFloat32 && t.is_contiguous() && t.numel() == numel, what, ": contiguous fp32 tensor of ", numel,
+              " elements expected");
+}
+const float* turns(const OptTensor& inv_ts, int64_t rot, int64_t dk) {
+  TORCH_CHECK(rot >= 0 && rot % 2 == 0 && rot <= dk && bool(inv_ts) == (rot > 0), "retention: bad rotation");
+  if (!inv_ts) return nullptr;
+  check_fp32(*inv_ts, rot / 2, "inverse timescales");
+  return inv_ts->data_ptr<float>();
+}
+
+// x rows: q H*dk | k H*dk | v H*dv | gate H*dv -> out [B, H * dv], normalised and gated
+void retention_decode(const Tensor& x, const Tensor& log_decay, const OptTensor& inv_ts, int64_t rot, double eps, int64_t H, int64_t dk, int64_t dv, Tensor& rec,
+                      const Tensor& slots, const Tensor& lengths, Tensor& out) {
+  const bool f = f32(x);
+  const int64_t B = x.size(0);
+  rows2d(x, x, B, 2 * H * (dk + dv), "packed projection");
+  check_fp32(log_decay, H, "log decay");
+  same(out, x, B * H * dv, "out");
+  float* rp = state(rec, {H, dk, dv}, "rec");
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_retention_decode(f, x.data_ptr(), x.stride(0), log_decay.data_ptr<float>(), turns(inv_ts, rot, dk), (int)rot, (float)eps, (int)H, (int)dk, (int)dv,
+                           rp, longs(slots, B, "slots"), longs(lengths, B, "lengths"), out.data_ptr(), (int)B, stream()), "retention_decode");
+}
+
+// token scan, any widths up to 256: x rows as above -> o [B*S, H * dv]
+void retention_scan(const Tensor& x, const Tensor& log_decay, const OptTensor& inv_ts, int64_t rot, int64_t H, int64_t dk, int64_t dv, int64_t S, Tensor& rec,
+                    const Tensor& slots, const Tensor& lengths, const OptTensor& new_lens, Tensor& o) {
+  const bool f = f32(x);
+  const int64_t B = slots.numel();
+  rows2d(x, x, B * S, 2 * H * (dk + dv), "packed projection");
+  check_fp32(log_decay, H, "log decay");
+  same(o, x, B * S * H * dv, "o");
+  float* rp = state(rec, {H, dk, dv}, "rec");
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_retention_scan(f, x.data_ptr(), x.stride(0), log_decay.data_ptr<float>(), turns(inv_ts, rot, dk), (int)rot, (int)H, (int)dk, (int)dv, (int)S, rp,
+                         longs(slots, B, "slots"), longs(lengths, B, "lengths"), longs(new_lens, B, "new_lens"), o.data_ptr(), (int)B, stream()),
+       "retention_scan");
+}
+
+// the chunked form of retention_scan (bf16)
+void retention_chunks(const Tensor& x, const Tensor& log_decay, const OptTensor& inv_ts, int64_t rot, int64_t H, int64_t dk, int64_t dv, int64_t S, Tensor& rec,
+                      const Tensor& slots, const Tensor& lengths, const OptTensor& new_lens, Tensor& o) {
+  TORCH_CHECK(!f32(x) && chunk_supported(dk, dv), "retention_chunks: bf16 and head widths of 16 .. 128 in steps of 16");
+  const int64_t B = slots.numel();
+  rows2d(x, x, B * S, 2 * H * (dk + dv), "packed projection");
+  TORCH_CHECK((reinterpret_cast<uintptr_t>(x.data_ptr()) % 16) == 0 && x.stride(0) % 8 == 0);
+  check_fp32(log_decay, H, "log decay");
+  same(o, x, B * S * H * dv, "o");
+  float* rp = state(rec, {H, dk, dv}, "rec");
+  const int64_t *sl = longs(slots, B, "slots"), *le = longs(lengths, B, "lengths"), *nl = longs(new_lens, B, "new_lens");
+  const float* iv = turns(inv_ts, rot, dk);
+  c10::cuda::CUDAGuard guard(x.device());
+  const int64_t seg = chunk_segment(B, H, S, 2 * 64 * 2 + 4 * dk * 2), tiles = B * (seg / 64) * H;
+  auto aa = torch::empty({tiles * 2 * 64 * 64}, x.options()), qkg = torch::empty({tiles * 4 * 64 * dk}, x.options());
+  auto ends = torch::empty({tiles * dk}, torch::dtype(torch::kFloat32).device(x.device()));
+  for (int64_t t = 0; t < S; t += seg)
+    done(mt_retention_chunks(x.data_ptr(), x.stride(0), log_decay.data_ptr<float>(), iv, (int)rot, (int)H, (int)dk, (int)dv, (int)S, (int)t,
+                             (int)std::min(S, t + seg), rp, sl, le, nl, aa.data_ptr(), qkg.data_ptr(), ends.data_ptr<float>(), o.data_ptr(), (int)B, stream()),
+         "retention_chunks", 2);
+}
+
+// x rows: q hk*dk | k hk*dk | v hv*dv; beta rows [B, >= hv]; da fp32 [B, hv*dk]; z rows [B, >= hv*dv] -> out [B, hv * dv], normalised and gated
+void channel_delta_decode(const Tensor& x, const Tensor& beta, const Tensor& conv_w, const Tensor& da, const Tensor& A_log, const Tensor& dt_bias,
+                          const Tensor& z, const Tensor& norm, double eps, int64_t hk, int64_t hv, int64_t dk, int64_t dv, Tensor& conv, Tensor& rec,
+                          const Tensor& slots, const Tensor& lengths, Tensor& out) {
+  const bool f = f32(x);
+  const int64_t B = x.size(0), cd = 2 * hk * dk + hv * dv;
+  TORCH_CHECK(hk > 0 && hv % hk == 0 && conv_w.dim() == 2 && conv_w.size(0) >= 1, "channel-wise gated delta: bad sizes");
+  const int64_t taps = conv_w.size(0);
+  rows2d(x, x, B, cd, "packed projection"); rows2d(beta, x, B, hv, "beta"); rows2d(z, x, B, hv * dv, "gate");
+  same(conv_w, x, taps * cd, "convolution"); same(A_log, x, hv, "A_log"); same(dt_bias, x, hv * dk, "dt_bias"); same(norm, x, dv, "norm");
+  same(out, x, B * hv * dv, "out");
+  check_fp32(da, B * hv * dk, "decay");
+  float* cp = state(conv, {taps - 1, cd}, "conv");
+  float* rp = state(rec, {hv, dk, dv}, "rec");
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_channel_delta_decode(f, x.data_ptr(), x.stride(0), beta.data_ptr(), beta.stride(0), conv_w.data_ptr(), (int)taps, da.data_ptr<float>(),
+                               A_log.data_ptr(), dt_bias.data_ptr(), z.data_ptr(), z.stride(0), norm.data_ptr(), (float)eps, (int)hk, (int)hv, (int)dk, (int)dv,
+                               cp, rp, longs(slots, B, "slots"), longs(lengths, B, "lengths"), out.data_ptr(), (int)B, stream()), "channel_delta_decode");
+}
+
+// mixed [B*S, 2 hk dk + hv dv] after the convolution -> o [B*S, hv * dv]; `chunked` (bf16, head widths of 16 .. 128 in steps of 16): in chunks of 64 tokens
+void channel_delta_scan(const Tensor& mixed, const Tensor& beta, const Tensor& da, const Tensor& A_log, const Tensor& dt_bias, int64_t hk, int64_t hv,
+                        int64_t dk, int64_t dv, int64_t S, Tensor& rec, const Tensor& slots, const Tensor& lengths, const OptTensor& new_lens, Tensor& o,
+                        bool chunked) {
+  const bool f = f32(mixed);
+  const int64_t B = slots.numel(), cd = 2 * hk * dk + hv * dv;
+  TORCH_CHECK(hk > 0 && hv % hk == 0, "channel-wise gated delta: bad sizes");
+  same(mixed, mixed, B * S * cd, "mixed");
+  rows2d(beta, mixed, B * S, hv, "beta");
+  same(A_log, mixed, hv, "A_log"); same(dt_bias, mixed, hv * dk, "dt_bias"); same(o, mixed, B * S * hv * dv, "o");
+  check_fp32(da, B * S * hv * dk, "decay");
+  float* rp = state(rec, {hv, dk, dv}, "rec");
+  const int64_t *sl = longs(slots, B, "slots"), *le = longs(lengths, B, "lengths"), *nl = longs(new_lens, B, "new_lens");
+  c10::cuda::CUDAGuard guard(mixed.device());
+  if (!chunked) {
+    done(mt_channel_delta_scan(f, mixed.data_ptr(), beta.data_ptr(), beta.stride(0), da.data_ptr<float>(), A_log.data_ptr(), dt_bias.data_ptr(), (int)hk, (int)hv,
+                               (int)dk, (int)dv, (int)S, rp, sl, le, nl, o.data_ptr(), (int)B, stream()), "channel_delta_scan");
+    return;
+  }
+  TORCH_CHECK(!f && chunk_supported(dk, dv) && cd % 8 == 0 && (reinterpret_cast<uintptr_t>(mixed.data_ptr()) % 16) == 0, "channel_delta_scan: not chunkable");
+  const int64_t seg = chunk_segment(B, hv, S, 4 * 64 * 2 + 6 * dk * 2), tiles = B * (seg / 64) * hv;
+  auto tp = torch::empty({tiles * 4 * 64 * 64}, mixed.options()), qkg = torch::empty({tiles * 6 * 64 * dk}, mixed.options());
+  auto fo = torch::dtype(torch::kFloat32).device(mixed.device());
+  auto betas = torch::empty({tiles * 64}, fo), ends = torch::empty({tiles * dk}, fo);
+  for (int64_t t = 0; t < S; t += seg)
+    done(mt_channel_delta_chunks(mixed.data_ptr(), cd, beta.data_ptr(), beta.stride(0), da.data_ptr<float>(), A_log.data_ptr(), dt_bias.data_ptr(), (int)hk,
+                                 (int)hv, (int)dk, (int)dv, (int)S, (int)t, (int)std::min(S, t + seg), rp, sl, le, nl, tp.data_ptr(), qkg.data_ptr(),
+                                 betas.data_ptr<float>(), ends.data_ptr<float>(), o.data_ptr(), (int)B, stream()), "channel_delta_chunks", 2);
 }
 
 void mla_prep(const OptTensor& qa, const OptTensor& qw, const Tensor& kva, const Tensor& kw, double eps, const Tensor& pos, const Tensor& inv_ts,
@@ -334,6 +500,8 @@ void mla_value_up(const Tensor& part, const Tensor& ml, const Tensor& w, int64_t
 
 void register_serving(pybind11::module_& m) {
   m.def("residual_norm", &residual_norm);
+  m.def("residual_join", &residual_join);
+  m.def("token_gate", &token_gate);
   m.def("act_fwd", &act_fwd);
   m.def("delta_decode", &delta_decode);
   m.def("delta_conv", &delta_conv);
@@ -344,7 +512,14 @@ void register_serving(pybind11::module_& m) {
   m.def("chunk_supported", &chunk_supported);
   m.def("delta_chunks", &delta_chunks);
   m.def("gla_chunks", &gla_chunks);
-  m.def("gated_head_norm", &gated_head_norm);
+  using pybind11::arg;
+  m.def("gated_head_norm", &gated_head_norm, arg("o"), arg("x"), arg("H"), arg("dv"), arg("r"), arg("zoff"), arg("zstride"), arg("w"), arg("eps"), arg("out"),
+        arg("sig") = false);
+  m.def("retention_decode", &retention_decode);
+  m.def("retention_scan", &retention_scan);
+  m.def("retention_chunks", &retention_chunks);
+  m.def("channel_delta_decode", &channel_delta_decode);
+  m.def("channel_delta_scan", &channel_delta_scan);
   m.def("mla_prep", &mla_prep);
   m.def("mla_pack", &mla_pack);
   m.def("mla_absorb", &mla_absorb);

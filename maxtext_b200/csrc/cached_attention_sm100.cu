@@ -1,7 +1,9 @@
 // Softmax attention over a slot-indexed key/value cache at inference: [slots, max_len, G, D] keys, [slots, max_len, G, Dv] values, any head
-// widths, with soft-capped scores, a per-head sink in the denominator, a sliding window and a sigmoid output gate.
+// widths, with soft-capped scores, a per-head sink in the denominator, a sliding window or chunks, and a sigmoid output gate per lane or head.
 //
-//   qkv_prep   projections -> rotated (first `rot` lanes, halves paired) and RMS-normalised q and k, cache rows, operands of the flash kernel
+//   qkv_prep   projections (plus bias) -> RMS-normalised and rotated q and k (first `rot` lanes; halves or neighbours paired; the norm after the
+//              rotation without a weight, or before it with one, per head or over the whole projection), a query temperature, cache rows,
+//              operands of the flash kernel
 //   decode     one new token per sequence: keys split over CTAs and, inside a CTA, over four warps that each stream their own 16-key tiles
 //              through a cp.async ring; up to 16 query heads of a key head sit in the M position of mma.sync m16n8k16; softmax in registers,
 //              weights as (high, low) bf16 pairs. No barrier between tiles. tcgen05 has no use here: a step is bound by reading the cache
@@ -9,6 +11,10 @@
 //   merge      joins the splits, adds the sink, applies the gate
 //   plain      fp32 arithmetic on CUDA cores over the cache, any widths up to 512 and any number of new tokens
 //   head_gate  gate of the prompt path, drops the flash kernel's width padding
+//   diff       differential attention: a head's two maps share the values. The cache holds the head's two keys side by side as one key, and each
+//              map's query is zero over the other map's half, so that the kernels above see two query heads of ordinary grouped attention;
+//              here the second result is subtracted from the first, times lambda, normalised per head, scaled and gated
+#include "cached_attention.h"
 #include "serving_common.cuh"
 #include "warp_mma.cuh"
 
@@ -21,46 +27,73 @@ __device__ __forceinline__ float capped(float s, float cap, float two_over_cap) 
 }
 
 // ------------------------------------------------------------------------------------------------ prep
-// One CTA per token; a warp per head. Lanes hold VEC neighbouring elements, ITER times.
+// One CTA per token; a warp per head and map. Lanes hold VEC neighbouring elements, ITER times.
 template <typename T, int VEC, int ITER>
 __global__ void __launch_bounds__(128)
-qkv_prep_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, long ldk, const T* __restrict__ v, long ldv, int H, int G, int D, int Dv,
-                const int64_t* __restrict__ pos, const float* __restrict__ inv_ts, int rot, float eps, int S, T* __restrict__ qp, int dq, T* __restrict__ kp,
-                T* __restrict__ vp, int dvp, T* __restrict__ kc, T* __restrict__ vc, long max_len, const int64_t* __restrict__ slots,
-                const int64_t* __restrict__ lengths, const int64_t* __restrict__ new_lens) {
+qkv_prep_kernel(const PrepArgs a) {
   extern __shared__ float2 cs[];                            // (cos, sin) of the rot / 2 angles
+  __shared__ float red[2][4];
   const long n = blockIdx.x;
-  const int b = (int)(n / S), s = (int)(n % S), half = rot / 2;
-  const float p = (float)pos[n];
+  const int b = (int)(n / a.S), s = (int)(n % a.S), half = a.rot / 2, D = a.D, HM = a.H * a.maps, GM = a.G * a.maps;
+  const float p = (float)a.pos[n];
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float sn, c;
-    sincosf(p * inv_ts[i], &sn, &c);
+    sincosf(p * a.inv_ts[i], &sn, &c);
     cs[i] = make_float2(c, sn);
   }
-  __syncthreads();
-  const long at = lengths[b] + s;
-  const bool keep = at < max_len && s < (new_lens ? new_lens[b] : (int64_t)S);
-  const long row = slots[b] * max_len + at;
+  const float warm = a.temp_every > 0.f ? 1.f + a.temp_coef * logf(floorf((p + 1.f) / a.temp_every) + 1.f) : 1.f;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int h = warp; h < H + G; h += 4) {
-    const bool key = h >= H;
-    const T* src = key ? k + n * ldk + (long)(h - H) * D : q + n * ldq + (long)h * D;
-    float x[ITER][VEC], ss = 0.f;
+  // raw elements of a head (with its bias), at lane offset e0
+  auto raw = [&](bool key, int head, int e0, float (&x)[VEC]) {
+    load_vec<VEC>(static_cast<const T*>(key ? a.k : a.q) + n * (key ? a.ldk : a.ldq) + (long)head * D + e0, x);
+    const T* bias = static_cast<const T*>(key ? a.bk : a.bq);
+    if (bias) {
+      float y[VEC];
+      load_vec<VEC>(bias + (long)head * D + e0, y);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] += y[e];
+    }
+  };
+  float rstd_q = 1.f, rstd_k = 1.f;
+  if (a.norm == NORM_ALL) {
+    float ss[2] = {0.f, 0.f};
+    for (int h = warp; h < HM + GM; h += 4) {
+      const bool key = h >= HM;
+      float t = 0.f;
+#pragma unroll
+      for (int it = 0; it < ITER; ++it) {
+        const int e0 = (it * 32 + lane) * VEC;
+        if (e0 < D) {
+          float x[VEC];
+          raw(key, key ? h - HM : h, e0, x);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) t += x[e] * x[e];
+        }
+      }
+      if (key) ss[1] += t; else ss[0] += t;
+    }
+    ss[0] = warp_add(ss[0]);
+    ss[1] = warp_add(ss[1]);
+    if (lane == 0) { red[0][warp] = ss[0]; red[1][warp] = ss[1]; }
+  }
+  __syncthreads();
+  if (a.norm == NORM_ALL) {
+    rstd_q = rsqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)(HM * D) + a.eps);
+    rstd_k = rsqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)(GM * D) + a.eps);
+  }
+  const long at = a.lengths[b] + s;
+  const bool keep = at < a.max_len && s < (a.new_lens ? a.new_lens[b] : (int64_t)a.S);
+  const long row = a.slots[b] * a.max_len + at;
+  for (int h = warp; h < HM + GM; h += 4) {
+    const bool key = h >= HM;
+    const int head = key ? h - HM : h;
+    const T* w = a.norm >= NORM_HEAD ? static_cast<const T*>(key ? a.wk : a.wq) + (a.norm == NORM_ALL ? (long)head * D : 0) : nullptr;
+    float x[ITER][VEC], ss = 0.f, r = key ? rstd_k : rstd_q;
 #pragma unroll
     for (int it = 0; it < ITER; ++it) {
       const int e0 = (it * 32 + lane) * VEC;
       if (e0 < D) {
-        load_vec<VEC>(src + e0, x[it]);
-        if (e0 < rot) {
-          const bool low = e0 < half;
-          float y[VEC];
-          load_vec<VEC>(src + (low ? e0 + half : e0 - half), y);
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) {
-            const float2 a = cs[(low ? e0 : e0 - half) + e];
-            x[it][e] = x[it][e] * a.x + (low ? -y[e] : y[e]) * a.y;
-          }
-        }
+        raw(key, head, e0, x[it]);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) ss += x[it][e] * x[it][e];
       } else {
@@ -68,32 +101,87 @@ qkv_prep_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, long
         for (int e = 0; e < VEC; ++e) x[it][e] = 0.f;
       }
     }
-    if (eps >= 0.f) {
-      const float r = rsqrtf(warp_add(ss) / (float)D + eps);
+    if (a.norm == NORM_HEAD || a.norm == NORM_AFTER) r = rsqrtf(warp_add(ss) / (float)D + a.eps);   // a rotation leaves the norm as it is
+    // the factor of an element in front of the rotation
+    auto scaled = [&](int e0, float (&y)[VEC]) {
+      float g[VEC];
+      if (w) load_vec<VEC>(w + e0, g);
 #pragma unroll
-      for (int it = 0; it < ITER; ++it)
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) x[it][e] *= r;
-    }
-    T* dst = key ? (kp ? kp + (n * G + h - H) * dq : nullptr) : qp + (n * H + h) * dq;
-    T* cache = key && keep ? kc + (row * G + h - H) * D : nullptr;
+      for (int e = 0; e < VEC; ++e) y[e] *= w ? r * g[e] : r;
+    };
 #pragma unroll
     for (int it = 0; it < ITER; ++it) {
       const int e0 = (it * 32 + lane) * VEC;
-      if (dst && e0 < dq) store_vec<VEC>(dst + e0, x[it]);
-      if (cache && e0 < D) store_vec<VEC>(cache + e0, x[it]);
+      if (e0 >= D) continue;
+      scaled(e0, x[it]);
+      if (e0 < a.rot) {
+        if (!a.paired) {
+          const bool low = e0 < half;
+          const int o0 = low ? e0 + half : e0 - half;
+          float y[VEC];
+          raw(key, head, o0, y);
+          scaled(o0, y);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            const float2 c = cs[(low ? e0 : e0 - half) + e];
+            x[it][e] = x[it][e] * c.x + (low ? -y[e] : y[e]) * c.y;
+          }
+        } else if constexpr (VEC > 1) {
+#pragma unroll
+          for (int e = 0; e < VEC; e += 2) {
+            const float2 c = cs[(e0 + e) / 2];
+            const float u = x[it][e], v = x[it][e + 1];
+            x[it][e] = u * c.x - v * c.y;
+            x[it][e + 1] = v * c.x + u * c.y;
+          }
+        } else {
+          float y[VEC];
+          raw(key, head, e0 ^ 1, y);
+          scaled(e0 ^ 1, y);
+          const float2 c = cs[e0 / 2];
+          x[it][0] = x[it][0] * c.x + (e0 & 1 ? y[0] : -y[0]) * c.y;
+        }
+      }
+      if (!key) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[it][e] *= warm;
+      }
+    }
+    const int m = head % a.maps;                            // this map's lanes of the head
+    T* dst = key ? (a.kp ? static_cast<T*>(a.kp) + (n * a.G + head / a.maps) * a.dq : nullptr) : static_cast<T*>(a.qp) + (n * HM + head) * a.dq;
+    T* cache = key && keep ? static_cast<T*>(a.kc) + (row * GM + head) * D : nullptr;
+#pragma unroll
+    for (int it = 0; it < ITER; ++it) {
+      const int e0 = (it * 32 + lane) * VEC;
+      if (e0 < D) {
+        if (dst) store_vec<VEC>(dst + m * D + e0, x[it]);
+        if (cache) store_vec<VEC>(cache + e0, x[it]);
+      }
+    }
+    // zeros: a query's other lanes, and what pads a key to the operand's width
+    if (dst && (key ? m == a.maps - 1 && a.dq > a.maps * D : a.dq > D)) {
+      const float zero[VEC] = {};
+      for (int e0 = lane * VEC; e0 < a.dq; e0 += 32 * VEC)
+        if (e0 >= (m + 1) * D || (!key && e0 < m * D)) store_vec<VEC>(dst + e0, zero);
     }
   }
-  if (keep || vp) {
-    for (int i = threadIdx.x * VEC; i < G * Dv; i += blockDim.x * VEC) {
+  if (keep || a.vp) {
+    T *vc = static_cast<T*>(a.vc), *vp = static_cast<T*>(a.vp);
+    for (int i = threadIdx.x * VEC; i < a.G * a.Dv; i += blockDim.x * VEC) {
       float x[VEC];
-      load_vec<VEC>(v + n * ldv + i, x);
-      if (keep) store_vec<VEC>(vc + row * G * Dv + i, x);
-      if (vp) store_vec<VEC>(vp + (n * G + i / Dv) * dvp + i % Dv, x);
+      load_vec<VEC>(static_cast<const T*>(a.v) + n * a.ldv + i, x);
+      if (a.bv) {
+        float y[VEC];
+        load_vec<VEC>(static_cast<const T*>(a.bv) + i, y);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] += y[e];
+      }
+      if (keep) store_vec<VEC>(vc + row * a.G * a.Dv + i, x);
+      if (vp) store_vec<VEC>(vp + (n * a.G + i / a.Dv) * a.dvp + i % a.Dv, x);
     }
-    if (vp && dvp > Dv) {
-      const int pad = dvp - Dv;
-      for (int i = threadIdx.x; i < G * pad; i += blockDim.x) vp[(n * G + i / pad) * dvp + Dv + i % pad] = from_f<T>(0.f);
+    if (vp && a.dvp > a.Dv) {
+      const int pad = a.dvp - a.Dv;
+      for (int i = threadIdx.x; i < a.G * pad; i += blockDim.x) vp[(n * a.G + i / pad) * a.dvp + a.Dv + i % pad] = from_f<T>(0.f);
     }
   }
 }
@@ -103,7 +191,7 @@ struct DecodeArgs {
   const __nv_bfloat16 *q, *k, *v;      // q [B, H, D]
   const int64_t *slots, *lengths;      // lengths without the new token
   long max_len;
-  int H, G, D, Dv, window, splits, head_blocks;
+  int H, G, D, Dv, window, chunk, splits, head_blocks;
   float scale, cap;
   float *part, *ml;                    // part [B, H, splits, Dv], ml [B, H, splits, 2]
 };
@@ -122,7 +210,8 @@ decode_kernel(const DecodeArgs a) {
   const int grp = a.H / a.G, h0 = g * grp + hb * 16, nh = min(16, grp - hb * 16);
   const int D16 = (a.D + 15) / 16, V16 = (a.Dv + 15) / 16;
   const long len = min(a.lengths[b] + 1, (int64_t)a.max_len);
-  const int first = (a.window > 0 && len > a.window) ? (int)(len - a.window) : 0;
+  int first = (a.window > 0 && len > a.window) ? (int)(len - a.window) : 0;
+  if (a.chunk > 0) first = max(first, (int)((len - 1) / a.chunk) * a.chunk);
   const int per = ((int)((len - first + a.splits - 1) / a.splits) + KEYS - 1) / KEYS * KEYS;
   const int lo = first + split * per, hi = (int)min((long)lo + per, len);
   const __nv_bfloat16* kb = a.k + (a.slots[b] * a.max_len * a.G + g) * a.D;
@@ -289,7 +378,7 @@ decode_kernel(const DecodeArgs a) {
 // out [B, H * Dv] = (splits joined, sink in the denominator) * sigmoid(gate)
 template <typename T>
 __global__ void merge_kernel(const float* __restrict__ part, const float* __restrict__ ml, int H, int Dv, int splits, const T* __restrict__ sinks,
-                             const T* __restrict__ gate, long ldg, T* __restrict__ out) {
+                             const T* __restrict__ gate, long ldg, int per_head, T* __restrict__ out) {
   const int h = blockIdx.x, b = blockIdx.y;
   const long at = ((long)b * H + h) * splits;
   float m = sinks ? to_f(sinks[h]) : -INFINITY;
@@ -302,8 +391,86 @@ __global__ void merge_kernel(const float* __restrict__ part, const float* __rest
     for (int s = 0; s < splits; ++s)
       if (ml[(at + s) * 2] != -INFINITY) o += part[(at + s) * Dv + d] * __expf(ml[(at + s) * 2] - m);
     o *= inv;
-    if (gate) o *= sigmoid_f(to_f(gate[b * ldg + (long)h * Dv + d]));
+    if (gate) o *= sigmoid_f(to_f(gate[b * ldg + (per_head ? h : (long)h * Dv + d)]));
     out[(long)b * H * Dv + (long)h * Dv + d] = from_f<T>(o);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ differential attention
+template <typename T>
+__device__ __forceinline__ float diff_lambda(const DiffArgs& a, int lane) {
+  float s1 = 0.f, s2 = 0.f;
+  for (int i = lane; i < a.D; i += 32) {
+    s1 += to_f(static_cast<const T*>(a.lq1)[i]) * to_f(static_cast<const T*>(a.lk1)[i]);
+    s2 += to_f(static_cast<const T*>(a.lq2)[i]) * to_f(static_cast<const T*>(a.lk2)[i]);
+  }
+  return expf(warp_add(s1)) - expf(warp_add(s2)) + a.diff;
+}
+
+// a head's lanes, held NV per thread by the nt threads of the group that owns it: (map 1 - lambda map 2) over its root mean square
+// times (1 - diff) and the gate. The sum over the group comes from `add`.
+template <typename T, int NV, typename Add>
+__device__ __forceinline__ void diff_finish(float (&x)[NV], const DiffArgs& a, int Dv, const T* gate, int per_head, int t, int nt, Add add, T* out) {
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) ss += x[j] * x[j];
+  const float r = rsqrtf(add(ss) / (float)Dv + a.eps) * (1.f - a.diff);
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int d = t + j * nt;
+    if (d < Dv) out[d] = from_f<T>(x[j] * r * (gate ? sigmoid_f(to_f(gate[per_head ? 0 : d])) : 1.f));
+  }
+}
+
+// decode: grid (heads, B), 128 threads. The maps of head h are the query heads 2 h and 2 h + 1 of `part`
+template <typename T>
+__global__ void __launch_bounds__(128)
+diff_merge_kernel(const float* __restrict__ part, const float* __restrict__ ml, const DiffArgs a, int H, int Dv, int splits, const T* __restrict__ gate,
+                  long ldg, int per_head, T* __restrict__ out) {
+  __shared__ float red[4];
+  const int h = blockIdx.x, b = blockIdx.y, t = threadIdx.x;
+  const float lam = diff_lambda<T>(a, t & 31);
+  float x[2] = {0.f, 0.f};                                  // Dv up to 256
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const long at = ((long)b * 2 * H + 2 * h + m) * splits;
+    float top = -INFINITY, den = 0.f, o[2] = {0.f, 0.f};
+    for (int s = 0; s < splits; ++s) top = fmaxf(top, ml[(at + s) * 2]);
+    for (int s = 0; s < splits; ++s) {
+      if (ml[(at + s) * 2] == -INFINITY) continue;
+      const float c = __expf(ml[(at + s) * 2] - top);
+      den += ml[(at + s) * 2 + 1] * c;
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (t + j * 128 < Dv) o[j] += part[(at + s) * Dv + t + j * 128] * c;
+    }
+    const float f = den > 0.f ? (m ? -lam : 1.f) / den : 0.f;
+    x[0] += f * o[0];
+    x[1] += f * o[1];
+  }
+  const long g0 = b * ldg + (per_head ? h : (long)h * Dv);
+  diff_finish<T, 2>(x, a, Dv, gate ? gate + g0 : nullptr, per_head, t, 128, [&](float v) { return block_add(v, red); }, out + ((long)b * H + h) * Dv);
+}
+
+// prompts: a warp per token and head; o [N, 2 H, dvp] -> out [N, H * Dv]
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+diff_combine_kernel(const T* __restrict__ o, int dvp, const DiffArgs a, long N, int H, int Dv, const T* __restrict__ gate, long ldg, int per_head,
+                    T* __restrict__ out) {
+  const int lane = threadIdx.x & 31;
+  const float lam = diff_lambda<T>(a, lane);
+  for (long i = (blockIdx.x * 256l + threadIdx.x) >> 5; i < N * H; i += gridDim.x * 8l) {
+    const long n = i / H;
+    const int h = (int)(i % H);
+    const T* o1 = o + (n * 2 * H + 2 * h) * dvp;
+    float x[NV];
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int d = lane + j * 32;
+      x[j] = d < Dv ? to_f(o1[d]) - lam * to_f(o1[dvp + d]) : 0.f;
+    }
+    const long g0 = n * ldg + (per_head ? h : (long)h * Dv);
+    diff_finish<T, NV>(x, a, Dv, gate ? gate + g0 : nullptr, per_head, lane, 32, [](float v) { return warp_add(v); }, out + i * Dv);
   }
 }
 
@@ -314,8 +481,8 @@ constexpr int PQ = 16, PK = 32;
 template <typename T, int NV>          // NV * 8 >= Dv
 __global__ void __launch_bounds__(128)
 plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long max_len, const int64_t* __restrict__ slots,
-             const int64_t* __restrict__ lengths, int S, int H, int G, int D, int Dv, float scale, float cap, int window, const T* __restrict__ sinks,
-             T* __restrict__ out) {
+             const int64_t* __restrict__ lengths, int S, int H, int G, int D, int Dv, float scale, float cap, int window, int chunk,
+             const T* __restrict__ sinks, T* __restrict__ out) {
   extern __shared__ __align__(16) float smf[];
   const int LD = D + 1, LV = Dv + 1;
   float* sq = smf;                     // [PQ][LD]
@@ -330,8 +497,10 @@ plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restri
     sq[t * LD + d] = s0 + t < S ? to_f(q[(((long)b * S + s0 + t) * H + h) * D + d]) : 0.f;
   }
   const long last = min(base + min(S, s0 + PQ) - 1, max_len - 1);               // position of the last query
-  const long firstk = window > 0 ? max(0l, base + s0 - window + 1) : 0l;
   const long mine = base + s0 + r;
+  long firstk = window > 0 ? max(0l, base + s0 - window + 1) : 0l;
+  if (chunk > 0) firstk = max(firstk, (base + s0) / chunk * chunk);
+  const long from = max(window > 0 ? mine - window + 1 : 0l, chunk > 0 ? mine / chunk * chunk : 0l);      // first key this query sees
   float acc[NV], m = -INFINITY, l = 0.f;
 #pragma unroll
   for (int j = 0; j < NV; ++j) acc[j] = 0.f;
@@ -355,7 +524,7 @@ plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restri
       x *= scale;
       if (cap > 0.f) x = cap * tanhf(x / cap);
       const long p = t0 + t;
-      if (p > mine || p > last || (window > 0 && p <= mine - window)) x = -INFINITY;
+      if (p > mine || p > last || p < from) x = -INFINITY;
       sc[j] = x;
       tm = fmaxf(tm, x);
     }
@@ -403,14 +572,20 @@ plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restri
 // ------------------------------------------------------------------------------------------------ gate
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
-head_gate_kernel(const T* __restrict__ o, int dvp, const T* __restrict__ g, long ldg, long rows, int HD, int Dv, T* __restrict__ out) {
+head_gate_kernel(const T* __restrict__ o, int dvp, const T* __restrict__ g, long ldg, long rows, int HD, int Dv, int per_head,
+                 T* __restrict__ out) {
   const long per = HD / VEC;
   for (long i = blockIdx.x * 256l + threadIdx.x; i < rows * per; i += gridDim.x * 256l) {
     const long r = i / per;
     const int c = (int)(i % per) * VEC, h = c / Dv, d = c % Dv;
     float x[VEC], y[VEC];
     load_vec<VEC>(o + (r * (HD / Dv) + h) * dvp + d, x);
-    load_vec<VEC>(g + r * ldg + c, y);
+    if (per_head) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = to_f(g[r * ldg + h]);
+    } else {
+      load_vec<VEC>(g + r * ldg + c, y);
+    }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) x[e] *= sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-y[e])) : sigmoid_f(y[e]);
     store_vec<VEC>(out + r * HD + c, x);
@@ -418,21 +593,19 @@ head_gate_kernel(const T* __restrict__ o, int dvp, const T* __restrict__ g, long
 }
 
 template <typename T>
-int prep_t(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int H, int G, int D, int Dv, const int64_t* pos, const float* inv_ts,
-           int rot, float eps, int S, void* qp, int dq, void* kp, void* vp, int dvp, void* kc, void* vc, long max_len, const int64_t* slots,
-           const int64_t* lengths, const int64_t* new_lens, long N, cudaStream_t st) {
-  const bool v4 = D % 4 == 0 && Dv % 4 == 0 && rot % 8 == 0 && dq % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 && (!vp || dvp % 4 == 0) &&
-                  (reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) % (4 * sizeof(T)) == 0;
-  const int wide = dq > D ? dq : D;
+int prep_t(const PrepArgs& a, long N, cudaStream_t st) {
+  uintptr_t bits = 0;
+  for (const void* p : {a.q, a.k, a.v, a.bq, a.bk, a.bv, a.wq, a.wk}) bits |= reinterpret_cast<uintptr_t>(p);
+  const bool v4 = a.D % 4 == 0 && a.Dv % 4 == 0 && a.rot % (a.paired ? 4 : 8) == 0 && a.dq % 4 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && a.ldv % 4 == 0 &&
+                  (!a.vp || a.dvp % 4 == 0) && bits % (4 * sizeof(T)) == 0;
   auto launch = [&](auto kernel) {
-    kernel<<<(unsigned)N, 128, (rot / 2) * 8 + 8, st>>>((const T*)q, ldq, (const T*)k, ldk, (const T*)v, ldv, H, G, D, Dv, pos, inv_ts, rot, eps, S, (T*)qp, dq,
-                                                        (T*)kp, (T*)vp, dvp, (T*)kc, (T*)vc, max_len, slots, lengths, new_lens);
+    kernel<<<(unsigned)N, 128, (a.rot / 2) * 8 + 8, st>>>(a);
     return cudaGetLastError() == cudaSuccess ? 0 : -3;
   };
-  if (wide > 512) return -1;
+  if (a.D > 512) return -1;
   if (!v4) return launch(qkv_prep_kernel<T, 1, 16>);
-  if (wide <= 128) return launch(qkv_prep_kernel<T, 4, 1>);
-  if (wide <= 256) return launch(qkv_prep_kernel<T, 4, 2>);
+  if (a.D <= 128) return launch(qkv_prep_kernel<T, 4, 1>);
+  if (a.D <= 256) return launch(qkv_prep_kernel<T, 4, 2>);
   return launch(qkv_prep_kernel<T, 4, 4>);
 }
 
@@ -454,12 +627,12 @@ int decode_dv(const DecodeArgs& a, int B, cudaStream_t st) {
 
 template <typename T>
 int plain_t(const void* q, const void* k, const void* v, long max_len, const int64_t* slots, const int64_t* lengths, int B, int S, int H, int G, int D, int Dv,
-            float scale, float cap, int window, const void* sinks, void* out, cudaStream_t st) {
+            float scale, float cap, int window, int chunk, const void* sinks, void* out, cudaStream_t st) {
   const int smem = ((PQ + PK) * (D + 1) + PK * (Dv + 1) + PQ * (PK + 1)) * 4;
   if (Dv > 512 || smem > 227 * 1024) return -1;
   auto launch = [&](auto kernel) {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
-    kernel<<<dim3((S + PQ - 1) / PQ, H, B), 128, smem, st>>>((const T*)q, (const T*)k, (const T*)v, max_len, slots, lengths, S, H, G, D, Dv, scale, cap, window,
+    kernel<<<dim3((S + PQ - 1) / PQ, H, B), 128, smem, st>>>((const T*)q, (const T*)k, (const T*)v, max_len, slots, lengths, S, H, G, D, Dv, scale, cap, window, chunk,
                                                              (const T*)sinks, (T*)out);
     return cudaGetLastError() == cudaSuccess ? 0 : -3;
   };
@@ -470,12 +643,12 @@ int plain_t(const void* q, const void* k, const void* v, long max_len, const int
 }
 
 template <typename T>
-int gate_t(const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, void* out, int sms, cudaStream_t st) {
-  const bool v8 = Dv % 8 == 0 && dvp % 8 == 0 && ldg % 8 == 0 && reinterpret_cast<uintptr_t>(g) % 16 == 0;
+int gate_t(const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, int per_head, void* out, int sms, cudaStream_t st) {
+  const bool v8 = Dv % 8 == 0 && dvp % 8 == 0 && (per_head || (ldg % 8 == 0 && reinterpret_cast<uintptr_t>(g) % 16 == 0));
   const long blocks = (rows * (HD / (v8 ? 8 : 1)) + 255) / 256;
   const unsigned grid = (unsigned)(blocks < sms * 16l ? (blocks < 1 ? 1 : blocks) : sms * 16l);
-  if (v8) head_gate_kernel<T, 8><<<grid, 256, 0, st>>>((const T*)o, dvp, (const T*)g, ldg, rows, HD, Dv, (T*)out);
-  else head_gate_kernel<T, 1><<<grid, 256, 0, st>>>((const T*)o, dvp, (const T*)g, ldg, rows, HD, Dv, (T*)out);
+  if (v8) head_gate_kernel<T, 8><<<grid, 256, 0, st>>>((const T*)o, dvp, (const T*)g, ldg, rows, HD, Dv, per_head, (T*)out);
+  else head_gate_kernel<T, 1><<<grid, 256, 0, st>>>((const T*)o, dvp, (const T*)g, ldg, rows, HD, Dv, per_head, (T*)out);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -485,34 +658,51 @@ int gate_t(const void* o, int dvp, const void* g, long ldg, long rows, int HD, i
 using namespace mt::cattn;
 using bf16 = __nv_bfloat16;
 
-extern "C" int mt_qkv_prep(int f32, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int H, int G, int D, int Dv, const int64_t* pos,
-                           const float* inv_ts, int rot, float eps, int S, void* qp, int dq, void* kp, void* vp, int dvp, void* kc, void* vc, long max_len,
-                           const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, long N, cudaStream_t st) {
+extern "C" int mt_qkv_prep(int f32, const PrepArgs* a, long N, cudaStream_t st) {
   if (N <= 0) return 0;
-  return f32 ? prep_t<float>(q, ldq, k, ldk, v, ldv, H, G, D, Dv, pos, inv_ts, rot, eps, S, qp, dq, kp, vp, dvp, kc, vc, max_len, slots, lengths, new_lens, N, st)
-             : prep_t<bf16>(q, ldq, k, ldk, v, ldv, H, G, D, Dv, pos, inv_ts, rot, eps, S, qp, dq, kp, vp, dvp, kc, vc, max_len, slots, lengths, new_lens, N, st);
+  return f32 ? prep_t<float>(*a, N, st) : prep_t<bf16>(*a, N, st);
 }
 
+// diff (or null): q holds two maps per head, H counts both, out is [B, H / 2 * Dv]
 extern "C" int mt_cached_decode(const void* q, const void* k, const void* v, const int64_t* slots, const int64_t* lengths, long max_len, int B, int H, int G,
-                                int D, int Dv, float scale, float cap, int window, const void* sinks, const void* gate, long ldg, int splits, float* part,
-                                float* ml, void* out, cudaStream_t st) {
+                                int D, int Dv, float scale, float cap, int window, int chunk, const void* sinks, const void* gate, long ldg, int per_head,
+                                const DiffArgs* diff, int splits, float* part, float* ml, void* out, cudaStream_t st) {
   if (B <= 0) return 0;
-  if (D % 8 || Dv % 8 || D > 256 || Dv > 256 || H % G || splits < 1) return -1;
-  DecodeArgs a{(const bf16*)q, (const bf16*)k, (const bf16*)v, slots, lengths, max_len, H, G, D, Dv, window, splits, (H / G + 15) / 16, scale, cap, part, ml};
+  if (D % 8 || Dv % 8 || D > 256 || Dv > 256 || H % G || splits < 1 || (diff && (H % 2 || sinks))) return -1;
+  DecodeArgs a{(const bf16*)q, (const bf16*)k, (const bf16*)v, slots, lengths, max_len, H, G, D, Dv, window, chunk, splits, (H / G + 15) / 16, scale, cap,
+               part, ml};
   const int rc = D <= 64 ? decode_dv<64>(a, B, st) : (D <= 128 ? decode_dv<128>(a, B, st) : decode_dv<256>(a, B, st));
   if (rc) return rc;
-  merge_kernel<bf16><<<dim3(H, B), Dv <= 64 ? 64 : 128, 0, st>>>(part, ml, H, Dv, splits, (const bf16*)sinks, (const bf16*)gate, ldg, (bf16*)out);
+  if (diff)
+    diff_merge_kernel<bf16><<<dim3(H / 2, B), 128, 0, st>>>(part, ml, *diff, H / 2, Dv, splits, (const bf16*)gate, ldg, per_head, (bf16*)out);
+  else
+    merge_kernel<bf16><<<dim3(H, B), Dv <= 64 ? 64 : 128, 0, st>>>(part, ml, H, Dv, splits, (const bf16*)sinks, (const bf16*)gate, ldg, per_head, (bf16*)out);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
 extern "C" int mt_cached_attention(int f32, const void* q, const void* k, const void* v, long max_len, const int64_t* slots, const int64_t* lengths, int B, int S,
-                                   int H, int G, int D, int Dv, float scale, float cap, int window, const void* sinks, void* out, cudaStream_t st) {
+                                   int H, int G, int D, int Dv, float scale, float cap, int window, int chunk, const void* sinks, void* out, cudaStream_t st) {
   if (B <= 0 || S <= 0) return 0;
-  return f32 ? plain_t<float>(q, k, v, max_len, slots, lengths, B, S, H, G, D, Dv, scale, cap, window, sinks, out, st)
-             : plain_t<bf16>(q, k, v, max_len, slots, lengths, B, S, H, G, D, Dv, scale, cap, window, sinks, out, st);
+  return f32 ? plain_t<float>(q, k, v, max_len, slots, lengths, B, S, H, G, D, Dv, scale, cap, window, chunk, sinks, out, st)
+             : plain_t<bf16>(q, k, v, max_len, slots, lengths, B, S, H, G, D, Dv, scale, cap, window, chunk, sinks, out, st);
 }
 
-extern "C" int mt_head_gate(int f32, const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, void* out, int sms, cudaStream_t st) {
+extern "C" int mt_head_gate(int f32, const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, int per_head, void* out, int sms,
+                            cudaStream_t st) {
   if (rows <= 0) return 0;
-  return f32 ? gate_t<float>(o, dvp, g, ldg, rows, HD, Dv, out, sms, st) : gate_t<bf16>(o, dvp, g, ldg, rows, HD, Dv, out, sms, st);
+  return f32 ? gate_t<float>(o, dvp, g, ldg, rows, HD, Dv, per_head, out, sms, st) : gate_t<bf16>(o, dvp, g, ldg, rows, HD, Dv, per_head, out, sms, st);
+}
+
+extern "C" int mt_diff_combine(int f32, const void* o, int dvp, const DiffArgs* a, long N, int H, int Dv, const void* gate, long ldg, int per_head, void* out,
+                               int sms, cudaStream_t st) {
+  if (N <= 0) return 0;
+  if (Dv > 256) return -1;
+  const long blocks = (N * H + 7) / 8;
+  const unsigned grid = (unsigned)(blocks < sms * 16l ? blocks : sms * 16l);
+#define GO(T, NV) diff_combine_kernel<T, NV><<<grid, 256, 0, st>>>((const T*)o, dvp, *a, N, H, Dv, (const T*)gate, ldg, per_head, (T*)out)
+  if (Dv <= 64) { if (f32) GO(float, 2); else GO(bf16, 2); }
+  else if (Dv <= 128) { if (f32) GO(float, 4); else GO(bf16, 4); }
+  else { if (f32) GO(float, 8); else GO(bf16, 8); }
+#undef GO
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

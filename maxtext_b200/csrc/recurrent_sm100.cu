@@ -1,6 +1,8 @@
 // Inference kernels of the recurrent layers. Per head a matrix state S [dk, dv] in fp32, per token
 //   gated delta:               S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q       (g, beta scalars per head)
 //   gated linear attention:    S <- diag(alpha) S + k v^T;                        o = S^T q       (alpha per key channel)
+//   retention:                 S <- d S + k v^T;                                  o = S^T q       (d fixed per head; q and k rotated)
+//   channel-wise gated delta:  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q  (g per key channel)
 // Three families:
 //  * decode (one token per sequence): one CTA per sequence and key head does everything between the input and the output projection:
 //    short convolution, unit norms, gates, state update, read-out, head norm and output gate. Bound by reading and writing S once: it passes through
@@ -44,15 +46,46 @@ struct GlaArgs {
   int rank; float inv_tau;
 };
 
+template <typename T>
+struct RetArgs {
+  const T* x; long ldx;          // q H*dk | k H*dk | v H*dv | gate H*dv
+  const float* log_decay;        // [H]
+  const float* inv_ts; int rot;  // rotated lanes, halves paired
+};
+
+template <typename T>
+struct ChanArgs {
+  const T* x; long ldx;          // decode: q hk*dk | k hk*dk | v hv*dv before the convolution
+  const T* beta; long ldb;       // logits [N, >= hv]
+  const T* conv_w; int taps;     // [taps, conv_dim]
+  float* conv;                   // [slots, taps - 1, conv_dim]
+  const float* da;               // product of the decay projection [N, hv*dk]
+  const T* A_log; const T* dt_bias;        // [hv], [hv*dk]
+  const T* z; long ldz;          // decode: gate logits [N, >= hv*dv]
+};
+
+enum { DELTA = 0, GLA = 1, RET = 2, CHAN = 3 };
+
 __device__ __forceinline__ float beta_gate(float b) { return sigmoid_f(b); }
 __device__ __forceinline__ float log_decay(float a, float A_log, float dt) { return -expf(A_log) * softplus_f(a + dt); }
+
+// lane e of a head (at x) turned by pos * inv_ts; halves paired
+template <typename T>
+__device__ __forceinline__ float turned(const T* x, int e, int rot, float c, float sn) {
+  const float v = to_f(x[e]);
+  if (e >= rot) return v;
+  const int half = rot / 2;
+  return e < half ? v * c - to_f(x[e + half]) * sn : v * c + to_f(x[e - half]) * sn;
+}
 
 // ------------------------------------------------------------------------------------------------ decode
 // grid (hk, B). TILE: the state of a head passes through shared memory (cp.async, several CTAs per SM hide each other's phases); otherwise it is read
 // twice from global memory (states too wide for shared memory, or not a multiple of 16 bytes).
-template <typename T, bool DELTA, bool TILE>
-__global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, DeltaArgs<T> d, GlaArgs<T> gl, const T* __restrict__ norm_w, float eps,
-                                                                 T* __restrict__ out, int dvp, int rows) {
+template <typename T, int KIND, bool TILE>
+__global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, DeltaArgs<T> d, GlaArgs<T> gl, RetArgs<T> rt, ChanArgs<T> ch_,
+                                                                 const T* __restrict__ norm_w, float eps, T* __restrict__ out, int dvp, int rows) {
+  constexpr bool RULE = KIND == DELTA || KIND == CHAN;  // the write removes what the key retrieves
+  constexpr bool VECDEC = KIND == GLA || KIND == CHAN;  // a decay per key channel
   extern __shared__ __align__(16) float sm[];
   const int kh = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const int dk = a.dk, dv = a.dv, r = a.r, H = a.hk * r;
@@ -61,8 +94,10 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
   float* tile = sm;                                     // [dk * dv]
   float* qs = tile + (TILE ? dk * dv : 0);              // [rows * nrg] each
   float* ks = qs + rows * nrg;
-  float* al = ks + rows * nrg;                          // alpha - 1 (GLA)
-  float* redk = al + (DELTA ? 0 : rows * nrg);          // [DEC_NT]
+  float* al = ks + rows * nrg;                          // decay - 1 per key channel
+  float* qa = al + (VECDEC ? rows * nrg : 0);           // decayed q and k (CHAN: they differ between the value heads of a key head)
+  float* ka = qa + (KIND == CHAN ? rows * nrg : 0);
+  float* redk = ka + (KIND == CHAN ? rows * nrg : 0);   // [DEC_NT]
   float* redq = redk + DEC_NT;
   float* wsum = redq + DEC_NT;                          // [DEC_NT / 32]
   float* vs = wsum + DEC_NT / 32;                       // [r * dv]
@@ -85,17 +120,18 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
   load_tile(kh * r);                                    // in flight while the convolution and the gates are computed
 
   const T* xr;
-  if constexpr (DELTA) {
-    const int per = 2 * dk + 2 * r * dv, key_dim = a.hk * dk, conv_dim = 2 * key_dim + H * dv, K = d.taps;
-    xr = d.x + b * d.ldx + (long)kh * per;
-    float* cs = d.conv + slot * (long)(K - 1) * conv_dim;
+  if constexpr (RULE) {
+    const int per = 2 * dk + 2 * r * dv, key_dim = a.hk * dk, conv_dim = 2 * key_dim + H * dv, K = KIND == DELTA ? d.taps : ch_.taps;
+    xr = KIND == DELTA ? d.x + b * d.ldx + (long)kh * per : ch_.x + b * ch_.ldx;
+    float* cs = (KIND == DELTA ? d.conv : ch_.conv) + slot * (long)(K - 1) * conv_dim;
+    const T* conv_w = KIND == DELTA ? d.conv_w : ch_.conv_w;
     for (int i = tid; i < 2 * dk + r * dv; i += DEC_NT) {
       const int ch = i < dk ? kh * dk + i : (i < 2 * dk ? key_dim + kh * dk + (i - dk) : 2 * key_dim + kh * r * dv + (i - 2 * dk));
-      const float xv = to_f(xr[i]);
-      float acc = to_f(d.conv_w[(long)(K - 1) * conv_dim + ch]) * xv;
+      const float xv = to_f(xr[KIND == DELTA ? i : ch]);
+      float acc = to_f(conv_w[(long)(K - 1) * conv_dim + ch]) * xv;
       for (int j = 0; j < K - 1; ++j) {
         const float old = fresh ? 0.f : cs[(long)j * conv_dim + ch];
-        acc += to_f(d.conv_w[(long)j * conv_dim + ch]) * old;
+        acc += to_f(conv_w[(long)j * conv_dim + ch]) * old;
         if (j > 0) cs[(long)(j - 1) * conv_dim + ch] = old;
       }
       if (K > 1) cs[(long)(K - 2) * conv_dim + ch] = xv;
@@ -104,6 +140,17 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
       else if (i < 2 * dk) ks[i - dk] = y;
       else vs[i - 2 * dk] = y;
     }
+  } else if constexpr (KIND == RET) {
+    xr = rt.x + b * rt.ldx;
+    const float pos = (float)a.lengths[b];
+    const T *xq = xr + (long)kh * dk, *xk = xr + (long)H * dk + (long)kh * dk;
+    for (int i = tid; i < dk; i += DEC_NT) {
+      float sn = 0.f, c = 1.f;
+      if (i < rt.rot) sincosf(pos * rt.inv_ts[i % (rt.rot / 2)], &sn, &c);
+      qs[i] = turned(xq, i, rt.rot, c, sn);
+      ks[i] = turned(xk, i, rt.rot, c, sn);
+    }
+    for (int i = tid; i < dv; i += DEC_NT) vs[i] = to_f(xr[2L * H * dk + kh * dv + i]);
   } else {
     xr = gl.x + b * gl.ldx;
     for (int i = tid; i < dk; i += DEC_NT) {
@@ -130,18 +177,27 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
   }
   qk = warp_add(qk);
   float rq = rsqrtf((float)dk), rk = 1.f;
-  if constexpr (DELTA) {
+  if constexpr (RULE) {
     rq *= rsqrtf(warp_add(qq) + 1e-6f);
     rk = rsqrtf(warp_add(kk) + 1e-6f);
   }
   qk *= rq * rk;
-  if (!DELTA) {                                         // S_new^T q = S^T (alpha q) + (k . q) v
+  if (KIND == GLA) {                                         // S_new^T q = S^T (alpha q) + (k . q) v
     __syncthreads();
     for (int i = tid; i < dk; i += DEC_NT) qs[i] += al[i] * qs[i];
   }
   for (int j = 0; j < r; ++j) {
     const int h = kh * r + j;
     if (j > 0) load_tile(h);
+    if constexpr (KIND == CHAN) {
+      const float rate = -expf(to_f(ch_.A_log[h]));
+      for (int i = tid; i < dk; i += DEC_NT) {
+        const float g = expm1f(rate * softplus_f(ch_.da[((long)b * H + h) * dk + i] + to_f(ch_.dt_bias[(long)h * dk + i])));
+        al[i] = g;
+        qa[i] = qs[i] + g * qs[i];
+        ka[i] = ks[i] + g * ks[i];
+      }
+    }
     la_wait<0>();
     __syncthreads();
     float* gp = state_of(h);
@@ -152,27 +208,33 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
 #pragma unroll 8
       for (int i = 0; i < nrows; ++i) {
         const float s = sp[(long)i * dv];
-        if (DELTA) pk += s * ks[row0 + i];
-        pq += s * qs[row0 + i];
+        if (RULE) pk += s * (KIND == CHAN ? ka : ks)[row0 + i];
+        pq += s * (KIND == CHAN ? qa : qs)[row0 + i];
       }
     }
-    if (DELTA) redk[tid] = pk;
+    if (RULE) redk[tid] = pk;
     redq[tid] = pq;
     __syncthreads();
     float sk = 0.f, sq = 0.f;
     for (int g = 0; g < nrg; ++g) {
-      if (DELTA) sk += redk[g * dvp + c];
+      if (RULE) sk += redk[g * dvp + c];
       sq += redq[g * dvp + c];
     }
     float dm1 = 0.f, u = 0.f;
     const float v = col ? vs[j * dv + c] : 0.f;
-    if constexpr (DELTA) {
+    if constexpr (KIND == DELTA) {
       const T* bb = d.ba + b * d.ldb + (long)kh * 2 * r;
       dm1 = expm1f(log_decay(to_f(bb[r + j]), to_f(d.A_log[h]), to_f(d.dt_bias[h])));
       sk += dm1 * sk;
       sq += dm1 * sq;
       u = beta_gate(to_f(bb[j])) * (v - rk * sk);
+    } else if constexpr (KIND == CHAN) {
+      u = beta_gate(to_f(ch_.beta[b * ch_.ldb + h])) * (v - rk * sk);
     } else {
+      if constexpr (KIND == RET) {
+        dm1 = expm1f(rt.log_decay[h]);
+        sq += dm1 * sq;
+      }
       u = v;
     }
     const float o = col ? rq * sq + qk * u : 0.f;
@@ -182,7 +244,7 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
 #pragma unroll 8
       for (int i = 0; i < nrows; ++i) {
         const float s = read ? sp[(long)i * dv] : 0.f;
-        wp[(long)i * dv] = s + (DELTA ? dm1 : al[row0 + i]) * s + ks[row0 + i] * ku;
+        wp[(long)i * dv] = s + (VECDEC ? al[row0 + i] : dm1) * s + ks[row0 + i] * ku;
       }
     }
     // head norm over dv and output gate
@@ -193,8 +255,10 @@ __global__ void __launch_bounds__(DEC_NT) recurrent_decode_kernel(RecArgs a, Del
     for (int g = 0; g < dvp / 32; ++g) ss += wsum[g];                 // row group 0 sees every column once
     if (rg == 0 && col) {
       const float rstd = rsqrtf(ss / (float)dv + eps);
-      const T* zp = DELTA ? xr + 2 * dk + r * dv + j * dv : xr + 2L * H * dk + (long)H * dv + kh * dv;
-      out[((long)b * H + h) * dv + c] = from_f<T>(o * rstd * to_f(norm_w[c]) * silu_t<T>(to_f(zp[c])));
+      const T* zp = KIND == DELTA ? xr + 2 * dk + r * dv + j * dv : KIND == CHAN ? ch_.z + b * ch_.ldz + (long)h * dv
+                                  : xr + 2L * H * dk + (long)H * dv + kh * dv;
+      const float z = to_f(zp[c]);
+      out[((long)b * H + h) * dv + c] = from_f<T>(o * rstd * (norm_w ? to_f(norm_w[c]) : 1.f) * (KIND == CHAN ? sigmoid_f(z) : silu_t<T>(z)));
     }
   }
 }
@@ -368,18 +432,20 @@ __global__ void __launch_bounds__(128) gla_decay_tc_kernel(const __nv_bfloat16* 
 
 // ------------------------------------------------------------------------------------------------ scan over a prompt
 // grid (ceil(dv / 16), heads, B). q / k of token n sit at q[n * ldq + (h / r) * dk]; likewise v and, for GLA, log_alpha (fp32).
-template <typename T, bool DELTA, int RPT>
+template <typename T, int KIND, int RPT>
 __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v,
                                                                 long ldx, const float* __restrict__ log_alpha, const T* __restrict__ ba, long ldb,
-                                                                const T* __restrict__ A_log, const T* __restrict__ dt_bias, T* __restrict__ o) {
+                                                                const T* __restrict__ A_log, const T* __restrict__ dt_bias, RetArgs<T> rt, ChanArgs<T> ch,
+                                                                T* __restrict__ o) {
+  constexpr bool RULE = KIND == DELTA || KIND == CHAN, VECDEC = KIND == GLA || KIND == CHAN;
   constexpr int GS = RPT + 4;                            // floats per row group: the eight groups start in different banks
   extern __shared__ __align__(16) float sm[];
   const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dk = a.dk, dv = a.dv, r = a.r, H = a.hk * r, kh = h / r;
   float* qs = sm;                                        // [TC][8 * GS]
   float* ks = qs + SCAN_TC * 8 * GS;
-  float* as = ks + SCAN_TC * 8 * GS;                     // GLA only
-  float* vs = as + (DELTA ? 0 : SCAN_TC * 8 * GS);       // [TC][16]
+  float* as = ks + SCAN_TC * 8 * GS;                     // decay - 1 per key channel
+  float* vs = as + (VECDEC ? SCAN_TC * 8 * GS : 0);      // [TC][16]
   float* sc = vs + SCAN_TC * SCAN_COLS;                  // [TC][4]: decay - 1, beta, rq, k.q (normalised); rk is folded into ks
   const int c0 = blockIdx.x * SCAN_COLS, cl = warp * 4 + (lane & 3), c = c0 + cl, rg = lane >> 2;
   const bool col = c < dv;
@@ -393,8 +459,9 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
   const float qscale = rsqrtf((float)dk);
   for (int i = tid; i < SCAN_TC * 8 * GS; i += SCAN_NT) {      // padding rows stay zero
     qs[i] = 0.f; ks[i] = 0.f;
-    if (!DELTA) as[i] = 0.f;
+    if (VECDEC) as[i] = 0.f;
   }
+  const float rate = KIND == CHAN ? -expf(to_f(ch.A_log[h])) : 0.f;
   for (int t0 = 0; t0 < n; t0 += SCAN_TC) {
     const int m = min(SCAN_TC, n - t0);
     __syncthreads();
@@ -402,9 +469,17 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
       const int t = i / dk, e = i % dk;
       const long row = (long)b * a.S + t0 + t;
       const int at = t * 8 * GS + (e / RPT) * GS + e % RPT;
-      qs[at] = to_f(q[row * ldx + (long)kh * dk + e]);
-      ks[at] = to_f(k[row * ldx + (long)kh * dk + e]);
-      if (!DELTA) as[at] = expm1f(log_alpha[row * (long)H * dk + (long)h * dk + e]);
+      if constexpr (KIND == RET) {
+        float sn = 0.f, c_ = 1.f;
+        if (e < rt.rot) sincosf((float)(a.lengths[b] + t0 + t) * rt.inv_ts[e % (rt.rot / 2)], &sn, &c_);
+        qs[at] = turned(q + row * ldx + (long)kh * dk, e, rt.rot, c_, sn);
+        ks[at] = turned(k + row * ldx + (long)kh * dk, e, rt.rot, c_, sn);
+      } else {
+        qs[at] = to_f(q[row * ldx + (long)kh * dk + e]);
+        ks[at] = to_f(k[row * ldx + (long)kh * dk + e]);
+      }
+      if (KIND == GLA) as[at] = expm1f(log_alpha[row * (long)H * dk + (long)h * dk + e]);
+      if (KIND == CHAN) as[at] = expm1f(rate * softplus_f(ch.da[row * (long)H * dk + (long)h * dk + e] + to_f(ch.dt_bias[(long)h * dk + e])));
     }
     for (int i = tid; i < m * SCAN_COLS; i += SCAN_NT) {
       const int t = i / SCAN_COLS, e = c0 + i % SCAN_COLS;
@@ -419,11 +494,13 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
       }
       qk = warp_add(qk);
       float rq = qscale, rk = 1.f;
-      if constexpr (DELTA) {
+      if (KIND == RET && lane == 0) sc[t * 4] = expm1f(rt.log_decay[h]);
+      if (KIND == CHAN && lane == 0) sc[t * 4 + 1] = beta_gate(to_f(ch.beta[((long)b * a.S + t0 + t) * ch.ldb + h]));
+      if constexpr (RULE) {
         rq *= rsqrtf(warp_add(qq) + 1e-6f);
         rk = rsqrtf(warp_add(kk) + 1e-6f);
         for (int e = lane; e < dk; e += 32) ks[t * 8 * GS + (e / RPT) * GS + e % RPT] *= rk;
-        if (lane == 0) {
+        if (KIND == DELTA && lane == 0) {
           const T* bb = ba + ((long)b * a.S + t0 + t) * ldb + (long)kh * 2 * r + (h - kh * r);
           sc[t * 4] = expm1f(log_decay(to_f(bb[r]), to_f(A_log[h]), to_f(dt_bias[h])));
           sc[t * 4 + 1] = beta_gate(to_f(bb[0]));
@@ -439,21 +516,23 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
       float sk = 0.f, sq = 0.f;
 #pragma unroll
       for (int i = 0; i < RPT; ++i) {
-        if constexpr (DELTA) { sk += S[i] * kt[i]; sq += S[i] * qt[i]; }
-        else { S[i] += at[i] * S[i]; sq += S[i] * qt[i]; }
+        if constexpr (VECDEC) S[i] += at[i] * S[i];
+        if constexpr (RULE) sk += S[i] * kt[i];
+        sq += S[i] * qt[i];
       }
 #pragma unroll
       for (int w = 4; w <= 16; w <<= 1) {
-        if (DELTA) sk += __shfl_xor_sync(0xffffffffu, sk, w);
+        if (RULE) sk += __shfl_xor_sync(0xffffffffu, sk, w);
         sq += __shfl_xor_sync(0xffffffffu, sq, w);
       }
       const float rq = sc[t * 4 + 2], kq = sc[t * 4 + 3];
       float u = vs[t * SCAN_COLS + cl];
-      if constexpr (DELTA) {
+      if constexpr (KIND == CHAN) u = sc[t * 4 + 1] * (u - sk);
+      if constexpr (!VECDEC) {
         const float dm1 = sc[t * 4];
         sk += dm1 * sk;
         sq += dm1 * sq;
-        u = sc[t * 4 + 1] * (u - sk);
+        if (KIND == DELTA) u = sc[t * 4 + 1] * (u - sk);
 #pragma unroll
         for (int i = 0; i < RPT; ++i) S[i] += dm1 * S[i];
       }
@@ -473,9 +552,9 @@ __global__ void __launch_bounds__(SCAN_NT) recurrent_scan_kernel(RecArgs a, cons
 }
 
 // ------------------------------------------------------------------------------------------------ head norm + output gate
-// out[n, h, :] = rms(o[n, h, :]) * w * silu(z), one warp per (n, h); z of head h sits at x[n * ldx + zoff + (h / r) * zstride + (h % r) * dv].
+// out[n, h, :] = rms(o[n, h, :]) * w * silu(z) (without w: no weight; SIG: sigmoid(z)), one warp per (n, h); z of head h sits at x[n * ldx + zoff + (h / r) * zstride + (h % r) * dv].
 // LPR lanes share a row.
-template <typename T, int VEC, int LPR>
+template <typename T, int VEC, int LPR, bool SIG>
 __global__ void __launch_bounds__(256) gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ x, long ldx, long rows, int H, int dv, int r,
                                                               long zoff, long zstride, const T* __restrict__ w, float eps, T* __restrict__ out) {
   const long row = ((long)blockIdx.x * blockDim.x + threadIdx.x) / LPR;
@@ -500,44 +579,45 @@ __global__ void __launch_bounds__(256) gated_head_norm_kernel(const T* __restric
     float z[VEC], g[VEC];
     if (!once) load_vec<VEC>(op + c, v);
     load_vec<VEC>(zp + c, z);
-    load_vec<VEC>(w + c, g);
+    if (w) load_vec<VEC>(w + c, g);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) v[e] = v[e] * rstd * g[e] * silu_t<T>(z[e]);
+    for (int e = 0; e < VEC; ++e) v[e] = v[e] * (w ? rstd * g[e] : rstd) * (SIG ? sigmoid_t<T>(z[e]) : silu_t<T>(z[e]));
     store_vec<VEC>(out + row * dv + c, v);
   }
 }
 
 // ------------------------------------------------------------------------------------------------ launchers
-template <typename T, bool DELTA>
-int launch_decode(const RecArgs& a, const DeltaArgs<T>& d, const GlaArgs<T>& g, const void* norm, float eps, void* out, int B, cudaStream_t st) {
+template <typename T, int KIND>
+int launch_decode(const RecArgs& a, const DeltaArgs<T>& d, const GlaArgs<T>& g, const RetArgs<T>& rt, const ChanArgs<T>& ch, const void* norm, float eps,
+                  void* out, int B, cudaStream_t st) {
   int dvp = 32;
   while (dvp < a.dv) dvp <<= 1;
   if (dvp > DEC_NT) return -1;
   const int nrg = DEC_NT / dvp, rows = ((a.dk + nrg - 1) / nrg + 3) & ~3;
   const size_t state = sizeof(float) * (size_t)a.dk * a.dv;
   const bool tile = state % 16 == 0 && state <= 160 * 1024;
-  const size_t smem = (tile ? state : 0) + sizeof(float) * ((DELTA ? 2 : 3) * (size_t)rows * nrg + (size_t)a.r * a.dv + 2 * DEC_NT + DEC_NT / 32);
+  const size_t smem = (tile ? state : 0) + sizeof(float) * ((KIND == CHAN ? 5 : KIND == GLA ? 3 : 2) * (size_t)rows * nrg + (size_t)a.r * a.dv + 2 * DEC_NT + DEC_NT / 32);
   if (smem > 220 * 1024) return -1;
-  auto k1 = recurrent_decode_kernel<T, DELTA, true>;
-  auto k0 = recurrent_decode_kernel<T, DELTA, false>;
+  auto k1 = recurrent_decode_kernel<T, KIND, true>;
+  auto k0 = recurrent_decode_kernel<T, KIND, false>;
   auto k = tile ? k1 : k0;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return -2;
-  k<<<dim3(a.hk, B), DEC_NT, smem, st>>>(a, d, g, (const T*)norm, eps, (T*)out, dvp, rows);
+  k<<<dim3(a.hk, B), DEC_NT, smem, st>>>(a, d, g, rt, ch, (const T*)norm, eps, (T*)out, dvp, rows);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-template <typename T, bool DELTA>
+template <typename T, int KIND>
 int launch_scan(const RecArgs& a, const void* q, const void* k, const void* v, long ldx, const float* la, const void* ba, long ldb, const void* A,
-                const void* dt, void* o, int B, cudaStream_t st) {
+                const void* dt, const RetArgs<T>& rt, const ChanArgs<T>& ch, void* o, int B, cudaStream_t st) {
   const int need = (a.dk + 7) / 8;
   const int rpt = need <= 4 ? 4 : need <= 8 ? 8 : need <= 16 ? 16 : need <= 32 ? 32 : 0;
   if (!rpt) return -1;
-  const size_t smem = sizeof(float) * ((DELTA ? 2 : 3) * (size_t)SCAN_TC * 8 * (rpt + 4) + SCAN_TC * SCAN_COLS + SCAN_TC * 4);
-  auto kern = rpt == 4 ? recurrent_scan_kernel<T, DELTA, 4> : rpt == 8 ? recurrent_scan_kernel<T, DELTA, 8> : rpt == 16
-      ? recurrent_scan_kernel<T, DELTA, 16> : recurrent_scan_kernel<T, DELTA, 32>;
+  const size_t smem = sizeof(float) * ((KIND == GLA || KIND == CHAN ? 3 : 2) * (size_t)SCAN_TC * 8 * (rpt + 4) + SCAN_TC * SCAN_COLS + SCAN_TC * 4);
+  auto kern = rpt == 4 ? recurrent_scan_kernel<T, KIND, 4> : rpt == 8 ? recurrent_scan_kernel<T, KIND, 8> : rpt == 16
+      ? recurrent_scan_kernel<T, KIND, 16> : recurrent_scan_kernel<T, KIND, 32>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return -2;
   kern<<<dim3((a.dv + SCAN_COLS - 1) / SCAN_COLS, a.hk * a.r, B), SCAN_NT, smem, st>>>(
-      a, (const T*)q, (const T*)k, (const T*)v, ldx, la, (const T*)ba, ldb, (const T*)A, (const T*)dt, (T*)o);
+      a, (const T*)q, (const T*)k, (const T*)v, ldx, la, (const T*)ba, ldb, (const T*)A, (const T*)dt, rt, ch, (T*)o);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -559,16 +639,18 @@ int launch_conv(const RecArgs& a, const DeltaArgs<T>& d, void* y, int B, cudaStr
 }
 
 template <typename T>
-int launch_head_norm(const void* o, const void* x, long ldx, long rows, int H, int dv, int r, long zoff, long zstride, const void* w, float eps, void* out,
-                     cudaStream_t st) {
-  const bool v8 = dv % 8 == 0 && ldx % 8 == 0 && zoff % 8 == 0 && zstride % 8 == 0;
-#define GO(V, L) gated_head_norm_kernel<T, V, L><<<(unsigned)((rows * L + 255) / 256), 256, 0, st>>>((const T*)o, (const T*)x, ldx, rows, H, dv, r, zoff, \
-                                                                                                  zstride, (const T*)w, eps, (T*)out)
+int launch_head_norm(const void* o, const void* x, long ldx, long rows, int H, int dv, int r, long zoff, long zstride, const void* w, float eps, int sig,
+                     void* out, cudaStream_t st) {
+  const bool v8 = dv % 8 == 0 && ldx % 8 == 0 && zoff % 8 == 0 && zstride % 8 == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0;
+#define GO_(V, L, S) gated_head_norm_kernel<T, V, L, S><<<(unsigned)((rows * L + 255) / 256), 256, 0, st>>>((const T*)o, (const T*)x, ldx, rows, H, dv, r, \
+                                                                                                         zoff, zstride, (const T*)w, eps, (T*)out)
+#define GO(V, L) do { if (sig) GO_(V, L, true); else GO_(V, L, false); } while (0)
   if (!v8) GO(1, 32);
   else if (dv <= 64) GO(8, 8);
   else if (dv <= 128) GO(8, 16);
   else GO(8, 32);
 #undef GO
+#undef GO_
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -583,8 +665,8 @@ extern "C" int mt_delta_decode(int f32, const void* x, long ldx, const void* ba,
                                const int64_t* slots, const int64_t* lengths, void* out, int B, cudaStream_t st) {
   if (B <= 0) return 0;
   const RecArgs a{hk, hv / hk, dk, dv, 1, slots, lengths, nullptr, rec};
-#define CALL(T) launch_decode<T, true>(a, DeltaArgs<T>{(const T*)x, ldx, (const T*)ba, ldb, (const T*)conv_w, taps, conv, (const T*)A_log, \
-                                                       (const T*)dt_bias}, GlaArgs<T>{}, norm, eps, out, B, st)
+#define CALL(T) launch_decode<T, DELTA>(a, DeltaArgs<T>{(const T*)x, ldx, (const T*)ba, ldb, (const T*)conv_w, taps, conv, (const T*)A_log, \
+                                                       (const T*)dt_bias}, GlaArgs<T>{}, RetArgs<T>{}, ChanArgs<T>{}, norm, eps, out, B, st)
   return MT_BY_TYPE(f32, CALL);
 #undef CALL
 }
@@ -593,7 +675,8 @@ extern "C" int mt_gla_decode(int f32, const void* x, long ldx, const void* w, co
                              int H, int dk, int dv, float* rec, const int64_t* slots, const int64_t* lengths, void* out, int B, cudaStream_t st) {
   if (B <= 0) return 0;
   const RecArgs a{H, 1, dk, dv, 1, slots, lengths, nullptr, rec};
-#define CALL(T) launch_decode<T, false>(a, DeltaArgs<T>{}, GlaArgs<T>{(const T*)x, ldx, (const T*)w, (const T*)bias, rank, inv_tau}, norm, eps, out, B, st)
+#define CALL(T) launch_decode<T, GLA>(a, DeltaArgs<T>{}, GlaArgs<T>{(const T*)x, ldx, (const T*)w, (const T*)bias, rank, inv_tau}, RetArgs<T>{}, \
+                                      ChanArgs<T>{}, norm, eps, out, B, st)
   return MT_BY_TYPE(f32, CALL);
 #undef CALL
 }
@@ -612,8 +695,8 @@ extern "C" int mt_delta_scan(int f32, const void* mixed, const void* ba, long ld
   if (B <= 0 || S <= 0) return 0;
   const RecArgs a{hk, hv / hk, dk, dv, S, slots, lengths, new_lens, rec};
   const long ld = 2L * hk * dk + (long)hv * dv;
-#define CALL(T) launch_scan<T, true>(a, (const T*)mixed, (const T*)mixed + (long)hk * dk, (const T*)mixed + 2L * hk * dk, ld, nullptr, ba, ldb, A_log, \
-                                     dt_bias, o, B, st)
+#define CALL(T) launch_scan<T, DELTA>(a, (const T*)mixed, (const T*)mixed + (long)hk * dk, (const T*)mixed + 2L * hk * dk, ld, nullptr, ba, ldb, A_log, \
+                                     dt_bias, RetArgs<T>{}, ChanArgs<T>{}, o, B, st)
   return MT_BY_TYPE(f32, CALL);
 #undef CALL
 }
@@ -622,8 +705,8 @@ extern "C" int mt_gla_scan(int f32, const void* x, long ldx, const float* log_al
                            const int64_t* lengths, const int64_t* new_lens, void* o, int B, cudaStream_t st) {
   if (B <= 0 || S <= 0) return 0;
   const RecArgs a{H, 1, dk, dv, S, slots, lengths, new_lens, rec};
-#define CALL(T) launch_scan<T, false>(a, (const T*)x, (const T*)x + (long)H * dk, (const T*)x + 2L * H * dk, ldx, log_alpha, nullptr, 0, nullptr, nullptr, \
-                                      o, B, st)
+#define CALL(T) launch_scan<T, GLA>(a, (const T*)x, (const T*)x + (long)H * dk, (const T*)x + 2L * H * dk, ldx, log_alpha, nullptr, 0, nullptr, nullptr, \
+                                      RetArgs<T>{}, ChanArgs<T>{}, o, B, st)
   return MT_BY_TYPE(f32, CALL);
 #undef CALL
 }
@@ -646,8 +729,52 @@ extern "C" int mt_gla_decay(int f32, const void* lo, long ldx, const void* w, co
 }
 
 extern "C" int mt_gated_head_norm(int f32, const void* o, const void* x, long ldx, long rows, int H, int dv, int r, long zoff, long zstride, const void* w,
-                                  float eps, void* out, cudaStream_t st) {
+                                  float eps, int sig, void* out, cudaStream_t st) {
   if (rows <= 0) return 0;
-  return f32 ? launch_head_norm<float>(o, x, ldx, rows, H, dv, r, zoff, zstride, w, eps, out, st)
-             : launch_head_norm<__nv_bfloat16>(o, x, ldx, rows, H, dv, r, zoff, zstride, w, eps, out, st);
+  return f32 ? launch_head_norm<float>(o, x, ldx, rows, H, dv, r, zoff, zstride, w, eps, sig, out, st)
+             : launch_head_norm<__nv_bfloat16>(o, x, ldx, rows, H, dv, r, zoff, zstride, w, eps, sig, out, st);
+}
+
+extern "C" int mt_retention_decode(int f32, const void* x, long ldx, const float* log_decay, const float* inv_ts, int rot, float eps, int H, int dk, int dv,
+                                   float* rec, const int64_t* slots, const int64_t* lengths, void* out, int B, cudaStream_t st) {
+  if (B <= 0) return 0;
+  const RecArgs a{H, 1, dk, dv, 1, slots, lengths, nullptr, rec};
+#define CALL(T) launch_decode<T, RET>(a, DeltaArgs<T>{}, GlaArgs<T>{}, RetArgs<T>{(const T*)x, ldx, log_decay, inv_ts, rot}, ChanArgs<T>{}, nullptr, eps, out, B, st)
+  return MT_BY_TYPE(f32, CALL);
+#undef CALL
+}
+
+extern "C" int mt_retention_scan(int f32, const void* x, long ldx, const float* log_decay, const float* inv_ts, int rot, int H, int dk, int dv, int S, float* rec,
+                                 const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* o, int B, cudaStream_t st) {
+  if (B <= 0 || S <= 0) return 0;
+  const RecArgs a{H, 1, dk, dv, S, slots, lengths, new_lens, rec};
+#define CALL(T) launch_scan<T, RET>(a, (const T*)x, (const T*)x + (long)H * dk, (const T*)x + 2L * H * dk, ldx, nullptr, nullptr, 0, nullptr, nullptr, \
+                                    RetArgs<T>{(const T*)x, ldx, log_decay, inv_ts, rot}, ChanArgs<T>{}, o, B, st)
+  return MT_BY_TYPE(f32, CALL);
+#undef CALL
+}
+
+extern "C" int mt_channel_delta_decode(int f32, const void* x, long ldx, const void* beta, long ldb, const void* conv_w, int taps, const float* da,
+                                       const void* A_log, const void* dt_bias, const void* z, long ldz, const void* norm, float eps, int hk, int hv, int dk,
+                                       int dv, float* conv, float* rec, const int64_t* slots, const int64_t* lengths, void* out, int B, cudaStream_t st) {
+  if (B <= 0) return 0;
+  const RecArgs a{hk, hv / hk, dk, dv, 1, slots, lengths, nullptr, rec};
+#define CALL(T) launch_decode<T, CHAN>(a, DeltaArgs<T>{}, GlaArgs<T>{}, RetArgs<T>{}, ChanArgs<T>{(const T*)x, ldx, (const T*)beta, ldb, (const T*)conv_w, \
+                                       taps, conv, da, (const T*)A_log, (const T*)dt_bias, (const T*)z, ldz}, norm, eps, out, B, st)
+  return MT_BY_TYPE(f32, CALL);
+#undef CALL
+}
+
+// mixed [B*S, 2 hk dk + hv dv]: q | k | v after the convolution
+extern "C" int mt_channel_delta_scan(int f32, const void* mixed, const void* beta, long ldb, const float* da, const void* A_log, const void* dt_bias, int hk,
+                                     int hv, int dk, int dv, int S, float* rec, const int64_t* slots, const int64_t* lengths, const int64_t* new_lens, void* o,
+                                     int B, cudaStream_t st) {
+  if (B <= 0 || S <= 0) return 0;
+  const RecArgs a{hk, hv / hk, dk, dv, S, slots, lengths, new_lens, rec};
+  const long ld = 2L * hk * dk + (long)hv * dv;
+#define CALL(T) launch_scan<T, CHAN>(a, (const T*)mixed, (const T*)mixed + (long)hk * dk, (const T*)mixed + 2L * hk * dk, ld, nullptr, nullptr, 0, nullptr, \
+                                     nullptr, RetArgs<T>{}, ChanArgs<T>{nullptr, 0, (const T*)beta, ldb, nullptr, 1, nullptr, da, (const T*)A_log, \
+                                     (const T*)dt_bias, nullptr, 0}, o, B, st)
+  return MT_BY_TYPE(f32, CALL);
+#undef CALL
 }

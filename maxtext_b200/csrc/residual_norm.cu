@@ -1,7 +1,9 @@
 // The border between two sublayers of a model with an fp32 residual stream and sandwich norms, in one pass per row:
 //   x += mult * rms(branch) * (offset + w_post);    y = rms(x) * (offset + w_next)
 // The branch comes in the compute type (a GEMM output), x stays fp32, y is rounded once for the next GEMM. Without a branch it is the
-// plain norm of the stream. Also here: the ungated activation between the two products of a feed-forward. Bandwidth-bound.
+// plain norm of the stream. residual_join is the same for pre-norm layers: one or two branches, each with a factor, a bias and a norm of its own
+// or without, one factor per lane on their sum, and the stream handed on normalised or as it is. Also here: the ungated activation between the
+// two products of a feed-forward, and the gate of a per-layer token embedding. Bandwidth-bound.
 #include "serving_common.cuh"
 
 namespace mt {
@@ -54,6 +56,109 @@ __global__ void residual_norm_kernel(float* __restrict__ x, const T* __restrict_
   }
 }
 
+struct JoinBranch {
+  const void *out, *bias, *norm;       // [rows, D]; bias [D] or null; norm weight [D] or null: not normalised
+  float factor;
+};
+
+// x += lanes * (a + b);   y = rms(x) * w_next, or x. One CTA per row, a thread holds VEC neighbouring lanes ITER times.
+template <typename T, int VEC, int ITER>
+__global__ void __launch_bounds__(256)
+residual_join_kernel(float* __restrict__ x, const JoinBranch a, const JoinBranch b, const T* __restrict__ lanes, const T* __restrict__ w_next,
+                     T* __restrict__ y, int D, float eps) {
+  __shared__ float red[2][8];
+  const long r = blockIdx.x;
+  const int nt = blockDim.x;
+  float* xr = x + r * D;
+  float add[ITER][VEC], xv[ITER][VEC], t[ITER][VEC];
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int c = (i * nt + threadIdx.x) * VEC;
+    if (c < D) load_vec<VEC>(xr + c, xv[i]);
+  }
+  auto load = [&](const JoinBranch& j, float (&v)[ITER][VEC]) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < ITER; ++i) {
+      const int c = (i * nt + threadIdx.x) * VEC;
+      if (c < D) {
+        load_vec<VEC>(static_cast<const T*>(j.out) + r * D + c, v[i]);
+        if (j.bias) {
+          float w[VEC];
+          load_vec<VEC>(static_cast<const T*>(j.bias) + c, w);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[i][e] += w[e];
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss += v[i][e] * v[i][e];
+      }
+    }
+    return ss;
+  };
+  auto scale = [&](const JoinBranch& j, float (&v)[ITER][VEC], float rstd) {
+#pragma unroll
+    for (int i = 0; i < ITER; ++i) {
+      const int c = (i * nt + threadIdx.x) * VEC;
+      if (c < D) {
+        float w[VEC];
+        if (j.norm) load_vec<VEC>(static_cast<const T*>(j.norm) + c, w);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[i][e] *= j.norm ? j.factor * rstd * w[e] : j.factor;
+      }
+    }
+  };
+  float sa = load(a, add), sb = 0.f;
+  if (b.out) sb = load(b, t);
+  if (a.norm || b.norm) {
+    sa = warp_add(sa);
+    sb = warp_add(sb);
+    if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sa; red[1][threadIdx.x >> 5] = sb; }
+    __syncthreads();
+    sa = sb = 0.f;
+    for (int i = 0; i < (nt + 31) / 32; ++i) { sa += red[0][i]; sb += red[1][i]; }
+  }
+  scale(a, add, rsqrtf(sa / (float)D + eps));
+  if (b.out) {
+    scale(b, t, rsqrtf(sb / (float)D + eps));
+#pragma unroll
+    for (int i = 0; i < ITER; ++i)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) add[i][e] += t[i][e];
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int c = (i * nt + threadIdx.x) * VEC;
+    if (c < D) {
+      float w[VEC];
+      if (lanes) load_vec<VEC>(lanes + c, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        xv[i][e] += lanes ? w[e] * add[i][e] : add[i][e];
+        ss += xv[i][e] * xv[i][e];
+      }
+      store_vec<VEC>(xr + c, xv[i]);
+    }
+  }
+  if (!y) return;
+  float rstd = 1.f;
+  if (w_next) {
+    __syncthreads();                                     // the sums of the branches have been read
+    rstd = rsqrtf(block_add(ss, red[0]) / (float)D + eps);
+  }
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int c = (i * nt + threadIdx.x) * VEC;
+    if (c < D) {
+      float w[VEC];
+      if (w_next) load_vec<VEC>(w_next + c, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) xv[i][e] *= w_next ? rstd * w[e] : 1.f;
+      store_vec<VEC>(y + r * D + c, xv[i]);
+    }
+  }
+}
+
 __device__ __forceinline__ float act_value(float x, int code) {
   switch (code) {
     case 0: return silu_f(x);
@@ -88,6 +193,44 @@ __global__ void act_kernel(const T* __restrict__ x, T* __restrict__ y, long n, i
   if (blockIdx.x == 0 && threadIdx.x < n - nv * 8) y[nv * 8 + threadIdx.x] = from_f<T>(act_typed<T>(to_f(x[nv * 8 + threadIdx.x]), code));
 }
 
+// out[n, c] = gelu_tanh(g[n, c]) * table[token[n], c]
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+token_gate_kernel(const T* __restrict__ g, const T* __restrict__ table, const int64_t* __restrict__ tokens, long N, int dim, long vocab, T* __restrict__ out) {
+  const long per = dim / VEC;
+  for (long i = blockIdx.x * 256l + threadIdx.x; i < N * per; i += gridDim.x * 256l) {
+    const long n = i / per;
+    const int c = (int)(i % per) * VEC;
+    const long tok = min(max((long)tokens[n], 0l), vocab - 1);
+    float v[VEC], e[VEC];
+    load_vec<VEC>(g + n * dim + c, v);
+    load_vec<VEC>(table + tok * dim + c, e);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] = act_value(v[k], 1) * e[k];
+    store_vec<VEC>(out + n * dim + c, v);
+  }
+}
+
+template <typename T>
+int residual_join_t(float* x, const JoinBranch& a, const JoinBranch& b, const void* lanes, const void* w_next, void* y, long rows, int D, float eps,
+                    cudaStream_t st) {
+  auto go = [&](auto kernel, int vec, int iter) {
+    int threads = (((D + vec * iter - 1) / (vec * iter)) + 31) / 32 * 32;
+    if (threads > 256) return -1;
+    kernel<<<(unsigned)rows, threads, 0, st>>>(x, a, b, (const T*)lanes, (const T*)w_next, (T*)y, D, eps);
+    return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  };
+  uintptr_t bits = 0;
+  for (const void* p : {a.out, a.bias, a.norm, b.out, b.bias, b.norm, lanes, w_next, (const void*)x, (const void*)y}) bits |= reinterpret_cast<uintptr_t>(p);
+  if (D % 4 == 0 && bits % 16 == 0) {
+    if (D <= 1024) return go(residual_join_kernel<T, 4, 1>, 4, 1);
+    if (D <= 2048) return go(residual_join_kernel<T, 4, 2>, 4, 2);
+    if (D <= 4096) return go(residual_join_kernel<T, 4, 4>, 4, 4);
+    return go(residual_join_kernel<T, 4, 16>, 4, 16);
+  }
+  return D <= 1024 ? go(residual_join_kernel<T, 1, 4>, 1, 4) : go(residual_join_kernel<T, 1, 32>, 1, 32);
+}
+
 template <typename T>
 int residual_norm_t(float* x, const void* b, const void* wp, float mult, const void* wn, void* y, long rows, int D, float e1, float e2, float off,
                     cudaStream_t st) {
@@ -119,5 +262,26 @@ extern "C" int mt_act_fwd(const void* x, void* y, int f32, long n, int code, int
   const int grid = (int)(blocks < 1 ? 1 : (blocks < (long)sms * 8 ? blocks : (long)sms * 8));
   if (f32) act_kernel<float><<<grid, 256, 0, st>>>((const float*)x, (float*)y, n, code);
   else act_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, n, code);
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int mt_residual_join(float* x, const void* a, const void* a_bias, const void* a_norm, float a_factor, const void* b, const void* b_bias,
+                                const void* b_norm, float b_factor, const void* lanes, const void* w_next, void* y, int f32, long rows, int D, float eps,
+                                cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const JoinBranch ja{a, a_bias, a_norm, a_factor}, jb{b, b_bias, b_norm, b_factor};
+  return f32 ? residual_join_t<float>(x, ja, jb, lanes, w_next, y, rows, D, eps, st) : residual_join_t<__nv_bfloat16>(x, ja, jb, lanes, w_next, y, rows, D, eps, st);
+}
+
+extern "C" int mt_token_gate(const void* g, const void* table, const int64_t* tokens, void* out, int f32, long N, int dim, long vocab, int sms,
+                             cudaStream_t st) {
+  if (N <= 0 || dim <= 0) return 0;
+  const bool v8 = dim % 8 == 0 && (reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+  const long blocks = (N * (dim / (v8 ? 8 : 1)) + 255) / 256;
+  const unsigned grid = (unsigned)(blocks < sms * 8l ? blocks : sms * 8l);
+#define GO(T, V) token_gate_kernel<T, V><<<grid, 256, 0, st>>>((const T*)g, (const T*)table, tokens, N, dim, vocab, (T*)out)
+  if (f32) { if (v8) GO(float, 8); else GO(float, 1); }
+  else { if (v8) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
+#undef GO
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

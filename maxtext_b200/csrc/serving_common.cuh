@@ -101,6 +101,8 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); 
 // for results that are rounded to bf16 a hardware exponential and reciprocal are exact enough
 template <typename T> __device__ __forceinline__ float silu_t(float x) { return silu_f(x); }
 template <> __device__ __forceinline__ float silu_t<__nv_bfloat16>(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+template <typename T> __device__ __forceinline__ float sigmoid_t(float x) { return sigmoid_f(x); }
+template <> __device__ __forceinline__ float sigmoid_t<__nv_bfloat16>(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 

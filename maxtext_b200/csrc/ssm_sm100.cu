@@ -42,7 +42,12 @@ conv_kernel(const T* __restrict__ x, long ldx, const T* __restrict__ w, const T*
   const T* xb = x + (long)b * S * ldx + c;
   T* yb = y + (long)b * S * C + c;
   float bv[VEC];
-  load_vec<VEC>(bias + c, bv);
+  if (bias) {
+    load_vec<VEC>(bias + c, bv);
+  } else {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) bv[e] = 0.f;
+  }
   // input at token s (negative: history)
   auto at = [&](int s, float (&v)[VEC]) {
     if (s >= 0) load_vec<VEC>(xb + (long)s * ldx, v);

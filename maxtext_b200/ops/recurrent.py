@@ -1,6 +1,7 @@
-"""Inference kernels of the recurrent layers (gated delta network, gated linear attention): `csrc/recurrent_sm100.cu`.
+"""Inference kernels of the recurrent layers (gated delta network, gated linear attention, retention, channel-wise gated delta rule):
+`csrc/recurrent_sm100.cu`, `csrc/recurrent_chunk_sm100.cu`.
 
-Both layers keep a matrix state per head; the kernels take the layer's raw projections and return its gated, normalised head outputs
+All of them keep a matrix state per head; the kernels take the layer's raw projections and return its gated, normalised head outputs
 [B, S, H * Dv] ready for the output projection. One token per sequence is one fused launch (convolution, gates, state update,
 read-out, norm); longer inputs run convolution -> recurrence -> norm. States are read and written in the rows `slot_ids` of the
 layer's `RecurrentState`; rows with `lengths` 0 start from zero, and only the first `new_lens` tokens of a row count.
@@ -78,3 +79,45 @@ def gla_forward(layer, p, st):
   scan(p2, log_alpha, H, dk, dv, S, st.rec, st.slot_ids, st.lengths, st.new_lens, o)
   E.gated_head_norm(o, p2, H, dv, 1, 2 * H * dk + H * dv, dv, layer.norm.data, eps, out.view(N, -1))
   return out
+
+
+def retention_forward(layer, p, B, S, st):
+  """layer: Retention; p [B*S, >= 2H(dk+dv)] rows of the input projection."""
+  E = backend.ext()
+  H, dk, dv = layer.heads, layer.dk, layer.dv
+  eps = float(layer.c.normalization_layer_epsilon)
+  out = torch.empty(B * S, H * dv, dtype=p.dtype, device=p.device)
+  turn = (layer.log_decay, layer.inv_ts, layer.rot)
+  if S == 1:
+    E.retention_decode(p, *turn, eps, H, dk, dv, st.rec, st.slot_ids, st.lengths, out)
+    return out.view(B, S, -1)
+  o = torch.empty(B * S, H * dv, dtype=p.dtype, device=p.device)
+  chunked = chunked_ok(p, S, dk, dv) and p.stride(0) % 8 == 0 and p.data_ptr() % 16 == 0
+  (E.retention_chunks if chunked else E.retention_scan)(p, *turn, H, dk, dv, S, st.rec, st.slot_ids, st.lengths, st.new_lens, o)
+  E.gated_head_norm(o, p, H, dv, 1, 2 * H * dk + H * dv, dv, None, eps, out)
+  return out.view(B, S, -1)
+
+
+def channel_delta_forward(layer, p, B, S, st):
+  """layer: ChannelDeltaNet; p [B*S, >= sum(columns)] rows of the input projection."""
+  from . import functional as F
+  E, s = backend.ext(), layer.s
+  N, dev, dt = B * S, p.device, p.dtype
+  eps = float(layer.c.normalization_layer_epsilon)
+  qkv, beta, a1, g1 = torch.split(p, s.columns, dim=-1)
+  # the decay's fp32 accumulators go straight into softplus
+  da = F.mm(a1, layer.decay.data, False, True, out_dtype=torch.float32)
+  z = F.mm(g1, layer.gate.data, False, True)
+  out = torch.empty(N, s.hv * s.dv, dtype=dt, device=dev)
+  w = layer.conv.data.view(s.taps, s.conv_dim)
+  if S == 1:
+    E.channel_delta_decode(qkv, beta, w, da, layer.A_log.data, layer.dt_bias.data, z, layer.norm.data, eps, s.hk, s.hv, s.dk, s.dv, st.conv, st.rec,
+                           st.slot_ids, st.lengths, out)
+    return out.view(B, S, -1)
+  mixed = torch.empty(N, s.conv_dim, dtype=dt, device=dev)
+  E.ssm_conv(qkv, w, None, S, st.conv, st.slot_ids, st.lengths, st.new_lens, mixed)
+  o = torch.empty(N, s.hv * s.dv, dtype=dt, device=dev)
+  E.channel_delta_scan(mixed, beta, da, layer.A_log.data, layer.dt_bias.data, s.hk, s.hv, s.dk, s.dv, S, st.rec, st.slot_ids, st.lengths, st.new_lens, o,
+                       chunked_ok(mixed, S, s.dk, s.dv) and s.conv_dim % 8 == 0)
+  E.gated_head_norm(o, z, s.hv, s.dv, 1, 0, s.dv, layer.norm.data, eps, out, True)
+  return out.view(B, S, -1)
