@@ -406,7 +406,7 @@ class Attention:
     self.lam = None
     if self.maps == 2:
       assert tp == 1, "differential attention is not split over the tensor axis"
-      self.lam = [ab.sub("lambda").vector(n, self.dh, ("norm",), init="zeros") for n in ("q1", "k1", "q2", "k2")]
+      self.lam = [ab.sub("lambda").vector(n, self.dh, ("norm",), init="fan_in_normal") for n in ("q1", "k1", "q2", "k2")]
 
   def sink_data(self, dtype):
     """The sink scores in the compute type, or None."""

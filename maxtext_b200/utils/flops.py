@@ -79,10 +79,27 @@ def _sized_mixer(bp, B, S, d):
   if bp.attention == "ssm":
     c, n, r = m["inner"], m["state"], m["dt_rank"]
     return 2 * bs * (3 * d * c + c * (r + 2 * n) + r * c + m["conv"] * c), 7 * bs * c * n
+  if bp.attention == "parallel":
+    left, right = (_sized_mixer(p, B, S, d) for p in bp.pair)
+    return left[0] + right[0], left[1] + right[1]
   H, dv = m["heads"], m["vdim"]
   if bp.attention == "gqa":
-    w = d * (H * m["dim"] + m["kv_heads"] * (m["dim"] + dv) + 2 * H * dv)
-    return 2 * bs * w, bs * S * H * (m["dim"] + dv)
+    maps = 2 if "diff" in m else 1
+    w = d * (H * maps * m["dim"] + m["kv_heads"] * (maps * m["dim"] + dv) + H * dv + (H if bp.gate == "head" else H * dv))
+    size = int(m["mask"]["size"]) if bp.mask else 0
+    if bp.mask == "window":
+      pairs = S * min(size, S) - 0.5 * min(size, S) ** 2
+    elif bp.mask == "chunk":
+      n, rem = divmod(S, size)
+      pairs = (n * size ** 2 + rem ** 2) / 2
+    else:
+      pairs = S * S / 2
+    return 2 * bs * w, 2 * B * pairs * H * maps * (m["dim"] + dv)
+  if bp.attention == "retention":
+    return 2 * bs * d * (2 * H * m["dim"] + 3 * H * dv), bs * H * m["dim"] * dv * 5
+  if bp.attention == "channel_delta":
+    kd, ra, rg = m["kv_heads"] * m["dim"], m["decay_rank"], m["gate_rank"]
+    return 2 * bs * (d * (2 * kd + 2 * H * dv + H + ra + rg) + ra * H * m["dim"] + rg * H * dv + m["conv"] * (2 * kd + H * dv)), bs * H * m["dim"] * dv * 8
   if bp.attention == "mla":
     qk = m["dim"] + m["rot_dim"]
     w = d * m["q_rank"] + m["q_rank"] * H * qk + d * (m["kv_rank"] + m["rot_dim"]) + m["kv_rank"] * H * (m["dim"] + dv) + H * dv * d
@@ -140,6 +157,8 @@ def _block(c, bp, B, S, n_act):
       ffn += _ffn(bs, d, c.mlp_dim, n_act)                                         # the dense MLP next to the routed experts
   else:
     ffn = _ffn(bs, d, int(bp.mlp_hidden or c.mlp_dim), n_act)
+  if bp.token_side:
+    ffn += 4 * bs * d * bp.token_side
   return proj_w + ffn, attn
 
 
