@@ -6,7 +6,7 @@
   decode:  tokens/s of a full decode state per slot count, every slot holding `context` tokens, CUDA-graph replay
   kernels: device microseconds per launch by kernel (PyTorch profiler, a separate untimed pass), one prompt and one decode step
 
-and one last line `rooflines`: every serving kernel at silinex-1b's and tipidra-1b's layer sizes (8192 prompt tokens; 128 sequences with 2048 cached tokens),
+and one last line `rooflines`: every serving kernel at the layer sizes of silinex-1b, tipidra-1b and sitivik-1b (8192 prompt tokens; 128 sequences with 2048 cached tokens),
 its time by CUDA events with L2 flushed, its algorithmic bytes or products, and the fraction of the measured copy bandwidth or GEMM rate,
 beside the like operation of the models that existed before (`like`).
 
@@ -19,6 +19,8 @@ Weights are random; the work does not depend on their values. The models:
   tipidra-1b   the catalog entry: capped attention and selective-scan layers in turn, every other pair with routed experts, two residual streams
   moe-1b       the same width, depth and active weights with the Mixtral block (grouped-query attention, routed experts in every layer)
   tipidra-5b, moe-5b   the same two at width 4096, 32 heads, 24 layers
+  sitivik-1b   the catalog entry: windowed attention beside retention, chunked attention beside the channel-wise gated delta rule, differential attention
+  sitivik-5b   the same at width 4096, 32 heads, 24 layers
 """
 from __future__ import annotations
 
@@ -67,6 +69,21 @@ def _moe(width, heads, expert_ff, layers):
               base_moe_mlp_dim=expert_ff, num_experts=16, num_experts_per_tok=2, base_num_decoder_layers=layers, vocab_size=65536, logits_via_embedding=False)
 
 
+def _sitivik(width, heads, ff, layers):
+  """Pairs (window 2048 beside retention, chunks of 2048 beside the channel-wise delta rule) and differential attention in turn."""
+  rot = {"base": 500000.0, "dims": 128}
+  left = {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 2048}, "rot": rot}
+  stretched = {**left, "rot": {**rot, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+  ret = {"heads": heads, "dim": 64, "vdim": 128, "rot": {"base": 10000.0, "dims": 64}, "decay": [1.0 - 2.0 ** (-5.0 - 5.0 * i / (heads - 1)) for i in range(heads)]}
+  delta = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128, "gate_rank": 128}
+  diff = {"heads": heads, "kv_heads": heads // 4, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.4, "q_temp": {"coef": 0.1, "every": 8192}}
+  kinds = [("parallel", {"left": stretched, "right": ret}), ("attention", diff), ("parallel", {"left": stretched, "right": ret}),
+           ("parallel_2", {"left": left, "right": delta, "left_scale": 0.7, "right_scale": 0.7})]
+  return dict(decoder_block="sitivik", base_emb_dim=width, base_num_decoder_layers=layers, token_side_dim=64, vocab_size=65536, logits_via_embedding=True,
+              normalize_embedding_logits=False, mlp_activations=["silu", "linear"], embedding_multiplier=width ** 0.5,
+              layer_specs=[{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)])
+
+
 MODELS = {
     "silinex-1b": dict(model_name="silinex-1b"),
     "mla-1b": _plain(2048, 16, 8192, 18, 768),
@@ -77,6 +94,8 @@ MODELS = {
     "moe-1b": _moe(2048, 16, 2560, 16),
     "tipidra-5b": _tipidra(4096, 32, 12288, 4096, 24),
     "moe-5b": _moe(4096, 32, 5120, 24),
+    "sitivik-1b": dict(model_name="sitivik-1b"),
+    "sitivik-5b": _sitivik(4096, 32, 9216, 24),
 }
 
 
@@ -277,6 +296,44 @@ def rooflines(iters: int = 10) -> dict:
   plan = moe_ops.GroupPlan(idx, nE)
   gu, he = t(plan.rows_max, 2 * Fe), t(plan.rows_max, Fe)
   add("expert_act", lambda: E.expert_act(gu, wts.view(-1), plan.row_pair, plan.offs, 7.0, he), 6 * N * top * Fe, like="gated_act")
+  # two mixers side by side, retention, channel-wise delta rule, differential attention
+  b2 = t(N, D)
+  add("residual_join, two normed branches", lambda: E.residual_join(x32, b, w, w, 0.5, b2, None, w, 0.5, w, w, y, 1e-6), N * D * (8 + 3 * 2), like="residual_norm")
+  add("residual_join, one branch", lambda: E.residual_join(x32, b, None, None, 1.0, None, None, None, 1.0, w, w, y, 1e-6), N * D * (8 + 2 * 2), like="residual_norm")
+  sg, stab, stok, so = t(N, 64), t(65536, 64), torch.randint(0, 65536, (N,), device=dev), t(N, 64)
+  add("token_gate", lambda: E.token_gate(sg, stab, stok, so), 6 * N * 64, like="gated_act, small")
+  add("gated_act, small", lambda: E.gated_act_fwd(so, sg.view(-1)[: N * 32].view(N, 32), 0), 3 * N * 64)
+  qb, kb_, vb_, qnw, knw, inv128, vo = t(HQ * hd), t(HG * hd), t(HG * hd), t(HQ * hd), t(HG * hd), torch.rand(64, device=dev), t(N, HG, hd)
+  add("qkv_prep, bias, norm over all heads, pairs", lambda: E.qkv_prep(qs, ks, vs, hd, hd, pos0, inv128, 128, 1e-5, qo, ko, vo, ck, cv, one, one, None, qb, kb_, vb_, qnw,
+                                                                       knw, True, 1, 0.0, 0.0), 2 * N * hd * (2 * HQ + 6 * HG), like="qkv_prep")
+  add("qkv_prep, bias, norm per head, pairs", lambda: E.qkv_prep(qs, ks, vs, hd, hd, pos0, inv128, 128, 1e-5, qo, ko, vo, ck, cv, one, one, None, qb, kb_, vb_, qnw[:hd],
+                                                                 knw[:hd], True, 1, 0.0, 0.0), 2 * N * hd * (2 * HQ + 6 * HG), like="qkv_prep")
+  q2o = t(N, 2 * HQ, hd)
+  add("qkv_prep, two maps, temperature", lambda: E.qkv_prep(qs, ks, vs, 64, hd, pos0, None, 0, -1.0, q2o, ko, vo, ck, cv, one, one, None, qb, kb_, vb_, None, None, False, 2,
+                                                            0.1, 8192.0), 2 * N * hd * (3 * HQ + 6 * HG), like="qkv_prep")
+  with torch.no_grad():
+    add("flash forward, window 2048, 128", lambda: F.attention_fwd(qn, kn, vo[None], None, None, 0.09, 0.0, win), 0, 2 * pairs * HQ * 2 * hd,
+        like="flash forward, window 2048")
+    cpairs = N * 2048 // 2
+    add("flash forward, chunks of 2048, sink", lambda: F.attention_fwd(qn, kn, vo[None], None, None, 0.09, 0.0, 0, chunk=2048, sinks=sink), 0,
+        2 * cpairs * HQ * 2 * hd, like="flash forward, window 2048")
+    q2n = q2o[None] * 0.1
+    add("flash forward, two maps of 64", lambda: F.attention_fwd(q2n, kn, vo[None], None, None, 0.12, 0.0, 0), 0, N * N * 2 * HQ * (64 + hd),
+        like="flash forward, causal, 128")
+  o2, lam = t(N, 2 * HQ, hd), [t(64) * 0.1 for _ in range(4)]
+  gh = t(N, 64)
+  add("diff_combine", lambda: E.diff_combine(o2, lam, 0.4, 1e-6, gh, hd, go_, True), 2 * N * hd * 3 * HQ, like="head_gate")
+  rx, rrec, ro = t(N, 2 * H * (gk + dv)), t(1, H, gk, dv, dtype=torch.float32), t(N, H * dv)
+  ld, rinv = torch.log(torch.rand(H, device=dev) * 0.05 + 0.95), torch.rand(gk // 2, device=dev)
+  add("retention_chunks (both kernels)", lambda: E.retention_chunks(rx, ld, rinv, gk, H, gk, dv, N, rrec, one, one, None, ro), 2 * N * 2 * H * (gk + dv),
+      like="gla_chunks (both kernels)")
+  ccd = H * 3 * 128
+  cmix, cbeta, cda, cA, cdt = t(N, ccd), t(N, H), t(N, H * 128, dtype=torch.float32), t(H) * 0.1 - 1.0, t(H * 128)
+  crec, cconv, craw, ccw = t(1, H, 128, 128, dtype=torch.float32), t(1, 3, ccd, dtype=torch.float32), t(N, ccd + 512), t(4, ccd)
+  add("channel_delta_scan, chunks (both kernels)", lambda: E.channel_delta_scan(cmix, cbeta, cda, cA, cdt, H, H, 128, 128, N, crec, one, one, None, ro, True),
+      N * H * (2 * 4 * 128 + 4 * 128 + 2), like="delta_chunks (both kernels)")
+  add("ssm_conv, no bias", lambda: E.ssm_conv(craw[:, :ccd], ccw, None, N, cconv, one, one, None, cmix), 4 * N * ccd, like="delta_conv")
+  add("gated_head_norm, sigmoid", lambda: E.gated_head_norm(ro, go_, H, 128, 1, 0, 128, nw, 1e-6, o, True), 6 * N * H * 128, like="gated_head_norm")
   # ---- decoding: 128 sequences, 2048 cached tokens
   B, L = 128, 2048
   ids, lens = torch.arange(B, device=dev), longs(B, L - 1)
@@ -324,6 +381,20 @@ def rooflines(iters: int = 10) -> dict:
     pt, ml2, od = t(Bd, HQ, sp, hd, dtype=torch.float32), t(Bd, HQ, sp, 2, dtype=torch.float32), t(Bd, HQ * hd)
     add(f"cached_decode, {Bd} sequences", lambda: E.cached_decode(q16[:Bd], kc4[:Bd], vc4[:Bd], ids[:Bd], lens[:Bd], 0.09, 40.0, 0, sinkb, g16[:Bd], sp, pt, ml2, od),
         2 * 2 * Bd * L * HG * hd, like="mla_decode_attn")
+  q32, ghd = t(B, 2 * HQ, hd), t(B, HQ)
+  for Bd in (1, 128):
+    sp = E.cached_decode_splits(Bd, 2 * HQ, HG, L)
+    pt, ml2, od = t(Bd, 2 * HQ, sp, hd, dtype=torch.float32), t(Bd, 2 * HQ, sp, 2, dtype=torch.float32), t(Bd, HQ * hd)
+    add(f"cached_decode, two maps, {Bd} sequences", lambda: E.cached_decode(q32[:Bd], kc4[:Bd], vc4[:Bd], ids[:Bd], lens[:Bd], 0.12, 0.0, 0, None, ghd[:Bd], sp, pt, ml2,
+                                                                           od, per_head=True, lam=lam, diff=0.4, eps=1e-6), 2 * 2 * Bd * L * HG * hd,
+        like=f"cached_decode, {Bd} sequences")
+  brr = t(B, H, gk, dv, dtype=torch.float32)
+  add("retention_decode", lambda: E.retention_decode(rx[:B], ld, rinv, gk, 1e-6, H, gk, dv, brr, ids, lens, dout), 8 * B * H * gk * dv, like="gla_decode")
+  bcr, bcc = t(B, H, 128, 128, dtype=torch.float32), t(B, 3, ccd, dtype=torch.float32)
+  add("channel_delta_decode", lambda: E.channel_delta_decode(craw[:B, :ccd], cbeta[:B], ccw, cda[:B], cA, cdt, go_[:B], nw, 1e-6, H, H, 128, 128, bcc, bcr, ids, lens,
+                                                             dout), 8 * B * H * 128 * 128 + 8 * B * 3 * ccd, like="delta_decode")
+  add("residual_join, 128 tokens", lambda: E.residual_join(x32[:B], b[:B], w, w, 0.5, b2[:B], None, w, 0.5, w, w, y[:B], 1e-6), B * D * 14,
+      like="rmsnorm, 128 tokens")
   add("stream_mix, 128 tokens", lambda: E.stream_mix(xs[:B], b[:B], None, 1, mix, wr, wr, w, w, y[:B], 1e-5), B * D * (2 * 2 * 4 + 4), like="rmsnorm, 128 tokens")
   add("rmsnorm, 128 tokens", lambda: E.rmsnorm_fwd(b[:B], w, 1e-6, 0.0, y[:B], None), 4 * B * D)
   return {"rooflines": rows, "hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "peaks": peaks["source"]}
