@@ -186,6 +186,153 @@ qkv_prep_kernel(const PrepArgs a) {
   }
 }
 
+// The same for head widths up to 8 * LPH that are multiples of 8: LPH lanes share a head, a warp takes 32 / LPH heads at a time, and the lanes that
+// rotate together meet by a shuffle. (Halves that are paired begin at a multiple of 8.)
+template <typename T, int LPH>
+__global__ void __launch_bounds__(128)
+qkv_prep_wide_kernel(const PrepArgs a) {
+  constexpr int VEC = 8, STEP = 4 * (32 / LPH);
+  extern __shared__ float2 cs[];                            // (cos, sin) of the rot / 2 angles
+  __shared__ float red[2][4];
+  const long n = blockIdx.x;
+  const int b = (int)(n / a.S), s = (int)(n % a.S), half = a.rot / 2, D = a.D, HM = a.H * a.maps, GM = a.G * a.maps, all = HM + GM;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, e0 = (lane % LPH) * VEC, first = warp * (32 / LPH) + lane / LPH;
+  const bool on = e0 < D;
+  auto raw = [&](int h, float (&x)[VEC]) {                  // elements of head h (keys follow the queries) with their bias
+    const bool key = h >= HM;
+    const int head = key ? h - HM : h;
+    if (on && h < all) {
+      load_vec<VEC>(static_cast<const T*>(key ? a.k : a.q) + n * (key ? a.ldk : a.ldq) + (long)head * D + e0, x);
+      const T* bias = static_cast<const T*>(key ? a.bk : a.bq);
+      if (bias) {
+        float y[VEC];
+        load_vec<VEC>(bias + (long)head * D + e0, y);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] += y[e];
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] = 0.f;
+    }
+  };
+  float x[VEC];
+  raw(first, x);
+  const float p = (float)a.pos[n];
+  const long at = a.lengths[b] + s;
+  const bool keep = at < a.max_len && s < (a.new_lens ? a.new_lens[b] : (int64_t)a.S);
+  const long row = a.slots[b] * a.max_len + at;
+  if (keep || a.vp) {
+    T *vc = static_cast<T*>(a.vc), *vp = static_cast<T*>(a.vp);
+    for (int i = threadIdx.x * VEC; i < a.G * a.Dv; i += 128 * VEC) {
+      float v[VEC];
+      load_vec<VEC>(static_cast<const T*>(a.v) + n * a.ldv + i, v);
+      if (a.bv) {
+        float y[VEC];
+        load_vec<VEC>(static_cast<const T*>(a.bv) + i, y);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] += y[e];
+      }
+      if (keep) store_vec<VEC>(vc + row * a.G * a.Dv + i, v);
+      if (vp) store_vec<VEC>(vp + (n * a.G + i / a.Dv) * a.dvp + i % a.Dv, v);
+    }
+    if (vp && a.dvp > a.Dv) {
+      const int pad = (a.dvp - a.Dv) / VEC;
+      const float zero[VEC] = {};
+      for (int i = threadIdx.x; i < a.G * pad; i += 128) store_vec<VEC>(vp + (n * a.G + i / pad) * a.dvp + a.Dv + (i % pad) * VEC, zero);
+    }
+  }
+  for (int i = threadIdx.x; i < half; i += 128) {
+    float sn, c;
+    sincosf(p * a.inv_ts[i], &sn, &c);
+    cs[i] = make_float2(c, sn);
+  }
+  const float warm = a.temp_every > 0.f ? 1.f + a.temp_coef * logf(floorf((p + 1.f) / a.temp_every) + 1.f) : 1.f;
+  if (a.norm == NORM_ALL) {
+    float sq = 0.f, sk = 0.f;
+    for (int h = first; h < all; h += STEP) {
+      float y[VEC], t = 0.f;
+      raw(h, y);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) t += y[e] * y[e];
+      if (h >= HM) sk += t; else sq += t;
+    }
+    sq = warp_add(sq);
+    sk = warp_add(sk);
+    if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  }
+  __syncthreads();
+  float rstd_q = 1.f, rstd_k = 1.f;
+  if (a.norm == NORM_ALL) {
+    rstd_q = rsqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)(HM * D) + a.eps);
+    rstd_k = rsqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)(GM * D) + a.eps);
+  }
+  for (int h0 = 0; h0 < all; h0 += STEP) {                  // every lane takes part in the shuffles
+    const int h = h0 + first;
+    const bool key = h >= HM, live = on && h < all;
+    const int head = key ? h - HM : h;
+    float next[VEC];
+    raw(h + STEP, next);
+    float r = key ? rstd_k : rstd_q;
+    if (a.norm == NORM_HEAD || a.norm == NORM_AFTER) {      // a rotation leaves the norm as it is
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += x[e] * x[e];
+#pragma unroll
+      for (int w = LPH / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+      r = rsqrtf(ss / (float)D + a.eps);
+    }
+    if (a.norm >= NORM_HEAD && live) {
+      float g[VEC];
+      load_vec<VEC>(static_cast<const T*>(key ? a.wk : a.wq) + (a.norm == NORM_ALL ? (long)head * D : 0) + e0, g);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] *= r * g[e];
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] *= r;
+    }
+    if (a.rot && a.paired) {
+#pragma unroll
+      for (int e = 0; e < VEC; e += 2) {
+        if (e0 + e < a.rot) {
+          const float2 c = cs[(e0 + e) / 2];
+          const float u = x[e], v = x[e + 1];
+          x[e] = u * c.x - v * c.y;
+          x[e + 1] = v * c.x + u * c.y;
+        }
+      }
+    } else if (a.rot) {
+      const bool turn = e0 < a.rot, low = e0 < half;
+      const int src = (lane & ~(LPH - 1)) | ((turn ? (low ? e0 + half : e0 - half) : e0) / VEC);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const float y = __shfl_sync(0xffffffffu, x[e], src);
+        if (turn) {
+          const float2 c = cs[(low ? e0 : e0 - half) + e];
+          x[e] = x[e] * c.x + (low ? -y : y) * c.y;
+        }
+      }
+    }
+    const int m = head % a.maps;                            // this map's lanes of the head
+    if (live) {
+      if (!key) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] *= warm;
+      }
+      T* dst = key ? (a.kp ? static_cast<T*>(a.kp) + (n * a.G + head / a.maps) * a.dq : nullptr) : static_cast<T*>(a.qp) + (n * HM + head) * a.dq;
+      if (dst) store_vec<VEC>(dst + m * D + e0, x);
+      if (key && keep) store_vec<VEC>(static_cast<T*>(a.kc) + (row * GM + head) * D + e0, x);
+    }
+    if (h < all && (key ? a.kp && m == a.maps - 1 && a.dq > a.maps * D : a.dq > D)) {
+      T* dst = key ? static_cast<T*>(a.kp) + (n * a.G + head / a.maps) * a.dq : static_cast<T*>(a.qp) + (n * HM + head) * a.dq;
+      const float zero[VEC] = {};
+      for (int z = e0; z < a.dq; z += LPH * VEC)
+        if (z >= (m + 1) * D || (!key && z < m * D)) store_vec<VEC>(dst + z, zero);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[e] = next[e];
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ decode
 struct DecodeArgs {
   const __nv_bfloat16 *q, *k, *v;      // q [B, H, D]
@@ -407,21 +554,6 @@ __device__ __forceinline__ float diff_lambda(const DiffArgs& a, int lane) {
   return expf(warp_add(s1)) - expf(warp_add(s2)) + a.diff;
 }
 
-// a head's lanes, held NV per thread by the nt threads of the group that owns it: (map 1 - lambda map 2) over its root mean square
-// times (1 - diff) and the gate. The sum over the group comes from `add`.
-template <typename T, int NV, typename Add>
-__device__ __forceinline__ void diff_finish(float (&x)[NV], const DiffArgs& a, int Dv, const T* gate, int per_head, int t, int nt, Add add, T* out) {
-  float ss = 0.f;
-#pragma unroll
-  for (int j = 0; j < NV; ++j) ss += x[j] * x[j];
-  const float r = rsqrtf(add(ss) / (float)Dv + a.eps) * (1.f - a.diff);
-#pragma unroll
-  for (int j = 0; j < NV; ++j) {
-    const int d = t + j * nt;
-    if (d < Dv) out[d] = from_f<T>(x[j] * r * (gate ? sigmoid_f(to_f(gate[per_head ? 0 : d])) : 1.f));
-  }
-}
-
 // decode: grid (heads, B), 128 threads. The maps of head h are the query heads 2 h and 2 h + 1 of `part`
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -448,29 +580,60 @@ diff_merge_kernel(const float* __restrict__ part, const float* __restrict__ ml, 
     x[0] += f * o[0];
     x[1] += f * o[1];
   }
-  const long g0 = b * ldg + (per_head ? h : (long)h * Dv);
-  diff_finish<T, 2>(x, a, Dv, gate ? gate + g0 : nullptr, per_head, t, 128, [&](float v) { return block_add(v, red); }, out + ((long)b * H + h) * Dv);
+  const float r = rsqrtf(block_add(x[0] * x[0] + x[1] * x[1], red) / (float)Dv + a.eps) * (1.f - a.diff);
+  const T* g = gate ? gate + b * ldg + (per_head ? h : (long)h * Dv) : nullptr;
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int d = t + j * 128;
+    if (d < Dv) out[((long)b * H + h) * Dv + d] = from_f<T>(x[j] * r * (g ? sigmoid_f(to_f(g[per_head ? 0 : d])) : 1.f));
+  }
 }
 
-// prompts: a warp per token and head; o [N, 2 H, dvp] -> out [N, H * Dv]
-template <typename T, int NV>
+// prompts: LPR lanes per token and head, VEC neighbouring elements each, NV times; o [N, 2 H, dvp] -> out [N, H * Dv]
+template <typename T, int VEC, int LPR, int NV>
 __global__ void __launch_bounds__(256)
 diff_combine_kernel(const T* __restrict__ o, int dvp, const DiffArgs a, long N, int H, int Dv, const T* __restrict__ gate, long ldg, int per_head,
                     T* __restrict__ out) {
-  const int lane = threadIdx.x & 31;
+  const int lane = threadIdx.x & 31, t = lane % LPR;
   const float lam = diff_lambda<T>(a, lane);
-  for (long i = (blockIdx.x * 256l + threadIdx.x) >> 5; i < N * H; i += gridDim.x * 8l) {
-    const long n = i / H;
-    const int h = (int)(i % H);
+  const long rows = N * H, step = gridDim.x * (256l / LPR);
+  for (long i = (blockIdx.x * 256l + threadIdx.x) / LPR; i - lane / LPR < rows; i += step) {         // a warp leaves the loop together
+    const bool in = i < rows;
+    const long n = in ? i / H : 0;
+    const int h = in ? (int)(i % H) : 0;
     const T* o1 = o + (n * 2 * H + 2 * h) * dvp;
-    float x[NV];
+    float x[NV][VEC], ss = 0.f;
 #pragma unroll
     for (int j = 0; j < NV; ++j) {
-      const int d = lane + j * 32;
-      x[j] = d < Dv ? to_f(o1[d]) - lam * to_f(o1[dvp + d]) : 0.f;
+      const int d = (j * LPR + t) * VEC;
+      if (d < Dv) {
+        float y[VEC];
+        load_vec<VEC>(o1 + d, x[j]);
+        load_vec<VEC>(o1 + dvp + d, y);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          x[j][e] -= lam * y[e];
+          ss += x[j][e] * x[j][e];
+        }
+      }
     }
-    const long g0 = n * ldg + (per_head ? h : (long)h * Dv);
-    diff_finish<T, NV>(x, a, Dv, gate ? gate + g0 : nullptr, per_head, lane, 32, [](float v) { return warp_add(v); }, out + i * Dv);
+#pragma unroll
+    for (int w = LPR / 2; w > 0; w >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w);
+    if (!in) continue;
+    float r = rsqrtf(ss / (float)Dv + a.eps) * (1.f - a.diff);
+    const T* g = gate ? gate + n * ldg + (per_head ? h : (long)h * Dv) : nullptr;
+    if (g && per_head) r *= sigmoid_f(to_f(g[0]));
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int d = (j * LPR + t) * VEC;
+      if (d < Dv) {
+        float z[VEC];
+        if (g && !per_head) load_vec<VEC>(g + d, z);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[j][e] *= g && !per_head ? r * sigmoid_f(z[e]) : r;
+        store_vec<VEC>(out + i * Dv + d, x[j]);
+      }
+    }
   }
 }
 
@@ -603,6 +766,11 @@ int prep_t(const PrepArgs& a, long N, cudaStream_t st) {
     return cudaGetLastError() == cudaSuccess ? 0 : -3;
   };
   if (a.D > 512) return -1;
+  const bool v8 = a.D % 8 == 0 && a.Dv % 8 == 0 && (a.paired || a.rot % 16 == 0) && a.dq % 8 == 0 && a.ldq % 8 == 0 && a.ldk % 8 == 0 && a.ldv % 8 == 0 &&
+                  (!a.vp || a.dvp % 8 == 0) && bits % 16 == 0;
+  if (v8 && a.D <= 64) return launch(qkv_prep_wide_kernel<T, 8>);
+  if (v8 && a.D <= 128) return launch(qkv_prep_wide_kernel<T, 16>);
+  if (v8 && a.D <= 256) return launch(qkv_prep_wide_kernel<T, 32>);
   if (!v4) return launch(qkv_prep_kernel<T, 1, 16>);
   if (a.D <= 128) return launch(qkv_prep_kernel<T, 4, 1>);
   if (a.D <= 256) return launch(qkv_prep_kernel<T, 4, 2>);
@@ -697,12 +865,18 @@ extern "C" int mt_diff_combine(int f32, const void* o, int dvp, const DiffArgs* 
                                int sms, cudaStream_t st) {
   if (N <= 0) return 0;
   if (Dv > 256) return -1;
-  const long blocks = (N * H + 7) / 8;
-  const unsigned grid = (unsigned)(blocks < sms * 16l ? blocks : sms * 16l);
-#define GO(T, NV) diff_combine_kernel<T, NV><<<grid, 256, 0, st>>>((const T*)o, dvp, *a, N, H, Dv, (const T*)gate, ldg, per_head, (T*)out)
-  if (Dv <= 64) { if (f32) GO(float, 2); else GO(bf16, 2); }
-  else if (Dv <= 128) { if (f32) GO(float, 4); else GO(bf16, 4); }
-  else { if (f32) GO(float, 8); else GO(bf16, 8); }
+  const bool v8 = Dv % 8 == 0 && dvp % 8 == 0 && (per_head || !gate || (ldg % 8 == 0 && reinterpret_cast<uintptr_t>(gate) % 16 == 0));
+  auto grid = [&](int lpr) {
+    const long blocks = (N * H * lpr + 255) / 256;
+    return (unsigned)(blocks < sms * 16l ? blocks : sms * 16l);
+  };
+#define GO(T, VEC, LPR, NV) diff_combine_kernel<T, VEC, LPR, NV><<<grid(LPR), 256, 0, st>>>((const T*)o, dvp, *a, N, H, Dv, (const T*)gate, ldg, per_head, (T*)out)
+#define BY(VEC, LPR, NV) do { if (f32) GO(float, VEC, LPR, NV); else GO(bf16, VEC, LPR, NV); } while (0)
+  if (!v8) BY(1, 32, 8);
+  else if (Dv <= 64) BY(8, 8, 1);
+  else if (Dv <= 128) BY(8, 16, 1);
+  else BY(8, 32, 1);
+#undef BY
 #undef GO
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

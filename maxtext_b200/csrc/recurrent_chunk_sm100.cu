@@ -467,27 +467,32 @@ __global__ void __launch_bounds__(256) retention_chunk_prepare_kernel(ChunkArgs 
 }
 
 // ------------------------------------------------------------------------------------------------ channel-wise gated delta: prepare
-// grid (chunks, H, B), 512 threads. mixed: q | k | v after the convolution; da fp32 [B*S, H*dk]: product of the decay projection. tp: T high, T low,
+// grid (chunks, H, B), 256 threads. mixed: q | k | v after the convolution; da fp32 [B*S, H*dk]: product of the decay projection. tp: T high, T low,
 // P high, P low as for the gated delta rule; qkg: six [64][dk] tiles: k e^G, q e^G, k e^(G_end - G), each high, low; betas [64]; end: e^G_end [dk].
+//
+// Warp (I, which) owns the 16 rows of block I of P (which 0, rows of q) or of L (1, rows of k). Its rows, scaled by e^(G - r_I) with r_I the sum at
+// the last token before the block, stay in registers as fragments; the keys of block J sit in shared memory scaled by e^(G_end(J) - G), so that
+// blocks I and J meet through the factor e^(r_I - G_end(J)), which is one for neighbours. No factor exceeds one.
 template <int DK>
-__global__ void __launch_bounds__(512) channel_chunk_prepare_kernel(ChunkArgs a, const bf16* __restrict__ mixed, long ldx, const bf16* __restrict__ bl, long ldb,
-                                                                    const float* __restrict__ da, const bf16* __restrict__ A_log,
-                                                                    const bf16* __restrict__ dt_bias, bf16* __restrict__ tp, bf16* __restrict__ qkg,
-                                                                    float* __restrict__ betas, float* __restrict__ end) {
+__global__ void __launch_bounds__(256, 2) channel_chunk_prepare_kernel(ChunkArgs a, const bf16* __restrict__ mixed, long ldx, const bf16* __restrict__ bl,
+                                                                       long ldb, const float* __restrict__ da, const bf16* __restrict__ A_log,
+                                                                       const bf16* __restrict__ dt_bias, bf16* __restrict__ tp, bf16* __restrict__ qkg,
+                                                                       float* __restrict__ betas, float* __restrict__ end) {
   extern __shared__ __align__(16) float sm[];
   const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  constexpr int dk = DK, LD = DK + 4, QLD = DK + 8, NT = 512;
+  constexpr int dk = DK, LD = DK + 4, QLD = DK + 8, NT = 256;
   const int H = a.H, r = a.r, kh = h / r, t0 = a.t_lo + c * CH;
   const int m = min(CH, real_tokens(a, b) - t0);
   if (m <= 0) return;
-  constexpr int KS = CH * LD > 96 * 36 ? CH * LD : 96 * 36;
+  constexpr int QK = CH * QLD > CH * 68 ? CH * QLD : CH * 68;            // floats: a pair of bf16 tiles, or L
   float* G = sm;                                         // [64][LD]
-  float* ksc = G + CH * LD;                              // [64][LD] scaled keys up to the diagonal block; later the inverse's tiles
-  float* rows = ksc + KS;                                // [2][16][LD] scaled rows of q and of k
-  float* L = rows + 2 * 16 * LD;                         // [64][68]
-  bf16* q = reinterpret_cast<bf16*>(L + CH * 68);        // [64][QLD]
+  bf16* q = reinterpret_cast<bf16*>(G + CH * LD);        // [64][QLD]
   bf16* k = q + CH * QLD;
+  float* L = G + CH * LD;                                // [64][68], over q and k once they are in registers
+  bf16* ksh = reinterpret_cast<bf16*>(G + CH * LD + QK); // scaled keys [64][QLD], high and low; later the inverse's tiles
+  bf16* ksl = ksh + CH * QLD;
   __shared__ float rk[CH], rq[CH], beta[CH];
+  __shared__ int steep;                                  // blocks whose own decay is too strong for one split of the exponents
   const bf16* row0 = mixed + ((long)b * a.S + t0) * ldx;
   tile_async<dk>(q, QLD, row0 + (long)kh * dk, ldx, m, tid, NT);
   tile_async<dk>(k, QLD, row0 + (long)(H / r + kh) * dk, ldx, m, tid, NT);
@@ -503,11 +508,12 @@ __global__ void __launch_bounds__(512) channel_chunk_prepare_kernel(ChunkArgs a,
     beta[tid] = be;
     betas[id * CH + tid] = be;
   }
+  if (tid == 0) steep = 0;
   const float rate = -expf(to_f(A_log[h])) * 1.4426950408889634f, scale = rsqrtf((float)dk);
   la_wait<0>();
   __syncthreads();
-  {                                                      // inverse norms: eight lanes per row, four rows of q and k per warp
-    const int row = warp * 4 + (lane >> 3);
+  for (int i = 0; i < 8; i += 4) {                       // inverse norms: eight lanes per row, eight rows of q and k per warp
+    const int row = warp * 8 + i + (lane >> 3);
     float sk = 0.f, sq = 0.f;
     for (int d = (lane & 7) * 2; d < dk; d += 16) {
       const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + row * QLD + d));
@@ -525,104 +531,181 @@ __global__ void __launch_bounds__(512) channel_chunk_prepare_kernel(ChunkArgs a,
       rq[row] = rsqrtf(sq + 1e-6f) * scale;
     }
   }
-  // log decays in base 2, summed down the 64 tokens: a segment of 16 tokens per thread, then the segments' offsets
-  const int seg = tid / dk, sd = tid % dk;               // 4 dk <= 512 segments
-  if (seg < 4) {
-    const float dt = to_f(dt_bias[(long)h * dk + sd]);
-    float s = 0.f;
+  // log decays in base 2, summed down the 64 tokens: segments of 16 tokens, then the segments' offsets
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      float* g = G + (seg * 16 + i) * LD + sd;
-      if (seg * 16 + i < m) s += rate * softplus_f(*g + dt);
-      *g = s;
+  for (int x = 0; x < 2; ++x) {                          // 4 dk <= 512 segments over 256 threads
+    const int w = tid + x * NT, seg = w / dk, d = w % dk;
+    if (seg < 4) {
+      const float dt = to_f(dt_bias[(long)h * dk + d]);
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        float* g = G + (seg * 16 + i) * LD + d;
+        if (seg * 16 + i < m) s += rate * softplus_f(*g + dt);
+        *g = s;
+      }
+      if (s < -60.f) atomicOr(&steep, 1 << seg);
     }
   }
   __syncthreads();
-  float off = 0.f;
-  if (seg < 4)
-    for (int s = 0; s < seg; ++s) off += G[(s * 16 + 15) * LD + sd];
-  __syncthreads();
-  if (seg < 4) {
+  float off[2] = {0.f, 0.f};
 #pragma unroll
-    for (int i = 0; i < 16; ++i) G[(seg * 16 + i) * LD + sd] += off;
+  for (int x = 0; x < 2; ++x) {
+    const int w = tid + x * NT;
+    if (w < 4 * dk)
+      for (int s = 0; s < w / dk; ++s) off[x] += G[(s * 16 + 15) * LD + w % dk];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int w = tid + x * NT;
+    if (w < 4 * dk && w >= dk) {
+      float* g = G + (w / dk) * 16 * LD + w % dk;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) g[i * LD] += off[x];
+    }
   }
   __syncthreads();
   bf16* qg = qkg + id * 6 * CH * dk;
-  for (int i = tid; i < CH * dk / 2; i += NT) {
-    const int t = i / (dk / 2), d = (i % (dk / 2)) * 2, at = t * dk + d;
-    float2 qv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(q + t * QLD + d));
-    float2 kv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(k + t * QLD + d));
-    kv.x *= rk[t]; kv.y *= rk[t]; qv.x *= rq[t]; qv.y *= rq[t];
-    const float g0 = G[t * LD + d], g1 = G[t * LD + d + 1], e0 = G[(CH - 1) * LD + d], e1 = G[(CH - 1) * LD + d + 1];
-    const float x0 = exp2f(g0), x1 = exp2f(g1);
-    auto pair = [&](int tile, float u, float v) {
-      la_split2(u, v, *reinterpret_cast<__nv_bfloat162*>(qg + tile * CH * dk + at), *reinterpret_cast<__nv_bfloat162*>(qg + (tile + 1) * CH * dk + at));
-    };
-    pair(0, kv.x * x0, kv.y * x1);
-    pair(2, qv.x * x0, qv.y * x1);
-    pair(4, kv.x * exp2f(e0 - g0), kv.y * exp2f(e1 - g1));
-  }
-  if (tid < dk) end[id * dk + tid] = exp2f(G[(CH - 1) * LD + tid]);
-  bf16* out = tp + id * 4 * CH * CH;
-  // block row by block row, exponents split as in gla_chunk_prepare_kernel; half of the threads take the rows of q, the others those of k
-  const int which = tid >> 8, i0 = (tid & 255) >> 4, j0 = tid & 15;
-  for (int I = 0; I < 4; ++I) {
-    const float* ref = G + (I * 16 - 1) * LD;            // not read for I = 0: nothing has decayed there
-    bool mild = true;
-    if (tid < dk) mild = (I ? ref[tid] : 0.f) - G[(I * 16 + 15) * LD + tid] <= 60.f;
-    mild = __syncthreads_and(mild);
-    for (int i = tid; i < 16 * dk; i += NT) {
-      const int t = i / dk, d = i % dk, at = I * 16 + t;
-      const float x = exp2f(G[at * LD + d] - (I ? ref[d] : 0.f));
-      rows[t * LD + d] = to_f(q[at * QLD + d]) * rq[at] * x;
-      rows[(16 + t) * LD + d] = to_f(k[at * QLD + d]) * rk[at] * x;
-    }
-    const int krows = mild ? I * 16 + 16 : I * 16;
-    for (int i = tid; i < krows * dk; i += NT) {
-      const int t = i / dk, d = i % dk;
-      ksc[t * LD + d] = to_f(k[t * QLD + d]) * rk[t] * exp2f((I ? ref[d] : 0.f) - G[t * LD + d]);
-    }
-    __syncthreads();
-    float s[4] = {0.f, 0.f, 0.f, 0.f};
-    const float* mine = rows + (which * 16 + i0) * LD;
-    for (int d = 0; d < dk; d += 4) {
-      const float4 u = *reinterpret_cast<const float4*>(mine + d);
+  for (int i = tid; i < CH * dk / 8; i += NT) {
+    const int t = i / (dk / 8), d = (i % (dk / 8)) * 8;
+    float qv[8], kv[8], g[8], x[8], y[8];
+    load_vec<8>(q + t * QLD + d, qv);
+    load_vec<8>(k + t * QLD + d, kv);
+    load_vec<8>(G + t * LD + d, g);
+    auto pair = [&](bf16* hi, bf16* lo) {                // x as a (high, low) pair
 #pragma unroll
-      for (int J = 0; J < 4; ++J) {
-        if (J * 16 < krows) {
-          const float4 w = *reinterpret_cast<const float4*>(ksc + (J * 16 + j0) * LD + d);
-          s[J] += u.x * w.x + u.y * w.y + u.z * w.z + u.w * w.w;
+      for (int e = 0; e < 8; ++e) y[e] = x[e] - __bfloat162float(__float2bfloat16_rn(x[e]));
+      store_vec<8>(hi, x);
+      store_vec<8>(lo, y);
+    };
+    bf16* at = qg + t * dk + d;
+    float eg[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { kv[e] *= rk[t]; eg[e] = exp2f(g[e]); x[e] = kv[e] * eg[e]; }
+    pair(at, at + CH * dk);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = qv[e] * rq[t] * eg[e];
+    pair(at + 2 * CH * dk, at + 3 * CH * dk);
+    load_vec<8>(G + (CH - 1) * LD + d, eg);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = kv[e] * exp2f(eg[e] - g[e]);
+    pair(at + 4 * CH * dk, at + 5 * CH * dk);
+    load_vec<8>(G + (t | 15) * LD + d, eg);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = kv[e] * exp2f(eg[e] - g[e]);
+    pair(ksh + t * QLD + d, ksl + t * QLD + d);
+  }
+  for (int d = tid; d < dk; d += NT) end[id * dk + d] = exp2f(G[(CH - 1) * LD + d]);
+  const int I = warp >> 1, which = warp & 1, ra = I * 16 + (lane >> 2), rb = ra + 8, c2 = (lane & 3) * 2;
+  const bf16* X = which ? k : q;
+  const float fa = which ? rk[ra] : rq[ra], fb = which ? rk[rb] : rq[rb], ka = rk[ra], kb = rk[rb];
+  const bool mild = !(steep >> I & 1);
+  unsigned ah[DK / 16][4], al[DK / 16][4];
+  float d0[4] = {}, d1[4] = {};                          // the diagonal block: columns 0 .. 7 and 8 .. 15
+  auto split = [](float u, float v, unsigned& hi, unsigned& lo) {
+    __nv_bfloat162 x, y;
+    la_split2(u, v, x, y);
+    hi = *reinterpret_cast<unsigned*>(&x);
+    lo = *reinterpret_cast<unsigned*>(&y);
+  };
+  auto two = [](const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); };
+#pragma unroll
+  for (int kk = 0; kk < DK / 16; ++kk) {
+    unsigned bh[4], bo[4];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int col = kk * 16 + e * 8 + c2;
+      const float2 ref = I ? *reinterpret_cast<const float2*>(G + (I * 16 - 1) * LD + col) : make_float2(0.f, 0.f);
+      const float2 ga = *reinterpret_cast<const float2*>(G + ra * LD + col), gb = *reinterpret_cast<const float2*>(G + rb * LD + col);
+      const float2 xa = two(X + ra * QLD + col), xb = two(X + rb * QLD + col);
+      split(xa.x * fa * exp2f(ga.x - ref.x), xa.y * fa * exp2f(ga.y - ref.y), ah[kk][2 * e], al[kk][2 * e]);
+      split(xb.x * fb * exp2f(gb.x - ref.x), xb.y * fb * exp2f(gb.y - ref.y), ah[kk][2 * e + 1], al[kk][2 * e + 1]);
+      if (mild) {
+        const float2 ya = two(k + ra * QLD + col), yb = two(k + rb * QLD + col);
+        split(ya.x * ka * exp2f(ref.x - ga.x), ya.y * ka * exp2f(ref.y - ga.y), bh[e], bo[e]);
+        split(yb.x * kb * exp2f(ref.x - gb.x), yb.y * kb * exp2f(ref.y - gb.y), bh[2 + e], bo[2 + e]);
+      }
+    }
+    if (mild) {
+      la_mma(d0, al[kk], bh[0], bh[1]);
+      la_mma(d1, al[kk], bh[2], bh[3]);
+      la_mma(d0, ah[kk], bo[0], bo[1]);
+      la_mma(d1, ah[kk], bo[2], bo[3]);
+      la_mma(d0, ah[kk], bh[0], bh[1]);
+      la_mma(d1, ah[kk], bh[2], bh[3]);
+    }
+  }
+  if (!mild) {                                           // every term with its own exponents
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      const int i = e & 2 ? rb : ra, j = I * 16 + (e & 4 ? 8 : 0) + c2 + (e & 1);
+      float s = 0.f;
+      if (j <= i)
+        for (int d = 0; d < dk; ++d) s += to_f(X[i * QLD + d]) * to_f(k[j * QLD + d]) * exp2f(G[i * LD + d] - G[j * LD + d]);
+      s *= (e & 2 ? fb : fa) * rk[j];
+      if (e & 4) d1[e & 3] = s; else d0[e & 3] = s;
+    }
+  }
+  __syncthreads();                                       // L takes the place of q and k; the scaled keys are visible
+  bf16* out = tp + id * 4 * CH * CH;
+  const float ba = beta[ra], bb = beta[rb];
+  auto put = [&](int j, const float* s) {                // columns j, j + 1 of rows ra and rb
+#pragma unroll
+    for (int e = 0; e < 4; e += 2) {
+      const int i = e ? rb : ra;
+      if (which) {
+        const float be = e ? bb : ba;
+        *reinterpret_cast<float2*>(L + i * 68 + j) = make_float2(j < i ? be * s[e] : 0.f, j + 1 < i ? be * s[e + 1] : 0.f);
+      } else {
+        la_split2(j <= i ? s[e] : 0.f, j + 1 <= i ? s[e + 1] : 0.f, *reinterpret_cast<__nv_bfloat162*>(out + 2 * CH * CH + i * CH + j),
+                  *reinterpret_cast<__nv_bfloat162*>(out + 3 * CH * CH + i * CH + j));
+      }
+    }
+  };
+  put(I * 16 + c2, d0);
+  put(I * 16 + 8 + c2, d1);
+  if (which) {
+    const float zero[4] = {};
+    for (int j = (I + 1) * 16 + c2; j < CH; j += 8) put(j, zero);
+  }
+  for (int J = 0; J < I; ++J) {
+    float s0[4] = {}, s1[4] = {};
+    const int off2 = (J * 16 + (lane & 7) + ((lane >> 4) << 3)) * QLD + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      unsigned th[4], tl[4], bh[4], bo[4];
+      la_ldm4(bh, ksh + off2 + kk * 16);
+      la_ldm4(bo, ksl + off2 + kk * 16);
+      if (J + 1 == I) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { th[e] = ah[kk][e]; tl[e] = al[kk][e]; }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int col = kk * 16 + e * 8 + c2;
+          const float2 ref = *reinterpret_cast<const float2*>(G + (I * 16 - 1) * LD + col), ge = *reinterpret_cast<const float2*>(G + (J * 16 + 15) * LD + col);
+          const float f0 = exp2f(ref.x - ge.x), f1 = exp2f(ref.y - ge.y);
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&ah[kk][2 * e + x]));
+            const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&al[kk][2 * e + x]));
+            split((u.x + v.x) * f0, (u.y + v.y) * f1, th[2 * e + x], tl[2 * e + x]);
+          }
         }
       }
+      la_mma(s0, tl, bh[0], bh[1]);
+      la_mma(s1, tl, bh[2], bh[3]);
+      la_mma(s0, th, bo[0], bo[1]);
+      la_mma(s1, th, bo[2], bo[3]);
+      la_mma(s0, th, bh[0], bh[1]);
+      la_mma(s1, th, bh[2], bh[3]);
     }
-    const int i = I * 16 + i0;
-    if (!mild) {
-      const int j = I * 16 + j0;
-      float t = 0.f;
-      if (j <= i) {
-        const bf16* x = which ? k : q;
-        for (int d = 0; d < dk; ++d) t += to_f(x[i * QLD + d]) * to_f(k[j * QLD + d]) * exp2f(G[i * LD + d] - G[j * LD + d]);
-        t *= (which ? rk[i] : rq[i]) * rk[j];
-      }
-#pragma unroll
-      for (int J = 0; J < 4; ++J)
-        if (J == I) s[J] = t;
-    }
-#pragma unroll
-    for (int J = 0; J < 4; ++J) {
-      const int j = J * 16 + j0;
-      if (which) {
-        L[i * 68 + j] = j < i ? beta[i] * s[J] : 0.f;
-      } else if (J <= I) {
-        const float p = j <= i ? s[J] : 0.f;
-        const bf16 hi = __float2bfloat16_rn(p);
-        out[2 * CH * CH + i * CH + j] = hi;
-        out[3 * CH * CH + i * CH + j] = __float2bfloat16_rn(p - __bfloat162float(hi));
-      }
-    }
+    put(J * 16 + c2, s0);
+    put(J * 16 + 8 + c2, s1);
   }
   __syncthreads();
-  float (*Ts)[36] = reinterpret_cast<float (*)[36]>(ksc);
+  float (*Ts)[36] = reinterpret_cast<float (*)[36]>(ksh);
   unit_lower_inverse(L, Ts, Ts + CH, out, tid);
 }
 
@@ -794,12 +877,12 @@ __global__ void __launch_bounds__(256) channel_carry_kernel(ChunkArgs a, const b
 template <int DK>
 int launch_channel(const ChunkArgs& a, const bf16* mixed, long ldx, long voff, const bf16* beta, long ldb, const float* da, const bf16* A_log, const bf16* dt,
                    bf16* tp, bf16* qkg, float* betas, float* ends, bf16* o, int B, cudaStream_t st) {
-  constexpr int LD = DK + 4, KS = CH * LD > 96 * 36 ? CH * LD : 96 * 36;
-  constexpr int s1 = 4 * (CH * LD + KS + 32 * LD + CH * 68) + 2 * 2 * CH * (DK + 8);
+  constexpr int two = CH * (DK + 8), QK = two > CH * 68 ? two : CH * 68, KS = two > 96 * 36 ? two : 96 * 36;       // floats: a pair of bf16 tiles each
+  constexpr int s1 = 4 * (CH * (DK + 4) + QK + KS);
   constexpr int s2 = 2 * (6 * CH * (DK + 8) + 4 * CH * CLD + CH * NLD + 2 * DK * NLD + 4 * CH * NLD) + 4 * (CH + DK);
   if (cudaFuncSetAttribute(channel_chunk_prepare_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, s1) != cudaSuccess) return -2;
   if (cudaFuncSetAttribute(channel_carry_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, s2) != cudaSuccess) return -2;
-  channel_chunk_prepare_kernel<DK><<<dim3(a.chunks, a.H, B), 512, s1, st>>>(a, mixed, ldx, beta, ldb, da, A_log, dt, tp, qkg, betas, ends);
+  channel_chunk_prepare_kernel<DK><<<dim3(a.chunks, a.H, B), 256, s1, st>>>(a, mixed, ldx, beta, ldb, da, A_log, dt, tp, qkg, betas, ends);
   channel_carry_kernel<DK><<<dim3(a.dv / CN, a.H, B), 256, s2, st>>>(a, mixed, ldx, voff, tp, qkg, betas, ends, o);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

@@ -222,6 +222,10 @@ int residual_join_t(float* x, const JoinBranch& a, const JoinBranch& b, const vo
   };
   uintptr_t bits = 0;
   for (const void* p : {a.out, a.bias, a.norm, b.out, b.bias, b.norm, lanes, w_next, (const void*)x, (const void*)y}) bits |= reinterpret_cast<uintptr_t>(p);
+  if (D % 8 == 0 && bits % 16 == 0) {
+    if (D <= 2048) return go(residual_join_kernel<T, 8, 1>, 8, 1);
+    if (D <= 4096) return go(residual_join_kernel<T, 8, 2>, 8, 2);
+  }
   if (D % 4 == 0 && bits % 16 == 0) {
     if (D <= 1024) return go(residual_join_kernel<T, 4, 1>, 4, 1);
     if (D <= 2048) return go(residual_join_kernel<T, 4, 2>, 4, 2);
