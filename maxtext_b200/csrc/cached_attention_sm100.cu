@@ -189,7 +189,7 @@ qkv_prep_kernel(const PrepArgs a) {
 // The same for head widths up to 8 * LPH that are multiples of 8: LPH lanes share a head, a warp takes 32 / LPH heads at a time, and the lanes that
 // rotate together meet by a shuffle. (Halves that are paired begin at a multiple of 8.)
 template <typename T, int LPH>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 12)
 qkv_prep_wide_kernel(const PrepArgs a) {
   constexpr int VEC = 8, STEP = 4 * (32 / LPH);
   extern __shared__ float2 cs[];                            // (cos, sin) of the rot / 2 angles

@@ -636,15 +636,26 @@ __global__ void __launch_bounds__(256, 2) channel_chunk_prepare_kernel(ChunkArgs
       la_mma(d1, ah[kk], bh[2], bh[3]);
     }
   }
-  if (!mild) {                                           // every term with its own exponents
+  if (!mild) {                                           // every term with its own exponents; entries above the diagonal are dropped later
+    const int j0 = I * 16 + c2;
+    float s00[2] = {}, s10[2] = {}, s11[2] = {};         // rows ra and rb on columns 0 .. 7, row rb on columns 8 .. 15
+    for (int d = 0; d < dk; d += 2) {
+      const float2 xa = two(X + ra * QLD + d), xb = two(X + rb * QLD + d);
+      const float2 ga = *reinterpret_cast<const float2*>(G + ra * LD + d), gb = *reinterpret_cast<const float2*>(G + rb * LD + d);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      const int i = e & 2 ? rb : ra, j = I * 16 + (e & 4 ? 8 : 0) + c2 + (e & 1);
-      float s = 0.f;
-      if (j <= i)
-        for (int d = 0; d < dk; ++d) s += to_f(X[i * QLD + d]) * to_f(k[j * QLD + d]) * exp2f(G[i * LD + d] - G[j * LD + d]);
-      s *= (e & 2 ? fb : fa) * rk[j];
-      if (e & 4) d1[e & 3] = s; else d0[e & 3] = s;
+      for (int e = 0; e < 2; ++e) {
+        const float2 k0 = two(k + (j0 + e) * QLD + d), k1 = two(k + (j0 + 8 + e) * QLD + d);
+        const float2 g0 = *reinterpret_cast<const float2*>(G + (j0 + e) * LD + d), g1 = *reinterpret_cast<const float2*>(G + (j0 + 8 + e) * LD + d);
+        s00[e] += xa.x * k0.x * exp2f(ga.x - g0.x) + xa.y * k0.y * exp2f(ga.y - g0.y);
+        s10[e] += xb.x * k0.x * exp2f(gb.x - g0.x) + xb.y * k0.y * exp2f(gb.y - g0.y);
+        s11[e] += xb.x * k1.x * exp2f(gb.x - g1.x) + xb.y * k1.y * exp2f(gb.y - g1.y);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      d0[e] = s00[e] * fa * rk[j0 + e];
+      d0[2 + e] = s10[e] * fb * rk[j0 + e];
+      d1[2 + e] = s11[e] * fb * rk[j0 + 8 + e];
     }
   }
   __syncthreads();                                       // L takes the place of q and k; the scaled keys are visible
