@@ -559,24 +559,39 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 diff_merge_kernel(const float* __restrict__ part, const float* __restrict__ ml, const DiffArgs a, int H, int Dv, int splits, const T* __restrict__ gate,
                   long ldg, int per_head, T* __restrict__ out) {
-  __shared__ float red[4];
-  const int h = blockIdx.x, b = blockIdx.y, t = threadIdx.x;
+  __shared__ float red[4], top[4], den[4], wt[2][64];
+  const int h = blockIdx.x, b = blockIdx.y, t = threadIdx.x, warp = t >> 5;
   const float lam = diff_lambda<T>(a, t & 31);
+  // the weights of the splits: 64 threads per map
+  const long at0 = ((long)b * 2 * H + 2 * h) * splits;
+  float mx = -INFINITY, l = 0.f;
+  if ((t & 63) < splits) {
+    const float2 v = *reinterpret_cast<const float2*>(ml + (at0 + (t >> 6) * splits + (t & 63)) * 2);
+    mx = v.x;
+    l = v.y;
+  }
+  float wm = mx;
+#pragma unroll
+  for (int d = 16; d > 0; d >>= 1) wm = fmaxf(wm, __shfl_xor_sync(0xffffffffu, wm, d));
+  if ((t & 31) == 0) top[warp] = wm;
+  __syncthreads();
+  const float c = mx == -INFINITY ? 0.f : __expf(mx - fmaxf(top[warp & 2], top[warp | 1]));
+  l = warp_add(c * l);
+  if ((t & 31) == 0) den[warp] = l;
+  wt[t >> 6][t & 63] = c;
+  __syncthreads();
   float x[2] = {0.f, 0.f};                                  // Dv up to 256
 #pragma unroll
   for (int m = 0; m < 2; ++m) {
-    const long at = ((long)b * 2 * H + 2 * h + m) * splits;
-    float top = -INFINITY, den = 0.f, o[2] = {0.f, 0.f};
-    for (int s = 0; s < splits; ++s) top = fmaxf(top, ml[(at + s) * 2]);
+    const float* p = part + (at0 + m * splits) * Dv;
+    const float sum = den[2 * m] + den[2 * m + 1], f = sum > 0.f ? (m ? -lam : 1.f) / sum : 0.f;
+    float o[2] = {0.f, 0.f};
+#pragma unroll 4
     for (int s = 0; s < splits; ++s) {
-      if (ml[(at + s) * 2] == -INFINITY) continue;
-      const float c = __expf(ml[(at + s) * 2] - top);
-      den += ml[(at + s) * 2 + 1] * c;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
-        if (t + j * 128 < Dv) o[j] += part[(at + s) * Dv + t + j * 128] * c;
+        if (t + j * 128 < Dv && wt[m][s] != 0.f) o[j] += p[(long)s * Dv + t + j * 128] * wt[m][s];
     }
-    const float f = den > 0.f ? (m ? -lam : 1.f) / den : 0.f;
     x[0] += f * o[0];
     x[1] += f * o[1];
   }
@@ -836,7 +851,7 @@ extern "C" int mt_cached_decode(const void* q, const void* k, const void* v, con
                                 int D, int Dv, float scale, float cap, int window, int chunk, const void* sinks, const void* gate, long ldg, int per_head,
                                 const DiffArgs* diff, int splits, float* part, float* ml, void* out, cudaStream_t st) {
   if (B <= 0) return 0;
-  if (D % 8 || Dv % 8 || D > 256 || Dv > 256 || H % G || splits < 1 || (diff && (H % 2 || sinks))) return -1;
+  if (D % 8 || Dv % 8 || D > 256 || Dv > 256 || H % G || splits < 1 || (diff && (H % 2 || sinks || splits > 64))) return -1;
   DecodeArgs a{(const bf16*)q, (const bf16*)k, (const bf16*)v, slots, lengths, max_len, H, G, D, Dv, window, chunk, splits, (H / G + 15) / 16, scale, cap,
                part, ml};
   const int rc = D <= 64 ? decode_dv<64>(a, B, st) : (D <= 128 ? decode_dv<128>(a, B, st) : decode_dv<256>(a, B, st));
