@@ -24,12 +24,12 @@ AXIS_TO_KEY["sequence"] = "sequence"
 DECODER_BLOCKS = (
     "default", "llama2", "mistral", "mixtral", "deepseek", "gemma", "gemma2", "gemma3", "gemma4",
     "gemma4_small", "qwen2", "qwen3", "qwen3_moe", "qwen3_custom_moe", "qwen3_next", "qwen3_5", "gpt3",
-    "gpt_oss", "simple", "simple_mlp", "llama4", "olmo3", "deepseek4", "envy", "silinex", "sitivik", "tipidra",
+    "gpt_oss", "simple", "simple_mlp", "llama4", "olmo3", "deepseek4", "envy", "gukirax", "silinex", "sitivik", "tipidra",
 )
 # families with a model implementation in maxtext_b200.models
 IMPLEMENTED_DECODER_BLOCKS = (
     "default", "llama2", "mistral", "mixtral", "deepseek", "gemma", "gemma2", "gemma3", "qwen2", "qwen3",
-    "qwen3_moe", "gpt3", "gpt_oss", "olmo3", "simple", "simple_mlp", "silinex", "sitivik", "tipidra",
+    "qwen3_moe", "gpt3", "gpt_oss", "olmo3", "simple", "simple_mlp", "gukirax", "silinex", "sitivik", "tipidra",
 )
 REMAT_POLICIES = (
     "minimal_with_context", "minimal", "save_dot_with_context_except_mlp", "save_dot_except_mlpwi",

@@ -300,8 +300,8 @@ def check_misc(t):
 
 
 def check_layer_specs(t):
-  from ..models import silinex, sitivik, tipidra
-  family = {"silinex": silinex, "sitivik": sitivik, "tipidra": tipidra}.get(t.get("decoder_block"))
+  from ..models import gukirax, silinex, sitivik, tipidra
+  family = {"gukirax": gukirax, "silinex": silinex, "sitivik": sitivik, "tipidra": tipidra}.get(t.get("decoder_block"))
   if family is None:
     return
   try:

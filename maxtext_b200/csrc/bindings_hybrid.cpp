@@ -21,6 +21,14 @@ int mt_cached_decode(const void* q, const void* k, const void* v, const int64_t*
                      const mt::cattn::DiffArgs* diff, int splits, float* part, float* ml, void* out, cudaStream_t st);
 int mt_cached_attention(int f32, const void* q, const void* k, const void* v, long max_len, const int64_t* slots, const int64_t* lengths, int B, int S, int H,
                         int G, int D, int Dv, float scale, float cap, int window, int chunk, const void* sinks, void* out, cudaStream_t st);
+int mt_wide_decode(const void* q, const void* k, const void* v, const int64_t* slots, const int64_t* lengths, long max_len, int B, int H, int G, int D, int Dv,
+                   float scale, int window, int chunk, const void* sinks, int splits, float* part, float* ml, void* out, cudaStream_t st);
+int mt_wide_attention(int f32, const void* q, const void* k, const void* v, long max_len, const int64_t* slots, const int64_t* lengths, int B, int S, int H, int G,
+                      int D, int Dv, float scale, int window, int chunk, const void* sinks, void* out, cudaStream_t st);
+int mt_wide_flash(const void* q, const void* k, const void* v, void* out, const int* seg_q, const int* seg_k, const int* pos_q, const int* pos_k, int* tiles,
+                  const void* sinks, int B, int Sq, int Skv, int H, int G, int D, int Dv, long ldk, long bsk, long ldv, long bsv, float scale, int window,
+                  int chunk, int q_off, int* status, cudaStream_t st);
+long mt_attn_tile_ints(int B, int Sq, int Skv);
 int mt_head_gate(int f32, const void* o, int dvp, const void* g, long ldg, long rows, int HD, int Dv, int per_head, void* out, int sms, cudaStream_t st);
 int mt_diff_combine(int f32, const void* o, int dvp, const mt::cattn::DiffArgs* a, long N, int H, int Dv, const void* gate, long ldg, int per_head, void* out,
                     int sms, cudaStream_t st);
@@ -28,12 +36,13 @@ int mt_expert_up(int f32, const void* x, const void* w0, const void* w1, const f
                  const int* row_pair, int n, int k, int E, int F, int D, float limit, void* h, int sms, cudaStream_t st);
 int mt_expert_down(int f32, const void* h, const void* w, const int* idx, const int* sizes, const int* offs, const int* row_pair, int n, int E, int D, int F,
                    void* y, int sms, cudaStream_t st);
-int mt_expert_act(const void* gu, const float* wts, const int* row_pair, const int* offs, int E, int F, float limit, void* h, int rows_max, int sms,
+int mt_expert_act(const void* gu, int gated, const float* wts, const int* row_pair, const int* offs, int E, int F, float limit, void* h, int rows_max, int sms,
                   cudaStream_t st);
 }
 
 void mt_count_launches(int n); // defined in bindings.cpp
 int mt_num_sms();              // defined in bindings.cpp
+int* mt_status_ptr();          // defined in bindings.cpp
 
 namespace {
 
@@ -147,16 +156,16 @@ void check_cache(const Tensor& k, const Tensor& v, const Tensor& like, int64_t D
 void qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, int64_t D, int64_t Dv, const Tensor& pos, const OptTensor& inv_ts, int64_t rot, double eps,
               Tensor& qp, const OptTensor& kp, const OptTensor& vp, Tensor& kc, Tensor& vc, const Tensor& slots, const Tensor& lengths,
               const OptTensor& new_lens, const OptTensor& bq, const OptTensor& bk, const OptTensor& bv, const OptTensor& wq, const OptTensor& wk, bool paired,
-              int64_t maps, double temp_coef, double temp_every) {
+              int64_t maps, double temp_coef, double temp_every, const OptTensor& talk) {
   const bool f = f32(q);
   TORCH_CHECK(qp.dim() == 3 && rot % 2 == 0 && rot >= 0 && rot <= D && bool(inv_ts) == (rot > 0) && maps >= 1 && qp.size(1) % maps == 0);
   const int64_t N = q.size(0), H = qp.size(1) / maps, dq = qp.size(2), B = slots.numel();
   check_cache(kc, vc, q, D * maps);
   const int64_t G = kc.size(2);
-  TORCH_CHECK(vc.size(3) == Dv && B > 0 && N % B == 0 && dq >= D * maps && H % G == 0);
+  TORCH_CHECK(vc.size(3) == Dv && B > 0 && N % B == 0 && dq >= D * maps && H % G == 0 && (!talk || (maps == 1 && dq == G * D)));
   rows2d(q, q, N, H * maps * D, "q"); rows2d(k, q, N, G * maps * D, "k"); rows2d(v, q, N, G * Dv, "v");
   same(qp, q, N * H * maps * dq, "packed q");
-  if (kp) same(*kp, q, N * G * dq, "packed k");
+  if (kp) same(*kp, q, N * G * (talk ? D : dq), "packed k");
   int64_t dvp = Dv;
   if (vp) { dvp = vp->size(vp->dim() - 1); TORCH_CHECK(dvp >= Dv); same(*vp, q, N * G * dvp, "packed v"); }
   if (inv_ts) floats(*inv_ts, rot / 2, "inverse timescales");
@@ -174,6 +183,7 @@ void qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, int64_t D, int6
   a.rot = (int)rot; a.paired = paired;
   a.eps = (float)eps; a.temp_coef = (float)temp_coef; a.temp_every = (float)temp_every;
   a.S = (int)(N / B);
+  a.talk = same(talk, q, H * H, "mixing matrix");
   a.qp = qp.data_ptr(); a.kp = kp ? kp->data_ptr() : nullptr; a.vp = vp ? vp->data_ptr() : nullptr;
   a.dq = (int)dq; a.dvp = (int)dvp;
   a.kc = kc.data_ptr(); a.vc = vc.data_ptr(); a.max_len = kc.size(1);
@@ -240,6 +250,61 @@ void cached_attention(const Tensor& q, const Tensor& k, const Tensor& v, const T
                            (int)G, (int)D, (int)Dv, (float)scale, (float)cap, (int)window, (int)chunk, sk, out.data_ptr(), stream()), "cached_attention");
 }
 
+// q [B, H, G * D] (one key of all key heads side by side), k [slots, max_len, G, D], v [.., G, Dv] -> out [B, H * Dv]
+void wide_decode(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& slots, const Tensor& lengths, double scale, int64_t window, int64_t chunk,
+                 const OptTensor& sinks, int64_t splits, Tensor& part, Tensor& ml, Tensor& out) {
+  TORCH_CHECK(!f32(q) && q.dim() == 3 && q.is_contiguous() && k.dim() == 4 && v.dim() == 4);
+  const int64_t B = q.size(0), H = q.size(1), G = k.size(2), D = k.size(3), Dv = v.size(3);
+  check_cache(k, v, q, D);
+  TORCH_CHECK(q.size(2) == G * D && H % G == 0 && splits >= 1);
+  floats(part, B * H * splits * Dv, "part"); floats(ml, B * H * splits * 2, "ml");
+  same(out, q, B * H * Dv, "out");
+  const void* sk = same(sinks, q, H, "sinks");
+  c10::cuda::CUDAGuard guard(q.device());
+  done(mt_wide_decode(q.data_ptr(), k.data_ptr(), v.data_ptr(), longs(slots, B, "slots"), longs(lengths, B, "lengths"), k.size(1), (int)B, (int)H, (int)G,
+                      (int)D, (int)Dv, (float)scale, (int)window, (int)chunk, sk, (int)splits, part.data_ptr<float>(), ml.data_ptr<float>(), out.data_ptr(),
+                      stream()), "wide_decode", 2);
+}
+
+void wide_attention(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& slots, const Tensor& lengths, int64_t S, double scale, int64_t window,
+                    int64_t chunk, const OptTensor& sinks, Tensor& out) {
+  const bool f = f32(q);
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && k.dim() == 4 && v.dim() == 4);
+  const int64_t B = slots.numel(), H = q.size(1), G = k.size(2), D = k.size(3), Dv = v.size(3);
+  check_cache(k, v, q, D);
+  TORCH_CHECK(q.size(0) == B * S && q.size(2) == G * D && H % G == 0);
+  same(out, q, B * S * H * Dv, "out");
+  const void* sk = same(sinks, q, H, "sinks");
+  c10::cuda::CUDAGuard guard(q.device());
+  done(mt_wide_attention(f, q.data_ptr(), k.data_ptr(), v.data_ptr(), k.size(1), longs(slots, B, "slots"), longs(lengths, B, "lengths"), (int)B, (int)S, (int)H,
+                         (int)G, (int)D, (int)Dv, (float)scale, (int)window, (int)chunk, sk, out.data_ptr(), stream()), "wide_attention");
+}
+
+// q [B, Sq, H, G * D] contiguous, k [B, Skv, G, D] and v [B, Skv, G, Dv] rows whose heads lie side by side -> out [B, Sq, H * Dv]
+void wide_flash(const Tensor& q, const Tensor& k, const Tensor& v, Tensor& out, const OptTensor& seg_q, const OptTensor& seg_k, const OptTensor& pos_q,
+                const OptTensor& pos_k, const OptTensor& sinks, double scale, int64_t window, int64_t chunk, int64_t q_off) {
+  TORCH_CHECK(!f32(q) && q.dim() == 4 && q.is_contiguous() && k.dim() == 4 && v.dim() == 4);
+  const int64_t B = q.size(0), Sq = q.size(1), H = q.size(2), Skv = k.size(1), G = k.size(2), D = k.size(3), Dv = v.size(3);
+  auto rows = [&](const Tensor& t, int64_t w) {
+    return t.is_cuda() && t.scalar_type() == torch::kBFloat16 && t.size(0) == B && t.size(1) == Skv && t.size(2) == G && t.size(3) == w && t.stride(3) == 1 &&
+           (G == 1 || t.stride(2) == w) && t.stride(1) % 8 == 0 && t.stride(1) >= G * w && (B == 1 || t.stride(0) % 8 == 0) &&
+           reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0;
+  };
+  TORCH_CHECK(rows(k, D) && rows(v, Dv) && q.size(3) == G * D && H % G == 0 && D % 8 == 0 && Dv % 8 == 0 && Dv <= 128 && Skv >= 1 && Sq >= 1,
+              "wide_flash: unsupported operands");
+  same(out, q, B * Sq * H * Dv, "out");
+  TORCH_CHECK(bool(seg_q) == bool(seg_k) && bool(pos_q) == bool(pos_k));
+  auto opt = [&](const OptTensor& t, int64_t n, const char* what) { return t ? ints(*t, n, what) : nullptr; };
+  const void* sk = same(sinks, q, H, "sinks");
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor tiles;
+  if (pos_q) tiles = torch::empty({mt_attn_tile_ints((int)B, (int)Sq, (int)Skv)}, torch::dtype(torch::kInt32).device(q.device()));
+  done(mt_wide_flash(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), opt(seg_q, B * Sq, "seg_q"), opt(seg_k, B * Skv, "seg_k"),
+                     opt(pos_q, B * Sq, "pos_q"), opt(pos_k, B * Skv, "pos_k"), pos_q ? tiles.data_ptr<int>() : nullptr, sk, (int)B, (int)Sq, (int)Skv, (int)H,
+                     (int)G, (int)D, (int)Dv, k.stride(1), k.stride(0), v.stride(1), v.stride(0), (float)scale, (int)window, (int)chunk, (int)q_off,
+                     mt_status_ptr(), stream()), "wide_flash", pos_q ? 3 : 1);
+}
+
 // o [N, H, >= dv], g [N, >= H * dv] (or [N, >= H]) -> out [N, H * dv]
 void head_gate(const Tensor& o, const Tensor& g, int64_t dv, Tensor& out, bool per_head) {
   const bool f = f32(o);
@@ -269,16 +334,17 @@ void check_plan(const Tensor& sizes, const Tensor& offs, const Tensor& row_pair,
   ints(sizes, E, "sizes"); ints(offs, E + 1, "offs"); ints(row_pair, row_pair.numel(), "row_pair");
 }
 
-void expert_up(const Tensor& x, const Tensor& w0, const Tensor& w1, const Tensor& wts, const Tensor& idx, const Tensor& sizes, const Tensor& offs,
+// w1 absent: ungated experts
+void expert_up(const Tensor& x, const Tensor& w0, const OptTensor& w1, const Tensor& wts, const Tensor& idx, const Tensor& sizes, const Tensor& offs,
                const Tensor& row_pair, int64_t k, double limit, Tensor& h) {
   const bool f = f32(x);
-  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w0.dim() == 3 && w0.sizes() == w1.sizes() && w0.size(2) == x.size(1));
+  TORCH_CHECK(x.dim() == 2 && x.is_contiguous() && w0.dim() == 3 && w0.size(2) == x.size(1));
   const int64_t E = w0.size(0), F = w0.size(1), D = w0.size(2), n = x.size(0) * k;
   same(w0, x, E * F * D, "w0"); same(w1, x, E * F * D, "w1"); same(h, x, n * F, "h");
   floats(wts, n, "scores");
   check_plan(sizes, offs, row_pair, E);
   c10::cuda::CUDAGuard guard(x.device());
-  done(mt_expert_up(f, x.data_ptr(), w0.data_ptr(), w1.data_ptr(), wts.data_ptr<float>(), ints(idx, n, "idx"), sizes.data_ptr<int>(), offs.data_ptr<int>(),
+  done(mt_expert_up(f, x.data_ptr(), w0.data_ptr(), w1 ? w1->data_ptr() : nullptr, wts.data_ptr<float>(), ints(idx, n, "idx"), sizes.data_ptr<int>(), offs.data_ptr<int>(),
                     row_pair.data_ptr<int>(), (int)n, (int)k, (int)E, (int)F, (int)D, (float)limit, h.data_ptr(), mt_num_sms(), stream()), "expert_up");
 }
 
@@ -293,13 +359,13 @@ void expert_down(const Tensor& h, const Tensor& w, const Tensor& idx, const Tens
                       (int)D, (int)F, y.data_ptr(), mt_num_sms(), stream()), "expert_down");
 }
 
-// gu [rows_max, 2F] of the padded layout -> h [rows_max, F]
+// gu [rows_max, 2F] (ungated experts: [rows_max, F]) of the padded layout -> h [rows_max, F]
 void expert_act(const Tensor& gu, const Tensor& wts, const Tensor& row_pair, const Tensor& offs, double limit, Tensor& h) {
-  TORCH_CHECK(!f32(gu) && gu.dim() == 2 && gu.is_contiguous() && h.dim() == 2 && gu.size(1) == 2 * h.size(1) && h.size(1) % 8 == 0);
+  TORCH_CHECK(!f32(gu) && gu.dim() == 2 && gu.is_contiguous() && h.dim() == 2 && (gu.size(1) == 2 * h.size(1) || gu.size(1) == h.size(1)) && h.size(1) % 8 == 0);
   same(h, gu, gu.size(0) * h.size(1), "h");
   ints(row_pair, gu.size(0), "row_pair"); ints(offs, offs.numel(), "offs"); floats(wts, wts.numel(), "scores");
   c10::cuda::CUDAGuard guard(gu.device());
-  done(mt_expert_act(gu.data_ptr(), wts.data_ptr<float>(), row_pair.data_ptr<int>(), offs.data_ptr<int>(), (int)offs.numel() - 1, (int)h.size(1), (float)limit,
+  done(mt_expert_act(gu.data_ptr(), gu.size(1) == 2 * h.size(1), wts.data_ptr<float>(), row_pair.data_ptr<int>(), offs.data_ptr<int>(), (int)offs.numel() - 1, (int)h.size(1), (float)limit,
                      h.data_ptr(), (int)gu.size(0), mt_num_sms(), stream()), "expert_act");
 }
 
@@ -313,13 +379,16 @@ void register_hybrid(pybind11::module_& m) {
   const auto none = pybind11::none();
   m.def("qkv_prep", &qkv_prep, arg("q"), arg("k"), arg("v"), arg("D"), arg("Dv"), arg("pos"), arg("inv_ts"), arg("rot"), arg("eps"), arg("qp"), arg("kp"),
         arg("vp"), arg("kc"), arg("vc"), arg("slots"), arg("lengths"), arg("new_lens"), arg("bq") = none, arg("bk") = none, arg("bv") = none, arg("wq") = none,
-        arg("wk") = none, arg("paired") = false, arg("maps") = 1, arg("temp_coef") = 0.0, arg("temp_every") = 0.0);
+        arg("wk") = none, arg("paired") = false, arg("maps") = 1, arg("temp_coef") = 0.0, arg("temp_every") = 0.0, arg("talk") = none);
   m.def("cached_decode_splits", &cached_decode_splits);
   m.def("cached_decode", &cached_decode, arg("q"), arg("k"), arg("v"), arg("slots"), arg("lengths"), arg("scale"), arg("cap"), arg("window"), arg("sinks"),
         arg("gate"), arg("splits"), arg("part"), arg("ml"), arg("out"), arg("chunk") = 0, arg("per_head") = false, arg("lam") = std::vector<Tensor>{},
         arg("diff") = 0.0, arg("eps") = 0.0);
   m.def("cached_attention", &cached_attention, arg("q"), arg("k"), arg("v"), arg("slots"), arg("lengths"), arg("S"), arg("scale"), arg("cap"), arg("window"),
         arg("sinks"), arg("out"), arg("chunk") = 0);
+  m.def("wide_decode", &wide_decode);
+  m.def("wide_attention", &wide_attention);
+  m.def("wide_flash", &wide_flash);
   m.def("head_gate", &head_gate, arg("o"), arg("g"), arg("dv"), arg("out"), arg("per_head") = false);
   m.def("diff_combine", &diff_combine);
   m.def("expert_up", &expert_up);

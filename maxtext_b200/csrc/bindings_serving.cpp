@@ -4,8 +4,11 @@
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
 #include <cuda_runtime.h>
+#include "residual_gate.h"
 
 extern "C" {
+int mt_residual_gate(const mt::ResidualGate* a, int f32, long rows, int D, cudaStream_t st);
+int mt_act_rows(const void* x, long ldx, void* y, int f32, long rows, int F, int code, const void* par, int sms, cudaStream_t st);
 int mt_residual_norm(float* x, const void* branch, const void* w_post, float mult, const void* w_next, void* y, int f32, long rows, int D, float eps_post,
                      float eps_next, float offset, cudaStream_t st);
 int mt_residual_join(float* x, const void* a, const void* a_bias, const void* a_norm, float a_factor, const void* b, const void* b_bias, const void* b_norm,
@@ -136,6 +139,56 @@ void residual_join(Tensor& x, const Tensor& a, const OptTensor& a_bias, const Op
                         b ? b->data_ptr() : nullptr, lane_vector(b_bias, a, D, "bias"), lane_vector(b_norm, a, D, "norm"), (float)b_factor,
                         lane_vector(lanes, a, D, "lane factors"), lane_vector(w_next, a, D, "next norm"), y ? y->data_ptr() : nullptr, f, x.size(0), (int)D,
                         (float)eps, stream()), "residual_join");
+}
+
+// x [N, D] fp32 += norm(b * sigmoid(gate + bias)) * w_post with b the sum of `per_token` of `rows` (dest: which) and `extra`; y: norm(x) * w_next, x itself
+// without w_next, or None. gate and y may be columns of wider matrices. centred: layer norms, otherwise RMS norms. fresh: x is only written.
+void residual_gate(Tensor& x, const OptTensor& rows, const OptTensor& dest, int64_t per_token, const OptTensor& extra, const OptTensor& gate,
+                   const OptTensor& bias, const OptTensor& w_post, const OptTensor& w_next, const OptTensor& y, double eps, bool centred, bool fresh) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.is_contiguous() && x.scalar_type() == torch::kFloat32 && x.size(1) <= 8192, "residual_gate: x fp32 [rows, <= 8192]");
+  TORCH_CHECK((rows && w_post) || (y && !rows && !fresh), "residual_gate: nothing to do");
+  TORCH_CHECK(bool(rows) == bool(w_post) && (!w_next || y) && bool(gate) == bool(bias) && (rows || !(gate || extra || dest)) && per_token >= 1);
+  const Tensor& like = rows ? *rows : *y;
+  const bool f = f32(like);
+  const int64_t N = x.size(0), D = x.size(1);
+  mt::ResidualGate a{};
+  a.x = x.data_ptr<float>(); a.per_token = (int)per_token; a.eps = (float)eps; a.centred = centred; a.fresh = fresh;
+  if (rows) {
+    TORCH_CHECK(rows->dim() == 2 && rows->is_contiguous() && rows->size(1) == D && rows->size(0) >= 1, "residual_gate: branch rows of the model width");
+    a.rows = rows->data_ptr(); a.n_rows = rows->size(0);
+    if (dest) {
+      TORCH_CHECK(dest->is_cuda() && dest->scalar_type() == torch::kInt32 && dest->is_contiguous() && dest->numel() == N * per_token, "residual_gate: int32 row numbers");
+      a.dest = dest->data_ptr<int>();
+    } else {
+      TORCH_CHECK(rows->size(0) == N * per_token, "residual_gate: ", per_token, " branch rows per token");
+    }
+    same(*w_post, like, D, "w_post"); a.w_post = w_post->data_ptr();
+    a.extra = lane_vector(extra, like, N * D, "extra rows");
+    if (gate) {
+      TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == like.scalar_type() && gate->dim() == 2 && gate->size(0) == N && gate->size(1) == D &&
+                  gate->stride(1) == 1, "residual_gate: gate [rows, D]");
+      a.gate = gate->data_ptr(); a.ldg = gate->stride(0);
+      a.bias = lane_vector(bias, like, D, "gate bias");
+    }
+  }
+  a.w_next = lane_vector(w_next, like, D, "w_next");
+  if (y) {
+    TORCH_CHECK(y->is_cuda() && y->scalar_type() == like.scalar_type() && y->dim() == 2 && y->size(0) == N && y->size(1) == D && y->stride(1) == 1,
+                "residual_gate: y [rows, D]");
+    a.y = y->data_ptr(); a.ldy = y->stride(0);
+  }
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_residual_gate(&a, f, N, (int)D, stream()), "residual_gate");
+}
+
+// x [N, F] rows (columns of a wider matrix allowed) -> y [N, F]; par: the two numbers of xIELU (code 6)
+void act_rows(const Tensor& x, Tensor& y, int64_t code, const OptTensor& par) {
+  const bool f = f32(x);
+  TORCH_CHECK(x.dim() == 2 && (x.size(1) == 1 || x.stride(1) == 1) && bool(par) == (code == 6));
+  same(y, x, x.numel(), "act_rows output");
+  const void* pp = lane_vector(par, x, 2, "activation parameters");
+  c10::cuda::CUDAGuard guard(x.device());
+  done(mt_act_rows(x.data_ptr(), x.stride(0), y.data_ptr(), f, x.size(0), (int)x.size(1), (int)code, pp, mt_num_sms(), stream()), "act_rows");
 }
 
 // g [N, dim], table [V, dim], tokens [N] -> out [N, dim]
@@ -501,6 +554,8 @@ void mla_value_up(const Tensor& part, const Tensor& ml, const Tensor& w, int64_t
 void register_serving(pybind11::module_& m) {
   m.def("residual_norm", &residual_norm);
   m.def("residual_join", &residual_join);
+  m.def("residual_gate", &residual_gate);
+  m.def("act_rows", &act_rows);
   m.def("token_gate", &token_gate);
   m.def("act_fwd", &act_fwd);
   m.def("delta_decode", &delta_decode);

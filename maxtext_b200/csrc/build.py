@@ -40,7 +40,7 @@ SERVING_NAME = "maxtext_b200_serving_C"
 SERVING_SOURCES = ("bindings.cpp", "bindings_attention.cpp", "bindings_serving.cpp", "bindings_hybrid.cpp", "bindings_moe.cpp", "gemm_sm100.cu",
                    "gemm_small_m.cu", "elementwise.cu", "attention_fwd_sm100.cu", "sampling_sm100.cu", "residual_norm.cu",
                    "recurrent_sm100.cu", "recurrent_chunk_sm100.cu", "latent_attention_sm100.cu", "stream_mix.cu", "ssm_sm100.cu",
-                   "cached_attention_sm100.cu", "expert_serving.cu", "router_sm100.cu", "moe_sm100.cu")
+                   "cached_attention_sm100.cu", "attention_wide_sm100.cu", "expert_serving.cu", "router_sm100.cu", "moe_sm100.cu")
 
 
 def build_serving_extension(verbose: bool = True):

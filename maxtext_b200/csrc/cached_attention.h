@@ -23,6 +23,8 @@ struct PrepArgs {
   void *kc, *vc;                       // cache [slots, max_len, G, maps * D], [.., Dv]
   long max_len;
   const int64_t *slots, *lengths, *new_lens;
+  const void* talk;                    // [H, H] or null: the heads' scores are mixed by this matrix. Then qp is [N, H, G * D]: a query over the keys of
+                                       // all key heads side by side (dq = G * D, no operand padding, one map)
 };
 
 // differential attention: lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff

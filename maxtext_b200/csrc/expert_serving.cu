@@ -3,6 +3,7 @@
 // up-projections in fp32, in front of the clamps:
 //   up:    h[pair] = act(s (Wg x), s (Wu x)),  act(g, u) = min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1)
 //   down:  y[pair] = Wd h[pair]
+// Ungated experts have one up-projection, whose activation the score multiplies:  h[pair] = s relu(W x)^2.
 // A persistent CTA works through items of 16 * MW weight rows of one expert. Its four warps sit MW along the rows and 4 / MW along the
 // contraction, operands pass through a cp.async ring of three or four stages, mma.sync m16n8k16 takes the weights in the M position (a step is bound by
 // reading weights: with a handful of tokens per expert the 128-row tiles of tcgen05 would be empty). Also here: the activation of the padded path, and plain kernels for fp32
@@ -18,6 +19,9 @@ __device__ __forceinline__ float clamped_act(float g, float u, float limit) {
   u = fminf(fmaxf(u, -limit), limit);
   return g * sigmoid_f(1.702f * g) * (u + 1.f);
 }
+
+enum { DOWN = 0, GATED = 1, RELU2 = 2 };
+__device__ __forceinline__ float relu2(float s, float v) { return v > 0.f ? s * v * v : 0.f; }
 
 struct Args {
   const void* x;              // up: [T, K]; down: [n, K]
@@ -58,10 +62,11 @@ __device__ __forceinline__ bool find(const Args& a, int E, int number, Item& it)
 }
 
 // The ring runs on over item borders: while an item's sums are finished the loads of the next one are in flight.
-template <bool UP, int MW>
+template <int MODE, int MW>
 __global__ void __launch_bounds__(128)
 stream_kernel(const Args a, int E) {
-  constexpr int KW = 4 / MW, BM = 16 * MW, BK = depth(MW), STAGES = stages(MW), LD = BK + 8, NWT = UP ? 2 : 1, PL = BM + 1;
+  constexpr int KW = 4 / MW, BM = 16 * MW, BK = depth(MW), STAGES = stages(MW), LD = BK + 8, NWT = MODE == GATED ? 2 : 1, PL = BM + 1;
+  constexpr bool UP = MODE != DOWN;
   constexpr int V = BK / 8, XR = NT * V / 128;                        // 16-byte pieces of a row; pieces of x per thread
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16* sw = sm;                                             // [STAGES][NWT][BM][LD]
@@ -80,7 +85,7 @@ stream_kernel(const Args a, int E) {
   auto enter = [&]() {
     if (!ld_more) return;
     w0 = reinterpret_cast<const __nv_bfloat16*>(a.w0) + ((long)ld.e * a.M + ld.m0) * a.K;
-    if (UP) w1 = reinterpret_cast<const __nv_bfloat16*>(a.w1) + ((long)ld.e * a.M + ld.m0) * a.K;
+    if (MODE == GATED) w1 = reinterpret_cast<const __nv_bfloat16*>(a.w1) + ((long)ld.e * a.M + ld.m0) * a.K;
     const int size = a.sizes[ld.e], off = a.offs[ld.e];
 #pragma unroll
     for (int j = 0; j < XR; ++j) {
@@ -98,7 +103,7 @@ stream_kernel(const Args a, int E) {
         const bool ok = ld.m0 + r < a.M && k0 + c < a.K;
         const long at = ok ? (long)r * a.K + k0 + c : 0;
         la_cp_async16(sw + ((ld_stage * NWT) * BM + r) * LD + c, w0 + at, ok ? 16 : 0);
-        if (UP) la_cp_async16(sw + ((ld_stage * NWT + NWT - 1) * BM + r) * LD + c, w1 + at, ok ? 16 : 0);
+        if (MODE == GATED) la_cp_async16(sw + ((ld_stage * NWT + NWT - 1) * BM + r) * LD + c, w1 + at, ok ? 16 : 0);
       }
 #pragma unroll
       for (int j = 0; j < XR; ++j) {
@@ -176,7 +181,8 @@ stream_kernel(const Args a, int E) {
         for (int q = 0; q < KW; ++q) v[wt] += part[((q * NWT + wt) * NT + t) * PL + r];
       }
       float o = v[0];
-      if constexpr (UP) o = clamped_act(a.wts[p] * v[0], a.wts[p] * v[NWT - 1], a.limit);
+      if constexpr (MODE == GATED) o = clamped_act(a.wts[p] * v[0], a.wts[p] * v[NWT - 1], a.limit);
+      if constexpr (MODE == RELU2) o = relu2(a.wts[p], v[0]);
       reinterpret_cast<__nv_bfloat16*>(a.out)[(long)p * a.M + it.m0 + r] = __float2bfloat16_rn(o);
     }
   }
@@ -184,9 +190,10 @@ stream_kernel(const Args a, int E) {
 }
 
 // one warp per output row, one pair at a time
-template <typename T, bool UP>
+template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 plain_kernel(const Args a) {
+  constexpr bool UP = MODE != DOWN;
   const int m = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (m >= a.M) return;
   for (int p = blockIdx.y; p < a.n; p += gridDim.y) {
@@ -196,10 +203,11 @@ plain_kernel(const Args a) {
     for (int c = lane; c < a.K; c += 32) {
       const float v = to_f(x[c]);
       g += to_f(reinterpret_cast<const T*>(a.w0)[wrow + c]) * v;
-      if (UP) u += to_f(reinterpret_cast<const T*>(a.w1)[wrow + c]) * v;
+      if (MODE == GATED) u += to_f(reinterpret_cast<const T*>(a.w1)[wrow + c]) * v;
     }
     g = warp_add(g);
-    if (UP) g = clamped_act(a.wts[p] * g, a.wts[p] * warp_add(u), a.limit);
+    if (MODE == GATED) g = clamped_act(a.wts[p] * g, a.wts[p] * warp_add(u), a.limit);
+    if (MODE == RELU2) g = relu2(a.wts[p], g);
     if (lane == 0) reinterpret_cast<T*>(a.out)[(long)p * a.M + m] = from_f<T>(g);
   }
 }
@@ -226,11 +234,28 @@ act_kernel(const __nv_bfloat16* __restrict__ gu, const float* __restrict__ wts, 
   }
 }
 
-template <bool UP, int MW>
+// the same for ungated experts: u [rows, F] -> h [rows, F]
+__global__ void __launch_bounds__(256)
+relu2_kernel(const __nv_bfloat16* __restrict__ u, const float* __restrict__ wts, const int* __restrict__ row_pair, const int* __restrict__ offs, int E, int F,
+             __nv_bfloat16* __restrict__ h) {
+  const long used = offs[E], per = F / 8;
+  for (long i = blockIdx.x * 256l + threadIdx.x; i < used * per; i += gridDim.x * 256l) {
+    const long r = i / per;
+    const int c = (int)(i % per) * 8, p = row_pair[r];
+    const float s = p < 0 ? 0.f : wts[p];
+    float v[8];
+    load_vec<8>(u + r * F + c, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = relu2(s, v[e]);
+    store_vec<8>(h + r * F + c, v);
+  }
+}
+
+template <int MODE, int MW>
 int stream(const Args& a, int E, int sms, cudaStream_t st) {
-  constexpr int BM = 16 * MW, STAGES = stages(MW), LD = depth(MW) + 8, NWT = UP ? 2 : 1, KW = 4 / MW;
+  constexpr int BM = 16 * MW, STAGES = stages(MW), LD = depth(MW) + 8, NWT = MODE == GATED ? 2 : 1, KW = 4 / MW;
   constexpr int smem = STAGES * (NWT * BM + NT) * LD * 2 + KW * NWT * NT * (BM + 1) * 4;
-  auto k = stream_kernel<UP, MW>;
+  auto k = stream_kernel<MODE, MW>;
   if (cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
   const long items = ((long)(a.n < E ? a.n : E) + a.n / NT) * ((a.M + BM - 1) / BM);       // at most
   const long slots = (long)sms * (227 * 1024 / (smem + 1024));
@@ -238,18 +263,18 @@ int stream(const Args& a, int E, int sms, cudaStream_t st) {
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
-template <bool UP>
+template <int MODE>
 int run(int f32, const Args& a, int E, int sms, cudaStream_t st) {
   if (a.n <= 0) return 0;
   if (!f32 && a.K % 8 == 0) {
     const long hit = a.n < E ? a.n : E;                     // experts that will find rows, at most
-    if (hit * ((a.M + 63) / 64) >= 2l * sms) return stream<UP, 4>(a, E, sms, st);
-    if (hit * ((a.M + 31) / 32) >= 2l * sms) return stream<UP, 2>(a, E, sms, st);
-    return stream<UP, 1>(a, E, sms, st);
+    if (hit * ((a.M + 63) / 64) >= 2l * sms) return stream<MODE, 4>(a, E, sms, st);
+    if (hit * ((a.M + 31) / 32) >= 2l * sms) return stream<MODE, 2>(a, E, sms, st);
+    return stream<MODE, 1>(a, E, sms, st);
   }
   const dim3 grid((a.M + 7) / 8, a.n < 65535 ? a.n : 65535);
-  if (f32) plain_kernel<float, UP><<<grid, 256, 0, st>>>(a);
-  else plain_kernel<__nv_bfloat16, UP><<<grid, 256, 0, st>>>(a);
+  if (f32) plain_kernel<float, MODE><<<grid, 256, 0, st>>>(a);
+  else plain_kernel<__nv_bfloat16, MODE><<<grid, 256, 0, st>>>(a);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }
 
@@ -258,22 +283,29 @@ int run(int f32, const Args& a, int E, int sms, cudaStream_t st) {
 
 using namespace mt::expert;
 
-// x [T, D], w0 / w1 [E, F, D], wts / idx [n] (pair t * k + c), sizes / offs / row_pair of mt_moe_sort -> h [n, F]
+// w1 null: ungated experts. x [T, D], w0 / w1 [E, F, D], wts / idx [n] (pair t * k + c), sizes / offs / row_pair of mt_moe_sort -> h [n, F]
 extern "C" int mt_expert_up(int f32, const void* x, const void* w0, const void* w1, const float* wts, const int* idx, const int* sizes, const int* offs,
                             const int* row_pair, int n, int k, int E, int F, int D, float limit, void* h, int sms, cudaStream_t st) {
-  return run<true>(f32, Args{x, w0, w1, wts, idx, sizes, offs, row_pair, n, k, F, D, limit, h}, E, sms, st);
+  const Args a{x, w0, w1, wts, idx, sizes, offs, row_pair, n, k, F, D, limit, h};
+  return w1 ? run<GATED>(f32, a, E, sms, st) : run<RELU2>(f32, a, E, sms, st);
 }
 
 // h [n, F], w [E, D, F] -> y [n, D]
 extern "C" int mt_expert_down(int f32, const void* h, const void* w, const int* idx, const int* sizes, const int* offs, const int* row_pair, int n, int E,
                               int D, int F, void* y, int sms, cudaStream_t st) {
-  return run<false>(f32, Args{h, w, nullptr, nullptr, idx, sizes, offs, row_pair, n, 1, D, F, 0.f, y}, E, sms, st);
+  return run<DOWN>(f32, Args{h, w, nullptr, nullptr, idx, sizes, offs, row_pair, n, 1, D, F, 0.f, y}, E, sms, st);
 }
 
-extern "C" int mt_expert_act(const void* gu, const float* wts, const int* row_pair, const int* offs, int E, int F, float limit, void* h, int rows_max, int sms,
-                             cudaStream_t st) {
+// gated: gu [rows, 2F] holds both up-projections; otherwise [rows, F]
+extern "C" int mt_expert_act(const void* gu, int gated, const float* wts, const int* row_pair, const int* offs, int E, int F, float limit, void* h, int rows_max,
+                             int sms, cudaStream_t st) {
   if (F % 8) return -1;
   const long blocks = ((long)rows_max * (F / 8) + 255) / 256;
+  if (!gated) {
+    relu2_kernel<<<(unsigned)(blocks < sms * 16l ? blocks : sms * 16l), 256, 0, st>>>(reinterpret_cast<const __nv_bfloat16*>(gu), wts, row_pair, offs, E, F,
+                                                                                     reinterpret_cast<__nv_bfloat16*>(h));
+    return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  }
   act_kernel<<<(unsigned)(blocks < sms * 16l ? blocks : sms * 16l), 256, 0, st>>>(reinterpret_cast<const __nv_bfloat16*>(gu), wts, row_pair, offs, E, F, limit,
                                                                                  reinterpret_cast<__nv_bfloat16*>(h));
   return cudaGetLastError() == cudaSuccess ? 0 : -3;

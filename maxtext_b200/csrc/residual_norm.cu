@@ -2,9 +2,11 @@
 //   x += mult * rms(branch) * (offset + w_post);    y = rms(x) * (offset + w_next)
 // The branch comes in the compute type (a GEMM output), x stays fp32, y is rounded once for the next GEMM. Without a branch it is the
 // plain norm of the stream. residual_join is the same for pre-norm layers: one or two branches, each with a factor, a bias and a norm of its own
-// or without, one factor per lane on their sum, and the stream handed on normalised or as it is. Also here: the ungated activation between the
-// two products of a feed-forward, and the gate of a per-layer token embedding. Bandwidth-bound.
+// or without, one factor per lane on their sum, and the stream handed on normalised or as it is. residual_gate is the same for sandwich-normed layers
+// whose branch is gated lane by lane, with layer or RMS norms; the branch may be a sum of rows that an index picks. Also here: the ungated
+// activations between the two products of a feed-forward, and the gate of a per-layer token embedding. Bandwidth-bound.
 #include "serving_common.cuh"
+#include "residual_gate.h"
 
 namespace mt {
 
@@ -159,11 +161,127 @@ residual_join_kernel(float* __restrict__ x, const JoinBranch a, const JoinBranch
   }
 }
 
+// Mean and sum of squared deviations of the row that a block holds in registers, `n` of its elements in this warp: the deviations are taken
+// from the warp's own mean, and the warps are joined by the shift of their means, so that one barrier is enough. `sh` holds one entry per warp.
+template <int VEC, int ITER>
+__device__ __forceinline__ float2 row_moments(const float (&v)[ITER][VEC], int D, bool centred, float3* sh) {
+  const int nt = blockDim.x, w0 = threadIdx.x & ~31;
+  int n = 0;
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    n += min(max(D - (i * nt + w0) * VEC, 0), 32 * VEC);
+    if ((i * nt + (int)threadIdx.x) * VEC < D) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) s += v[i][e];
+    }
+  }
+  const float mean = centred && n > 0 ? warp_add(s) / (float)n : 0.f;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < ITER; ++i)
+    if ((i * nt + (int)threadIdx.x) * VEC < D) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss += (v[i][e] - mean) * (v[i][e] - mean);
+    }
+  ss = warp_add(ss);
+  if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = make_float3(mean, ss, (float)n);
+  __syncthreads();
+  const int warps = (nt + 31) / 32;
+  float all = 0.f;
+  for (int i = 0; i < warps; ++i) all += sh[i].x * sh[i].z;
+  all /= (float)D;
+  float m2 = 0.f;
+  for (int i = 0; i < warps; ++i) m2 += sh[i].y + sh[i].z * (sh[i].x - all) * (sh[i].x - all);
+  return make_float2(all, m2);
+}
+
+// x += norm(b * sigmoid(g + bias)) * w_post;   y = norm(x) * w_next, or x, where b is the sum of `per_token` rows (dest: their numbers) and
+// `extra`, and norm subtracts the mean (centred) or not. Without a gate the factor is one; without rows x is only read; `fresh`: x is written
+// without being read. One CTA per row, a thread holds VEC neighbouring lanes ITER times.
+template <typename T, int VEC, int ITER>
+__global__ void __launch_bounds__(256)
+residual_gate_kernel(const ResidualGate a, int D) {
+  __shared__ float3 red[2][8];
+  const long r = blockIdx.x;
+  const int nt = blockDim.x;
+  float* xr = a.x + r * D;
+  float xv[ITER][VEC];
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int c = (i * nt + threadIdx.x) * VEC;
+    if (c < D && !a.fresh) load_vec<VEC>(xr + c, xv[i]);
+    else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) xv[i][e] = 0.f;
+    }
+  }
+  if (a.rows) {
+    float b[ITER][VEC];
+#pragma unroll
+    for (int i = 0; i < ITER; ++i) {
+      const int c = (i * nt + threadIdx.x) * VEC;
+      if (c >= D) continue;
+      float t[VEC];
+      if (a.extra) load_vec<VEC>(static_cast<const T*>(a.extra) + r * D + c, b[i]);
+      else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) b[i][e] = 0.f;
+      }
+      for (int j = 0; j < a.per_token; ++j) {
+        const long at = a.dest ? min(max((long)a.dest[r * a.per_token + j], 0l), a.n_rows - 1) : r * a.per_token + j;
+        load_vec<VEC>(static_cast<const T*>(a.rows) + at * D + c, t);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) b[i][e] += t[e];
+      }
+      if (a.gate) {
+        float g[VEC];
+        load_vec<VEC>(static_cast<const T*>(a.gate) + r * a.ldg + c, g);
+        load_vec<VEC>(static_cast<const T*>(a.bias) + c, t);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) b[i][e] *= sigmoid_t<T>(g[e] + t[e]);
+      }
+    }
+    const float2 m = row_moments<VEC, ITER>(b, D, a.centred, red[0]);
+    const float rstd = rsqrtf(m.y / (float)D + a.eps);
+#pragma unroll
+    for (int i = 0; i < ITER; ++i) {
+      const int c = (i * nt + threadIdx.x) * VEC;
+      if (c >= D) continue;
+      float w[VEC];
+      load_vec<VEC>(static_cast<const T*>(a.w_post) + c, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) xv[i][e] += (b[i][e] - m.x) * rstd * w[e];
+      store_vec<VEC>(xr + c, xv[i]);
+    }
+  }
+  if (!a.y) return;
+  float2 m = make_float2(0.f, 0.f);
+  float rstd = 1.f;
+  if (a.w_next) {
+    m = row_moments<VEC, ITER>(xv, D, a.centred, red[1]);
+    rstd = rsqrtf(m.y / (float)D + a.eps);
+  }
+#pragma unroll
+  for (int i = 0; i < ITER; ++i) {
+    const int c = (i * nt + threadIdx.x) * VEC;
+    if (c >= D) continue;
+    if (a.w_next) {
+      float w[VEC];
+      load_vec<VEC>(static_cast<const T*>(a.w_next) + c, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) xv[i][e] = (xv[i][e] - m.x) * rstd * w[e];
+    }
+    store_vec<VEC>(static_cast<T*>(a.y) + r * a.ldy + c, xv[i]);
+  }
+}
+
 __device__ __forceinline__ float act_value(float x, int code) {
   switch (code) {
     case 0: return silu_f(x);
     case 1: return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
     case 2: return fmaxf(x, 0.f);
+    case 5: return x > 0.f ? x * x : 0.f;
     default: return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
   }
 }
@@ -191,6 +309,32 @@ __global__ void act_kernel(const T* __restrict__ x, T* __restrict__ y, long n, i
     store_vec<8>(y + i * 8, v);
   }
   if (blockIdx.x == 0 && threadIdx.x < n - nv * 8) y[nv * 8 + threadIdx.x] = from_f<T>(act_typed<T>(to_f(x[nv * 8 + threadIdx.x]), code));
+}
+
+// The same over rows that lie in a wider matrix, x [rows, ldx] -> y [rows, F]. Code 6 is xIELU with its two numbers in `par`:
+// a z^2 + z / 2 for positive z, b (e^z - 1 - z) + z / 2 for the others, a = softplus(par 0), b = 1/2 + softplus(par 1).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+act_rows_kernel(const T* __restrict__ x, long ldx, T* __restrict__ y, long rows, int F, int code, const T* __restrict__ par) {
+  const long per = F / VEC;
+  const float a = code == 6 ? softplus_f(to_f(par[0])) : 0.f, b = code == 6 ? 0.5f + softplus_f(to_f(par[1])) : 0.f;
+  for (long i = blockIdx.x * 256l + threadIdx.x; i < rows * per; i += gridDim.x * 256l) {
+    const long r = i / per;
+    const int c = (int)(i % per) * VEC;
+    float v[VEC];
+    load_vec<VEC>(x + r * ldx + c, v);
+    if (code == 6) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const float z = v[e], neg = fminf(z, 0.f);
+        v[e] = (z > 0.f ? a * z * z : b * ((sizeof(T) == 2 && neg < -0.25f ? __expf(neg) - 1.f : expm1f(neg)) - neg)) + 0.5f * z;
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] = act_typed<T>(v[e], code);
+    }
+    store_vec<VEC>(y + r * F + c, v);
+  }
 }
 
 // out[n, c] = gelu_tanh(g[n, c]) * table[token[n], c]
@@ -233,6 +377,25 @@ int residual_join_t(float* x, const JoinBranch& a, const JoinBranch& b, const vo
     return go(residual_join_kernel<T, 4, 16>, 4, 16);
   }
   return D <= 1024 ? go(residual_join_kernel<T, 1, 4>, 1, 4) : go(residual_join_kernel<T, 1, 32>, 1, 32);
+}
+
+template <typename T>
+int residual_gate_t(const ResidualGate& a, long rows, int D, cudaStream_t st) {
+  auto go = [&](auto kernel, int vec, int iter) {
+    const int threads = (((D + vec * iter - 1) / (vec * iter)) + 31) / 32 * 32;
+    if (threads > 256) return -1;
+    kernel<<<(unsigned)rows, threads, 0, st>>>(a, D);
+    return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  };
+  uintptr_t bits = 0;
+  for (const void* p : {a.rows, a.extra, a.gate, a.bias, a.w_post, a.w_next, (const void*)a.x, (const void*)a.y}) bits |= reinterpret_cast<uintptr_t>(p);
+  const bool al = bits % 16 == 0;
+  if (D % 8 == 0 && al && (!a.gate || a.ldg % 8 == 0) && a.ldy % 8 == 0) {
+    if (D <= 2048) return go(residual_gate_kernel<T, 8, 1>, 8, 1);
+    if (D <= 4096) return go(residual_gate_kernel<T, 8, 2>, 8, 2);
+    if (D <= 8192) return go(residual_gate_kernel<T, 8, 4>, 8, 4);
+  }
+  return D <= 1024 ? go(residual_gate_kernel<T, 1, 4>, 1, 4) : go(residual_gate_kernel<T, 1, 32>, 1, 32);
 }
 
 template <typename T>
@@ -284,6 +447,24 @@ extern "C" int mt_token_gate(const void* g, const void* table, const int64_t* to
   const long blocks = (N * (dim / (v8 ? 8 : 1)) + 255) / 256;
   const unsigned grid = (unsigned)(blocks < sms * 8l ? blocks : sms * 8l);
 #define GO(T, V) token_gate_kernel<T, V><<<grid, 256, 0, st>>>((const T*)g, (const T*)table, tokens, N, dim, vocab, (T*)out)
+  if (f32) { if (v8) GO(float, 8); else GO(float, 1); }
+  else { if (v8) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
+#undef GO
+  return cudaGetLastError() == cudaSuccess ? 0 : -3;
+}
+
+extern "C" int mt_residual_gate(const ResidualGate* a, int f32, long rows, int D, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  return f32 ? residual_gate_t<float>(*a, rows, D, st) : residual_gate_t<__nv_bfloat16>(*a, rows, D, st);
+}
+
+extern "C" int mt_act_rows(const void* x, long ldx, void* y, int f32, long rows, int F, int code, const void* par, int sms, cudaStream_t st) {
+  if (rows <= 0 || F <= 0) return 0;
+  if (code == 6 && !par) return -1;
+  const bool v8 = F % 8 == 0 && ldx % 8 == 0 && (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y)) % 16 == 0;
+  const long blocks = (rows * (F / (v8 ? 8 : 1)) + 255) / 256;
+  const unsigned grid = (unsigned)(blocks < sms * 16l ? blocks : sms * 16l);
+#define GO(T, V) act_rows_kernel<T, V><<<grid, 256, 0, st>>>((const T*)x, ldx, (T*)y, rows, F, code, (const T*)par)
   if (f32) { if (v8) GO(float, 8); else GO(float, 1); }
   else { if (v8) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
 #undef GO

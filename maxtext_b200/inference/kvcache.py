@@ -122,11 +122,13 @@ class LayerKVCache:
       return self.quant.dequantize(x, sbuf[self.slot_ids, :upto], self.dtype)
     return x
 
-  def attend(self, q, k, v, ctx, window=0, soft_cap=0.0, sinks=None, chunk=0):
+  def attend(self, q, k, v, ctx, window=0, soft_cap=0.0, sinks=None, chunk=0, wide=False):
     """Append k/v of the S new tokens at each row's current length, then attend over everything cached (that `window` and `chunk` leave
-    visible)."""
+    visible). `wide`: q reads the keys of all key heads side by side."""
     B, S = q.shape[:2]
     if self.seq_size > 1:
+      if wide:
+        raise NotImplementedError("a sequence-split cache does not take heads that mix their scores")
       if chunk:
         raise NotImplementedError("a sequence-split cache does not take chunked attention")
       if getattr(ctx, "bidir", None) is not None:
@@ -136,13 +138,16 @@ class LayerKVCache:
     self._write(self.k, getattr(self, "ks", None), k)
     self._write(self.v, getattr(self, "vs", None), v)
     from ..ops import cached_attention as CA
-    if CA.attends(q, self, ctx):
+    if not wide and CA.attends(q, self, ctx):
       # flash kernel for prompts, split decode kernel for one new token per sequence (lengths stay on the device, no host sync)
       return CA.attend(q, k, v, self, ctx, window, soft_cap, sinks, chunk)
     upto = int((self.lengths.max() + S).item()) if ctx.mode != "prefill" else int(S + self.lengths.max().item())
     if self.new_lens is not None:
       upto = min(upto, self.max_len)                      # padding may run past the end of the cache
     K, V = self._read(self.k, getattr(self, "ks", None), upto), self._read(self.v, getattr(self, "vs", None), upto)
+    if wide:
+      from ..layers.blocks import side_by_side
+      K = side_by_side(K)
     kv_pos = torch.arange(upto, device=q.device)[None].expand(B, upto)
     valid_len = (self.lengths + S)[:, None]
     packed = ctx.segment_ids is not None and ctx.mode == "prefill" and ctx.segment_ids.shape[1] == upto
@@ -230,7 +235,7 @@ def _block_cache(attn, plan, slots, max_len, dt, device, quant, seq):
 
 
 def make_caches(model, slots: int, max_len: int, device, quantize: bool = False):
-  """One cache per attention block of the model, in layer order."""
+  """One cache per attention block and run of its layer (a layer that runs several times has a cache for each pass), in running order."""
   c = model.config
   dt = model.store.compute_dtype
   quant = KVQuant(c.kv_quant_dtype) if (quantize or c.quantize_kvcache) else None
@@ -238,7 +243,7 @@ def make_caches(model, slots: int, max_len: int, device, quantize: bool = False)
   seq_size = mesh.axis_size("context_autoregressive") if mesh is not None else 1
   seq = dict(seq_group=mesh.group("context_autoregressive"), seq_rank=mesh.axis_index("context_autoregressive"), seq_size=seq_size) if seq_size > 1 else {}
   out = []
-  for layer in model.layers:
+  for layer in model.runs:
     per_layer = []
     for blk in layer.blocks:
       if seq_size > 1 and (blk.plan.attention in ("mla", "parallel", "compressed") or recurrent(blk.plan)):

@@ -211,6 +211,15 @@ class FusedParam:
     return (sum(self.rows), self.parts[0].shape[1])
 
 
+def back_to_back(b: Builder, parts: list):
+  """Moves parameters of a unit under construction next to each other, so that everything which reads one input can be one operand. Returns it,
+  or None when the parts do not fit together (vector loads need every part to begin on 16 bytes)."""
+  at = min(i for i, p in enumerate(b.params) if any(p is q for q in parts))
+  rest = [p for p in b.params[at:] if not any(p is q for q in parts)]
+  b.params[at:] = parts + rest
+  return FusedParam(parts) if FusedParam.possible(parts) and all(p.shape[0] % 8 == 0 for p in parts) else None
+
+
 # ------------------------------------------------------------------------------------------ tensor-parallel glue
 class _CopyToTP(torch.autograd.Function):
   """Identity forward, all-reduce backward (input of a column-parallel linear)."""
@@ -275,8 +284,8 @@ class Norm:
     self.bias = nb.vector("bias", dim, axes, init="zeros") if kind == "layernorm" else None
 
   def __call__(self, x):
-    if self.kind == "layernorm":
-      return ref.layernorm(x, self.scale.leaf(), self.bias.leaf(), self.eps)
+    if self.kind in ("layernorm", "layernorm_scale"):
+      return ref.layernorm(x, self.scale.leaf(), self.bias.leaf() if self.bias is not None else None, self.eps)
     if self.scale is None:
       xf = x.float()
       return (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + self.eps)).to(x.dtype)
@@ -289,7 +298,8 @@ class HeadSizes:
   """Sizes of one attention layer; `scale` multiplies q . k, `soft_cap` (0: none) bounds the result. `gate`: an output gate per lane
   ("lane"), per head ("head") or none. `q_temp` = (coef, every): q grows by 1 + coef ln(floor((p + 1) / every) + 1) at position p.
   `diff`: differential attention (Ye et al., "Differential Transformer"): two maps per head over the same values, the second subtracted
-  with a learned weight around `diff`. `sink`: a constant score in the softmax denominator, without a value."""
+  with a learned weight around `diff`. `sink`: a constant score in the softmax denominator, without a value. `talk`: a matrix mixes the heads'
+  scores in front of the softmax (Shazeer et al., "Talking-Heads Attention")."""
   heads: int
   kv_heads: int
   dim: int
@@ -300,6 +310,12 @@ class HeadSizes:
   q_temp: tuple | None = None
   diff: float | None = None
   sink: float | None = None
+  talk: bool = False
+
+
+def side_by_side(k: torch.Tensor) -> torch.Tensor:
+  """Keys [B, S, G, D] as every key head sees them where heads mix their scores: all of them in one, [B, S, G, G * D]."""
+  return k.flatten(2)[:, :, None].expand(-1, -1, k.shape[2], -1)
 
 
 class Constant:
@@ -339,6 +355,7 @@ class Attention:
     self.window, self.inv_ts, self.interleaved, self.use_rope = window, rope_inv_ts, interleaved, use_rope
     self.qk_norm, self.query_scalar, self.soft_cap, self.rotary_dim = qk_norm, query_scalar, soft_cap, rotary_dim
     self.l2_qk_norm, self.temperature_tuning, self.chunk = l2_qk_norm, temperature_tuning, int(chunk)
+    self.talk = None
     # maps per head (two in differential attention); the cache keeps them side by side as one key of width kw
     self.maps = 2 if sizes is not None and sizes.diff is not None else 1
     self.kw = self.dh * self.maps
@@ -403,6 +420,9 @@ class Attention:
     self.sinks = ab.vector("sinks", self.hq, ("q_heads",), init="zeros", tp=True) if sinks else None
     if sizes is not None and sizes.sink is not None:
       self.sinks = Constant(torch.full((self.hq * self.maps,), float(sizes.sink), device=rope_inv_ts.device))
+    if sizes is not None and sizes.talk:
+      assert tp == 1 and self.maps == 1 and not gated and not soft_cap, "heads that mix their scores: no second map, gate, cap or tensor split"
+      self.talk = ab.sub("talk").table("kernel", (self.hq, self.hq), (None, None), init="identity")
     self.lam = None
     if self.maps == 2:
       assert tp == 1, "differential attention is not split over the tensor axis"
@@ -413,6 +433,12 @@ class Attention:
     if isinstance(self.sinks, Constant) and self.sinks.data.dtype != dtype:
       self.sinks.data = self.sinks.data.to(dtype)
     return self.sinks.data if self.sinks is not None else None
+
+  def _mix_scores(self, q):
+    """q [B, S, H, D] -> [B, S, H, G * D]: sum_g T[h, g] (q_g . k_g) as one product with the keys of all key heads side by side."""
+    B, S, H, D = q.shape
+    T = self.talk.leaf().float().view(H, self.hkv_l, H // self.hkv_l)
+    return torch.einsum("hcj,bscjd->bshcd", T, q.float().view(B, S, self.hkv_l, -1, D)).reshape(B, S, H, -1).to(q.dtype)
 
   def _maps_apart(self, q):
     """q [B, S, heads * 2, dim] -> [B, S, heads * 2, 2 * dim]: map j of a head meets its own half of the cached key (both halves share the
@@ -460,8 +486,9 @@ class Attention:
         rows = torch.split(F.linear(x, self.qkvg).view(B * S, -1), self.qkvg.rows, dim=-1)
       else:
         rows = [F.linear(x, w).view(B * S, -1) for w in self.in_parts]
-    q, k, v = rows[:3]
-    return F.linear(CA.serve(self, q, k, v, rows[3] if self.g is not None else None, ctx).view(B, S, -1), self.o)
+    q, k = rows[:2]
+    v = k if self.share_kv else rows[2]
+    return F.linear(CA.serve(self, q, k, v, rows[-1] if self.g is not None else None, ctx).view(B, S, -1), self.o)
 
   def __call__(self, x, ctx, rows=None, out_bias=True):
     """`out_bias=False` leaves the output projection's bias to the caller (it may join a later step)."""
@@ -523,6 +550,8 @@ class Attention:
         q = (q.float() * sc[:, :, None, None]).to(q.dtype)
       if self.maps == 2:
         q, k = self._maps_apart(q), k.reshape(B, S, self.hkv_l, self.kw)
+      if self.talk is not None:
+        q = self._mix_scores(q)
       if moba:
         # mixture-of-block attention: each query attends its own block and the best `moba_topk` earlier key blocks
         seg = None
@@ -537,7 +566,11 @@ class Attention:
         out = F.attention(q, k, v, ctx.positions, ctx.segment_ids, 1.0, self.soft_cap, self.window, chunk=self.chunk,
                           sinks=self.sinks.leaf() if self.sinks is not None else None)
       elif ctx.cache is not None:
-        out = ctx.cache.attend(q, k, v, ctx, window=self.window, soft_cap=self.soft_cap, sinks=self.sinks, chunk=self.chunk)
+        out = ctx.cache.attend(q, k, v, ctx, window=self.window, soft_cap=self.soft_cap, sinks=self.sinks, chunk=self.chunk, wide=self.talk is not None)
+      elif self.talk is not None:
+        assert ctx.cp_size == 1, "heads that mix their scores are not split along the sequence"
+        m = ref.attention_mask(ctx.positions, ctx.positions, ctx.segment_ids, ctx.segment_ids, True, self.window, self.chunk)
+        out = ref.attention(q, side_by_side(k), v, m, 1.0, sinks=self.sinks.leaf() if self.sinks is not None else None)
       elif ctx.cp_size > 1:
         from ..parallel.context_parallel import context_attention
         out = context_attention(q, k, v, ctx.positions, ctx.segment_ids, ctx, 1.0, self.soft_cap, self.window)
@@ -691,7 +724,8 @@ def _max_logit_per_head(q, k, positions, segment_ids, chunk: int = 512) -> torch
 
 # ------------------------------------------------------------------------------------------ dense MLP
 class MLP:
-  """wo( act(wi_0 x) * (wi_1 x) ) (src/maxtext/layers/linears.py:422-625)."""
+  """wo( act(wi_0 x) * (wi_1 x) ) (src/maxtext/layers/linears.py:422-625); with one activation wo( act(wi x) ), where "xielu" has two learned
+  numbers (Huang and Schlag, "Deriving Activation Functions Using Integration")."""
 
   def __init__(self, b: Builder, config, name="mlp", hidden: int | None = None, acts=None, bias=False):
     c = config
@@ -703,13 +737,18 @@ class MLP:
     self.wi_0 = mb.sub("wi_0" if self.gated else "wi").linear("kernel", (d,), (f,), ("embed", "mlp"), tp="col")
     self.wi_1 = mb.sub("wi_1").linear("kernel", (d,), (f,), ("embed", "mlp"), tp="col") if self.gated else None
     self.wo = mb.sub("wo").linear("kernel", (f,), (d,), ("mlp", "embed"), tp="row")
+    self.in_parts = [p for p in (self.wi_0, self.wi_1) if p is not None]
+    self.act_params = mb.vector("act", 2, (None,)) if self.acts[0] == "xielu" else None
     self.wi = FusedParam([self.wi_0, self.wi_1]) if self.gated and FusedParam.possible([self.wi_0, self.wi_1]) else None
     self.bi = mb.sub("wi_0" if self.gated else "wi").vector("bias", f, ("mlp",), init="zeros", tp=True) if bias else None
     self.bo = mb.sub("wo").vector("bias", d, ("embed",), init="zeros") if bias else None
     if self.bo is not None and b.tp_size > 1 and sp_enabled(c):
       self.bo.pdef.tp_partial = True
 
-  def __call__(self, x, ctx):
+  def __call__(self, x, ctx, rows=None):
+    """`rows`: the up-projection of an ungated layer, when it was part of a wider product."""
+    if rows is not None:
+      return F.linear(F.act(rows, self.acts[0], self.act_params).view(*x.shape[:-1], -1), self.wo, bias=self.bo)
     tp_rt = tp_fused.runtime_for(ctx, x, x.shape[-1]) if ctx.tp_size > 1 else None
     fuse_in = tp_rt is not None and self.gated and self.wi is not None and self.wi.fusable()
     if not fuse_in:
@@ -724,7 +763,7 @@ class MLP:
       h = F.gated_act(gu, self.acts[0])
     else:
       h = F.linear(x, self.wi_0, bias=self.bi)
-      h = F.act(h, self.acts[0])
+      h = F.act(h, self.acts[0], self.act_params)
     if tp_rt is not None and ctx.reuse("mlpwo") is None and self.bo is None and self.wo.lora is None:
       y = F.linear(h, self.wo, tp_reduce=tp_rt)
     else:

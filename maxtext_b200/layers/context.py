@@ -75,6 +75,8 @@ class LayerCtx:
   new_lens: torch.Tensor | None = None  # [B] real tokens per row of a right-padded inference batch (None: all of them)
   next_norm: object = None           # fp32 residual streams: the norm that reads the stream after the current layer ...
   normed: torch.Tensor | None = None  # ... and its output, handed from the layer that computed it to the one that reads it
+  origin: torch.Tensor | None = None  # models whose layers run in a loop: the embedding output in the compute type, which every pass reads again ...
+  beside: torch.Tensor | None = None  # ... and (inference) the rows [stream | embedding output] that it reads them from
   name_prefix: str = ""              # disambiguates blocks that share a layer (gemma2 local/global)
   batch_split: int = 1               # > 1: every decoder layer runs the batch as that many micro-batches on alternating streams
   micro_slot: int = 0                # which micro-batch of a split layer this context describes

@@ -102,7 +102,8 @@ class RoutedMoE:
     src/maxtext/layers/moe.py:752,902-906,1051-1053) or "gpt_oss" (router bias on the logits, per-expert biases and the
     clamped x * sigmoid(1.702 x) * (up + 1) activation; moe.py:617-637,841-853,2239-2242), or "scaled_input": the top-k sigmoid
     scores, not renormalised, scale what each chosen expert reads, experts with the clamped activation and no biases; the router and
-    the scores are fp32. `sizes` replaces the config's sizes."""
+    the scores are fp32; or "prob_weighted": the top-k soft-max probabilities, not renormalised, weight what each chosen expert gives, experts
+    wo relu(wi x)^2 without a gate and biases, fp32 router. `sizes` replaces the config's sizes."""
     c = config
     self.c = c
     self.style = style
@@ -113,14 +114,15 @@ class RoutedMoE:
     mb = b.sub(name)
     d, f = c.emb_dim, sizes.ff
     self.gate = mb.sub("gate").linear("kernel", (d,), (self.E,), ("embed", None))
-    self.gate_bias = mb.sub("gate").vector("bias", self.E, (None,), init="zeros") if c.routed_bias and style != "scaled_input" else None
+    plain = style in ("scaled_input", "prob_weighted")         # fp32 router without a bias, experts without biases
+    self.gate_bias = mb.sub("gate").vector("bias", self.E, (None,), init="zeros") if c.routed_bias and not plain else None
     self.wi_0 = mb.experts("wi_0", self.E, d, f, ("exp", "embed_moe", "mlp_moe"), tp="col")
-    self.wi_1 = mb.experts("wi_1", self.E, d, f, ("exp", "embed_moe", "mlp_moe"), tp="col")
+    self.wi_1 = mb.experts("wi_1", self.E, d, f, ("exp", "embed_moe", "mlp_moe"), tp="col") if style != "prob_weighted" else None
     self.wo = mb.experts("wo", self.E, f, d, ("exp", "mlp_moe", "embed_moe"), tp="row")
     self.act = c.mlp_activations[0]
     self.e_local = self.E // b.ep_size
     self.b0 = self.b1 = self.bo = None
-    if c.mlp_bias and style != "scaled_input":
+    if c.mlp_bias and not plain:
       self.b0 = mb.table("wi_0_bias", (self.E, f), ("exp", "activation_mlp"), init="zeros")
       self.b1 = mb.table("wi_1_bias", (self.E, f), ("exp", "activation_mlp"), init="zeros")
       self.bo = mb.table("wo_bias", (self.E, d), ("exp", "activation_embed"), init="zeros")
@@ -142,6 +144,10 @@ class RoutedMoE:
     w = self.gate.leaf()
     if self.style == "scaled_input":
       probs = torch.sigmoid(torch.nn.functional.linear(src.float(), w.float()))
+      wts, idx = probs.topk(self.k, dim=-1)
+      return wts, idx, self._aux(probs, idx, B, S, ctx)
+    if self.style == "prob_weighted":
+      probs = torch.softmax(torch.nn.functional.linear(src.float(), w.float()), -1)
       wts, idx = probs.topk(self.k, dim=-1)
       return wts, idx, self._aux(probs, idx, B, S, ctx)
     logits = torch.nn.functional.linear(xg, w.to(xg.dtype))
@@ -235,6 +241,8 @@ class RoutedMoE:
   # ---- expert FFN on rows grouped by (local) expert
   def experts_ffn(self, rows, sizes):
     g = moe_ops.grouped_linear(rows, self.wi_0, sizes)
+    if self.wi_1 is None:
+      return moe_ops.grouped_linear(F.act(g, "relu2"), self.wo, sizes)
     u = moe_ops.grouped_linear(rows, self.wi_1, sizes)
     row_e = None
     if self.b0 is not None:
@@ -276,8 +284,8 @@ class RoutedMoE:
 
   def __call__(self, x, ctx, gate_inputs=None, rows_ok=False):
     """`rows_ok`: a GPU inference pass may return the experts' output rows (`moe_ops.ExpertRows`) instead of their sum per token."""
-    if self.style == "scaled_input" and moe_ops.serve_ok(x, ctx):
-      out = moe_ops.serve_scaled(x.reshape(-1, x.shape[-1]), self)
+    if self.style in ("scaled_input", "prob_weighted") and moe_ops.serve_ok(x, ctx):
+      out = moe_ops.serve_scored(x.reshape(-1, x.shape[-1]), self)
       return out if rows_ok else out.combine(x)
     if ctx.sp and ctx.tp_size > 1:
       assert gate_inputs is None, "a separate router input is not implemented under tensor-sequence parallelism"
@@ -319,7 +327,7 @@ class RoutedMoE:
       x2, wts_fused = tp_enter(x2, ctx), tp_enter(wts, ctx)
     else:
       wts_fused = wts
-    plain_ffn = self.b0 is None and self.style not in ("gpt_oss", "scaled_input")
+    plain_ffn = self.b0 is None and self.style not in ("gpt_oss", "scaled_input", "prob_weighted")
     if plain_ffn and ctx.ep_size == 1 and self.act in F._ACT_CODE and moe_ops.padded_path_supported(x2, D, self.wi_0.data.shape[1], self.E):
       # GPU path: device-side stable sort into 128-row-padded expert groups, grouped tcgen05 GEMMs, no host synchronisation
       out = moe_ops.moe_ffn_padded(x2, wts_fused, idx, self.wi_0, self.wi_1, self.wo, self.E, self.act)
@@ -392,9 +400,17 @@ class Gemma4MoE:
 class RoutedAndSharedMoE:
   """Routed experts plus always-on shared experts (src/maxtext/layers/moe.py:3259-3371)."""
 
-  def __init__(self, b: Builder, config, name="DeepSeekMoeBlock_0", style: str = "", hash_routing: bool = False):
+  def __init__(self, b: Builder, config, name="DeepSeekMoeBlock_0", style: str = "", hash_routing: bool = False, sizes: MoESizes | None = None,
+               shared_ff: int | None = None):
+    """With `sizes` the routed layer has sizes of its own, and `shared_ff` is the width of the shared expert (None: there is none), whose form is
+    that of the routed ones."""
     mb = b.sub(name)
     self.shared_gate = None
+    if sizes is not None:
+      assert style == "prob_weighted", f"routed layers of style {style!r} with sizes of their own have no shared expert"
+      self.routed = RoutedMoE(mb, config, "routed_experts", style=style, sizes=sizes)
+      self.shared = MLP(mb, config, "shared_expert", hidden=shared_ff, acts=["relu2"]) if shared_ff else None
+      return
     if style == "qwen3_next":
       # src/maxtext/models/qwen3.py:1107-1193: softmax top-k router, one shared expert whose output is scaled per token by
       # sigmoid(x . w_gate)
@@ -406,10 +422,14 @@ class RoutedAndSharedMoE:
     self.shared = MLP(mb, config, "shared_experts", hidden=config.shared_experts * config.moe_mlp_dim) \
         if config.shared_experts > 0 else None
 
-  def __call__(self, x, ctx):
-    y = self.routed(x, ctx)
+  def __call__(self, x, ctx, rows_ok=False, shared_rows=None):
+    """`rows_ok`: see `RoutedMoE`; `shared_rows`: the shared expert's up-projection, when it was part of a wider product."""
+    y = self.routed(x, ctx, rows_ok=rows_ok)
     if self.shared is not None:
-      sh = self.shared(x, ctx)
+      sh = self.shared(x, ctx, rows=shared_rows) if shared_rows is not None else self.shared(x, ctx)
+      if isinstance(y, moe_ops.ExpertRows):
+        y.extra = sh
+        return y
       if self.shared_gate is not None:
         gate = torch.nn.functional.linear(x.float(), self.shared_gate.leaf().float())
         sh = (sh.float() * torch.sigmoid(gate)).to(sh.dtype)

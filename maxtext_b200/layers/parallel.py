@@ -9,7 +9,7 @@ from __future__ import annotations
 import torch
 
 from ..ops import functional as F
-from .blocks import Builder, FusedParam, Norm
+from .blocks import Builder, Norm, back_to_back
 
 
 class ParallelMixer:
@@ -21,13 +21,7 @@ class ParallelMixer:
     self.left, self.right, self.factors = build_left(ab, "left"), build_right(ab, "right"), (float(join[0]), float(join[1]))
     self.norms = tuple(Norm(ab, n, c.emb_dim, c.normalization_layer_epsilon) if join[2] else None for n in ("left_norm", "right_norm"))
     self.parts = self.left.in_parts + self.right.in_parts
-    # back to back in the unit, so that they can be one operand
-    at = max(i for i, p in enumerate(ab.params) if any(p is q for q in self.left.in_parts))
-    rest = [p for p in ab.params[at + 1:] if not any(p is q for q in self.right.in_parts)]
-    ab.params[at + 1:] = self.right.in_parts + rest
-    # vector loads need every part to begin on 16 bytes
-    fits = FusedParam.possible(self.parts) and all(p.shape[0] % 8 == 0 for p in self.parts)
-    self.fused = FusedParam(self.parts) if fits else None
+    self.fused = back_to_back(ab, self.parts)
 
   def __call__(self, x, ctx):
     cache = ctx.cache

@@ -19,6 +19,7 @@ class Family:
   norm_offset: float = 0.0
   scale_embedding: bool = False
   residual_fp32: bool = False              # the residual stream and the logits are fp32 whatever the compute dtype
+  embed_norm: bool = False                 # a norm on the token embeddings
   static_streams: bool = False             # mhc_expansion_rate fp32 streams, mixed by constants of the model instead of per-token maps
 
 
@@ -31,6 +32,8 @@ def describe(c) -> Family:
     return Family(norm_kind="layernorm")
   if blk in ("qwen3_next", "qwen3_5"):
     return Family(norm_offset=1.0)           # every RMS scale is stored zero-centred and applied as (1 + scale)
+  if blk == "gukirax":
+    return Family(norm_kind="layernorm_scale", residual_fp32=True, embed_norm=True)
   if blk == "silinex":
     return Family(norm_offset=1.0, residual_fp32=True)
   if blk == "sitivik":
@@ -70,6 +73,15 @@ def rope_tables(c, device) -> dict:
     tables["gemma4_global"] = (prop(g_dim, float(c.global_rope_proportion), g_max), False)
     tables["gemma4_local"] = (prop(int(c.head_dim), float(c.local_rope_proportion), local_max), False)
   return tables
+
+
+def layer_runs(c) -> list[int]:
+  """Layer numbers in running order (`layer_loop`: layers start .. stop - 1 run `times` times in a row, with the same weights)."""
+  n, loop = len(layer_plans(c)), c.layer_loop
+  if not loop:
+    return list(range(n))
+  a, b = int(loop["start"]), int(loop["stop"])
+  return [*range(a), *(list(range(a, b)) * int(loop["times"])), *range(b, n)]
 
 
 def _llama_like(c, **kw) -> BlockPlan:
@@ -172,6 +184,9 @@ def layer_plans(c) -> list[LayerPlan]:
     for i in range(nh, n, 2):
       plans.append(LayerPlan("scanned_blocks", [v4(ratios[i], "layers_0"), v4(ratios[i + 1], "layers_1")]))
     return plans
+  if blk == "gukirax":
+    from .gukirax import layer_plans as gukirax_plans
+    return gukirax_plans(c)
   if blk == "silinex":
     from .silinex import layer_plans as silinex_plans
     return silinex_plans(c)
@@ -238,4 +253,4 @@ def layer_plans(c) -> list[LayerPlan]:
     return plans
   raise NotImplementedError(
       f"decoder_block={blk!r} parses but has no model implementation here yet (implemented: llama2, mistral, mixtral, "
-      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, silinex, sitivik, tipidra, simple)")
+      "deepseek, gemma, gemma2, gemma3, qwen2, qwen3, qwen3_moe, qwen3_next, qwen3_5, gpt3, gpt_oss, olmo3, llama4, envy, gemma4, deepseek4, gukirax, silinex, sitivik, tipidra, simple)")

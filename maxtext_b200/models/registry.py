@@ -13,9 +13,9 @@ import struct
 
 import torch
 
-from . import silinex, sitivik, tipidra
+from . import gukirax, silinex, sitivik, tipidra
 
-ARCHITECTURES = {"Silinex": silinex, "Sitivik": sitivik, "Tipidra": tipidra}
+ARCHITECTURES = {"Gukirax": gukirax, "Silinex": silinex, "Sitivik": sitivik, "Tipidra": tipidra}
 
 
 def _safetensors_files(path: str) -> list[str]:

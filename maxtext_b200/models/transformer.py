@@ -57,7 +57,7 @@ class BlockPlan:
   l2_qk_norm: bool = False               # llama4: scale-free RMS normalisation of q and k after RoPE
   temperature_tuning: bool = False       # llama4 NoPE layers: position-dependent query scale
   chunk: int = 0                         # llama4 RoPE layers: attention restricted to chunks of this many tokens
-  moe_style: str = ""                    # "" | "llama4" | "gpt_oss" | "scaled_input"
+  moe_style: str = ""                    # "" | "llama4" | "gpt_oss" | "scaled_input" | "prob_weighted"
   moe: dict | None = None                # router and expert sizes of this block, for families whose layers differ (None: the config's)
   head_dim: int | None = None            # gemma4 global layers: own head width ...
   kv_heads: int | None = None            # ... and key / value head count
@@ -74,6 +74,8 @@ class BlockPlan:
   gate: str = "lane"                     # `mixer` attention: one output gate per "lane" or per "head"
   sink_value: float | None = None        # `mixer` attention: a constant sink score instead of learned ones
   layer_scale: bool = False              # one learned factor per lane on every branch before it joins the stream
+  residual_gate: bool = False            # sigmoid of a projection of the sublayer's input, lane by lane, on every branch in front of its norm (sandwich norms)
+  talk: bool = False                     # `mixer` attention: a matrix mixes the heads' scores
   token_side: int = 0                    # width of the per-layer token input that joins the stream after the feed-forward (0: none)
   compress_ratio: int = 0                # DeepSeek-V4 compressed attention: 0 (window only), 4 (sparse) or 128 (heavy)
 
@@ -82,6 +84,7 @@ class BlockPlan:
 class LayerPlan:
   stack: str = "layers"                  # name of the stacked collection in the checkpoint tree
   blocks: list = field(default_factory=lambda: [BlockPlan()])
+  pass_input: bool = False               # first layer of a loop: reads a projection of [stream | embedding output]
 
 
 def build_mixer(b: L.Builder, c, plan: BlockPlan, name: str, rope_tables: dict):
@@ -126,7 +129,7 @@ def build_mixer(b: L.Builder, c, plan: BlockPlan, name: str, rope_tables: dict):
     inv_ts = ref.rope_inv_timescale(rot, 1.0, float(turn["base"]), stretch=turn.get("scaling")).to(inv_ts.device)
     temp = m.get("q_temp")
     sizes = L.HeadSizes(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), float(m.get("softcap", 0.0)), plan.gate,
-                        (float(temp["coef"]), float(temp["every"])) if temp else None, float(m["diff"]) if "diff" in m else None, plan.sink_value)
+                        (float(temp["coef"]), float(temp["every"])) if temp else None, float(m["diff"]) if "diff" in m else None, plan.sink_value, plan.talk)
     window, chunk = (int(m["mask"]["size"]) if plan.mask == kind else 0 for kind in ("window", "chunk"))
   return L.Attention(b, c, name, window, inv_ts, interleaved, plan.use_rope and rot != 0, plan.qk_norm,
                      plan.query_scalar, plan.soft_cap, plan.attn_bias,
@@ -155,10 +158,14 @@ class DecoderBlock:
     self.attn = build_mixer(b, c, plan, plan.attn_name + s, rope_tables)
     self.n1b = mk(plan.post_attn_norm) if plan.post_attn_norm else None
     self.n2 = mk(plan.pre_mlp_norm) if plan.pre_mlp_norm else None
+    r = plan.moe
+    moe_sizes = M.MoESizes(int(r["router"]["experts"]), int(r["router"]["top"]), int(r["expert"]["ff"]), float(r["expert"].get("limit", 0.0))) \
+        if r is not None else None
     if plan.mlp == "moe":
-      r = plan.moe
-      self.mlp = M.RoutedMoE(b, c, plan.mlp_name + s, style=plan.moe_style, sizes=M.MoESizes(
-          int(r["router"]["experts"]), int(r["router"]["top"]), int(r["expert"]["ff"]), float(r["expert"]["limit"])) if r is not None else None)
+      self.mlp = M.RoutedMoE(b, c, plan.mlp_name + s, style=plan.moe_style, sizes=moe_sizes)
+    elif plan.mlp == "moe_shared" and r is not None:
+      self.mlp = M.RoutedAndSharedMoE(b, c, plan.mlp_name + s, style=plan.moe_style, sizes=moe_sizes,
+                                      shared_ff=int(r["shared"]["ff"]) if r.get("shared") is not None else None)
     elif plan.mlp == "moe_shared":
       hashed = layer_index is not None and layer_index < int(getattr(c, "first_num_hash_layers", 0) or 0) and plan.moe_style == ""
       self.mlp = M.RoutedAndSharedMoE(b, c, plan.mlp_name + s, style=plan.moe_style, hash_routing=hashed)
@@ -171,6 +178,16 @@ class DecoderBlock:
     self.n2b = mk(plan.post_mlp_norm) if plan.post_mlp_norm else None
     self.ls1 = b.sub("layer_scale").vector("mixer" + s, c.emb_dim) if plan.layer_scale else None
     self.ls2 = b.sub("layer_scale").vector("mlp" + s, c.emb_dim) if plan.layer_scale and self.mlp is not None else None
+    self.rg1 = self.rg2 = None
+    if plan.residual_gate:
+      gate = lambda name: (b.sub("residual_gate", name).linear("kernel", (c.emb_dim,), (c.emb_dim,), ("embed", "embed_out"), "fan_in_normal"),  # noqa: E731
+                           b.sub("residual_gate", name).vector("bias", c.emb_dim, ("norm",), init="zeros"))
+      self.rg1 = gate("mixer" + s)
+      self.rg2 = gate("mlp" + s) if self.mlp is not None else None
+      # a gate and what else reads its input as one product (inference)
+      up = self.mlp if isinstance(self.mlp, L.MLP) else getattr(self.mlp, "shared", None)
+      self.mixer_in = L.back_to_back(b, self.attn.in_parts + [self.rg1[0]])
+      self.mlp_in = L.back_to_back(b, up.in_parts + [self.rg2[0]]) if up is not None and not up.gated else None
     self.side = None
     if plan.token_side:
       from ..layers.parallel import TokenSide
@@ -204,6 +221,8 @@ class DecoderBlock:
       return self.mhc_mlp(self.n2, lambda h: self.mlp(h, ctx), x)
     if self.hc1 is not None:
       return self._call_static_streams(x, ctx)
+    if self.plan.residual_gate:
+      return self._call_gated_stream(x, ctx)
     if self.plan.residual_fp32:
       return self._call_fp32_stream(x, ctx) if self.n1b is not None else self._call_joined_stream(x, ctx)
     a = self.attn(self.n1(x) if self.n1 is not None else x, ctx)
@@ -254,6 +273,27 @@ class DecoderBlock:
     return x
 
 
+  def _call_gated_stream(self, x, ctx: LayerCtx):
+    """x fp32 [B, S, D], sandwich norms. One product for everything that reads a sublayer's input, the branch's gate included, and one kernel per
+    border between sublayers: gate, the branch's norm, the residual add and what reads the stream next."""
+    h = ctx.normed if ctx.normed is not None else F.stream_norm(x, self.n1, self.n1.scale.data.dtype)
+    ctx.normed = None
+    if self.mixer_in is not None and self.attn.serves(h, ctx) and self.mixer_in.fusable():
+      rows = torch.split(F.linear(h, self.mixer_in).flatten(0, 1), self.mixer_in.rows, dim=-1)
+      a, g = self.attn(h, ctx, rows=rows[:-1]), rows[-1]
+    else:
+      a, g = self.attn(h, ctx), F.linear(h, self.rg1[0])
+    if self.mlp is None:
+      x, ctx.normed = F.residual_gate(x, a, g, self.rg1[1], self.n1b, ctx.next_norm)
+      return x
+    x, h = F.residual_gate(x, a, g, self.rg1[1], self.n1b, self.n2)
+    dense, up, g = isinstance(self.mlp, L.MLP), None, None
+    if self.mlp_in is not None and not torch.is_grad_enabled() and ctx.tp_size == 1 and self.mlp_in.fusable():
+      up, g = torch.split(F.linear(h, self.mlp_in).flatten(0, 1), self.mlp_in.rows, dim=-1)
+    f = self.mlp(h, ctx, rows=up) if dense else self.mlp(h, ctx, rows_ok=True, shared_rows=up)
+    x, ctx.normed = F.residual_gate(x, f, g if g is not None else F.linear(h, self.rg2[0]), self.rg2[1], self.n2b, ctx.next_norm)
+    return x
+
   def _call_joined_stream(self, x, ctx: LayerCtx):
     """x fp32 [B, S, D], pre-norm. One kernel per border between sublayers: the branches (weighted, normalised, scaled lane by lane) join the
     stream, and what reads it next comes out of the same pass: a norm, or the stream itself in the compute type for the token input."""
@@ -276,6 +316,7 @@ class DecoderLayer:
     self.index, self.plan = index, plan
     self.unit = f"layer_{index}"
     b = L.Builder(config, self.unit, stack_index, plan.stack, **par)
+    self.entry = b.sub("pass_input").linear("kernel", (2 * config.emb_dim,), (config.emb_dim,), ("concat_embed", "embed")) if plan.pass_input else None
     self.blocks = [DecoderBlock(b, config, bp, rope_tables, layer_index=index, hash_mapping=hash_mapping) for bp in plan.blocks]
     self.params = b.params
 
@@ -320,6 +361,8 @@ class DecoderLayer:
     return torch.cat(outs, 0)
 
   def _call_one(self, x, ctx: LayerCtx):
+    if self.entry is not None:
+      x = self._enter(x, ctx)
     caches = ctx.cache                      # inference: one cache per block of this layer
     for i, blk in enumerate(self.blocks):
       ctx.name_prefix = f"b{i}/" if len(self.blocks) > 1 else ""
@@ -334,6 +377,19 @@ class DecoderLayer:
       from ..multimodal.utils import merge_mm_embeddings
       x = x + merge_mm_embeddings(torch.zeros_like(x), ds[1][self.index], ds[0])
     return x
+
+
+  def reader(self, ctx: LayerCtx):
+    """What reads the residual stream first in this layer."""
+    return F.Beside(ctx.beside) if self.entry is not None else self.blocks[0].reader()
+
+  def _enter(self, x, ctx: LayerCtx):
+    """First layer of a loop: the stream becomes a projection of [stream | embedding output], at the start of every pass."""
+    h = ctx.normed if ctx.normed is not None else torch.cat([x.to(ctx.origin.dtype), ctx.origin], -1)
+    ctx.normed = None
+    if torch.is_grad_enabled():
+      return F.linear(h, self.entry).float()
+    return F.mm(h.reshape(-1, h.shape[-1]), self.entry.data, False, True, out_dtype=torch.float32).view(x.shape)
 
 
 _LANES: dict = {}
@@ -366,7 +422,7 @@ class _StreamNorm:
   """Final norm of a model with an fp32 residual stream: reads fp32, returns the compute dtype."""
 
   def __init__(self, norm):
-    self.norm, self.scale, self.bias, self.eps, self.offset = norm, norm.scale, norm.bias, norm.eps, norm.offset
+    self.norm, self.scale, self.bias, self.eps, self.offset, self.kind = norm, norm.scale, norm.bias, norm.eps, norm.offset, norm.kind
 
   def __call__(self, x):
     return F.stream_norm(x, self.norm, self.scale.data.dtype)
@@ -445,6 +501,8 @@ class Transformer:
     # ---- embedding unit
     eb = L.Builder(c, "embed", None, None, **self.par)
     self.embedding = eb.sub("token_embedder").table("embedding", (c.vocab_size, c.emb_dim), ("vocab", "embed_vocab"))
+    self.embed_norm = L.Norm(eb.sub("decoder"), "embedding_norm", c.emb_dim, c.normalization_layer_epsilon, self.family.norm_offset,
+                             kind=self.family.norm_kind) if self.family.embed_norm else None
     self.pos_embedding = None
     if c.trainable_position_size > 0:
       self.pos_embedding = eb.sub("decoder", "position_embedder").table(
@@ -468,6 +526,8 @@ class Transformer:
         continue
       self.layers.append(DecoderLayer(c, i, si, plan, self.rope_tables, self.par, hash_mapping=self.hash_mapping))
     self.stack_sizes = counters
+    # the layers in running order: a loop runs a stretch of them several times
+    self.runs = list(self.layers) if stage is not None else [self.layers[i] for i in families.layer_runs(c)]
     # ---- multi-token prediction unit (training only; the last stage owns it)
     self.mtp_layers: list[MTPLayer] = []
     self.mtp_params = []
@@ -589,7 +649,10 @@ class Transformer:
   def embed(self, tokens, positions, mm=None):
     """mm: (soft tokens, mask) of one modality, or a list of such pairs (images, audio) merged one after the other."""
     c = self.config
-    x = F.embedding(tokens, self.embedding)
+    if self.embed_norm is not None:
+      x = F.embedding_norm(tokens, self.embedding, self.embed_norm)
+    else:
+      x = F.embedding(tokens, self.embedding)
     if self.family.residual_fp32:
       x = x.float()
     if float(c.embedding_multiplier) != 1.0:
@@ -618,9 +681,8 @@ class Transformer:
 
   def head_logit_scale(self) -> float:
     c = self.config
-    if c.logits_via_embedding and c.normalize_embedding_logits:
-      return 1.0 / math.sqrt(c.emb_dim)
-    return 1.0
+    s = float(c.final_logits_scale)
+    return s / math.sqrt(c.emb_dim) if c.logits_via_embedding and c.normalize_embedding_logits else s
 
   def logits(self, x, normed=None):
     """`normed`: the final norm's output when the last layer already produced it (fp32 residual streams)."""
@@ -655,12 +717,16 @@ class Transformer:
       am = self.encode_audio(audio, audio_mask)
       mm = am if mm is None else [mm, am]
     x = self.embed(tokens, positions, mm)
-    for i, layer in enumerate(self.layers):
-      ctx.layer_index = i
+    if len(self.runs) != len(self.layers) or any(layer.entry is not None for layer in self.layers):
+      D = x.shape[-1]
+      ctx.beside = torch.empty(*x.shape[:-1], 2 * D, dtype=self.store.compute_dtype, device=x.device)
+      ctx.beside[..., D:] = x
+      ctx.origin = ctx.beside[..., D:]
+    for i, layer in enumerate(self.runs):
+      ctx.layer_index = layer.index
       ctx.cache = caches[i] if caches is not None else None
       if self.family.residual_fp32 and not torch.is_grad_enabled():
-        nxt = self.layers[i + 1].blocks[0] if i + 1 < len(self.layers) else self.final_norm
-        ctx.next_norm = nxt.reader()
+        ctx.next_norm = self.runs[i + 1].reader(ctx) if i + 1 < len(self.runs) else self.final_norm.reader()
       x = layer(x, ctx)
     normed = ctx.normed
     if logit_rows is None:

@@ -3,8 +3,9 @@
 `serve` is the whole attention part of a layer with sizes of its own (`layers.blocks.HeadSizes`): one kernel adds biases, normalises, rotates,
 fills the cache and lays the operands out for what follows; prompts run the flash kernel (head widths padded to the next variant), one new
 token per sequence runs the split decode kernel, and everything else (fp32, unusual widths) a plain kernel that reads the cache. Sinks,
-soft caps, windows, chunks, a query temperature, a second map per head (differential attention) and a sigmoid output gate are parameters. `attend` is the same for layers that prepare q, k and v themselves
-(`inference.kvcache.LayerKVCache.attend`).
+soft caps, windows, chunks, a query temperature, a second map per head (differential attention) and a sigmoid output gate are parameters. Where
+the heads mix their scores (`layer.talk`) the first kernel folds the mixing into the queries, which then meet the keys of all key heads side by side
+(`wide`). `attend` is the same for layers that prepare q, k and v themselves (`inference.kvcache.LayerKVCache.attend`).
 """
 from __future__ import annotations
 
@@ -24,9 +25,9 @@ def servable(x, layer, ctx) -> bool:
   from ..inference.kvcache import LayerKVCache
   c = ctx.cache
   return (kernels_ok(x) and type(c) is LayerKVCache and c.quant is None and c.seq_size == 1 and c.k.dtype == x.dtype and ctx.tp_size == 1
-          and ctx.positions3 is None and ctx.bidir is None and layer.vn is None and not layer.share_kv
+          and ctx.positions3 is None and ctx.bidir is None and layer.vn is None and (not layer.share_kv or layer.sizes is not None)
           and not (layer.qk_norm and (layer.l2_qk_norm or layer.qn.scale is None or layer.qn.offset != 0))
-          and not (ctx.segment_ids is not None and (x.dtype != torch.bfloat16 or flash_widths(layer.kw, layer.dv) is None)))
+          and not (ctx.segment_ids is not None and (x.dtype != torch.bfloat16 or not prompt_kernel(layer))))
 
 
 def flash_widths(qk: int, vd: int):
@@ -35,6 +36,17 @@ def flash_widths(qk: int, vd: int):
     if qk <= dq and vd <= dv:
       return dq, dv
   return None
+
+
+def wide_flash_ok(D: int, Dv: int, scale: float) -> bool:
+  return D % 8 == 0 and Dv % 8 == 0 and Dv <= 128 and scale >= 0.0
+
+
+def prompt_kernel(layer) -> bool:
+  """Does a flash kernel hold this layer's heads?"""
+  if layer.talk is not None:
+    return wide_flash_ok(layer.dh, layer.dv, float(layer.query_scalar))
+  return flash_widths(layer.kw, layer.dv) is not None
 
 
 def attends(q, cache, ctx) -> bool:
@@ -96,6 +108,8 @@ def serve(layer, q, k, v, g, ctx):
   norms = (layer.qn.scale.data, layer.kn.scale.data) if layer.qk_norm else (None, None)
   eps = float(layer.config.normalization_layer_epsilon) if layer.l2_qk_norm or layer.qk_norm else -1.0
   temp = layer.q_temp or (0.0, 0.0)
+  if layer.talk is not None:
+    return _serve_mixed(layer, q, k, v, ctx, scale, win, chunk, sinks, rot, eps, bias, norms, temp)
   kw = layer.kw                                          # width of a cached key: the maps' keys side by side
   widths = flash_widths(kw, Dv) if bf and S > 1 else None
   # two maps whose keys are too wide together run the flash kernel one after the other
@@ -129,6 +143,47 @@ def serve(layer, q, k, v, g, ctx):
   return _gate(o.view(N, H * maps, dvp), g, H, Dv, layer)
 
 
+def _serve_mixed(layer, q, k, v, ctx, scale, win, chunk, sinks, rot, eps, bias, norms, temp):
+  """`serve` for heads that mix their scores."""
+  E, cache = backend.ext(), ctx.cache
+  B, S = ctx.positions.shape
+  N, H, G, D, Dv = B * S, layer.hq_l, layer.hkv_l, layer.dh, layer.dv
+  flash = q.dtype == torch.bfloat16 and S > 1 and prompt_kernel(layer)
+  fresh = ctx.mode == "prefill"
+  qp = torch.empty(N, H, G * D, dtype=q.dtype, device=q.device)
+  kp = torch.empty(N, G, D, dtype=q.dtype, device=q.device) if flash and fresh else None
+  copy_v = flash and fresh and (bias[2] is not None or v.stride(0) % 8 != 0 or v.data_ptr() % 16 != 0)
+  vp = torch.empty(N, G, Dv, dtype=q.dtype, device=q.device) if copy_v else None
+  E.qkv_prep(q, k, v, D, Dv, ctx.positions.contiguous(), layer.inv_ts if rot else None, rot, eps, qp, kp, vp, cache.k, cache.v, cache.slot_ids,
+             cache.lengths, cache.new_lens, *bias, *norms, layer.interleaved, 1, *temp, talk=layer.talk.data)
+  if S == 1 and decode_widths_ok(D, Dv, q.dtype) and wide_decode_ok(G, D, Dv):
+    splits = E.cached_decode_splits(B, H, 1, min(x for x in (cache.max_len, win, chunk) if x > 0))
+    part = torch.empty(B, H, splits, Dv, dtype=torch.float32, device=q.device)
+    ml = torch.empty(B, H, splits, 2, dtype=torch.float32, device=q.device)
+    out = torch.empty(B, H * Dv, dtype=q.dtype, device=q.device)
+    E.wide_decode(qp, cache.k, cache.v, cache.slot_ids, cache.lengths, scale, win, chunk, sinks, splits, part, ml, out)
+    return out
+  out = torch.empty(N, H * Dv, dtype=q.dtype, device=q.device)
+  if not flash:
+    E.wide_attention(qp, cache.k, cache.v, cache.slot_ids, cache.lengths, S, scale, win, chunk, sinks, out)
+    return out
+  qw = qp.view(B, S, H, G * D)
+  if fresh:
+    seg = F._i32(ctx.segment_ids)
+    pos = F._i32(ctx.positions) if seg is not None and chunk else None
+    E.wide_flash(qw, kp.view(B, S, G, D), vp.view(B, S, G, Dv) if vp is not None else _rows(v, B, S, G, Dv), out, seg, seg, pos, pos, sinks, scale, win, chunk, 0)
+  else:
+    kc, vc, kv_pos = _cached_rows(cache, S, win)
+    E.wide_flash(qw, kc, vc, out, None, None, F._i32(ctx.positions), F._i32(kv_pos), sinks, scale, win, chunk, 0)
+  return out
+
+
+def wide_decode_ok(G: int, D: int, Dv: int) -> bool:
+  """Do the wide queries of 16 heads and the ring fit in shared memory?"""
+  w = next(x for x in (64, 128, 256) if max(D, Dv) <= x)
+  return (16 * (G * -(-D // 16) * 16 + 8) + 4 * 4 * 16 * (w + 8)) * 2 <= 227 * 1024
+
+
 def _rows(v, B, S, G, Dv):
   """[N, G*Dv] rows of a wider matrix as [B, S, G, Dv] without a copy."""
   return v.as_strided((B, S, G, Dv), (S * v.stride(0), v.stride(0), Dv, 1), v.storage_offset())
@@ -138,18 +193,24 @@ def _flash(q, k, v, positions, segment_ids, scale, cap, win, sinks, mode, kv_pos
   return F.attention_fwd(q, k, v, positions, segment_ids, scale, cap, win, kv_positions=kv_positions, sinks=sinks, cap_mode=mode, chunk=chunk)[0]
 
 
+def _cached_rows(cache, S, win):
+  """What S new tokens per sequence can see of the cache: keys, values and their positions."""
+  dev = cache.lengths.device
+  if win > 0:
+    idx = cache.lengths[:, None] - (win - 1) + torch.arange(win - 1 + S, device=dev)[None]
+  else:
+    idx = torch.arange(int((cache.lengths.max() + S).item()), device=dev)[None].expand(cache.lengths.numel(), -1)
+  kv_pos = torch.where((idx < 0) | (idx >= (cache.lengths + S)[:, None]), torch.full_like(idx, FAR), idx)
+  rows = idx.clamp(0, cache.max_len - 1)
+  slots = cache.slot_ids[:, None].expand_as(rows)
+  return cache.k[slots, rows], cache.v[slots, rows], kv_pos
+
+
 def _portion(q, cache, ctx, scale, cap, win, sinks, mode, D, Dv, chunk=0):
   """Queries that follow cached tokens: the keys they can see are gathered from the cache (padded to the flash widths)."""
   B, S, H, dq = q.shape
   dvp = flash_widths(D, Dv)[1]
-  if win > 0:
-    idx = cache.lengths[:, None] - (win - 1) + torch.arange(win - 1 + S, device=q.device)[None]
-  else:
-    idx = torch.arange(int((cache.lengths.max() + S).item()), device=q.device)[None].expand(B, -1)
-  kv_pos = torch.where((idx < 0) | (idx >= (cache.lengths + S)[:, None]), torch.full_like(idx, FAR), idx)
-  rows = idx.clamp(0, cache.max_len - 1)
-  slots = cache.slot_ids[:, None].expand_as(rows)
-  k, v = cache.k[slots, rows], cache.v[slots, rows]
+  k, v, kv_pos = _cached_rows(cache, S, win)
   k = torch.nn.functional.pad(k, (0, dq - D)) if dq != D else k
   v = torch.nn.functional.pad(v, (0, dvp - Dv)) if dvp != Dv else v
   return _flash(q, k, v, ctx.positions, None, scale, cap, win, sinks, mode, kv_pos, chunk)

@@ -268,7 +268,14 @@ def _stream_kernel_ok(*ts) -> bool:
 
 
 def stream_norm(x: torch.Tensor, norm, dtype) -> torch.Tensor:
-  """RMS norm of an fp32 stream, rounded once to `dtype` (`norm` is a `layers.blocks.Norm`)."""
+  """Norm of an fp32 stream, rounded once to `dtype` (`norm` is a `layers.blocks.Norm`: RMS, or a layer norm without a bias)."""
+  if norm.kind == "layernorm_scale":
+    if _stream_kernel_ok(x) and x.dtype == torch.float32:
+      x2 = x.reshape(-1, x.shape[-1]).contiguous()
+      y = torch.empty(x2.shape, dtype=dtype, device=x.device)
+      backend.ext().residual_gate(x2, None, None, 1, None, None, None, None, norm.scale.data, y, float(norm.eps), True, False)
+      return y.view(x.shape)
+    return ref.layernorm_f32(x, norm.scale.leaf(), norm.eps).to(dtype)
   if _stream_kernel_ok(x) and x.dtype == torch.float32:
     x2 = x.reshape(-1, x.shape[-1]).contiguous()
     y = torch.empty(x2.shape, dtype=dtype, device=x.device)
@@ -338,6 +345,57 @@ def residual_join(x: torch.Tensor, branch, lanes=None, nxt=None):
   return x, (x if nxt is AS_IS else ref.rmsnorm_f32(x, nxt.scale.leaf(), nxt.eps, nxt.offset)).to(dt)
 
 
+class Beside:
+  """`residual_gate(nxt=Beside(buffer))`: the stream as it is goes to the first half of each row of `buffer`, whose second half is set already."""
+
+  def __init__(self, buffer: torch.Tensor):
+    self.buffer = buffer
+
+
+def _norm_f32(x, norm):
+  if norm.kind == "layernorm_scale":
+    return ref.layernorm_f32(x, norm.scale.leaf(), norm.eps)
+  return ref.rmsnorm_f32(x, norm.scale.leaf(), norm.eps, norm.offset)
+
+
+def residual_gate(x: torch.Tensor, branch, gate, bias, post, nxt=None):
+  """(x + post(branch * sigmoid(gate + bias)), nxt(of that) or None) for a sandwich-normed branch whose lanes are gated. `branch`: a tensor or
+  `moe_ops.ExpertRows`; `gate`: logits like the branch or columns of a wider product, `bias` a parameter (both None: no gate); `nxt`: a norm or
+  `Beside`. Norms are RMS or layer norms without a bias. On a GPU one kernel, which updates x in place."""
+  rows, dest, per_token, extra = (branch, None, 1, None) if isinstance(branch, torch.Tensor) else (branch.rows, branch.dest, branch.k, branch.extra)
+  D = x.shape[-1]
+  if _stream_kernel_ok(x, rows) and x.dtype == torch.float32 and x.is_contiguous():
+    x2 = x.view(-1, D)
+    N, dt = x2.shape[0], rows.dtype
+    side = isinstance(nxt, Beside)
+    y = None if nxt is None else nxt.buffer.view(N, -1)[:, :D] if side else torch.empty(N, D, dtype=dt, device=x.device)
+    assert all(n is None or isinstance(n, Beside) or (n.eps == post.eps and n.kind == post.kind and n.offset == 0) for n in (post, nxt))
+    backend.ext().residual_gate(x2, rows.reshape(-1, D).contiguous(), dest, per_token, extra.reshape(N, D).contiguous() if extra is not None else None,
+                                gate.reshape(N, D) if gate is not None and gate.dim() != 2 else gate, bias.data if bias is not None else None, post.scale.data,
+                                nxt.scale.data if nxt is not None and not side else None, y, float(post.eps), post.kind == "layernorm_scale", False)
+    return x, (None if nxt is None else nxt.buffer if side else y.view(x.shape))
+  b = (branch if isinstance(branch, torch.Tensor) else branch.combine(x, torch.float32)).float()
+  if gate is not None:
+    b = b * torch.sigmoid(gate.float().view(b.shape) + bias.leaf().float())
+  x = x.float() + _norm_f32(b, post)
+  if nxt is None:
+    return x, None
+  if isinstance(nxt, Beside):
+    return x, torch.cat([x.to(nxt.buffer.dtype), nxt.buffer[..., D:]], -1)
+  return x, _norm_f32(x, nxt).to(rows.dtype)
+
+
+def embedding_norm(tokens: torch.Tensor, table, norm) -> torch.Tensor:
+  """norm(table[tokens]) as an fp32 stream."""
+  t = table.data
+  if not torch.is_grad_enabled() and backend.use_cuda_kernels(t) and t.dtype in (torch.bfloat16, torch.float32):
+    x = torch.empty(*tokens.shape, t.shape[1], dtype=torch.float32, device=t.device)
+    backend.ext().residual_gate(x.view(-1, t.shape[1]), t, tokens.reshape(-1).to(torch.int32), 1, None, None, None, norm.scale.data, None, None,
+                                float(norm.eps), norm.kind == "layernorm_scale", True)
+    return x
+  return _norm_f32(embedding(tokens, table).float(), norm)
+
+
 def token_gate(g: torch.Tensor, table, tokens: torch.Tensor) -> torch.Tensor:
   """gelu_tanh(g) * table[tokens] for g [B, S, dim]."""
   if not torch.is_grad_enabled() and backend.use_cuda_kernels(g) and g.dtype in (torch.bfloat16, torch.float32) and table.data.dtype == g.dtype:
@@ -395,13 +453,21 @@ def stream_mix(x: torch.Tensor, branch, connection, nxt: StreamReader | None = N
 
 
 # =============================================================================== activation (ungated)
-_PLAIN_ACT_CODE = {"silu": 0, "swish": 0, "gelu": 1, "relu": 2, "gelu_exact": 4}
+_PLAIN_ACT_CODE = {"silu": 0, "swish": 0, "gelu": 1, "relu": 2, "gelu_exact": 4, "relu2": 5, "xielu": 6}
 
 
-def act(h: torch.Tensor, name: str) -> torch.Tensor:
-  """act(h) elementwise, fp32 inside, in h's dtype."""
+def act(h: torch.Tensor, name: str, params=None) -> torch.Tensor:
+  """act(h) elementwise, fp32 inside, in h's dtype. `params`: the two numbers of "xielu". On a GPU h may be columns of a wider matrix."""
   if name == "linear":
     return h
+  if not torch.is_grad_enabled() and name in _PLAIN_ACT_CODE and backend.use_cuda_kernels(h) and h.dtype in (torch.bfloat16, torch.float32) \
+      and (name == "xielu" or not h.is_contiguous()):
+    h2 = h if h.dim() == 2 else h.reshape(-1, h.shape[-1])
+    out = torch.empty(h2.shape, dtype=h.dtype, device=h.device)
+    backend.ext().act_rows(h2 if h2.stride(1) == 1 else h2.contiguous(), out, _PLAIN_ACT_CODE[name], params.data if params is not None else None)
+    return out.view(h.shape)
+  if name == "xielu":
+    return ref.xielu(h.float(), params.leaf().float()).to(h.dtype)
   if not torch.is_grad_enabled() and name in _PLAIN_ACT_CODE and backend.use_cuda_kernels(h) and h.is_contiguous() \
       and h.dtype in (torch.bfloat16, torch.float32):
     out = torch.empty_like(h)

@@ -328,16 +328,19 @@ def router_kernel_ok(logits: torch.Tensor, E: int, k: int) -> bool:
   return backend.use_cuda_kernels(logits) and logits.dtype in (torch.float32, torch.bfloat16) and E <= 512 and k <= 32 and k <= E
 
 
-# =============================================================================== routed layers whose scores scale the expert inputs (inference)
+# =============================================================================== routed layers whose plain scores scale expert inputs or outputs (inference)
 class ExpertRows:
-  """Output rows of the chosen experts: token t sums rows[dest[t * k + c]] over c (dest None: rows[t * k + c])."""
+  """Output rows of the chosen experts: token t sums rows[dest[t * k + c]] over c (dest None: rows[t * k + c]), and row t of `extra` if given."""
 
-  def __init__(self, rows: torch.Tensor, dest, k: int):
-    self.rows, self.dest, self.k = rows, dest, k
+  def __init__(self, rows: torch.Tensor, dest, k: int, extra=None):
+    self.rows, self.dest, self.k, self.extra = rows, dest, k, extra
 
-  def combine(self, like: torch.Tensor) -> torch.Tensor:
+  def combine(self, like: torch.Tensor, dtype=None) -> torch.Tensor:
     r = self.rows if self.dest is None else self.rows[self.dest.long()]
-    return r.view(-1, self.k, r.shape[-1]).float().sum(1).to(like.dtype).view(like.shape)
+    y = r.view(-1, self.k, r.shape[-1]).float().sum(1)
+    if self.extra is not None:
+      y = y + self.extra.reshape(y.shape).float()
+    return y.to(dtype or like.dtype).view(like.shape)
 
 
 def serve_ok(x: torch.Tensor, ctx) -> bool:
@@ -348,24 +351,26 @@ def serve_ok(x: torch.Tensor, ctx) -> bool:
 TENSOR_CORE_FROM = 64       # rows per expert, on average, from which padded groups on the tcgen05 GEMM beat streaming the weights
 
 
-def serve_scaled(x2: torch.Tensor, layer) -> ExpertRows:
-  """x2 [T, D] through a `layers.moe.RoutedMoE` of style "scaled_input". A score s multiplies its expert's input, so by linearity it
-  multiplies both up-projections; it is applied there in fp32, in front of the clamps."""
+def serve_scored(x2: torch.Tensor, layer) -> ExpertRows:
+  """x2 [T, D] through a `layers.moe.RoutedMoE` of style "scaled_input" or "prob_weighted". A score that multiplies its expert's input multiplies
+  both up-projections, by linearity; it is applied there in fp32, in front of the clamps. A score that weights its expert's output multiplies
+  the activation, in fp32."""
   E_ = backend.ext()
   T, D = x2.shape
   k, E, Fdim = layer.k, layer.E, layer.wi_0.data.shape[1]
   n = T * k
   dev, dt = x2.device, x2.dtype
   logits = F.mm(x2, layer.gate.data, False, True, out_dtype=torch.float32)
-  idx, wts, _, _ = E_.router_topk(logits, None, k, 1, True, True, 1.0)
+  idx, wts, _, _ = E_.router_topk(logits, None, k, 1, layer.style == "scaled_input", True, 1.0)
   plan = GroupPlan(idx, E)
-  w0, w1, wo = layer.wi_0.data, layer.wi_1.data, layer.wo.data
+  w0, w1, wo = layer.wi_0.data, layer.wi_1.data if layer.wi_1 is not None else None, layer.wo.data
   if dt == torch.bfloat16 and n >= TENSOR_CORE_FROM * E and D % 128 == 0 and Fdim % 128 == 0:
     rows = torch.empty(plan.rows_max, D, dtype=dt, device=dev)
     E_.moe_gather(x2, plan.row_pair, plan.offs, k, rows)
-    gu = torch.empty(plan.rows_max, 2 * Fdim, dtype=dt, device=dev)
-    E_.grouped_gemm(1, rows, w0, gu[:, :Fdim], plan.offs, plan.blk_expert, False)
-    E_.grouped_gemm(1, rows, w1, gu[:, Fdim:], plan.offs, plan.blk_expert, False)
+    ups = [w for w in (w0, w1) if w is not None]
+    gu = torch.empty(plan.rows_max, len(ups) * Fdim, dtype=dt, device=dev)
+    for j, w in enumerate(ups):
+      E_.grouped_gemm(1, rows, w, gu[:, j * Fdim:(j + 1) * Fdim], plan.offs, plan.blk_expert, False)
     h = torch.empty(plan.rows_max, Fdim, dtype=dt, device=dev)
     E_.expert_act(gu, wts.view(-1), plan.row_pair, plan.offs, float(layer.limit), h)
     E_.grouped_gemm(1, h, wo, rows, plan.offs, plan.blk_expert, False)

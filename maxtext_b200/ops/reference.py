@@ -31,6 +31,13 @@ def rmsnorm_f32(x: torch.Tensor, scale: torch.Tensor | None, eps: float, offset:
   return y if scale is None else y * (scale.float() + offset)
 
 
+def layernorm_f32(x: torch.Tensor, scale: torch.Tensor, eps: float) -> torch.Tensor:
+  """Layer norm without a bias, everything in fp32; fp32 result."""
+  xf = x.float()
+  c = xf - xf.mean(-1, keepdim=True)
+  return c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * scale.float()
+
+
 def rmsnorm_bwd(dy, x, scale, eps, offset=0.0):
   xf, dyf = x.float(), dy.float()
   rstd = torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
@@ -146,8 +153,15 @@ def apply_mrope(x: torch.Tensor, positions3: torch.Tensor, inv_ts: torch.Tensor,
 # ----------------------------------------------------------------------------- activations
 _ACTS = {
     "silu": F.silu, "swish": F.silu, "gelu": lambda t: F.gelu(t, approximate="tanh"), "gelu_exact": F.gelu,
-    "relu": F.relu, "linear": lambda t: t, "sigmoid": torch.sigmoid, "tanh": torch.tanh,
+    "relu": F.relu, "relu2": lambda t: F.relu(t).square(), "linear": lambda t: t, "sigmoid": torch.sigmoid, "tanh": torch.tanh,
 }
+
+
+def xielu(z: torch.Tensor, params: torch.Tensor) -> torch.Tensor:
+  """a z^2 + z / 2 for positive z, b (e^z - 1 - z) + z / 2 for the others, a = softplus(p), b = 1/2 + softplus(q), params = (p, q)."""
+  a, b = F.softplus(params[0]), 0.5 + F.softplus(params[1])
+  neg = z.clamp(max=0.0)
+  return torch.where(z > 0, a * z * z, b * (torch.expm1(neg) - neg)) + 0.5 * z
 
 
 def act_fn(name: str):

@@ -64,8 +64,11 @@ def training_tflops_per_device(c, batch_per_device: float | None = None) -> tupl
     # walk the layer plans: every block contributes its own projections, feed-forward kind and attention pattern, so families with
     # mixed layers (local / global, chunked, dense / routed, gated-delta) are counted layer by layer
     weight, attention = 2 * bs * d * c.vocab_size, 0.0
-    for plan in families.layer_plans(c):
-      for bp in plan.blocks:
+    plans = families.layer_plans(c)
+    for i in families.layer_runs(c):
+      if plans[i].pass_input:
+        weight += 4 * bs * d * d
+      for bp in plans[i].blocks:
         w_, a_ = _block(c, bp, B, S, n_act)
         weight += w_
         attention += a_
@@ -85,7 +88,8 @@ def _sized_mixer(bp, B, S, d):
   H, dv = m["heads"], m["vdim"]
   if bp.attention == "gqa":
     maps = 2 if "diff" in m else 1
-    w = d * (H * maps * m["dim"] + m["kv_heads"] * (maps * m["dim"] + dv) + H * dv + (H if bp.gate == "head" else H * dv))
+    gate = (H if bp.gate == "head" else H * dv) if bp.gated_attn else 0
+    w = d * (H * maps * m["dim"] + m["kv_heads"] * (maps * m["dim"] + (0 if bp.share_kv else dv)) + H * dv + gate)
     size = int(m["mask"]["size"]) if bp.mask else 0
     if bp.mask == "window":
       pairs = S * min(size, S) - 0.5 * min(size, S) ** 2
@@ -94,7 +98,7 @@ def _sized_mixer(bp, B, S, d):
       pairs = (n * size ** 2 + rem ** 2) / 2
     else:
       pairs = S * S / 2
-    return 2 * bs * w, 2 * B * pairs * H * maps * (m["dim"] + dv)
+    return 2 * bs * w, 2 * B * pairs * (H * maps * (m["dim"] + dv) + (H * H if bp.talk else 0))
   if bp.attention == "retention":
     return 2 * bs * d * (2 * H * m["dim"] + 3 * H * dv), bs * H * m["dim"] * dv * 5
   if bp.attention == "channel_delta":
@@ -149,6 +153,8 @@ def _block(c, bp, B, S, n_act):
   elif bp.moe is not None:
     r = bp.moe["router"]
     ffn = 2 * bs * d * r["experts"] + _ffn(bs, d, bp.moe["expert"]["ff"], n_act) * r["top"]
+    if bp.moe.get("shared") is not None:
+      ffn += _ffn(bs, d, bp.moe["shared"]["ff"], n_act)
   elif bp.mlp in ("moe", "moe_shared", "gemma4_moe"):
     ffn = 2 * bs * d * c.num_experts + _ffn(bs, d, c.moe_mlp_dim, n_act) * c.num_experts_per_tok
     if bp.mlp == "moe_shared" and c.shared_experts > 0:
@@ -157,6 +163,8 @@ def _block(c, bp, B, S, n_act):
       ffn += _ffn(bs, d, c.mlp_dim, n_act)                                         # the dense MLP next to the routed experts
   else:
     ffn = _ffn(bs, d, int(bp.mlp_hidden or c.mlp_dim), n_act)
+  if bp.residual_gate:
+    ffn += 2 * bs * d * d * (1 if bp.mlp == "none" else 2)
   if bp.token_side:
     ffn += 4 * bs * d * bp.token_side
   return proj_w + ffn, attn
