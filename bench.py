@@ -239,7 +239,7 @@ def main():
   ap.add_argument("--no-precheck", action="store_true", help="skip the untimed fused-vs-NCCL equivalence check that multi-GPU runs do first")
   ap.add_argument("--comm", default="fused", choices=["fused", "nccl"],
                   help="FSDP collectives: this repository's NVLink kernels fused with the GEMMs (default) or plain NCCL (comparison arm)")
-  ap.add_argument("--serving", action="store_true", help="instead of the training step: prefill and decode throughput of silinex-1b, tipidra-1b, sitivik-1b and "
+  ap.add_argument("--serving", action="store_true", help="instead of the training step: prefill and decode throughput of silinex-1b, tipidra-1b, sitivik-1b, gukirax-1b and "
                   "plain models of equal size, one JSON line per model (maxtext_b200/benchmarks/serving_bench.py; one GPU)")
   ap.add_argument("--serving-models", default="")
   ap.add_argument("--serving-lengths", default="512,2048,8192")

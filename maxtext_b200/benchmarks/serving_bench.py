@@ -6,7 +6,7 @@
   decode:  tokens/s of a full decode state per slot count, every slot holding `context` tokens, CUDA-graph replay
   kernels: device microseconds per launch by kernel (PyTorch profiler, a separate untimed pass), one prompt and one decode step
 
-and one last line `rooflines`: every serving kernel at the layer sizes of silinex-1b, tipidra-1b and sitivik-1b (8192 prompt tokens; 128 sequences with 2048 cached tokens),
+and one last line `rooflines`: every serving kernel at the layer sizes of silinex-1b, tipidra-1b, sitivik-1b and gukirax-1b (8192 prompt tokens; 128 sequences with 2048 cached tokens),
 its time by CUDA events with L2 flushed, its algorithmic bytes or products, and the fraction of the measured copy bandwidth or GEMM rate,
 beside the like operation of the models that existed before (`like`).
 
@@ -21,6 +21,8 @@ Weights are random; the work does not depend on their values. The models:
   tipidra-5b, moe-5b   the same two at width 4096, 32 heads, 24 layers
   sitivik-1b   the catalog entry: windowed attention beside retention, chunked attention beside the channel-wise gated delta rule, differential attention
   sitivik-5b   the same at width 4096, 32 heads, 24 layers
+  gukirax-1b   the catalog entry: heads that mix their scores, gated branches, dense and routed feed-forwards, 12 layers of which four run twice
+  gukirax-5b   the same at width 4096, 32 heads, 18 layers of which six run twice
 """
 from __future__ import annotations
 
@@ -84,6 +86,16 @@ def _sitivik(width, heads, ff, layers):
               layer_specs=[{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)])
 
 
+def _gukirax(width, heads, ff, expert_ff, layers, loop):
+  """Heads that mix their scores in every layer; the first and the last feed-forward dense, the others routed beside a shared expert."""
+  a = {"heads": heads, "kv_heads": 4, "dim": 128, "vdim": 128, "rot": {"base": 500000.0, "dims": 64}, "scale": 128 ** -0.5}
+  routed = {"kind": "moe", "router": {"experts": 16, "top": 2}, "expert": {"ff": expert_ff}, "shared": {"ff": expert_ff}}
+  mlps = [{"kind": "dense", "ff": ff} if i in (0, layers - 1) else routed for i in range(layers)]
+  return dict(decoder_block="gukirax", base_emb_dim=width, base_num_decoder_layers=layers, layer_loop=dict(zip(("start", "stop", "times"), loop)),
+              layer_specs=[{"type": "attention", "mixer": a, "mlp": m} for m in mlps], mlp_activations=["xielu"], final_logits_scale=1.0,
+              final_logits_soft_cap=30.0, vocab_size=65536, logits_via_embedding=True, normalize_embedding_logits=False)
+
+
 MODELS = {
     "silinex-1b": dict(model_name="silinex-1b"),
     "mla-1b": _plain(2048, 16, 8192, 18, 768),
@@ -96,6 +108,8 @@ MODELS = {
     "moe-5b": _moe(4096, 32, 5120, 24),
     "sitivik-1b": dict(model_name="sitivik-1b"),
     "sitivik-5b": _sitivik(4096, 32, 9216, 24),
+    "gukirax-1b": dict(model_name="gukirax-1b"),
+    "gukirax-5b": _gukirax(4096, 32, 12288, 4096, 18, (6, 12, 2)),
 }
 
 
@@ -287,11 +301,11 @@ def rooflines(iters: int = 10) -> dict:
   from ..ops import moe_ops
   nE, top, Fe = 16, 2, 2048
   P = lambda *s: type("P", (), {"data": t(*s)})()  # noqa: E731
-  lay = type("L", (), dict(k=top, E=nE, limit=7.0, gate=P(nE, D), wi_0=P(nE, Fe, D), wi_1=P(nE, Fe, D), wo=P(nE, D, Fe)))()
+  lay = type("L", (), dict(style="scaled_input", k=top, E=nE, limit=7.0, gate=P(nE, D), wi_0=P(nE, Fe, D), wi_1=P(nE, Fe, D), wo=P(nE, D, Fe)))()
   xin = t(N, D)
   idx, wts, _, _ = E.router_topk(F.mm(xin, lay.gate.data, False, True, out_dtype=torch.float32), None, top, 1, True, True, 1.0)
   with torch.no_grad():
-    add("experts, scaled inputs (whole layer)", lambda: moe_ops.serve_scaled(xin, lay), 0, 6 * N * top * D * Fe, like="experts, silu (whole layer)")
+    add("experts, scaled inputs (whole layer)", lambda: moe_ops.serve_scored(xin, lay), 0, 6 * N * top * D * Fe, like="experts, silu (whole layer)")
     add("experts, silu (whole layer)", lambda: moe_ops.moe_ffn_padded(xin, wts, idx, lay.wi_0, lay.wi_1, lay.wo, nE, "silu"), 0, 6 * N * top * D * Fe)
   plan = moe_ops.GroupPlan(idx, nE)
   gu, he = t(plan.rows_max, 2 * Fe), t(plan.rows_max, Fe)
@@ -334,6 +348,34 @@ def rooflines(iters: int = 10) -> dict:
       N * H * (2 * 4 * 128 + 4 * 128 + 2), like="delta_chunks (both kernels)")
   add("ssm_conv, no bias", lambda: E.ssm_conv(craw[:, :ccd], ccw, None, N, cconv, one, one, None, cmix), 4 * N * ccd, like="delta_conv")
   add("gated_head_norm, sigmoid", lambda: E.gated_head_norm(ro, go_, H, 128, 1, 0, 128, nw, 1e-6, o, True), 6 * N * H * 128, like="gated_head_norm")
+  # heads that mix their scores, gated sandwich-normed branches, xIELU, ungated experts
+  talk, pk2 = t(HQ, HQ) * 0.2, t(N, (HQ + HG) * hd + D)
+  tq, tk, tg = torch.split(pk2, [HQ * hd, HG * hd, D], -1)
+  qf, ow = t(N, HQ, HG * hd), t(N, HQ * hd)
+  add("qkv_prep, mixing folded into the queries", lambda: E.qkv_prep(tq, tk, tk, hd, hd, pos0, inv64, 64, 1e-5, qf, ko, None, ck, cv, one, one, None, talk=talk),
+      2 * N * hd * (HQ + HQ * HG + 4 * HG), like="qkv_prep")
+  vr = tk.as_strided((1, N, HG, hd), (N * tk.stride(0), tk.stride(0), hd, 1), tk.storage_offset())
+  qf4 = qf[None] * 0.1
+  sinkh = t(HQ)
+  add("wide_flash (mixed scores, sink)", lambda: E.wide_flash(qf4, ko[None], vr, ow, None, None, None, None, sinkh, 0.09, 0, 0, 0), 0, N * N * HQ * (2 * hd + HQ),
+      like="flash forward, causal, 128")
+  rows["wide_flash (mixed scores, sink)"]["products_issued"] = int(N * N * HQ * (HG * hd + hd))
+  bd = t(D)
+  add("residual_gate", lambda: E.residual_gate(x32, b, None, 1, None, tg, bd, w, w, y, 1e-6, True, False), N * D * (8 + 3 * 2), like="residual_norm")
+  er, edest = t(2 * N + 2048, D), torch.randperm(2 * N + 2048, device=dev)[:2 * N].int()
+  add("residual_gate, rows of two experts and a shared one", lambda: E.residual_gate(x32, er, edest, 2, b, tg, bd, w, w, y, 1e-6, True, False),
+      N * D * (8 + 5 * 2), like="residual_norm")
+  hx, ha, par = t(N, 6144 + D), t(N, 6144), t(2)
+  add("act xielu", lambda: E.act_rows(hx[:, :6144], ha, 6, par), 4 * N * 6144, like="gated_act")
+  add("act relu2", lambda: E.act_rows(hx[:, :2048], ha.view(-1)[: N * 2048].view(N, 2048), 5, None), 4 * N * 2048, like="gated_act")
+  glay = type("L", (), dict(style="prob_weighted", k=top, E=nE, limit=0.0, gate=lay.gate, wi_0=lay.wi_0, wi_1=None, wo=lay.wo))()
+  with torch.no_grad():
+    add("experts, squared relu (whole layer)", lambda: moe_ops.serve_scored(xin, glay), 0, 4 * N * top * D * Fe, like="experts, silu (whole layer)")
+  add("expert_act, squared relu", lambda: E.expert_act(he, wts.view(-1), plan.row_pair, plan.offs, 0.0, gu.view(-1)[: he.numel()].view(he.shape)), 4 * N * top * Fe,
+      like="expert_act")
+  cat, wl, xl = t(N, 2 * D), t(D, 2 * D), t(N, D, dtype=torch.float32)
+  add("gemm, input of a pass (fp32 result)", lambda: F.mm(cat, wl, False, True, out=xl), 0, 4 * N * D * D, like="gemm, 8192 rows")
+  add("gemm, 8192 rows", lambda: F.mm(cat, wl, False, True, out=y), 0, 4 * N * D * D)
   # ---- decoding: 128 sequences, 2048 cached tokens
   B, L = 128, 2048
   ids, lens = torch.arange(B, device=dev), longs(B, L - 1)
@@ -367,7 +409,7 @@ def rooflines(iters: int = 10) -> dict:
     add(f"expert_down, {Bd} tokens", lambda: E.expert_down(hd_, lay.wo.data, idx.view(-1), plan.sizes, plan.offs, plan.row_pair, yd), 2 * hit * Fe * D,
         like=f"experts, silu (whole layer), {Bd} tokens")
     with torch.no_grad():
-      add(f"experts, scaled inputs (whole layer), {Bd} tokens", lambda: moe_ops.serve_scaled(xd, lay), 2 * hit * 3 * Fe * D,
+      add(f"experts, scaled inputs (whole layer), {Bd} tokens", lambda: moe_ops.serve_scored(xd, lay), 2 * hit * 3 * Fe * D,
           like=f"experts, silu (whole layer), {Bd} tokens")
       add(f"experts, silu (whole layer), {Bd} tokens", lambda: moe_ops.moe_ffn_padded(xd, wts, idx, lay.wi_0, lay.wi_1, lay.wo, nE, "silu"), 2 * hit * 3 * Fe * D)
   brec, bhist = t(B, 1, C, NS, dtype=torch.float32), t(B, 3, C, dtype=torch.float32)
@@ -388,6 +430,24 @@ def rooflines(iters: int = 10) -> dict:
     add(f"cached_decode, two maps, {Bd} sequences", lambda: E.cached_decode(q32[:Bd], kc4[:Bd], vc4[:Bd], ids[:Bd], lens[:Bd], 0.12, 0.0, 0, None, ghd[:Bd], sp, pt, ml2,
                                                                            od, per_head=True, lam=lam, diff=0.4, eps=1e-6), 2 * 2 * Bd * L * HG * hd,
         like=f"cached_decode, {Bd} sequences")
+  qw, sinkw = t(B, HQ, HG * hd) * 0.1, t(HQ)
+  for Bd in (1, 32, 128):
+    sp = E.cached_decode_splits(Bd, HQ, 1, L)
+    pt, ml2, od = t(Bd, HQ, sp, hd, dtype=torch.float32), t(Bd, HQ, sp, 2, dtype=torch.float32), t(Bd, HQ * hd)
+    add(f"wide_decode, {Bd} sequences", lambda: E.wide_decode(qw[:Bd], kc4[:Bd], vc4[:Bd], ids[:Bd], lens[:Bd], 0.09, 0, 0, sinkw, sp, pt, ml2, od),
+        2 * 2 * Bd * L * HG * hd, like=f"cached_decode, {Bd} sequences")
+  add("qkv_prep, mixing folded, 128 tokens", lambda: E.qkv_prep(tq[:B], tk[:B], tk[:B], hd, hd, lens, inv64, 64, 1e-5, qw, None, None, kc4, vc4, ids, lens, None,
+                                                                talk=talk), 2 * B * hd * (HQ + HQ * HG + 3 * HG), like="rmsnorm, 128 tokens")
+  add("residual_gate, 128 tokens", lambda: E.residual_gate(x32[:B], b[:B], None, 1, None, tg[:B], bd, w, w, y[:B], 1e-6, True, False), B * D * 14,
+      like="rmsnorm, 128 tokens")
+  add("act xielu, 128 tokens", lambda: E.act_rows(hx[:B, :6144], ha[:B], 6, par), 4 * B * 6144, like="rmsnorm, 128 tokens")
+  for Bd in (1, 128):
+    xd = xin[:Bd].contiguous()
+    with torch.no_grad():
+      gidx = E.router_topk(F.mm(xd, lay.gate.data, False, True, out_dtype=torch.float32), None, top, 1, False, True, 1.0)[0]
+      hit = int((moe_ops.GroupPlan(gidx, nE).sizes > 0).sum())
+      add(f"experts, squared relu (whole layer), {Bd} tokens", lambda: moe_ops.serve_scored(xd, glay), 2 * hit * 2 * Fe * D,
+          like=f"experts, silu (whole layer), {Bd} tokens")
   brr = t(B, H, gk, dv, dtype=torch.float32)
   add("retention_decode", lambda: E.retention_decode(rx[:B], ld, rinv, gk, 1e-6, H, gk, dv, brr, ids, lens, dout), 8 * B * H * gk * dv, like="gla_decode")
   bcr, bcc = t(B, H, 128, 128, dtype=torch.float32), t(B, 3, ccd, dtype=torch.float32)

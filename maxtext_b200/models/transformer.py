@@ -717,7 +717,7 @@ class Transformer:
       am = self.encode_audio(audio, audio_mask)
       mm = am if mm is None else [mm, am]
     x = self.embed(tokens, positions, mm)
-    if len(self.runs) != len(self.layers) or any(layer.entry is not None for layer in self.layers):
+    if any(layer.entry is not None for layer in self.layers):
       D = x.shape[-1]
       ctx.beside = torch.empty(*x.shape[:-1], 2 * D, dtype=self.store.compute_dtype, device=x.device)
       ctx.beside[..., D:] = x

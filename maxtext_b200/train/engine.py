@@ -75,7 +75,8 @@ class TrainEngine:
     self._units = self._ordered_units()
     from ..models import families as _fam
     # all MoE blocks of the model, also those that live on other pipeline stages (the balance loss is averaged over them)
-    self.n_moe_layers = sum(1 for pl in _fam.layer_plans(c) for b in pl.blocks if b.mlp in ("moe", "moe_shared"))
+    plans = _fam.layer_plans(c)
+    self.n_moe_layers = sum(1 for i in _fam.layer_runs(c) for b in plans[i].blocks if b.mlp in ("moe", "moe_shared"))
     self.all_group = None  # WORLD
 
   # ------------------------------------------------------------------ unit bookkeeping
@@ -196,20 +197,23 @@ class TrainEngine:
       x = sp.local_seq(x, ctx.tp_group)
     self._release(0) if self._units[0] and self._units[0][0].group_size > 1 and not c.logits_via_embedding else None
     ckpts = []
-    for i, layer in enumerate(model.layers):
-      ui = i + 1
+    if any(layer.entry is not None for layer in model.layers):
+      ctx.origin = x.to(store.compute_dtype)
+    for i, layer in enumerate(model.runs):
+      ui = layer.index + 1
       self._wait_gather(ui)
-      self._gather(ui + 1)
+      self._gather(model.runs[i + 1].index + 1 if i + 1 < len(model.runs) else len(model.layers) + 1)
       saved = {}
-      ctx.saved, ctx.recompute, ctx.layer_index, ctx.aux_losses = saved, False, i, []
+      ctx.saved, ctx.recompute, ctx.layer_index, ctx.aux_losses = saved, False, layer.index, []
       with torch.no_grad():
-        y = layer(x, ctx)
+        # kernels of an fp32 stream update it in place; the recompute pass needs the layer's input
+        y = layer(x.clone() if model.family.residual_fp32 else x, ctx)
       aux_val = sum(a for _, a in ctx.aux_losses) if ctx.aux_losses else None
       if aux_val is not None:
         acc["aux"] += aux_val.detach().float()
       ckpts.append((x, saved))
       x = y
-      if not (i == len(model.layers) - 1):
+      if i + 1 < len(model.runs) and model.runs[i + 1] is not layer:
         self._release(ui)
     # ---- head: loss and d(hidden) in one pass
     hi = n_units - 1
@@ -253,19 +257,23 @@ class TrainEngine:
       # the update divides every gradient by the global token weight; the balance loss is a mean over each rank's own rows,
       # and the ranks' gradients are summed, so it is seeded with weight / (layers x data shards)
       aux_scale = self._global_weight(total_w) / self.n_moe_layers / self._data_shards()
-    self._gather(len(model.layers) - 1)  # unit index of layer L-2 is L-1
+    self._gather(model.runs[-2].index + 1 if len(model.runs) > 1 else 0)
     train_towers = mm is not None and not bool(getattr(c, "freeze_vision_encoder_params", True))
     deep_grads: dict = {}
-    for i in reversed(range(len(model.layers))):
-      ui = i + 1
-      layer = model.layers[i]
+    d_origin, met = None, set()
+    for i in reversed(range(len(model.runs))):
+      layer = model.runs[i]
+      ui = layer.index + 1
       self._wait_gather(ui)
-      self._gather(ui - 1)
-      for u in self._units[ui]:
+      self._gather(model.runs[i - 1].index + 1 if i > 0 else 0)
+      for u in self._units[ui] if ui not in met else ():
         store.acquire_full_grad(u)
+      met.add(ui)
       x_in, saved = ckpts.pop()
       x_in = x_in.detach().requires_grad_(True)
-      ctx.saved, ctx.recompute, ctx.layer_index, ctx.aux_losses = saved, True, i, []
+      ctx.saved, ctx.recompute, ctx.layer_index, ctx.aux_losses = saved, True, layer.index, []
+      if layer.entry is not None:
+        ctx.origin = ctx.origin.detach().requires_grad_(True)
       deep_leaf = None
       if train_towers and ctx.deepstack is not None and layer.index < len(ctx.deepstack[1]):
         # a trainable tower also feeds this layer directly (deepstack): differentiate with respect to that feature as well
@@ -282,13 +290,19 @@ class TrainEngine:
             grads.append(aux_scale.to(a.dtype))
       torch.autograd.backward(outs, grads)
       dx = x_in.grad
+      if layer.entry is not None:
+        d_origin = ctx.origin.grad.float() if d_origin is None else d_origin + ctx.origin.grad.float()
       if deep_leaf is not None and deep_leaf.grad is not None:
         deep_grads[layer.index] = deep_leaf.grad
       del y, outs, grads, x_in, saved
       for p in layer.params:
         p.collect_leaf_grad()
+      if layer in model.runs[:i]:
+        continue                                 # an earlier pass adds to the same gradients
       self._finish_unit_grads(ui, accumulate_rs)
       self._release(ui)
+    if d_origin is not None:
+      dx = dx + d_origin.to(dx.dtype)
     # ---- embedding backward
     self._wait_gather(0)
     emb_units = self._units[0]
@@ -711,8 +725,9 @@ class TrainEngine:
     for i in range(len(self._units)):
       self._gather(i, async_op=False)
     x = model.embed(tokens, positions)
-    for i, layer in enumerate(model.layers):
-      ctx.layer_index, ctx.saved, ctx.aux_losses = i, None, []
+    ctx.origin = x.to(self.store.compute_dtype) if any(layer.entry is not None for layer in model.layers) else None
+    for layer in model.runs:
+      ctx.layer_index, ctx.saved, ctx.aux_losses = layer.index, None, []
       x = layer(x, ctx)
     h = model.final_norm(x).reshape(B * S, -1)
     out = torch.empty(B * S, dtype=torch.float32, device=self.device)

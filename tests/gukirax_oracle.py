@@ -53,15 +53,15 @@ def talking_attention(q, k, v, scale, talk, sink):
   """q [T, H, D]; k [T, G, D]; v [T, G, Dv]; talk [H, H]; sink [H]. Causal; before the softmax every head's scores become a weighted sum of
   all heads' scores; exp(sink) joins the denominator only."""
   T, H, G = q.shape[0], q.shape[1], k.shape[1]
-  out = torch.zeros(T, H, v.shape[-1], dtype=q.dtype)
-  for i in range(T):
-    own = torch.stack([(k[:i + 1, h // (H // G)] @ q[i, h]) * scale for h in range(H)])
-    for h in range(H):
-      s = sum(talk[h, g] * own[g] for g in range(H))
-      top = torch.maximum(s.max(), sink[h])
-      p = torch.exp(s - top)
-      out[i, h] = (p @ v[:i + 1, h // (H // G)]) / (p.sum() + torch.exp(sink[h] - top))
-  return out
+  own = [(q[:, h] @ k[:, h // (H // G)].T) * scale for h in range(H)]
+  future = torch.triu(torch.ones(T, T, dtype=torch.bool), 1)
+  out = []
+  for h in range(H):
+    s = sum(talk[h, g] * own[g] for g in range(H)).masked_fill(future, float("-inf"))
+    top = torch.maximum(s.max(-1, keepdim=True).values, sink[h])
+    p = torch.exp(s - top)
+    out.append((p @ v[:, h // (H // G)]) / (p.sum(-1, keepdim=True) + torch.exp(sink[h] - top)))
+  return torch.stack(out, 1)
 
 
 def attention_mixer(h, w, m, eps):
@@ -75,7 +75,7 @@ def attention_mixer(h, w, m, eps):
 MIXERS = {"attention": attention_mixer}
 
 
-def dense_mlp(h, w, m):
+def dense_mlp(h, w, m, margins):
   return xielu(h @ w["up"].T, w["act"][0], w["act"][1]) @ w["down"].T
 
 
@@ -83,11 +83,15 @@ def expert(h, up, down):
   return relu_squared(h @ up.T) @ down.T
 
 
-def moe_mlp(h, w, m):
-  """Softmax scores over all experts; the `top` largest weight what their experts give; one more expert runs for every token."""
+def moe_mlp(h, w, m, margins):
+  """Softmax scores over all experts; the `top` largest weight what their experts give; one more expert runs for every token. `margins` (a list)
+  collects by how much the last chosen logit of every token exceeds the next one."""
   out = torch.zeros_like(h)
   for t in range(h.shape[0]):
     z = w["router"] @ h[t]
+    if margins is not None and m["router"]["top"] < m["router"]["experts"]:
+      ranked = torch.sort(z, descending=True).values
+      margins.append((t, float(ranked[m["router"]["top"] - 1] - ranked[m["router"]["top"]])))
     s = torch.exp(z - z.max())
     s = s / s.sum()
     for e in torch.argsort(s, descending=True)[:m["router"]["top"]].tolist():
@@ -119,7 +123,7 @@ def layer_runs(spec):
   return [(i, False) for i in range(a)] + [(i, i == a) for _ in range(loop["times"]) for i in range(a, b)] + [(i, False) for i in range(b, n)]
 
 
-def forward(weights, spec, tokens, layers_out=None):
+def forward(weights, spec, tokens, layers_out=None, margins=None):
   """tokens: list of ids -> logits [T, vocab]; `layers_out` (a list) collects the residual stream after every layer run."""
   eps = spec["norm"]["eps"]
   x = layer_norm(weights["embed"][torch.tensor(tokens)], weights["embed.norm"], eps)
@@ -135,7 +139,7 @@ def forward(weights, spec, tokens, layers_out=None):
     x = gated_sublayer(x, norm("norm1"), lambda h: MIXERS[lay["type"]](h, mix, lay["mixer"], eps), weights[f"l{i}.rg1"], weights[f"l{i}.rg1.b"], norm("norm1b"))
     if lay["mlp"] is not None:
       mlp = part(weights, f"l{i}.mlp.")
-      x = gated_sublayer(x, norm("norm2"), lambda h: MLPS[lay["mlp"]["kind"]](h, mlp, lay["mlp"]), weights[f"l{i}.rg2"], weights[f"l{i}.rg2.b"], norm("norm2b"))
+      x = gated_sublayer(x, norm("norm2"), lambda h: MLPS[lay["mlp"]["kind"]](h, mlp, lay["mlp"], margins), weights[f"l{i}.rg2"], weights[f"l{i}.rg2.b"], norm("norm2b"))
     if layers_out is not None:
       layers_out.append(x)
   h = layer_norm(x, weights["final.norm"], eps)

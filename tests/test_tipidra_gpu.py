@@ -293,7 +293,7 @@ def test_flash_soft_cap_is_exact(mode, reach):
 # ------------------------------------------------------------------------------------------ experts
 def _layer(E_n, k, D, Fd, limit, dtype, g):
   P = lambda *s: type("P", (), {"data": (torch.randn(*s, generator=g) * s[-1] ** -0.5 * 1.5).to(dtype).cuda()})()  # noqa: E731
-  return type("L", (), dict(k=k, E=E_n, limit=limit, gate=P(E_n, D), wi_0=P(E_n, Fd, D), wi_1=P(E_n, Fd, D), wo=P(E_n, D, Fd)))()
+  return type("L", (), dict(style="scaled_input", k=k, E=E_n, limit=limit, gate=P(E_n, D), wi_0=P(E_n, Fd, D), wi_1=P(E_n, Fd, D), wo=P(E_n, D, Fd)))()
 
 
 @pytest.mark.parametrize("T, E_n, k, D, Fd", [(1, 8, 2, 64, 48), (5, 4, 4, 40, 24), (130, 3, 1, 72, 40), (40, 16, 3, 33, 21), (200, 2, 2, 128, 128), (513, 4, 2, 256, 128),
@@ -306,7 +306,7 @@ def test_experts(T, E_n, k, D, Fd):
     layer = _layer(E_n, k, D, Fd, limit, dtype, g)
     x = torch.randn(T, D, generator=g).to(dtype)
     with torch.no_grad():
-      rows = moe_ops.serve_scaled(x.cuda(), layer)
+      rows = moe_ops.serve_scored(x.cuda(), layer)
       got = rows.combine(torch.empty(T, D, device="cuda"))
     s = torch.sigmoid(x.double() @ layer.gate.data.double().cpu().t())
     top = torch.topk(s, min(k + 1, E_n), dim=-1).values
@@ -331,7 +331,7 @@ def test_every_row_of_an_expert_is_computed():
     layer.gate.data.zero_()
     layer.gate.data[3, 0], layer.gate.data[5, 0] = 0.5, 0.25
     with torch.no_grad():
-      got = moe_ops.serve_scaled(x.cuda(), layer).combine(torch.empty(T, D, device="cuda"))
+      got = moe_ops.serve_scored(x.cuda(), layer).combine(torch.empty(T, D, device="cuda"))
     w0, w1, wo = (p.data.double().cpu() for p in (layer.wi_0, layer.wi_1, layer.wo))
     want = sum(O.clamped_expert(float(torch.sigmoid(torch.tensor(v, dtype=torch.float64))) * x.double(), w0[e], w1[e], wo[e], 1.0) for e, v in ((3, 2.0), (5, 1.0)))
     assert _rows(got, want) < 2.5e-2
