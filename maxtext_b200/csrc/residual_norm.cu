@@ -327,7 +327,10 @@ act_rows_kernel(const T* __restrict__ x, long ldx, T* __restrict__ y, long rows,
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
         const float z = v[e], neg = fminf(z, 0.f);
-        v[e] = (z > 0.f ? a * z * z : b * ((sizeof(T) == 2 && neg < -0.25f ? __expf(neg) - 1.f : expm1f(neg)) - neg)) + 0.5f * z;
+        float t;                                         // e^z - 1 - z of a negative z; for a bf16 result two terms are enough near zero
+        if constexpr (sizeof(T) == 2) t = neg > -0.015625f ? neg * neg * (0.5f + neg * (1.f / 6.f)) : __expf(neg) - 1.f - neg;
+        else t = expm1f(neg) - neg;
+        v[e] = (z > 0.f ? a * z * z : b * t) + 0.5f * z;
       }
     } else {
 #pragma unroll

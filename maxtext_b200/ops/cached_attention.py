@@ -39,7 +39,7 @@ def flash_widths(qk: int, vd: int):
 
 
 def wide_flash_ok(D: int, Dv: int, scale: float) -> bool:
-  return D % 8 == 0 and Dv % 8 == 0 and Dv <= 128 and scale >= 0.0
+  return D % 8 == 0 and Dv % 8 == 0 and Dv <= 128 and scale > 0.0
 
 
 def prompt_kernel(layer) -> bool:
