@@ -10,11 +10,10 @@
 //   warps 2..9  softmax, two threads per query row (64 keys each)
 // The contraction W passes in boxes of 64 lanes with 128-byte swizzle through a ring that keys and values share; each CTA fetches half of the keys (and
 // half of the value columns) of a 128-key tile, the products read both halves. That halves what the long contraction costs in shared memory and in
-// traffic: with the whole tile in each CTA the products wait for their operands. Up to W = 512 the query stays on the SM, its first four boxes in shared
-// memory and the others in tensor memory, so that the ring is deep enough for the traffic; beyond that its boxes pass through the ring next to the
-// keys'. W is several times the head width, so the score products of the next key tile are long enough to cover the softmax of the current one: S is
-// double buffered in tensor memory,
-//   S(0), [S(1), P(0) V], [S(2), P(1) V], ...
+// traffic: with the whole tile in each CTA the products wait for their operands. The query's boxes stay in shared memory when they fit (W <= 512) and
+// pass through the ring next to the keys' otherwise. W is several times the head width, so the score products of the next key tiles are long enough to
+// cover the softmax of the current one: S has three buffers in tensor memory,
+//   S(0), S(1), [S(2), P(0) V], [S(3), P(1) V], ...
 // A row's two threads agree on its maximum through shared memory; by then all scores of the tile are in registers, so P may overwrite S as the TMEM
 // operand. Masks, the lazy rescaling and the bounded waits are those of attention_fwd_sm100.cu. Boxes that reach into a neighbour head's columns meet
 // zero-filled lanes of the other operand (keys), or fill accumulator columns that are not stored (values; their width counts as 128).
@@ -28,7 +27,7 @@ namespace wide {
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float RESCALE_THRESHOLD = 8.f;     // log2 units
 constexpr int QBOX = 128 * 64 * 2, KBOX = 64 * 64 * 2, VBOX = 128 * 64 * 2;      // bytes of a box, per CTA
-constexpr int STAGES_MAX = 12, RESIDENT_MAX = 8, QSMEM = 4;     // boxes of a query on the SM, and those of them in shared memory
+constexpr int STAGES_MAX = 12, RESIDENT_MAX = 8;
 
 struct Params {
   int B, H, G, Dv, W;
@@ -37,14 +36,13 @@ struct Params {
   int n_pairs;           // of 256 queries
   attn::Mask mk;
   float scale;
-  const __nv_bfloat16* q;
   const __nv_bfloat16* sinks;    // [H] or nullptr
   __nv_bfloat16* out;
   int* status;
 };
 
 struct alignas(8) Ctl {
-  uint64_t bars[8 + 2 * STAGES_MAX];
+  uint64_t bars[10 + 2 * STAGES_MAX];
   uint32_t tmem_base;
   int abort_flag;
   int pad[2];
@@ -61,15 +59,14 @@ __device__ __forceinline__ float fmax3(float a, float b, float c) {
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(320, 1)
 wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                   const __grid_constant__ Params p) {
-  constexpr uint32_t TMEM_COLS = 512, COL_S = 0, COL_O = 256, COL_Q = 384;       // S of a tile at (its parity) * 128
+  constexpr uint32_t TMEM_COLS = 512, COL_S = 0, COL_O = 384;        // S of tile i at (i % 3) * 128
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  const int nq = p.resident ? min(p.boxes, QSMEM) : 0;   // query boxes in shared memory
-  const uint32_t sQ = base, sR = base + nq * QBOX;
+  const uint32_t sQ = base, sR = base + (p.resident ? p.boxes * QBOX : 0);
   Ctl* ctl = reinterpret_cast<Ctl*>(smem_raw + (sR - smem_u32(smem_raw)) + p.stages * p.stage_bytes);
   const uint32_t bar0 = smem_u32(&ctl->bars[0]);
-  // leader only: Q_FULL, QT_READY, P_READY, FULL; in both CTAs: S_FULL, PV_DONE, EMPTY
-  enum { Q_FULL = 0, S_FULL0 = 1, P_READY0 = 3, PV_DONE = 5, QT_READY = 6, FULL0 = 8, EMPTY0 = 8 + STAGES_MAX };
+  // leader only: Q_FULL, P_READY, FULL; in both CTAs: S_FULL, PV_DONE, EMPTY
+  enum { Q_FULL = 0, S_FULL0 = 1, P_READY0 = 4, PV_DONE0 = 7, FULL0 = 9, EMPTY0 = 9 + STAGES_MAX };
   auto bar = [&](int i) { return bar0 + 8u * i; };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t rank = cluster_ctarank();               // 0 = leader
@@ -96,9 +93,9 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
   if (threadIdx.x == 0) {
     ctl->abort_flag = 0;
     mbar_init(bar(Q_FULL), 1);
-    mbar_init(bar(PV_DONE), 1);
-    mbar_init(bar(QT_READY), 16);
-    for (int s = 0; s < 2; ++s) {
+    mbar_init(bar(PV_DONE0), 1);
+    mbar_init(bar(PV_DONE0 + 1), 1);
+    for (int s = 0; s < 3; ++s) {
       mbar_init(bar(S_FULL0 + s), 1);
       mbar_init(bar(P_READY0 + s), 16);                  // one arrival per softmax warp of the pair
     }
@@ -141,14 +138,16 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
       int kt = seek(kt_lo);
       bool ok = kt < kt_hi;
       if (ok && p.resident) {
-        if (rank == 0) mbar_arrive_expect_tx(bar(Q_FULL), 2 * nq * QBOX);
+        if (rank == 0) mbar_arrive_expect_tx(bar(Q_FULL), 2 * p.boxes * QBOX);
         const uint32_t qb = mapa_shared(bar(Q_FULL), 0);
-        for (int j = 0; j < nq; ++j) tma_load_3d_pair(sQ + j * QBOX, &map_q, qb, h * p.W + j * 64, q0, b);
+        for (int j = 0; j < p.boxes; ++j) tma_load_3d_pair(sQ + j * QBOX, &map_q, qb, h * p.W + j * 64, q0, b);
       }
       ok = ok && keys(kt);
+      if (ok && seek(kt + 1) < kt_hi) ok = keys(seek(kt + 1));
       while (ok) {
         const int nx = seek(kt + 1);
-        if (nx < kt_hi && !keys(nx)) break;
+        const int ahead = nx < kt_hi ? seek(nx + 1) : kt_hi;
+        if (ahead < kt_hi && !keys(ahead)) break;
         if (!stage(VBOX)) break;
         tma_load_3d_pair(sR + s * p.stage_bytes, &map_v, mapa_shared(bar(FULL0 + s), 0), g * p.Dv + (int)rank * 64, kt * 128, b);
         advance();
@@ -180,22 +179,12 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         if (elected) umma_commit_pair(bar(EMPTY0 + s));
         if (++s == p.stages) { s = 0; ph ^= 1; }
       };
-      auto scores = [&](int i) {                         // S of the i-th tile
-        const uint32_t d = tm + COL_S + (i & 1) * 128;
+      auto scores = [&](int buf) {                       // S of a tile
+        const uint32_t d = tm + COL_S + buf * 128;
         for (int j = 0; j < p.boxes; j += 2) {
           if (!wait(FULL0 + s, ph)) return false;
           const uint64_t dk = dk0 + (uint64_t)((s * p.stage_bytes) >> 4), dq = p.resident ? dq0 + (uint64_t)(j * (QBOX >> 4)) : dk + (2 * KBOX >> 4);
-          if (p.resident && j >= QSMEM) {
-            const uint32_t tq = tm + COL_Q + (j - QSMEM) * 32;
-            if (elected) {
-#pragma unroll
-              for (int k = 0; k < 4; ++k) umma_f16_ts_2cta(d, tq + k * 8, dk + k * KSTEP, idesc_qk, 1);
-              if (j + 1 < p.boxes) {
-#pragma unroll
-                for (int k = 0; k < 4; ++k) umma_f16_ts_2cta(d, tq + 32 + k * 8, dk + (KBOX >> 4) + k * KSTEP, idesc_qk, 1);
-              }
-            }
-          } else if (elected) {
+          if (elected) {
 #pragma unroll
             for (int k = 0; k < 4; ++k) umma_f16_ss_2cta(d, dq + k * KSTEP, dk + k * KSTEP, idesc_qk, (j | k) != 0);
             if (j + 1 < p.boxes) {
@@ -205,23 +194,27 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
           }
           release();
         }
-        if (elected) umma_commit_pair(bar(S_FULL0 + (i & 1)));
+        if (elected) umma_commit_pair(bar(S_FULL0 + buf));
         return true;
       };
       bool ok = n > 0;
-      if (ok && p.resident) ok = wait(Q_FULL, 0) && (p.boxes <= QSMEM || wait(QT_READY, 0));
+      if (ok && p.resident) ok = wait(Q_FULL, 0);
       ok = ok && scores(0);
+      if (ok && n > 1) ok = scores(1);
+      int buf = 0;                                       // of tile i
+      uint32_t par = 0;
       for (int i = 0; i < n && ok; ++i) {
-        if (i + 1 < n && !scores(i + 1)) break;
-        if (!wait(FULL0 + s, ph) || !wait(P_READY0 + (i & 1), (i >> 1) & 1)) break;
+        if (i + 2 < n && !scores(buf == 0 ? 2 : buf - 1)) break;
+        if (!wait(FULL0 + s, ph) || !wait(P_READY0 + buf, par)) break;
         const uint64_t dv = dv0 + (uint64_t)((s * p.stage_bytes) >> 4);
-        const uint32_t tp = tm + COL_S + (i & 1) * 128;
+        const uint32_t tp = tm + COL_S + buf * 128;
         if (elected) {
 #pragma unroll
           for (int k = 0; k < 8; ++k) umma_f16_ts_2cta(tm + COL_O, tp + k * 8, dv + k * VSTEP, idesc_pv, (i | k) != 0);
         }
         release();
-        if (elected) umma_commit_pair(bar(PV_DONE));
+        if (elected) umma_commit_pair(bar(PV_DONE0 + (i & 1)));
+        if (++buf == 3) { buf = 0; par ^= 1; }
       }
     }
   } else {
@@ -237,31 +230,14 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     const uint32_t span = (uint32_t)hi_p - (uint32_t)lo_p;
     const bool none = hi_p < lo_p;
     const float a = p.scale * LOG2E;                     // scores in log2 units
-    if (p.resident && p.boxes > QSMEM) {
-      // the query's later boxes go to tensor memory, two lanes of the contraction per column
-      const __nv_bfloat16* src = p.q + (((long)b * mk.Sq + qg) * p.H + h) * p.W;
-      for (int j = QSMEM + half; j < p.boxes; j += 2) {
-        uint32_t r[32];
-#pragma unroll
-        for (int c = 0; c < 8; ++c) {
-          const int col = j * 64 + c * 8;
-          const uint4 v = row_ok && col < p.W ? *reinterpret_cast<const uint4*>(src + col) : make_uint4(0, 0, 0, 0);
-          r[4 * c] = v.x; r[4 * c + 1] = v.y; r[4 * c + 2] = v.z; r[4 * c + 3] = v.w;
-        }
-        tmem_st_32x32b_x32(tmem + lane_off + COL_Q + (j - QSMEM) * 32, r);
-      }
-      tmem_st_wait();
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive_cluster(mapa_shared(bar(QT_READY), 0));
-    }
     float m = -INFINITY, l = 0.f;                        // reference maximum; this half's part of the row sum
-    int cnt = 0;
+    int cnt = 0, buf = 0;
+    uint32_t phase = 0;                                  // of the buffer of tile cnt
     bool ok = true;
     for (int kt = seek(kt_lo); kt < kt_hi; kt = seek(kt + 1), ++cnt) {
       const int par = cnt & 1, k0 = kt * 128 + half * 64;
       const bool masked = attn::classify(mk, t, attn::k_span(mk, b, kt)) != 1;
-      const uint32_t tS = tmem + lane_off + COL_S + par * 128;
+      const uint32_t tS = tmem + lane_off + COL_S + buf * 128;
       if (arrays || has_seg) {
         if (wt < 128) {
           const int kg = kt * 128 + wt;
@@ -270,7 +246,7 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         }
         named_bar_sync(1, 256);
       }
-      if (ok && !mbar_wait(bar(S_FULL0 + par), (cnt >> 1) & 1, abort_flag, p.status, ST_TIMEOUT_EPILOGUE)) ok = false;
+      if (ok && !mbar_wait(bar(S_FULL0 + buf), phase, abort_flag, p.status, ST_TIMEOUT_EPILOGUE)) ok = false;
       tc_fence_after();
       uint32_t r0[32], r1[32];
       auto mask32 = [&](uint32_t (&r)[32], int c0) {
@@ -312,8 +288,9 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
       if (__any_sync(0xffffffffu, grow)) {
         const float alpha = grow ? fast_exp2(m - tm) : 1.f;
         if (cnt > 0) {
-          // O may only be touched once the previous P V product has retired; each half scales its columns
-          if (ok && !mbar_wait(bar(PV_DONE), (cnt - 1) & 1, abort_flag, p.status, ST_TIMEOUT_EPILOGUE)) ok = false;
+          // O may only be touched once the previous P V product has retired (the scores of this tile follow the one before that); each half scales
+          // its columns
+          if (ok && !mbar_wait(bar(PV_DONE0 + (par ^ 1)), ((cnt - 1) >> 1) & 1, abort_flag, p.status, ST_TIMEOUT_EPILOGUE)) ok = false;
           __syncwarp();
           tc_fence_after();
 #pragma unroll 1
@@ -350,10 +327,11 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive_cluster(mapa_shared(bar(P_READY0 + par), 0));
+      if (lane == 0) mbar_arrive_cluster(mapa_shared(bar(P_READY0 + buf), 0));
+      if (++buf == 3) { buf = 0; phase ^= 1; }
     }
     // ---------------------------------------------------------------- epilogue: each half stores its columns
-    if (ok && cnt > 0 && !mbar_wait(bar(PV_DONE), (cnt - 1) & 1, abort_flag, p.status, ST_TIMEOUT_EPILOGUE)) ok = false;
+    if (ok && cnt > 0 && !mbar_wait(bar(PV_DONE0 + ((cnt - 1) & 1)), ((cnt - 1) >> 1) & 1, abort_flag, p.status, ST_TIMEOUT_EPILOGUE)) ok = false;
     __syncwarp();
     tc_fence_after();
     named_bar_sync(2, 256);                              // the last maxima have been read
@@ -446,7 +424,7 @@ int mt_wide_flash(const void* q, const void* k, const void* v, void* out, const 
   p.boxes = (p.W + 63) / 64;
   p.resident = p.boxes <= RESIDENT_MAX;
   p.stage_bytes = p.resident ? VBOX : 2 * (KBOX + QBOX);
-  const int fixed = 1024 + (int)sizeof(Ctl), held = p.resident ? (p.boxes < QSMEM ? p.boxes : QSMEM) * QBOX : 0;
+  const int fixed = 1024 + (int)sizeof(Ctl), held = p.resident ? p.boxes * QBOX : 0;
   p.stages = (227 * 1024 - fixed - held) / p.stage_bytes;
   if (p.stages > STAGES_MAX) p.stages = STAGES_MAX;
   const int smem = fixed + held + p.stages * p.stage_bytes;
@@ -455,7 +433,6 @@ int mt_wide_flash(const void* q, const void* k, const void* v, void* out, const 
       box_map(&mv, v, B, Skv, (long)G * Dv, ldv, bsv, 128))
     return -3;
   p.n_pairs = (Sq + 255) / 256;
-  p.q = static_cast<const __nv_bfloat16*>(q);
   p.scale = scale; p.sinks = static_cast<const __nv_bfloat16*>(sinks); p.out = static_cast<__nv_bfloat16*>(out); p.status = status;
   mt::attn::Mask& msk = p.mk;
   msk.Sq = Sq; msk.Skv = Skv; msk.n_qt = (Sq + 127) / 128; msk.n_kt = (Skv + 127) / 128;
