@@ -327,7 +327,7 @@ wide_flash_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive_cluster(mapa_shared(bar(P_READY0 + buf), 0));
+      if (lane == 0) mbar_arrive_cluster_tmem(mapa_shared(bar(P_READY0 + buf), 0));
       if (++buf == 3) { buf = 0; phase ^= 1; }
     }
     // ---------------------------------------------------------------- epilogue: each half stores its columns

@@ -269,7 +269,7 @@ def _stream_kernel_ok(*ts) -> bool:
 
 def stream_norm(x: torch.Tensor, norm, dtype) -> torch.Tensor:
   """Norm of an fp32 stream, rounded once to `dtype` (`norm` is a `layers.blocks.Norm`: RMS, or a layer norm without a bias)."""
-  if norm.kind == "layernorm_scale":
+  if getattr(norm, "kind", "rms") == "layernorm_scale":
     if _stream_kernel_ok(x) and x.dtype == torch.float32:
       x2 = x.reshape(-1, x.shape[-1]).contiguous()
       y = torch.empty(x2.shape, dtype=dtype, device=x.device)

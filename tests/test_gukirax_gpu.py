@@ -184,6 +184,22 @@ def test_wide_flash(H, G, D):
   assert E.kernel_status(True) == 0
 
 
+@pytest.mark.parametrize("H, G, D", [(8, 4, 128), (12, 12, 56)])
+def test_wide_flash_over_many_tiles(H, G, D):
+  """Rings and score buffers that go around many times; the last keys of a row outgrow the first, so that its reference maximum moves."""
+  E = _ext()
+  g = torch.Generator().manual_seed(3)
+  bf, S = torch.bfloat16, 1500
+  q, k, v = torch.randn(1, S, H, G * D, generator=g).to(bf), torch.randn(1, S, G, D, generator=g), torch.randn(1, S, G, D, generator=g).to(bf)
+  k = (k * torch.linspace(0.2, 4.0, S)[None, :, None, None]).to(bf)
+  sink = torch.randn(H, generator=g).to(bf)
+  scale = 2.0 / (G * D) ** 0.5
+  out = torch.empty(1, S, H * D, dtype=bf, device="cuda")
+  E.wide_flash(q.cuda(), k.cuda(), v.cuda(), out, None, None, None, None, sink.cuda(), scale, 0, 0, 0)
+  assert _rows(out.view(S, H, D), _attend(q[0].double(), k[0].double(), v[0].double(), S, S, scale, sink.double())) < 2e-2
+  assert E.kernel_status(True) == 0
+
+
 @pytest.mark.parametrize("H, G, D", [(4, 2, 64), (20, 5, 40), (16, 16, 64)])
 def test_wide_flash_segments_and_positions(H, G, D):
   """Several prompts in one row; and portions that follow cached tokens of unequal number."""
